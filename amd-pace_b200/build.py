@@ -13,7 +13,10 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 ROOT = os.path.dirname(HERE)
 CSRC = os.path.join(HERE, "csrc")
 OUT = os.path.join(HERE, "pace_b200", "libpace_b200.so")
-SOURCES = ["kv_pool.cu", "attn_decode.cu", "attn_mma.cu", "attn_api.cu", "linear_skinny.cu"]
+SOURCES = ["kv_pool.cu", "attn_decode.cu", "attn_mma.cu", "attn_api.cu", "linear_skinny.cu",
+           "hybrid_ops.cu", "attn_general.cu", "recurrent.cu"]
+# fp32 exp, log and divide of these files are the accurate ones (they serve 32-bit models)
+PRECISE = {"hybrid_ops.cu", "attn_general.cu", "recurrent.cu"}
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
          "--use_fast_math", "-Xcompiler", "-fPIC", "-I", os.path.join(ROOT, "include"), "-I", CSRC] + \
@@ -36,7 +39,8 @@ def build(force=False, verbose=False):
         o = os.path.join(objdir, os.path.basename(s) + ".o")
         objs.append(o)
         if force or any(_newer(d, o) for d in [s] + headers):
-            cmd = [NVCC] + FLAGS + (["-Xptxas", "-v"] if verbose else []) + ["-c", s, "-o", o]
+            flags = [f for f in FLAGS if f != "--use_fast_math" or os.path.basename(s) not in PRECISE]
+            cmd = [NVCC] + flags + (["-Xptxas", "-v"] if verbose else []) + ["-c", s, "-o", o]
             procs.append((s, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
     failed = False
     for s, pr in procs:

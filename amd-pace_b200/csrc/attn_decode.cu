@@ -681,6 +681,7 @@ uint64_t decode_workspace_bytes(int batch, int n_q_heads, int n_kv_heads, int he
 namespace pace {
 int decode_cuda_cores(const pace_attn_args_t* a, void* stream) {
   if (!a || !a->pool || a->q_len != 1 || a->layer < 0 || a->layer >= a->pool->n_layers) return PACE_ERR_INVALID;
+  if (a->pool->row_format != PACE_ROWS_BF16) return PACE_ERR_UNSUPPORTED;
   if (a->batch > a->pool->max_seqs) return PACE_ERR_INVALID;
   const KVView kv = make_view(a->pool, a->layer, a->seq_ids);
   return run_decode(kv, a->batch, a->n_q_heads, a->q, a->q_stride_b, a->q_stride_h, a->out, a->o_stride_b,

@@ -1739,6 +1739,7 @@ int run_mma(const KVView& kv, const CUtensorMap& tmK, const CUtensorMap& tmV, in
 
 int run_mma_paged(const pace_attn_args_t* a, int causal, cudaStream_t stream) {
   if (!a || !a->pool || a->q_len < 1 || a->layer < 0 || a->layer >= a->pool->n_layers) return PACE_ERR_INVALID;
+  if (a->pool->row_format != PACE_ROWS_BF16) return PACE_ERR_UNSUPPORTED;
   if (a->batch > a->pool->max_seqs) return PACE_ERR_INVALID;
   CUtensorMap tm, tm_sub;
   const int rc = pool_map(a->pool, &tm, &tm_sub);

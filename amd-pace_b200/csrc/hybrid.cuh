@@ -1,0 +1,120 @@
+// Helpers of the hybrid-decoder kernels (norms, general attention, recurrences): activations are bf16 or
+// fp32 (template parameter T), everything else is fp32.
+#pragma once
+
+#include "common.cuh"
+
+namespace pace {
+
+template <typename T> __device__ __forceinline__ float to_f(T v);
+template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+// a value as an activation of type T holds it
+template <typename T> __device__ __forceinline__ float round_to(float v) { return to_f<T>(from_f<T>(v)); }
+
+// N consecutive elements <-> fp32 registers; N is 1 or makes an 8- or 16-byte access the caller has aligned
+template <typename T, int N> struct Vec;
+template <> struct Vec<float, 1> {
+  static __device__ __forceinline__ void load(const float* p, float* o) { o[0] = *p; }
+  static __device__ __forceinline__ void store(float* p, const float* v) { *p = v[0]; }
+};
+template <> struct Vec<float, 2> {
+  static __device__ __forceinline__ void load(const float* p, float* o) {
+    const float2 t = *reinterpret_cast<const float2*>(p);
+    o[0] = t.x; o[1] = t.y;
+  }
+  static __device__ __forceinline__ void store(float* p, const float* v) {
+    *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+  }
+};
+template <> struct Vec<float, 4> {
+  static __device__ __forceinline__ void load(const float* p, float* o) {
+    const float4 t = *reinterpret_cast<const float4*>(p);
+    o[0] = t.x; o[1] = t.y; o[2] = t.z; o[3] = t.w;
+  }
+  static __device__ __forceinline__ void store(float* p, const float* v) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  }
+};
+template <> struct Vec<float, 8> {
+  static __device__ __forceinline__ void load(const float* p, float* o) {
+    Vec<float, 4>::load(p, o);
+    Vec<float, 4>::load(p + 4, o + 4);
+  }
+  static __device__ __forceinline__ void store(float* p, const float* v) {
+    Vec<float, 4>::store(p, v);
+    Vec<float, 4>::store(p + 4, v + 4);
+  }
+};
+template <> struct Vec<__nv_bfloat16, 1> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float* o) { o[0] = __bfloat162float(*p); }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float* v) { *p = __float2bfloat16_rn(v[0]); }
+};
+template <> struct Vec<__nv_bfloat16, 4> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float* o) {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    const float2 a = bf2_to_f2(t.x), b = bf2_to_f2(t.y);
+    o[0] = a.x; o[1] = a.y; o[2] = b.x; o[3] = b.y;
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float* v) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(f2_to_bf2(v[0], v[1]), f2_to_bf2(v[2], v[3]));
+  }
+};
+template <> struct Vec<__nv_bfloat16, 8> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float* o) {
+    const uint4 t = *reinterpret_cast<const uint4*>(p);
+    const float2 a = bf2_to_f2(t.x), b = bf2_to_f2(t.y), c = bf2_to_f2(t.z), d = bf2_to_f2(t.w);
+    o[0] = a.x; o[1] = a.y; o[2] = b.x; o[3] = b.y; o[4] = c.x; o[5] = c.y; o[6] = d.x; o[7] = d.y;
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float* v) {
+    *reinterpret_cast<uint4*>(p) =
+        make_uint4(f2_to_bf2(v[0], v[1]), f2_to_bf2(v[2], v[3]), f2_to_bf2(v[4], v[5]), f2_to_bf2(v[6], v[7]));
+  }
+};
+
+// fp32 with a few ulp of error.  T names the activation type of the caller: fp32 models take the library's
+// exp and divide, bf16 models the hardware's approximate ones (relative error about 1e-6).
+template <typename T> __device__ __forceinline__ float exp_t(float x) { return __expf(x); }
+template <> __device__ __forceinline__ float exp_t<float>(float x) { return expf(x); }
+template <typename T> __device__ __forceinline__ float div_t(float a, float b) { return __fdividef(a, b); }
+template <> __device__ __forceinline__ float div_t<float>(float a, float b) { return a / b; }
+// sigmoid(x) = 1 / (1 + e^-x); the exponent is clamped so that the approximate divide never sees infinity
+template <typename T> __device__ __forceinline__ float sigmoid_t(float x) {
+  return div_t<T>(1.0f, 1.0f + exp_t<T>(fminf(-x, 80.0f)));
+}
+template <typename T> __device__ __forceinline__ float silu_t(float x) { return x * sigmoid_t<T>(x); }
+// 0.5 z (1 + tanh w) = z sigmoid(2 w)
+template <typename T> __device__ __forceinline__ float gelu_tanh_t(float z) {
+  return z * sigmoid_t<T>(1.5957691216057308f * (z + 0.044715f * z * z * z));
+}
+// 1 - e^x for x <= 0 without cancellation: the series of expm1 near zero, the plain difference further out
+template <typename T> __device__ __forceinline__ float one_minus_exp(float x, float exp_x) {
+  const float s = -x * (1.0f + x * (1.0f / 2) * (1.0f + x * (1.0f / 3) * (1.0f + x * (1.0f / 4) *
+                  (1.0f + x * (1.0f / 5) * (1.0f + x * (1.0f / 6) * (1.0f + x * (1.0f / 7)))))));
+  return x > -0.25f ? s : 1.0f - exp_x;
+}
+
+// Sum over the thread block, the same value in every thread; `red` holds one float per warp.
+__device__ __forceinline__ float block_sum(float v, float* red) {
+#pragma unroll
+  for (int o = 16; o; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  const int warps = (blockDim.x + 31) >> 5;
+  if (warps == 1) return v;
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float s = 0.f;
+  for (int w = 0; w < warps; ++w) s += red[w];
+  return s;
+}
+
+inline bool step_ok(const pace_step_t* s) {
+  return s && s->n_tokens >= 0 && s->n_entries >= 0 && s->n_tokens >= s->n_entries &&
+         (s->n_tokens == 0 || (s->token && s->tok_entry && s->tok_pos && s->q_row && s->cu && s->start && s->slot));
+}
+inline bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
+
+}  // namespace pace

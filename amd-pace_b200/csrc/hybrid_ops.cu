@@ -1,0 +1,404 @@
+// Token-wise kernels of hybrid decoders: residual + norms, the append of normalised keys, output gates,
+// squared ReLU.  One thread block per token row where a row has to be summed over; fp32 arithmetic.
+#include "hybrid.cuh"
+
+namespace pace {
+namespace {
+
+// ---------------------------------------------------------------------------
+// x' = x + rms(y) w_post (+ embedding row);  h = rms(x') w_next
+// ---------------------------------------------------------------------------
+template <typename T, int V, int ITEMS>
+__global__ void __launch_bounds__(512) residual_norm_kernel(pace_step_t st, pace_residual_norm_args_t a) {
+  __shared__ float red[32];
+  const int t = blockIdx.x, W = a.width;
+  float xv[ITEMS][V], yv[ITEMS][V];
+  float* x = a.x + (size_t)t * W;
+  const T* y = a.y ? static_cast<const T*>(a.y) + (size_t)t * a.y_stride : nullptr;
+  const T* em = nullptr;
+  if (a.embed) {
+    const int tok = st.token[t];
+    if (tok >= 0 && tok < a.vocab) em = static_cast<const T*>(a.embed) + (size_t)tok * W;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * V;
+    if (c < W) {
+      if (!a.restart) Vec<float, V>::load(x + c, xv[i]);
+      else
+#pragma unroll
+        for (int j = 0; j < V; ++j) xv[i][j] = 0.f;
+      if (y) {
+        Vec<T, V>::load(y + c, yv[i]);
+#pragma unroll
+        for (int j = 0; j < V; ++j) ss += yv[i][j] * yv[i][j];
+      }
+    }
+  }
+  if (y) {
+    float r = 1.f;
+    if (a.w_post) r = 1.0f / sqrtf(block_sum(ss, red) / (float)W + a.eps);
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * V;
+      if (c < W) {
+        float w[V];
+        if (a.w_post) Vec<float, V>::load(a.w_post + c, w);
+#pragma unroll
+        for (int j = 0; j < V; ++j) xv[i][j] += a.w_post ? yv[i][j] * r * (a.weight_offset + w[j]) : yv[i][j];
+      }
+    }
+  }
+  ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * V;
+    if (c < W) {
+      if (em) {
+        float e[V];
+        Vec<T, V>::load(em + c, e);
+#pragma unroll
+        for (int j = 0; j < V; ++j) xv[i][j] += e[j];
+      }
+      Vec<float, V>::store(x + c, xv[i]);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += xv[i][j] * xv[i][j];
+    }
+  }
+  if (!a.w_next) return;
+  const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)W + a.eps);
+  T* h = static_cast<T*>(a.h) + (size_t)t * W;
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * V;
+    if (c < W) {
+      float w[V];
+      Vec<float, V>::load(a.w_next + c, w);
+#pragma unroll
+      for (int j = 0; j < V; ++j) w[j] = xv[i][j] * r * (a.weight_offset + w[j]);
+      Vec<T, V>::store(h + c, w);
+    }
+  }
+}
+
+// Threads for a row of `groups` vectors and how many vectors each of them takes (1, 2, 4, 8 or 16), 0 = too wide.
+int row_items(int groups, int* threads) {
+  int th = (groups + 31) / 32 * 32;
+  if (th > 512) th = 512;
+  *threads = th;
+  const int need = (groups + th - 1) / th;
+  for (int i = 1; i <= 16; i *= 2)
+    if (need <= i) return i;
+  return 0;
+}
+
+template <typename T, int V>
+int launch_residual_norm(const pace_step_t& st, const pace_residual_norm_args_t& a, cudaStream_t s) {
+  int threads = 0;
+  const int items = row_items((a.width + V - 1) / V, &threads);
+  switch (items) {
+    case 1: residual_norm_kernel<T, V, 1><<<st.n_tokens, threads, 0, s>>>(st, a); break;
+    case 2: residual_norm_kernel<T, V, 2><<<st.n_tokens, threads, 0, s>>>(st, a); break;
+    case 4: residual_norm_kernel<T, V, 4><<<st.n_tokens, threads, 0, s>>>(st, a); break;
+    case 8: residual_norm_kernel<T, V, 8><<<st.n_tokens, threads, 0, s>>>(st, a); break;
+    case 16: residual_norm_kernel<T, V, 16><<<st.n_tokens, threads, 0, s>>>(st, a); break;
+    default: return PACE_ERR_UNSUPPORTED;
+  }
+  PACE_LAUNCH_CHECK("residual_norm_kernel");
+  return PACE_OK;
+}
+
+// ---------------------------------------------------------------------------
+// q / k norms over the whole projections, query temperature, rows to the staging buffer and to the pages
+// ---------------------------------------------------------------------------
+struct PageRows {
+  const int32_t* block_table;
+  int32_t* status;
+  char *k, *v;       // this layer's K and V regions
+  int page_tokens, n_kv_heads, max_pages_per_seq, max_seqs, n_pages;
+};
+
+template <typename T, int V>
+__global__ void append_norm_kernel(pace_step_t st, PageRows pg, pace_append_norm_args_t a, int row) {
+  __shared__ float red[32];
+  const int t = blockIdx.x;
+  const int H = a.n_q_heads, G = pg.n_kv_heads, d = a.dim, vd = a.vdim;
+  const int nq = H * d, nk = G * d;
+  const T* src = static_cast<const T*>(a.qkv) + (size_t)t * a.qkv_stride;
+  const T *qs = src, *ks = src + nq, *vs = ks + nk;
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x * V; c < nq + nk; c += blockDim.x * V) {  // (V divides dim: a vector never straddles)
+    float x[V];
+    Vec<T, V>::load(src + c, x);
+    float s = 0.f;
+#pragma unroll
+    for (int j = 0; j < V; ++j) s += x[j] * x[j];
+    if (c < nq) sq += s; else sk += s;
+  }
+  const float rq0 = a.q_norm ? 1.0f / sqrtf(block_sum(sq, red) / (float)nq + a.eps) : 1.f;
+  const float rk = a.k_norm ? 1.0f / sqrtf(block_sum(sk, red) / (float)nk + a.eps) : 1.f;
+  const int pos = st.tok_pos[t];
+  float temp = a.q_mul;
+  if (a.temp_coef != 0.f) temp *= 1.0f + a.temp_coef * logf((float)(floor((double)(pos + 1) / a.temp_every) + 1.0));
+  const int slot = st.slot[st.tok_entry[t]];
+  const int lp = pos / pg.page_tokens;
+  int page = -1;
+  if (slot >= 0 && slot < pg.max_seqs && lp < pg.max_pages_per_seq)
+    page = pg.block_table[(size_t)slot * pg.max_pages_per_seq + lp];
+  if (page < 0 || page >= pg.n_pages) {
+    if (threadIdx.x == 0) raise_status(pg.status, PACE_DEV_BAD_INDEX);
+    page = -1;
+  }
+  const int per_row = row / V;  // vectors of one padded row
+  T* qo = static_cast<T*>(a.q_out) + (size_t)st.q_row[t] * H * row;
+  for (int i = threadIdx.x; i < (H + 2 * G) * per_row; i += blockDim.x) {
+    const int hh = i / per_row, c = (i - hh * per_row) * V;
+    float x[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[j] = 0.f;
+    if (hh < H) {
+      if (c < d) {
+        Vec<T, V>::load(qs + hh * d + c, x);
+        if (a.q_norm) {
+          float w[V];
+          Vec<float, V>::load(a.q_norm + hh * d + c, w);
+#pragma unroll
+          for (int j = 0; j < V; ++j) x[j] *= rq0 * w[j];
+        }
+#pragma unroll
+        for (int j = 0; j < V; ++j) x[j] *= temp;
+      }
+      Vec<T, V>::store(qo + (size_t)hh * row + c, x);
+      continue;
+    }
+    const int g = hh < H + G ? hh - H : hh - H - G;
+    const bool is_v = hh >= H + G;
+    if (is_v) {
+      if (c < vd) Vec<T, V>::load(vs + g * vd + c, x);
+    } else if (c < d) {
+      Vec<T, V>::load(ks + g * d + c, x);
+      if (a.k_norm) {
+        float w[V];
+        Vec<float, V>::load(a.k_norm + g * d + c, w);
+#pragma unroll
+        for (int j = 0; j < V; ++j) x[j] *= rk * w[j];
+      }
+    }
+    if (page >= 0) {
+      const size_t off = (((size_t)page * G + g) * pg.page_tokens + (pos - lp * pg.page_tokens)) * row + c;
+      Vec<T, V>::store(reinterpret_cast<T*>(is_v ? pg.v : pg.k) + off, x);
+    }
+  }
+}
+
+template <typename T>
+int launch_append_norm(const pace_kv_pool_t* p, int layer, const pace_step_t& st, const pace_append_norm_args_t& a,
+                       cudaStream_t s) {
+  const int row = p->head_dim * 2 / (int)sizeof(T);  // elements of a pool row
+  if (a.dim > row || a.vdim > row) return PACE_ERR_INVALID;
+  const size_t region = (size_t)p->n_pages * p->n_kv_heads * p->page_tokens * p->head_dim * 2;  // bytes
+  PageRows pg;
+  pg.block_table = p->block_table;
+  pg.status = p->status;
+  pg.k = static_cast<char*>(p->pages) + (size_t)layer * 2 * region;
+  pg.v = pg.k + region;
+  pg.page_tokens = p->page_tokens;
+  pg.n_kv_heads = p->n_kv_heads;
+  pg.max_pages_per_seq = p->max_pages_per_seq;
+  pg.max_seqs = p->max_seqs;
+  pg.n_pages = p->n_pages;
+  constexpr int V = 16 / sizeof(T);
+  const bool vec = a.dim % V == 0 && a.vdim % V == 0 && row % V == 0 && a.qkv_stride % V == 0 && aligned16(a.qkv) &&
+                   aligned16(a.q_out) && (!a.q_norm || aligned16(a.q_norm)) && (!a.k_norm || aligned16(a.k_norm));
+  const int groups = (a.n_q_heads + 2 * p->n_kv_heads) * row / (vec ? V : 1);
+  const int threads = groups < 512 ? (groups + 31) / 32 * 32 : 512;
+  if (vec)
+    append_norm_kernel<T, V><<<st.n_tokens, threads, 0, s>>>(st, pg, a, row);
+  else
+    append_norm_kernel<T, 1><<<st.n_tokens, threads, 0, s>>>(st, pg, a, row);
+  PACE_LAUNCH_CHECK("append_norm_kernel");
+  note_pool_write(s);
+  return PACE_OK;
+}
+
+// ---------------------------------------------------------------------------
+// gates and activation
+// ---------------------------------------------------------------------------
+template <typename T, int V>
+__global__ void gate_heads_kernel(pace_step_t st, const T* __restrict__ attn, const T* __restrict__ gate, int64_t gs,
+                                  T* __restrict__ out, int H, int vd, int row) {
+  const int n = H * vd, per = n / V;
+  const size_t total = (size_t)st.n_tokens * per;
+  for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const int t = (int)(i / per), c = (int)(i % per) * V;
+    const int h = c / vd;
+    float o[V], g[V];
+    Vec<T, V>::load(attn + ((size_t)st.q_row[t] * H + h) * row + (c - h * vd), o);
+    Vec<T, V>::load(gate + (size_t)t * gs + c, g);
+#pragma unroll
+    for (int j = 0; j < V; ++j) o[j] *= sigmoid_t<T>(g[j]);
+    Vec<T, V>::store(out + (size_t)t * n + c, o);
+  }
+}
+
+template <typename T, int V>
+__global__ void norm_gate_kernel(const T* __restrict__ o, const float* __restrict__ w, const T* __restrict__ gate,
+                                 int64_t gs, T* __restrict__ out, int n, float eps) {
+  __shared__ float red[32];
+  const int t = blockIdx.x;
+  const T* src = o + (size_t)t * n;
+  float ss = 0.f;
+  for (int c = threadIdx.x * V; c < n; c += blockDim.x * V) {
+    float x[V];
+    Vec<T, V>::load(src + c, x);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += x[j] * x[j];
+  }
+  const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
+  for (int c = threadIdx.x * V; c < n; c += blockDim.x * V) {
+    float x[V], g[V], wv[V];
+    Vec<T, V>::load(src + c, x);
+    Vec<T, V>::load(gate + (size_t)t * gs + c, g);
+    Vec<float, V>::load(w + c, wv);
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[j] = x[j] * r * wv[j] * sigmoid_t<T>(g[j]);
+    Vec<T, V>::store(out + (size_t)t * n + c, x);
+  }
+}
+
+template <typename T, int V>
+__global__ void relu_squared_kernel(T* __restrict__ x, int64_t n) {
+  for (int64_t i = (blockIdx.x * (int64_t)blockDim.x + threadIdx.x) * V; i < n; i += (int64_t)gridDim.x * blockDim.x * V) {
+    float v[V];
+    Vec<T, V>::load(x + i, v);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const float p = fmaxf(v[j], 0.f);
+      v[j] = p * p;
+    }
+    Vec<T, V>::store(x + i, v);
+  }
+}
+
+unsigned elementwise_blocks(size_t threads_wanted) {
+  size_t b = (threads_wanted + 255) / 256;
+  return (unsigned)(b < 1 ? 1 : b > 148 * 16 ? 148 * 16 : b);
+}
+
+__global__ void step_decode_kernel(int32_t* token, int32_t* tok_pos, int32_t* start, const int64_t* next, const int64_t* pos,
+                                   int n) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  token[i] = (int32_t)next[i];
+  tok_pos[i] = start[i] = (int32_t)pos[i];
+}
+
+template <typename T>
+int gate_heads_t(const pace_step_t& st, const void* attn, const void* gate, int64_t gs, void* out, int H, int vd, int row,
+                 cudaStream_t s) {
+  constexpr int V = 16 / sizeof(T);
+  const bool vec = vd % V == 0 && row % V == 0 && gs % V == 0 && aligned16(attn) && aligned16(gate) && aligned16(out);
+  const size_t n = (size_t)st.n_tokens * H * vd;
+  if (vec)
+    gate_heads_kernel<T, V><<<elementwise_blocks(n / V), 256, 0, s>>>(st, (const T*)attn, (const T*)gate, gs, (T*)out, H, vd, row);
+  else
+    gate_heads_kernel<T, 1><<<elementwise_blocks(n), 256, 0, s>>>(st, (const T*)attn, (const T*)gate, gs, (T*)out, H, vd, row);
+  PACE_LAUNCH_CHECK("gate_heads_kernel");
+  return PACE_OK;
+}
+
+template <typename T>
+int norm_gate_t(const void* o, const float* w, const void* gate, int64_t gs, void* out, int n_tokens, int n, float eps,
+                cudaStream_t s) {
+  constexpr int V = 16 / sizeof(T);
+  const bool vec = n % V == 0 && gs % V == 0 && aligned16(o) && aligned16(gate) && aligned16(out) && aligned16(w);
+  const int groups = vec ? n / V : n;
+  const int threads = groups < 512 ? (groups + 31) / 32 * 32 : 512;
+  if (vec)
+    norm_gate_kernel<T, V><<<n_tokens, threads, 0, s>>>((const T*)o, w, (const T*)gate, gs, (T*)out, n, eps);
+  else
+    norm_gate_kernel<T, 1><<<n_tokens, threads, 0, s>>>((const T*)o, w, (const T*)gate, gs, (T*)out, n, eps);
+  PACE_LAUNCH_CHECK("norm_gate_kernel");
+  return PACE_OK;
+}
+
+template <typename T>
+int relu_squared_t(void* x, int64_t n, cudaStream_t s) {
+  constexpr int V = 16 / sizeof(T);
+  if (n % V == 0 && aligned16(x))
+    relu_squared_kernel<T, V><<<elementwise_blocks((size_t)n / V), 256, 0, s>>>((T*)x, n);
+  else
+    relu_squared_kernel<T, 1><<<elementwise_blocks((size_t)n), 256, 0, s>>>((T*)x, n);
+  PACE_LAUNCH_CHECK("relu_squared_kernel");
+  return PACE_OK;
+}
+
+bool dtype_ok(int dtype) { return dtype == PACE_DTYPE_BF16 || dtype == PACE_DTYPE_FP32; }
+
+}  // namespace
+}  // namespace pace
+
+using namespace pace;
+
+extern "C" {
+
+int pace_residual_norm(const pace_step_t* st, const pace_residual_norm_args_t* a, void* stream) {
+  if (!step_ok(st) || !a || !a->x || a->width < 1 || !dtype_ok(a->dtype)) return PACE_ERR_INVALID;
+  if ((a->w_next && !a->h) || (a->embed && a->vocab < 1) || (a->y && a->y_stride < a->width)) return PACE_ERR_INVALID;
+  if (st->n_tokens == 0) return PACE_OK;
+  PACE_PROFILE("residual_norm", stream, "tokens=%d width=%d", st->n_tokens, a->width);
+  const cudaStream_t s = (cudaStream_t)stream;
+  // four elements per access: 16 bytes of fp32, 8 of bf16
+  const bool vec = a->width % 4 == 0 && a->y_stride % 4 == 0 && aligned16(a->x) && aligned16(a->y) && aligned16(a->h) &&
+                   aligned16(a->embed) && aligned16(a->w_post) && aligned16(a->w_next);
+  if (a->dtype == PACE_DTYPE_BF16)
+    return vec ? launch_residual_norm<__nv_bfloat16, 4>(*st, *a, s) : launch_residual_norm<__nv_bfloat16, 1>(*st, *a, s);
+  return vec ? launch_residual_norm<float, 4>(*st, *a, s) : launch_residual_norm<float, 1>(*st, *a, s);
+}
+
+int pace_kv_append_norm(const pace_kv_pool_t* p, int32_t layer, const pace_step_t* st, const pace_append_norm_args_t* a,
+                        void* stream) {
+  if (!p || !p->pages || !p->block_table || !step_ok(st) || !a || layer < 0 || layer >= p->n_layers) return PACE_ERR_INVALID;
+  if (!a->qkv || !a->q_out || a->n_q_heads < 1 || a->dim < 1 || a->vdim < 1 || !dtype_ok(a->dtype)) return PACE_ERR_INVALID;
+  if (a->n_q_heads % p->n_kv_heads || (a->temp_coef != 0.f && !(a->temp_every > 0.0))) return PACE_ERR_INVALID;
+  if (p->row_format == PACE_ROWS_BF16 && a->dtype != PACE_DTYPE_BF16) return PACE_ERR_INVALID;
+  if (st->n_tokens == 0) return PACE_OK;
+  PACE_PROFILE("kv_append_norm", stream, "layer=%d tokens=%d", layer, st->n_tokens);
+  return a->dtype == PACE_DTYPE_BF16 ? launch_append_norm<__nv_bfloat16>(p, layer, *st, *a, (cudaStream_t)stream)
+                                     : launch_append_norm<float>(p, layer, *st, *a, (cudaStream_t)stream);
+}
+
+int pace_gate_heads(const pace_step_t* st, const void* attn, const void* gate, int64_t gs, void* out, int32_t H, int32_t vd,
+                    int32_t row, int32_t dtype, void* stream) {
+  if (!step_ok(st) || !attn || !gate || !out || H < 1 || vd < 1 || row < vd || !dtype_ok(dtype)) return PACE_ERR_INVALID;
+  if (st->n_tokens == 0) return PACE_OK;
+  return dtype == PACE_DTYPE_BF16 ? gate_heads_t<__nv_bfloat16>(*st, attn, gate, gs, out, H, vd, row, (cudaStream_t)stream)
+                                  : gate_heads_t<float>(*st, attn, gate, gs, out, H, vd, row, (cudaStream_t)stream);
+}
+
+int pace_norm_gate(const void* o, const float* w, const void* gate, int64_t gs, void* out, int32_t n_tokens, int32_t n,
+                   float eps, int32_t dtype, void* stream) {
+  if (!o || !w || !gate || !out || n_tokens < 0 || n < 1 || !dtype_ok(dtype)) return PACE_ERR_INVALID;
+  if (n_tokens == 0) return PACE_OK;
+  return dtype == PACE_DTYPE_BF16 ? norm_gate_t<__nv_bfloat16>(o, w, gate, gs, out, n_tokens, n, eps, (cudaStream_t)stream)
+                                  : norm_gate_t<float>(o, w, gate, gs, out, n_tokens, n, eps, (cudaStream_t)stream);
+}
+
+int pace_relu_squared(void* x, int64_t n, int32_t dtype, void* stream) {
+  if (!x || n < 0 || !dtype_ok(dtype)) return PACE_ERR_INVALID;
+  if (n == 0) return PACE_OK;
+  return dtype == PACE_DTYPE_BF16 ? relu_squared_t<__nv_bfloat16>(x, n, (cudaStream_t)stream)
+                                  : relu_squared_t<float>(x, n, (cudaStream_t)stream);
+}
+
+int pace_step_decode(int32_t* token, int32_t* tok_pos, int32_t* start, const int64_t* next, const int64_t* pos, int32_t n,
+                     void* stream) {
+  if (!token || !tok_pos || !start || !next || !pos || n < 0) return PACE_ERR_INVALID;
+  if (n == 0) return PACE_OK;
+  step_decode_kernel<<<(n + 127) / 128, 128, 0, (cudaStream_t)stream>>>(token, tok_pos, start, next, pos, n);
+  PACE_LAUNCH_CHECK("step_decode_kernel");
+  return PACE_OK;
+}
+
+}  // extern "C"

@@ -56,8 +56,8 @@ bool geometry_ok(const pace_kv_pool_t* g) {
   if (g->n_layers <= 0 || g->n_kv_heads <= 0 || g->page_tokens <= 0 || g->n_pages <= 0 || g->max_seqs <= 0 ||
       g->max_pages_per_seq <= 0)
     return false;
-  if (g->head_dim != 64 && g->head_dim != 128) return false;
-  return true;
+  if (g->row_format == PACE_ROWS_OPAQUE) return g->head_dim > 0 && g->head_dim % 8 == 0 && g->head_dim <= 2048;
+  return g->row_format == PACE_ROWS_BF16 && (g->head_dim == 64 || g->head_dim == 128);
 }
 
 // ---------------------------------------------------------------------------
@@ -711,6 +711,8 @@ bool pool_ok(const pace_kv_pool_t* p) {
   return geometry_ok(p) && p->pages && p->block_table && p->seq_len && p->seq_pages && p->page_ref &&
          p->free_stack && p->counters && p->status && p->table_tmp;
 }
+// the entry points that move or interpret bf16 rows
+bool bf16_rows(const pace_kv_pool_t* p) { return p->row_format == PACE_ROWS_BF16; }
 
 }  // namespace
 }  // namespace pace
@@ -831,6 +833,7 @@ int pace_kv_append(const pace_kv_pool_t* p, int32_t layer, const int32_t* seq_id
       layer >= p->n_layers)
     return PACE_ERR_INVALID;
   if (batch == 0 || n_new == 0) return PACE_OK;
+  if (!bf16_rows(p)) return PACE_ERR_UNSUPPORTED;
   if (!k_new || !v_new) return PACE_ERR_INVALID;
   PACE_PROFILE("kv_append", stream, "layer=%d batch=%d n_new=%d", layer, batch, n_new);
   // 16-byte vector moves: bases and strides must keep rows 16-byte aligned
@@ -871,6 +874,7 @@ int pace_kv_append_layers(const pace_kv_pool_t* p, int32_t layer_begin, int32_t 
   PACE_PROFILE("kv_append_layers", stream, "layers=%d..%d batch=%d n_new=%d rows=%d", layer_begin, layer_end, batch, n_new,
                lengths_only ? 0 : 1);
   if (!lengths_only && (!k_new || !v_new)) return PACE_ERR_INVALID;
+  if (!lengths_only && !bf16_rows(p)) return PACE_ERR_UNSUPPORTED;
   if (!lengths_only &&
       (((uintptr_t)k_new & 15) || ((uintptr_t)v_new & 15) || (sl & 7) || (sb & 7) || (sh & 7) || (st & 7)))
     return PACE_ERR_INVALID;
@@ -910,6 +914,7 @@ int pace_kv_append_rope(const pace_kv_pool_t* p, int32_t layer, const int32_t* s
       layer >= p->n_layers)
     return PACE_ERR_INVALID;
   if (batch == 0 || n_new == 0) return PACE_OK;
+  if (!bf16_rows(p)) return PACE_ERR_UNSUPPORTED;
   if (!a->q || !a->k || !a->v || !a->q_out || !a->table_row || !a->cos_table || !a->sin_table) return PACE_ERR_INVALID;
   PACE_PROFILE("kv_append_rope", stream, "layer=%d batch=%d n_new=%d", layer, batch, n_new);
   if (a->n_q_heads < 1 || a->table_rows < 1 || a->rotary_dim < 16 || a->rotary_dim > p->head_dim || (a->rotary_dim & 15))
@@ -1009,6 +1014,7 @@ int pace_kv_read_dense(const pace_kv_pool_t* p, int32_t layer, const int32_t* se
                        void* v_out, int32_t cap, void* stream) {
   if (!pool_ok(p) || !seq_ids || batch < 0 || cap < 0 || layer < 0 || layer >= p->n_layers) return PACE_ERR_INVALID;
   if (batch == 0 || cap == 0) return PACE_OK;
+  if (!bf16_rows(p)) return PACE_ERR_UNSUPPORTED;
   if (!k_out || !v_out || ((uintptr_t)k_out & 15) || ((uintptr_t)v_out & 15)) return PACE_ERR_INVALID;
   const size_t total = (size_t)batch * p->n_kv_heads * cap * (p->head_dim / 8);
   size_t blocks = (total + 255) / 256;

@@ -28,8 +28,12 @@ class KVPoolStruct(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("n_layers", "n_kv_heads", "head_dim", "page_tokens", "n_pages",
                                           "max_seqs", "max_pages_per_seq", "owns_memory")] + \
                [(n, C.c_void_p) for n in ("pages", "block_table", "seq_len", "seq_pages", "page_ref",
-                                          "free_stack", "counters", "status", "table_tmp")]
+                                          "free_stack", "counters", "status", "table_tmp")] + \
+               [("row_format", C.c_int32)]
 
+
+ROWS_BF16, ROWS_OPAQUE = 0, 1   # PACE_ROWS_*
+DTYPE_BF16, DTYPE_FP32 = 0, 1   # PACE_DTYPE_*
 
 ATTN_WHOLE_UNITS = 1      # PACE_ATTN_WHOLE_UNITS
 ATTN_PENDING_ROW = 2      # PACE_ATTN_PENDING_ROW
@@ -61,7 +65,38 @@ class RopeArgs(C.Structure):
                 ("stage_stride_h", C.c_int64), ("stage_stride_t", C.c_int64)]
 
 
+class StepStruct(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("n_tokens", "n_entries", "max_count", "reserved")] + \
+               [(n, C.c_void_p) for n in ("token", "tok_entry", "tok_pos", "q_row", "cu", "start", "slot")]
+
+
+class ResidualNormArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("x", "y", "w_post", "embed", "w_next", "h")] + [("y_stride", C.c_int64)] + \
+               [(n, C.c_int32) for n in ("width", "vocab", "restart", "dtype")] + \
+               [("eps", C.c_float), ("weight_offset", C.c_float)]
+
+
+class AppendNormArgs(C.Structure):
+    _fields_ = [("qkv", C.c_void_p), ("qkv_stride", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("q_norm", "k_norm", "q_out")] + \
+               [(n, C.c_int32) for n in ("n_q_heads", "dim", "vdim", "dtype")] + \
+               [("eps", C.c_float), ("q_mul", C.c_float), ("temp_coef", C.c_float), ("temp_every", C.c_double)]
+
+
+class RglruArgs(C.Structure):
+    _fields_ = [("yx", C.c_void_p), ("yx_stride", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("u", "gates", "gate_w", "taps", "conv_bias", "ra_bias", "ri_bias", "decay_base",
+                                          "state", "conv_state", "out")] + \
+               [(n, C.c_int32) for n in ("width", "blocks", "n_taps", "dtype")]
+
+
+class LightningArgs(C.Structure):
+    _fields_ = [("qkv", C.c_void_p), ("qkv_stride", C.c_int64), ("decay", C.c_void_p), ("state", C.c_void_p),
+                ("out", C.c_void_p)] + [(n, C.c_int32) for n in ("heads", "dim", "vdim", "dtype")]
+
+
 byref = C.byref
+_S = C.POINTER(StepStruct)
 _P = C.POINTER(KVPoolStruct)
 _SIGS = {
     "pace_last_cuda_error": (C.c_char_p, []),
@@ -100,6 +135,22 @@ _SIGS = {
     "pace_linear_workspace_bytes": (C.c_uint64, [C.c_int32]),
     "pace_linear_skinny": (C.c_int, [C.c_void_p, C.c_int64, C.c_void_p, C.c_int64, C.c_void_p, C.c_int64, C.c_int32,
                                      C.c_int32, C.c_int32, C.c_void_p, C.c_uint64, C.c_void_p, C.c_void_p]),
+    "pace_residual_norm": (C.c_int, [_S, C.POINTER(ResidualNormArgs), C.c_void_p]),
+    "pace_kv_append_norm": (C.c_int, [_P, C.c_int32, _S, C.POINTER(AppendNormArgs), C.c_void_p]),
+    "pace_attn_general": (C.c_int, [_P, C.c_int32, _S, C.c_void_p, C.c_void_p, C.c_int32, C.c_int32, C.c_int32, C.c_float,
+                                    C.c_int32, C.c_void_p]),
+    "pace_gate_heads": (C.c_int, [_S, C.c_void_p, C.c_void_p, C.c_int64, C.c_void_p, C.c_int32, C.c_int32, C.c_int32,
+                                  C.c_int32, C.c_void_p]),
+    "pace_norm_gate": (C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int64, C.c_void_p, C.c_int32, C.c_int32, C.c_float,
+                                 C.c_int32, C.c_void_p]),
+    "pace_relu_squared": (C.c_int, [C.c_void_p, C.c_int64, C.c_int32, C.c_void_p]),
+    "pace_causal_conv": (C.c_int, [_S, C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_int32, C.c_void_p, C.c_void_p,
+                                   C.c_int32, C.c_int32, C.c_void_p]),
+    "pace_rglru_scan": (C.c_int, [_S, C.POINTER(RglruArgs), C.c_void_p]),
+    "pace_rglru_step": (C.c_int, [_S, C.POINTER(RglruArgs), C.c_void_p]),
+    "pace_lightning_prefill": (C.c_int, [_S, C.POINTER(LightningArgs), C.c_void_p]),
+    "pace_lightning_step": (C.c_int, [_S, C.POINTER(LightningArgs), C.c_void_p]),
+    "pace_step_decode": (C.c_int, [C.c_void_p] * 5 + [C.c_int32, C.c_void_p]),
     "pace_attention_dense": (C.c_int, [C.c_void_p] * 4 + [C.c_int32, C.c_int32, C.c_void_p] + [C.c_int32] * 6 +
                              [C.c_void_p, C.c_uint64, C.c_void_p]),
 }

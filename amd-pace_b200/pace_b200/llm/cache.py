@@ -95,14 +95,14 @@ class KVPool:
     """Device memory + descriptor of one paged pool (C struct pace_kv_pool_t)."""
 
     def __init__(self, n_layers: int, n_kv_heads: int, head_dim: int, page_tokens: int, n_pages: int,
-                 max_seqs: int, max_pages_per_seq: int, device):
+                 max_seqs: int, max_pages_per_seq: int, device, row_format: int = _C.ROWS_BF16):
         device = torch.device(device)
         if device.type != "cuda":
             raise RuntimeError("pace_b200 KV pools live in CUDA memory; got device " + str(device))
         self.device = device
         self.desc = _C.KVPoolStruct(n_layers=n_layers, n_kv_heads=n_kv_heads, head_dim=head_dim,
                                     page_tokens=page_tokens, n_pages=n_pages, max_seqs=max_seqs,
-                                    max_pages_per_seq=max_pages_per_seq)
+                                    max_pages_per_seq=max_pages_per_seq, row_format=row_format)
         pb, mb = C.c_uint64(), C.c_uint64()
         _C.check(_C.lib.pace_kv_pool_bytes(C.byref(self.desc), C.byref(pb), C.byref(mb)), "pace_kv_pool_bytes")
         # zero-filled like the reference's fresh segments (cache.py:255-256)
@@ -279,6 +279,28 @@ class KVCacheManager:
         self.slots = self.pool.alloc_slots(batch)
         self.slots_dev = torch.tensor(self.slots, dtype=torch.int32, device=self.pool.device)
         self.identity_slots = self.slots == list(range(batch))
+
+    def open_batch(self, batch: int) -> None:
+        """Takes ``batch`` slots of a shared pool at once, for callers whose layers write the pool themselves
+        (``advance_step``) instead of handing tensors to ``update_cache``."""
+        pool = self.pool
+        self._ensure_pool(batch, pool.n_kv_heads, pool.head_dim, pool.device)
+        for c in self.cache_objects:
+            c._lens, c.concat_dim = [0] * batch, 2
+            c.key, c.value = PagedKV(c, "k"), PagedKV(c, "v")
+
+    def advance_step(self, counts: Sequence[int], slots: torch.Tensor, counts_dev: torch.Tensor, n_max: int) -> None:
+        """Reserves the pages of a step's tokens and advances every layer's lengths by ``counts`` (one per batch
+        row), before the layers' own kernels store the rows.  ``slots`` / ``counts_dev`` (int32, device) list the
+        sequences that take part, at most ``n_max`` tokens each."""
+        pool, first = self.pool, self.cache_objects[0]
+        grow = first._host_account(counts, dry_run=self.capturing)
+        if not self.capturing:
+            for c in self.cache_objects[1:]:
+                c._lens, c._capacity = list(first._lens), first._capacity
+        if (not self.skip_reserve) if self.static_launch else (grow or pool.shared_pages):
+            _OPS.kv_reserve(pool.handle, pool.meta, 0, slots, n_max, counts_dev)
+        _OPS.kv_append_layers(pool.handle, pool.pages, pool.meta, 0, self.num_layers, slots, None, None, n_max, counts_dev)
 
     def __len__(self) -> int:
         return int(self.cache_objects[0].seq_len)

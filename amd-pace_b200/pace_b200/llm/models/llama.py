@@ -14,8 +14,8 @@ Differences that come from the path being on the GPU:
   * ``forward_tokens`` takes only the NEW tokens and allows ragged counts per sequence, which
     batched speculative decoding needs; ``forward`` is the reference signature on top of it.
 """
-import math
-from typing import List, Optional, Sequence
+from types import SimpleNamespace
+from typing import Dict, Optional, Sequence
 
 import torch
 import torch.nn.functional as F
@@ -23,6 +23,7 @@ from torch import nn
 
 from pace_b200.llm.cache import KVCacheBase, KVCacheManager
 from pace_b200.llm.outputs import ModelOutput
+from pace_b200.llm.registry import model_registry
 from pace_b200.ops import MultiHeadAttention, RotaryEmbedding
 from pace_b200.ops.linear import linear
 
@@ -255,19 +256,43 @@ class LlamaForCausalLM(nn.Module):
         return ModelOutput(logits=_lin(self.lm_head, hidden))
 
     # -- packed form used by continuous batching ----------------------------------------------------
-    def forward_packed(self, tokens: torch.Tensor, counts: Sequence[int], kv_cache: KVCacheManager) -> ModelOutput:
+    def forward_packed(self, tokens: torch.Tensor, counts: Sequence[int], kv_cache: KVCacheManager,
+                       rows: Optional[Sequence[int]] = None) -> ModelOutput:
         """``tokens`` [T] holds the new tokens of every sequence back to back, ``counts[b]`` of them for
         sequence b (zero for a sequence that sits this step out); positions continue from each
         sequence's cached length.  Returns the logits of the LAST new token of every sequence that had
-        any, as ``[B, vocab]`` (rows of idle sequences are zero): the LM head runs on those rows only."""
+        any, as ``[B, vocab]`` (rows of idle sequences are zero): the LM head runs on those rows only.
+        With ``rows`` (places in ``tokens``) it returns the logits of those instead, ``[len(rows), vocab]``."""
         B = len(counts)
+        tokens = tokens.to(self.lm_head.weight.device)
         cached = kv_cache[0].seq_lens if kv_cache[0].seq_lens else [0] * B
         pk = Packed(counts, cached, self.model.rotary_emb, self.config, tokens.device,
                     self.config.max_position_embeddings)
         hidden = self.model.forward_packed(tokens, pk, kv_cache)
+        if rows is not None:
+            return ModelOutput(logits=self.lm_head(hidden[torch.tensor(list(rows), dtype=torch.long, device=hidden.device)]))
         logits = torch.zeros(B, self.vocab_size, dtype=hidden.dtype, device=hidden.device)
         logits[torch.tensor(pk.live, device=hidden.device)] = self.lm_head(hidden[pk.last_rows])
         return ModelOutput(logits=logits)
+
+    def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
+        """Checkpoint names: the reference's state dict, or the plain ``mlp.up_proj.weight`` form of it."""
+        fused = {f"{n}.weight": f"{n}.linear.weight" for n, m in self.named_modules() if isinstance(m, _FusedLinear)}
+        renamed = {fused.get(k, k): v for k, v in tensors.items() if not k.endswith("rotary_emb.inv_freq")}
+        if "lm_head.weight" not in renamed and "model.embed_tokens.weight" in renamed:
+            renamed["lm_head.weight"] = renamed["model.embed_tokens.weight"]     # tied embeddings
+        self.load_state_dict(renamed, strict=True)
+
+
+def _from_config_json(config: dict, dtype: torch.dtype) -> LlamaForCausalLM:
+    cfg = SimpleNamespace(**config)
+    cfg.num_key_value_heads = getattr(cfg, "num_key_value_heads", None) or cfg.num_attention_heads
+    cfg.rope_theta = getattr(cfg, "rope_theta", 10000.0)
+    cfg.pad_token_id = getattr(cfg, "pad_token_id", None)
+    return LlamaForCausalLM(cfg).to(dtype)
+
+
+model_registry.register("LlamaForCausalLM", _from_config_json)
 
 
 def random_init_(model: nn.Module, seed: int, std: float = 0.02) -> nn.Module:

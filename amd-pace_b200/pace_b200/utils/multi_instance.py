@@ -35,11 +35,17 @@ def _init_instance(rank, args):
     import torch
     from pace_b200.llm.models.llama import LlamaForCausalLM, random_init_
     from pace_b200.llm.serving import ContinuousBatcher, WaveServer
+    dev = torch.device("cuda", torch.cuda.current_device())
+    if args.model:
+        from pace_b200.llm.registry import load_model
+        model = load_model(args.model, getattr(torch, args.dtype), dev)
+        server = ContinuousBatcher(model, pool_tokens=args.pool_tokens, max_batch=args.max_batch,
+                                   max_seq_len=args.max_len + args.new_tokens, prefill_chunk=512)
+        return {"rank": rank, "server": server, "cfg": model.config}
     cfg = _Cfg(hidden_size=args.hidden, intermediate_size=args.ffn, num_hidden_layers=args.layers,
                num_attention_heads=args.heads, num_key_value_heads=args.kv_heads, vocab_size=args.vocab,
                max_position_embeddings=args.max_len + args.new_tokens + 64, rope_theta=500000.0, rms_norm_eps=1e-5,
                pad_token_id=0)
-    dev = torch.device("cuda", torch.cuda.current_device())
     model = random_init_(LlamaForCausalLM(cfg).to(torch.bfloat16), seed=1).to(dev).eval()
     cls = ContinuousBatcher if args.scheduler == "continuous" else WaveServer
     server = cls(model, pool_tokens=args.pool_tokens, max_batch=args.max_batch,
@@ -52,12 +58,13 @@ def _serve(state, args, world, in_queue, out_queue):
     instances that died when the dispatcher hands them out again."""
     import torch
     rank = state["rank"]
+    vocab = state["cfg"].vocab_size
     lengths = make_prompt_lengths(args.requests_per_gpu * world, args.min_len, args.max_len, seed=7)
 
     def one_shard(shard):
         mine = shard_requests(len(lengths), world, shard)
         g = torch.Generator().manual_seed(100 + shard)
-        prompts = [torch.randint(1, args.vocab, (lengths[i],), generator=g) for i in mine]
+        prompts = [torch.randint(1, vocab, (lengths[i],), generator=g) for i in mine]
         t0 = time.perf_counter()
         _, stats = state["server"].run(prompts, args.new_tokens)
         dt = time.perf_counter() - t0
@@ -83,9 +90,14 @@ def main():
     ap.add_argument("--heads", type=int, default=32)
     ap.add_argument("--kv-heads", type=int, default=8)
     ap.add_argument("--vocab", type=int, default=128256)
+    ap.add_argument("--model", help="serve the checkpoint of this folder (config.json + model.safetensors, any registered "
+                                    "architecture) instead of a random model of the given shape")
+    ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16", help="number format of --model")
     ap.add_argument("--scheduler", choices=["continuous", "wave"], default="continuous")
     ap.add_argument("--timeout-s", type=float, default=3600.0, help="give up when the shards are not served by then")
     args = ap.parse_args()
+    if args.model and args.scheduler != "continuous":
+        ap.error("--model is served by the continuous scheduler")
     ctx = mp.get_context("spawn")
     inq, out = ctx.Queue(), ctx.Queue()
     # every instance keeps its own slice of the host cores (the reference gives each instance

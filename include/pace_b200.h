@@ -69,6 +69,7 @@ typedef struct pace_kv_pool {
   int32_t* counters;    /* device */
   int32_t* status;      /* device */
   int32_t* table_tmp;   /* device */
+  int32_t row_format;   /* PACE_ROWS_*: 0 = bf16 rows of 64 or 128 */
 } pace_kv_pool_t;
 
 const char* pace_last_cuda_error(void);
@@ -375,6 +376,154 @@ uint64_t pace_linear_workspace_bytes(int32_t n_max);
 int pace_linear_skinny(const void* x, int64_t x_stride, const void* w, int64_t w_stride, void* y, int64_t y_stride,
                        int32_t M, int32_t N, int32_t K, void* workspace, uint64_t workspace_bytes, int32_t* status,
                        void* stream);
+
+/* ==== layers of hybrid decoders (attention beside recurrent layers) =====================================
+ * Building blocks for models whose layers are not all softmax attention over the pool: fused norms, the
+ * append of normalised keys, an attention kernel for any row format, short convolutions, gated linear
+ * recurrences and decayed linear attention.  They work on a step's tokens packed back to back ([n_tokens]
+ * rows, all sequences), described by pace_step_t.  `dtype` is the type of activations, projection outputs
+ * and cache rows: PACE_DTYPE_BF16 or PACE_DTYPE_FP32; the residual stream, norms, gates, attention scores
+ * and recurrent states are fp32 with either.  (No counterpart in the reference, which serves attention-only
+ * decoders.) */
+#define PACE_DTYPE_BF16 0
+#define PACE_DTYPE_FP32 1
+
+/* Values of pace_kv_pool_t::row_format.
+ * PACE_ROWS_BF16: K and V rows are head_dim bf16 values, head_dim 64 or 128; every entry point takes them.
+ * PACE_ROWS_OPAQUE: rows are head_dim 16-bit units of any content (head_dim a multiple of 8, at most 2048):
+ * fp32 rows, other head sizes.  The allocator's entry points (reserve, release, truncate, gather,
+ * append_layers without rows, query), pace_kv_append_norm and pace_attn_general take them; the rest answers
+ * PACE_ERR_UNSUPPORTED. */
+#define PACE_ROWS_BF16 0
+#define PACE_ROWS_OPAQUE 1
+
+/* The tokens of one step.  Entry e (a sequence that takes part) owns rows [cu[e], cu[e + 1]); its first
+ * token has position start[e]; `slot` is its slot in the pool and in the recurrent states.  A state is
+ * never cleared: an entry with start[e] == 0 begins from zeros whatever its slot holds.  All device. */
+typedef struct pace_step {
+  int32_t n_tokens, n_entries, max_count; /* max_count: most tokens any entry has */
+  int32_t reserved;
+  const int32_t* token;     /* [n_tokens] token ids (embedding lookup) */
+  const int32_t* tok_entry; /* [n_tokens] */
+  const int32_t* tok_pos;   /* [n_tokens] position in the sequence */
+  const int32_t* q_row;     /* [n_tokens] row of the attention staging buffers the token uses */
+  const int32_t* cu;        /* [n_entries + 1] */
+  const int32_t* start;     /* [n_entries] */
+  const int32_t* slot;      /* [n_entries] */
+} pace_step_t;
+
+/* One pass over the residual stream x (fp32 [n_tokens][width]) between two sublayers:
+ *     x' = (restart ? 0 : x) + rms(y) * w_post + (embed ? embed[token] : 0)
+ *     h  = rms(x') * w_next,       rms(z) = z / sqrt(mean(z^2) + eps)
+ * y (the sublayer's output) may be NULL, embed may be NULL (with restart and embed it is the embedding
+ * lookup in front of the first layer; with y and embed the re-injection of the embeddings between two
+ * passes of a loop), w_next / h may be NULL.  w_post == NULL adds y as it is.  Norm weights are fp32
+ * [width] and used as weight_offset + w (1 for "one plus weight" norms).  embed is dtype [vocab][width]. */
+typedef struct {
+  float* x;
+  const void* y;
+  const float* w_post;
+  const void* embed;
+  const float* w_next;
+  void* h;
+  int64_t y_stride;
+  int32_t width, vocab, restart, dtype;
+  float eps, weight_offset;
+} pace_residual_norm_args_t;
+int pace_residual_norm(const pace_step_t* step, const pace_residual_norm_args_t* a, void* stream);
+
+/* Projection output -> attention operands, in one pass per token: RMS norm of the whole query and the whole
+ * key projection (q_norm / k_norm fp32 weights over all heads; NULL = no norm), queries times
+ *     q_mul * (1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1))        (temp_coef 0: no temperature)
+ * to q_out rows [q_row][n_q_heads][row elements], keys and values into the pages of pool layer `layer` at
+ * positions tok_pos.  The pages must be reserved; lengths are left alone (pace_kv_append_layers without rows
+ * advances them).  qkv is dtype [n_tokens][qkv_stride]: q (n_q_heads x dim), k (kv_heads x dim), v (kv_heads
+ * x vdim).  A pool row holds max(dim, vdim) or more elements; what a row has beyond dim / vdim is zeroed. */
+typedef struct {
+  const void* qkv;
+  int64_t qkv_stride;
+  const float* q_norm;
+  const float* k_norm;
+  void* q_out;
+  int32_t n_q_heads, dim, vdim, dtype;
+  float eps, q_mul, temp_coef;
+  double temp_every;
+} pace_append_norm_args_t;
+int pace_kv_append_norm(const pace_kv_pool_t* pool, int32_t layer, const pace_step_t* step,
+                        const pace_append_norm_args_t* a, void* stream);
+
+/* Causal softmax attention over the pool for any row format: q and out are dtype [q_row][n_q_heads][row
+ * elements]; scores, weights and sums in fp32.  dim, vdim <= 512.  CUDA cores; the tensor-core kernels
+ * (pace_attn_decode / pace_attn_prefill) take the PACE_ROWS_BF16 pools. */
+int pace_attn_general(const pace_kv_pool_t* pool, int32_t layer, const pace_step_t* step, const void* q, void* out,
+                      int32_t n_q_heads, int32_t dim, int32_t vdim, float scale, int32_t dtype, void* stream);
+
+/* out[t][h * vdim + i] = attn[q_row[t]][h][i] * sigmoid(gate[t][h * vdim + i]);
+ * attn rows are [n_heads][row_elems], gate has gate_stride elements per token. */
+int pace_gate_heads(const pace_step_t* step, const void* attn, const void* gate, int64_t gate_stride, void* out,
+                    int32_t n_heads, int32_t vdim, int32_t row_elems, int32_t dtype, void* stream);
+/* out[t] = rms(o[t]) * w * sigmoid(gate[t]) over n elements (w fp32). */
+int pace_norm_gate(const void* o, const float* w, const void* gate, int64_t gate_stride, void* out, int32_t n_tokens,
+                   int32_t n, float eps, int32_t dtype, void* stream);
+/* x = relu(x)^2 in place, n elements. */
+int pace_relu_squared(void* x, int64_t n, int32_t dtype, void* stream);
+
+/* Causal depthwise convolution: out[t][c] = bias[c] + sum_j taps[c][j] in[c](pos - (n_taps - 1) + j), zeros
+ * in front of the sequence.  conv_state fp32 [slots][n_taps][channels] holds each slot's newest inputs in row
+ * position % n_taps (a row is overwritten only when no later token needs it).  This entry point reads it;
+ * the recurrence behind it stores the new inputs. */
+int pace_causal_conv(const pace_step_t* step, const void* in, int64_t in_stride, const float* taps, const float* bias,
+                     int32_t n_taps, const float* conv_state, void* out, int32_t channels, int32_t dtype, void* stream);
+
+/* Real-gated linear recurrence (RG-LRU) with its branch product:
+ *     r = sigmoid(gates_r + ra_bias), i = sigmoid(gates_i + ri_bias), log a = decay_base * r
+ *     S_t = a S_(t-1) + sqrt(1 - a^2) i u,    out = S * gelu_tanh(y)
+ * decay_base fp32 [width] (= -8 softplus(lam)); state fp32 [slots][width].  yx is dtype [n_tokens][yx_stride]
+ * with y in columns [0, width) and the convolution's input in [width, 2 width): its newest rows go to
+ * conv_state.
+ * pace_rglru_scan: gates fp32 [blocks][n_tokens][2][width / blocks] (r, i) and u dtype [n_tokens][width] come
+ * from launches in front (any counts per entry).
+ * pace_rglru_step: one token per entry (n_tokens == n_entries); convolution and block-diagonal gates
+ * (gate_w dtype [blocks][2][out][in]) are part of the launch. */
+typedef struct {
+  const void* yx;
+  int64_t yx_stride;
+  const void* u;          /* scan only */
+  const float* gates;     /* scan only */
+  const void* gate_w;     /* step only */
+  const float* taps;      /* step only: fp32 [width][n_taps] */
+  const float* conv_bias; /* step only */
+  const float* ra_bias;
+  const float* ri_bias;
+  const float* decay_base;
+  float* state;
+  float* conv_state;
+  void* out;              /* dtype [n_tokens][width] */
+  int32_t width, blocks, n_taps, dtype;
+} pace_rglru_args_t;
+int pace_rglru_scan(const pace_step_t* step, const pace_rglru_args_t* a, void* stream);
+int pace_rglru_step(const pace_step_t* step, const pace_rglru_args_t* a, void* stream);
+
+/* Linear attention with a fixed decay per head: with q, k, v = silu of the projections (rounded to dtype),
+ *     S_t = decay S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t.
+ * qkv dtype [n_tokens][qkv_stride]: q (heads x dim), k (heads x dim), v (heads x vdim).  state fp32
+ * [slots][heads][dim][vdim].  out dtype [n_tokens][heads x vdim].  dim <= 512 (vdim any).
+ * pace_lightning_step: one token per entry; pace_lightning_prefill: any counts. */
+typedef struct {
+  const void* qkv;
+  int64_t qkv_stride;
+  const float* decay;     /* fp32 [heads] */
+  float* state;
+  void* out;
+  int32_t heads, dim, vdim, dtype;
+} pace_lightning_args_t;
+int pace_lightning_prefill(const pace_step_t* step, const pace_lightning_args_t* a, void* stream);
+int pace_lightning_step(const pace_step_t* step, const pace_lightning_args_t* a, void* stream);
+
+/* Step arrays of a decode step whose tokens and positions the device holds (one token per entry):
+ * token[i] = next_token[i], tok_pos[i] = start[i] = position[i]. */
+int pace_step_decode(int32_t* token, int32_t* tok_pos, int32_t* start, const int64_t* next_token,
+                     const int64_t* position, int32_t n_entries, void* stream);
 
 #ifdef __cplusplus
 }

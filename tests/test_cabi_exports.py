@@ -66,7 +66,9 @@ def test_dispatcher_ops_are_registered_without_a_gpu():
     import pace_b200.torch_ops  # noqa: F401
     names = ["kv_reserve", "kv_append", "kv_append_layers", "kv_append_rope", "kv_truncate", "kv_gather",
              "kv_read_dense", "pard_accept", "linear_skinny", "attn_decode", "attn_decode_cuda_cores",
-             "attn_verify", "attn_prefill"]
+             "attn_verify", "attn_prefill", "residual_norm", "kv_append_norm", "attn_general", "gate_heads", "norm_gate",
+             "relu_squared", "causal_conv", "rglru_scan", "rglru_step", "lightning_prefill", "lightning_step",
+             "step_decode"]
     for n in names:
         op = getattr(torch.ops.pace_b200, n)
         assert torch._C._dispatch_has_kernel_for_dispatch_key(f"pace_b200::{n}", "CUDA"), n
