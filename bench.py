@@ -887,6 +887,250 @@ def run_linear(args):
     print(json.dumps(linear_measure()), flush=True)
 
 
+# ---------------------------------------------------------------------------------------------------
+# hybrid decoder (Garupel) beside the attention-only decoder at equal size
+# ---------------------------------------------------------------------------------------------------
+HYBRID_SIZES = {
+    "w2048": dict(width=2048, ff=8192, heads=16, kv_heads=4, dim=128, blocks=8, lin_heads=16),
+    "w4096": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, blocks=16, lin_heads=32),
+}
+HYBRID_VOCAB, HYBRID_LAYERS = 32000, 8
+
+
+def hybrid_models(size: str, dev):
+    """(Garupel, Llama) of one size with random weights: 8 layer runs each, of which Garupel's are 4 x rglru,
+    2 x lightning and 2 x attention."""
+    from pace_b200.llm.models.garupel import GarupelForCausalLM
+    from pace_b200.llm.models.llama import LlamaForCausalLM
+    from pace_b200.llm.registry import build_model
+    z = HYBRID_SIZES[size]
+    W, mlp = z["width"], {"kind": "dense", "ff": z["ff"]}
+    lru = {"type": "rglru", "mlp": mlp, "mixer": {"width": W, "blocks": z["blocks"], "conv": 4}}
+    lin = {"type": "lightning", "mlp": mlp, "mixer": {
+        "heads": z["lin_heads"], "dim": z["dim"], "vdim": z["dim"],
+        "decay": [2.0 ** -(8.0 * h / z["lin_heads"] / 8.0) for h in range(z["lin_heads"])]}}
+    att = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+        "q_temp": {"coef": 0.1, "every": 2048}}}
+    cfg = {"architecture": "Garupel", "vocab": HYBRID_VOCAB, "width": W, "norm": {"eps": 1e-5},
+           "layers": [lru, lru, lin, att] * (HYBRID_LAYERS // 4)}
+    garupel = build_model(cfg, torch.bfloat16, dev)
+    assert isinstance(garupel, GarupelForCausalLM)
+    garupel.random_init_(5)
+
+    class Cfg:
+        hidden_size, intermediate_size, num_hidden_layers = W, z["ff"], HYBRID_LAYERS
+        num_attention_heads, num_key_value_heads, vocab_size = z["heads"], z["kv_heads"], HYBRID_VOCAB
+        max_position_embeddings, rope_theta, rms_norm_eps, pad_token_id = 8192, 500000.0, 1e-5, 0
+        rope_scaling = None
+
+    with torch.device(dev):
+        llama = LlamaForCausalLM(Cfg()).to(torch.bfloat16).eval()
+    g = torch.Generator(device=dev).manual_seed(5)
+    with torch.no_grad():
+        for p_ in llama.parameters():
+            if p_.dim() >= 2:
+                p_.normal_(0.0, 0.02, generator=g)
+    return garupel, llama
+
+
+def hybrid_cache(model, batch: int, max_len: int, dev):
+    from pace_b200.llm.cache import KVCacheManager, KVCacheType, KVPool
+    if hasattr(model, "new_cache"):
+        return model.new_cache(batch, batch * (max_len + 128), max_len + 128)
+    c = model.config
+    per = (max_len + 128) // 64 + 2
+    pool = KVPool(c.num_hidden_layers, c.num_key_value_heads, c.hidden_size // c.num_attention_heads, 64, batch * per, batch,
+                  per, dev)
+    return KVCacheManager(c, max_len + 128, KVCacheType.BMC, pool=pool)
+
+
+@torch.inference_mode()
+def hybrid_throughput(model, dev):
+    """Prompt tokens/s of packed prefill passes and decode tokens/s of the device-resident greedy loop."""
+    from pace_b200.llm.device_loop import GreedyDeviceLoop
+    res, g = {}, torch.Generator().manual_seed(1)
+    for batch, n in ((1, 4096), (8, 512)):
+        toks = torch.randint(1, HYBRID_VOCAB, (batch * n,), generator=g)
+        cache = hybrid_cache(model, batch, n, dev)
+        times = []
+        for it in range(8):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            e0.record()
+            model.forward_packed(toks, [n] * batch, cache)
+            e1.record()
+            torch.cuda.synchronize()
+            times.append(e0.elapsed_time(e1))
+            cache.recycle(range(batch))
+        cache.pool.check_status()
+        ms = statistics.median(times[3:])
+        res[f"prefill_{batch}x{n}"] = {"ms": ms, "tokens_per_s": batch * n / ms * 1e3}
+        del cache
+    for batch, past in ((32, 512), (8, 4096)):
+        cache = hybrid_cache(model, batch, past + 160, dev)
+        ids = torch.randint(1, HYBRID_VOCAB, (batch, 512), generator=g).to(dev)
+        for done in range(0, past, 512):
+            pos = (torch.arange(512, device=dev) + done).expand(batch, 512)
+            model.model.forward_tokens(ids, cache, pos)
+        loop = GreedyDeviceLoop(model, cache, ids[:, -1], torch.full((batch,), past, device=dev), max_new_tokens=128)
+        for _ in range(16):
+            loop.graph.replay()
+        times = []
+        for _ in range(3):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            e0.record()
+            for _ in range(32):
+                loop.graph.replay()
+            e1.record()
+            torch.cuda.synchronize()
+            times.append(e0.elapsed_time(e1) / 32)
+        cache.pool.check_status()
+        ms = statistics.median(times)
+        res[f"decode_b{batch}_past{past}"] = {"ms_per_step": ms, "tokens_per_s": batch / ms * 1e3}
+        del loop, cache
+        torch.cuda.empty_cache()
+    return res
+
+
+def graph_us(launches, reps=5):
+    """Microseconds per launch of a list of launches recorded back to back (their operands together exceed L2)."""
+    side = torch.cuda.Stream()
+    side.wait_stream(torch.cuda.current_stream())
+    with torch.cuda.stream(side):
+        for f in launches:
+            f()
+    side.synchronize()
+    gr = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(gr, stream=side):
+        for f in launches:
+            f()
+    for _ in range(3):
+        gr.replay()
+    times = []
+    for _ in range(3):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        for _ in range(reps):
+            gr.replay()
+        e1.record()
+        torch.cuda.synchronize()
+        times.append(e0.elapsed_time(e1) * 1e3 / (reps * len(launches)))
+    return statistics.median(times)
+
+
+@torch.inference_mode()
+def hybrid_kernels(size: str, dev):
+    """Each kernel of the hybrid decoder alone, against its own roofline: bytes that must move over the measured
+    copy rate, or flops over the measured bf16 rate (sustained), whichever takes longer.  Shapes of `size`:
+    prefill = one sequence of 4096 tokens, decode = 32 sequences over 512 cached tokens."""
+    from pace_b200.llm.hybrid_cache import HybridCacheManager, KVSpec, StateSpec
+    from pace_b200.ops import hybrid
+    z = HYBRID_SIZES[size]
+    W, H, G, D, nb, LH, FF = z["width"], z["heads"], z["kv_heads"], z["dim"], z["blocks"], z["lin_heads"], z["ff"]
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(
+        os.path.join(ROOT, "MEASURED_PEAKS.json")) else {"hbm_gbs": FALLBACK_HBM_GBS, "bf16_tflops_sustained": 1400.0}
+    bw, fl = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops_sustained"] * 1e12
+    g = torch.Generator(device=dev).manual_seed(2)
+
+    def rnd(*shape, dtype=torch.bfloat16):
+        return torch.randn(*shape, device=dev, generator=g, dtype=torch.float32).to(dtype)
+
+    out = {}
+    for phase, batch, n, past in (("prefill", 1, 4096, 0), ("decode", 32, 1, 512)):
+        T, E, m = batch * n, batch, W // nb
+        dec = n == 1
+        N = 8 if dec else 3                        # copies of every operand
+        specs = [KVSpec(G, D, D)] * N + [StateSpec((("S", (W,)), ("conv", (4, W))))] * N + \
+                [StateSpec((("S", (LH, D, D)),))] * N
+        cache = HybridCacheManager(specs, batch, batch * (past + n + 64), past + n + 64, torch.bfloat16, dev)
+        if past:
+            cache.begin_step(cache.step([past] * batch, torch.zeros(batch * past, dtype=torch.long), 1))
+        step = cache.step([n] * batch, torch.zeros(T, dtype=torch.long), 1)
+        cache.begin_step(step)
+        vec = lambda k: rnd(k, dtype=torch.float32)                          # noqa: E731
+        x, y = [rnd(T, W, dtype=torch.float32) for _ in range(N)], [rnd(T, W) for _ in range(N)]
+        wp, wn = vec(W), vec(W)
+        nq, nk = H * D, G * D
+        qkvg = [rnd(T, nq * 2 + nk * 2) for _ in range(N)]
+        qn, kn = vec(nq), vec(nk)
+        yx = [rnd(T, 2 * W) for _ in range(N)]
+        gw = [rnd(nb, 2, m, m) * m ** -0.5 for _ in range(N)]
+        taps, cb, ra, ri, base = rnd(W, 4, dtype=torch.float32), vec(W), vec(W), vec(W), -vec(W).abs()
+        lq = [rnd(T, 4 * LH * D) for _ in range(N)]
+        decay = torch.linspace(0.9, 0.999, LH, device=dev)
+        lo = [rnd(T, LH * D) for _ in range(N)]
+        up = [rnd(T, FF) for _ in range(N)]
+        att_out = [rnd(step.staging_rows, H, D) for _ in range(N)]
+        kv_read = 2 * nk * 2 * (E * (past + 1) if dec else T)
+        flops = 4 * nq * (E * (past + 1) if dec else sum(range(1, n + 1)) * E)
+        rows = {}
+
+        def add(name, launches, nbytes, nflops=0.0):
+            us = graph_us(launches)
+            roof = max(nbytes / bw, nflops / fl) * 1e6
+            rows[name] = {"us": us, "roofline_us": roof, "frac": roof / us, "bound": "hbm" if nbytes / bw >= nflops / fl else "tensor"}
+
+        add("residual_norm", [lambda i=i: hybrid.residual_norm(step, x[i], y[i], wp, w_next=wn, eps=1e-5) for i in range(N)],
+            T * W * (4 + 4 + 2 + 2))
+        pool = cache[0].pool
+        qb = [torch.empty(step.staging_rows, H, D, dtype=torch.bfloat16, device=dev) for _ in range(N)]
+        add("append_norm", [lambda i=i: torch.ops.pace_b200.kv_append_norm(
+            pool.handle, pool.pages, i, step.handle, qkvg[i], qn, kn, qb[i], D, D, 1e-5, 1.0, 0.1, 2048.0) for i in range(N)],
+            T * (nq + 2 * nk) * 4)
+        add("append_norm+attention", [lambda i=i: hybrid.step_attention(
+            step, cache[i], qkvg[i], H, D, D, D ** -0.5, qn, kn, 1e-5, 0.1, 2048.0) for i in range(N)],
+            T * (nq + 2 * nk) * 4 + kv_read + T * nq * 4, flops)
+        add("gate_heads", [lambda i=i: hybrid.gate_heads(step, att_out[i], qkvg[i][:, nq + 2 * nk:], D) for i in range(N)],
+            T * nq * 6)
+        rg = E * W * 4 * (2 + 4)                  # state read and written, three ring rows read and one written
+        add("rglru", [lambda i=i: hybrid.rglru(step, yx[i], gw[i], taps, cb, ra, ri, base, cache[N + i]["S"],
+                                               cache[N + i]["conv"]) for i in range(N)],
+            T * W * 2 * 3 + nb * 2 * m * m * 2 + rg, T * W * m * 4.0)
+        add("lightning", [lambda i=i: hybrid.lightning(step, lq[i], decay, cache[2 * N + i]["S"]) for i in range(N)],
+            T * LH * D * 2 * 4 + E * LH * D * D * 8, 0.0 if dec else T * LH * (4 * D * D + 4 * D * 64.0))
+        add("norm_gate", [lambda i=i: hybrid.norm_gate(lo[i], wp[:LH * D] if LH * D <= W else vec(LH * D),
+                                                       lq[i][:, 3 * LH * D:], 1e-5) for i in range(N)], T * LH * D * 6)
+        add("relu_squared", [lambda i=i: hybrid.relu_squared_(up[i]) for i in range(N)], T * FF * 4)
+        cache.pool.check_status()
+        if not dec:                               # the parts of the recurrence's prefill
+            u = [rnd(T, W) for _ in range(N)]
+            gates = [rnd(nb, T, 2 * m, dtype=torch.float32) for _ in range(N)]
+            ro = torch.empty(T, W, dtype=torch.bfloat16, device=dev)
+            ops = torch.ops.pace_b200
+            add("rglru.conv", [lambda i=i: ops.causal_conv(step.handle, yx[i][:, W:], taps, cb, cache[N + i]["conv"], u[i])
+                               for i in range(N)], T * W * 4)
+            add("rglru.scan", [lambda i=i: ops.rglru_scan(step.handle, yx[i], u[i], gates[i], ra, ri, base, cache[N + i]["S"],
+                                                          cache[N + i]["conv"], ro, nb) for i in range(N)], T * W * 14)
+        out[phase] = rows
+        del cache
+        torch.cuda.empty_cache()
+    return out
+
+
+def run_hybrid(args):
+    """Side measurement: prefill and decode throughput of the Garupel decoder beside the Llama decoder at equal
+    width, heads, feed-forward and layer count (random weights), and every kernel of the former against its
+    roofline.  Prints one JSON line per size."""
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    for size in HYBRID_SIZES:
+        sampler = ClockSampler(0)
+        sampler.start()
+        garupel, llama = hybrid_models(size, dev)
+        line = {"workload": "hybrid", "size": size, **HYBRID_SIZES[size], "layer_runs": HYBRID_LAYERS,
+                "params": {"garupel": sum(p.numel() for p in garupel.parameters()),
+                           "llama": sum(p.numel() for p in llama.parameters())},
+                "garupel": hybrid_throughput(garupel, dev), "llama": hybrid_throughput(llama, dev)}
+        del garupel, llama
+        torch.cuda.empty_cache()
+        line["kernels"] = hybrid_kernels(size, dev)
+        line["clocks"] = sampler.stop()
+        print(json.dumps(line), flush=True)
+
+
 def main():
     # stdout carries the JSON line and nothing else: whatever native libraries print to file descriptor 1
     # (NCCL's version banner on some ranks) goes to stderr, Python's own prints keep the real stdout
@@ -904,7 +1148,8 @@ def main():
     ap.add_argument("--no-sweep", action="store_true", help="profiling aid: skip the timed blocks at other cache lengths")
     ap.add_argument("--layers", type=int, default=CFG["n_layers"],
                     help="profiling aid: fewer layers = less device memory; the bench line is only valid at 32")
-    ap.add_argument("--workload", default="decode", choices=["decode", "verify", "prefill", "rope_append", "device_loop", "serving", "linear"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "verify", "prefill", "rope_append", "device_loop", "serving", "linear",
+                                                                 "hybrid"],
                     help="decode = the bench line; verify / prefill = side measurements of the multi-token kernels")
     ap.add_argument("--past", type=int, default=3584, help="prefill side measurement: tokens cached before the chunk")
     ap.add_argument("--head-dim", type=int, default=128, choices=[64, 128])
@@ -919,10 +1164,10 @@ def main():
         return
     global RANK_CORES
     RANK_CORES = pin_rank_to_cores(local_rank, world)
-    if args.workload in ("rope_append", "device_loop", "serving", "linear"):
+    if args.workload in ("rope_append", "device_loop", "serving", "linear", "hybrid"):
         if rank == 0:
             {"rope_append": run_rope, "device_loop": run_device_loop, "serving": run_serving,
-             "linear": run_linear}[args.workload](args)
+             "linear": run_linear, "hybrid": run_hybrid}[args.workload](args)
         return
     if args.workload != "decode":
         if rank == 0:

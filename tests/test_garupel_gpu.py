@@ -161,8 +161,8 @@ def test_norms_and_temperature_of_queries_and_keys(dtype):
     assert float((got - want).abs().max()) < tol
     if dtype == BF16:      # a scale the tensor-core kernels do not take by themselves
         cache.recycle([1])
-        neg = _attend(qkv, cache, 1, [n], heads, dim, vdim, -0.4, **kw)
-        w = torch.stack([read(69, h, -0.4) for h in range(heads)])
+        neg = _attend(qkv, cache, 1, [n], heads, dim, vdim, -0.5, **kw)      # (a power of two: the same rounding of q)
+        w = torch.stack([read(69, h, -0.5) for h in range(heads)])
         assert float((neg[69] - w).abs().max()) < tol
 
 
