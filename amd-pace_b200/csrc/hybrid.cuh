@@ -90,11 +90,19 @@ template <typename T> __device__ __forceinline__ float silu_t(float x) { return 
 template <typename T> __device__ __forceinline__ float gelu_tanh_t(float z) {
   return z * sigmoid_t<T>(1.5957691216057308f * (z + 0.044715f * z * z * z));
 }
-// 1 - e^x for x <= 0 without cancellation: the series of expm1 near zero, the plain difference further out
-template <typename T> __device__ __forceinline__ float one_minus_exp(float x, float exp_x) {
+// sqrt(1 - e^x) for x <= 0 (exp_x = e^x) without cancellation: near zero 1 - e^x is the Taylor series
+// -x (1 + x/2 (1 + x/3 (1 + ...))), further out the plain difference
+template <typename T> __device__ __forceinline__ float sqrt_one_minus_exp(float x, float exp_x) {
+  // |x| < 1/16: the first term left out, x^4 / 120, is below 2e-7; the difference has lost four bits at most
+  const float s = -x * fmaf(x * (1.0f / 2), fmaf(x * (1.0f / 3), fmaf(x, 1.0f / 4, 1.0f), 1.0f), 1.0f);
+  float r;
+  asm("sqrt.approx.f32 %0, %1;" : "=f"(r) : "f"(x > -0.0625f ? s : 1.0f - exp_x));
+  return r;
+}
+template <> __device__ __forceinline__ float sqrt_one_minus_exp<float>(float x, float exp_x) {
   const float s = -x * (1.0f + x * (1.0f / 2) * (1.0f + x * (1.0f / 3) * (1.0f + x * (1.0f / 4) *
                   (1.0f + x * (1.0f / 5) * (1.0f + x * (1.0f / 6) * (1.0f + x * (1.0f / 7)))))));
-  return x > -0.25f ? s : 1.0f - exp_x;
+  return sqrtf(x > -0.25f ? s : 1.0f - exp_x);
 }
 
 // Sum over the thread block, the same value in every thread; `red` holds one float per warp.

@@ -1,0 +1,353 @@
+// Linear attention with a fixed decay per head over many tokens, in chunks of 64 on the tensor cores.
+//
+// With d = decay and a chunk whose state in front is S:
+//     out_i = d^(i+1) S^T q_i + sum_{j <= i} d^(i-j) (q_i . k_j) v_j,      S' = d^n S + sum_j d^(n-1-j) k_j v_j^T
+// q, k, v are bf16 values (silu of the projections); everything else is fp32: the state stays in fp32
+// accumulators, and where an fp32 quantity is the operand of a bf16 product it is split into two or three bf16
+// terms whose sum carries 16 or 24 bits (weights and the state that is read: two, the keys that enter the state
+// with their decay: three).
+//
+// A block owns (entry, head, up to 128 value columns) and a segment of chunks.  Sequences that would leave the
+// GPU half empty are cut into several segments: a first launch computes what each segment adds to the state, a
+// second one turns those into the states in front of the segments, then all segments run side by side.
+#include "hybrid.cuh"
+
+namespace pace {
+namespace {
+
+constexpr int kChunk = 64, kThreads = 256;
+
+struct SegmentArgs {
+  float* scratch;     // [entries][segments][heads][dim][vdim]: what a segment adds, then the state in front of it
+  int segments, seg_tokens;
+};
+
+__device__ __forceinline__ void mma16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldsm4(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p)));
+}
+// 16 bytes global -> shared, zeros when `live` is false
+__device__ __forceinline__ void copy16(void* dst, const void* src, bool live) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
+}
+// a pair of fp32 values as bf16 pairs hi + lo
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = f2_to_bf2(x, y);
+  const float2 h = bf2_to_f2(hi);
+  lo = f2_to_bf2(x - h.x, y - h.y);
+}
+
+template <int DP, int VP>
+struct Tiles {
+  static constexpr int QP = DP + 8, VQ = VP + 8;  // row pitches: 16 bytes beyond a power of two, ldmatrix without conflicts
+  static constexpr int kStage = kChunk * (2 * QP + VQ);   // q, k, v of one chunk
+  static constexpr int kState = DP * VQ;
+  static constexpr size_t bytes = sizeof(__nv_bfloat16) * (2 * kStage + 2 * kState) + sizeof(float) * (kChunk + 1);
+};
+
+template <int DP, int VP, bool STATE_ONLY>
+__global__ void __launch_bounds__(kThreads, 1)
+    lightning_chunk_kernel(pace_step_t st, pace_lightning_args_t a, SegmentArgs sg) {
+  using TL = Tiles<DP, VP>;
+  constexpr int QP = TL::QP, VQ = TL::VQ;
+  constexpr int RG = DP / 16, CG = 8 / RG, SC = VP / CG;   // state tile of a warp: 16 rows x SC columns
+  constexpr int NT = SC / 8;                               // its 8-column tiles
+  constexpr int OT = VP / 16;                              // output tiles of a warp (half of the columns)
+  extern __shared__ __align__(16) __nv_bfloat16 sm[];
+  __nv_bfloat16* s_hi = sm + 2 * TL::kStage;
+  __nv_bfloat16* s_lo = s_hi + TL::kState;
+  float* pw = reinterpret_cast<float*>(s_lo + TL::kState);
+
+  const int e = blockIdx.z / sg.segments, seg = blockIdx.z % sg.segments, h = blockIdx.y, v0 = blockIdx.x * VP;
+  const int d = a.dim, vd = a.vdim, H = a.heads;
+  const int t0 = st.cu[e], count = st.cu[e + 1] - t0, first = seg * sg.seg_tokens;
+  if (first >= count) return;
+  const int end = min(count, first + sg.seg_tokens);
+  const bool last = end == count;
+  if (STATE_ONLY && last) return;                          // nobody starts behind the last segment
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const float decay = a.decay[h];
+  if (tid <= kChunk) pw[tid] = powf(decay, (float)tid);
+
+  const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(a.qkv) + (size_t)t0 * a.qkv_stride;
+  auto fetch = [&](int l0, int buf) {
+    __nv_bfloat16* q = sm + buf * TL::kStage;
+    constexpr int per = (2 * DP + VP) / 8;                 // 16-byte pieces of one token
+    for (int i = tid; i < kChunk * per; i += kThreads) {
+      const int j = i / per, p = i - j * per;
+      const bool tok = l0 + j < end;
+      const __nv_bfloat16* row = base + (size_t)(tok ? l0 + j : first) * a.qkv_stride;
+      if (p < 2 * DP / 8) {
+        const int which = p / (DP / 8), c = (p - which * (DP / 8)) * 8;
+        if (STATE_ONLY && which == 0) continue;
+        copy16(q + which * kChunk * QP + j * QP + c, row + (size_t)(which * H + h) * d + (c < d ? c : 0), tok && c < d);
+      } else {
+        const int c = (p - 2 * DP / 8) * 8;
+        copy16(q + 2 * kChunk * QP + j * VQ + c, row + 2 * (size_t)H * d + (size_t)h * vd + (v0 + c < vd ? v0 + c : 0),
+               tok && v0 + c < vd);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  fetch(first, 0);
+
+  // the state in front of the segment
+  const int sr = (warp % RG) * 16 + (lane >> 2), sc = (warp / RG) * SC + (lane & 3) * 2;
+  float S[NT][4];
+  const float* from = nullptr;
+  if (!STATE_ONLY) {
+    if (sg.segments > 1) from = sg.scratch + (((size_t)e * sg.segments + seg) * H + h) * d * vd;
+    else if (st.start[e] != 0) from = a.state + ((size_t)st.slot[e] * H + h) * d * vd;
+  }
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const int r = sr + (q >> 1) * 8, c = v0 + sc + n * 8 + (q & 1);
+      S[n][q] = (from && r < d && c < vd) ? from[(size_t)r * vd + c] : 0.f;
+    }
+
+  int buf = 0;
+  for (int l0 = first; l0 < end; l0 += kChunk, buf ^= 1) {
+    const int n_tok = min(kChunk, end - l0);
+    __nv_bfloat16* q_s = sm + buf * TL::kStage;
+    __nv_bfloat16* k_s = q_s + kChunk * QP;
+    __nv_bfloat16* v_s = k_s + kChunk * QP;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                       // the chunk is here, the previous one is done with
+    constexpr int per = (2 * DP + VP) / 8;
+    for (int i = tid; i < kChunk * per; i += kThreads) {   // silu in place
+      const int j = i / per, p = i - j * per;
+      if (STATE_ONLY && p < DP / 8) continue;
+      __nv_bfloat16* x = p < 2 * DP / 8 ? q_s + (p / (DP / 8)) * kChunk * QP + j * QP + (p % (DP / 8)) * 8
+                                        : v_s + j * VQ + (p - 2 * DP / 8) * 8;
+      float f[8];
+      Vec<__nv_bfloat16, 8>::load(x, f);
+#pragma unroll
+      for (int u = 0; u < 8; ++u) f[u] = silu_t<__nv_bfloat16>(f[u]);
+      Vec<__nv_bfloat16, 8>::store(x, f);
+    }
+    if (!STATE_ONLY) {
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int q = 0; q < 4; q += 2) {
+          uint32_t hi, lo;
+          split2(S[n][q], S[n][q + 1], hi, lo);
+          const int at = (sr + (q >> 1) * 8) * VQ + sc + n * 8;
+          *reinterpret_cast<uint32_t*>(s_hi + at) = hi;
+          *reinterpret_cast<uint32_t*>(s_lo + at) = lo;
+        }
+    }
+    __syncthreads();
+    if (l0 + kChunk < end) fetch(l0 + kChunk, buf ^ 1);
+
+    if (!STATE_ONLY) {
+      // rows 16 (warp % 4), value columns VP / 2 (warp / 4)
+      const int m0 = (warp & 3) * 16, c0 = (warp >> 2) * (VP / 2);
+      float O[OT][4], P[8][4];
+#pragma unroll
+      for (int n = 0; n < OT; ++n) O[n][0] = O[n][1] = O[n][2] = O[n][3] = 0.f;
+#pragma unroll
+      for (int n = 0; n < 8; ++n) P[n][0] = P[n][1] = P[n][2] = P[n][3] = 0.f;
+      const int live_tiles = 2 * ((m0 >> 4) + 1);          // keys up to the tile's last row
+#pragma unroll
+      for (int k0 = 0; k0 < DP; k0 += 16) {
+        uint32_t A[4], B[4];
+        ldsm4(A, q_s + (m0 + (lane & 15)) * QP + k0 + (lane >> 4) * 8);
+#pragma unroll
+        for (int n = 0; n < OT; n += 2) {
+          const int at = (k0 + (lane & 15)) * VQ + c0 + n * 8 + (lane >> 4) * 8;
+          ldsm4t(B, s_hi + at);
+          mma16816(O[n], A, B[0], B[1]);
+          mma16816(O[n + 1], A, B[2], B[3]);
+          ldsm4t(B, s_lo + at);
+          mma16816(O[n], A, B[0], B[1]);
+          mma16816(O[n + 1], A, B[2], B[3]);
+        }
+#pragma unroll
+        for (int n = 0; n < 8; n += 2) {
+          if (n < live_tiles) {
+            ldsm4(B, k_s + (n * 8 + (lane & 7) + (lane >> 4) * 8) * QP + k0 + ((lane >> 3) & 1) * 8);
+            mma16816(P[n], A, B[0], B[1]);
+            mma16816(P[n + 1], A, B[2], B[3]);
+          }
+        }
+      }
+      const int i0 = m0 + (lane >> 2);
+      const float f0 = pw[i0 + 1], f1 = pw[i0 + 9];
+#pragma unroll
+      for (int n = 0; n < OT; ++n) {
+        O[n][0] *= f0; O[n][1] *= f0;
+        O[n][2] *= f1; O[n][3] *= f1;
+      }
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) {
+        if (2 * kk >= live_tiles) break;
+        uint32_t hi[4], lo[4], B[4];
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {                      // operand registers: (row half, key half)
+          const int n = 2 * kk + (x >> 1), r = i0 + (x & 1) * 8, j = n * 8 + (lane & 3) * 2;
+          float* p = &P[n][(x & 1) * 2];
+          const float w0 = j <= r ? p[0] * pw[r - j] : 0.f;
+          const float w1 = j + 1 <= r ? p[1] * pw[r - j - 1] : 0.f;
+          split2(w0, w1, hi[x], lo[x]);
+        }
+#pragma unroll
+        for (int n = 0; n < OT; n += 2) {
+          ldsm4t(B, v_s + (kk * 16 + (lane & 15)) * VQ + c0 + n * 8 + (lane >> 4) * 8);
+          mma16816(O[n], hi, B[0], B[1]);
+          mma16816(O[n + 1], hi, B[2], B[3]);
+          mma16816(O[n], lo, B[0], B[1]);
+          mma16816(O[n + 1], lo, B[2], B[3]);
+        }
+      }
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (size_t)(t0 + l0) * H * vd + (size_t)h * vd;
+#pragma unroll
+      for (int n = 0; n < OT; ++n) {
+        const int c = v0 + c0 + n * 8 + (lane & 3) * 2;    // (vdim is a multiple of 8: pairs are whole)
+        if (c < vd) {
+          if (i0 < n_tok) *reinterpret_cast<uint32_t*>(out + (size_t)i0 * H * vd + c) = f2_to_bf2(O[n][0], O[n][1]);
+          if (i0 + 8 < n_tok) *reinterpret_cast<uint32_t*>(out + (size_t)(i0 + 8) * H * vd + c) = f2_to_bf2(O[n][2], O[n][3]);
+        }
+      }
+    }
+
+    // the state behind the chunk
+    const float fs = pw[n_tok];
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      S[n][0] *= fs; S[n][1] *= fs; S[n][2] *= fs; S[n][3] *= fs;
+    }
+    const int m0 = (warp % RG) * 16, c0 = (warp / RG) * SC;
+#pragma unroll
+    for (int k0 = 0; k0 < kChunk; k0 += 16) {
+      uint32_t K[4], hi[4], mid[4], lo[4], B[4];
+      ldsm4t(K, k_s + (k0 + (lane & 7) + (lane >> 4) * 8) * QP + m0 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int j = k0 + (x >> 1) * 8 + (lane & 3) * 2;  // (keys beyond the chunk's end are zero)
+        const float2 k = bf2_to_f2(K[x]);
+        const float x0 = k.x * pw[max(n_tok - 1 - j, 0)], x1 = k.y * pw[max(n_tok - 2 - j, 0)];
+        hi[x] = f2_to_bf2(x0, x1);
+        const float2 g = bf2_to_f2(hi[x]);
+        split2(x0 - g.x, x1 - g.y, mid[x], lo[x]);
+      }
+#pragma unroll
+      for (int n = 0; n < NT; n += 2) {
+        ldsm4t(B, v_s + (k0 + (lane & 15)) * VQ + c0 + n * 8 + (lane >> 4) * 8);
+        mma16816(S[n], hi, B[0], B[1]);
+        mma16816(S[n + 1], hi, B[2], B[3]);
+        mma16816(S[n], mid, B[0], B[1]);
+        mma16816(S[n + 1], mid, B[2], B[3]);
+        mma16816(S[n], lo, B[0], B[1]);
+        mma16816(S[n + 1], lo, B[2], B[3]);
+      }
+    }
+  }
+
+  float* to = nullptr;
+  if (STATE_ONLY) to = sg.scratch + (((size_t)e * sg.segments + seg) * H + h) * d * vd;
+  else if (last) to = a.state + ((size_t)st.slot[e] * H + h) * d * vd;
+  if (!to) return;
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const int r = sr + (q >> 1) * 8, c = v0 + sc + n * 8 + (q & 1);
+      if (r < d && c < vd) to[(size_t)r * vd + c] = S[n][q];
+    }
+}
+
+// What the segments add -> the states in front of them, in place.
+__global__ void lightning_prefix_kernel(pace_step_t st, pace_lightning_args_t a, SegmentArgs sg) {
+  const int e = blockIdx.z, h = blockIdx.y, n = a.dim * a.vdim;
+  const int count = st.cu[e + 1] - st.cu[e];
+  const int used = (count + sg.seg_tokens - 1) / sg.seg_tokens;
+  const float f = powf(a.decay[h], (float)sg.seg_tokens);
+  const float* state = a.state + ((size_t)st.slot[e] * a.heads + h) * n;
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
+    float s = st.start[e] != 0 ? state[i] : 0.f;
+    for (int r = 0; r < used; ++r) {
+      float* p = sg.scratch + (((size_t)e * sg.segments + r) * a.heads + h) * n + i;
+      const float add = r + 1 < used ? *p : 0.f;
+      *p = s;
+      s = fmaf(f, s, add);
+    }
+  }
+}
+
+SegmentArgs plan_segments(int entries, int max_count, int heads, int vdim) {
+  SegmentArgs s;
+  s.scratch = nullptr;
+  const int blocks = entries * heads * ((vdim + 127) / 128);
+  int want = 2 * 148 / (blocks > 0 ? blocks : 1);
+  const int most = max_count / (4 * kChunk);               // a segment is worth its own blocks from four chunks on
+  if (want > most) want = most;
+  if (want < 1) want = 1;
+  s.seg_tokens = (max_count + want - 1) / want;
+  s.seg_tokens = (s.seg_tokens + kChunk - 1) / kChunk * kChunk;
+  s.segments = (max_count + s.seg_tokens - 1) / s.seg_tokens;
+  if (s.segments < 1) s.segments = 1;
+  return s;
+}
+
+template <int DP, int VP>
+int launch_chunked(const pace_step_t& st, const pace_lightning_args_t& a, const SegmentArgs& sg, cudaStream_t s) {
+  const size_t smem = Tiles<DP, VP>::bytes;
+  const dim3 grid((unsigned)((a.vdim + VP - 1) / VP), (unsigned)a.heads, (unsigned)(st.n_entries * sg.segments));
+  if (sg.segments > 1) {
+    PACE_CUDA_TRY(cudaFuncSetAttribute(lightning_chunk_kernel<DP, VP, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                       (int)smem));
+    lightning_chunk_kernel<DP, VP, true><<<grid, kThreads, smem, s>>>(st, a, sg);
+    PACE_LAUNCH_CHECK("lightning_chunk_kernel (states)");
+    const int blocks = (a.dim * a.vdim + 255) / 256;
+    lightning_prefix_kernel<<<dim3((unsigned)(blocks < 64 ? blocks : 64), (unsigned)a.heads, (unsigned)st.n_entries), 256, 0, s>>>(
+        st, a, sg);
+    PACE_LAUNCH_CHECK("lightning_prefix_kernel");
+  }
+  PACE_CUDA_TRY(cudaFuncSetAttribute(lightning_chunk_kernel<DP, VP, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                     (int)smem));
+  lightning_chunk_kernel<DP, VP, false><<<grid, kThreads, smem, s>>>(st, a, sg);
+  PACE_LAUNCH_CHECK("lightning_chunk_kernel");
+  return PACE_OK;
+}
+
+}  // namespace
+
+// bf16, head sizes that the tiles cover and 16-byte pieces; everything else is the token-by-token kernel's
+bool lightning_chunked_fits(const pace_lightning_args_t& a) {
+  return a.dtype == PACE_DTYPE_BF16 && a.dim <= 128 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.qkv_stride % 8 == 0 &&
+         aligned16(a.qkv) && aligned16(a.out);
+}
+
+int lightning_chunked(const pace_step_t& st, const pace_lightning_args_t& a, cudaStream_t s) {
+  SegmentArgs sg = plan_segments(st.n_entries, st.max_count, a.heads, a.vdim);
+  sg.scratch = a.workspace;
+  const uint64_t need = sizeof(float) * (uint64_t)st.n_entries * sg.segments * a.heads * a.dim * a.vdim;
+  if (sg.segments > 1 && (!a.workspace || a.workspace_bytes < need)) return PACE_ERR_INVALID;
+  if ((int64_t)st.n_entries * sg.segments > 65535) return PACE_ERR_UNSUPPORTED;
+  if (a.dim <= 64) return a.vdim <= 64 ? launch_chunked<64, 64>(st, a, sg, s) : launch_chunked<64, 128>(st, a, sg, s);
+  return a.vdim <= 64 ? launch_chunked<128, 64>(st, a, sg, s) : launch_chunked<128, 128>(st, a, sg, s);
+}
+
+}  // namespace pace
+
+extern "C" uint64_t pace_lightning_workspace_bytes(int32_t n_entries, int32_t max_count, int32_t heads, int32_t dim,
+                                                   int32_t vdim) {
+  if (n_entries <= 0 || max_count <= 0 || heads <= 0 || dim <= 0 || vdim <= 0) return 0;
+  const pace::SegmentArgs sg = pace::plan_segments(n_entries, max_count, heads, vdim);
+  return sg.segments > 1 ? sizeof(float) * (uint64_t)n_entries * sg.segments * heads * dim * vdim : 0;
+}

@@ -4,138 +4,200 @@
 #include "hybrid.cuh"
 
 namespace pace {
+bool lightning_chunked_fits(const pace_lightning_args_t& a);   // lightning.cu
+int lightning_chunked(const pace_step_t& st, const pace_lightning_args_t& a, cudaStream_t s);
+
 namespace {
 
 // ---------------------------------------------------------------------------
 // causal depthwise convolution
 // ---------------------------------------------------------------------------
-// Input of channel c at `back` tokens in front of local token l of an entry: from the step's rows, from the
-// slot's ring of newest inputs, or zero in front of the sequence.
-template <typename T>
-__device__ __forceinline__ float conv_input(const T* __restrict__ in, int64_t in_stride, const float* __restrict__ ring,
-                                            int n_taps, int channels, int t, int l, int pos, int back, int c) {
-  if (l >= back) return to_f<T>(in[(size_t)(t - back) * in_stride + c]);
-  if (pos < back) return 0.f;
-  return ring[(size_t)((pos - back) % n_taps) * channels + c];
-}
+// A thread takes V channels of kConvTokens consecutive rows: the taps are read once for all of them, a row's
+// inputs come from the cache after their first use.
+constexpr int kConvTokens = 4;
 
 template <typename T, int V>
-__global__ void causal_conv_kernel(pace_step_t st, const T* __restrict__ in, int64_t in_stride, const float* __restrict__ taps,
-                                   const float* __restrict__ bias, int n_taps, const float* __restrict__ conv_state,
-                                   T* __restrict__ out, int channels) {
+__global__ void __launch_bounds__(256)
+    causal_conv_kernel(pace_step_t st, const T* __restrict__ in, int64_t in_stride, const float* __restrict__ taps,
+                       const float* __restrict__ bias, int n_taps, const float* __restrict__ conv_state, T* __restrict__ out,
+                       int channels) {
   const int per = channels / V;
-  const size_t total = (size_t)st.n_tokens * per;
+  const size_t total = (size_t)((st.n_tokens + kConvTokens - 1) / kConvTokens) * per;
   for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
-    const int t = (int)(i / per), c = (int)(i % per) * V;
-    const int e = st.tok_entry[t], l = t - st.cu[e], pos = st.tok_pos[t];
-    float acc[V];
-    Vec<float, V>::load(bias + c, acc);
+    const int t0 = (int)(i / per) * kConvTokens, c = (int)(i % per) * V;
+    float acc[kConvTokens][V];
+    int local[kConvTokens], pos[kConvTokens];
+    const float* ring[kConvTokens];
+#pragma unroll
+    for (int r = 0; r < kConvTokens; ++r) {
+      const int t = min(t0 + r, st.n_tokens - 1), e = st.tok_entry[t];
+      local[r] = t - st.cu[e];
+      pos[r] = st.tok_pos[t];
+      ring[r] = conv_state + (size_t)st.slot[e] * n_taps * channels + c;
+      Vec<float, V>::load(bias + c, acc[r]);
+    }
     for (int j = 0; j < n_taps; ++j) {
       const int back = n_taps - 1 - j;
-      float x[V];
-      if (l >= back) {
-        Vec<T, V>::load(in + (size_t)(t - back) * in_stride + c, x);
-      } else if (pos >= back) {
-        Vec<float, V>::load(conv_state + ((size_t)st.slot[e] * n_taps + (pos - back) % n_taps) * channels + c, x);
-      } else {
-        continue;
-      }
+      float w[V];
+      Vec<float, V>::load(taps + (size_t)j * channels + c, w);
 #pragma unroll
-      for (int v = 0; v < V; ++v) acc[v] = fmaf(taps[(size_t)(c + v) * n_taps + j], x[v], acc[v]);
+      for (int r = 0; r < kConvTokens; ++r) {
+        const int t = min(t0 + r, st.n_tokens - 1);
+        float x[V];
+        if (local[r] >= back) Vec<T, V>::load(in + (size_t)(t - back) * in_stride + c, x);
+        else if (pos[r] >= back) Vec<float, V>::load(ring[r] + (size_t)((pos[r] - back) % n_taps) * channels, x);
+        else continue;                                     // in front of the sequence
+#pragma unroll
+        for (int v = 0; v < V; ++v) acc[r][v] = fmaf(w[v], x[v], acc[r][v]);
+      }
     }
-    Vec<T, V>::store(out + (size_t)t * channels + c, acc);
+#pragma unroll
+    for (int r = 0; r < kConvTokens; ++r)
+      if (t0 + r < st.n_tokens) Vec<T, V>::store(out + (size_t)(t0 + r) * channels + c, acc[r]);
   }
 }
 
 // ---------------------------------------------------------------------------
 // RG-LRU over any number of tokens: gates and convolution come from launches in front
 // ---------------------------------------------------------------------------
-constexpr int kSegs = 16, kSegTokens = 8, kTile = kSegs * kSegTokens;
+constexpr int kSegs = 16, kSegTokens = 4, kTile = kSegs * kSegTokens;
 
 // coefficients of S_t = a S_(t-1) + b for pre-activations of the two gates
 template <typename T>
 __device__ __forceinline__ void rglru_coefficients(float r_pre, float i_pre, float u, float decay_base, float& a, float& b) {
   const float log_a = decay_base * sigmoid_t<T>(r_pre);
   a = exp_t<T>(log_a);
-  b = sqrtf(one_minus_exp<T>(2.0f * log_a, a * a)) * sigmoid_t<T>(i_pre) * u;
+  b = sqrt_one_minus_exp<T>(2.0f * log_a, a * a) * sigmoid_t<T>(i_pre) * u;
 }
 
-// A block walks 32 channels of one entry in tiles of 128 tokens: warp = a segment of 8 tokens, lane = a
-// channel.  A thread composes its 8 steps into one affine map, the 16 maps of a channel meet in shared
-// memory, every thread then replays its 8 steps from the state in front of them.  The next tile's operands
-// are on their way meanwhile.
+// The blocks of a cluster walk 32 channels of one entry together: tiles of 64 tokens go round the cluster, in a
+// block warp = a segment of 4 tokens, lane = a channel.  A thread composes its 4 steps into one affine map; the
+// maps of a tile meet in shared memory, their products in the shared memory of every block of the cluster; then
+// each thread replays its 8 steps from the state in front of them.  The next tile's operands are on their way
+// meanwhile.  All blocks of a cluster take the same number of rounds.
+constexpr int kMaxCluster = 4;
+
 template <typename T>
-__global__ void __launch_bounds__(512)
+__global__ void __launch_bounds__(512, 2)
     rglru_scan_kernel(pace_step_t st, pace_rglru_args_t a) {
   __shared__ float2 maps[2][kSegs][32];
-  const int e = blockIdx.y, lane = threadIdx.x & 31, seg = threadIdx.x >> 5;
-  const int W = a.width, c = blockIdx.x * 32 + lane;
+  __shared__ float2 tiles_map[2][kMaxCluster][32];   // the round's tiles, written by the cluster's blocks
+  uint32_t rank, n_rank;
+  asm("mov.u32 %0, %%cluster_ctarank;" : "=r"(rank));
+  asm("mov.u32 %0, %%cluster_nctarank;" : "=r"(n_rank));
+  const int e = blockIdx.z, lane = threadIdx.x & 31, seg = threadIdx.x >> 5;
+  const int W = a.width, c = blockIdx.y * 32 + lane;
   const bool live = c < W;
   const int cc = live ? c : 0;
   const int bs = W / a.blocks, blk = cc / bs, in_blk = cc - blk * bs;
   const int t0 = st.cu[e], count = st.cu[e + 1] - t0, start = st.start[e], slot = st.slot[e];
-  const T* u = static_cast<const T*>(a.u) + cc;
-  const T* yx = static_cast<const T*>(a.yx) + cc;
-  const float* gr = a.gates + (size_t)blk * st.n_tokens * 2 * bs + in_blk;
-  T* out = static_cast<T*>(a.out) + cc;
+  const T* u = static_cast<const T*>(a.u) + (size_t)t0 * W + cc;
+  const T* yx = static_cast<const T*>(a.yx) + (size_t)t0 * a.yx_stride + cc;
+  const float* gr = a.gates + ((size_t)blk * st.n_tokens + t0) * 2 * bs + in_blk;
+  T* out = static_cast<T*>(a.out) + (size_t)t0 * W + cc;
   const float rb = a.ra_bias[cc], ib = a.ri_bias[cc], base = a.decay_base[cc];
   float* state = a.state + (size_t)slot * W + cc;
   float carry = start == 0 ? 0.f : *state;
 
-  float g0[kSegTokens], g1[kSegTokens], uu[kSegTokens], yy[kSegTokens];
-  auto fetch = [&](int tile) {
+  float g0[kSegTokens], g1[kSegTokens];
+  T uu[kSegTokens], yy[kSegTokens];
+  auto fetch = [&](int l0) {
 #pragma unroll
     for (int j = 0; j < kSegTokens; ++j) {
-      const int l = tile * kTile + seg * kSegTokens + j;
-      if (l < count) {
-        const size_t t = (size_t)(t0 + l);
-        g0[j] = gr[t * 2 * bs];
-        g1[j] = gr[t * 2 * bs + bs];
-        uu[j] = to_f<T>(u[t * W]);
-        yy[j] = to_f<T>(yx[t * a.yx_stride]);
-      }
+      const int l = min(l0 + j, count - 1);          // (rows behind the end are read but not used)
+      g0[j] = gr[(size_t)l * 2 * bs];
+      g1[j] = gr[(size_t)l * 2 * bs + bs];
+      uu[j] = u[(size_t)l * W];
+      yy[j] = yx[(size_t)l * a.yx_stride];
     }
   };
-  fetch(0);
-  const int tiles = (count + kTile - 1) / kTile;
-  for (int tile = 0; tile < tiles; ++tile) {
-    float ca[kSegTokens], cb[kSegTokens], y[kSegTokens], A = 1.f, B = 0.f;
-    const int l0 = tile * kTile + seg * kSegTokens;
+  const int stride = kTile * (int)n_rank;
+  int l0 = (int)rank * kTile + seg * kSegTokens;
+  fetch(l0);
+  const int rounds = (count + stride - 1) / stride;
+  if (n_rank > 1) {                                  // every block of the cluster runs before anyone writes into it
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+  }
+  for (int round = 0; round < rounds; ++round, l0 += stride) {
+    float ca[kSegTokens], cb[kSegTokens], A = 1.f, B = 0.f;
+    T y[kSegTokens];
 #pragma unroll
     for (int j = 0; j < kSegTokens; ++j) {
-      if (l0 + j < count) {
-        rglru_coefficients<T>(g0[j] + rb, g1[j] + ib, uu[j], base, ca[j], cb[j]);
-        y[j] = yy[j];
-        A *= ca[j];
-        B = fmaf(ca[j], B, cb[j]);
-      }
+      rglru_coefficients<T>(g0[j] + rb, g1[j] + ib, to_f<T>(uu[j]), base, ca[j], cb[j]);
+      if (l0 + j >= count) ca[j] = 1.f, cb[j] = 0.f;
+      y[j] = yy[j];
+      A *= ca[j];
+      B = fmaf(ca[j], B, cb[j]);
     }
-    if (tile + 1 < tiles) fetch(tile + 1);
-    maps[tile & 1][seg][lane] = make_float2(A, B);
+    if (round + 1 < rounds) fetch(l0 + stride);
+    const int buf = round & 1;
+    maps[buf][seg][lane] = make_float2(A, B);
     __syncthreads();
-    float s = carry, mine = 0.f;
+    // the map of the segments in front, and the tile's
+    float fa = 1.f, fb = 0.f, ma = 1.f, mb = 0.f;
 #pragma unroll
     for (int k = 0; k < kSegs; ++k) {
-      if (k == seg) mine = s;
-      const float2 m = maps[tile & 1][k][lane];
-      s = fmaf(m.x, s, m.y);
+      if (k == seg) ma = fa, mb = fb;
+      const float2 m = maps[buf][k][lane];
+      fb = fmaf(m.x, fb, m.y);
+      fa *= m.x;
     }
-    carry = s;
+    float mine;
+    if (n_rank == 1) {
+      mine = fmaf(ma, carry, mb);
+      carry = fmaf(fa, carry, fb);
+    } else {
+      if (seg < (int)n_rank) {                       // warp k sends the tile's map to block k
+        uint32_t addr;
+        asm volatile("mapa.shared::cluster.u32 %0, %1, %2;"
+                     : "=r"(addr) : "r"(smem_u32(&tiles_map[buf][rank][lane])), "r"((uint32_t)seg));
+        asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(addr), "f"(fa), "f"(fb) : "memory");
+      }
+      asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+      asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+      float s = carry;
+      for (int k = 0; k < (int)n_rank; ++k) {
+        if (k == (int)rank) mine = fmaf(ma, s, mb);
+        const float2 m = tiles_map[buf][k][lane];
+        s = fmaf(m.x, s, m.y);
+      }
+      carry = s;
+    }
 #pragma unroll
     for (int j = 0; j < kSegTokens; ++j) {
-      if (l0 + j < count) {
-        mine = fmaf(ca[j], mine, cb[j]);
-        if (live) out[(size_t)(t0 + l0 + j) * W] = from_f<T>(mine * gelu_tanh_t<T>(y[j]));
-      }
+      mine = fmaf(ca[j], mine, cb[j]);
+      if (l0 + j < count && live) out[(size_t)(l0 + j) * W] = from_f<T>(mine * gelu_tanh_t<T>(to_f<T>(y[j])));
     }
   }
-  if (!live) return;
+  // (a block's last sends were received in front of the last barrier: nobody writes into a block that has left)
+  if (!live || rank != 0) return;
   if (seg == 0) *state = carry;
   for (int j = seg; j < a.n_taps && j < count; j += kSegs) {
     const int l = count - 1 - j;
-    a.conv_state[((size_t)slot * a.n_taps + (start + l) % a.n_taps) * W + c] =
-        to_f<T>(yx[(size_t)(t0 + l) * a.yx_stride + W]);
+    a.conv_state[((size_t)slot * a.n_taps + (start + l) % a.n_taps) * W + c] = to_f<T>(yx[(size_t)l * a.yx_stride + W]);
   }
+}
+
+template <typename T>
+int launch_rglru_scan(const pace_step_t& st, const pace_rglru_args_t& a, cudaStream_t s) {
+  const int groups = (a.width + 31) / 32;
+  int cluster = 1;                                   // blocks that share an entry's tiles, while the GPU has room for them
+  while (cluster < kMaxCluster && cluster * 2 * kTile <= st.max_count && (int64_t)groups * st.n_entries * cluster < 296)
+    cluster *= 2;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3((unsigned)cluster, (unsigned)groups, (unsigned)st.n_entries);
+  cfg.blockDim = dim3(32 * kSegs);
+  cfg.stream = s;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = (unsigned)cluster;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = 1;
+  PACE_CUDA_TRY(cudaLaunchKernelEx(&cfg, rglru_scan_kernel<T>, st, a));
+  PACE_LAUNCH_CHECK("rglru_scan_kernel");
+  return PACE_OK;
 }
 
 // ---------------------------------------------------------------------------
@@ -148,15 +210,6 @@ __device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
-// two consecutive weights of a row of `n`, zero behind its end; rows of odd length are not word aligned
-__device__ __forceinline__ uint32_t load_pair(const __nv_bfloat16* row, int k, int n, bool even) {
-  if (even) return k < n ? *reinterpret_cast<const uint32_t*>(row + k) : 0u;
-  uint32_t lo = 0, hi = 0;
-  if (k < n) lo = *reinterpret_cast<const uint16_t*>(row + k);
-  if (k + 1 < n) hi = *reinterpret_cast<const uint16_t*>(row + k + 1);
-  return lo | (hi << 16);
 }
 
 template <typename T>
@@ -173,69 +226,91 @@ __device__ __forceinline__ void rglru_finish(const pace_step_t& st, const pace_r
   static_cast<T*>(a.out)[(size_t)st.cu[e] * W + c] = from_f<T>(S * gelu_tanh_t<T>(to_f<T>(row[c])));
 }
 
-// Block (slice, batch tile): 32 output channels of one gate block for 32 entries.  bf16: warp w multiplies
-// entries [16 (w / 4), +16) with channels [8 (w % 4), +8) of both gates on the tensor cores (fp32
-// accumulators are the pre-activations); fp32: one thread per (entry, channel).
-template <typename T>
+// Block (slice, batch tile): 32 output channels of one gate block for 32 entries.  The slice's gate weights and the
+// convolved inputs of the whole gate block go to shared memory (V elements per access), then bf16: warp w multiplies
+// entries [16 (w / 4), +16) with channels [8 (w % 4), +8) of both gates on the tensor cores (fp32 accumulators
+// are the pre-activations); fp32: one thread per (entry, channel).
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
     rglru_step_kernel(pace_step_t st, pace_rglru_args_t a, int slices, int ld) {
   extern __shared__ __align__(16) char smem_raw[];
+  __shared__ int row_of[kStepEntries], pos_of[kStepEntries], slot_of[kStepEntries];
   T* us = reinterpret_cast<T*>(smem_raw);  // [kStepEntries][ld]
+  T* ws = us + kStepEntries * ld;          // [2][kStepChannels][ld]
   const int W = a.width, bs = W / a.blocks;
   const int blk = blockIdx.x / slices, o0 = (blockIdx.x % slices) * kStepChannels;
-  const int e0 = blockIdx.y * kStepEntries, E = st.n_entries;
-  const T* x0 = static_cast<const T*>(a.yx) + W;
-  for (int i = threadIdx.x; i < kStepEntries * ld; i += 256) {
-    const int r = i / ld, k = i - r * ld, e = e0 + r, c = blk * bs + k;
-    float acc = 0.f;
-    if (e < E && k < bs) {
-      acc = a.conv_bias[c];
-      const int pos = st.start[e], t = st.cu[e];
-      const float* ring = a.conv_state + (size_t)st.slot[e] * a.n_taps * W;
-      for (int j = 0; j < a.n_taps; ++j)
-        acc = fmaf(a.taps[(size_t)c * a.n_taps + j],
-                   conv_input<T>(x0, a.yx_stride, ring, a.n_taps, W, t, 0, pos, a.n_taps - 1 - j, c), acc);
-    }
-    us[i] = from_f<T>(acc);
+  const int e0 = blockIdx.y * kStepEntries, n_e = min(kStepEntries, st.n_entries - e0);
+  const int lv = ld / V;                   // vectors of a shared row
+  const T* wg = static_cast<const T*>(a.gate_w) + (size_t)blk * 2 * bs * bs;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < 2 * kStepChannels * lv; i += 256) {
+    const int r = i / lv, k = (i - r * lv) * V, o = o0 + (r & (kStepChannels - 1));
+    float x[V];
+#pragma unroll
+    for (int v = 0; v < V; ++v) x[v] = 0.f;
+    if (o < bs && k < bs) Vec<T, V>::load(wg + ((size_t)(r / kStepChannels) * bs + o) * bs + k, x);
+    Vec<T, V>::store(ws + r * ld + k, x);
+  }
+  if (threadIdx.x < n_e) {
+    row_of[threadIdx.x] = st.cu[e0 + threadIdx.x];
+    pos_of[threadIdx.x] = st.start[e0 + threadIdx.x];
+    slot_of[threadIdx.x] = st.slot[e0 + threadIdx.x];
   }
   __syncthreads();
-  const T* wr = static_cast<const T*>(a.gate_w) + (size_t)blk * 2 * bs * bs;
-  const T* wi = wr + (size_t)bs * bs;
+  const T* x0 = static_cast<const T*>(a.yx) + W;
+#pragma unroll 2
+  for (int i = threadIdx.x; i < kStepEntries * lv; i += 256) {
+    const int r = i / lv, k = (i - r * lv) * V, c = blk * bs + k;
+    float acc[V];
+#pragma unroll
+    for (int v = 0; v < V; ++v) acc[v] = 0.f;
+    if (r < n_e && k < bs) {
+      const int pos = pos_of[r];
+      const float* ring = a.conv_state + (size_t)slot_of[r] * a.n_taps * W + c;
+      Vec<float, V>::load(a.conv_bias + c, acc);
+      for (int j = 0; j < a.n_taps; ++j) {
+        const int back = a.n_taps - 1 - j;
+        if (pos < back) continue;
+        float x[V], w[V];
+        if (back == 0) Vec<T, V>::load(x0 + (size_t)row_of[r] * a.yx_stride + c, x);
+        else Vec<float, V>::load(ring + (size_t)((pos - back) % a.n_taps) * W, x);
+        Vec<float, V>::load(a.taps + (size_t)j * W + c, w);
+#pragma unroll
+        for (int v = 0; v < V; ++v) acc[v] = fmaf(w[v], x[v], acc[v]);
+      }
+    }
+    Vec<T, V>::store(us + r * ld + k, acc);
+  }
+  __syncthreads();
   if constexpr (sizeof(T) == 2) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
     const int m0 = (warp >> 2) * 16;
-    if (e0 + m0 >= E) return;
-    const int n = o0 + (warp & 3) * 8 + gid;  // the channel whose weights this lane feeds
-    const bool even = (bs & 1) == 0;
-    const __nv_bfloat16* rr = reinterpret_cast<const __nv_bfloat16*>(wr) + (size_t)(n < bs ? n : 0) * bs;
-    const __nv_bfloat16* ri = reinterpret_cast<const __nv_bfloat16*>(wi) + (size_t)(n < bs ? n : 0) * bs;
+    if (m0 >= n_e) return;
     const __nv_bfloat16* up = reinterpret_cast<const __nv_bfloat16*>(us) + (m0 + gid) * ld + tig * 2;
+    const __nv_bfloat16* rp = reinterpret_cast<const __nv_bfloat16*>(ws) + ((warp & 3) * 8 + gid) * ld + tig * 2;
+    const __nv_bfloat16* ip = rp + kStepChannels * ld;
+    auto pair = [](const __nv_bfloat16* p) { return *reinterpret_cast<const uint32_t*>(p); };
     float cr[4] = {0.f, 0.f, 0.f, 0.f}, ci[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll 4
     for (int k = 0; k < bs; k += 16) {
-      uint32_t A[4];
-      A[0] = *reinterpret_cast<const uint32_t*>(up + k);
-      A[1] = *reinterpret_cast<const uint32_t*>(up + 8 * ld + k);
-      A[2] = *reinterpret_cast<const uint32_t*>(up + k + 8);
-      A[3] = *reinterpret_cast<const uint32_t*>(up + 8 * ld + k + 8);
-      const int kk = k + tig * 2;
-      mma_bf16(cr, A, load_pair(rr, kk, bs, even), load_pair(rr, kk + 8, bs, even));
-      mma_bf16(ci, A, load_pair(ri, kk, bs, even), load_pair(ri, kk + 8, bs, even));
+      const uint32_t A[4] = {pair(up + k), pair(up + 8 * ld + k), pair(up + k + 8), pair(up + 8 * ld + k + 8)};
+      mma_bf16(cr, A, pair(rp + k), pair(rp + k + 8));
+      mma_bf16(ci, A, pair(ip + k), pair(ip + k + 8));
     }
 #pragma unroll
     for (int q = 0; q < 4; ++q) {
       const int r = m0 + gid + (q >> 1) * 8, o = o0 + (warp & 3) * 8 + tig * 2 + (q & 1);
-      if (e0 + r < E && o < bs) rglru_finish<T>(st, a, e0 + r, blk * bs + o, cr[q], ci[q], to_f<T>(us[r * ld + o]));
+      if (r < n_e && o < bs) rglru_finish<T>(st, a, e0 + r, blk * bs + o, cr[q], ci[q], to_f<T>(us[r * ld + o]));
     }
   } else {
     for (int i = threadIdx.x; i < kStepEntries * kStepChannels; i += 256) {
-      const int r = i / kStepChannels, o = o0 + i % kStepChannels;
-      if (e0 + r >= E || o >= bs) continue;
+      const int r = i / kStepChannels, oo = i % kStepChannels, o = o0 + oo;
+      if (r >= n_e || o >= bs) continue;
       float sr = 0.f, si = 0.f;
       for (int k = 0; k < bs; ++k) {
         const float x = to_f<T>(us[r * ld + k]);
-        sr = fmaf(to_f<T>(wr[(size_t)o * bs + k]), x, sr);
-        si = fmaf(to_f<T>(wi[(size_t)o * bs + k]), x, si);
+        sr = fmaf(to_f<T>(ws[oo * ld + k]), x, sr);
+        si = fmaf(to_f<T>(ws[(kStepChannels + oo) * ld + k]), x, si);
       }
       rglru_finish<T>(st, a, e0 + r, blk * bs + o, sr, si, to_f<T>(us[r * ld + o]));
     }
@@ -404,8 +479,8 @@ template <typename T>
 int causal_conv_t(const pace_step_t& st, const void* in, int64_t is, const float* taps, const float* bias, int n_taps,
                   const float* cs, void* out, int channels, cudaStream_t s) {
   constexpr int V = 16 / sizeof(T);
-  const bool vec = channels % V == 0 && is % V == 0 && aligned16(in) && aligned16(out) && aligned16(bias) && aligned16(cs);
-  const size_t groups = (size_t)st.n_tokens * (channels / (vec ? V : 1));
+  const bool vec = channels % V == 0 && is % V == 0 && aligned16(in) && aligned16(out) && aligned16(bias) && aligned16(cs) && aligned16(taps);
+  const size_t groups = (size_t)((st.n_tokens + kConvTokens - 1) / kConvTokens) * (channels / (vec ? V : 1));
   size_t blocks = (groups + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   if (vec)
@@ -416,17 +491,25 @@ int causal_conv_t(const pace_step_t& st, const void* in, int64_t is, const float
   return PACE_OK;
 }
 
+template <typename T, int V>
+int launch_rglru_step(const pace_step_t& st, const pace_rglru_args_t& a, int slices, int ld, size_t smem, cudaStream_t s) {
+  PACE_CUDA_TRY(cudaFuncSetAttribute(rglru_step_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  const dim3 grid((unsigned)(a.blocks * slices), (unsigned)((st.n_entries + kStepEntries - 1) / kStepEntries));
+  rglru_step_kernel<T, V><<<grid, 256, smem, s>>>(st, a, slices, ld);
+  PACE_LAUNCH_CHECK("rglru_step_kernel");
+  return PACE_OK;
+}
+
 template <typename T>
 int rglru_step_t(const pace_step_t& st, const pace_rglru_args_t& a, cudaStream_t s) {
   const int bs = a.width / a.blocks, slices = (bs + kStepChannels - 1) / kStepChannels;
-  const int ld = sizeof(T) == 2 ? (bs + 15) / 16 * 16 + 8 : bs;
-  const size_t smem = (size_t)kStepEntries * ld * sizeof(T);
+  const int ld = (bs + 15) / 16 * 16 + 16 / (int)sizeof(T);   // whole k steps of the tensor cores, rows 16 bytes apart
+  const size_t smem = (size_t)(kStepEntries + 2 * kStepChannels) * ld * sizeof(T);
   if (smem > 200 * 1024) return PACE_ERR_UNSUPPORTED;
-  PACE_CUDA_TRY(cudaFuncSetAttribute(rglru_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  const dim3 grid((unsigned)(a.blocks * slices), (unsigned)((st.n_entries + kStepEntries - 1) / kStepEntries));
-  rglru_step_kernel<T><<<grid, 256, smem, s>>>(st, a, slices, ld);
-  PACE_LAUNCH_CHECK("rglru_step_kernel");
-  return PACE_OK;
+  constexpr int V = 16 / sizeof(T);
+  const bool vec = bs % V == 0 && a.yx_stride % V == 0 && aligned16(a.yx) && aligned16(a.gate_w) && aligned16(a.taps) &&
+                   aligned16(a.conv_bias) && aligned16(a.conv_state);
+  return vec ? launch_rglru_step<T, V>(st, a, slices, ld, smem, s) : launch_rglru_step<T, 1>(st, a, slices, ld, smem, s);
 }
 
 bool dtype_ok(int dtype) { return dtype == PACE_DTYPE_BF16 || dtype == PACE_DTYPE_FP32; }
@@ -461,15 +544,10 @@ int pace_causal_conv(const pace_step_t* st, const void* in, int64_t is, const fl
 int pace_rglru_scan(const pace_step_t* st, const pace_rglru_args_t* a, void* stream) {
   if (!rglru_ok(st, a) || !a->u || !a->gates) return PACE_ERR_INVALID;
   if (st->n_tokens == 0) return PACE_OK;
-  if (st->n_entries > 65535) return PACE_ERR_UNSUPPORTED;
+  if (st->n_entries > 65535 || a->width > 32 * 65535) return PACE_ERR_UNSUPPORTED;
   PACE_PROFILE("rglru_scan", stream, "entries=%d tokens=%d width=%d", st->n_entries, st->n_tokens, a->width);
-  const dim3 grid((unsigned)((a->width + 31) / 32), (unsigned)st->n_entries);
-  if (a->dtype == PACE_DTYPE_BF16)
-    rglru_scan_kernel<__nv_bfloat16><<<grid, 32 * kSegs, 0, (cudaStream_t)stream>>>(*st, *a);
-  else
-    rglru_scan_kernel<float><<<grid, 32 * kSegs, 0, (cudaStream_t)stream>>>(*st, *a);
-  PACE_LAUNCH_CHECK("rglru_scan_kernel");
-  return PACE_OK;
+  return a->dtype == PACE_DTYPE_BF16 ? launch_rglru_scan<__nv_bfloat16>(*st, *a, (cudaStream_t)stream)
+                                     : launch_rglru_scan<float>(*st, *a, (cudaStream_t)stream);
 }
 
 int pace_rglru_step(const pace_step_t* st, const pace_rglru_args_t* a, void* stream) {
@@ -485,6 +563,7 @@ int pace_lightning_prefill(const pace_step_t* st, const pace_lightning_args_t* a
   if (st->n_tokens == 0) return PACE_OK;
   if (a->dim > 512 || a->heads > 65535 || st->n_entries > 65535) return PACE_ERR_UNSUPPORTED;
   PACE_PROFILE("lightning_prefill", stream, "entries=%d tokens=%d heads=%d", st->n_entries, st->n_tokens, a->heads);
+  if (lightning_chunked_fits(*a)) return lightning_chunked(*st, *a, (cudaStream_t)stream);
   return a->dtype == PACE_DTYPE_BF16 ? lightning_seq<__nv_bfloat16>(*st, *a, (cudaStream_t)stream)
                                      : lightning_seq<float>(*st, *a, (cudaStream_t)stream);
 }

@@ -94,7 +94,7 @@ def rglru(step: Step, yx: torch.Tensor, gate_w: torch.Tensor, taps: torch.Tensor
     T, W = yx.shape[0], yx.shape[1] // 2
     blocks, n = gate_w.shape[0], gate_w.shape[2]
     out = torch.empty(T, W, dtype=yx.dtype, device=yx.device)
-    if step.decode_only and n <= 2048:
+    if step.decode_only and 96 * (n + 32) * yx.element_size() <= 200 * 1024:      # what the launch keeps in shared memory
         _OPS.rglru_step(step.handle, yx, gate_w, taps, conv_bias, ra_bias, ri_bias, decay_base, state, conv_state, out, blocks)
         return out
     u = torch.empty(T, W, dtype=yx.dtype, device=yx.device)

@@ -1058,7 +1058,7 @@ def hybrid_kernels(size: str, dev):
         qn, kn = vec(nq), vec(nk)
         yx = [rnd(T, 2 * W) for _ in range(N)]
         gw = [rnd(nb, 2, m, m) * m ** -0.5 for _ in range(N)]
-        taps, cb, ra, ri, base = rnd(W, 4, dtype=torch.float32), vec(W), vec(W), vec(W), -vec(W).abs()
+        taps, cb, ra, ri, base = rnd(4, W, dtype=torch.float32), vec(W), vec(W), vec(W), -vec(W).abs()
         lq = [rnd(T, 4 * LH * D) for _ in range(N)]
         decay = torch.linspace(0.9, 0.999, LH, device=dev)
         lo = [rnd(T, LH * D) for _ in range(N)]

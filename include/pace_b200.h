@@ -468,7 +468,7 @@ int pace_norm_gate(const void* o, const float* w, const void* gate, int64_t gate
 /* x = relu(x)^2 in place, n elements. */
 int pace_relu_squared(void* x, int64_t n, int32_t dtype, void* stream);
 
-/* Causal depthwise convolution: out[t][c] = bias[c] + sum_j taps[c][j] in[c](pos - (n_taps - 1) + j), zeros
+/* Causal depthwise convolution: out[t][c] = bias[c] + sum_j taps[j][c] in[c](pos - (n_taps - 1) + j), zeros
  * in front of the sequence.  conv_state fp32 [slots][n_taps][channels] holds each slot's newest inputs in row
  * position % n_taps (a row is overwritten only when no later token needs it).  This entry point reads it;
  * the recurrence behind it stores the new inputs. */
@@ -491,7 +491,7 @@ typedef struct {
   const void* u;          /* scan only */
   const float* gates;     /* scan only */
   const void* gate_w;     /* step only */
-  const float* taps;      /* step only: fp32 [width][n_taps] */
+  const float* taps;      /* step only: fp32 [n_taps][width] */
   const float* conv_bias; /* step only */
   const float* ra_bias;
   const float* ri_bias;
@@ -508,15 +508,20 @@ int pace_rglru_step(const pace_step_t* step, const pace_rglru_args_t* a, void* s
  *     S_t = decay S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t.
  * qkv dtype [n_tokens][qkv_stride]: q (heads x dim), k (heads x dim), v (heads x vdim).  state fp32
  * [slots][heads][dim][vdim].  out dtype [n_tokens][heads x vdim].  dim <= 512 (vdim any).
- * pace_lightning_step: one token per entry; pace_lightning_prefill: any counts. */
+ * pace_lightning_step: one token per entry; pace_lightning_prefill: any counts (bf16 with dim <= 128 and sizes that
+ * are multiples of 8: chunks of 64 tokens on the tensor cores; otherwise token by token). */
 typedef struct {
   const void* qkv;
   int64_t qkv_stride;
   const float* decay;     /* fp32 [heads] */
   float* state;
   void* out;
+  float* workspace;       /* prefill: pace_lightning_workspace_bytes() of scratch, any content */
+  uint64_t workspace_bytes;
   int32_t heads, dim, vdim, dtype;
 } pace_lightning_args_t;
+/* Scratch of a prefill (0: none).  Long sequences are cut into segments that run side by side. */
+uint64_t pace_lightning_workspace_bytes(int32_t n_entries, int32_t max_count, int32_t heads, int32_t dim, int32_t vdim);
 int pace_lightning_prefill(const pace_step_t* step, const pace_lightning_args_t* a, void* stream);
 int pace_lightning_step(const pace_step_t* step, const pace_lightning_args_t* a, void* stream);
 

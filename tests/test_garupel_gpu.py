@@ -229,7 +229,7 @@ def test_gated_recurrence(dtype, width, blocks, taps):
         want.append(S * ref.gelu_tanh(yx[t, :width].double()))
     want = torch.stack(want)
     base = (-8 * torch.nn.functional.softplus(lam)).float()
-    args = [z.to(DEV) for z in (gw, tp, cb, ra, ri, base)]
+    args = [z.to(DEV) for z in (gw, tp.t().contiguous(), cb, ra, ri, base)]
     cache = HybridCacheManager([StateSpec((("S", (width,)), ("conv", (taps, width))))], 3, 64, 4096, dtype, DEV)
     for a in cache[0].arrays.values():
         a.fill_(float("nan"))
