@@ -77,14 +77,16 @@ template <> struct Vec<__nv_bfloat16, 8> {
 
 // fp32 with a few ulp of error.  T names the activation type of the caller: fp32 models take the library's
 // exp and divide, bf16 models the hardware's approximate ones (relative error about 1e-6).
-template <typename T> __device__ __forceinline__ float exp_t(float x) { return __expf(x); }
+template <typename T> __device__ __forceinline__ float exp_t(float x) { return fast_exp2(x * kLog2e); }
 template <> __device__ __forceinline__ float exp_t<float>(float x) { return expf(x); }
-template <typename T> __device__ __forceinline__ float div_t(float a, float b) { return __fdividef(a, b); }
-template <> __device__ __forceinline__ float div_t<float>(float a, float b) { return a / b; }
-// sigmoid(x) = 1 / (1 + e^-x); the exponent is clamped so that the approximate divide never sees infinity
-template <typename T> __device__ __forceinline__ float sigmoid_t(float x) {
-  return div_t<T>(1.0f, 1.0f + exp_t<T>(fminf(-x, 80.0f)));
+template <typename T> __device__ __forceinline__ float rcp_t(float x) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
 }
+template <> __device__ __forceinline__ float rcp_t<float>(float x) { return 1.0f / x; }
+// sigmoid(x) = 1 / (1 + e^-x)   (1 / infinity = 0 at the far end)
+template <typename T> __device__ __forceinline__ float sigmoid_t(float x) { return rcp_t<T>(1.0f + exp_t<T>(-x)); }
 template <typename T> __device__ __forceinline__ float silu_t(float x) { return x * sigmoid_t<T>(x); }
 // 0.5 z (1 + tanh w) = z sigmoid(2 w)
 template <typename T> __device__ __forceinline__ float gelu_tanh_t(float z) {
@@ -96,7 +98,7 @@ template <typename T> __device__ __forceinline__ float sqrt_one_minus_exp(float 
   // |x| < 1/16: the first term left out, x^4 / 120, is below 2e-7; the difference has lost four bits at most
   const float s = -x * fmaf(x * (1.0f / 2), fmaf(x * (1.0f / 3), fmaf(x, 1.0f / 4, 1.0f), 1.0f), 1.0f);
   float r;
-  asm("sqrt.approx.f32 %0, %1;" : "=f"(r) : "f"(x > -0.0625f ? s : 1.0f - exp_x));
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x > -0.0625f ? s : 1.0f - exp_x));
   return r;
 }
 template <> __device__ __forceinline__ float sqrt_one_minus_exp<float>(float x, float exp_x) {

@@ -192,6 +192,105 @@ __global__ void append_norm_kernel(pace_step_t st, PageRows pg, pace_append_norm
   }
 }
 
+// The same for rows that fit in registers (ITEMS vectors of V elements per thread): one pass over the projection row,
+// one reduction for both sums.
+template <typename T, int V, int ITEMS>
+__global__ void __launch_bounds__(512) append_norm_regs_kernel(pace_step_t st, PageRows pg, pace_append_norm_args_t a, int row) {
+  __shared__ float2 red[16];
+  const int t = blockIdx.x, tid = threadIdx.x;
+  const int H = a.n_q_heads, G = pg.n_kv_heads, d = a.dim, vd = a.vdim;
+  const int nq = H * d, nk = G * d, n = nq + nk + G * vd;
+  const T* src = static_cast<const T*>(a.qkv) + (size_t)t * a.qkv_stride;
+  uint4 raw[ITEMS];
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * blockDim.x + tid) * V;
+    if (c < n) raw[i] = *reinterpret_cast<const uint4*>(src + c);
+  }
+  const int pos = st.tok_pos[t], slot = st.slot[st.tok_entry[t]];
+  const size_t q_row = (size_t)st.q_row[t];
+  const int lp = pos / pg.page_tokens;
+  int page = -1;
+  if (slot >= 0 && slot < pg.max_seqs && lp < pg.max_pages_per_seq)
+    page = pg.block_table[(size_t)slot * pg.max_pages_per_seq + lp];
+  float2 ss = make_float2(0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * blockDim.x + tid) * V;
+    if (c < nq + nk) {
+      float x[V], s = 0.f;
+      Vec<T, V>::load(reinterpret_cast<const T*>(&raw[i]), x);
+#pragma unroll
+      for (int j = 0; j < V; ++j) s = fmaf(x[j], x[j], s);
+      if (c < nq) ss.x += s; else ss.y += s;
+    }
+  }
+#pragma unroll
+  for (int o = 16; o; o >>= 1) {
+    ss.x += __shfl_xor_sync(0xffffffffu, ss.x, o);
+    ss.y += __shfl_xor_sync(0xffffffffu, ss.y, o);
+  }
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  ss = make_float2(0.f, 0.f);
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) {
+    ss.x += red[w].x;
+    ss.y += red[w].y;
+  }
+  float temp = a.q_mul;
+  if (a.temp_coef != 0.f) temp *= 1.0f + a.temp_coef * logf((float)(floor((double)(pos + 1) / a.temp_every) + 1.0));
+  const float fq = (a.q_norm ? 1.0f / sqrtf(ss.x / (float)nq + a.eps) : 1.f) * temp;
+  const float fk = a.k_norm ? 1.0f / sqrtf(ss.y / (float)nk + a.eps) : 1.f;
+  if (page < 0 || page >= pg.n_pages) {
+    if (tid == 0) raise_status(pg.status, PACE_DEV_BAD_INDEX);
+    page = -1;
+  }
+  T* qo = static_cast<T*>(a.q_out) + q_row * H * row;
+  const size_t in_page = (size_t)pos - (size_t)lp * pg.page_tokens;
+  auto page_row = [&](bool is_v, int g) {
+    return reinterpret_cast<T*>(is_v ? pg.v : pg.k) + (((size_t)page * G + g) * pg.page_tokens + in_page) * row;
+  };
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * blockDim.x + tid) * V;
+    if (c >= n) continue;
+    if (c >= nq + nk) {                                    // values go as they are
+      const int o = c - nq - nk, g = o / vd;
+      if (page >= 0) *reinterpret_cast<uint4*>(page_row(true, g) + (o - g * vd)) = raw[i];
+      continue;
+    }
+    const bool is_q = c < nq;
+    const float* w = is_q ? (a.q_norm ? a.q_norm + c : nullptr) : (a.k_norm ? a.k_norm + c - nq : nullptr);
+    const float f = is_q ? fq : fk;
+    float x[V];
+    Vec<T, V>::load(reinterpret_cast<const T*>(&raw[i]), x);
+    if (w) {
+      float wv[V];
+      Vec<float, V>::load(w, wv);
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] *= f * wv[j];
+    } else {
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] *= f;
+    }
+    const int o = is_q ? c : c - nq, h = o / d;
+    if (is_q) Vec<T, V>::store(qo + (size_t)h * row + (o - h * d), x);
+    else if (page >= 0) Vec<T, V>::store(page_row(false, h) + (o - h * d), x);
+  }
+  // what a row has beyond its head size
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  const int pd = (row - d) / V, pv = (row - vd) / V, heads_d = H + (page >= 0 ? G : 0);
+  for (int i = tid; i < heads_d * pd; i += blockDim.x) {
+    const int h = i / pd, c = d + (i - h * pd) * V;
+    *reinterpret_cast<uint4*>((h < H ? qo + (size_t)h * row : page_row(false, h - H)) + c) = zero;
+  }
+  if (page >= 0)
+    for (int i = tid; i < G * pv; i += blockDim.x) {
+      const int g = i / pv;
+      *reinterpret_cast<uint4*>(page_row(true, g) + vd + (i - g * pv) * V) = zero;
+    }
+}
+
 template <typename T>
 int launch_append_norm(const pace_kv_pool_t* p, int layer, const pace_step_t& st, const pace_append_norm_args_t& a,
                        cudaStream_t s) {
@@ -213,10 +312,18 @@ int launch_append_norm(const pace_kv_pool_t* p, int layer, const pace_step_t& st
                    aligned16(a.q_out) && (!a.q_norm || aligned16(a.q_norm)) && (!a.k_norm || aligned16(a.k_norm));
   const int groups = (a.n_q_heads + 2 * p->n_kv_heads) * row / (vec ? V : 1);
   const int threads = groups < 512 ? (groups + 31) / 32 * 32 : 512;
-  if (vec)
+  const int n_vec = (a.n_q_heads * a.dim + p->n_kv_heads * (a.dim + a.vdim)) / V;
+  int per = n_vec <= 4 * 128 ? 2 : n_vec <= 4 * 512 ? 4 : 8;   // vectors a thread holds
+  const int nt = ((n_vec + per - 1) / per + 31) / 32 * 32;
+  if (vec && nt <= 512) {
+    if (per == 2) append_norm_regs_kernel<T, V, 2><<<st.n_tokens, nt, 0, s>>>(st, pg, a, row);
+    else if (per == 4) append_norm_regs_kernel<T, V, 4><<<st.n_tokens, nt, 0, s>>>(st, pg, a, row);
+    else append_norm_regs_kernel<T, V, 8><<<st.n_tokens, nt, 0, s>>>(st, pg, a, row);
+  } else if (vec) {
     append_norm_kernel<T, V><<<st.n_tokens, threads, 0, s>>>(st, pg, a, row);
-  else
+  } else {
     append_norm_kernel<T, 1><<<st.n_tokens, threads, 0, s>>>(st, pg, a, row);
+  }
   PACE_LAUNCH_CHECK("append_norm_kernel");
   note_pool_write(s);
   return PACE_OK;

@@ -49,18 +49,19 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
   lo = f2_to_bf2(x - h.x, y - h.y);
 }
 
-template <int DP, int VP>
+template <int DP, int VP, bool STATE_ONLY>
 struct Tiles {
   static constexpr int QP = DP + 8, VQ = VP + 8;  // row pitches: 16 bytes beyond a power of two, ldmatrix without conflicts
-  static constexpr int kStage = kChunk * (2 * QP + VQ);   // q, k, v of one chunk
-  static constexpr int kState = DP * VQ;
+  static constexpr int kK = 0, kV = kChunk * QP, kQ = kV + kChunk * VQ;           // one chunk: k, v, q
+  static constexpr int kStage = STATE_ONLY ? kQ : kQ + kChunk * QP;
+  static constexpr int kState = STATE_ONLY ? 0 : DP * VQ;                         // the state's high and low halves
   static constexpr size_t bytes = sizeof(__nv_bfloat16) * (2 * kStage + 2 * kState) + sizeof(float) * (kChunk + 1);
 };
 
 template <int DP, int VP, bool STATE_ONLY>
-__global__ void __launch_bounds__(kThreads, 1)
+__global__ void __launch_bounds__(kThreads, STATE_ONLY ? 2 : 1)
     lightning_chunk_kernel(pace_step_t st, pace_lightning_args_t a, SegmentArgs sg) {
-  using TL = Tiles<DP, VP>;
+  using TL = Tiles<DP, VP, STATE_ONLY>;
   constexpr int QP = TL::QP, VQ = TL::VQ;
   constexpr int RG = DP / 16, CG = 8 / RG, SC = VP / CG;   // state tile of a warp: 16 rows x SC columns
   constexpr int NT = SC / 8;                               // its 8-column tiles
@@ -83,7 +84,7 @@ __global__ void __launch_bounds__(kThreads, 1)
 
   const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(a.qkv) + (size_t)t0 * a.qkv_stride;
   auto fetch = [&](int l0, int buf) {
-    __nv_bfloat16* q = sm + buf * TL::kStage;
+    __nv_bfloat16* stage = sm + buf * TL::kStage;
     constexpr int per = (2 * DP + VP) / 8;                 // 16-byte pieces of one token
     for (int i = tid; i < kChunk * per; i += kThreads) {
       const int j = i / per, p = i - j * per;
@@ -92,10 +93,10 @@ __global__ void __launch_bounds__(kThreads, 1)
       if (p < 2 * DP / 8) {
         const int which = p / (DP / 8), c = (p - which * (DP / 8)) * 8;
         if (STATE_ONLY && which == 0) continue;
-        copy16(q + which * kChunk * QP + j * QP + c, row + (size_t)(which * H + h) * d + (c < d ? c : 0), tok && c < d);
+        copy16(stage + (which == 0 ? TL::kQ : TL::kK) + j * QP + c, row + (size_t)(which * H + h) * d + (c < d ? c : 0), tok && c < d);
       } else {
         const int c = (p - 2 * DP / 8) * 8;
-        copy16(q + 2 * kChunk * QP + j * VQ + c, row + 2 * (size_t)H * d + (size_t)h * vd + (v0 + c < vd ? v0 + c : 0),
+        copy16(stage + TL::kV + j * VQ + c, row + 2 * (size_t)H * d + (size_t)h * vd + (v0 + c < vd ? v0 + c : 0),
                tok && v0 + c < vd);
       }
     }
@@ -122,17 +123,18 @@ __global__ void __launch_bounds__(kThreads, 1)
   int buf = 0;
   for (int l0 = first; l0 < end; l0 += kChunk, buf ^= 1) {
     const int n_tok = min(kChunk, end - l0);
-    __nv_bfloat16* q_s = sm + buf * TL::kStage;
-    __nv_bfloat16* k_s = q_s + kChunk * QP;
-    __nv_bfloat16* v_s = k_s + kChunk * QP;
+    __nv_bfloat16* q_s = sm + buf * TL::kStage + TL::kQ;
+    __nv_bfloat16* k_s = sm + buf * TL::kStage + TL::kK;
+    __nv_bfloat16* v_s = sm + buf * TL::kStage + TL::kV;
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                       // the chunk is here, the previous one is done with
     constexpr int per = (2 * DP + VP) / 8;
     for (int i = tid; i < kChunk * per; i += kThreads) {   // silu in place
       const int j = i / per, p = i - j * per;
       if (STATE_ONLY && p < DP / 8) continue;
-      __nv_bfloat16* x = p < 2 * DP / 8 ? q_s + (p / (DP / 8)) * kChunk * QP + j * QP + (p % (DP / 8)) * 8
-                                        : v_s + j * VQ + (p - 2 * DP / 8) * 8;
+      __nv_bfloat16* x = p < DP / 8       ? q_s + j * QP + p * 8
+                         : p < 2 * DP / 8 ? k_s + j * QP + (p - DP / 8) * 8
+                                          : v_s + j * VQ + (p - 2 * DP / 8) * 8;
       float f[8];
       Vec<__nv_bfloat16, 8>::load(x, f);
 #pragma unroll
@@ -293,7 +295,7 @@ SegmentArgs plan_segments(int entries, int max_count, int heads, int vdim) {
   SegmentArgs s;
   s.scratch = nullptr;
   const int blocks = entries * heads * ((vdim + 127) / 128);
-  int want = 2 * 148 / (blocks > 0 ? blocks : 1);
+  int want = 148 / (blocks > 0 ? blocks : 1);
   const int most = max_count / (4 * kChunk);               // a segment is worth its own blocks from four chunks on
   if (want > most) want = most;
   if (want < 1) want = 1;
@@ -306,12 +308,12 @@ SegmentArgs plan_segments(int entries, int max_count, int heads, int vdim) {
 
 template <int DP, int VP>
 int launch_chunked(const pace_step_t& st, const pace_lightning_args_t& a, const SegmentArgs& sg, cudaStream_t s) {
-  const size_t smem = Tiles<DP, VP>::bytes;
+  constexpr size_t smem = Tiles<DP, VP, false>::bytes, smem_state = Tiles<DP, VP, true>::bytes;
   const dim3 grid((unsigned)((a.vdim + VP - 1) / VP), (unsigned)a.heads, (unsigned)(st.n_entries * sg.segments));
   if (sg.segments > 1) {
     PACE_CUDA_TRY(cudaFuncSetAttribute(lightning_chunk_kernel<DP, VP, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                       (int)smem));
-    lightning_chunk_kernel<DP, VP, true><<<grid, kThreads, smem, s>>>(st, a, sg);
+                                       (int)smem_state));
+    lightning_chunk_kernel<DP, VP, true><<<grid, kThreads, smem_state, s>>>(st, a, sg);
     PACE_LAUNCH_CHECK("lightning_chunk_kernel (states)");
     const int blocks = (a.dim * a.vdim + 255) / 256;
     lightning_prefix_kernel<<<dim3((unsigned)(blocks < 64 ? blocks : 64), (unsigned)a.heads, (unsigned)st.n_entries), 256, 0, s>>>(

@@ -16,7 +16,7 @@ namespace {
 // inputs come from the cache after their first use.
 constexpr int kConvTokens = 4;
 
-template <typename T, int V>
+template <typename T, int V, int NT>   // NT: number of taps where it is known at compile time, else 0
 __global__ void __launch_bounds__(256)
     causal_conv_kernel(pace_step_t st, const T* __restrict__ in, int64_t in_stride, const float* __restrict__ taps,
                        const float* __restrict__ bias, int n_taps, const float* __restrict__ conv_state, T* __restrict__ out,
@@ -26,6 +26,34 @@ __global__ void __launch_bounds__(256)
   for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const int t0 = (int)(i / per) * kConvTokens, c = (int)(i % per) * V;
     float acc[kConvTokens][V];
+    if constexpr (NT > 0) {
+      // the usual place: four tokens of one entry with all their inputs among the step's rows
+      const int tl = min(t0 + kConvTokens, st.n_tokens) - 1, e = st.tok_entry[tl];
+      if (tl - t0 == kConvTokens - 1 && t0 - (NT - 1) >= st.cu[e]) {
+        float x[kConvTokens + NT - 1][V];
+        const T* row = in + (size_t)(t0 - (NT - 1)) * in_stride + c;
+#pragma unroll
+        for (int r = 0; r < kConvTokens + NT - 1; ++r, row += in_stride) Vec<T, V>::load(row, x[r]);
+        float b[V];
+        Vec<float, V>::load(bias + c, b);
+#pragma unroll
+        for (int r = 0; r < kConvTokens; ++r)
+#pragma unroll
+          for (int v = 0; v < V; ++v) acc[r][v] = b[v];
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          float w[V];
+          Vec<float, V>::load(taps + (size_t)j * channels + c, w);
+#pragma unroll
+          for (int r = 0; r < kConvTokens; ++r)
+#pragma unroll
+            for (int v = 0; v < V; ++v) acc[r][v] = fmaf(w[v], x[r + j][v], acc[r][v]);
+        }
+#pragma unroll
+        for (int r = 0; r < kConvTokens; ++r) Vec<T, V>::store(out + (size_t)(t0 + r) * channels + c, acc[r]);
+        continue;
+      }
+    }
     int local[kConvTokens], pos[kConvTokens];
     const float* ring[kConvTokens];
 #pragma unroll
@@ -60,7 +88,7 @@ __global__ void __launch_bounds__(256)
 // ---------------------------------------------------------------------------
 // RG-LRU over any number of tokens: gates and convolution come from launches in front
 // ---------------------------------------------------------------------------
-constexpr int kSegs = 16, kSegTokens = 4, kTile = kSegs * kSegTokens;
+constexpr int kSegs = 8, kSegTokens = 8, kTile = kSegs * kSegTokens;
 
 // coefficients of S_t = a S_(t-1) + b for pre-activations of the two gates
 template <typename T>
@@ -71,14 +99,14 @@ __device__ __forceinline__ void rglru_coefficients(float r_pre, float i_pre, flo
 }
 
 // The blocks of a cluster walk 32 channels of one entry together: tiles of 64 tokens go round the cluster, in a
-// block warp = a segment of 4 tokens, lane = a channel.  A thread composes its 4 steps into one affine map; the
+// block warp = a segment of 8 tokens, lane = a channel.  A thread composes its 8 steps into one affine map; the
 // maps of a tile meet in shared memory, their products in the shared memory of every block of the cluster; then
 // each thread replays its 8 steps from the state in front of them.  The next tile's operands are on their way
 // meanwhile.  All blocks of a cluster take the same number of rounds.
 constexpr int kMaxCluster = 4;
 
 template <typename T>
-__global__ void __launch_bounds__(512, 2)
+__global__ void __launch_bounds__(32 * kSegs, 2)
     rglru_scan_kernel(pace_step_t st, pace_rglru_args_t a) {
   __shared__ float2 maps[2][kSegs][32];
   __shared__ float2 tiles_map[2][kMaxCluster][32];   // the round's tiles, written by the cluster's blocks
@@ -102,13 +130,30 @@ __global__ void __launch_bounds__(512, 2)
   float g0[kSegTokens], g1[kSegTokens];
   T uu[kSegTokens], yy[kSegTokens];
   auto fetch = [&](int l0) {
+    // (rows behind the end are read from its last row and not used)
+    const int from = min(l0, count - 1);
+    const float* gp = gr + (size_t)from * 2 * bs;
+    const T *up = u + (size_t)from * W, *yp = yx + (size_t)from * a.yx_stride;
+    if (l0 + kSegTokens <= count) {
 #pragma unroll
-    for (int j = 0; j < kSegTokens; ++j) {
-      const int l = min(l0 + j, count - 1);          // (rows behind the end are read but not used)
-      g0[j] = gr[(size_t)l * 2 * bs];
-      g1[j] = gr[(size_t)l * 2 * bs + bs];
-      uu[j] = u[(size_t)l * W];
-      yy[j] = yx[(size_t)l * a.yx_stride];
+      for (int j = 0; j < kSegTokens; ++j) {
+        g0[j] = gp[0];
+        g1[j] = gp[bs];
+        uu[j] = *up;
+        yy[j] = *yp;
+        gp += 2 * bs;
+        up += W;
+        yp += a.yx_stride;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < kSegTokens; ++j) {
+        const int l = min(l0 + j, count - 1);
+        g0[j] = gr[(size_t)l * 2 * bs];
+        g1[j] = gr[(size_t)l * 2 * bs + bs];
+        uu[j] = u[(size_t)l * W];
+        yy[j] = yx[(size_t)l * a.yx_stride];
+      }
     }
   };
   const int stride = kTile * (int)n_rank;
@@ -164,10 +209,21 @@ __global__ void __launch_bounds__(512, 2)
       }
       carry = s;
     }
+    if (live) {
+      T* o = out + (size_t)l0 * W;
+      if (l0 + kSegTokens <= count) {
 #pragma unroll
-    for (int j = 0; j < kSegTokens; ++j) {
-      mine = fmaf(ca[j], mine, cb[j]);
-      if (l0 + j < count && live) out[(size_t)(l0 + j) * W] = from_f<T>(mine * gelu_tanh_t<T>(to_f<T>(y[j])));
+        for (int j = 0; j < kSegTokens; ++j, o += W) {
+          mine = fmaf(ca[j], mine, cb[j]);
+          *o = from_f<T>(mine * gelu_tanh_t<T>(to_f<T>(y[j])));
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < kSegTokens; ++j, o += W) {
+          mine = fmaf(ca[j], mine, cb[j]);
+          if (l0 + j < count) *o = from_f<T>(mine * gelu_tanh_t<T>(to_f<T>(y[j])));
+        }
+      }
     }
   }
   // (a block's last sends were received in front of the last barrier: nobody writes into a block that has left)
@@ -183,7 +239,7 @@ template <typename T>
 int launch_rglru_scan(const pace_step_t& st, const pace_rglru_args_t& a, cudaStream_t s) {
   const int groups = (a.width + 31) / 32;
   int cluster = 1;                                   // blocks that share an entry's tiles, while the GPU has room for them
-  while (cluster < kMaxCluster && cluster * 2 * kTile <= st.max_count && (int64_t)groups * st.n_entries * cluster < 296)
+  while (cluster < kMaxCluster && cluster * 2 * kTile <= st.max_count && (int64_t)groups * st.n_entries * cluster * 2 <= 296)
     cluster *= 2;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3((unsigned)cluster, (unsigned)groups, (unsigned)st.n_entries);
@@ -212,80 +268,130 @@ __device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+// The operands of one (entry, channel) besides the gates' sums, fetched before they are needed.
+struct StepOperands {
+  float y, x, state, ra, ri, base;
+};
 template <typename T>
-__device__ __forceinline__ void rglru_finish(const pace_step_t& st, const pace_rglru_args_t& a, int e, int c, float r_pre,
-                                             float i_pre, float u) {
-  const int W = a.width, slot = st.slot[e], pos = st.start[e];
+__device__ __forceinline__ StepOperands rglru_operands(const pace_rglru_args_t& a, int row, int pos, int slot, int c) {
+  const T* in = static_cast<const T*>(a.yx) + (size_t)row * a.yx_stride + c;
+  StepOperands o;
+  o.y = to_f<T>(in[0]);
+  o.x = to_f<T>(in[a.width]);
+  o.state = pos == 0 ? 0.f : a.state[(size_t)slot * a.width + c];
+  o.ra = a.ra_bias[c];
+  o.ri = a.ri_bias[c];
+  o.base = a.decay_base[c];
+  return o;
+}
+template <typename T>
+__device__ __forceinline__ void rglru_finish(const pace_rglru_args_t& a, const StepOperands& o, int row, int pos, int slot, int c,
+                                             float r_pre, float i_pre, float u) {
   float ca, cb;
-  rglru_coefficients<T>(r_pre + a.ra_bias[c], i_pre + a.ri_bias[c], u, a.decay_base[c], ca, cb);
-  float* s = a.state + (size_t)slot * W + c;
-  const float S = pos == 0 ? cb : fmaf(ca, *s, cb);
-  *s = S;
-  const T* row = static_cast<const T*>(a.yx) + (size_t)st.cu[e] * a.yx_stride;
-  a.conv_state[((size_t)slot * a.n_taps + pos % a.n_taps) * W + c] = to_f<T>(row[W + c]);
-  static_cast<T*>(a.out)[(size_t)st.cu[e] * W + c] = from_f<T>(S * gelu_tanh_t<T>(to_f<T>(row[c])));
+  rglru_coefficients<T>(r_pre + o.ra, i_pre + o.ri, u, o.base, ca, cb);
+  const float S = fmaf(ca, o.state, cb);
+  a.state[(size_t)slot * a.width + c] = S;
+  a.conv_state[((size_t)slot * a.n_taps + pos % a.n_taps) * a.width + c] = o.x;
+  static_cast<T*>(a.out)[(size_t)row * a.width + c] = from_f<T>(S * gelu_tanh_t<T>(o.y));
 }
 
 // Block (slice, batch tile): 32 output channels of one gate block for 32 entries.  The slice's gate weights and the
 // convolved inputs of the whole gate block go to shared memory (V elements per access), then bf16: warp w multiplies
 // entries [16 (w / 4), +16) with channels [8 (w % 4), +8) of both gates on the tensor cores (fp32 accumulators
 // are the pre-activations); fp32: one thread per (entry, channel).
-template <typename T, int V>
-__global__ void __launch_bounds__(256)
+constexpr int kStepThreads = 512;
+
+template <typename T, int V, int NT>   // NT: taps known at compile time (their inputs are fetched together), else 0
+__global__ void __launch_bounds__(kStepThreads)
     rglru_step_kernel(pace_step_t st, pace_rglru_args_t a, int slices, int ld) {
   extern __shared__ __align__(16) char smem_raw[];
   __shared__ int row_of[kStepEntries], pos_of[kStepEntries], slot_of[kStepEntries];
   T* us = reinterpret_cast<T*>(smem_raw);  // [kStepEntries][ld]
   T* ws = us + kStepEntries * ld;          // [2][kStepChannels][ld]
-  const int W = a.width, bs = W / a.blocks;
+  const int W = a.width, bs = W / a.blocks, tid = threadIdx.x;
   const int blk = blockIdx.x / slices, o0 = (blockIdx.x % slices) * kStepChannels;
   const int e0 = blockIdx.y * kStepEntries, n_e = min(kStepEntries, st.n_entries - e0);
   const int lv = ld / V;                   // vectors of a shared row
   const T* wg = static_cast<const T*>(a.gate_w) + (size_t)blk * 2 * bs * bs;
-#pragma unroll 4
-  for (int i = threadIdx.x; i < 2 * kStepChannels * lv; i += 256) {
+  for (int i = tid; i < 2 * kStepChannels * lv; i += kStepThreads) {
     const int r = i / lv, k = (i - r * lv) * V, o = o0 + (r & (kStepChannels - 1));
-    float x[V];
-#pragma unroll
-    for (int v = 0; v < V; ++v) x[v] = 0.f;
-    if (o < bs && k < bs) Vec<T, V>::load(wg + ((size_t)(r / kStepChannels) * bs + o) * bs + k, x);
-    Vec<T, V>::store(ws + r * ld + k, x);
+    const bool in = o < bs && k < bs;
+    const T* src = wg + (in ? ((size_t)(r / kStepChannels) * bs + o) * bs + k : 0);
+    if constexpr (V * sizeof(T) == 16) {
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(ws + r * ld + k)), "l"(src), "r"(in ? 16 : 0)
+                   : "memory");
+    } else {
+      ws[r * ld + k] = in ? *src : from_f<T>(0.f);
+    }
   }
-  if (threadIdx.x < n_e) {
-    row_of[threadIdx.x] = st.cu[e0 + threadIdx.x];
-    pos_of[threadIdx.x] = st.start[e0 + threadIdx.x];
-    slot_of[threadIdx.x] = st.slot[e0 + threadIdx.x];
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  if (tid < n_e) {
+    row_of[tid] = st.cu[e0 + tid];
+    pos_of[tid] = st.start[e0 + tid];
+    slot_of[tid] = st.slot[e0 + tid];
   }
   __syncthreads();
+  // bf16: the outputs of a multiplying lane, their operands on the way while the inputs are convolved
+  const int warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tig = lane & 3, m0 = ((warp >> 2) & 1) * 16;
+  StepOperands ops[4];
+  if constexpr (sizeof(T) == 2) {
+    if (warp < 8) {
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const int r = m0 + gid + (q >> 1) * 8, o = o0 + (warp & 3) * 8 + tig * 2 + (q & 1);
+        if (r < n_e && o < bs) ops[q] = rglru_operands<T>(a, row_of[r], pos_of[r], slot_of[r], blk * bs + o);
+      }
+    }
+  }
   const T* x0 = static_cast<const T*>(a.yx) + W;
-#pragma unroll 2
-  for (int i = threadIdx.x; i < kStepEntries * lv; i += 256) {
+  for (int i = tid; i < kStepEntries * lv; i += kStepThreads) {
     const int r = i / lv, k = (i - r * lv) * V, c = blk * bs + k;
     float acc[V];
 #pragma unroll
     for (int v = 0; v < V; ++v) acc[v] = 0.f;
     if (r < n_e && k < bs) {
       const int pos = pos_of[r];
+      const T* now = x0 + (size_t)row_of[r] * a.yx_stride + c;
       const float* ring = a.conv_state + (size_t)slot_of[r] * a.n_taps * W + c;
-      Vec<float, V>::load(a.conv_bias + c, acc);
-      for (int j = 0; j < a.n_taps; ++j) {
-        const int back = a.n_taps - 1 - j;
-        if (pos < back) continue;
-        float x[V], w[V];
-        if (back == 0) Vec<T, V>::load(x0 + (size_t)row_of[r] * a.yx_stride + c, x);
-        else Vec<float, V>::load(ring + (size_t)((pos - back) % a.n_taps) * W, x);
-        Vec<float, V>::load(a.taps + (size_t)j * W + c, w);
+      if constexpr (NT > 0) {
+        float x[NT][V];
 #pragma unroll
-        for (int v = 0; v < V; ++v) acc[v] = fmaf(w[v], x[v], acc[v]);
+        for (int j = 0; j < NT; ++j) {
+          const int back = NT - 1 - j;
+          if (back == 0) Vec<T, V>::load(now, x[j]);
+          else if (pos >= back) Vec<float, V>::load(ring + (size_t)((pos - back) % NT) * W, x[j]);
+          else
+#pragma unroll
+            for (int v = 0; v < V; ++v) x[j][v] = 0.f;
+        }
+        Vec<float, V>::load(a.conv_bias + c, acc);
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          float w[V];
+          Vec<float, V>::load(a.taps + (size_t)j * W + c, w);
+#pragma unroll
+          for (int v = 0; v < V; ++v) acc[v] = fmaf(w[v], x[j][v], acc[v]);
+        }
+      } else {
+        Vec<float, V>::load(a.conv_bias + c, acc);
+        for (int j = 0; j < a.n_taps; ++j) {
+          const int back = a.n_taps - 1 - j;
+          if (pos < back) continue;
+          float x[V], w[V];
+          if (back == 0) Vec<T, V>::load(now, x);
+          else Vec<float, V>::load(ring + (size_t)((pos - back) % a.n_taps) * W, x);
+          Vec<float, V>::load(a.taps + (size_t)j * W + c, w);
+#pragma unroll
+          for (int v = 0; v < V; ++v) acc[v] = fmaf(w[v], x[v], acc[v]);
+        }
       }
     }
     Vec<T, V>::store(us + r * ld + k, acc);
   }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
   if constexpr (sizeof(T) == 2) {
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
-    const int m0 = (warp >> 2) * 16;
-    if (m0 >= n_e) return;
+    if (warp >= 8 || m0 >= n_e) return;
     const __nv_bfloat16* up = reinterpret_cast<const __nv_bfloat16*>(us) + (m0 + gid) * ld + tig * 2;
     const __nv_bfloat16* rp = reinterpret_cast<const __nv_bfloat16*>(ws) + ((warp & 3) * 8 + gid) * ld + tig * 2;
     const __nv_bfloat16* ip = rp + kStepChannels * ld;
@@ -300,11 +406,12 @@ __global__ void __launch_bounds__(256)
 #pragma unroll
     for (int q = 0; q < 4; ++q) {
       const int r = m0 + gid + (q >> 1) * 8, o = o0 + (warp & 3) * 8 + tig * 2 + (q & 1);
-      if (r < n_e && o < bs) rglru_finish<T>(st, a, e0 + r, blk * bs + o, cr[q], ci[q], to_f<T>(us[r * ld + o]));
+      if (r < n_e && o < bs)
+        rglru_finish<T>(a, ops[q], row_of[r], pos_of[r], slot_of[r], blk * bs + o, cr[q], ci[q], to_f<T>(us[r * ld + o]));
     }
   } else {
-    for (int i = threadIdx.x; i < kStepEntries * kStepChannels; i += 256) {
-      const int r = i / kStepChannels, oo = i % kStepChannels, o = o0 + oo;
+    for (int i = tid; i < kStepEntries * kStepChannels; i += kStepThreads) {
+      const int r = i / kStepChannels, oo = i % kStepChannels, o = o0 + oo, c = blk * bs + o;
       if (r >= n_e || o >= bs) continue;
       float sr = 0.f, si = 0.f;
       for (int k = 0; k < bs; ++k) {
@@ -312,7 +419,8 @@ __global__ void __launch_bounds__(256)
         sr = fmaf(to_f<T>(ws[oo * ld + k]), x, sr);
         si = fmaf(to_f<T>(ws[(kStepChannels + oo) * ld + k]), x, si);
       }
-      rglru_finish<T>(st, a, e0 + r, blk * bs + o, sr, si, to_f<T>(us[r * ld + o]));
+      rglru_finish<T>(a, rglru_operands<T>(a, row_of[r], pos_of[r], slot_of[r], c), row_of[r], pos_of[r], slot_of[r], c, sr, si,
+                      to_f<T>(us[r * ld + o]));
     }
   }
 }
@@ -478,24 +586,26 @@ int lightning_step_t(const pace_step_t& st, const pace_lightning_args_t& a, cuda
 template <typename T>
 int causal_conv_t(const pace_step_t& st, const void* in, int64_t is, const float* taps, const float* bias, int n_taps,
                   const float* cs, void* out, int channels, cudaStream_t s) {
-  constexpr int V = 16 / sizeof(T);
+  constexpr int V = 8 / sizeof(T);      // (four bf16 or two fp32 channels: the window of rows stays in registers)
   const bool vec = channels % V == 0 && is % V == 0 && aligned16(in) && aligned16(out) && aligned16(bias) && aligned16(cs) && aligned16(taps);
   const size_t groups = (size_t)((st.n_tokens + kConvTokens - 1) / kConvTokens) * (channels / (vec ? V : 1));
   size_t blocks = (groups + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
-  if (vec)
-    causal_conv_kernel<T, V><<<(unsigned)blocks, 256, 0, s>>>(st, (const T*)in, is, taps, bias, n_taps, cs, (T*)out, channels);
+  if (vec && n_taps == 4)
+    causal_conv_kernel<T, V, 4><<<(unsigned)blocks, 256, 0, s>>>(st, (const T*)in, is, taps, bias, n_taps, cs, (T*)out, channels);
+  else if (vec)
+    causal_conv_kernel<T, V, 0><<<(unsigned)blocks, 256, 0, s>>>(st, (const T*)in, is, taps, bias, n_taps, cs, (T*)out, channels);
   else
-    causal_conv_kernel<T, 1><<<(unsigned)blocks, 256, 0, s>>>(st, (const T*)in, is, taps, bias, n_taps, cs, (T*)out, channels);
+    causal_conv_kernel<T, 1, 0><<<(unsigned)blocks, 256, 0, s>>>(st, (const T*)in, is, taps, bias, n_taps, cs, (T*)out, channels);
   PACE_LAUNCH_CHECK("causal_conv_kernel");
   return PACE_OK;
 }
 
-template <typename T, int V>
+template <typename T, int V, int NT>
 int launch_rglru_step(const pace_step_t& st, const pace_rglru_args_t& a, int slices, int ld, size_t smem, cudaStream_t s) {
-  PACE_CUDA_TRY(cudaFuncSetAttribute(rglru_step_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  PACE_CUDA_TRY(cudaFuncSetAttribute(rglru_step_kernel<T, V, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   const dim3 grid((unsigned)(a.blocks * slices), (unsigned)((st.n_entries + kStepEntries - 1) / kStepEntries));
-  rglru_step_kernel<T, V><<<grid, 256, smem, s>>>(st, a, slices, ld);
+  rglru_step_kernel<T, V, NT><<<grid, kStepThreads, smem, s>>>(st, a, slices, ld);
   PACE_LAUNCH_CHECK("rglru_step_kernel");
   return PACE_OK;
 }
@@ -509,7 +619,8 @@ int rglru_step_t(const pace_step_t& st, const pace_rglru_args_t& a, cudaStream_t
   constexpr int V = 16 / sizeof(T);
   const bool vec = bs % V == 0 && a.yx_stride % V == 0 && aligned16(a.yx) && aligned16(a.gate_w) && aligned16(a.taps) &&
                    aligned16(a.conv_bias) && aligned16(a.conv_state);
-  return vec ? launch_rglru_step<T, V>(st, a, slices, ld, smem, s) : launch_rglru_step<T, 1>(st, a, slices, ld, smem, s);
+  if (vec && a.n_taps == 4) return launch_rglru_step<T, V, 4>(st, a, slices, ld, smem, s);
+  return vec ? launch_rglru_step<T, V, 0>(st, a, slices, ld, smem, s) : launch_rglru_step<T, 1, 0>(st, a, slices, ld, smem, s);
 }
 
 bool dtype_ok(int dtype) { return dtype == PACE_DTYPE_BF16 || dtype == PACE_DTYPE_FP32; }
