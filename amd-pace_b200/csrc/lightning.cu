@@ -15,11 +15,14 @@
 namespace pace {
 namespace {
 
-constexpr int kChunk = 64, kThreads = 256;
+constexpr int kChunk = 64;
 
+// `segments` blocks of seg_tokens tokens side by side, per launch: the first launch uses `ratio` times as many (it
+// needs fewer registers, so more of its blocks are resident).
 struct SegmentArgs {
-  float* scratch;     // [entries][segments][heads][dim][vdim]: what a segment adds, then the state in front of it
+  float* scratch;     // [entries][stored][heads][dim][vdim]: what a segment adds, then the state in front of it
   int segments, seg_tokens;
+  int stored, ratio;  // states in scratch per entry, and how many of them one segment of this launch spans
 };
 
 __device__ __forceinline__ void mma16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
@@ -55,21 +58,25 @@ struct Tiles {
   static constexpr int kK = 0, kV = kChunk * QP, kQ = kV + kChunk * VQ;           // one chunk: k, v, q
   static constexpr int kStage = STATE_ONLY ? kQ : kQ + kChunk * QP;
   static constexpr int kState = STATE_ONLY ? 0 : DP * VQ;                         // the state's high and low halves
-  static constexpr size_t bytes = sizeof(__nv_bfloat16) * (2 * kStage + 2 * kState) + sizeof(float) * (kChunk + 1);
+  static constexpr int PP = kChunk + 8, kP = STATE_ONLY ? 0 : kChunk * PP;       // the weights' high and low halves
+  static constexpr size_t bytes = sizeof(__nv_bfloat16) * (2 * kStage + 2 * kState + 2 * kP) + sizeof(float) * (kChunk + 1);
+  static constexpr int kThreads = STATE_ONLY ? 256 : 512;
 };
 
 template <int DP, int VP, bool STATE_ONLY>
-__global__ void __launch_bounds__(kThreads, STATE_ONLY ? 2 : 1)
+__global__ void __launch_bounds__(STATE_ONLY ? 256 : 512, STATE_ONLY ? 2 : 1)
     lightning_chunk_kernel(pace_step_t st, pace_lightning_args_t a, SegmentArgs sg) {
   using TL = Tiles<DP, VP, STATE_ONLY>;
-  constexpr int QP = TL::QP, VQ = TL::VQ;
-  constexpr int RG = DP / 16, CG = 8 / RG, SC = VP / CG;   // state tile of a warp: 16 rows x SC columns
+  constexpr int QP = TL::QP, VQ = TL::VQ, PP = TL::PP, kThreads = TL::kThreads;
+  constexpr int RG = DP / 16, CG = kThreads / 32 / RG, SC = VP / CG;   // state tile of a warp: 16 rows x SC columns
   constexpr int NT = SC / 8;                               // its 8-column tiles
-  constexpr int OT = VP / 16;                              // output tiles of a warp (half of the columns)
+  constexpr int OT = VP / 32;                              // output tiles of a warp: 16 rows x a quarter of the columns
   extern __shared__ __align__(16) __nv_bfloat16 sm[];
   __nv_bfloat16* s_hi = sm + 2 * TL::kStage;
   __nv_bfloat16* s_lo = s_hi + TL::kState;
-  float* pw = reinterpret_cast<float*>(s_lo + TL::kState);
+  __nv_bfloat16* p_hi = s_lo + TL::kState;
+  __nv_bfloat16* p_lo = p_hi + TL::kP;
+  float* pw = reinterpret_cast<float*>(p_lo + TL::kP);
 
   const int e = blockIdx.z / sg.segments, seg = blockIdx.z % sg.segments, h = blockIdx.y, v0 = blockIdx.x * VP;
   const int d = a.dim, vd = a.vdim, H = a.heads;
@@ -109,7 +116,7 @@ __global__ void __launch_bounds__(kThreads, STATE_ONLY ? 2 : 1)
   float S[NT][4];
   const float* from = nullptr;
   if (!STATE_ONLY) {
-    if (sg.segments > 1) from = sg.scratch + (((size_t)e * sg.segments + seg) * H + h) * d * vd;
+    if (sg.segments > 1) from = sg.scratch + (((size_t)e * sg.stored + seg * sg.ratio) * H + h) * d * vd;
     else if (st.start[e] != 0) from = a.state + ((size_t)st.slot[e] * H + h) * d * vd;
   }
 #pragma unroll
@@ -157,14 +164,37 @@ __global__ void __launch_bounds__(kThreads, STATE_ONLY ? 2 : 1)
     if (l0 + kChunk < end) fetch(l0 + kChunk, buf ^ 1);
 
     if (!STATE_ONLY) {
-      // rows 16 (warp % 4), value columns VP / 2 (warp / 4)
-      const int m0 = (warp & 3) * 16, c0 = (warp >> 2) * (VP / 2);
-      float O[OT][4], P[8][4];
+      // the four warps of 16 rows each score 16 keys, then own a quarter of the value columns
+      const int m0 = (warp & 3) * 16, quarter = warp >> 2, c0 = quarter * (VP / 4);
+      const int i0 = m0 + (lane >> 2);
+      if (quarter <= (warp & 3)) {                         // (later keys are out of sight)
+        float P[2][4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n) P[n][0] = P[n][1] = P[n][2] = P[n][3] = 0.f;
+#pragma unroll
+        for (int k0 = 0; k0 < DP; k0 += 16) {
+          uint32_t A[4], B[4];
+          ldsm4(A, q_s + (m0 + (lane & 15)) * QP + k0 + (lane >> 4) * 8);
+          ldsm4(B, k_s + (quarter * 16 + (lane & 7) + (lane >> 4) * 8) * QP + k0 + ((lane >> 3) & 1) * 8);
+          mma16816(P[0], A, B[0], B[1]);
+          mma16816(P[1], A, B[2], B[3]);
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            const int r = i0 + x * 8, j = quarter * 16 + n * 8 + (lane & 3) * 2;
+            const float w0 = j <= r ? P[n][2 * x] * pw[r - j] : 0.f;
+            const float w1 = j + 1 <= r ? P[n][2 * x + 1] * pw[r - j - 1] : 0.f;
+            uint32_t hi, lo;
+            split2(w0, w1, hi, lo);
+            *reinterpret_cast<uint32_t*>(p_hi + r * PP + j) = hi;
+            *reinterpret_cast<uint32_t*>(p_lo + r * PP + j) = lo;
+          }
+      }
+      float O[OT][4];
 #pragma unroll
       for (int n = 0; n < OT; ++n) O[n][0] = O[n][1] = O[n][2] = O[n][3] = 0.f;
-#pragma unroll
-      for (int n = 0; n < 8; ++n) P[n][0] = P[n][1] = P[n][2] = P[n][3] = 0.f;
-      const int live_tiles = 2 * ((m0 >> 4) + 1);          // keys up to the tile's last row
 #pragma unroll
       for (int k0 = 0; k0 < DP; k0 += 16) {
         uint32_t A[4], B[4];
@@ -179,34 +209,20 @@ __global__ void __launch_bounds__(kThreads, STATE_ONLY ? 2 : 1)
           mma16816(O[n], A, B[0], B[1]);
           mma16816(O[n + 1], A, B[2], B[3]);
         }
-#pragma unroll
-        for (int n = 0; n < 8; n += 2) {
-          if (n < live_tiles) {
-            ldsm4(B, k_s + (n * 8 + (lane & 7) + (lane >> 4) * 8) * QP + k0 + ((lane >> 3) & 1) * 8);
-            mma16816(P[n], A, B[0], B[1]);
-            mma16816(P[n + 1], A, B[2], B[3]);
-          }
-        }
       }
-      const int i0 = m0 + (lane >> 2);
       const float f0 = pw[i0 + 1], f1 = pw[i0 + 9];
 #pragma unroll
       for (int n = 0; n < OT; ++n) {
         O[n][0] *= f0; O[n][1] *= f0;
         O[n][2] *= f1; O[n][3] *= f1;
       }
+      asm volatile("bar.sync %0, 128;" ::"r"(1 + (warp & 3)) : "memory");   // the weights of these rows are there
 #pragma unroll
       for (int kk = 0; kk < 4; ++kk) {
-        if (2 * kk >= live_tiles) break;
+        if (kk > (warp & 3)) break;
         uint32_t hi[4], lo[4], B[4];
-#pragma unroll
-        for (int x = 0; x < 4; ++x) {                      // operand registers: (row half, key half)
-          const int n = 2 * kk + (x >> 1), r = i0 + (x & 1) * 8, j = n * 8 + (lane & 3) * 2;
-          float* p = &P[n][(x & 1) * 2];
-          const float w0 = j <= r ? p[0] * pw[r - j] : 0.f;
-          const float w1 = j + 1 <= r ? p[1] * pw[r - j - 1] : 0.f;
-          split2(w0, w1, hi[x], lo[x]);
-        }
+        ldsm4(hi, p_hi + (m0 + (lane & 15)) * PP + kk * 16 + (lane >> 4) * 8);
+        ldsm4(lo, p_lo + (m0 + (lane & 15)) * PP + kk * 16 + (lane >> 4) * 8);
 #pragma unroll
         for (int n = 0; n < OT; n += 2) {
           ldsm4t(B, v_s + (kk * 16 + (lane & 15)) * VQ + c0 + n * 8 + (lane >> 4) * 8);
@@ -261,7 +277,7 @@ __global__ void __launch_bounds__(kThreads, STATE_ONLY ? 2 : 1)
   }
 
   float* to = nullptr;
-  if (STATE_ONLY) to = sg.scratch + (((size_t)e * sg.segments + seg) * H + h) * d * vd;
+  if (STATE_ONLY) to = sg.scratch + (((size_t)e * sg.stored + seg) * H + h) * d * vd;
   else if (last) to = a.state + ((size_t)st.slot[e] * H + h) * d * vd;
   if (!to) return;
 #pragma unroll
@@ -283,7 +299,7 @@ __global__ void lightning_prefix_kernel(pace_step_t st, pace_lightning_args_t a,
   for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
     float s = st.start[e] != 0 ? state[i] : 0.f;
     for (int r = 0; r < used; ++r) {
-      float* p = sg.scratch + (((size_t)e * sg.segments + r) * a.heads + h) * n + i;
+      float* p = sg.scratch + (((size_t)e * sg.stored + r) * a.heads + h) * n + i;
       const float add = r + 1 < used ? *p : 0.f;
       *p = s;
       s = fmaf(f, s, add);
@@ -299,10 +315,19 @@ SegmentArgs plan_segments(int entries, int max_count, int heads, int vdim) {
   const int most = max_count / (4 * kChunk);               // a segment is worth its own blocks from four chunks on
   if (want > most) want = most;
   if (want < 1) want = 1;
-  s.seg_tokens = (max_count + want - 1) / want;
-  s.seg_tokens = (s.seg_tokens + kChunk - 1) / kChunk * kChunk;
+  s.ratio = max_count / want >= 8 * kChunk ? 2 : 1;
+  const int unit = s.ratio * kChunk;
+  s.seg_tokens = ((max_count + want - 1) / want + unit - 1) / unit * unit;
   s.segments = (max_count + s.seg_tokens - 1) / s.seg_tokens;
   if (s.segments < 1) s.segments = 1;
+  s.stored = s.segments * s.ratio;
+  return s;
+}
+// the first launch's view: one segment per stored state
+SegmentArgs state_segments(SegmentArgs s) {
+  s.segments = s.stored;
+  s.seg_tokens /= s.ratio;
+  s.ratio = 1;
   return s;
 }
 
@@ -313,16 +338,18 @@ int launch_chunked(const pace_step_t& st, const pace_lightning_args_t& a, const 
   if (sg.segments > 1) {
     PACE_CUDA_TRY(cudaFuncSetAttribute(lightning_chunk_kernel<DP, VP, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                        (int)smem_state));
-    lightning_chunk_kernel<DP, VP, true><<<grid, kThreads, smem_state, s>>>(st, a, sg);
+    const SegmentArgs ss = state_segments(sg);
+    const dim3 grid_state(grid.x, grid.y, (unsigned)(st.n_entries * ss.segments));
+    lightning_chunk_kernel<DP, VP, true><<<grid_state, 256, smem_state, s>>>(st, a, ss);
     PACE_LAUNCH_CHECK("lightning_chunk_kernel (states)");
     const int blocks = (a.dim * a.vdim + 255) / 256;
     lightning_prefix_kernel<<<dim3((unsigned)(blocks < 64 ? blocks : 64), (unsigned)a.heads, (unsigned)st.n_entries), 256, 0, s>>>(
-        st, a, sg);
+        st, a, ss);
     PACE_LAUNCH_CHECK("lightning_prefix_kernel");
   }
   PACE_CUDA_TRY(cudaFuncSetAttribute(lightning_chunk_kernel<DP, VP, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                      (int)smem));
-  lightning_chunk_kernel<DP, VP, false><<<grid, kThreads, smem, s>>>(st, a, sg);
+  lightning_chunk_kernel<DP, VP, false><<<grid, 512, smem, s>>>(st, a, sg);
   PACE_LAUNCH_CHECK("lightning_chunk_kernel");
   return PACE_OK;
 }
@@ -338,9 +365,9 @@ bool lightning_chunked_fits(const pace_lightning_args_t& a) {
 int lightning_chunked(const pace_step_t& st, const pace_lightning_args_t& a, cudaStream_t s) {
   SegmentArgs sg = plan_segments(st.n_entries, st.max_count, a.heads, a.vdim);
   sg.scratch = a.workspace;
-  const uint64_t need = sizeof(float) * (uint64_t)st.n_entries * sg.segments * a.heads * a.dim * a.vdim;
+  const uint64_t need = sizeof(float) * (uint64_t)st.n_entries * sg.stored * a.heads * a.dim * a.vdim;
   if (sg.segments > 1 && (!a.workspace || a.workspace_bytes < need)) return PACE_ERR_INVALID;
-  if ((int64_t)st.n_entries * sg.segments > 65535) return PACE_ERR_UNSUPPORTED;
+  if ((int64_t)st.n_entries * sg.stored > 65535) return PACE_ERR_UNSUPPORTED;
   if (a.dim <= 64) return a.vdim <= 64 ? launch_chunked<64, 64>(st, a, sg, s) : launch_chunked<64, 128>(st, a, sg, s);
   return a.vdim <= 64 ? launch_chunked<128, 64>(st, a, sg, s) : launch_chunked<128, 128>(st, a, sg, s);
 }
@@ -351,5 +378,5 @@ extern "C" uint64_t pace_lightning_workspace_bytes(int32_t n_entries, int32_t ma
                                                    int32_t vdim) {
   if (n_entries <= 0 || max_count <= 0 || heads <= 0 || dim <= 0 || vdim <= 0) return 0;
   const pace::SegmentArgs sg = pace::plan_segments(n_entries, max_count, heads, vdim);
-  return sg.segments > 1 ? sizeof(float) * (uint64_t)n_entries * sg.segments * heads * dim * vdim : 0;
+  return sg.segments > 1 ? sizeof(float) * (uint64_t)n_entries * sg.stored * heads * dim * vdim : 0;
 }

@@ -207,6 +207,48 @@ def test_decayed_linear_attention_remembers_exactly(dtype, heads, dim, vdim):
         assert float((state - S).abs().max() / S.abs().max()) < 2e-5, counts      # fp32 states with either dtype
 
 
+@pytest.mark.parametrize("heads,dim,vdim", [(2, 64, 128), (64, 32, 40), (3, 128, 136)])
+def test_decayed_linear_attention_over_long_prompts(heads, dim, vdim):
+    """Prompts long enough to be cut into segments that run side by side, of unequal lengths in one batch, in front
+    of them a state from earlier tokens (or none)."""
+    from pace_b200.llm.hybrid_cache import HybridCacheManager, StateSpec
+    from pace_b200.ops import hybrid
+    g = torch.Generator().manual_seed(heads)
+    lens = [1500, 70, 900, 1]
+    decay = torch.linspace(0.9, 0.9999, heads)
+    dec = decay.double()[:, None, None]
+    xs = [torch.randn(n, heads * (2 * dim + vdim), generator=g).to(BF16) for n in lens]
+    cache = HybridCacheManager([StateSpec((("S", (heads, dim, vdim)),))], 4, 64, 4096, BF16, DEV)
+    cache[0]["S"].fill_(float("nan"))
+    at = [0] * 4
+    outs = [[] for _ in lens]
+
+    def go(counts):
+        x = torch.cat([xs[b][at[b]: at[b] + c] for b, c in enumerate(counts)])
+        step = cache.step(counts, torch.zeros(sum(counts), dtype=torch.long), 1)
+        cache.begin_step(step)
+        order = torch.cat([torch.arange(sum(counts[:b]), sum(counts[:b + 1])) for b in step.rows])
+        o = hybrid.lightning(step, x[order].to(DEV), decay.to(DEV), cache[0]["S"]).double().cpu()
+        for b in step.rows:
+            outs[b].append(o[step.first_row[b]: step.first_row[b] + counts[b]])
+            at[b] += counts[b]
+    go([0, 0, 65, 0])
+    go([1, 0, 30, 0])
+    go([1499, 70, 805, 1])
+    silu = lambda z: torch.nn.functional.silu(z.double()).to(BF16).double()     # noqa: E731
+    for b, n in enumerate(lens):
+        q, k, v = (silu(xs[b][:, a: z]).view(n, heads, -1) for a, z in ((0, heads * dim), (heads * dim, 2 * heads * dim),
+                                                                        (2 * heads * dim, xs[b].shape[1])))
+        S, want = torch.zeros(heads, dim, vdim, dtype=torch.float64), []
+        for t in range(n):
+            S = dec * S + k[t, :, :, None] * v[t, :, None, :]
+            want.append(torch.einsum("hdv,hd->hv", S, q[t]))
+        want, got = torch.stack(want), torch.cat(outs[b]).view(n, heads, vdim)
+        rel = (got - want).abs().amax(-1) / want.abs().amax(-1).clamp_min(1e-3)
+        assert float(rel.max()) < 0.012, b
+        assert float((cache[0]["S"][b].double().cpu() - S).abs().max() / S.abs().max()) < 2e-5, b
+
+
 @pytest.mark.parametrize("dtype", [BF16, FP32])
 @pytest.mark.parametrize("width,blocks,taps", [(60, 3, 3), (66, 2, 4), (128, 1, 1), (320, 5, 6), (33, 3, 2)])
 def test_gated_recurrence(dtype, width, blocks, taps):
