@@ -296,13 +296,22 @@ __global__ void lightning_prefix_kernel(pace_step_t st, pace_lightning_args_t a,
   const int used = (count + sg.seg_tokens - 1) / sg.seg_tokens;
   const float f = powf(a.decay[h], (float)sg.seg_tokens);
   const float* state = a.state + ((size_t)st.slot[e] * a.heads + h) * n;
+  constexpr int kBatch = 8;                                // loads of a batch are in flight together
+  const size_t step = (size_t)a.heads * n;
   for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
     float s = st.start[e] != 0 ? state[i] : 0.f;
-    for (int r = 0; r < used; ++r) {
-      float* p = sg.scratch + (((size_t)e * sg.stored + r) * a.heads + h) * n + i;
-      const float add = r + 1 < used ? *p : 0.f;
-      *p = s;
-      s = fmaf(f, s, add);
+    float* p = sg.scratch + ((size_t)e * sg.stored * a.heads + h) * n + i;
+    for (int r = 0; r < used; r += kBatch, p += kBatch * step) {
+      float add[kBatch];
+#pragma unroll
+      for (int j = 0; j < kBatch; ++j)
+        if (r + j + 1 < used) add[j] = p[j * step];
+#pragma unroll
+      for (int j = 0; j < kBatch; ++j) {
+        if (r + j >= used) break;
+        p[j * step] = s;
+        if (r + j + 1 < used) s = fmaf(f, s, add[j]);
+      }
     }
   }
 }
