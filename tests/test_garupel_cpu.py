@@ -110,3 +110,27 @@ def test_plain_recurrences_match_closed_forms():
     outs = [float(ref.causal_conv_token(torch.tensor([x]), taps, torch.tensor([0.5]), past)) for x in (1.0, 2.0, 3.0, 4.0)]
     assert outs == [100.5, 210.5, 321.5, 432.5]
     assert ref.query_temperature(14, 0.3, 16) == 1.0 and ref.query_temperature(15, 0.3, 16) == 1 + 0.3 * math.log(2)
+
+
+def test_llama_checkpoints_load_through_the_registry(tmp_path):
+    """The attention-only decoder takes the same road: config.json, safetensors, plain MLP names, tied head."""
+    import json
+    from pace_b200.llm.registry import load_model
+    from pace_b200.llm.weights import write_safetensors
+    cfg = {"architectures": ["LlamaForCausalLM"], "hidden_size": 128, "intermediate_size": 96, "num_hidden_layers": 1,
+           "num_attention_heads": 2, "num_key_value_heads": 1, "vocab_size": 40, "max_position_embeddings": 64,
+           "rms_norm_eps": 1e-5}
+    g = torch.Generator().manual_seed(0)
+    names = {"model.embed_tokens.weight": (40, 128), "model.norm.weight": (128,)}
+    pre = "model.layers.0."
+    names.update({pre + "input_layernorm.weight": (128,), pre + "post_attention_layernorm.weight": (128,),
+                  pre + "self_attn.q_proj.weight": (128, 128), pre + "self_attn.k_proj.weight": (64, 128),
+                  pre + "self_attn.v_proj.weight": (64, 128), pre + "self_attn.o_proj.weight": (128, 128),
+                  pre + "mlp.gate_proj.weight": (96, 128), pre + "mlp.up_proj.weight": (96, 128),
+                  pre + "mlp.down_proj.weight": (128, 96)})
+    w = {k: torch.randn(*s, generator=g).bfloat16() for k, s in names.items()}
+    (tmp_path / "config.json").write_text(json.dumps(cfg))
+    write_safetensors(str(tmp_path / "model.safetensors"), w)
+    m = load_model(str(tmp_path), torch.bfloat16, "cpu")
+    assert torch.equal(m.model.layers[0].mlp.gate_proj.linear.weight, w[pre + "mlp.gate_proj.weight"])
+    assert torch.equal(m.lm_head.weight, w["model.embed_tokens.weight"])
