@@ -147,7 +147,7 @@ struct SmemPlan {
 // (umma: the tcgen05 variant keeps its Q tile in tensor memory and needs neither the padded Q rows,
 // the merge buffer nor the result slots)
 __host__ __device__ inline SmemPlan plan_smem(int D, int MT, int NS, int n_stages, int live_max, int batch,
-                                              int n_items, bool umma = false) {
+                                              int n_items, bool umma = false, bool split = false) {
   SmemPlan s;
   const int MR = 16 * MT, QS = D * 2 + 16;
   int off = 0;
@@ -161,8 +161,9 @@ __host__ __device__ inline SmemPlan plan_smem(int D, int MT, int NS, int n_stage
   // (mma.sync kernels: only the live rows are ever written; a fragment load of the padding rows of the
   // last 8-row group and beyond reads whatever follows in shared memory, which no live row depends on)
   const int q_rows = MR < ((live_max + 7) & ~7) ? MR : ((live_max + 7) & ~7);
-  // (the tcgen05 variant keeps its Q tile in tensor memory; with two tiles per unit the second one's is here)
-  s.qbuf = umma ? (MT == 16 ? take(128 * D * 2, 1024) : take(16, 16)) : take(q_rows * QS, 128);
+  // (the tcgen05 variant keeps its Q tile in tensor memory; with two tiles per unit the second one's is here, with split
+  // weights every tile's)
+  s.qbuf = umma ? (split ? take((MT / 8) * 128 * D * 2, 1024) : MT == 16 ? take(128 * D * 2, 1024) : take(16, 16)) : take(q_rows * QS, 128);
   s.mg_stride = D + 8;  // floats; the pad spreads the rows of a fragment over the banks
   s.mg = take(umma ? 16 : (NS > 1 ? NS * live_max * (s.mg_stride + 2) * 4 : 16), 16);
   s.n_res = live_max <= 64 ? 2 : 1;
@@ -323,7 +324,7 @@ __device__ __forceinline__ void fence_proxy_async_all() {
   asm volatile("fence.proxy.async;" ::: "memory");
 }
 
-template <int D, int MT, int NS, bool UMMA = false>
+template <int D, int MT, int NS, bool UMMA = false, bool X = false>  // X: weights as two bf16 terms (PACE_ATTN_SPLIT_WEIGHTS)
 __global__ void __launch_bounds__(threads_of(UMMA, UMMA ? 8 : MT * NS), (!UMMA && MT * NS == 4) ? 2 : 1)
     attn_mma_kernel(const MmaParams p, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                     const __grid_constant__ CUtensorMap tmS) {
@@ -363,7 +364,7 @@ __global__ void __launch_bounds__(threads_of(UMMA, UMMA ? 8 : MT * NS), (!UMMA &
   // pend: every sequence has one more key than the pool says, whose row this launch first stores in
   // its slot of the sequence's last page (position seq_len; seq_len itself is left alone)
   const bool pend = !UMMA && p.k_pend != nullptr;
-  const SmemPlan sp = plan_smem(D, MT, NS, n_stages, p.live_max, p.batch, n_items, UMMA);
+  const SmemPlan sp = plan_smem(D, MT, NS, n_stages, p.live_max, p.batch, n_items, UMMA, X);
   unsigned char* ring = smem + sp.ring;  // [n_stages][K | V]
   MetaM* metas = reinterpret_cast<MetaM*>(smem + sp.metas);
   unsigned char* qbuf = smem + sp.qbuf;
@@ -991,7 +992,7 @@ __global__ void __launch_bounds__(threads_of(UMMA, UMMA ? 8 : MT * NS), (!UMMA &
     uc.n_stages = n_stages;
     uc.cta = cta;
     uc.qsw = qbuf;
-    umma_consumer<D, WIDE>(p, uc, tid);
+    umma_consumer<D, WIDE, X>(p, uc, tid);
     return;
   }
 
@@ -1160,7 +1161,17 @@ __global__ void __launch_bounds__(threads_of(UMMA, UMMA ? 8 : MT * NS), (!UMMA &
           o[t][3] *= a1;
         }
         // P (keys x query rows) -> B fragments of P^T: one 8x8 transpose per 8 keys
-        const uint32_t pb0 = movmatrix_t(f2_to_bf2(p00, p01)), pb1 = movmatrix_t(f2_to_bf2(p10, p11));
+        uint32_t ph0, ph1, pl0 = 0, pl1 = 0;
+        if constexpr (X) {
+          split_bf2(p00, p01, ph0, pl0);
+          split_bf2(p10, p11, ph1, pl1);
+          pl0 = movmatrix_t(pl0);
+          pl1 = movmatrix_t(pl1);
+        } else {
+          ph0 = f2_to_bf2(p00, p01);
+          ph1 = f2_to_bf2(p10, p11);
+        }
+        const uint32_t pb0 = movmatrix_t(ph0), pb1 = movmatrix_t(ph1);
         // ---- O^T += V^T P^T: tiles of 16 head dimensions x 8 query rows ----
         {
           const int row = tw0 + (mi >> 1) * 8 + (lane & 7);
@@ -1170,6 +1181,7 @@ __global__ void __launch_bounds__(threads_of(UMMA, UMMA ? 8 : MT * NS), (!UMMA &
             uint32_t a[4];
             ldsm_x4_t(vb + (cg >> 3) * HALF_B + row * 128 + (((cg & 7) ^ (row & 7)) << 4), a[0], a[1], a[2], a[3]);
             mma16816(o[t], a, pb0, pb1);
+            if constexpr (X) mma16816(o[t], a, pl0, pl1);
           }
         }
       } else {
@@ -1263,15 +1275,20 @@ __global__ void __launch_bounds__(threads_of(UMMA, UMMA ? 8 : MT * NS), (!UMMA &
         o[n][2] *= a1;
         o[n][3] *= a1;
       }
-      uint32_t pk[NT][2];
+      uint32_t pk[NT][2], pl[NT][2];
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt) {
         const float p00 = fast_exp2(sc[nt][0] - e0), p01 = fast_exp2(sc[nt][1] - e0);
         const float p10 = fast_exp2(sc[nt][2] - e1), p11 = fast_exp2(sc[nt][3] - e1);
         l0 += p00 + p01;
         l1 += p10 + p11;
-        pk[nt][0] = f2_to_bf2(p00, p01);
-        pk[nt][1] = f2_to_bf2(p10, p11);
+        if constexpr (X) {
+          split_bf2(p00, p01, pk[nt][0], pl[nt][0]);
+          split_bf2(p10, p11, pk[nt][1], pl[nt][1]);
+        } else {
+          pk[nt][0] = f2_to_bf2(p00, p01);
+          pk[nt][1] = f2_to_bf2(p10, p11);
+        }
       }
       // ---- O += P V ----
       if constexpr (NT == 1) {
@@ -1285,6 +1302,12 @@ __global__ void __launch_bounds__(threads_of(UMMA, UMMA ? 8 : MT * NS), (!UMMA &
           mma1688(o[n4 * 4 + 1], pk[0][0], pk[0][1], b1);
           mma1688(o[n4 * 4 + 2], pk[0][0], pk[0][1], b2);
           mma1688(o[n4 * 4 + 3], pk[0][0], pk[0][1], b3);
+          if constexpr (X) {
+            mma1688(o[n4 * 4 + 0], pl[0][0], pl[0][1], b0);
+            mma1688(o[n4 * 4 + 1], pl[0][0], pl[0][1], b1);
+            mma1688(o[n4 * 4 + 2], pl[0][0], pl[0][1], b2);
+            mma1688(o[n4 * 4 + 3], pl[0][0], pl[0][1], b3);
+          }
         }
       } else {
 #pragma unroll
@@ -1300,6 +1323,11 @@ __global__ void __launch_bounds__(threads_of(UMMA, UMMA ? 8 : MT * NS), (!UMMA &
               ldsm_x4_t(vb + (cg >> 3) * HALF_B + row * 128 + (((cg & 7) ^ (row & 7)) << 4), b0, b1, b2, b3);
               mma16816(o[2 * n2], a, b0, b1);
               mma16816(o[2 * n2 + 1], a, b2, b3);
+              if constexpr (X) {
+                const uint32_t al[4] = {pl[2 * kb2][0], pl[2 * kb2][1], pl[2 * kb2 + 1][0], pl[2 * kb2 + 1][1]};
+                mma16816(o[2 * n2], al, b0, b1);
+                mma16816(o[2 * n2 + 1], al, b2, b3);
+              }
             }
           }
         }
@@ -1550,7 +1578,7 @@ struct MmaExtra {
   const CUtensorMap* tm_sub = nullptr;  // the pool seen in 16-row boxes (64-token pages only)
 };
 
-template <int D, int MT, int NS, bool UMMA = false>
+template <int D, int MT, int NS, bool UMMA = false, bool X = false>
 int launch_mma(MmaParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, int grid, cudaStream_t stream,
                const MmaExtra& ex) {
   constexpr int MR = 16 * MT;
@@ -1560,10 +1588,10 @@ int launch_mma(MmaParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, int
   // two CTAs per SM (four consumer warps): 228 KB of shared memory less 1 KB the system keeps per CTA
   const int budget = NW == 4 ? kHalfSmemBudget : 227 * 1024;  // (227 KB: the most one CTA may ask for)
   int ns = kMaxStagesM;
-  while (ns >= 2 && plan_smem(D, MT, NS, ns, p.live_max, p.batch, n_items, UMMA).total > budget) --ns;
+  while (ns >= 2 && plan_smem(D, MT, NS, ns, p.live_max, p.batch, n_items, UMMA, X).total > budget) --ns;
   if (ns < 2) return PACE_ERR_UNSUPPORTED;
   p.n_stages = ns;
-  const size_t smem_bytes = plan_smem(D, MT, NS, ns, p.live_max, p.batch, n_items, UMMA).total;
+  const size_t smem_bytes = plan_smem(D, MT, NS, ns, p.live_max, p.batch, n_items, UMMA, X).total;
   // Early K/V streaming: only the short prologue of whole-unit decode has it, and only when this
   // library's newest launch on the stream was an attention launch (nothing wrote the pool since).
   p.early_kv = (!UMMA && MT == 1 && p.whole_units && !ex.no_early_kv && ex.pages && !p.q_lens &&
@@ -1574,9 +1602,9 @@ int launch_mma(MmaParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, int
   int dev = 0;
   PACE_CUDA_TRY(cudaGetDevice(&dev));
   if (dev >= 16 || !configured[dev]) {
-    PACE_CUDA_TRY(cudaFuncSetAttribute(attn_mma_kernel<D, MT, NS, UMMA>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    PACE_CUDA_TRY(cudaFuncSetAttribute(attn_mma_kernel<D, MT, NS, UMMA, X>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                        budget));
-    PACE_CUDA_TRY(cudaFuncSetAttribute(attn_mma_kernel<D, MT, NS, UMMA>,
+    PACE_CUDA_TRY(cudaFuncSetAttribute(attn_mma_kernel<D, MT, NS, UMMA, X>,
                                        cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared));
     if (dev < 16) configured[dev] = true;
   }
@@ -1591,7 +1619,7 @@ int launch_mma(MmaParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, int
   cfg.attrs = attr;
   cfg.numAttrs = 1;
   p.sub_boxes = (ex.tm_sub && !UMMA && MT == 1 && p.pages_per_chunk == 1 && p.kv.page_tokens == kChunk) ? 1 : 0;
-  PACE_CUDA_TRY(cudaLaunchKernelEx(&cfg, attn_mma_kernel<D, MT, NS, UMMA>, p, tmK, tmV, ex.tm_sub ? *ex.tm_sub : tmK));
+  PACE_CUDA_TRY(cudaLaunchKernelEx(&cfg, attn_mma_kernel<D, MT, NS, UMMA, X>, p, tmK, tmV, ex.tm_sub ? *ex.tm_sub : tmK));
   PACE_LAUNCH_CHECK("attn_mma_kernel");
   note_attention_launch(stream, /*uses_workspace=*/!p.whole_units, ex.pages, ex.layer, p.q);
   return PACE_OK;
@@ -1708,6 +1736,22 @@ int run_mma(const KVView& kv, const CUtensorMap& tmK, const CUtensorMap& tmV, in
       p.v_pend = (const __nv_bfloat16*)ex.v_pend + (size_t)b0 * ex.pend_sb;
     }
     int rc = PACE_ERR_UNSUPPORTED;
+    if (flags & PACE_ATTN_SPLIT_WEIGHTS) {
+      // (tiles of 33 rows and more only on the tcgen05 variant)
+#define PACE_SPLIT_CASE(DD)                                                                           \
+  if (D == DD) {                                                                                      \
+    if (umma) rc = wide ? launch_mma<DD, 16, 1, true, true>(p, tmK, tmV, grid, stream, ex)            \
+                        : launch_mma<DD, 8, 1, true, true>(p, tmK, tmV, grid, stream, ex);            \
+    else if (MT == 1) rc = half ? launch_mma<DD, 1, 4, false, true>(p, tmK, tmV, grid, stream, ex)    \
+                                : launch_mma<DD, 1, 8, false, true>(p, tmK, tmV, grid, stream, ex);   \
+    else if (MT == 2) rc = launch_mma<DD, 2, 4, false, true>(p, tmK, tmV, grid, stream, ex);          \
+  }
+      PACE_SPLIT_CASE(128)
+      PACE_SPLIT_CASE(64)
+#undef PACE_SPLIT_CASE
+      if (rc != PACE_OK) return rc;
+      continue;
+    }
 #define PACE_MMA_CASE(DD, MM, NN) \
   if (D == DD && MT == MM) rc = launch_mma<DD, MM, NN>(p, tmK, tmV, grid, stream, ex);
     if (umma && wide) {

@@ -26,6 +26,10 @@
 // row's running maximum grows by more than 2^8 (the result is exact either way: numerator and
 // denominator share whatever maximum was used).
 //
+// Split weights (template flag X, PACE_ATTN_SPLIT_WEIGHTS): P enters the second product as two bf16 terms, high and
+// low, so the weights keep 16 bits of mantissa instead of 8.  The low halves take the tensor-memory columns of the Q
+// tile; all of Q is then in shared memory, in the form the wide form's second tile uses.
+//
 // Included by attn_mma.cu, which provides MmaParams, MetaM, the ring and its producer warp.
 #pragma once
 
@@ -41,6 +45,7 @@ constexpr int kUmmaQkWarp = 9, kUmmaPvWarp = 10, kUmmaWarpB = 11;
 constexpr int kTmemCols = 512;          // the whole tensor memory of the SM:
 constexpr uint32_t kTmemO = 256;        //   [0, 128) S_A S_B, [128, 192) P_A P_B, [192, 256) Q, [256, 512) O_A O_B
 constexpr uint32_t kTmemP = 128, kTmemQ = 192;
+constexpr uint32_t kTmemPLow = kTmemQ;  // split weights (X): [192, 224) / [224, 256) the low halves of P_A / P_B, Q in shared memory
 constexpr float kLazyRescale = 8.0f;    // log2 units
 // Wide form: every n-th pair of a row's scores takes 2^x on the FMA pipe (0: none).  Both groups are in
 // their exp2 phase at the same time there (they wait for the same K/V chunk) and the one exp2 unit per
@@ -60,7 +65,7 @@ struct UmmaCtx {
   uint64_t* q_ready;      // the Q tile of a unit part is in tensor memory (one arrival per softmax warp)
   uint64_t* drain;        // [2] every MMA an issuer warp issued has completed
   uint64_t* drain_b;      // the same for warp 11 (second QK issuer or second PV issuer)
-  unsigned char* qsw;     // wide form: tile B's Q, K-major 128-byte-swizzled: [D/64][128 rows][128 B]
+  unsigned char* qsw;     // wide form: tile B's Q, K-major 128-byte-swizzled: [D/64][128 rows][128 B]; split weights: every tile's
   uint64_t* pub;          // meeting point of the 256 softmax threads while a cut unit is published
   uint64_t* xch;          // the two groups have posted their (max, sum) of a part (one arrival per warp)
   uint32_t* tmem_slot;    // where tcgen05.alloc wrote the base address
@@ -145,6 +150,32 @@ __device__ __forceinline__ void exp2_poly2(float x0, float x1, float& p0, float&
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(q) : "l"(c3), "l"(f), "l"(c2));
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(q) : "l"(q), "l"(f), "l"(c1));
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(q) : "l"(q), "l"(f), "l"(c0));
+  uint32_t r0, r1, q0, q1;
+  asm("mov.b64 {%0, %1}, %2;" : "=r"(r0), "=r"(r1) : "l"(r));
+  asm("mov.b64 {%0, %1}, %2;" : "=r"(q0), "=r"(q1) : "l"(q));
+  p0 = __uint_as_float(q0 + (r0 << 23));
+  p1 = __uint_as_float(q1 + (r1 << 23));
+}
+// The same with a degree-5 polynomial (minimax for the relative error on [-0.5, 0.5], found with the Remez exchange:
+// 7e-8, 2.4e-7 with fp32 arithmetic): weights that are split keep what this gives them.
+__device__ __forceinline__ void exp2_poly2_fine(float x0, float x1, float& p0, float& p1) {
+  x0 = fmaxf(x0, -126.f);
+  x1 = fmaxf(x1, -126.f);
+  uint64_t x, r, f, q;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(x) : "r"(__float_as_uint(x0)), "r"(__float_as_uint(x1)));
+  auto both = [](float v) {
+    uint64_t d;
+    asm("mov.b64 %0, {%1, %1};" : "=l"(d) : "r"(__float_as_uint(v)));
+    return d;
+  };
+  r = add2(x, both(12582912.0f));        // 1.5 * 2^23: the low mantissa bits are the rounded integer
+  f = add2(r, both(-12582912.0f));
+  f = fma2(f, both(-1.0f), x);           // x - round(x)
+  q = fma2(both(0.0013276472632f), f, both(0.0096755413431f));
+  q = fma2(q, f, both(0.0555071327186f));
+  q = fma2(q, f, both(0.2402211972371f));
+  q = fma2(q, f, both(0.6931469670651f));
+  q = fma2(q, f, both(1.0000000716547f));
   uint32_t r0, r1, q0, q1;
   asm("mov.b64 {%0, %1}, %2;" : "=r"(r0), "=r"(r1) : "l"(r));
   asm("mov.b64 {%0, %1}, %2;" : "=r"(q0), "=r"(q1) : "l"(q));
@@ -262,7 +293,7 @@ __device__ __forceinline__ bool elect_one() {
 // every chunk paced the whole pipeline).
 // Wide form (W): warp 9 issues both tiles' QK of every chunk: tile A's Q from tensor memory into S_A, tile B's
 // from shared memory into S_B.
-template <int D, bool W>
+template <int D, bool W, bool X>
 __device__ __forceinline__ void umma_issue_qk(const UmmaCtx& c, uint32_t tmem, int lane, int mine) {
   constexpr int HALF_B = kChunk * 128;
   constexpr uint32_t IDESC_QK1 = umma_idesc(kChunk, false);
@@ -272,8 +303,19 @@ __device__ __forceinline__ void umma_issue_qk(const UmmaCtx& c, uint32_t tmem, i
   const uint32_t k_lo0 = (smem_u32(c.ring) >> 4) | (1u << 16);  // K-major: LBO unused (1)
   const uint32_t k_half = (uint32_t)c.n_stages * (HALF_B >> 4);  // from one 64-column block of K to the next
   const uint32_t tQ = tmem + kTmemQ;  // 16 elements of every row per MMA: 8 columns
-  const uint32_t q_lo = (smem_u32(c.qsw) >> 4) | (1u << 16);  // (wide form: tile B's Q, K-major in shared memory)
-  constexpr int QHALF = kUmmaRows * 128;
+  constexpr int QHALF = kUmmaRows * 128, QTILE = (D / 64) * QHALF;
+  // Q tiles in shared memory, K-major: the wide form's tile B, with split weights every tile (A first)
+  const uint32_t qa_lo = (smem_u32(c.qsw) >> 4) | (1u << 16), q_lo = qa_lo + (X ? (QTILE >> 4) : 0);
+  auto product_a = [&](uint32_t tS, uint32_t k_lo) {   // scores of the tile whose Q is A's (or the only one)
+#pragma unroll
+    for (int kk = 0; kk < D / 16; ++kk) {
+      const uint64_t kd = pack64(k_lo + (kk >> 2) * k_half + (kk & 3) * 2, kDescHi);
+      if constexpr (X)
+        umma_bf16(tS, pack64(qa_lo + (kk >> 2) * (QHALF >> 4) + (kk & 3) * 2, kDescHi), kd, IDESC_QK1, kk ? 1u : 0u);
+      else
+        umma_bf16_ts(tS, tQ + kk * 8, kd, IDESC_QK1, kk ? 1u : 0u);
+    }
+  };
   const bool leader = elect_one();
   int s = 0, ph = 0;       // ring stage / its phase
   int part = 0, left = 0;  // chunks left in the current unit part
@@ -296,9 +338,7 @@ __device__ __forceinline__ void umma_issue_qk(const UmmaCtx& c, uint32_t tmem, i
       if (used_a > 0 && !issuer_wait(c, &c.s_free[0], (used_a - 1) & 1)) break;
       tc_fence_after();
       if (leader) {
-#pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk)
-          umma_bf16_ts(tmem, tQ + kk * 8, pack64(k_lo + (kk >> 2) * k_half + (kk & 3) * 2, kDescHi), IDESC_QK1, kk ? 1u : 0u);
+        product_a(tmem, k_lo);
         umma_commit(&c.s_full[0]);
       }
       __syncwarp();
@@ -335,9 +375,7 @@ __device__ __forceinline__ void umma_issue_qk(const UmmaCtx& c, uint32_t tmem, i
       const uint32_t k_lo = k_lo0 + (uint32_t)s * (HALF_B >> 4);
       const uint32_t tS = tmem + (uint32_t)g * kChunk;
       if (leader) {
-#pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk)
-          umma_bf16_ts(tS, tQ + kk * 8, pack64(k_lo + (kk >> 2) * k_half + (kk & 3) * 2, kDescHi), IDESC_QK1, kk ? 1u : 0u);
+        product_a(tS, k_lo);
         umma_commit(&c.s_full[g]);
       }
       __syncwarp();
@@ -362,7 +400,7 @@ __device__ __forceinline__ void umma_issue_qk(const UmmaCtx& c, uint32_t tmem, i
 
 // mine: -1 = every PV (narrow form); 0 / 1 = group A's / B's of every chunk (wide form: the two groups do
 // not wait for one another anywhere, the ring stage goes back once both PVs have read it)
-template <int D, bool W>
+template <int D, bool W, bool X>
 __device__ __forceinline__ void umma_issue_pv(const UmmaCtx& c, uint32_t tmem, int lane, int mine) {
   constexpr int KVB = kChunk * D * 2, HALF_B = kChunk * 128;
   constexpr uint32_t IDESC_PV = umma_idesc(D, true);
@@ -400,6 +438,12 @@ __device__ __forceinline__ void umma_issue_pv(const UmmaCtx& c, uint32_t tmem, i
 #pragma unroll
         for (int k = 1; k < 4; ++k)  // 16 keys per instruction
           umma_bf16_ts(tO, tP + k * 8, pack64(v_lo + k * (2048 >> 4), kDescHi), IDESC_PV, 1u);
+        if constexpr (X) {
+          const uint32_t tPl = tmem + kTmemPLow + (uint32_t)w * 32;
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            umma_bf16_ts(tO, tPl + k * 8, pack64(v_lo + k * (2048 >> 4), kDescHi), IDESC_PV, 1u);
+        }
         umma_commit(&c.empty_bar[s]);  // K and V of this stage have been consumed (wide form: by this group)
         umma_commit(&c.o_full[w]);                          // O_w holds the chunk; P_w may be rewritten
       }
@@ -496,7 +540,7 @@ __device__ __forceinline__ void umma_merge(const MmaParams& p, const ResMeta& rm
 // chunk - two query tiles share each K/V chunk the CTA fetches, which halves the L2 -> SM traffic per flop
 // (with one tile per fetch the launch was pinned at about 5 TB/s of it, sixteen tiles pulling every K/V
 // byte).  Tile A's Q sits in tensor memory, tile B's in shared memory.
-template <int D, bool W>
+template <int D, bool W, bool X>
 __device__ __forceinline__ void umma_softmax(const MmaParams& p, const UmmaCtx& c, uint32_t tmem, int tid) {
   constexpr int MR = W ? 2 * kUmmaRows : kUmmaRows, REC = MR * (D + 2);
   const int wg = tid >> 7, row = tid & 127, lane = tid & 31, G = p.G;
@@ -544,7 +588,19 @@ __device__ __forceinline__ void umma_softmax(const MmaParams& p, const UmmaCtx& 
       const uint4* src = reinterpret_cast<const uint4*>(p.q + (size_t)fin.b * p.q_sb + (size_t)(fin.h * G + g) * p.q_sh +
                                                         (size_t)sq * p.q_ss);
       out_row = p.out + (size_t)fin.b * p.o_sb + (size_t)(fin.h * G + g) * p.o_sh + (size_t)sq * p.o_ss;
-      if constexpr (!W) {
+      if constexpr (X) {
+        // every tile's rows into shared memory (narrow: each group stores half of the row)
+        unsigned char* qrow = c.qsw + (W ? wg * (D / 64) * (kUmmaRows * 128) : 0) + row * 128;
+        constexpr int N = W ? D / 8 : D / 16;
+        const int c0 = W ? 0 : wg * N;
+#pragma unroll
+        for (int k = 0; k < N; ++k) {
+          const int cc = c0 + k;
+          const uint4 v = live ? __ldg(src + cc) : make_uint4(0, 0, 0, 0);
+          *reinterpret_cast<uint4*>(qrow + (cc >> 3) * (kUmmaRows * 128) + (((cc & 7) ^ (row & 7)) << 4)) = v;
+        }
+        fence_proxy_async();  // generic-proxy writes before the tensor core's async-proxy reads
+      } else if constexpr (!W) {
         // each group stores half of the row: D / 2 elements = D / 4 columns (a 16-byte piece is four columns)
         uint32_t qv[D / 4];
 #pragma unroll
@@ -662,19 +718,22 @@ __device__ __forceinline__ void umma_softmax(const MmaParams& p, const UmmaCtx& 
         uint32_t pk[2][16];
 #pragma unroll
         for (int hf = 0; hf < 2; ++hf) {
+          uint32_t pl[16];
 #pragma unroll
           for (int k = 0; k < 16; ++k) {
             uint32_t x0, x1;
             unpack64(fma2(pack64(sr[hf][2 * k], sr[hf][2 * k + 1]), scale2, ne2), x0, x1);
             float p0, p1;
             if (W && kWidePolyEvery > 0 && (k % (kWidePolyEvery > 0 ? kWidePolyEvery : 1)) == kWidePolyEvery - 1) {
-              exp2_poly2(__uint_as_float(x0), __uint_as_float(x1), p0, p1);
+              if constexpr (X) exp2_poly2_fine(__uint_as_float(x0), __uint_as_float(x1), p0, p1);
+              else exp2_poly2(__uint_as_float(x0), __uint_as_float(x1), p0, p1);
             } else {
               p0 = fast_exp2(__uint_as_float(x0));
               p1 = fast_exp2(__uint_as_float(x1));
             }
             l2[k & 1] = add2(l2[k & 1], pack64(__float_as_uint(p0), __float_as_uint(p1)));
-            pk[hf][k] = f2_to_bf2(p0, p1);
+            if constexpr (X) split_bf2(p0, p1, pk[hf][k], pl[k]);
+            else pk[hf][k] = f2_to_bf2(p0, p1);
           }
           if (hf == 0) {
             // The PV of the group's previous chunk has to have read the buffer (its completion is o_full's
@@ -686,6 +745,7 @@ __device__ __forceinline__ void umma_softmax(const MmaParams& p, const UmmaCtx& 
             }
           }
           tmem_st16(tP + hf * 16, pk[hf]);
+          if constexpr (X) tmem_st16(t_lane + kTmemPLow + (uint32_t)wg * 32 + hf * 16, pl);
         }
         {
           uint32_t a0, a1, b0, b1;
@@ -841,7 +901,7 @@ __device__ __forceinline__ void umma_softmax(const MmaParams& p, const UmmaCtx& 
 // Entry of warps 0..7 and 9..11 of a CTA that has work: warp 9 owns the tensor memory and issues QK MMAs
 // (warp 11 those of group B's chunks on full tiles), warp 10 the PV MMAs, warps 0..7 are the two softmax groups.  Every wait inside is bounded and every path ends at
 // the barrier in front of the deallocation: a CTA never exits holding tensor memory.
-template <int D, bool W>
+template <int D, bool W, bool X>
 __device__ __forceinline__ void umma_consumer(const MmaParams& p, const UmmaCtx& c, int tid) {
   const int warp = tid >> 5, lane = tid & 31;
   const bool owner = warp == kUmmaQkWarp;
@@ -855,12 +915,12 @@ __device__ __forceinline__ void umma_consumer(const MmaParams& p, const UmmaCtx&
   asm volatile("bar.sync 3, 352;" ::: "memory");
   tc_fence_after();
   const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(c.tmem_slot);
-  if (warp == kUmmaQkWarp) umma_issue_qk<D, W>(c, tmem, lane, 0);
+  if (warp == kUmmaQkWarp) umma_issue_qk<D, W, X>(c, tmem, lane, 0);
   else if (warp == kUmmaWarpB) {
-    if (W) umma_issue_pv<D, W>(c, tmem, lane, 1);
-    else umma_issue_qk<D, W>(c, tmem, lane, 1);
-  } else if (warp == kUmmaPvWarp) umma_issue_pv<D, W>(c, tmem, lane, W ? 0 : -1);
-  else umma_softmax<D, W>(p, c, tmem, tid);
+    if (W) umma_issue_pv<D, W, X>(c, tmem, lane, 1);
+    else umma_issue_qk<D, W, X>(c, tmem, lane, 1);
+  } else if (warp == kUmmaPvWarp) umma_issue_pv<D, W, X>(c, tmem, lane, W ? 0 : -1);
+  else umma_softmax<D, W, X>(p, c, tmem, tid);
   if (lane == 0 && *c.abort) raise_status(p.kv.status, PACE_DEV_WAIT_TIMEOUT);
   tc_fence_before();
   asm volatile("bar.sync 3, 352;" ::: "memory");

@@ -294,6 +294,12 @@ __device__ __forceinline__ uint32_t f2_to_bf2(float a, float b) {
   __nv_bfloat162 t = __floats2bfloat162_rn(a, b);
   return *reinterpret_cast<uint32_t*>(&t);
 }
+// two fp32 values as bf16 pairs hi + lo that together carry 16 bits of mantissa
+__device__ __forceinline__ void split_bf2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = f2_to_bf2(a, b);
+  const float2 h = bf2_to_f2(hi);
+  lo = f2_to_bf2(a - h.x, b - h.y);
+}
 __device__ __forceinline__ float fast_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));

@@ -45,13 +45,6 @@ __device__ __forceinline__ void ldsm4t(uint32_t* r, const void* p) {
 __device__ __forceinline__ void copy16(void* dst, const void* src, bool live) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
 }
-// a pair of fp32 values as bf16 pairs hi + lo
-__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  hi = f2_to_bf2(x, y);
-  const float2 h = bf2_to_f2(hi);
-  lo = f2_to_bf2(x - h.x, y - h.y);
-}
-
 template <int DP, int VP, bool STATE_ONLY>
 struct Tiles {
   static constexpr int QP = DP + 8, VQ = VP + 8;  // row pitches: 16 bytes beyond a power of two, ldmatrix without conflicts
@@ -154,7 +147,7 @@ __global__ void __launch_bounds__(STATE_ONLY ? 256 : 512, STATE_ONLY ? 2 : 1)
 #pragma unroll
         for (int q = 0; q < 4; q += 2) {
           uint32_t hi, lo;
-          split2(S[n][q], S[n][q + 1], hi, lo);
+          split_bf2(S[n][q], S[n][q + 1], hi, lo);
           const int at = (sr + (q >> 1) * 8) * VQ + sc + n * 8;
           *reinterpret_cast<uint32_t*>(s_hi + at) = hi;
           *reinterpret_cast<uint32_t*>(s_lo + at) = lo;
@@ -187,7 +180,7 @@ __global__ void __launch_bounds__(STATE_ONLY ? 256 : 512, STATE_ONLY ? 2 : 1)
             const float w0 = j <= r ? P[n][2 * x] * pw[r - j] : 0.f;
             const float w1 = j + 1 <= r ? P[n][2 * x + 1] * pw[r - j - 1] : 0.f;
             uint32_t hi, lo;
-            split2(w0, w1, hi, lo);
+            split_bf2(w0, w1, hi, lo);
             *reinterpret_cast<uint32_t*>(p_hi + r * PP + j) = hi;
             *reinterpret_cast<uint32_t*>(p_lo + r * PP + j) = lo;
           }
@@ -261,7 +254,7 @@ __global__ void __launch_bounds__(STATE_ONLY ? 256 : 512, STATE_ONLY ? 2 : 1)
         const float x0 = k.x * pw[max(n_tok - 1 - j, 0)], x1 = k.y * pw[max(n_tok - 2 - j, 0)];
         hi[x] = f2_to_bf2(x0, x1);
         const float2 g = bf2_to_f2(hi[x]);
-        split2(x0 - g.x, x1 - g.y, mid[x], lo[x]);
+        split_bf2(x0 - g.x, x1 - g.y, mid[x], lo[x]);
       }
 #pragma unroll
       for (int n = 0; n < NT; n += 2) {

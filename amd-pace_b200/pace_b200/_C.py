@@ -39,6 +39,7 @@ ATTN_WHOLE_UNITS = 1      # PACE_ATTN_WHOLE_UNITS
 ATTN_PENDING_ROW = 2      # PACE_ATTN_PENDING_ROW
 ATTN_NO_EARLY_KV = 4      # PACE_ATTN_NO_EARLY_KV
 ATTN_ONE_CTA_PER_SM = 8   # PACE_ATTN_ONE_CTA_PER_SM
+ATTN_SPLIT_WEIGHTS = 16   # PACE_ATTN_SPLIT_WEIGHTS
 
 
 class AttnArgs(C.Structure):

@@ -307,6 +307,13 @@ typedef struct pace_attn_args {
  * back to it by themselves when the workspace or shared memory has no room for two blocks per SM). */
 #define PACE_ATTN_ONE_CTA_PER_SM 8u
 
+/* The softmax weights enter the product with V as two bf16 terms (high and low, 16 bits of mantissa together)
+ * instead of one rounded to bf16, and every exponential is good to fp32's last bits: for models that want weights
+ * kept in 32-bit.  Costs one more tensor-core product per key; the cache is read once all the same.  Not for
+ * tiles of 33 query rows and more whose output rows are not 16-byte aligned, nor for an additive mask.  (The CUDA-core
+ * decode kernel keeps its weights in fp32 anyway.) */
+#define PACE_ATTN_SPLIT_WEIGHTS 16u
+
 uint64_t pace_attn_workspace_bytes(int32_t batch, int32_t n_q_heads, int32_t n_kv_heads, int32_t head_dim,
                                    int32_t q_len);
 /* q_len == 1.  The grouped query heads of a KV head are packed into one mma.sync tile (any group

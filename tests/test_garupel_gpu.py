@@ -139,6 +139,31 @@ def test_one_key_far_away_at_every_page_border(dtype, heads, kv, dim, vdim):
             cache.recycle([row])
 
 
+@pytest.mark.parametrize("heads,kv,dim,vdim", [(4, 1, 128, 128), (12, 1, 64, 64), (20, 1, 96, 80), (2, 1, 64, 64)])
+def test_softmax_weights_are_not_rounded_to_bf16(heads, kv, dim, vdim):
+    """Every key but the first has a weight half way between two bf16 values: rounded, all of them would be off in
+    the same direction by 2^-8 of themselves, and half of the outputs would land on another bf16 value than the exact
+    result does."""
+    p = 0.5 + 2.0 ** -9 * 0.98
+    n = 500
+    for counts in ([n], [n - 1, 1], [n - 2, 2], [n - 3, 3], [n - 40, 40]):
+        qkv, cache = _attention_case(BF16, heads, kv, dim, vdim, n, 11)
+        v = (1.0 + torch.rand(n, kv * vdim, generator=torch.Generator().manual_seed(1))).to(BF16)
+        qkv[:, : (heads + kv) * dim] = 0
+        qkv[:, : heads * dim: dim] = 1
+        qkv[0, heads * dim: (heads + kv) * dim: dim] = 1
+        qkv[:, (heads + kv) * dim:] = v
+        got = _attend(qkv, cache, 0, counts, heads, dim, vdim, -math.log(p))[n - counts[-1]:]
+        w = torch.cat([torch.ones(1, dtype=torch.float64), torch.full((n - 1,), p, dtype=torch.float64)])
+        same = []
+        for i in range(0, counts[-1], 97):
+            t = n - counts[-1] + i
+            if t >= 300:
+                want = (w[: t + 1] @ v[: t + 1].double()) / w[: t + 1].sum()
+                same.append((got[i] == want.view(kv, vdim).to(BF16).double()).double().mean())
+        assert float(min(same)) > 0.9, (counts, same)
+
+
 @pytest.mark.parametrize("dtype", [BF16, FP32])
 def test_norms_and_temperature_of_queries_and_keys(dtype):
     heads, kv, dim, vdim, n, eps = 4, 2, 24, 40, 70, 0.05
