@@ -1094,6 +1094,37 @@ def hybrid_kernels(size: str, dev):
         add("norm_gate", [lambda i=i: hybrid.norm_gate(lo[i], wp[:LH * D] if LH * D <= W else vec(LH * D),
                                                        lq[i][:, 3 * LH * D:], 1e-5) for i in range(N)], T * LH * D * 6)
         add("relu_squared", [lambda i=i: hybrid.relu_squared_(up[i]) for i in range(N)], T * FF * 4)
+        # the like kernels of the attention-only decoder on the same operands: plain attention (its weights rounded to
+        # bf16), RoPE + append, norm and residual, gated activation (the last two are torch's)
+        from pace_b200.llm.cache import KVCacheManager, KVCacheType
+        from pace_b200.ops import MultiHeadAttention, RotaryEmbedding
+
+        class LlamaCfg:
+            num_hidden_layers = N
+        mgr = KVCacheManager(LlamaCfg(), past + n * (8 if not dec else 64) + 64, KVCacheType.BMC)
+        for i in range(N):
+            kv = rnd(E, G, past + n, D)
+            mgr[i].update_cache(kv, kv, concat_dim=2)
+        q4, mha = [t.view(E, n, H, D).transpose(1, 2) for t in qb], MultiHeadAttention()
+        o4 = torch.empty(E, n, H, D, dtype=torch.bfloat16, device=dev).transpose(1, 2)
+        add("llama.attention", [lambda i=i: mha(q4[i], mgr[i].key, mgr[i].value, out=o4) for i in range(N)],
+            kv_read + T * nq * 4, flops)
+        if not dec:                               # (a decode step stages its rows: profiled with the decode loop)
+            rope = RotaryEmbedding(None, D, 8192, 500000.0).to(dev)
+            rws = rope.table_rows(torch.arange(n, device=dev).expand(E, n))
+            xs = [t[:, : nq + 2 * nk].view(E, n, H + 2 * G, D) for t in qkvg]
+            qo = [t.view(E, n, H, D) for t in qb]
+            cos, sin = rope.device_tables(pool.device)
+            add("llama.append_rope", [lambda i=i: torch.ops.pace_b200.kv_append_rope(
+                mgr.pool.handle, mgr.pool.pages, mgr.pool.meta, i, mgr.slots_dev, xs[i][:, :, :H], xs[i][:, :, H:H + G],
+                xs[i][:, :, H + G:], qo[i], rws, cos, sin, D, False, None, xs[i][:, :, H:H + G].transpose(1, 2), xs[i][:, :, H + G:].transpose(1, 2))
+                for i in range(N)], T * (nq + 2 * nk) * 4)
+        w16 = wp.bfloat16()
+        add("llama.residual+norm (torch)", [lambda i=i: torch.nn.functional.rms_norm(y[i] + y[i - 1], (W,), w16, 1e-5)
+                                            for i in range(N)], T * W * 2 * 4)
+        add("llama.silu*up (torch)", [lambda i=i: up[i] * torch.nn.functional.silu(up[i - 1]) for i in range(N)], T * FF * 6)
+        mgr.pool.check_status()
+        del mgr
         cache.pool.check_status()
         if not dec:                               # the parts of the recurrence's prefill
             u = [rnd(T, W) for _ in range(N)]
