@@ -1,23 +1,37 @@
 // Causal softmax attention over the paged pool on the CUDA cores, for rows the tensor-core kernels do not
-// take: fp32 caches, head sizes beyond 128, any pair of key and value sizes up to 512.
+// take: fp32 caches, head sizes beyond 128, any pair of key and value sizes up to 640 and 512; with or without a span,
+// a distance bias and a sink.
 //
 // A thread block owns 32 query rows (token, grouped head) of one (sequence, KV head); its eight warps hold
 // four rows each.  Keys and values pass through shared memory 32 at a time: a lane scores one key for its
 // warp's rows, then owns value columns while the weights are passed round by shuffles.  Online softmax,
 // everything in fp32.
-#include "hybrid.cuh"
+#include "span.cuh"
 
 namespace pace {
 namespace {
+
+struct GeneralArgs {
+  const void* q;
+  void* out;
+  const int32_t* rows;   // row of q and out of a token, nullptr: the token itself
+  const float* slopes;
+  const float* sinks;
+  int H, d, vd, q_row, o_row, row;   // elements of a row of q, out and the pool
+  int entry0, span, span_size;
+  float scale;
+};
 
 constexpr int kRows = 32, kKeys = 32, kRowsPerWarp = 4, kThreads = 256;
 
 template <typename T, int VI>  // VI: value columns per lane
 __global__ void __launch_bounds__(kThreads)
-    attn_general_kernel(KVView kv, pace_step_t st, const T* __restrict__ q, T* __restrict__ out, int H, int d, int vd, int row,
-                        float scale) {
+    attn_general_kernel(KVView kv, pace_step_t st, GeneralArgs a) {
   extern __shared__ float smem[];
-  const int e = blockIdx.z, g = blockIdx.y;
+  const T* __restrict__ q = static_cast<const T*>(a.q);
+  T* __restrict__ out = static_cast<T*>(a.out);
+  const int H = a.H, d = a.d, vd = a.vd, row = a.row;
+  const int e = a.entry0 + blockIdx.z, g = blockIdx.y;
   const int Gq = H / kv.n_kv_heads;
   const int t0 = st.cu[e], count = st.cu[e + 1] - t0, start = st.start[e];
   const int r0 = blockIdx.x * kRows;
@@ -38,16 +52,20 @@ __global__ void __launch_bounds__(kThreads)
     float v = 0.f;
     if (r0 + r < count * Gq) {
       const int tok = (r0 + r) / Gq, hh = g * Gq + (r0 + r) % Gq;
-      v = to_f<T>(q[((size_t)st.q_row[t0 + tok] * H + hh) * row + c]);
+      v = to_f<T>(q[((size_t)(a.rows ? a.rows[t0 + tok] : t0 + tok) * H + hh) * a.q_row + c]);
     }
     qs[i] = v;
   }
-  int last[kRowsPerWarp];  // last visible position of the warp's rows, -1 for rows that do not exist
+  int last[kRowsPerWarp];   // last visible position of the warp's rows, -1 for rows that do not exist
+  int first[kRowsPerWarp];  // first one
+  float slope[kRowsPerWarp];
   float m[kRowsPerWarp], l[kRowsPerWarp], acc[kRowsPerWarp][VI];
 #pragma unroll
   for (int r = 0; r < kRowsPerWarp; ++r) {
     const int rr = r0 + warp * kRowsPerWarp + r;
     last[r] = rr < count * Gq ? start + rr / Gq : -1;
+    first[r] = last[r] < 0 ? 0 : span_first(a.span, a.span_size, last[r]);
+    slope[r] = (a.slopes && last[r] >= 0) ? a.slopes[g * Gq + rr % Gq] : 0.f;
     m[r] = -INFINITY;
     l[r] = 0.f;
 #pragma unroll
@@ -55,7 +73,7 @@ __global__ void __launch_bounds__(kThreads)
   }
   const int r_end = min(r0 + kRows, count * Gq) - 1;
   const int n_keys = start + r_end / Gq + 1;
-  for (int k0 = 0; k0 < n_keys; k0 += kKeys) {
+  for (int k0 = span_first(a.span, a.span_size, start + r0 / Gq) / kKeys * kKeys; k0 < n_keys; k0 += kKeys) {
     __syncthreads();
     for (int i = tid; i < kKeys * (d + vd); i += kThreads) {
       const bool is_v = i >= kKeys * d;
@@ -84,8 +102,10 @@ __global__ void __launch_bounds__(kThreads)
     }
 #pragma unroll
     for (int r = 0; r < kRowsPerWarp; ++r) {
-      if (last[r] < k0) continue;  // (the warp's rows agree: lanes differ in the key only)
-      float x = k0 + lane <= last[r] ? s[r] * scale : -INFINITY;
+      if (last[r] < k0 || first[r] >= k0 + kKeys) continue;  // (the warp's rows agree: lanes differ in the key only)
+      const int pos = k0 + lane;
+      float x = -INFINITY;
+      if (pos <= last[r] && pos >= first[r]) x = s[r] * a.scale + slope[r] * (float)(pos - last[r]);
       float mx = x;
 #pragma unroll
       for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -114,7 +134,13 @@ __global__ void __launch_bounds__(kThreads)
     const int rr = r0 + warp * kRowsPerWarp + r;
     if (last[r] < 0) continue;
     const int tok = rr / Gq, hh = g * Gq + rr % Gq;
-    T* o = out + ((size_t)st.q_row[t0 + tok] * H + hh) * row;
+    if (a.sinks) {  // one more term of the denominator
+      const float sink = a.sinks[hh], mx = fmaxf(m[r], sink), f = expf(m[r] - mx);
+      l[r] = l[r] * f + expf(sink - mx);
+#pragma unroll
+      for (int i = 0; i < VI; ++i) acc[r][i] *= f;
+    }
+    T* o = out + ((size_t)(a.rows ? a.rows[t0 + tok] : t0 + tok) * H + hh) * a.o_row;
 #pragma unroll
     for (int i = 0; i < VI; ++i) {
       const int c = lane + 32 * i;
@@ -124,28 +150,55 @@ __global__ void __launch_bounds__(kThreads)
 }
 
 template <typename T, int VI>
-int launch_general(const KVView& kv, const pace_step_t& st, const void* q, void* out, int H, int d, int vd, int row,
-                   float scale, cudaStream_t s) {
-  const size_t smem = sizeof(float) * ((size_t)kRows * d + (size_t)kKeys * (d | 1) + (size_t)kKeys * vd);
+int launch_general(const KVView& kv, const pace_step_t& st, const GeneralArgs& a, int entries, int max_tokens, cudaStream_t s) {
+  const size_t smem = sizeof(float) * ((size_t)kRows * a.d + (size_t)kKeys * (a.d | 1) + (size_t)kKeys * a.vd);
+  if (smem > 227 * 1024) return PACE_ERR_UNSUPPORTED;
   PACE_CUDA_TRY(cudaFuncSetAttribute(attn_general_kernel<T, VI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  const int Gq = H / kv.n_kv_heads;
-  const dim3 grid((unsigned)((st.max_count * Gq + kRows - 1) / kRows), (unsigned)kv.n_kv_heads, (unsigned)st.n_entries);
-  attn_general_kernel<T, VI><<<grid, kThreads, smem, s>>>(kv, st, (const T*)q, (T*)out, H, d, vd, row, scale);
+  const int Gq = a.H / kv.n_kv_heads;
+  const dim3 grid((unsigned)(((size_t)max_tokens * Gq + kRows - 1) / kRows), (unsigned)kv.n_kv_heads, (unsigned)entries);
+  attn_general_kernel<T, VI><<<grid, kThreads, smem, s>>>(kv, st, a);
   PACE_LAUNCH_CHECK("attn_general_kernel");
   return PACE_OK;
 }
 
 template <typename T>
-int general_t(const KVView& kv, const pace_step_t& st, const void* q, void* out, int H, int d, int vd, int row, float scale,
-              cudaStream_t s) {
-  if (vd <= 32) return launch_general<T, 1>(kv, st, q, out, H, d, vd, row, scale, s);
-  if (vd <= 64) return launch_general<T, 2>(kv, st, q, out, H, d, vd, row, scale, s);
-  if (vd <= 128) return launch_general<T, 4>(kv, st, q, out, H, d, vd, row, scale, s);
-  if (vd <= 256) return launch_general<T, 8>(kv, st, q, out, H, d, vd, row, scale, s);
-  return launch_general<T, 16>(kv, st, q, out, H, d, vd, row, scale, s);
+int general_t(const KVView& kv, const pace_step_t& st, const GeneralArgs& a, int entries, int max_tokens, cudaStream_t s) {
+  if (a.vd <= 32) return launch_general<T, 1>(kv, st, a, entries, max_tokens, s);
+  if (a.vd <= 64) return launch_general<T, 2>(kv, st, a, entries, max_tokens, s);
+  if (a.vd <= 128) return launch_general<T, 4>(kv, st, a, entries, max_tokens, s);
+  if (a.vd <= 256) return launch_general<T, 8>(kv, st, a, entries, max_tokens, s);
+  return launch_general<T, 16>(kv, st, a, entries, max_tokens, s);
+}
+
+int general(const KVView& kv, const pace_step_t& st, const GeneralArgs& a, int entries, int max_tokens, int dtype, cudaStream_t s) {
+  if (a.d > 640 || a.vd > 512 || kv.n_kv_heads > 65535 || entries > 65535) return PACE_ERR_UNSUPPORTED;
+  return dtype == PACE_DTYPE_BF16 ? general_t<__nv_bfloat16>(kv, st, a, entries, max_tokens, s)
+                                  : general_t<float>(kv, st, a, entries, max_tokens, s);
 }
 
 }  // namespace
+
+int attn_general_span(const pace_kv_pool_t* p, int layer, const pace_step_t& st, const pace_attn_span_args_t& a,
+                      cudaStream_t s) {
+  GeneralArgs ga;
+  ga.q = a.q;
+  ga.out = a.out;
+  ga.rows = nullptr;
+  ga.slopes = a.slopes;
+  ga.sinks = a.sinks;
+  ga.H = a.n_q_heads;
+  ga.d = a.dim;
+  ga.vd = a.vdim;
+  ga.q_row = a.q_elems;
+  ga.o_row = a.out_elems;
+  ga.row = a.dtype == PACE_DTYPE_BF16 ? p->head_dim : p->head_dim / 2;
+  ga.entry0 = a.entry_begin;
+  ga.span = a.span;
+  ga.span_size = a.span_size;
+  ga.scale = a.scale;
+  return general(make_view(p, layer, nullptr), st, ga, a.entry_end - a.entry_begin, a.max_tokens, a.dtype, s);
+}
+
 }  // namespace pace
 
 using namespace pace;
@@ -156,12 +209,21 @@ extern "C" int pace_attn_general(const pace_kv_pool_t* p, int32_t layer, const p
   if (H < 1 || H % p->n_kv_heads || d < 1 || vd < 1 || st->max_count < 0) return PACE_ERR_INVALID;
   if (dtype != PACE_DTYPE_BF16 && dtype != PACE_DTYPE_FP32) return PACE_ERR_INVALID;
   if (p->row_format == PACE_ROWS_BF16 && dtype != PACE_DTYPE_BF16) return PACE_ERR_INVALID;
-  const int row = dtype == PACE_DTYPE_BF16 ? p->head_dim : p->head_dim / 2;
-  if (d > row || vd > row) return PACE_ERR_INVALID;
-  if (d > 512 || vd > 512 || p->n_kv_heads > 65535 || st->n_entries > 65535) return PACE_ERR_UNSUPPORTED;
+  GeneralArgs ga;
+  ga.row = ga.q_row = ga.o_row = dtype == PACE_DTYPE_BF16 ? p->head_dim : p->head_dim / 2;
+  if (d > ga.row || vd > ga.row) return PACE_ERR_INVALID;
   if (st->n_tokens == 0) return PACE_OK;
   PACE_PROFILE("attn_general", stream, "layer=%d entries=%d tokens=%d", layer, st->n_entries, st->n_tokens);
-  const KVView kv = make_view(p, layer, nullptr);
-  return dtype == PACE_DTYPE_BF16 ? general_t<__nv_bfloat16>(kv, *st, q, out, H, d, vd, row, scale, (cudaStream_t)stream)
-                                  : general_t<float>(kv, *st, q, out, H, d, vd, row, scale, (cudaStream_t)stream);
+  ga.q = q;
+  ga.out = out;
+  ga.rows = st->q_row;
+  ga.slopes = ga.sinks = nullptr;
+  ga.H = H;
+  ga.d = d;
+  ga.vd = vd;
+  ga.entry0 = 0;
+  ga.span = PACE_SPAN_ALL;
+  ga.span_size = 0;
+  ga.scale = scale;
+  return general(make_view(p, layer, nullptr), *st, ga, st->n_entries, st->max_count, dtype, (cudaStream_t)stream);
 }

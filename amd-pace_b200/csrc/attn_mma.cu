@@ -26,6 +26,7 @@
 #include <mutex>
 
 #include "common.cuh"
+#include "umma.cuh"
 
 namespace pace {
 namespace {
@@ -1474,23 +1475,6 @@ __global__ void __launch_bounds__(threads_of(UMMA, UMMA ? 8 : MT * NS), (!UMMA &
 }
 
 // ------------------------------- host side -------------------------------
-typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                             const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                             CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-EncodeFn encode_fn() {
-  static EncodeFn fn = nullptr;
-  static std::once_flag once;
-  std::call_once(once, [] {
-    void* ptr = nullptr;
-    cudaDriverEntryPointQueryResult q;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &q) == cudaSuccess &&
-        q == cudaDriverEntryPointSuccess)
-      fn = reinterpret_cast<EncodeFn>(ptr);
-  });
-  return fn;
-}
-
 // bf16 tensor seen as [c3][tiles][rows][D]; box = 64 columns x box_rows rows, 128-byte swizzle
 int make_map(CUtensorMap* tm, const void* base, int D, int rows, uint64_t tiles, uint64_t c3, uint64_t c3_stride_elems,
              int box_rows) {

@@ -1,0 +1,492 @@
+// Softmax attention over the paged pool with a span (window or chunk), a distance bias and a sink: decode, short
+// portions of prompts and whatever the tcgen05 prompt kernel (attn_span_umma.cu) does not take.  bf16 rows of any size,
+// keys and values in two planes or (latents) in one.
+//
+// A thread block works on one tile of 16 * MT query rows (row = token * group + head of the group) of one (entry, KV
+// head) and a contiguous share of the tile's visible keys; the shares of a tile are the blocks of a thread-block cluster.
+// Tiles of 64 keys travel through a ring of shared-memory stages (cp.async, 16 bytes at a time, row strides that
+// are an odd number of 16-byte units: ldmatrix without bank conflicts).  Per tile
+//   scores   warp w: all query rows x keys 8 w .. 8 w + 7, mma.sync m16n8k16
+//   softmax  256 / rows threads per row, fp32, span and bias from positions; weights leave as two bf16 terms
+//   values   warp w: all query rows x the 16-column groups w, w + 8, ...
+// At the end every block has (maximum, sum, weighted values) of its keys in shared memory; the blocks of the cluster merge
+// them over distributed shared memory, each a part of the outputs.  No workspace, no atomics, no order that varies.
+#include <cooperative_groups.h>
+
+#include "span.cuh"
+
+namespace cg = cooperative_groups;
+
+namespace pace {
+namespace {
+
+constexpr int kKeys = 64, kThreads = 256, kPS = kKeys + 8, kSS = kKeys + 4;
+
+struct SpanParams {
+  KVView kv;
+  pace_step_t st;
+  const __nv_bfloat16* q;
+  __nv_bfloat16* out;
+  const float* slopes;
+  const float* sinks;
+  int q_elems, out_elems, H, Gq, dk, dv, row;  // row: elements of a pool row
+  int dk16, dv16, shared_rows;                // sizes rounded up to 16; one plane
+  int entry0, span, span_size, n_stages, tab_cap, page_shift;
+  float scale_log2;
+};
+
+struct SpanSmem {
+  int q, ring, k_bytes, stage_bytes, s, ph, pl, alpha, tab, obuf, ml, total;
+};
+__host__ __device__ inline SpanSmem span_smem(int MR, int dk16, int dv16, int shared_rows, int n_stages, int tab_cap) {
+  SpanSmem m;
+  int off = 0;
+  auto take = [&](int bytes) {
+    const int o = off;
+    off += (bytes + 15) / 16 * 16;
+    return o;
+  };
+  m.q = take(MR * (dk16 + 8) * 2);
+  m.k_bytes = kKeys * (dk16 + 8) * 2;
+  m.stage_bytes = m.k_bytes + (shared_rows ? 0 : kKeys * (dv16 + 8) * 2);
+  m.ring = take(n_stages * m.stage_bytes);
+  m.s = take(MR * kSS * 4);
+  m.ph = take(MR * kPS * 2);
+  m.pl = take(MR * kPS * 2);
+  m.alpha = take(MR * 4);
+  m.tab = take(tab_cap * 4);
+  // behind the last tile the ring's place holds the block's results
+  m.obuf = m.ring;
+  const int need = MR * (dv16 + 4) * 4;
+  if (m.ring + need > off) off = m.ring + need;
+  m.ml = take(MR * 8);
+  m.total = off;
+  return m;
+}
+
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm2(uint32_t addr, uint32_t& r0, uint32_t& r1) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// MT: 16-row tiles of query rows; NG: 16-column groups of the values a warp owns
+template <int MT, int NG>
+__global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kernel(const SpanParams p) {
+  constexpr int MR = 16 * MT, TPR = kThreads / MR, KPT = kKeys / TPR;
+  extern __shared__ __align__(16) unsigned char smem[];
+  const SpanSmem sm = span_smem(MR, p.dk16, p.dv16, p.shared_rows, p.n_stages, p.tab_cap);
+  const int ns = gridDim.x, share = blockIdx.x;  // the cluster is the grid's x extent
+  const int Hkv = p.kv.n_kv_heads, g = blockIdx.y % Hkv, e = p.entry0 + blockIdx.z;
+  const int t0 = p.st.cu[e], count = p.st.cu[e + 1] - t0, start = p.st.start[e];
+  const int R = count * p.Gq, r0 = (int)(blockIdx.y / Hkv) * MR;
+  if (r0 >= R) return;  // (the same for the whole cluster)
+  const int live = min(MR, R - r0);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int pos_a = start + r0 / p.Gq, pos_z = start + (r0 + live - 1) / p.Gq;
+  const int base = span_first(p.span, p.span_size, pos_a) & ~(kKeys - 1);
+  const int n_tiles = (pos_z - base) / kKeys + 1;
+  const int per = (n_tiles + ns - 1) / ns;
+  const int tile_a = min(share * per, n_tiles), tile_z = min(tile_a + per, n_tiles);
+  const int slot = p.st.slot[e], P = p.kv.page_tokens;
+  const uint32_t s_q = smem_u32(smem + sm.q), s_ring = smem_u32(smem + sm.ring);
+  const int KSB = (p.dk16 + 8) * 2, VSB = p.shared_rows ? KSB : (p.dv16 + 8) * 2;  // row strides, bytes
+  const int v_off = p.shared_rows ? 0 : sm.k_bytes;
+  int* tab = reinterpret_cast<int*>(smem + sm.tab);
+
+  // ---- the query rows, the share's page numbers ----
+  {
+    const int pieces = p.dk16 / 8;
+    for (int i = tid; i < MR * pieces; i += kThreads) {
+      const int r = i / pieces, c = i - r * pieces;
+      const int rr = min(r0 + r, R - 1), tok = rr / p.Gq, hh = g * p.Gq + rr - tok * p.Gq;
+      const bool ok = r < live && (c + 1) * 8 <= p.q_elems;
+      cp_async16(s_q + r * KSB + c * 16, p.q + ((size_t)(t0 + tok) * p.H + hh) * p.q_elems + (ok ? c * 8 : 0), ok);
+    }
+  }
+  const bool slot_ok = slot >= 0 && slot < p.kv.max_seqs;
+  const int lp0 = (base + tile_a * kKeys) / P;
+  const int last_pos = min(pos_z, base + tile_z * kKeys - 1);
+  int n_lp = tile_a < tile_z ? last_pos / P - lp0 + 1 : 0;
+  if (n_lp > p.tab_cap || !slot_ok) {
+    if (tid == 0) raise_status(p.kv.status, PACE_DEV_BAD_INDEX);
+    n_lp = slot_ok ? min(n_lp, p.tab_cap) : 0;
+  }
+  for (int i = tid; i < n_lp; i += kThreads) {
+    const int pg = view_page(p.kv, slot, lp0 + i);
+    if (pg < 0) raise_status(p.kv.status, PACE_DEV_BAD_INDEX);
+    tab[i] = pg;
+  }
+  __syncthreads();
+
+  auto load_tile = [&](int t) {
+    const uint32_t dst = s_ring + (uint32_t)((t - tile_a) % p.n_stages) * sm.stage_bytes;
+    auto plane = [&](const __nv_bfloat16* src, uint32_t to, int stride, int width16) {
+      const int pieces = width16 / 8;
+      for (int i = tid; i < kKeys * pieces; i += kThreads) {
+        const int j = i / pieces, c = i - j * pieces, pos = base + t * kKeys + j;
+        const int lp = (p.page_shift >= 0 ? pos >> p.page_shift : pos / P);
+        const int in = pos - lp * P;
+        int pg = -1;
+        if (pos <= pos_z && lp - lp0 < n_lp) pg = tab[lp - lp0];
+        const bool ok = pg >= 0 && (c + 1) * 8 <= p.row;
+        cp_async16(to + j * stride + c * 16, ok ? src + (((size_t)pg * Hkv + g) * P + in) * p.row + c * 8 : src, ok);
+      }
+    };
+    plane(p.kv.k, dst, KSB, p.dk16);
+    if (!p.shared_rows) plane(p.kv.v, dst + sm.k_bytes, VSB, p.dv16);
+  };
+
+  for (int k = 0; k < p.n_stages - 1; ++k) {
+    if (tile_a + k < tile_z) load_tile(tile_a + k);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+
+  // softmax role of this thread: one row, keys 4 (sub + TPR i) + 0..3
+  const int srow = tid / TPR, sub = tid % TPR;
+  const int srr = r0 + srow, stok = srr / p.Gq;
+  const int spos = srow < live ? start + stok : -1;
+  const int sfirst = srow < live ? span_first(p.span, p.span_size, spos) : 0;
+  const int shead = g * p.Gq + (srr - stok * p.Gq);
+  const float slope = (p.slopes && srow < live) ? p.slopes[shead] * kLog2e : 0.f;
+  float m = -INFINITY, l = 0.f;
+  float* S = reinterpret_cast<float*>(smem + sm.s);
+  float* alpha = reinterpret_cast<float*>(smem + sm.alpha);
+  const uint32_t s_ph = smem_u32(smem + sm.ph), s_pl = smem_u32(smem + sm.pl);
+
+  float o[MT][NG][2][4];
+#pragma unroll
+  for (int a = 0; a < MT; ++a)
+#pragma unroll
+    for (int b = 0; b < NG; ++b)
+#pragma unroll
+      for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int d = 0; d < 4; ++d) o[a][b][c][d] = 0.f;
+
+  const int n_groups = p.dv16 / 16, ksteps = p.dk16 / 16;
+  for (int t = tile_a; t < tile_z; ++t) {
+    // (one group is committed per tile, an empty one at the end: all but the newest n_stages - 2 are complete)
+    if (p.n_stages == 2) asm volatile("cp.async.wait_group 0;" ::: "memory");
+    else asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncthreads();  // the tile is here for everybody, and everybody is done with the stage that is filled next
+    if (t + p.n_stages - 1 < tile_z) load_tile(t + p.n_stages - 1);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    const uint32_t stage = s_ring + (uint32_t)((t - tile_a) % p.n_stages) * sm.stage_bytes;
+    // ---- scores ----
+    {
+      float c[MT][2][4];
+#pragma unroll
+      for (int a = 0; a < MT; ++a)
+#pragma unroll
+        for (int b = 0; b < 2; ++b)
+#pragma unroll
+          for (int d = 0; d < 4; ++d) c[a][b][d] = 0.f;
+      // ldmatrix x4 over two k-steps of this warp's eight keys; A: rows lane % 16, column half lane / 16
+      const uint32_t kb = stage + (warp * 8 + (lane & 7)) * KSB + (lane >> 3) * 16;
+      const uint32_t qa = s_q + (lane & 15) * KSB + (lane >> 4) * 16;
+      int kk = 0;
+      for (; kk + 2 <= ksteps; kk += 2) {
+        uint32_t b[4];
+        ldsm4(kb + kk * 32, b);
+#pragma unroll
+        for (int a = 0; a < MT; ++a) {
+          uint32_t q0[4], q1[4];
+          ldsm4(qa + a * 16 * KSB + kk * 32, q0);
+          ldsm4(qa + a * 16 * KSB + kk * 32 + 32, q1);
+          mma16816(c[a][0], q0, b[0], b[1]);
+          mma16816(c[a][1], q1, b[2], b[3]);
+        }
+      }
+      if (kk < ksteps) {
+        uint32_t b0, b1;
+        ldsm2(stage + (warp * 8 + (lane & 7)) * KSB + ((lane >> 3) & 1) * 16 + kk * 32, b0, b1);
+#pragma unroll
+        for (int a = 0; a < MT; ++a) {
+          uint32_t q0[4];
+          ldsm4(qa + a * 16 * KSB + kk * 32, q0);
+          mma16816(c[a][0], q0, b0, b1);
+        }
+      }
+      const int col = warp * 8 + (lane & 3) * 2;
+#pragma unroll
+      for (int a = 0; a < MT; ++a) {
+        const int r = a * 16 + (lane >> 2);
+        *reinterpret_cast<float2*>(S + r * kSS + col) = make_float2(c[a][0][0] + c[a][1][0], c[a][0][1] + c[a][1][1]);
+        *reinterpret_cast<float2*>(S + (r + 8) * kSS + col) = make_float2(c[a][0][2] + c[a][1][2], c[a][0][3] + c[a][1][3]);
+      }
+    }
+    __syncthreads();
+    // ---- softmax ----
+    {
+      float x[KPT];
+      float mx = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < KPT / 4; ++i) {
+        const int k = 4 * (sub + TPR * i), pos = base + t * kKeys + k;
+        const float4 s4 = *reinterpret_cast<const float4*>(S + srow * kSS + k);
+        const float sv[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const bool seen = pos + j <= spos && pos + j >= sfirst;
+          x[4 * i + j] = seen ? fmaf(sv[j], p.scale_log2, slope * (float)(pos + j - spos)) : -INFINITY;
+          mx = fmaxf(mx, x[4 * i + j]);
+        }
+      }
+#pragma unroll
+      for (int d = TPR / 2; d; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+      const float mn = fmaxf(m, mx);
+      const float f = m == -INFINITY ? (mn == -INFINITY ? 1.f : 0.f) : fast_exp2(m - mn);
+      const float ref = mn == -INFINITY ? 0.f : mn;
+      m = mn;
+      float sum = 0.f;
+      const uint32_t prow = (uint32_t)srow * (kPS * 2);
+#pragma unroll
+      for (int i = 0; i < KPT / 4; ++i) {
+        uint32_t h0, h1, l0, l1;
+        float w[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          w[j] = fast_exp2(x[4 * i + j] - ref);
+          sum += w[j];
+        }
+        split_bf2(w[0], w[1], h0, l0);
+        split_bf2(w[2], w[3], h1, l1);
+        const uint32_t at = prow + 8 * (sub + TPR * i);
+        asm volatile("st.shared.v2.b32 [%0], {%1, %2};" ::"r"(s_ph + at), "r"(h0), "r"(h1) : "memory");
+        asm volatile("st.shared.v2.b32 [%0], {%1, %2};" ::"r"(s_pl + at), "r"(l0), "r"(l1) : "memory");
+      }
+      l = l * f + sum;
+      if (sub == 0) alpha[srow] = f;
+    }
+    __syncthreads();
+    // ---- values ----
+    if (warp < n_groups) {
+#pragma unroll
+      for (int a = 0; a < MT; ++a) {
+        const float f0 = alpha[a * 16 + (lane >> 2)], f1 = alpha[a * 16 + (lane >> 2) + 8];
+        if (f0 != 1.f || f1 != 1.f) {
+#pragma unroll
+          for (int b = 0; b < NG; ++b)
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+              o[a][b][c][0] *= f0;
+              o[a][b][c][1] *= f0;
+              o[a][b][c][2] *= f1;
+              o[a][b][c][3] *= f1;
+            }
+        }
+      }
+      const uint32_t pa = (uint32_t)(lane & 15) * (kPS * 2) + (lane >> 4) * 16;
+      const uint32_t vb = stage + v_off + (lane & 15) * VSB + (lane >> 4) * 16;
+#pragma unroll
+      for (int ks = 0; ks < kKeys / 16; ++ks) {
+        uint32_t ah[MT][4], al[MT][4];
+#pragma unroll
+        for (int a = 0; a < MT; ++a) {
+          ldsm4(s_ph + pa + a * 16 * (kPS * 2) + ks * 32, ah[a]);
+          ldsm4(s_pl + pa + a * 16 * (kPS * 2) + ks * 32, al[a]);
+        }
+#pragma unroll
+        for (int b = 0; b < NG; ++b) {
+          const int gi = warp + 8 * b;
+          if (gi < n_groups) {
+            uint32_t v[4];
+            ldsm4_t(vb + ks * 16 * VSB + gi * 32, v);
+#pragma unroll
+            for (int a = 0; a < MT; ++a) {
+              mma16816(o[a][b][0], ah[a], v[0], v[1]);
+              mma16816(o[a][b][1], ah[a], v[2], v[3]);
+              mma16816(o[a][b][0], al[a], v[0], v[1]);
+              mma16816(o[a][b][1], al[a], v[2], v[3]);
+            }
+          }
+        }
+      }
+    }
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+
+  // ---- this block's results to shared memory, merge over the cluster ----
+  float* O = reinterpret_cast<float*>(smem + sm.obuf);
+  float2* ml = reinterpret_cast<float2*>(smem + sm.ml);
+  const int OS = p.dv16 + 4;
+#pragma unroll
+  for (int d = TPR / 2; d; d >>= 1) l += __shfl_xor_sync(0xffffffffu, l, d);
+  if (sub == 0) ml[srow] = make_float2(m, l);
+#pragma unroll
+  for (int b = 0; b < NG; ++b) {
+    const int gi = warp + 8 * b;
+    if (gi < n_groups) {
+#pragma unroll
+      for (int a = 0; a < MT; ++a)
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          const int r = a * 16 + (lane >> 2), col = gi * 16 + c * 8 + (lane & 3) * 2;
+          *reinterpret_cast<float2*>(O + r * OS + col) = make_float2(o[a][b][c][0], o[a][b][c][1]);
+          *reinterpret_cast<float2*>(O + (r + 8) * OS + col) = make_float2(o[a][b][c][2], o[a][b][c][3]);
+        }
+    }
+  }
+  cg::cluster_group cl = cg::this_cluster();
+  if (ns > 1) cl.sync();
+  else __syncthreads();
+  const int v4 = p.dv16 / 4;
+  for (int i = share * kThreads + tid; i < live * v4; i += ns * kThreads) {
+    const int r = i / v4, c = (i - r * v4) * 4;
+    const int rr = r0 + r, tok = rr / p.Gq, hh = g * p.Gq + rr - tok * p.Gq;
+    float top = -INFINITY, den = 0.f;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (p.sinks) {
+      top = p.sinks[hh] * kLog2e;
+      den = 1.f;
+    }
+    for (int k = 0; k < ns; ++k) {
+      const float2 st = ns > 1 ? *cl.map_shared_rank(ml + r, k) : ml[r];
+      if (st.x == -INFINITY) continue;
+      const float4 v = *reinterpret_cast<const float4*>(ns > 1 ? cl.map_shared_rank(O + r * OS + c, k) : O + r * OS + c);
+      const float tn = fmaxf(top, st.x);
+      const float fa = top == -INFINITY ? 0.f : fast_exp2(top - tn), fb = fast_exp2(st.x - tn);
+      top = tn;
+      den = den * fa + st.y * fb;
+      acc.x = acc.x * fa + v.x * fb;
+      acc.y = acc.y * fa + v.y * fb;
+      acc.z = acc.z * fa + v.z * fb;
+      acc.w = acc.w * fa + v.w * fb;
+    }
+    const float inv = den > 0.f ? 1.0f / den : 0.f;
+    __nv_bfloat16* dst = p.out + ((size_t)(t0 + tok) * p.H + hh) * p.out_elems + c;
+    const float y[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
+    if (c + 4 <= p.dv && (p.out_elems & 3) == 0) {
+      Vec<__nv_bfloat16, 4>::store(dst, y);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j < p.dv) dst[j] = __float2bfloat16_rn(y[j]);
+    }
+  }
+  if (ns > 1) cl.sync();  // nobody leaves while its shared memory is read
+}
+
+template <int MT, int NG>
+int launch_span(SpanParams& p, int ns, int tiles, int entries, int smem, cudaStream_t s) {
+  auto* fn = attn_span_kernel<MT, NG>;
+  PACE_CUDA_TRY(cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3((unsigned)ns, (unsigned)(tiles * p.kv.n_kv_heads), (unsigned)entries);
+  cfg.blockDim = dim3(kThreads);
+  cfg.dynamicSmemBytes = (size_t)smem;
+  cfg.stream = s;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = (unsigned)ns;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = 1;
+  PACE_CUDA_TRY(cudaLaunchKernelEx(&cfg, fn, p));
+  PACE_LAUNCH_CHECK("attn_span_kernel");
+  return PACE_OK;
+}
+
+constexpr int kSmemMax = 227 * 1024, kTargetBlocks = 2 * 148;
+
+// PACE_ERR_UNSUPPORTED: shapes beyond this kernel (the caller takes the CUDA-core one)
+int span_mma(const pace_kv_pool_t* pl, int layer, const pace_step_t& st, const pace_attn_span_args_t& a, cudaStream_t s) {
+  SpanParams p;
+  p.kv = make_view(pl, layer, nullptr);
+  p.st = st;
+  p.q = static_cast<const __nv_bfloat16*>(a.q);
+  p.out = static_cast<__nv_bfloat16*>(a.out);
+  p.slopes = a.slopes;
+  p.sinks = a.sinks;
+  p.q_elems = a.q_elems;
+  p.out_elems = a.out_elems;
+  p.H = a.n_q_heads;
+  p.Gq = a.n_q_heads / pl->n_kv_heads;
+  p.dk = a.dim;
+  p.dv = a.vdim;
+  p.row = pl->head_dim;
+  p.dk16 = (a.dim + 15) / 16 * 16;
+  p.dv16 = (a.vdim + 15) / 16 * 16;
+  p.shared_rows = pl->row_format == PACE_ROWS_SHARED;
+  p.entry0 = a.entry_begin;
+  p.span = a.span;
+  p.span_size = a.span_size;
+  p.scale_log2 = a.scale * kLog2e;
+  p.page_shift = -1;
+  for (int k = 0; k < 31; ++k)
+    if (pl->page_tokens == (1 << k)) p.page_shift = k;
+  if (a.q_elems % 8 || p.row % 8 || !aligned16(a.q) || !aligned16(pl->pages) || ((uintptr_t)a.out & 7) || p.dv16 > 512)
+    return PACE_ERR_UNSUPPORTED;
+  // (q rows are read in pieces of eight: the caller keeps what lies between dim and the next multiple of 8 zero)
+  if (p.shared_rows && p.dv16 > p.dk16) return PACE_ERR_UNSUPPORTED;
+  const int rows = a.max_tokens * p.Gq;
+  int keys = a.max_keys;   // visible keys of a tile, at most
+  int MT = rows <= 16 ? 1 : rows <= 32 ? 2 : 4;
+  const int NG = p.dv16 <= 128 ? 1 : p.dv16 <= 256 ? 2 : 4;
+  for (;; MT >>= 1) {
+    if (MT == 0) return PACE_ERR_UNSUPPORTED;
+    const int tok = (16 * MT - 1) / p.Gq + 2;   // tokens a tile can touch
+    int k = keys;
+    if (a.span != PACE_SPAN_ALL && (long long)a.span_size + tok < k) k = a.span_size + tok;
+    const int tiles_k = k / kKeys + 2;
+    const int tiles = (rows + 16 * MT - 1) / (16 * MT);
+    const long long units = (long long)tiles * pl->n_kv_heads * (a.entry_end - a.entry_begin);
+    int ns = 1;
+    while (ns < 8 && units * ns * 2 <= kTargetBlocks && tiles_k >= ns * 2) ns *= 2;
+    p.tab_cap = ((tiles_k + ns - 1) / ns + 1) * kKeys / pl->page_tokens + 2;
+    int smem = 0;
+    for (p.n_stages = 3; p.n_stages >= 2; --p.n_stages) {
+      smem = span_smem(16 * MT, p.dk16, p.dv16, p.shared_rows, p.n_stages, p.tab_cap).total;
+      // a third stage only where two blocks still share an SM, or where it is free
+      if (smem <= (p.n_stages == 3 ? kSmemMax / 2 - 1024 : kSmemMax)) break;
+    }
+    if (p.n_stages < 2) continue;
+    if (units > 0x7fffffffLL || (long long)tiles * pl->n_kv_heads > 65535 || a.entry_end - a.entry_begin > 65535)
+      return PACE_ERR_UNSUPPORTED;
+    const int E = a.entry_end - a.entry_begin;
+#define PACE_SPAN_CASE(mt, ng) \
+  if (MT == mt && NG == ng) return launch_span<mt, ng>(p, ns, tiles, E, smem, s);
+    PACE_SPAN_CASE(1, 1) PACE_SPAN_CASE(1, 2) PACE_SPAN_CASE(1, 4)
+    PACE_SPAN_CASE(2, 1) PACE_SPAN_CASE(2, 2) PACE_SPAN_CASE(2, 4)
+    PACE_SPAN_CASE(4, 1) PACE_SPAN_CASE(4, 2) PACE_SPAN_CASE(4, 4)
+#undef PACE_SPAN_CASE
+    return PACE_ERR_UNSUPPORTED;
+  }
+}
+
+}  // namespace
+}  // namespace pace
+
+using namespace pace;
+
+extern "C" int pace_attn_span(const pace_kv_pool_t* p, int32_t layer, const pace_step_t* st, const pace_attn_span_args_t* a,
+                              void* stream) {
+  if (!p || !p->pages || !p->block_table || !step_ok(st) || layer < 0 || layer >= p->n_layers) return PACE_ERR_INVALID;
+  if (!span_args_ok(st, a, p->n_kv_heads)) return PACE_ERR_INVALID;
+  const int row = a->dtype == PACE_DTYPE_BF16 ? p->head_dim : p->head_dim / 2;
+  if (a->dim > row || a->vdim > row || (p->row_format == PACE_ROWS_BF16 && a->dtype != PACE_DTYPE_BF16)) return PACE_ERR_INVALID;
+  if (st->n_tokens == 0 || a->entry_begin == a->entry_end || a->max_tokens == 0) return PACE_OK;
+  PACE_PROFILE("attn_span", stream, "layer=%d entries=%d tokens<=%d heads=%d dims=%d/%d", layer, a->entry_end - a->entry_begin,
+               a->max_tokens, a->n_q_heads, a->dim, a->vdim);
+  if (a->dtype == PACE_DTYPE_BF16) {
+    const int rc = span_mma(p, layer, *st, *a, (cudaStream_t)stream);
+    if (rc != PACE_ERR_UNSUPPORTED) return rc;
+  }
+  return attn_general_span(p, layer, *st, *a, (cudaStream_t)stream);
+}

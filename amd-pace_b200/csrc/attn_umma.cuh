@@ -36,7 +36,6 @@
 namespace pace {
 namespace {
 
-constexpr int kUmmaRows = 128;          // query rows per tile (UMMA M)
 constexpr int kUmmaSoftmaxThreads = 256;  // two warpgroups
 // Warps 0-7: softmax; 8: producer; 9: QK issuer (of group A's chunks when the work is split); 10: PV issuer;
 // 11: narrow form: QK issuer of group B's chunks; wide form: PV issuer of group B.  (Issuers on warps 10 and 11, away from
@@ -74,175 +73,6 @@ struct UmmaCtx {
   int n_my, n_stages, cta;
 };
 
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-
-// shared-memory matrix descriptor, 128-byte swizzle (layout type 2), descriptor version 1
-__device__ __forceinline__ uint64_t umma_desc(uint32_t smem_addr, uint32_t lbo_bytes, uint32_t sbo_bytes) {
-  const uint32_t lo = ((smem_addr >> 4) & 0x3FFFu) | (((lbo_bytes >> 4) & 0x3FFFu) << 16);
-  const uint32_t hi = ((sbo_bytes >> 4) & 0x3FFFu) | (1u << 14) | (2u << 29);
-  return ((uint64_t)hi << 32) | lo;
-}
-// instruction descriptor: bf16 x bf16 -> fp32, M = 128, A K-major
-__host__ __device__ constexpr uint32_t umma_idesc(int n, bool b_mn_major) {
-  return (1u << 4) | (1u << 7) | (1u << 10) | ((b_mn_major ? 1u : 0u) << 16) | ((uint32_t)(n >> 3) << 17) |
-         ((uint32_t)(kUmmaRows >> 4) << 24);
-}
-__device__ __forceinline__ void umma_bf16(uint32_t tmem_d, uint64_t a_desc, uint64_t b_desc, uint32_t idesc,
-                                          uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
-      :
-      : "r"(tmem_d), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate), "r"(0u)
-      : "memory");
-}
-// A operand in tensor memory (128 lanes x 8 columns of packed bf16 pairs per 16-wide k-step)
-__device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t b_desc, uint32_t idesc,
-                                             uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, {%5, %5, %5, %5}, p;\n\t}"
-      :
-      : "r"(tmem_d), "r"(tmem_a), "l"(b_desc), "r"(idesc), "r"(accumulate), "r"(0u)
-      : "memory");
-}
-// Blackwell's two-wide fp32 arithmetic and three-input maximum: a row of 64 scores takes 32 instructions
-// for the maximum, 32 for scale-and-shift and 32 for the row sum instead of 64 each - the softmax
-// warps share their schedulers' issue slots with each other and the exp2 unit is the pipe to keep busy.
-__device__ __forceinline__ float max3(float a, float b, float c) {
-  float d;
-  asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
-  return d;
-}
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
-  uint64_t d;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-// 2^x for two values at once on the FMA pipe (any x; below -126 the result is 2^-126): round to the
-// nearest integer with the 1.5 * 2^23 trick, a degree-3 polynomial for 2^f on [-0.5, 0.5] (relative error
-// 1e-4, a twentieth of the bf16 rounding of P) and the integer part added into the exponent field.
-__device__ __forceinline__ void exp2_poly2(float x0, float x1, float& p0, float& p1) {
-  const uint32_t kMagic = 0x4B400000u, kNegMagic = 0xCB400000u, kNegOne = 0xBF800000u;  // 1.5 * 2^23, -1.5 * 2^23, -1.0
-  x0 = fmaxf(x0, -126.f);
-  x1 = fmaxf(x1, -126.f);
-  uint64_t x, r, f, q;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(x) : "r"(__float_as_uint(x0)), "r"(__float_as_uint(x1)));
-  uint64_t magic, neg_magic, neg_one, c0, c1, c2, c3;
-  asm("mov.b64 %0, {%1, %1};" : "=l"(magic) : "r"(kMagic));
-  asm("mov.b64 %0, {%1, %1};" : "=l"(neg_magic) : "r"(kNegMagic));
-  asm("mov.b64 %0, {%1, %1};" : "=l"(neg_one) : "r"(kNegOne));
-  asm("mov.b64 %0, {%1, %1};" : "=l"(c0) : "r"(__float_as_uint(0.9999281764f)));
-  asm("mov.b64 %0, {%1, %1};" : "=l"(c1) : "r"(__float_as_uint(0.6932609677f)));
-  asm("mov.b64 %0, {%1, %1};" : "=l"(c2) : "r"(__float_as_uint(0.2426091731f)));
-  asm("mov.b64 %0, {%1, %1};" : "=l"(c3) : "r"(__float_as_uint(0.05517086014f)));
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(x), "l"(magic));  // low mantissa bits: the rounded integer
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(f) : "l"(r), "l"(neg_magic));
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(f) : "l"(f), "l"(neg_one), "l"(x));  // x - round(x)
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(q) : "l"(c3), "l"(f), "l"(c2));
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(q) : "l"(q), "l"(f), "l"(c1));
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(q) : "l"(q), "l"(f), "l"(c0));
-  uint32_t r0, r1, q0, q1;
-  asm("mov.b64 {%0, %1}, %2;" : "=r"(r0), "=r"(r1) : "l"(r));
-  asm("mov.b64 {%0, %1}, %2;" : "=r"(q0), "=r"(q1) : "l"(q));
-  p0 = __uint_as_float(q0 + (r0 << 23));
-  p1 = __uint_as_float(q1 + (r1 << 23));
-}
-// The same with a degree-5 polynomial (minimax for the relative error on [-0.5, 0.5], found with the Remez exchange:
-// 7e-8, 2.4e-7 with fp32 arithmetic): weights that are split keep what this gives them.
-__device__ __forceinline__ void exp2_poly2_fine(float x0, float x1, float& p0, float& p1) {
-  x0 = fmaxf(x0, -126.f);
-  x1 = fmaxf(x1, -126.f);
-  uint64_t x, r, f, q;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(x) : "r"(__float_as_uint(x0)), "r"(__float_as_uint(x1)));
-  auto both = [](float v) {
-    uint64_t d;
-    asm("mov.b64 %0, {%1, %1};" : "=l"(d) : "r"(__float_as_uint(v)));
-    return d;
-  };
-  r = add2(x, both(12582912.0f));        // 1.5 * 2^23: the low mantissa bits are the rounded integer
-  f = add2(r, both(-12582912.0f));
-  f = fma2(f, both(-1.0f), x);           // x - round(x)
-  q = fma2(both(0.0013276472632f), f, both(0.0096755413431f));
-  q = fma2(q, f, both(0.0555071327186f));
-  q = fma2(q, f, both(0.2402211972371f));
-  q = fma2(q, f, both(0.6931469670651f));
-  q = fma2(q, f, both(1.0000000716547f));
-  uint32_t r0, r1, q0, q1;
-  asm("mov.b64 {%0, %1}, %2;" : "=r"(r0), "=r"(r1) : "l"(r));
-  asm("mov.b64 {%0, %1}, %2;" : "=r"(q0), "=r"(q1) : "l"(q));
-  p0 = __uint_as_float(q0 + (r0 << 23));
-  p1 = __uint_as_float(q1 + (r1 << 23));
-}
-__device__ __forceinline__ void unpack64(uint64_t v, uint32_t& lo, uint32_t& hi) {
-  asm("mov.b64 {%0, %1}, %2;" : "=r"(lo), "=r"(hi) : "l"(v));
-}
-__device__ __forceinline__ uint64_t pack64(uint32_t lo, uint32_t hi) {
-  uint64_t d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "r"(lo), "r"(hi));
-  return d;
-}
-// arrive on an mbarrier once every tcgen05.mma issued so far by this thread has completed
-__device__ __forceinline__ void umma_commit(uint64_t* bar) {
-  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar))
-               : "memory");
-}
-// 32 TMEM lanes (this warp's) x 32 consecutive 32-bit columns -> 32 registers per thread
-__device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
-      "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]),
-        "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]),
-        "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-      : "r"(taddr));
-}
-__device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t (&r)[32]) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, "
-      "%17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};" ::"r"(taddr),
-      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]),
-      "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]),
-      "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]),
-      "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
-      : "memory");
-}
-__device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x16.b32 "
-      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
-      : "r"(taddr));
-}
-__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16]) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
-      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};" ::"r"(taddr),
-      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]),
-      "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
-      : "memory");
-}
-__device__ __forceinline__ void tmem_ld2(uint32_t taddr, uint32_t& r0, uint32_t& r1) {
-  asm volatile("tcgen05.ld.sync.aligned.32x32b.x2.b32 {%0, %1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(taddr));
-}
-__device__ __forceinline__ void tmem_st2(uint32_t taddr, uint32_t r0, uint32_t r1) {
-  asm volatile("tcgen05.st.sync.aligned.32x32b.x2.b32 [%0], {%1, %2};" ::"r"(taddr), "r"(r0), "r"(r1) : "memory");
-}
-__device__ __forceinline__ void tmem_wait_ld() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ void tmem_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-
 // Bounded wait that also gives up when another role has raised the abort flag.  Called by whole
 // warps; the answer is the same for every lane (the tcgen05 instructions that follow are .aligned).
 __device__ __forceinline__ bool umma_wait(uint64_t* bar, uint32_t parity, volatile int* abort) {
@@ -267,8 +97,6 @@ __device__ __forceinline__ bool umma_wait(uint64_t* bar, uint32_t parity, volati
 //               into registers, issue QK(i)
 //   PV issuer:  wait P(i), issue PV(i), release the ring stage and the group's O / P
 // so a group's next scores are computed while it works on the current ones.
-constexpr uint32_t kDescHi = (1024u >> 4) | (1u << 14) | (2u << 29);  // SBO 1024 B, version 1, 128-byte swizzle
-
 // The issuer warps run their loops with all 32 lanes in step and one elected lane issuing: every value
 // an MMA takes (descriptors, tensor-memory addresses) then depends only on votes and loop counters, which
 // the compiler can keep in the uniform datapath the instruction reads its operands from.  With a single
@@ -282,12 +110,6 @@ __device__ __forceinline__ bool issuer_wait(const UmmaCtx& c, uint64_t* bar, uin
   *c.abort = 1;
   return false;
 }
-__device__ __forceinline__ bool elect_one() {
-  uint32_t pred;
-  asm volatile("{\n\t.reg .pred p;\n\telect.sync _|p, 0xffffffff;\n\tselp.u32 %0, 1, 0, p;\n\t}" : "=r"(pred));
-  return pred != 0;
-}
-
 // Narrow form: mine = 0 / 1, this warp issues the QK of group A's / B's chunks (the loop's fixed cost -
 // barrier waits, votes, fences, the commit - is about as long as the MMAs themselves, and one warp walking
 // every chunk paced the whole pipeline).

@@ -80,13 +80,16 @@ struct KVView {
   int32_t n_pages;
 };
 
+// row planes of a layer: keys and values, or one that is both
+__host__ __device__ inline int pool_planes(const pace_kv_pool_t& p) { return p.row_format == PACE_ROWS_SHARED ? 1 : 2; }
+
 inline KVView make_view(const pace_kv_pool_t* p, int layer, const int32_t* seq_ids) {
   KVView v;
   const size_t page_elems = (size_t)p->n_kv_heads * p->page_tokens * p->head_dim;
   const size_t region = page_elems * (size_t)p->n_pages;
   const __nv_bfloat16* base = (const __nv_bfloat16*)p->pages;
-  v.k = base + ((size_t)layer * 2 + 0) * region;
-  v.v = base + ((size_t)layer * 2 + 1) * region;
+  v.k = base + (size_t)layer * pool_planes(*p) * region;
+  v.v = v.k + (pool_planes(*p) - 1) * region;
   v.block_table = p->block_table;
   v.seq_ids = seq_ids;
   v.slot_base = 0;

@@ -6,12 +6,32 @@ namespace pace {
 namespace {
 
 // ---------------------------------------------------------------------------
-// x' = x + rms(y) w_post (+ embedding row);  h = rms(x') w_next
+// x' = x + rms(y) w_post (+ embedding row);  h = rms(x') w_next, or x' itself
+// MOE: y is the weighted sum of the rows of the token's experts
 // ---------------------------------------------------------------------------
-template <typename T, int V, int ITEMS>
+constexpr int kMaxTop = 64;
+
+template <typename T, int V, int ITEMS, bool MOE>
 __global__ void __launch_bounds__(512) residual_norm_kernel(pace_step_t st, pace_residual_norm_args_t a) {
   __shared__ float red[32];
+  __shared__ int e_row[MOE ? kMaxTop : 1];
+  __shared__ float e_w[MOE ? kMaxTop : 1];
   const int t = blockIdx.x, W = a.width;
+  if constexpr (MOE) {
+    // one warp per chosen expert: the expert's first row is the number of tokens of all experts in front of it
+    for (int k = threadIdx.x >> 5; k < a.top; k += blockDim.x >> 5) {
+      const int e = a.slot_expert[(size_t)t * a.top + k];
+      int n = 0;
+      for (int i = threadIdx.x & 31; i < e; i += 32) n += a.expert_count[i];
+#pragma unroll
+      for (int o = 16; o; o >>= 1) n += __shfl_xor_sync(0xffffffffu, n, o);
+      if ((threadIdx.x & 31) == 0) {
+        e_row[k] = n + a.slot_rank[(size_t)t * a.top + k];
+        e_w[k] = a.slot_weight[(size_t)t * a.top + k];
+      }
+    }
+    __syncthreads();
+  }
   float xv[ITEMS][V], yv[ITEMS][V];
   float* x = a.x + (size_t)t * W;
   const T* y = a.y ? static_cast<const T*>(a.y) + (size_t)t * a.y_stride : nullptr;
@@ -29,8 +49,19 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(pace_step_t st, pace
       else
 #pragma unroll
         for (int j = 0; j < V; ++j) xv[i][j] = 0.f;
-      if (y) {
+      if (MOE) {
+#pragma unroll
+        for (int j = 0; j < V; ++j) yv[i][j] = 0.f;
+        for (int k = 0; k < a.top; ++k) {
+          float r[V];
+          Vec<T, V>::load(static_cast<const T*>(a.y) + (size_t)e_row[k] * a.y_stride + c, r);
+#pragma unroll
+          for (int j = 0; j < V; ++j) yv[i][j] = fmaf(e_w[k], r[j], yv[i][j]);
+        }
+      } else if (y) {
         Vec<T, V>::load(y + c, yv[i]);
+      }
+      if (y) {
 #pragma unroll
         for (int j = 0; j < V; ++j) ss += yv[i][j] * yv[i][j];
       }
@@ -59,16 +90,24 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(pace_step_t st, pace
         float e[V];
         Vec<T, V>::load(em + c, e);
 #pragma unroll
-        for (int j = 0; j < V; ++j) xv[i][j] += e[j];
+        for (int j = 0; j < V; ++j) xv[i][j] = fmaf(e[j], a.embed_scale, xv[i][j]);
       }
       Vec<float, V>::store(x + c, xv[i]);
 #pragma unroll
       for (int j = 0; j < V; ++j) ss += xv[i][j] * xv[i][j];
     }
   }
-  if (!a.w_next) return;
-  const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)W + a.eps);
+  if (!a.h) return;
   T* h = static_cast<T*>(a.h) + (size_t)t * W;
+  if (!a.w_next) {
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * V;
+      if (c < W) Vec<T, V>::store(h + c, xv[i]);
+    }
+    return;
+  }
+  const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)W + a.eps);
 #pragma unroll
   for (int i = 0; i < ITEMS; ++i) {
     const int c = (i * blockDim.x + threadIdx.x) * V;
@@ -97,14 +136,20 @@ template <typename T, int V>
 int launch_residual_norm(const pace_step_t& st, const pace_residual_norm_args_t& a, cudaStream_t s) {
   int threads = 0;
   const int items = row_items((a.width + V - 1) / V, &threads);
+#define PACE_NORM_CASE(n)                                                                          \
+  case n:                                                                                          \
+    if (a.top > 0) residual_norm_kernel<T, V, n, true><<<st.n_tokens, threads, 0, s>>>(st, a);     \
+    else residual_norm_kernel<T, V, n, false><<<st.n_tokens, threads, 0, s>>>(st, a);              \
+    break;
   switch (items) {
-    case 1: residual_norm_kernel<T, V, 1><<<st.n_tokens, threads, 0, s>>>(st, a); break;
-    case 2: residual_norm_kernel<T, V, 2><<<st.n_tokens, threads, 0, s>>>(st, a); break;
-    case 4: residual_norm_kernel<T, V, 4><<<st.n_tokens, threads, 0, s>>>(st, a); break;
-    case 8: residual_norm_kernel<T, V, 8><<<st.n_tokens, threads, 0, s>>>(st, a); break;
-    case 16: residual_norm_kernel<T, V, 16><<<st.n_tokens, threads, 0, s>>>(st, a); break;
+    PACE_NORM_CASE(1)
+    PACE_NORM_CASE(2)
+    PACE_NORM_CASE(4)
+    PACE_NORM_CASE(8)
+    PACE_NORM_CASE(16)
     default: return PACE_ERR_UNSUPPORTED;
   }
+#undef PACE_NORM_CASE
   PACE_LAUNCH_CHECK("residual_norm_kernel");
   return PACE_OK;
 }
@@ -291,6 +336,55 @@ __global__ void __launch_bounds__(512) append_norm_regs_kernel(pace_step_t st, P
     }
 }
 
+// Per-head norms without weights: a warp per head row of (queries, keys, values).
+template <typename T, int V>
+__global__ void append_heads_kernel(pace_step_t st, PageRows pg, pace_append_norm_args_t a, int row) {
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int H = a.n_q_heads, G = pg.n_kv_heads, d = a.dim, vd = a.vdim;
+  const T* src = static_cast<const T*>(a.qkv) + (size_t)t * a.qkv_stride;
+  const int pos = st.tok_pos[t], slot = st.slot[st.tok_entry[t]], lp = pos / pg.page_tokens;
+  int page = -1;
+  if (slot >= 0 && slot < pg.max_seqs && lp < pg.max_pages_per_seq)
+    page = pg.block_table[(size_t)slot * pg.max_pages_per_seq + lp];
+  if (page < 0 || page >= pg.n_pages) {
+    if (threadIdx.x == 0) raise_status(pg.status, PACE_DEV_BAD_INDEX);
+    page = -1;
+  }
+  float temp = a.q_mul;
+  if (a.temp_coef != 0.f) temp *= 1.0f + a.temp_coef * logf((float)(floor((double)(pos + 1) / a.temp_every) + 1.0));
+  for (int hh = threadIdx.x >> 5; hh < H + 2 * G; hh += warps) {
+    const bool is_q = hh < H, is_v = hh >= H + G;
+    const int g = is_v ? hh - H - G : hh - H, n = is_v ? vd : d;
+    const T* x = src + (is_q ? hh * d : is_v ? H * d + G * d + g * vd : H * d + g * d);
+    T* dst;
+    if (is_q) dst = static_cast<T*>(a.q_out) + ((size_t)t * H + hh) * row;
+    else dst = reinterpret_cast<T*>(is_v ? pg.v : pg.k) +
+               (((size_t)(page < 0 ? 0 : page) * G + g) * pg.page_tokens + (pos - lp * pg.page_tokens)) * row;
+    float f = 1.f;
+    if (!is_v) {
+      float ss = 0.f;
+      for (int c = lane * V; c < n; c += 32 * V) {
+        float v[V];
+        Vec<T, V>::load(x + c, v);
+#pragma unroll
+        for (int j = 0; j < V; ++j) ss = fmaf(v[j], v[j], ss);
+      }
+#pragma unroll
+      for (int o = 16; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      f = 1.0f / sqrtf(ss / (float)n + a.eps);
+      if (is_q) f *= temp;
+    }
+    if (!is_q && page < 0) continue;
+    for (int c = lane * V; c < row; c += 32 * V) {
+      float v[V];
+      if (c < n) Vec<T, V>::load(x + c, v);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] = c < n ? v[j] * f : 0.f;
+      Vec<T, V>::store(dst + c, v);
+    }
+  }
+}
+
 template <typename T>
 int launch_append_norm(const pace_kv_pool_t* p, int layer, const pace_step_t& st, const pace_append_norm_args_t& a,
                        cudaStream_t s) {
@@ -310,6 +404,17 @@ int launch_append_norm(const pace_kv_pool_t* p, int layer, const pace_step_t& st
   constexpr int V = 16 / sizeof(T);
   const bool vec = a.dim % V == 0 && a.vdim % V == 0 && row % V == 0 && a.qkv_stride % V == 0 && aligned16(a.qkv) &&
                    aligned16(a.q_out) && (!a.q_norm || aligned16(a.q_norm)) && (!a.k_norm || aligned16(a.k_norm));
+  if (a.per_head) {
+    const int heads = a.n_q_heads + 2 * p->n_kv_heads, th = heads < 16 ? heads * 32 : 512;
+    constexpr int V4 = 4;  // 8-byte accesses of bf16: a head of 128 fills a warp
+    const bool v4 = a.dim % V4 == 0 && a.vdim % V4 == 0 && row % V4 == 0 && a.qkv_stride % V4 == 0 && aligned16(a.qkv) &&
+                    aligned16(a.q_out);
+    if (v4) append_heads_kernel<T, V4><<<st.n_tokens, th, 0, s>>>(st, pg, a, row);
+    else append_heads_kernel<T, 1><<<st.n_tokens, th, 0, s>>>(st, pg, a, row);
+    PACE_LAUNCH_CHECK("append_heads_kernel");
+    note_pool_write(s);
+    return PACE_OK;
+  }
   const int groups = (a.n_q_heads + 2 * p->n_kv_heads) * row / (vec ? V : 1);
   const int threads = groups < 512 ? (groups + 31) / 32 * 32 : 512;
   const int n_vec = (a.n_q_heads * a.dim + p->n_kv_heads * (a.dim + a.vdim)) / V;
@@ -388,6 +493,21 @@ __global__ void relu_squared_kernel(T* __restrict__ x, int64_t n) {
   }
 }
 
+template <typename T, int V, int ACT>
+__global__ void glu_kernel(const T* __restrict__ x, int64_t xs, T* __restrict__ out, int n_tokens, int n) {
+  const int per = n / V;
+  const size_t total = (size_t)n_tokens * per;
+  for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const int t = (int)(i / per), c = (int)(i % per) * V;
+    float g[V], u[V];
+    Vec<T, V>::load(x + (size_t)t * xs + c, g);
+    Vec<T, V>::load(x + (size_t)t * xs + n + c, u);
+#pragma unroll
+    for (int j = 0; j < V; ++j) u[j] *= ACT == PACE_ACT_SILU ? silu_t<T>(g[j]) : gelu_tanh_t<T>(g[j]);
+    Vec<T, V>::store(out + (size_t)t * n + c, u);
+  }
+}
+
 unsigned elementwise_blocks(size_t threads_wanted) {
   size_t b = (threads_wanted + 255) / 256;
   return (unsigned)(b < 1 ? 1 : b > 148 * 16 ? 148 * 16 : b);
@@ -441,6 +561,18 @@ int relu_squared_t(void* x, int64_t n, cudaStream_t s) {
   return PACE_OK;
 }
 
+template <typename T, int ACT>
+int glu_t(const void* x, int64_t xs, void* out, int n_tokens, int n, cudaStream_t s) {
+  constexpr int V = 16 / sizeof(T);
+  const size_t total = (size_t)n_tokens * n;
+  if (n % V == 0 && xs % V == 0 && aligned16(x) && aligned16(out))
+    glu_kernel<T, V, ACT><<<elementwise_blocks(total / V), 256, 0, s>>>((const T*)x, xs, (T*)out, n_tokens, n);
+  else
+    glu_kernel<T, 1, ACT><<<elementwise_blocks(total), 256, 0, s>>>((const T*)x, xs, (T*)out, n_tokens, n);
+  PACE_LAUNCH_CHECK("glu_kernel");
+  return PACE_OK;
+}
+
 bool dtype_ok(int dtype) { return dtype == PACE_DTYPE_BF16 || dtype == PACE_DTYPE_FP32; }
 
 }  // namespace
@@ -453,6 +585,9 @@ extern "C" {
 int pace_residual_norm(const pace_step_t* st, const pace_residual_norm_args_t* a, void* stream) {
   if (!step_ok(st) || !a || !a->x || a->width < 1 || !dtype_ok(a->dtype)) return PACE_ERR_INVALID;
   if ((a->w_next && !a->h) || (a->embed && a->vocab < 1) || (a->y && a->y_stride < a->width)) return PACE_ERR_INVALID;
+  if (a->top < 0 || (a->top > 0 && (!a->y || a->top > kMaxTop || a->n_experts < a->top || !a->slot_expert || !a->slot_rank ||
+                                    !a->slot_weight || !a->expert_count)))
+    return PACE_ERR_INVALID;
   if (st->n_tokens == 0) return PACE_OK;
   PACE_PROFILE("residual_norm", stream, "tokens=%d width=%d", st->n_tokens, a->width);
   const cudaStream_t s = (cudaStream_t)stream;
@@ -468,6 +603,8 @@ int pace_kv_append_norm(const pace_kv_pool_t* p, int32_t layer, const pace_step_
                         void* stream) {
   if (!p || !p->pages || !p->block_table || !step_ok(st) || !a || layer < 0 || layer >= p->n_layers) return PACE_ERR_INVALID;
   if (!a->qkv || !a->q_out || a->n_q_heads < 1 || a->dim < 1 || a->vdim < 1 || !dtype_ok(a->dtype)) return PACE_ERR_INVALID;
+  if (p->row_format == PACE_ROWS_SHARED) return PACE_ERR_UNSUPPORTED;
+  if (a->per_head && (a->q_norm || a->k_norm)) return PACE_ERR_INVALID;
   if (a->n_q_heads % p->n_kv_heads || (a->temp_coef != 0.f && !(a->temp_every > 0.0))) return PACE_ERR_INVALID;
   if (p->row_format == PACE_ROWS_BF16 && a->dtype != PACE_DTYPE_BF16) return PACE_ERR_INVALID;
   if (st->n_tokens == 0) return PACE_OK;
@@ -497,6 +634,18 @@ int pace_relu_squared(void* x, int64_t n, int32_t dtype, void* stream) {
   if (n == 0) return PACE_OK;
   return dtype == PACE_DTYPE_BF16 ? relu_squared_t<__nv_bfloat16>(x, n, (cudaStream_t)stream)
                                   : relu_squared_t<float>(x, n, (cudaStream_t)stream);
+}
+
+int pace_glu(const void* x, int64_t x_stride, void* out, int32_t n_tokens, int32_t n, int32_t act, int32_t dtype, void* stream) {
+  if (!x || !out || n_tokens < 0 || n < 1 || x_stride < 2 * (int64_t)n || !dtype_ok(dtype)) return PACE_ERR_INVALID;
+  if (act != PACE_ACT_SILU && act != PACE_ACT_GELU_TANH) return PACE_ERR_INVALID;
+  if (n_tokens == 0) return PACE_OK;
+  const cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == PACE_DTYPE_BF16)
+    return act == PACE_ACT_SILU ? glu_t<__nv_bfloat16, PACE_ACT_SILU>(x, x_stride, out, n_tokens, n, s)
+                                : glu_t<__nv_bfloat16, PACE_ACT_GELU_TANH>(x, x_stride, out, n_tokens, n, s);
+  return act == PACE_ACT_SILU ? glu_t<float, PACE_ACT_SILU>(x, x_stride, out, n_tokens, n, s)
+                              : glu_t<float, PACE_ACT_GELU_TANH>(x, x_stride, out, n_tokens, n, s);
 }
 
 int pace_step_decode(int32_t* token, int32_t* tok_pos, int32_t* start, const int64_t* next, const int64_t* pos, int32_t n,

@@ -56,7 +56,7 @@ bool geometry_ok(const pace_kv_pool_t* g) {
   if (g->n_layers <= 0 || g->n_kv_heads <= 0 || g->page_tokens <= 0 || g->n_pages <= 0 || g->max_seqs <= 0 ||
       g->max_pages_per_seq <= 0)
     return false;
-  if (g->row_format == PACE_ROWS_OPAQUE) return g->head_dim > 0 && g->head_dim % 8 == 0 && g->head_dim <= 2048;
+  if (g->row_format == PACE_ROWS_OPAQUE || g->row_format == PACE_ROWS_SHARED) return g->head_dim > 0 && g->head_dim % 8 == 0 && g->head_dim <= 2048;
   return g->row_format == PACE_ROWS_BF16 && (g->head_dim == 64 || g->head_dim == 128);
 }
 
@@ -180,7 +180,7 @@ __global__ void reserve_kernel(pace_kv_pool_t p, int layer, const int32_t* __res
   for (int c = 0; c < nc; ++c) {
     const int src = cow[3 * c], dst = cow[3 * c + 1], rows = cow[3 * c + 2];
     const size_t per_head = (size_t)rows * vec_per_row;
-    const size_t total = (size_t)p.n_layers * 2 * p.n_kv_heads * per_head;
+    const size_t total = (size_t)p.n_layers * pool_planes(p) * p.n_kv_heads * per_head;
     for (size_t i = threadIdx.x; i < total; i += blockDim.x) {
       const size_t lk = i / (p.n_kv_heads * per_head);
       const size_t rem = i % (p.n_kv_heads * per_head);
@@ -726,7 +726,7 @@ const char* pace_version(void) { return "pace_b200 0.1 (sm_100a)"; }
 
 int pace_kv_pool_bytes(const pace_kv_pool_t* g, uint64_t* pages_bytes, uint64_t* meta_bytes) {
   if (!geometry_ok(g) || !pages_bytes || !meta_bytes) return PACE_ERR_INVALID;
-  *pages_bytes = (uint64_t)g->n_layers * 2 * g->n_pages * g->n_kv_heads * g->page_tokens * g->head_dim * 2;
+  *pages_bytes = (uint64_t)g->n_layers * pool_planes(*g) * g->n_pages * g->n_kv_heads * g->page_tokens * g->head_dim * 2;
   *meta_bytes = meta_layout(g).total;
   return PACE_OK;
 }

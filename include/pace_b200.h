@@ -399,10 +399,14 @@ int pace_linear_skinny(const void* x, int64_t x_stride, const void* w, int64_t w
  * PACE_ROWS_BF16: K and V rows are head_dim bf16 values, head_dim 64 or 128; every entry point takes them.
  * PACE_ROWS_OPAQUE: rows are head_dim 16-bit units of any content (head_dim a multiple of 8, at most 2048):
  * fp32 rows, other head sizes.  The allocator's entry points (reserve, release, truncate, gather,
- * append_layers without rows, query), pace_kv_append_norm and pace_attn_general take them; the rest answers
- * PACE_ERR_UNSUPPORTED. */
+ * append_layers without rows, query), pace_kv_append_norm, pace_attn_general and pace_attn_span take them; the rest
+ * answers PACE_ERR_UNSUPPORTED.
+ * PACE_ROWS_SHARED: as PACE_ROWS_OPAQUE, but a layer has one row per token and head, which is its key and, with its
+ * first elements, its value (latents): pages are [layer][page][kv_head][page_tokens][head_dim], half the memory.
+ * pace_kv_append_norm does not take them (pace_latent_append writes them). */
 #define PACE_ROWS_BF16 0
 #define PACE_ROWS_OPAQUE 1
+#define PACE_ROWS_SHARED 2
 
 /* The tokens of one step.  Entry e (a sequence that takes part) owns rows [cu[e], cu[e + 1]); its first
  * token has position start[e]; `slot` is its slot in the pool and in the recurrent states.  A state is
@@ -420,12 +424,15 @@ typedef struct pace_step {
 } pace_step_t;
 
 /* One pass over the residual stream x (fp32 [n_tokens][width]) between two sublayers:
- *     x' = (restart ? 0 : x) + rms(y) * w_post + (embed ? embed[token] : 0)
+ *     x' = (restart ? 0 : x) + rms(y) * w_post + (embed ? embed[token] * embed_scale : 0)
  *     h  = rms(x') * w_next,       rms(z) = z / sqrt(mean(z^2) + eps)
  * y (the sublayer's output) may be NULL, embed may be NULL (with restart and embed it is the embedding
  * lookup in front of the first layer; with y and embed the re-injection of the embeddings between two
- * passes of a loop), w_next / h may be NULL.  w_post == NULL adds y as it is.  Norm weights are fp32
- * [width] and used as weight_offset + w (1 for "one plus weight" norms).  embed is dtype [vocab][width]. */
+ * passes of a loop), w_next / h may be NULL; h without w_next takes x' as it is (sublayers that read the stream
+ * itself).  w_post == NULL adds y as it is.  Norm weights are fp32 [width] and used as weight_offset + w (1 for
+ * "one plus weight" norms).  embed is dtype [vocab][width].
+ * With `top` > 0, y holds the rows of a mixture's experts (pace_moe_experts) and the sublayer's output of token t is
+ *     sum over k < top of slot_weight[t][k] * y[expert_row(slot_expert[t][k], slot_rank[t][k])]. */
 typedef struct {
   float* x;
   const void* y;
@@ -435,7 +442,12 @@ typedef struct {
   void* h;
   int64_t y_stride;
   int32_t width, vocab, restart, dtype;
-  float eps, weight_offset;
+  float eps, weight_offset, embed_scale;
+  int32_t top, n_experts;
+  const int32_t* slot_expert;   /* [n_tokens][top], with top > 0 */
+  const int32_t* slot_rank;     /* [n_tokens][top] */
+  const float* slot_weight;     /* [n_tokens][top] */
+  const int32_t* expert_count;  /* [n_experts] */
 } pace_residual_norm_args_t;
 int pace_residual_norm(const pace_step_t* step, const pace_residual_norm_args_t* a, void* stream);
 
@@ -445,7 +457,9 @@ int pace_residual_norm(const pace_step_t* step, const pace_residual_norm_args_t*
  * to q_out rows [q_row][n_q_heads][row elements], keys and values into the pages of pool layer `layer` at
  * positions tok_pos.  The pages must be reserved; lengths are left alone (pace_kv_append_layers without rows
  * advances them).  qkv is dtype [n_tokens][qkv_stride]: q (n_q_heads x dim), k (kv_heads x dim), v (kv_heads
- * x vdim).  A pool row holds max(dim, vdim) or more elements; what a row has beyond dim / vdim is zeroed. */
+ * x vdim).  A pool row holds max(dim, vdim) or more elements; what a row has beyond dim / vdim is zeroed.
+ * per_head: the norms are taken over each head's dim elements instead, without weights (q_norm and k_norm NULL), and
+ * row t of q_out belongs to token t (no staging rows). */
 typedef struct {
   const void* qkv;
   int64_t qkv_stride;
@@ -455,6 +469,7 @@ typedef struct {
   int32_t n_q_heads, dim, vdim, dtype;
   float eps, q_mul, temp_coef;
   double temp_every;
+  int32_t per_head;
 } pace_append_norm_args_t;
 int pace_kv_append_norm(const pace_kv_pool_t* pool, int32_t layer, const pace_step_t* step,
                         const pace_append_norm_args_t* a, void* stream);
@@ -464,6 +479,136 @@ int pace_kv_append_norm(const pace_kv_pool_t* pool, int32_t layer, const pace_st
  * (pace_attn_decode / pace_attn_prefill) take the PACE_ROWS_BF16 pools. */
 int pace_attn_general(const pace_kv_pool_t* pool, int32_t layer, const pace_step_t* step, const void* q, void* out,
                       int32_t n_q_heads, int32_t dim, int32_t vdim, float scale, int32_t dtype, void* stream);
+
+/* Causal softmax attention with a span, a distance bias and a sink, for entries [entry_begin, entry_end) of a step.
+ * The query at position i sees key j <= i
+ *     PACE_SPAN_ALL     always,
+ *     PACE_SPAN_WINDOW  if i - j < span_size,
+ *     PACE_SPAN_CHUNK   if i / span_size == j / span_size (integer division, counted from position 0),
+ * its score is scale * (q . k) - slopes[h] * (i - j) (slopes NULL: no bias), and exp(sinks[h]) is added to the
+ * denominator (sinks NULL: ordinary softmax).  Query head h reads KV head h / (n_q_heads / n_kv_heads).
+ * Row t of q (dtype [n_tokens][n_q_heads][q_elems], dim elements used, zero up to the next multiple of 8) and of out
+ * ([n_tokens][n_q_heads][out_elems], vdim elements written) belongs to token t.  The pool holds the step's own rows already;
+ * lengths come from the step.  PACE_ROWS_SHARED pools: the value is the first vdim elements of the key row.
+ * Scores, weights and sums are fp32 (with bf16 rows the weights enter the second product as two bf16 terms).
+ * max_tokens / max_keys: upper bounds, over the entries, of their tokens and of their last position + 1.
+ * bf16: tensor cores (mma.sync), the keys of a query tile split over a thread-block cluster; fp32 and what does not fit
+ * that kernel: the CUDA-core kernel of pace_attn_general.  dim, vdim <= 640, 512. */
+#define PACE_SPAN_ALL 0
+#define PACE_SPAN_WINDOW 1
+#define PACE_SPAN_CHUNK 2
+typedef struct {
+  const void* q;
+  void* out;
+  const float* slopes;   /* fp32 [n_q_heads] or NULL */
+  const float* sinks;    /* fp32 [n_q_heads] or NULL */
+  int32_t n_q_heads, dim, vdim, dtype, q_elems, out_elems;
+  int32_t entry_begin, entry_end, max_tokens, max_keys;
+  int32_t span, span_size;
+  float scale;
+} pace_attn_span_args_t;
+int pace_attn_span(const pace_kv_pool_t* pool, int32_t layer, const pace_step_t* step, const pace_attn_span_args_t* a,
+                   void* stream);
+
+/* The same attention for prompts on the tcgen05 tensor cores (bf16): 256 query rows of one (entry, KV head) per thread
+ * block, K and V tiles by TMA.  Keys come from the pool (k NULL; PACE_ROWS_BF16), or from plain tensors of expanded
+ * rows: the keys of entry e are rows key_cu[e - entry_begin] .. key_cu[e - entry_begin + 1] - 1, of which the first has
+ * position key_pos[e - entry_begin]; a key is k[row][head][0 .. k_dim) followed by k2[row][0 .. k2_dim) shared by all heads
+ * (k2_dim may be 0), a value v[row][head][0 .. vdim).  Queries then are [0, k_dim) | [k_dim, k_dim + k2_dim).
+ * Answers PACE_ERR_UNSUPPORTED (nothing launched) for shapes it does not take: sizes and strides that are not
+ * multiples of 8, more than 256 key or 128 value elements (rounded up to 64 per part). */
+typedef struct {
+  pace_attn_span_args_t a;
+  const void* k;
+  const void* k2;
+  const void* v;
+  int64_t k_row, k_head, k2_row, v_row, v_head;   /* strides in elements */
+  int32_t k_dim, k2_dim, n_kv_heads, n_rows;
+  const int32_t* key_cu;    /* device, [entry_end - entry_begin + 1] */
+  const int32_t* key_pos;   /* device, [entry_end - entry_begin] */
+} pace_attn_span_prefill_args_t;
+int pace_attn_span_prefill(const pace_kv_pool_t* pool, int32_t layer, const pace_step_t* step,
+                           const pace_attn_span_prefill_args_t* a, void* stream);
+
+/* ---- latent attention: what surrounds the products ------------------------------------------------------------------
+ * pace_latent_append: one token's down projections, down [n_tokens][down_stride] = query latent (q_rank) | key/value
+ * latent (kv_rank) | rotated key part (rot_dim):
+ *     cq[t] = rms(query latent) * q_norm                                      (dtype [n_tokens][q_rank]; q_rank 0: none)
+ *     page row of token t = rms(kv latent) * kv_norm | rotate(key part) | 0
+ * rotate turns the pairs (2i, 2i + 1), i < rot_pairs, by the angles whose cosine and sine are cos[pos][i], sin[pos][i]
+ * (fp32 tables of table_rows rows).
+ * pace_rotate_heads: the same rotation for n_heads parts of rot_dim elements per token, src[t][h] -> dst[t][h] (strides in
+ * elements; may be the same place), zeros in dst up to pad_dim elements.
+ * pace_latent_gather: page rows of (slot[i], pos[i]), i < n, into out [n][row elements].
+ * The pool is PACE_ROWS_SHARED with one KV head. */
+typedef struct {
+  const void* down;
+  int64_t down_stride;
+  const float* q_norm;
+  const float* kv_norm;
+  const float* cos_table;
+  const float* sin_table;
+  void* cq;
+  int32_t q_rank, kv_rank, rot_dim, rot_pairs, table_rows, dtype;
+  float eps;
+} pace_latent_append_args_t;
+int pace_latent_append(const pace_kv_pool_t* pool, int32_t layer, const pace_step_t* step,
+                       const pace_latent_append_args_t* a, void* stream);
+typedef struct {
+  const void* src;
+  void* dst;
+  int64_t src_row, src_head, dst_row, dst_head;
+  const float* cos_table;
+  const float* sin_table;
+  int32_t token_begin, token_end, n_heads, rot_dim, rot_pairs, pad_dim, table_rows, dtype;
+} pace_rotate_args_t;
+int pace_rotate_heads(const pace_step_t* step, const pace_rotate_args_t* a, void* stream);
+int pace_latent_gather(const pace_kv_pool_t* pool, int32_t layer, const int32_t* slot, const int32_t* pos, int32_t n,
+                       void* out, void* stream);
+
+/* ---- gated feed-forwards and mixtures of experts --------------------------------------------------------------------
+ * pace_glu: out[t][i] = act(x[t][i]) * x[t][n + i], x rows of 2 n elements. */
+#define PACE_ACT_SILU 0
+#define PACE_ACT_GELU_TANH 1
+int pace_glu(const void* x, int64_t x_stride, void* out, int32_t n_tokens, int32_t n, int32_t act, int32_t dtype,
+             void* stream);
+
+/* Router: scores = sigmoid(logits) (logits fp32 [n_tokens][n_experts]); the `top` experts with the largest scores +
+ * correction (fp32 [n_experts] or NULL; ties go to the lower index) are chosen, their weights are the scores without
+ * it.  slot_expert / slot_weight [n_tokens][top]; expert_count [n_experts] and slot_rank [n_tokens][top] number the tokens
+ * of an expert, expert_list [n_experts][n_tokens] lists them.  top <= 64, n_experts <= 1024. */
+typedef struct {
+  const float* logits;
+  const float* correction;
+  int32_t* slot_expert;
+  int32_t* slot_rank;
+  float* slot_weight;
+  int32_t* expert_count;
+  int32_t* expert_list;
+  int32_t n_tokens, n_experts, top;
+} pace_moe_route_args_t;
+int pace_moe_route(const pace_moe_route_args_t* a, void* stream);
+
+/* The chosen experts' feed-forwards: for every (token, expert) pair of the router
+ *     hidden = act(gate x) * (up x),  y = down hidden
+ * x dtype [n_tokens][width], gate_up dtype [n_experts][2 ff][width] (gate rows first), down dtype [n_experts][width][ff].
+ * hidden [n_tokens * top][ff] and y [n_tokens * top][width] are written by expert: expert e's token of rank r is row
+ *     expert_row(e, r) = expert_count[0] + .. + expert_count[e - 1] + r.
+ * bf16 with width and ff multiples of 8: grouped products on the tcgen05 tensor cores, weights as the 128-row operand,
+ * the tokens' rows gathered by TMA.  Otherwise CUDA cores.  `status` (device int32, may be NULL) takes
+ * PACE_DEV_WAIT_TIMEOUT if a bounded wait runs out. */
+typedef struct {
+  const void* x;
+  const void* gate_up;
+  const void* down;
+  void* hidden;
+  void* y;
+  const int32_t* expert_count;
+  const int32_t* expert_list;
+  int32_t* status;
+  int32_t n_tokens, n_experts, top, width, ff, act, dtype;
+} pace_moe_experts_args_t;
+int pace_moe_experts(const pace_moe_experts_args_t* a, void* stream);
 
 /* out[t][h * vdim + i] = attn[q_row[t]][h][i] * sigmoid(gate[t][h * vdim + i]);
  * attn rows are [n_heads][row_elems], gate has gate_stride elements per token. */
