@@ -32,8 +32,10 @@ class KVPoolStruct(C.Structure):
                [("row_format", C.c_int32)]
 
 
-ROWS_BF16, ROWS_OPAQUE = 0, 1   # PACE_ROWS_*
+ROWS_BF16, ROWS_OPAQUE, ROWS_SHARED = 0, 1, 2   # PACE_ROWS_*
 DTYPE_BF16, DTYPE_FP32 = 0, 1   # PACE_DTYPE_*
+SPAN_ALL, SPAN_WINDOW, SPAN_CHUNK = 0, 1, 2   # PACE_SPAN_*
+ACT_SILU, ACT_GELU_TANH = 0, 1  # PACE_ACT_*
 
 ATTN_WHOLE_UNITS = 1      # PACE_ATTN_WHOLE_UNITS
 ATTN_PENDING_ROW = 2      # PACE_ATTN_PENDING_ROW
@@ -74,14 +76,55 @@ class StepStruct(C.Structure):
 class ResidualNormArgs(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("x", "y", "w_post", "embed", "w_next", "h")] + [("y_stride", C.c_int64)] + \
                [(n, C.c_int32) for n in ("width", "vocab", "restart", "dtype")] + \
-               [("eps", C.c_float), ("weight_offset", C.c_float)]
+               [("eps", C.c_float), ("weight_offset", C.c_float), ("embed_scale", C.c_float), ("top", C.c_int32),
+                ("n_experts", C.c_int32)] + \
+               [(n, C.c_void_p) for n in ("slot_expert", "slot_rank", "slot_weight", "expert_count")]
 
 
 class AppendNormArgs(C.Structure):
     _fields_ = [("qkv", C.c_void_p), ("qkv_stride", C.c_int64)] + \
                [(n, C.c_void_p) for n in ("q_norm", "k_norm", "q_out")] + \
                [(n, C.c_int32) for n in ("n_q_heads", "dim", "vdim", "dtype")] + \
-               [("eps", C.c_float), ("q_mul", C.c_float), ("temp_coef", C.c_float), ("temp_every", C.c_double)]
+               [("eps", C.c_float), ("q_mul", C.c_float), ("temp_coef", C.c_float), ("temp_every", C.c_double),
+                ("per_head", C.c_int32)]
+
+
+class AttnSpanArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("q", "out", "slopes", "sinks")] + \
+               [(n, C.c_int32) for n in ("n_q_heads", "dim", "vdim", "dtype", "q_elems", "out_elems", "entry_begin", "entry_end",
+                                         "max_tokens", "max_keys", "span", "span_size")] + [("scale", C.c_float)]
+
+
+class AttnSpanPrefillArgs(C.Structure):
+    _fields_ = [("a", AttnSpanArgs)] + [(n, C.c_void_p) for n in ("k", "k2", "v")] + \
+               [(n, C.c_int64) for n in ("k_row", "k_head", "k2_row", "v_row", "v_head")] + \
+               [(n, C.c_int32) for n in ("k_dim", "k2_dim", "n_kv_heads", "n_rows")] + \
+               [("key_cu", C.c_void_p), ("key_pos", C.c_void_p)]
+
+
+class LatentAppendArgs(C.Structure):
+    _fields_ = [("down", C.c_void_p), ("down_stride", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("q_norm", "kv_norm", "cos_table", "sin_table", "cq")] + \
+               [(n, C.c_int32) for n in ("q_rank", "kv_rank", "rot_dim", "rot_pairs", "table_rows", "dtype")] + \
+               [("eps", C.c_float)]
+
+
+class RotateArgs(C.Structure):
+    _fields_ = [("src", C.c_void_p), ("dst", C.c_void_p)] + \
+               [(n, C.c_int64) for n in ("src_row", "src_head", "dst_row", "dst_head")] + \
+               [("cos_table", C.c_void_p), ("sin_table", C.c_void_p)] + \
+               [(n, C.c_int32) for n in ("token_begin", "token_end", "n_heads", "rot_dim", "rot_pairs", "pad_dim", "table_rows",
+                                         "dtype")]
+
+
+class MoeRouteArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("logits", "correction", "slot_expert", "slot_rank", "slot_weight", "expert_count",
+                                          "expert_list")] + [(n, C.c_int32) for n in ("n_tokens", "n_experts", "top")]
+
+
+class MoeExpertsArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("x", "gate_up", "down", "hidden", "y", "expert_count", "expert_list", "status")] + \
+               [(n, C.c_int32) for n in ("n_tokens", "n_experts", "top", "width", "ff", "act", "dtype")]
 
 
 class RglruArgs(C.Structure):
@@ -141,6 +184,14 @@ _SIGS = {
     "pace_kv_append_norm": (C.c_int, [_P, C.c_int32, _S, C.POINTER(AppendNormArgs), C.c_void_p]),
     "pace_attn_general": (C.c_int, [_P, C.c_int32, _S, C.c_void_p, C.c_void_p, C.c_int32, C.c_int32, C.c_int32, C.c_float,
                                     C.c_int32, C.c_void_p]),
+    "pace_attn_span": (C.c_int, [_P, C.c_int32, _S, C.POINTER(AttnSpanArgs), C.c_void_p]),
+    "pace_attn_span_prefill": (C.c_int, [_P, C.c_int32, _S, C.POINTER(AttnSpanPrefillArgs), C.c_void_p]),
+    "pace_latent_append": (C.c_int, [_P, C.c_int32, _S, C.POINTER(LatentAppendArgs), C.c_void_p]),
+    "pace_rotate_heads": (C.c_int, [_S, C.POINTER(RotateArgs), C.c_void_p]),
+    "pace_latent_gather": (C.c_int, [_P, C.c_int32, C.c_void_p, C.c_void_p, C.c_int32, C.c_void_p, C.c_void_p]),
+    "pace_glu": (C.c_int, [C.c_void_p, C.c_int64, C.c_void_p, C.c_int32, C.c_int32, C.c_int32, C.c_int32, C.c_void_p]),
+    "pace_moe_route": (C.c_int, [C.POINTER(MoeRouteArgs), C.c_void_p]),
+    "pace_moe_experts": (C.c_int, [C.POINTER(MoeExpertsArgs), C.c_void_p]),
     "pace_gate_heads": (C.c_int, [_S, C.c_void_p, C.c_void_p, C.c_int64, C.c_void_p, C.c_int32, C.c_int32, C.c_int32,
                                   C.c_int32, C.c_void_p]),
     "pace_norm_gate": (C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int64, C.c_void_p, C.c_int32, C.c_int32, C.c_float,

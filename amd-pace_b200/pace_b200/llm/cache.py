@@ -175,6 +175,10 @@ class KVPool:
         return self._meta_view(self.desc.block_table, self.max_seqs * self.max_pages_per_seq).view(
             self.max_seqs, self.max_pages_per_seq)
 
+    def status_word(self) -> torch.Tensor:
+        """The sticky status word on the device (int32 [1]), for kernels that report to it."""
+        return self._meta_view(self.desc.status, 1)
+
     def seq_len(self) -> torch.Tensor:
         return self._meta_view(self.desc.seq_len, self.n_layers * self.max_seqs).view(self.n_layers, self.max_seqs)
 

@@ -6,12 +6,23 @@ positions, entry boundaries, slots, the rows of the attention staging buffers - 
 the host and copied once.
 """
 import ctypes as C
+from dataclasses import dataclass
 from typing import Dict, List, Optional, Sequence
 
 import numpy as np
 import torch
 
 from pace_b200 import _C
+
+
+@dataclass
+class KeyRows:
+    """Keys of several entries back to back: entry i owns [cu[i], cu[i + 1]), its first key has position first_pos[i]."""
+    total: int
+    slot: torch.Tensor
+    pos: torch.Tensor
+    cu: torch.Tensor
+    first_pos: torch.Tensor
 
 
 class Step:
@@ -36,6 +47,9 @@ class Step:
         if self.n_entries == 0:
             raise ValueError("a step needs at least one token")
         self.max_count = max(self.counts)
+        # last position of any entry + 1, as far as the host knows (``set_decode``: whoever supplies positions raises it)
+        self.max_keys = max(s + c for s, c in zip(self.starts, self.counts))
+        self._key_rows: Dict[tuple, "KeyRows"] = {}
         T, E, Ed = self.n_tokens, self.n_entries, self.n_decode
         n = np.asarray(self.counts, dtype=np.int64)
         cu = np.concatenate([[0], np.cumsum(n)])
@@ -54,6 +68,7 @@ class Step:
         # (batch row, local token) of a packed row, for callers that ask for logits by place
         self.first_row: Dict[int, int] = {b: int(cu[i]) for i, b in enumerate(self.rows)}
         self.last_rows: List[int] = [int(x) - 1 for x in cu[1:]]
+        self._slots = [int(slots[b]) for b in self.rows]
         parts = [tok, entry, pos, q_row, cu, np.asarray(self.starts), np.asarray([slots[b] for b in self.rows]), n]
         if tokens.is_cuda:
             parts.append(src)
@@ -81,6 +96,22 @@ class Step:
     @property
     def decode_only(self) -> bool:
         return self.max_count == 1
+
+    def key_rows(self, window: Optional[int], first_entry: int) -> "KeyRows":
+        """The keys that entries ``first_entry`` .. see through a sliding window (None: all), listed for gathering."""
+        key = (window, first_entry)
+        if key not in self._key_rows:
+            lo = [max(0, s - window + 1) if window else 0 for s in self.starts[first_entry:]]
+            hi = [s + c for s, c in zip(self.starts[first_entry:], self.counts[first_entry:])]
+            n = np.asarray(hi) - np.asarray(lo)
+            cu = np.concatenate([[0], np.cumsum(n)])
+            pos = np.arange(cu[-1]) - np.repeat(cu[:-1], n) + np.repeat(lo, n)
+            slot = np.repeat(self._slots[first_entry:], n)
+            host = torch.from_numpy(np.concatenate([slot, pos, cu, lo]).astype(np.int32))
+            dev = host if self.device.type != "cuda" else host.pin_memory().to(self.device, non_blocking=True)
+            T, E = int(cu[-1]), len(lo)
+            self._key_rows[key] = KeyRows(T, dev[:T], dev[T: 2 * T], dev[2 * T: 2 * T + E + 1], dev[2 * T + E + 1:])
+        return self._key_rows[key]
 
     def set_decode(self, next_token: torch.Tensor, position: torch.Tensor) -> None:
         """Token ids and positions (int64 ``[n_entries]``, on the device) of a one-token-per-entry step; stream

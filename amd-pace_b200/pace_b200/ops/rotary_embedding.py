@@ -15,6 +15,25 @@ import torch
 from torch import nn
 
 
+def _yarn_tables(theta: float, rotary_dim: int, n_rows: int, scaling: Optional[Dict[str, Any]]):
+    """fp32 tables from double-precision frequencies and angles.  ``scaling`` (``factor``,
+    ``original_max_position_embeddings``, ``beta_fast``, ``beta_slow``): pairs that turn at least ``beta_fast`` times
+    within the original length keep their frequency, those that turn at most ``beta_slow`` times have it divided by the
+    factor, a linear ramp over the pairs lies in between; cos and sin are multiplied by 0.1 ln(factor) + 1."""
+    i = torch.arange(rotary_dim // 2, dtype=torch.float64)
+    freq, gain = theta ** (-2.0 * i / rotary_dim), 1.0
+    if scaling is not None:
+        factor, window = float(scaling["factor"]), float(scaling["original_max_position_embeddings"])
+        pair = lambda turns: rotary_dim * math.log(window / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))   # noqa: E731
+        lo = max(math.floor(pair(scaling["beta_fast"])), 0)
+        hi = min(math.ceil(pair(scaling["beta_slow"])), rotary_dim - 1)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        freq = freq / factor * ramp + freq * (1.0 - ramp)
+        gain = 0.1 * math.log(factor) + 1.0
+    angle = torch.arange(n_rows, dtype=torch.float64)[:, None] * freq[None, :]
+    return (angle.cos() * gain).float(), (angle.sin() * gain).float()
+
+
 def _frequencies(theta: float, rotary_dim: int, divide_by=None) -> torch.Tensor:
     exponents = torch.arange(0, rotary_dim, 2, dtype=torch.float) / rotary_dim
     freq = theta ** exponents
@@ -33,7 +52,9 @@ class RotaryEmbedding(nn.Module):
     ``default``, ``linear`` (``scaling_factor``), ``dynamic`` (NTK, ``scaling_factor``), ``llama3``
     (``factor``, ``low_freq_factor``, ``high_freq_factor``, ``original_max_position_embeddings``) and
     ``longrope`` (``short_factor``, ``long_factor``, optional ``attention_factor``; keyword
-    ``original_max_position_embeddings``).  Tables are fp32 ``[rows, rotary_dim / 2]``."""
+    ``original_max_position_embeddings``), ``yarn`` (``factor``, ``original_max_position_embeddings``, ``beta_fast``,
+    ``beta_slow``) and ``precise`` (no scaling).  Tables are fp32 ``[rows, rotary_dim / 2]``; those of the last two come
+    from double-precision angles (an fp32 product of position and frequency is off by up to half an ulp of the angle)."""
 
     def __init__(self, rope_scaling: Optional[Dict[str, Any]], rotary_dim: int, max_position_embeddings: int,
                  rope_theta: float, partial_rotary_factor: float = 1.0, dtype: Optional[torch.dtype] = None,
@@ -80,6 +101,8 @@ class RotaryEmbedding(nn.Module):
             short = _tables(_frequencies(rope_theta, R, rope_scaling["short_factor"]), window, gain)
             long = _tables(_frequencies(rope_theta, R, rope_scaling["long_factor"]), N, gain)
             cos, sin = torch.cat([short[0], long[0]]), torch.cat([short[1], long[1]])
+        elif kind in ("yarn", "precise"):
+            cos, sin = _yarn_tables(rope_theta, R, N, rope_scaling if kind == "yarn" else None)
         else:
             raise ValueError(f"Unsupported RoPE type: {kind}")
         self.register_buffer("cos_cache", cos.contiguous(), persistent=False)

@@ -43,9 +43,25 @@ _DEFS["linear_skinny"] = "(Tensor x, Tensor weight, Tensor(a!) out, Tensor(b!) w
 # layers of hybrid decoders; a step is named by the address of its pace_step_t (``Step.handle``)
 _DEFS.update({
     "residual_norm": "(int step, Tensor(a!) x, Tensor? y, Tensor? w_post, Tensor? embed, Tensor? w_next, Tensor(b!)? h, "
-                     "float eps, bool restart, float weight_offset) -> ()",
+                     "float eps, bool restart, float weight_offset, float embed_scale=1.0, int top=0, Tensor? slot_expert=None, "
+                     "Tensor? slot_rank=None, Tensor? slot_weight=None, Tensor? expert_count=None) -> ()",
     "kv_append_norm": "(int pool, Tensor(a!) pages, int layer, int step, Tensor qkv, Tensor? q_norm, Tensor? k_norm, "
-                      "Tensor(b!) q_out, int dim, int vdim, float eps, float q_mul, float temp_coef, float temp_every) -> ()",
+                      "Tensor(b!) q_out, int dim, int vdim, float eps, float q_mul, float temp_coef, float temp_every, "
+                      "bool per_head=False) -> ()",
+    "attn_span": "(int pool, Tensor pages, int layer, int step, Tensor q, Tensor(a!) out, Tensor? slopes, Tensor? sinks, int dim, "
+                 "int vdim, float scale, int span, int span_size, int entry_begin, int entry_end, int max_tokens, int max_keys) -> ()",
+    "attn_span_prefill": "(int pool, Tensor? pages, int layer, int step, Tensor q, Tensor(a!) out, Tensor? slopes, Tensor? sinks, "
+                         "int dim, int vdim, float scale, int span, int span_size, int entry_begin, int entry_end, int max_tokens, "
+                         "int max_keys, Tensor? k, Tensor? k2, Tensor? v, Tensor? key_cu, Tensor? key_pos) -> bool",
+    "latent_append": "(int pool, Tensor(a!) pages, int layer, int step, Tensor down, Tensor q_norm, Tensor kv_norm, Tensor cos, "
+                     "Tensor sin, Tensor(b!) cq, int rot_dim, float eps) -> ()",
+    "rotate_heads": "(int step, Tensor src, Tensor(a!) dst, Tensor cos, Tensor sin, int token_begin, int token_end, int pad_dim) -> ()",
+    "latent_gather": "(int pool, Tensor pages, int layer, Tensor slot, Tensor pos, Tensor(a!) out) -> ()",
+    "glu": "(Tensor x, Tensor(a!) out, int act) -> ()",
+    "moe_route": "(Tensor logits, Tensor? correction, Tensor(a!) slot_expert, Tensor(b!) slot_rank, Tensor(c!) slot_weight, "
+                 "Tensor(d!) expert_count, Tensor(e!) expert_list) -> ()",
+    "moe_experts": "(Tensor x, Tensor gate_up, Tensor down, Tensor(a!) hidden, Tensor(b!) y, Tensor expert_count, "
+                   "Tensor expert_list, Tensor(c!)? status, int top, int act) -> ()",
     "attn_general": "(int pool, Tensor pages, int layer, int step, Tensor q, Tensor(a!) out, int dim, int vdim, "
                     "float scale) -> ()",
     "gate_heads": "(int step, Tensor attn, Tensor gate, Tensor(a!) out, int vdim) -> ()",
@@ -172,10 +188,16 @@ def _dtype(t: torch.Tensor) -> int:
     raise TypeError(f"activations must be bfloat16 or float32, got {t.dtype}")
 
 
-def _residual_norm(step, x, y, w_post, embed, w_next, h, eps, restart, weight_offset):
+def _residual_norm(step, x, y, w_post, embed, w_next, h, eps, restart, weight_offset, embed_scale=1.0, top=0,
+                   slot_expert=None, slot_rank=None, slot_weight=None, expert_count=None):
     a = _C.ResidualNormArgs()
     a.x, a.y, a.w_post, a.embed, a.w_next, a.h = x.data_ptr(), _ptr(y), _ptr(w_post), _ptr(embed), _ptr(w_next), _ptr(h)
     a.width, a.restart, a.eps, a.weight_offset = x.shape[1], int(restart), eps, weight_offset
+    a.embed_scale, a.top = embed_scale, top
+    if top:
+        a.n_experts = expert_count.numel()
+        a.slot_expert, a.slot_rank = slot_expert.data_ptr(), slot_rank.data_ptr()
+        a.slot_weight, a.expert_count = slot_weight.data_ptr(), expert_count.data_ptr()
     a.y_stride = y.stride(0) if y is not None else x.shape[1]
     a.vocab = embed.shape[0] if embed is not None else 0
     a.dtype = _dtype(next(t for t in (h, y, embed) if t is not None))
@@ -183,12 +205,13 @@ def _residual_norm(step, x, y, w_post, embed, w_next, h, eps, restart, weight_of
         _C.check(_C.lib.pace_residual_norm(_step(step), C.byref(a), _stream(x)), "pace_residual_norm")
 
 
-def _kv_append_norm(pool, pages, layer, step, qkv, q_norm, k_norm, q_out, dim, vdim, eps, q_mul, temp_coef, temp_every):
+def _kv_append_norm(pool, pages, layer, step, qkv, q_norm, k_norm, q_out, dim, vdim, eps, q_mul, temp_coef, temp_every,
+                    per_head=False):
     a = _C.AppendNormArgs()
     a.qkv, a.qkv_stride = qkv.data_ptr(), qkv.stride(0)
     a.q_norm, a.k_norm, a.q_out = _ptr(q_norm), _ptr(k_norm), q_out.data_ptr()
     a.n_q_heads, a.dim, a.vdim, a.dtype = q_out.shape[1], dim, vdim, _dtype(qkv)
-    a.eps, a.q_mul, a.temp_coef, a.temp_every = eps, q_mul, temp_coef, temp_every
+    a.eps, a.q_mul, a.temp_coef, a.temp_every, a.per_head = eps, q_mul, temp_coef, temp_every, int(per_head)
     with torch.cuda.device(pages.device):
         _C.check(_C.lib.pace_kv_append_norm(_pool(pool), layer, _step(step), C.byref(a), _stream(pages)),
                  "pace_kv_append_norm")
@@ -198,6 +221,93 @@ def _attn_general(pool, pages, layer, step, q, out, dim, vdim, scale):
     with torch.cuda.device(pages.device):
         _C.check(_C.lib.pace_attn_general(_pool(pool), layer, _step(step), q.data_ptr(), out.data_ptr(), q.shape[1], dim,
                                           vdim, scale, _dtype(q), _stream(pages)), "pace_attn_general")
+
+
+def _span_args(a, q, out, slopes, sinks, dim, vdim, scale, span, span_size, entry_begin, entry_end, max_tokens, max_keys):
+    a.q, a.out, a.slopes, a.sinks = q.data_ptr(), out.data_ptr(), _ptr(slopes), _ptr(sinks)
+    a.n_q_heads, a.dim, a.vdim, a.dtype = q.shape[1], dim, vdim, _dtype(q)
+    a.q_elems, a.out_elems = q.shape[2], out.shape[2]
+    a.entry_begin, a.entry_end, a.max_tokens, a.max_keys = entry_begin, entry_end, max_tokens, max_keys
+    a.span, a.span_size, a.scale = span, span_size, scale
+    return a
+
+
+def _attn_span(pool, pages, layer, step, q, out, *rule):
+    a = _span_args(_C.AttnSpanArgs(), q, out, *rule)
+    with torch.cuda.device(q.device):
+        _C.check(_C.lib.pace_attn_span(_pool(pool), layer, _step(step), C.byref(a), _stream(q)), "pace_attn_span")
+
+
+def _attn_span_prefill(pool, pages, layer, step, q, out, slopes, sinks, dim, vdim, scale, span, span_size, entry_begin, entry_end,
+                       max_tokens, max_keys, k=None, k2=None, v=None, key_cu=None, key_pos=None):
+    """False: the kernel does not take these shapes and nothing was launched."""
+    a = _C.AttnSpanPrefillArgs()
+    _span_args(a.a, q, out, slopes, sinks, dim, vdim, scale, span, span_size, entry_begin, entry_end, max_tokens, max_keys)
+    if k is not None:
+        a.k, a.k_row, a.k_head, a.k_dim = k.data_ptr(), k.stride(0), k.stride(1), k.shape[2]
+        a.v, a.v_row, a.v_head = v.data_ptr(), v.stride(0), v.stride(1)
+        a.n_rows, a.n_kv_heads = k.shape[:2]
+        a.key_cu, a.key_pos = key_cu.data_ptr(), key_pos.data_ptr()
+        if k2 is not None:
+            a.k2, a.k2_row, a.k2_dim = k2.data_ptr(), k2.stride(0), k2.shape[1]
+    with torch.cuda.device(q.device):
+        rc = _C.lib.pace_attn_span_prefill(_pool(pool), layer, _step(step), C.byref(a), _stream(q))
+        if rc != _C.PACE_ERR_UNSUPPORTED:
+            _C.check(rc, "pace_attn_span_prefill")
+    return rc == _C.PACE_OK
+
+
+def _latent_append(pool, pages, layer, step, down, q_norm, kv_norm, cos, sin, cq, rot_dim, eps):
+    a = _C.LatentAppendArgs()
+    a.down, a.down_stride, a.q_norm, a.kv_norm = down.data_ptr(), down.stride(0), q_norm.data_ptr(), kv_norm.data_ptr()
+    a.cos_table, a.sin_table, a.cq = cos.data_ptr(), sin.data_ptr(), cq.data_ptr()
+    a.q_rank, a.kv_rank, a.rot_dim, a.rot_pairs = q_norm.numel(), kv_norm.numel(), rot_dim, cos.shape[1]
+    a.table_rows, a.dtype, a.eps = cos.shape[0], _dtype(down), eps
+    with torch.cuda.device(pages.device):
+        _C.check(_C.lib.pace_latent_append(_pool(pool), layer, _step(step), C.byref(a), _stream(pages)), "pace_latent_append")
+
+
+def _rotate_heads(step, src, dst, cos, sin, token_begin, token_end, pad_dim):
+    a = _C.RotateArgs()
+    a.src, a.dst = src.data_ptr(), dst.data_ptr()
+    a.src_row, a.src_head, a.dst_row, a.dst_head = src.stride(0), src.stride(1), dst.stride(0), dst.stride(1)
+    a.cos_table, a.sin_table, a.token_begin, a.token_end = cos.data_ptr(), sin.data_ptr(), token_begin, token_end
+    a.n_heads, a.rot_dim, a.rot_pairs, a.pad_dim = src.shape[1], src.shape[2], cos.shape[1], pad_dim
+    a.table_rows, a.dtype = cos.shape[0], _dtype(src)
+    with torch.cuda.device(src.device):
+        _C.check(_C.lib.pace_rotate_heads(_step(step), C.byref(a), _stream(src)), "pace_rotate_heads")
+
+
+def _latent_gather(pool, pages, layer, slot, pos, out):
+    with torch.cuda.device(pages.device):
+        _C.check(_C.lib.pace_latent_gather(_pool(pool), layer, slot.data_ptr(), pos.data_ptr(), pos.numel(), out.data_ptr(),
+                                           _stream(pages)), "pace_latent_gather")
+
+
+def _glu(x, out, act):
+    with torch.cuda.device(x.device):
+        _C.check(_C.lib.pace_glu(x.data_ptr(), x.stride(0), out.data_ptr(), out.shape[0], out.shape[1], act, _dtype(x),
+                                 _stream(x)), "pace_glu")
+
+
+def _moe_route(logits, correction, slot_expert, slot_rank, slot_weight, expert_count, expert_list):
+    a = _C.MoeRouteArgs()
+    a.logits, a.correction, a.slot_expert, a.slot_rank = logits.data_ptr(), _ptr(correction), slot_expert.data_ptr(), slot_rank.data_ptr()
+    a.slot_weight, a.expert_count, a.expert_list = slot_weight.data_ptr(), expert_count.data_ptr(), expert_list.data_ptr()
+    (a.n_tokens, a.n_experts), a.top = logits.shape, slot_expert.shape[1]
+    with torch.cuda.device(logits.device):
+        _C.check(_C.lib.pace_moe_route(C.byref(a), _stream(logits)), "pace_moe_route")
+
+
+def _moe_experts(x, gate_up, down, hidden, y, expert_count, expert_list, status, top, act):
+    a = _C.MoeExpertsArgs()
+    a.x, a.gate_up, a.down, a.hidden, a.y = x.data_ptr(), gate_up.data_ptr(), down.data_ptr(), hidden.data_ptr(), y.data_ptr()
+    a.expert_count, a.expert_list, a.status = expert_count.data_ptr(), expert_list.data_ptr(), _ptr(status)
+    a.n_tokens, a.width = x.shape
+    a.n_experts, _, a.ff = down.shape
+    a.top, a.act, a.dtype = top, act, _dtype(x)
+    with torch.cuda.device(x.device):
+        _C.check(_C.lib.pace_moe_experts(C.byref(a), _stream(x)), "pace_moe_experts")
 
 
 def _gate_heads(step, attn, gate, out, vdim):
@@ -306,7 +416,9 @@ _IMPLS = {"kv_reserve": _kv_reserve, "kv_append": _kv_append, "kv_append_layers"
           "attn_general": _attn_general, "gate_heads": _gate_heads, "norm_gate": _norm_gate, "relu_squared": _relu_squared,
           "causal_conv": _causal_conv, "rglru_scan": _rglru_scan, "rglru_step": _rglru_step,
           "lightning_prefill": _lightning("pace_lightning_prefill"), "lightning_step": _lightning("pace_lightning_step"),
-          "step_decode": _step_decode}
+          "step_decode": _step_decode, "attn_span": _attn_span, "attn_span_prefill": _attn_span_prefill,
+          "latent_append": _latent_append, "rotate_heads": _rotate_heads, "latent_gather": _latent_gather, "glu": _glu,
+          "moe_route": _moe_route, "moe_experts": _moe_experts}
 for _n, _f in _IMPLS.items():
     _lib.impl(_n, _f, "CUDA")
     # shape propagation for tracers: nothing is returned, nothing to compute
