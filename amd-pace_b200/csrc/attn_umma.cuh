@@ -50,7 +50,6 @@ constexpr float kLazyRescale = 8.0f;    // log2 units
 // their exp2 phase at the same time there (they wait for the same K/V chunk) and the one exp2 unit per
 // scheduler serves two warps: 1150 cycles per chunk for 2 x 64 exp2 per lane, measured.
 constexpr int kWidePolyEvery = 2;
-constexpr unsigned kSoftmaxBackoffNs = 100;  // a waiting softmax warp leaves its scheduler's issue slots to the MMA issuer
 
 struct UmmaCtx {
   unsigned char* ring;    // [n_stages][K | V] as the TMA boxes land
@@ -72,23 +71,6 @@ struct UmmaCtx {
   volatile int* abort;
   int n_my, n_stages, cta;
 };
-
-// Bounded wait that also gives up when another role has raised the abort flag.  Called by whole
-// warps; the answer is the same for every lane (the tcgen05 instructions that follow are .aligned).
-__device__ __forceinline__ bool umma_wait(uint64_t* bar, uint32_t parity, volatile int* abort) {
-  bool ok = false;
-  for (int i = 0; i < (1 << 18); ++i) {
-    if (mbar_try_wait(bar, parity)) {
-      ok = true;
-      break;
-    }
-    if (*abort) break;
-    if (i >= 8) __nanosleep(i > 64 ? 256 : kSoftmaxBackoffNs);  // (the first probes back to back: most waits are nearly over)
-  }
-  if (!ok) *abort = 1;
-  return __all_sync(0xffffffffu, ok);
-}
-
 
 // ---- the two MMA issuers: warp 9 issues every QK, warp 10 every PV ----
 // Chunk i of this CTA's range (counted over the whole range, not per unit part) belongs to softmax

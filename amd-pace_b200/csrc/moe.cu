@@ -283,21 +283,13 @@ __global__ void __launch_bounds__(kThreads, 1)
     const bool leader = elect_one();
     int s = 0, ph = 0, n = 0;
     bool ok = true;
-    auto wait = [&](uint64_t* bar, uint32_t parity) {
-      for (int k = 0; k < (1 << 20); ++k) {
-        if (__all_sync(0xffffffffu, mbar_try_wait(bar, parity))) return true;
-        if ((k & 15) == 15 && __any_sync(0xffffffffu, *abort != 0)) break;
-      }
-      *abort = 1;
-      return false;
-    };
     for (int i = blockIdx.x; i < n_tiles && ok; i += gridDim.x, ++n) {
       const int buf = n & 1;
-      if (n >= 2 && !wait(&t_empty[buf], ((n >> 1) - 1) & 1)) break;
+      if (n >= 2 && !umma_issuer_wait(&t_empty[buf], ((n >> 1) - 1) & 1, abort)) break;
       tc_fence_after();
       const uint32_t d0 = tmem + buf * 2 * NT, d1 = d0 + NT;
       for (int ks = 0; ks < k_steps; ++ks) {
-        if (!wait(&full[s], ph)) {
+        if (!umma_issuer_wait(&full[s], ph, abort)) {
           ok = false;
           break;
         }

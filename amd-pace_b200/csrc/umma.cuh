@@ -233,6 +233,31 @@ __device__ __forceinline__ bool elect_one() {
   return pred != 0;
 }
 
+constexpr unsigned kSoftmaxBackoffNs = 100;  // a waiting softmax warp leaves its scheduler's issue slots to the MMA issuer
+// Bounded wait that also gives up when another role has raised the abort flag.  Called by whole
+// warps; the answer is the same for every lane (the tcgen05 instructions that follow are .aligned).
+__device__ __forceinline__ bool umma_wait(uint64_t* bar, uint32_t parity, volatile int* abort) {
+  bool ok = false;
+  for (int i = 0; i < (1 << 18); ++i) {
+    if (mbar_try_wait(bar, parity)) {
+      ok = true;
+      break;
+    }
+    if (*abort) break;
+    if (i >= 8) __nanosleep(i > 64 ? 256 : kSoftmaxBackoffNs);  // (the first probes back to back: most waits are nearly over)
+  }
+  if (!ok) *abort = 1;
+  return __all_sync(0xffffffffu, ok);
+}
+// The same for an issuer warp: no sleeping between the probes (each of them may wait up to a microsecond).
+__device__ __forceinline__ bool umma_issuer_wait(uint64_t* bar, uint32_t parity, volatile int* abort) {
+  for (int k = 0; k < (1 << 20); ++k) {
+    if (__all_sync(0xffffffffu, mbar_try_wait(bar, parity))) return true;
+    if ((k & 15) == 15 && __any_sync(0xffffffffu, *abort != 0)) break;
+  }
+  *abort = 1;
+  return false;
+}
 __device__ __forceinline__ void tma_load_2d(void* dst, const CUtensorMap* tm, int c0, int c1, uint64_t* bar) {
   asm volatile(
       "cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];" ::"r"(

@@ -183,7 +183,7 @@ def expand_pays(step: Step, dtype: torch.dtype, heads: int, dim: int, rot_dim: i
         pairs = c * min(s + c / 2.0, float(window or s + c))
         expanded += seen * rank * (dim + vdim) + pairs * (dim + rot_dim + vdim)
         absorbed += c * rank * (dim + vdim) + pairs * (2 * rank + rot_dim)
-    return False and step.max_count >= 32 and expanded < absorbed
+    return step.max_count >= 32 and expanded < absorbed
 
 
 def glu(x: torch.Tensor, act: int) -> torch.Tensor:
