@@ -897,11 +897,30 @@ HYBRID_SIZES = {
 HYBRID_VOCAB, HYBRID_LAYERS = 32000, 8
 
 
+def llama_model(z: dict, n_layers: int, dev):
+    """The attention-only decoder of one size with random weights."""
+    from pace_b200.llm.models.llama import LlamaForCausalLM
+
+    class Cfg:
+        hidden_size, intermediate_size, num_hidden_layers = z["width"], z["ff"], n_layers
+        num_attention_heads, num_key_value_heads, vocab_size = z["heads"], z["kv_heads"], HYBRID_VOCAB
+        max_position_embeddings, rope_theta, rms_norm_eps, pad_token_id = 8192, 500000.0, 1e-5, 0
+        rope_scaling = None
+
+    with torch.device(dev):
+        llama = LlamaForCausalLM(Cfg()).to(torch.bfloat16).eval()
+    g = torch.Generator(device=dev).manual_seed(5)
+    with torch.no_grad():
+        for p_ in llama.parameters():
+            if p_.dim() >= 2:
+                p_.normal_(0.0, 0.02, generator=g)
+    return llama
+
+
 def hybrid_models(size: str, dev):
     """(Garupel, Llama) of one size with random weights: 8 layer runs each, of which Garupel's are 4 x rglru,
     2 x lightning and 2 x attention."""
     from pace_b200.llm.models.garupel import GarupelForCausalLM
-    from pace_b200.llm.models.llama import LlamaForCausalLM
     from pace_b200.llm.registry import build_model
     z = HYBRID_SIZES[size]
     W, mlp = z["width"], {"kind": "dense", "ff": z["ff"]}
@@ -918,20 +937,7 @@ def hybrid_models(size: str, dev):
     assert isinstance(garupel, GarupelForCausalLM)
     garupel.random_init_(5)
 
-    class Cfg:
-        hidden_size, intermediate_size, num_hidden_layers = W, z["ff"], HYBRID_LAYERS
-        num_attention_heads, num_key_value_heads, vocab_size = z["heads"], z["kv_heads"], HYBRID_VOCAB
-        max_position_embeddings, rope_theta, rms_norm_eps, pad_token_id = 8192, 500000.0, 1e-5, 0
-        rope_scaling = None
-
-    with torch.device(dev):
-        llama = LlamaForCausalLM(Cfg()).to(torch.bfloat16).eval()
-    g = torch.Generator(device=dev).manual_seed(5)
-    with torch.no_grad():
-        for p_ in llama.parameters():
-            if p_.dim() >= 2:
-                p_.normal_(0.0, 0.02, generator=g)
-    return garupel, llama
+    return garupel, llama_model(z, HYBRID_LAYERS, dev)
 
 
 def hybrid_cache(model, batch: int, max_len: int, dev):
@@ -1021,6 +1027,41 @@ def graph_us(launches, reps=5):
     return statistics.median(times)
 
 
+def llama_kernels(add, dev, rnd, N, E, n, past, qkvg, qb, y, up, wp, sizes, kv_read, flops):
+    """The like kernels of the attention-only decoder on the same operands: plain attention (its weights rounded to
+    bf16), RoPE + append, norm and residual, gated activation (the last two are torch's)."""
+    from pace_b200.llm.cache import KVCacheManager, KVCacheType
+    from pace_b200.ops import MultiHeadAttention, RotaryEmbedding
+    W, H, G, D, FF = sizes
+    T, nq, nk, dec = E * n, H * D, G * D, n == 1
+
+    class LlamaCfg:
+        num_hidden_layers = N
+    mgr = KVCacheManager(LlamaCfg(), past + n * (8 if not dec else 64) + 64, KVCacheType.BMC)
+    for i in range(N):
+        kv = rnd(E, G, past + n, D)
+        mgr[i].update_cache(kv, kv, concat_dim=2)
+    q4, mha = [t.view(E, n, H, D).transpose(1, 2) for t in qb], MultiHeadAttention()
+    o4 = torch.empty(E, n, H, D, dtype=torch.bfloat16, device=dev).transpose(1, 2)
+    add("llama.attention", [lambda i=i: mha(q4[i], mgr[i].key, mgr[i].value, out=o4) for i in range(N)],
+        kv_read + T * nq * 4, flops)
+    if not dec:                               # (a decode step stages its rows: profiled with the decode loop)
+        rope = RotaryEmbedding(None, D, 8192, 500000.0).to(dev)
+        rws = rope.table_rows(torch.arange(n, device=dev).expand(E, n))
+        xs = [t[:, : nq + 2 * nk].view(E, n, H + 2 * G, D) for t in qkvg]
+        qo = [t.view(E, n, H, D) for t in qb]
+        cos, sin = rope.device_tables(mgr.pool.device)
+        add("llama.append_rope", [lambda i=i: torch.ops.pace_b200.kv_append_rope(
+            mgr.pool.handle, mgr.pool.pages, mgr.pool.meta, i, mgr.slots_dev, xs[i][:, :, :H], xs[i][:, :, H:H + G],
+            xs[i][:, :, H + G:], qo[i], rws, cos, sin, D, False, None, xs[i][:, :, H:H + G].transpose(1, 2), xs[i][:, :, H + G:].transpose(1, 2))
+            for i in range(N)], T * (nq + 2 * nk) * 4)
+    w16 = wp.bfloat16()
+    add("llama.residual+norm (torch)", [lambda i=i: torch.nn.functional.rms_norm(y[i] + y[i - 1], (W,), w16, 1e-5)
+                                        for i in range(N)], T * W * 2 * 4)
+    add("llama.silu*up (torch)", [lambda i=i: up[i] * torch.nn.functional.silu(up[i - 1]) for i in range(N)], T * FF * 6)
+    mgr.pool.check_status()
+
+
 @torch.inference_mode()
 def hybrid_kernels(size: str, dev):
     """Each kernel of the hybrid decoder alone, against its own roofline: bytes that must move over the measured
@@ -1094,37 +1135,7 @@ def hybrid_kernels(size: str, dev):
         add("norm_gate", [lambda i=i: hybrid.norm_gate(lo[i], wp[:LH * D] if LH * D <= W else vec(LH * D),
                                                        lq[i][:, 3 * LH * D:], 1e-5) for i in range(N)], T * LH * D * 6)
         add("relu_squared", [lambda i=i: hybrid.relu_squared_(up[i]) for i in range(N)], T * FF * 4)
-        # the like kernels of the attention-only decoder on the same operands: plain attention (its weights rounded to
-        # bf16), RoPE + append, norm and residual, gated activation (the last two are torch's)
-        from pace_b200.llm.cache import KVCacheManager, KVCacheType
-        from pace_b200.ops import MultiHeadAttention, RotaryEmbedding
-
-        class LlamaCfg:
-            num_hidden_layers = N
-        mgr = KVCacheManager(LlamaCfg(), past + n * (8 if not dec else 64) + 64, KVCacheType.BMC)
-        for i in range(N):
-            kv = rnd(E, G, past + n, D)
-            mgr[i].update_cache(kv, kv, concat_dim=2)
-        q4, mha = [t.view(E, n, H, D).transpose(1, 2) for t in qb], MultiHeadAttention()
-        o4 = torch.empty(E, n, H, D, dtype=torch.bfloat16, device=dev).transpose(1, 2)
-        add("llama.attention", [lambda i=i: mha(q4[i], mgr[i].key, mgr[i].value, out=o4) for i in range(N)],
-            kv_read + T * nq * 4, flops)
-        if not dec:                               # (a decode step stages its rows: profiled with the decode loop)
-            rope = RotaryEmbedding(None, D, 8192, 500000.0).to(dev)
-            rws = rope.table_rows(torch.arange(n, device=dev).expand(E, n))
-            xs = [t[:, : nq + 2 * nk].view(E, n, H + 2 * G, D) for t in qkvg]
-            qo = [t.view(E, n, H, D) for t in qb]
-            cos, sin = rope.device_tables(pool.device)
-            add("llama.append_rope", [lambda i=i: torch.ops.pace_b200.kv_append_rope(
-                mgr.pool.handle, mgr.pool.pages, mgr.pool.meta, i, mgr.slots_dev, xs[i][:, :, :H], xs[i][:, :, H:H + G],
-                xs[i][:, :, H + G:], qo[i], rws, cos, sin, D, False, None, xs[i][:, :, H:H + G].transpose(1, 2), xs[i][:, :, H + G:].transpose(1, 2))
-                for i in range(N)], T * (nq + 2 * nk) * 4)
-        w16 = wp.bfloat16()
-        add("llama.residual+norm (torch)", [lambda i=i: torch.nn.functional.rms_norm(y[i] + y[i - 1], (W,), w16, 1e-5)
-                                            for i in range(N)], T * W * 2 * 4)
-        add("llama.silu*up (torch)", [lambda i=i: up[i] * torch.nn.functional.silu(up[i - 1]) for i in range(N)], T * FF * 6)
-        mgr.pool.check_status()
-        del mgr
+        llama_kernels(add, dev, rnd, N, E, n, past, qkvg, qb, y, up, wp, (W, H, G, D, FF), kv_read, flops)
         cache.pool.check_status()
         if not dec:                               # the parts of the recurrence's prefill
             u = [rnd(T, W) for _ in range(N)]
@@ -1162,6 +1173,188 @@ def run_hybrid(args):
         print(json.dumps(line), flush=True)
 
 
+# ---------------------------------------------------------------------------------------------------
+# Gekupel (chunked attention, latent attention, mixtures of experts) beside the attention-only decoder
+# ---------------------------------------------------------------------------------------------------
+# top * expert_ff = ff: a token's feed-forward is as wide as the attention-only decoder's
+GEKUPEL_SIZES = {
+    "w2048": dict(width=2048, ff=8192, heads=16, kv_heads=4, dim=128, chunk=2048, lat_heads=16, lat_dim=128, rot=64, q_rank=768,
+                  kv_rank=512, window=1024, experts=64, top=8, expert_ff=1024),
+    "w4096": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, chunk=2048, lat_heads=32, lat_dim=128, rot=64, q_rank=1536,
+                  kv_rank=512, window=1024, experts=64, top=8, expert_ff=1792),
+}
+
+
+def gekupel_model(size: str, dev):
+    from pace_b200.llm.registry import build_model
+    z = GEKUPEL_SIZES[size]
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    lat = {"heads": z["lat_heads"], "dim": z["lat_dim"], "rot_dim": z["rot"], "vdim": z["lat_dim"], "q_rank": z["q_rank"],
+           "kv_rank": z["kv_rank"], "mask": {"size": z["window"]}, "scale": (z["lat_dim"] + z["rot"]) ** -0.5,
+           "rot": {"dims": z["rot"], "base": 1e6}}
+    lat2 = {**lat, "rot": {**lat["rot"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+           "mask": {"size": z["chunk"]}}
+    A = {"type": "attention", "mixer": att, "mlp": moe}
+    L = {"type": "latent_attention", "mixer": lat, "mlp": moe}
+    L2 = {"type": "latent_attention_2", "mixer": lat2, "mlp": moe}
+    cfg = {"architecture": "Gekupel", "vocab": HYBRID_VOCAB, "width": z["width"], "norm": {"eps": 1e-5}, "embedding": {"scale": 8.0},
+           "layers": [{**L2, "mlp": {"kind": "dense", "ff": z["ff"]}}, A, L, L2, A, L, L2, {**A, "weights_of": 1}]}
+    return build_model(cfg, torch.bfloat16, dev).random_init_(5)
+
+
+@torch.inference_mode()
+def gekupel_kernels(size: str, dev):
+    """Each kernel of the Gekupel decoder alone, against its own roofline, beside the like kernels of the attention-only
+    decoder; operands and phases as in ``hybrid_kernels``."""
+    from pace_b200 import _C
+    from pace_b200.llm.hybrid_cache import HybridCacheManager, KVSpec, LatentSpec
+    from pace_b200.ops import RotaryEmbedding, hybrid
+    z = GEKUPEL_SIZES[size]
+    W, H, G, D, FF = z["width"], z["heads"], z["kv_heads"], z["dim"], z["ff"]
+    LH, LD, r, R, QR, win = z["lat_heads"], z["lat_dim"], z["rot"], z["kv_rank"], z["q_rank"], z["window"]
+    X, top, XF, ops = z["experts"], z["top"], z["expert_ff"], torch.ops.pace_b200
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(
+        os.path.join(ROOT, "MEASURED_PEAKS.json")) else {"hbm_gbs": FALLBACK_HBM_GBS, "bf16_tflops_sustained": 1400.0}
+    bw, fl = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops_sustained"] * 1e12
+    g = torch.Generator(device=dev).manual_seed(2)
+
+    def rnd(*shape, dtype=torch.bfloat16):
+        return torch.randn(*shape, device=dev, generator=g, dtype=torch.float32).to(dtype)
+
+    def pairs(n, past, first):                 # (query, key) pairs of one sequence
+        return sum(t + 1 - first(t) for t in range(past, past + n))
+
+    out = {}
+    cos, sin = RotaryEmbedding({"rope_type": "precise"}, r, 8192, 1e6, is_neox_style=False).device_tables(dev)
+    for phase, E, n, past in (("prefill", 1, 4096, 0), ("decode", 32, 1, 512)):
+        T, dec = E * n, n == 1
+        N = 8 if dec else 3                    # copies of every operand
+        cache = HybridCacheManager([KVSpec(G, D, D)] * N + [LatentSpec(R, r)] * N, E, E * (past + n + 64), past + n + 64,
+                                   torch.bfloat16, dev)
+        if past:
+            cache.begin_step(cache.step([past] * E, torch.zeros(E * past, dtype=torch.long), 1))
+        step = cache.step([n] * E, torch.zeros(T, dtype=torch.long), 1)
+        cache.begin_step(step)
+        x, y = [rnd(T, W, dtype=torch.float32) for _ in range(N)], [rnd(T, W) for _ in range(N)]
+        wp = rnd(W, dtype=torch.float32)
+        nq, nk = H * D, G * D
+        qkv = [rnd(T, nq + 2 * nk) for _ in range(N)]
+        up = [rnd(T, FF) for _ in range(N)]
+        gu = [rnd(T, 2 * FF) for _ in range(N)]
+        qb = [rnd(step.staging_rows, H, D) for _ in range(N)]
+        slopes, sinks = torch.rand(H, device=dev) * 0.01, rnd(H, dtype=torch.float32)
+        pool, lpool = cache[0].pool, cache[N].pool
+        rows = {}
+
+        def add(name, launches, nbytes, nflops=0.0):
+            us = graph_us(launches)
+            roof = max(nbytes / bw, nflops / fl) * 1e6
+            rows[name] = {"us": us, "roofline_us": roof, "frac": roof / us, "bound": "hbm" if nbytes / bw >= nflops / fl else "tensor"}
+
+        add("residual_norm", [lambda i=i: hybrid.residual_norm(step, x[i], y[i], wp, plain=True, eps=1e-5) for i in range(N)],
+            T * W * (4 + 4 + 2 + 2))
+        add("append_heads", [lambda i=i: ops.kv_append_norm(pool.handle, pool.pages, i, step.handle, qkv[i], None, None, qb[i], D, D,
+                                                            1e-5, 1.0, 0.0, 1.0, True) for i in range(N)], T * (nq + 2 * nk) * 4)
+        pa = E * pairs(n, past, lambda t: t - t % z["chunk"])
+        keys_a = E * (past + n - (past - past % z["chunk"]))
+        ao = torch.empty(T, H, D, dtype=torch.bfloat16, device=dev)
+        rule = (slopes, sinks, D, D, D ** -0.5, _C.SPAN_CHUNK, z["chunk"], 0, E, n, past + n)
+
+        def attention(i):
+            if dec:
+                ops.attn_span(pool.handle, pool.pages, i, step.handle, qb[i], ao, *rule)
+            else:
+                assert ops.attn_span_prefill(pool.handle, pool.pages, i, step.handle, qb[i], ao, *rule, None, None, None, None, None)
+        add("attention (chunk, bias, sink)", [lambda i=i: attention(i) for i in range(N)], keys_a * nk * 4 + T * nq * 4, 4.0 * nq * pa)
+        # latent attention
+        down = [rnd(T, QR + R + r) for _ in range(N)]
+        cq, qn, kn = torch.empty(T, QR, dtype=torch.bfloat16, device=dev), rnd(QR, dtype=torch.float32), rnd(R, dtype=torch.float32)
+        add("latent_append", [lambda i=i: ops.latent_append(lpool.handle, lpool.pages, i, step.handle, down[i], qn, kn, cos, sin, cq,
+                                                            r, 1e-5) for i in range(N)], T * (QR + R + r) * 4)
+        q = [rnd(T, LH, LD + r) for _ in range(N)]
+        lsink = rnd(LH, dtype=torch.float32)
+        pl = E * pairs(n, past, lambda t: max(0, t - win + 1))
+        if dec:
+            row = R + r
+            qa = [rnd(T, LH, row) for _ in range(N)]
+            lo = torch.empty(T, LH, R, dtype=torch.bfloat16, device=dev)
+            add("rotate_heads", [lambda i=i: ops.rotate_heads(step.handle, q[i][:, :, LD:], qa[i][:, :, R:], cos, sin, 0, T, r)
+                                 for i in range(N)], T * LH * r * 4)
+            add("latent attention (absorbed)", [lambda i=i: ops.attn_span(
+                lpool.handle, lpool.pages, i, step.handle, qa[i], lo, None, lsink, row, R, 0.07, _C.SPAN_WINDOW, win, 0, E, 1, past + 1)
+                for i in range(N)], min(past + 1, win) * E * row * 2 + T * LH * (row + R) * 2, 2.0 * pl * LH * (row + R))
+        else:
+            add("rotate_heads", [lambda i=i: ops.rotate_heads(step.handle, q[i][:, :, LD:], q[i][:, :, LD:], cos, sin, 0, T, r)
+                                 for i in range(N)], T * LH * r * 4)
+            keys = step.key_rows(win, 0)
+            lat = [torch.empty(keys.total, R + r, dtype=torch.bfloat16, device=dev) for _ in range(N)]
+            add("latent_gather", [lambda i=i: ops.latent_gather(lpool.handle, lpool.pages, i, keys.slot, keys.pos, lat[i])
+                                  for i in range(N)], keys.total * (R + r) * 4)
+            kv = [rnd(keys.total, LH * 2 * LD) for _ in range(N)]
+            lo = torch.empty(T, LH, LD, dtype=torch.bfloat16, device=dev)
+
+            def expanded(i):
+                k, v = kv[i][:, : LH * LD].view(-1, LH, LD), kv[i][:, LH * LD:].view(-1, LH, LD)
+                assert ops.attn_span_prefill(lpool.handle, lpool.pages, i, step.handle, q[i], lo, None, lsink, LD + r, LD, 0.07,
+                                             _C.SPAN_WINDOW, win, 0, E, n, n, k, lat[i][:, R:], v, keys.cu, keys.first_pos)
+            add("latent attention (expanded)", [lambda i=i: expanded(i) for i in range(N)],
+                keys.total * (LH * 2 * LD + r) * 2 + T * LH * (2 * LD + r) * 2, 2.0 * pl * LH * (2 * LD + r))
+        # feed-forwards
+        add("glu", [lambda i=i: hybrid.glu(gu[i], _C.ACT_GELU_TANH) for i in range(N)], T * FF * 6)
+        M = 2                                   # sets of experts (each far beyond L2)
+        router = rnd(X, W) * W ** -0.5
+        logits = [hybrid.linear_f32(y[i], router) for i in range(N)]
+        routed = [hybrid.moe_route(y[i], router, None, top) for i in range(N)]
+        wg, wd = [rnd(X, 2 * XF, W) * 0.02 for _ in range(M)], [rnd(X, W, XF) * 0.02 for _ in range(M)]
+        used = int((routed[0].count > 0).sum())
+        add("moe_route", [lambda i=i: ops.moe_route(logits[i], None, routed[i].slot_expert, routed[i].slot_rank, routed[i].slot_weight,
+                                                    routed[i].count, routed[i].lists) for i in range(N)], T * X * 4 + T * top * 16)
+        add("moe_experts (both products)", [lambda i=i: hybrid.moe_experts(y[i % N], routed[i % N], wg[i % M], wd[i % M], _C.ACT_SILU)
+                                            for i in range(2 * M)],
+            used * 3 * XF * W * 2 + T * W * 2 + T * top * (XF * 4 + W * 2), 6.0 * T * top * XF * W)
+        for i in range(N):
+            hybrid.moe_experts(y[i], routed[i], wg[i % M], wd[i % M], _C.ACT_SILU)
+        add("residual_norm (experts' sum)", [lambda i=i: hybrid.residual_norm(step, x[i], w_post=wp, plain=True, eps=1e-5,
+                                                                              routed=routed[i]) for i in range(N)],
+            T * W * (4 + 4 + 2) + T * top * W * 2)
+        del wg, wd
+        llama_kernels(add, dev, rnd, N, E, n, past, qkv, qb, y, up, wp, (W, H, G, D, FF), 2 * nk * 2 * E * (past + n),
+                      4.0 * nq * E * pairs(n, past, lambda t: 0))
+        lg, ld = [rnd(2 * FF, W) for _ in range(M)], [rnd(W, FF) for _ in range(M)]
+        add("llama.mlp products (cuBLAS)", [lambda i=i: (torch.mm(y[i % N], lg[i % M].t()), torch.mm(up[i % N], ld[i % M].t()))
+                                            for i in range(2 * M)], 3 * FF * W * 2 + T * (W * 4 + FF * 6), 6.0 * T * FF * W)
+        cache.pool.check_status()
+        out[phase] = rows
+        del cache, lg, ld
+        torch.cuda.empty_cache()
+    return out
+
+
+def run_gekupel(args):
+    """Side measurement: prefill and decode throughput of the Gekupel decoder beside the Llama decoder at equal width,
+    heads, layer count and feed-forward width per token (random weights), and every kernel of the former against its
+    roofline.  Prints one JSON line per size."""
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    for size, z in GEKUPEL_SIZES.items():
+        sampler = ClockSampler(0)
+        sampler.start()
+        model = gekupel_model(size, dev)
+        line = {"workload": "gekupel", "size": size, **z, "layers": HYBRID_LAYERS,
+                "params": {"gekupel": sum(p.numel() for p in model.parameters())}, "gekupel": hybrid_throughput(model, dev)}
+        del model
+        torch.cuda.empty_cache()
+        llama = llama_model(z, HYBRID_LAYERS, dev)
+        line["params"]["llama"] = sum(p.numel() for p in llama.parameters())
+        line["llama"] = hybrid_throughput(llama, dev)
+        del llama
+        torch.cuda.empty_cache()
+        line["kernels"] = gekupel_kernels(size, dev)
+        line["clocks"] = sampler.stop()
+        print(json.dumps(line), flush=True)
+
+
 def main():
     # stdout carries the JSON line and nothing else: whatever native libraries print to file descriptor 1
     # (NCCL's version banner on some ranks) goes to stderr, Python's own prints keep the real stdout
@@ -1180,7 +1373,7 @@ def main():
     ap.add_argument("--layers", type=int, default=CFG["n_layers"],
                     help="profiling aid: fewer layers = less device memory; the bench line is only valid at 32")
     ap.add_argument("--workload", default="decode", choices=["decode", "verify", "prefill", "rope_append", "device_loop", "serving", "linear",
-                                                                 "hybrid"],
+                                                                 "hybrid", "gekupel"],
                     help="decode = the bench line; verify / prefill = side measurements of the multi-token kernels")
     ap.add_argument("--past", type=int, default=3584, help="prefill side measurement: tokens cached before the chunk")
     ap.add_argument("--head-dim", type=int, default=128, choices=[64, 128])
@@ -1195,10 +1388,10 @@ def main():
         return
     global RANK_CORES
     RANK_CORES = pin_rank_to_cores(local_rank, world)
-    if args.workload in ("rope_append", "device_loop", "serving", "linear", "hybrid"):
+    if args.workload in ("rope_append", "device_loop", "serving", "linear", "hybrid", "gekupel"):
         if rank == 0:
             {"rope_append": run_rope, "device_loop": run_device_loop, "serving": run_serving,
-             "linear": run_linear, "hybrid": run_hybrid}[args.workload](args)
+             "linear": run_linear, "hybrid": run_hybrid, "gekupel": run_gekupel}[args.workload](args)
         return
     if args.workload != "decode":
         if rank == 0:
