@@ -4,8 +4,8 @@
 //
 // A thread block works on one tile of 16 * MT query rows (row = token * group + head of the group) of one (entry, KV
 // head) and a contiguous share of the tile's visible keys; the shares of a tile are the blocks of a thread-block cluster.
-// Tiles of 64 keys travel through a ring of shared-memory stages (cp.async, 16 bytes at a time, row strides that
-// are an odd number of 16-byte units: ldmatrix without bank conflicts).  Per tile
+// A producer warp streams tiles of 64 keys (one page) through a ring of shared-memory stages: TMA boxes of 64 columns x 16
+// rows with the 128-byte swizzle, only those that hold visible keys.  Eight consumer warps, per tile
 //   scores   warp w: all query rows x keys 8 w .. 8 w + 7, mma.sync m16n8k16
 //   softmax  256 / rows threads per row, fp32, span and bias from positions; weights leave as two bf16 terms
 //   values   warp w: all query rows x the 16-column groups w, w + 8, ...
@@ -14,13 +14,15 @@
 #include <cooperative_groups.h>
 
 #include "span.cuh"
+#include "umma.cuh"
 
 namespace cg = cooperative_groups;
 
 namespace pace {
 namespace {
 
-constexpr int kKeys = 64, kThreads = 256, kPS = kKeys + 8, kSS = kKeys + 4;
+constexpr int kKeys = 64, kConsumers = 256, kThreads = kConsumers + 32, kPS = kKeys + 8, kSS = kKeys + 4;
+constexpr int kBlock = kKeys * 128, kBoxRows = 16, kBox = kBoxRows * 128;  // 64 columns x 64 keys, x 16 keys (bytes)
 
 struct SpanParams {
   KVView kv;
@@ -29,16 +31,16 @@ struct SpanParams {
   __nv_bfloat16* out;
   const float* slopes;
   const float* sinks;
-  int q_elems, out_elems, H, Gq, dk, dv, row;  // row: elements of a pool row
-  int dk16, dv16, shared_rows;                // sizes rounded up to 16; one plane
-  int entry0, span, span_size, n_stages, tab_cap, page_shift;
+  int q_elems, out_elems, H, Gq, dv;
+  int dk16, dv16, k_blocks, v_blocks;   // sizes rounded up to 16; 64-column blocks of a stage (v_blocks 0: one plane)
+  int entry0, span, span_size, n_stages;
   float scale_log2;
 };
 
 struct SpanSmem {
-  int q, ring, k_bytes, stage_bytes, s, ph, pl, alpha, tab, obuf, ml, total;
+  int ring, q, s, ph, pl, alpha, ml, bars, obuf, total;
 };
-__host__ __device__ inline SpanSmem span_smem(int MR, int dk16, int dv16, int shared_rows, int n_stages, int tab_cap) {
+__host__ __device__ inline SpanSmem span_smem(int MR, int dk16, int dv16, int blocks, int n_stages) {
   SpanSmem m;
   int off = 0;
   auto take = [&](int bytes) {
@@ -46,21 +48,17 @@ __host__ __device__ inline SpanSmem span_smem(int MR, int dk16, int dv16, int sh
     off += (bytes + 15) / 16 * 16;
     return o;
   };
+  m.ring = take(n_stages * blocks * kBlock);
+  m.obuf = 0;  // behind the last tile the ring's place (and the queries') holds the block's results
   m.q = take(MR * (dk16 + 8) * 2);
-  m.k_bytes = kKeys * (dk16 + 8) * 2;
-  m.stage_bytes = m.k_bytes + (shared_rows ? 0 : kKeys * (dv16 + 8) * 2);
-  m.ring = take(n_stages * m.stage_bytes);
+  if (off < MR * (dv16 + 4) * 4) off = (MR * (dv16 + 4) * 4 + 15) / 16 * 16;
   m.s = take(MR * kSS * 4);
   m.ph = take(MR * kPS * 2);
   m.pl = take(MR * kPS * 2);
   m.alpha = take(MR * 4);
-  m.tab = take(tab_cap * 4);
-  // behind the last tile the ring's place holds the block's results
-  m.obuf = m.ring;
-  const int need = MR * (dv16 + 4) * 4;
-  if (m.ring + need > off) off = m.ring + need;
   m.ml = take(MR * 8);
-  m.total = off;
+  m.bars = take(2 * 8 * 8 + 8);
+  m.total = off + 1024;  // (the ring starts at a multiple of 1024)
   return m;
 }
 
@@ -75,21 +73,23 @@ __device__ __forceinline__ void ldsm4_t(uint32_t addr, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
-__device__ __forceinline__ void ldsm2(uint32_t addr, uint32_t& r0, uint32_t& r1) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr) : "memory");
-}
 __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+__device__ __forceinline__ void consumer_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kConsumers) : "memory"); }
+
 // MT: 16-row tiles of query rows; NG: 16-column groups of the values a warp owns
 template <int MT, int NG>
-__global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kernel(const SpanParams p) {
-  constexpr int MR = 16 * MT, TPR = kThreads / MR, KPT = kKeys / TPR;
-  extern __shared__ __align__(16) unsigned char smem[];
-  const SpanSmem sm = span_smem(MR, p.dk16, p.dv16, p.shared_rows, p.n_stages, p.tab_cap);
+__global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1)
+    attn_span_kernel(const SpanParams p, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV) {
+  constexpr int MR = 16 * MT, TPR = kConsumers / MR, KPT = kKeys / TPR;
+  extern __shared__ unsigned char smem_raw[];
+  unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+  const int blocks = p.k_blocks + p.v_blocks, STAGE = blocks * kBlock;
+  const SpanSmem sm = span_smem(MR, p.dk16, p.dv16, blocks, p.n_stages);
   const int ns = gridDim.x, share = blockIdx.x;  // the cluster is the grid's x extent
   const int Hkv = p.kv.n_kv_heads, g = blockIdx.y % Hkv, e = p.entry0 + blockIdx.z;
   const int t0 = p.st.cu[e], count = p.st.cu[e + 1] - t0, start = p.st.start[e];
@@ -98,62 +98,91 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kern
   const int live = min(MR, R - r0);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int pos_a = start + r0 / p.Gq, pos_z = start + (r0 + live - 1) / p.Gq;
-  const int base = span_first(p.span, p.span_size, pos_a) & ~(kKeys - 1);
+  const int key_a = span_first(p.span, p.span_size, pos_a), base = key_a & ~(kKeys - 1);
   const int n_tiles = (pos_z - base) / kKeys + 1;
   const int per = (n_tiles + ns - 1) / ns;
   const int tile_a = min(share * per, n_tiles), tile_z = min(tile_a + per, n_tiles);
-  const int slot = p.st.slot[e], P = p.kv.page_tokens;
-  const uint32_t s_q = smem_u32(smem + sm.q), s_ring = smem_u32(smem + sm.ring);
-  const int KSB = (p.dk16 + 8) * 2, VSB = p.shared_rows ? KSB : (p.dv16 + 8) * 2;  // row strides, bytes
-  const int v_off = p.shared_rows ? 0 : sm.k_bytes;
-  int* tab = reinterpret_cast<int*>(smem + sm.tab);
+  uint64_t* full = reinterpret_cast<uint64_t*>(smem + sm.bars);
+  uint64_t* empty = full + 8;
+  int* abort_flag = reinterpret_cast<int*>(empty + 8);
+  volatile int* abort = abort_flag;
+  const uint32_t s_ring = smem_u32(smem + sm.ring), s_q = smem_u32(smem + sm.q);
+  const int QSB = (p.dk16 + 8) * 2;  // row stride of the queries, bytes: an odd number of 16-byte units
 
-  // ---- the query rows, the share's page numbers ----
-  {
-    const int pieces = p.dk16 / 8;
-    for (int i = tid; i < MR * pieces; i += kThreads) {
-      const int r = i / pieces, c = i - r * pieces;
-      const int rr = min(r0 + r, R - 1), tok = rr / p.Gq, hh = g * p.Gq + rr - tok * p.Gq;
-      const bool ok = r < live && (c + 1) * 8 <= p.q_elems;
-      cp_async16(s_q + r * KSB + c * 16, p.q + ((size_t)(t0 + tok) * p.H + hh) * p.q_elems + (ok ? c * 8 : 0), ok);
+  if (tid == kConsumers) {
+    *abort_flag = 0;
+    for (int i = 0; i < p.n_stages; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], kConsumers / 32);
     }
+    fence_mbar_init();
   }
-  const bool slot_ok = slot >= 0 && slot < p.kv.max_seqs;
-  const int lp0 = (base + tile_a * kKeys) / P;
-  const int last_pos = min(pos_z, base + tile_z * kKeys - 1);
-  int n_lp = tile_a < tile_z ? last_pos / P - lp0 + 1 : 0;
-  if (n_lp > p.tab_cap || !slot_ok) {
-    if (tid == 0) raise_status(p.kv.status, PACE_DEV_BAD_INDEX);
-    n_lp = slot_ok ? min(n_lp, p.tab_cap) : 0;
-  }
-  for (int i = tid; i < n_lp; i += kThreads) {
-    const int pg = view_page(p.kv, slot, lp0 + i);
-    if (pg < 0) raise_status(p.kv.status, PACE_DEV_BAD_INDEX);
-    tab[i] = pg;
+  // values of keys no box ever brings are multiplied by zero weights and must be numbers
+  {
+    uint4* z = reinterpret_cast<uint4*>(smem + sm.ring);
+    const int used = min(p.n_stages, tile_z - tile_a) * STAGE / 16;
+    for (int i = tid; i < used; i += kThreads) z[i] = make_uint4(0, 0, 0, 0);
+    fence_proxy_async();
   }
   __syncthreads();
 
-  auto load_tile = [&](int t) {
-    const uint32_t dst = s_ring + (uint32_t)((t - tile_a) % p.n_stages) * sm.stage_bytes;
-    auto plane = [&](const __nv_bfloat16* src, uint32_t to, int stride, int width16) {
-      const int pieces = width16 / 8;
-      for (int i = tid; i < kKeys * pieces; i += kThreads) {
-        const int j = i / pieces, c = i - j * pieces, pos = base + t * kKeys + j;
-        const int lp = (p.page_shift >= 0 ? pos >> p.page_shift : pos / P);
-        const int in = pos - lp * P;
-        int pg = -1;
-        if (pos <= pos_z && lp - lp0 < n_lp) pg = tab[lp - lp0];
-        const bool ok = pg >= 0 && (c + 1) * 8 <= p.row;
-        cp_async16(to + j * stride + c * 16, ok ? src + (((size_t)pg * Hkv + g) * P + in) * p.row + c * 8 : src, ok);
+  if (warp == kConsumers / 32) {
+    // ================================ producer ================================
+    const int slot = p.st.slot[e];
+    const bool slot_ok = slot >= 0 && slot < p.kv.max_seqs;
+    int page = 0, s = 0, ph = 0, issued = 0;
+    for (int t = tile_a; t < tile_z; ++t) {
+      if (((t - tile_a) & 31) == 0) {  // the next 32 tiles' pages, one per lane
+        page = 0;
+        if (t + lane < tile_z) {
+          page = slot_ok ? view_page(p.kv, slot, base / kKeys + t + lane) : -1;
+          if (page < 0) {
+            raise_status(p.kv.status, PACE_DEV_BAD_INDEX);
+            page = 0;
+          }
+        }
       }
-    };
-    plane(p.kv.k, dst, KSB, p.dk16);
-    if (!p.shared_rows) plane(p.kv.v, dst + sm.k_bytes, VSB, p.dv16);
-  };
+      const int pg = __shfl_sync(0xffffffffu, page, (t - tile_a) & 31);
+      if (issued >= p.n_stages && !__all_sync(0xffffffffu, mbar_wait(&empty[s], ph ^ 1, abort))) break;
+      const int p0 = base + t * kKeys;
+      const int box_a = max(0, key_a - p0) / kBoxRows, box_z = min(kKeys, pos_z + 1 - p0 + kBoxRows - 1) / kBoxRows;
+      if (lane == 0) mbar_arrive_expect_tx(&full[s], (uint32_t)((box_z - box_a) * blocks * kBox));
+      __syncwarp();
+      unsigned char* st = smem + sm.ring + (size_t)s * STAGE;
+      const int n = (box_z - box_a) * blocks;
+      for (int i = lane; i < n; i += 32) {
+        const int bx = box_a + i / blocks, b = i % blocks;
+        const bool is_v = b >= p.k_blocks;
+        tma_load_3d(st + b * kBlock + bx * kBox, is_v ? &tmV : &tmK, (is_v ? b - p.k_blocks : b) * 64, bx * kBoxRows, pg * Hkv + g,
+                    &full[s]);
+      }
+      ++issued;
+      if (++s == p.n_stages) s = 0, ph ^= 1;
+    }
+    if (*abort) {  // copies in flight land before the block's shared memory is released
+      for (int k = issued > p.n_stages ? issued - p.n_stages : 0; k < issued; ++k) mbar_wait(&full[k % p.n_stages], (k / p.n_stages) & 1);
+    }
+    if (ns > 1) {
+      cg::cluster_group cl = cg::this_cluster();
+      cl.sync();
+      cl.sync();
+    }
+    return;
+  }
 
-  for (int k = 0; k < p.n_stages - 1; ++k) {
-    if (tile_a + k < tile_z) load_tile(tile_a + k);
-    asm volatile("cp.async.commit_group;" ::: "memory");
+  // ---- consumers: the query rows ----
+  {
+    const int pieces = p.dk16 / 8;
+    for (int r = warp; r < MR; r += kConsumers / 32) {
+      const int rr = min(r0 + r, R - 1), tok = rr / p.Gq, hh = g * p.Gq + rr - tok * p.Gq;
+      const __nv_bfloat16* src = p.q + ((size_t)(t0 + tok) * p.H + hh) * p.q_elems;
+      for (int c = lane; c < pieces; c += 32) {
+        const bool ok = r < live && (c + 1) * 8 <= p.q_elems;
+        cp_async16(s_q + r * QSB + c * 16, src + (ok ? c * 8 : 0), ok);
+      }
+    }
+    asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
+    consumer_sync();
   }
 
   // softmax role of this thread: one row, keys 4 (sub + TPR i) + 0..3
@@ -179,14 +208,12 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kern
         for (int d = 0; d < 4; ++d) o[a][b][c][d] = 0.f;
 
   const int n_groups = p.dv16 / 16, ksteps = p.dk16 / 16;
+  const int v_off = p.v_blocks ? p.k_blocks * kBlock : 0;
+  int st_i = 0, st_ph = 0;
   for (int t = tile_a; t < tile_z; ++t) {
-    // (one group is committed per tile, an empty one at the end: all but the newest n_stages - 2 are complete)
-    if (p.n_stages == 2) asm volatile("cp.async.wait_group 0;" ::: "memory");
-    else asm volatile("cp.async.wait_group 1;" ::: "memory");
-    __syncthreads();  // the tile is here for everybody, and everybody is done with the stage that is filled next
-    if (t + p.n_stages - 1 < tile_z) load_tile(t + p.n_stages - 1);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    const uint32_t stage = s_ring + (uint32_t)((t - tile_a) % p.n_stages) * sm.stage_bytes;
+    // (a wait that ran out raises the flag, which cuts the waits behind it short; nobody leaves the common barriers)
+    mbar_wait(&full[st_i], st_ph, abort);
+    const uint32_t stage = s_ring + (uint32_t)st_i * STAGE;
     // ---- scores ----
     {
       float c[MT][2][4];
@@ -196,30 +223,33 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kern
         for (int b = 0; b < 2; ++b)
 #pragma unroll
           for (int d = 0; d < 4; ++d) c[a][b][d] = 0.f;
-      // ldmatrix x4 over two k-steps of this warp's eight keys; A: rows lane % 16, column half lane / 16
-      const uint32_t kb = stage + (warp * 8 + (lane & 7)) * KSB + (lane >> 3) * 16;
-      const uint32_t qa = s_q + (lane & 15) * KSB + (lane >> 4) * 16;
+      // ldmatrix x4 over two k-steps of this warp's eight keys; A: rows lane % 16, column half lane / 16.
+      // Key tiles: 64-column blocks, 16-byte piece c of row r at ((c ^ r % 8) * 16)
+      const uint32_t kb = stage + (warp * 8 + (lane & 7)) * 128;
+      const uint32_t kc = (uint32_t)((lane >> 3) ^ (lane & 7)) << 4;   // piece 0 .. 3 of this lane's matrix; 4 .. 7: bit 6 flipped
+      const uint32_t qa = s_q + (lane & 15) * QSB + (lane >> 4) * 16;
       int kk = 0;
+#pragma unroll 2
       for (; kk + 2 <= ksteps; kk += 2) {
         uint32_t b[4];
-        ldsm4(kb + kk * 32, b);
+        ldsm4(kb + (kk >> 2) * kBlock + (kc ^ ((kk & 2) << 5)), b);
 #pragma unroll
         for (int a = 0; a < MT; ++a) {
           uint32_t q0[4], q1[4];
-          ldsm4(qa + a * 16 * KSB + kk * 32, q0);
-          ldsm4(qa + a * 16 * KSB + kk * 32 + 32, q1);
+          ldsm4(qa + a * 16 * QSB + kk * 32, q0);
+          ldsm4(qa + a * 16 * QSB + kk * 32 + 32, q1);
           mma16816(c[a][0], q0, b[0], b[1]);
           mma16816(c[a][1], q1, b[2], b[3]);
         }
       }
       if (kk < ksteps) {
-        uint32_t b0, b1;
-        ldsm2(stage + (warp * 8 + (lane & 7)) * KSB + ((lane >> 3) & 1) * 16 + kk * 32, b0, b1);
+        uint32_t b[4];   // (the second step's pieces lie in the same block: zeros or what follows, not used)
+        ldsm4(kb + (kk >> 2) * kBlock + (kc ^ ((kk & 2) << 5)), b);
 #pragma unroll
         for (int a = 0; a < MT; ++a) {
           uint32_t q0[4];
-          ldsm4(qa + a * 16 * KSB + kk * 32, q0);
-          mma16816(c[a][0], q0, b0, b1);
+          ldsm4(qa + a * 16 * QSB + kk * 32, q0);
+          mma16816(c[a][0], q0, b[0], b[1]);
         }
       }
       const int col = warp * 8 + (lane & 3) * 2;
@@ -230,7 +260,7 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kern
         *reinterpret_cast<float2*>(S + (r + 8) * kSS + col) = make_float2(c[a][0][2] + c[a][1][2], c[a][0][3] + c[a][1][3]);
       }
     }
-    __syncthreads();
+    consumer_sync();
     // ---- softmax ----
     {
       float x[KPT];
@@ -273,7 +303,7 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kern
       l = l * f + sum;
       if (sub == 0) alpha[srow] = f;
     }
-    __syncthreads();
+    consumer_sync();
     // ---- values ----
     if (warp < n_groups) {
 #pragma unroll
@@ -292,7 +322,9 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kern
         }
       }
       const uint32_t pa = (uint32_t)(lane & 15) * (kPS * 2) + (lane >> 4) * 16;
-      const uint32_t vb = stage + v_off + (lane & 15) * VSB + (lane >> 4) * 16;
+      // rows lane % 16 of a k-step; the group's two pieces by lane / 16
+      const uint32_t vb = stage + v_off + (lane & 15) * 128;
+      const uint32_t vh = (uint32_t)(lane >> 4), vx = (uint32_t)(lane & 7);
 #pragma unroll
       for (int ks = 0; ks < kKeys / 16; ++ks) {
         uint32_t ah[MT][4], al[MT][4];
@@ -306,7 +338,7 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kern
           const int gi = warp + 8 * b;
           if (gi < n_groups) {
             uint32_t v[4];
-            ldsm4_t(vb + ks * 16 * VSB + gi * 32, v);
+            ldsm4_t(vb + (gi >> 2) * kBlock + ks * 16 * 128 + (((((uint32_t)gi & 3) * 2 + vh) ^ vx) << 4), v);
 #pragma unroll
             for (int a = 0; a < MT; ++a) {
               mma16816(o[a][b][0], ah[a], v[0], v[1]);
@@ -318,9 +350,12 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kern
         }
       }
     }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[st_i]);
+    if (++st_i == p.n_stages) st_i = 0, st_ph ^= 1;
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
-  __syncthreads();
+  consumer_sync();
+  if (tid == 0 && *abort) raise_status(p.kv.status, PACE_DEV_WAIT_TIMEOUT);
 
   // ---- this block's results to shared memory, merge over the cluster ----
   float* O = reinterpret_cast<float*>(smem + sm.obuf);
@@ -345,9 +380,9 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kern
   }
   cg::cluster_group cl = cg::this_cluster();
   if (ns > 1) cl.sync();
-  else __syncthreads();
+  else consumer_sync();
   const int v4 = p.dv16 / 4;
-  for (int i = share * kThreads + tid; i < live * v4; i += ns * kThreads) {
+  for (int i = share * kConsumers + tid; i < live * v4; i += ns * kConsumers) {
     const int r = i / v4, c = (i - r * v4) * 4;
     const int rr = r0 + r, tok = rr / p.Gq, hh = g * p.Gq + rr - tok * p.Gq;
     float top = -INFINITY, den = 0.f;
@@ -384,7 +419,8 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1) attn_span_kern
 }
 
 template <int MT, int NG>
-int launch_span(SpanParams& p, int ns, int tiles, int entries, int smem, cudaStream_t s) {
+int launch_span(SpanParams& p, const CUtensorMap& tk, const CUtensorMap& tv, int ns, int tiles, int entries, int smem,
+                cudaStream_t s) {
   auto* fn = attn_span_kernel<MT, NG>;
   PACE_CUDA_TRY(cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
   cudaLaunchConfig_t cfg = {};
@@ -398,16 +434,23 @@ int launch_span(SpanParams& p, int ns, int tiles, int entries, int smem, cudaStr
   attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
   cfg.attrs = attr;
   cfg.numAttrs = 1;
-  PACE_CUDA_TRY(cudaLaunchKernelEx(&cfg, fn, p));
+  PACE_CUDA_TRY(cudaLaunchKernelEx(&cfg, fn, p, tk, tv));
   PACE_LAUNCH_CHECK("attn_span_kernel");
   return PACE_OK;
 }
 
-constexpr int kSmemMax = 227 * 1024, kTargetBlocks = 2 * 148;
+constexpr int kSmemMax = 227 * 1024, kSmemHalf = 113 * 1024, kMaxCluster = 8;
+
+int sm_count() {
+  int dev = 0, n = 148;
+  if (cudaGetDevice(&dev) == cudaSuccess) cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev);
+  return n;
+}
 
 // PACE_ERR_UNSUPPORTED: shapes beyond this kernel (the caller takes the CUDA-core one)
 int span_mma(const pace_kv_pool_t* pl, int layer, const pace_step_t& st, const pace_attn_span_args_t& a, cudaStream_t s) {
   SpanParams p;
+  const bool shared = pl->row_format == PACE_ROWS_SHARED;
   p.kv = make_view(pl, layer, nullptr);
   p.st = st;
   p.q = static_cast<const __nv_bfloat16*>(a.q);
@@ -418,56 +461,58 @@ int span_mma(const pace_kv_pool_t* pl, int layer, const pace_step_t& st, const p
   p.out_elems = a.out_elems;
   p.H = a.n_q_heads;
   p.Gq = a.n_q_heads / pl->n_kv_heads;
-  p.dk = a.dim;
   p.dv = a.vdim;
-  p.row = pl->head_dim;
   p.dk16 = (a.dim + 15) / 16 * 16;
   p.dv16 = (a.vdim + 15) / 16 * 16;
-  p.shared_rows = pl->row_format == PACE_ROWS_SHARED;
+  p.k_blocks = (a.dim + 63) / 64;
+  p.v_blocks = shared ? 0 : (a.vdim + 63) / 64;
   p.entry0 = a.entry_begin;
   p.span = a.span;
   p.span_size = a.span_size;
   p.scale_log2 = a.scale * kLog2e;
-  p.page_shift = -1;
-  for (int k = 0; k < 31; ++k)
-    if (pl->page_tokens == (1 << k)) p.page_shift = k;
-  if (a.q_elems % 8 || p.row % 8 || !aligned16(a.q) || !aligned16(pl->pages) || ((uintptr_t)a.out & 7) || p.dv16 > 512)
-    return PACE_ERR_UNSUPPORTED;
   // (q rows are read in pieces of eight: the caller keeps what lies between dim and the next multiple of 8 zero)
-  if (p.shared_rows && p.dv16 > p.dk16) return PACE_ERR_UNSUPPORTED;
-  const int rows = a.max_tokens * p.Gq;
-  int keys = a.max_keys;   // visible keys of a tile, at most
-  int MT = rows <= 16 ? 1 : rows <= 32 ? 2 : 4;
+  if (pl->page_tokens != kKeys || a.q_elems % 8 || pl->head_dim % 8 || !aligned16(a.q) || !aligned16(pl->pages) ||
+      ((uintptr_t)a.out & 7) || p.dv16 > 512 || (shared && p.dv16 > p.k_blocks * 64))
+    return PACE_ERR_UNSUPPORTED;
+  const int E = a.entry_end - a.entry_begin, rows = a.max_tokens * p.Gq, blocks = p.k_blocks + p.v_blocks, sms = sm_count();
   const int NG = p.dv16 <= 128 ? 1 : p.dv16 <= 256 ? 2 : 4;
-  for (;; MT >>= 1) {
-    if (MT == 0) return PACE_ERR_UNSUPPORTED;
-    const int tok = (16 * MT - 1) / p.Gq + 2;   // tokens a tile can touch
-    int k = keys;
-    if (a.span != PACE_SPAN_ALL && (long long)a.span_size + tok < k) k = a.span_size + tok;
-    const int tiles_k = k / kKeys + 2;
-    const int tiles = (rows + 16 * MT - 1) / (16 * MT);
-    const long long units = (long long)tiles * pl->n_kv_heads * (a.entry_end - a.entry_begin);
-    int ns = 1;
-    while (ns < 8 && units * ns * 2 <= kTargetBlocks && tiles_k >= ns * 2) ns *= 2;
-    p.tab_cap = ((tiles_k + ns - 1) / ns + 1) * kKeys / pl->page_tokens + 2;
-    int smem = 0;
-    for (p.n_stages = 3; p.n_stages >= 2; --p.n_stages) {
-      smem = span_smem(16 * MT, p.dk16, p.dv16, p.shared_rows, p.n_stages, p.tab_cap).total;
-      // a third stage only where two blocks still share an SM, or where it is free
-      if (smem <= (p.n_stages == 3 ? kSmemMax / 2 - 1024 : kSmemMax)) break;
+  for (int MT = rows <= 16 ? 1 : rows <= 32 ? 2 : 4; MT; MT >>= 1) {
+    int smem = 0, resident = 2;
+    p.n_stages = 3;
+    smem = span_smem(16 * MT, p.dk16, p.dv16, blocks, 3).total;
+    if (smem > kSmemHalf || MT * NG > 4) {
+      resident = 1;
+      for (p.n_stages = 6; p.n_stages >= 2; --p.n_stages) {
+        smem = span_smem(16 * MT, p.dk16, p.dv16, blocks, p.n_stages).total;
+        if (smem <= kSmemMax) break;
+      }
+      if (p.n_stages < 2) continue;
     }
-    if (p.n_stages < 2) continue;
-    if (units > 0x7fffffffLL || (long long)tiles * pl->n_kv_heads > 65535 || a.entry_end - a.entry_begin > 65535)
-      return PACE_ERR_UNSUPPORTED;
-    const int E = a.entry_end - a.entry_begin;
+    const int tok = (16 * MT - 1) / p.Gq + 2;   // tokens a tile can touch
+    int keys = a.max_keys;                      // visible keys of a tile, at most
+    if (a.span != PACE_SPAN_ALL && (long long)a.span_size + tok < keys) keys = a.span_size + tok;
+    const int tiles_k = keys / kKeys + 1, tiles = (rows + 16 * MT - 1) / (16 * MT);
+    const long long units = (long long)tiles * pl->n_kv_heads * E;
+    if ((long long)tiles * pl->n_kv_heads > 65535 || E > 65535) return PACE_ERR_UNSUPPORTED;
+    // the share count that leaves the fewest tiles per block while all blocks are resident at once
+    int ns = 1;
+    for (int k = 2; k <= kMaxCluster && units * k <= (long long)resident * sms; ++k)
+      if ((tiles_k + k - 1) / k < (tiles_k + ns - 1) / ns) ns = k;
+    CUtensorMap tk, tv;
+    const uint64_t row = (uint64_t)pl->head_dim;
+    const uint64_t dims[3] = {row, kKeys, (uint64_t)pl->n_pages * pl->n_kv_heads}, str[2] = {row * 2, row * 2 * kKeys};
+    const uint32_t box[3] = {64, kBoxRows, 1};
+    int rc = tensor_map_bf16(&tk, p.kv.k, 3, dims, str, box);
+    if (rc == PACE_OK) rc = tensor_map_bf16(&tv, p.kv.v, 3, dims, str, box);
+    if (rc != PACE_OK) return rc;
 #define PACE_SPAN_CASE(mt, ng) \
-  if (MT == mt && NG == ng) return launch_span<mt, ng>(p, ns, tiles, E, smem, s);
+  if (MT == mt && NG == ng) return launch_span<mt, ng>(p, tk, tv, ns, tiles, E, smem, s);
     PACE_SPAN_CASE(1, 1) PACE_SPAN_CASE(1, 2) PACE_SPAN_CASE(1, 4)
     PACE_SPAN_CASE(2, 1) PACE_SPAN_CASE(2, 2) PACE_SPAN_CASE(2, 4)
     PACE_SPAN_CASE(4, 1) PACE_SPAN_CASE(4, 2) PACE_SPAN_CASE(4, 4)
 #undef PACE_SPAN_CASE
-    return PACE_ERR_UNSUPPORTED;
   }
+  return PACE_ERR_UNSUPPORTED;
 }
 
 }  // namespace
