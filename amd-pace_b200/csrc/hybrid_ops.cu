@@ -336,53 +336,75 @@ __global__ void __launch_bounds__(512) append_norm_regs_kernel(pace_step_t st, P
     }
 }
 
-// Per-head norms without weights: a warp per head row of (queries, keys, values).
-template <typename T, int V>
+// Per-head norms without weights: LH lanes per head row of (queries, keys, values), V elements an access.
+template <typename T, int V, int LH>
 __global__ void append_heads_kernel(pace_step_t st, PageRows pg, pace_append_norm_args_t a, int row) {
-  const int t = blockIdx.x, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int t = blockIdx.x, lane = threadIdx.x % LH, groups = blockDim.x / LH;
   const int H = a.n_q_heads, G = pg.n_kv_heads, d = a.dim, vd = a.vdim;
   const T* src = static_cast<const T*>(a.qkv) + (size_t)t * a.qkv_stride;
   const int pos = st.tok_pos[t], slot = st.slot[st.tok_entry[t]], lp = pos / pg.page_tokens;
   int page = -1;
   if (slot >= 0 && slot < pg.max_seqs && lp < pg.max_pages_per_seq)
     page = pg.block_table[(size_t)slot * pg.max_pages_per_seq + lp];
-  if (page < 0 || page >= pg.n_pages) {
-    if (threadIdx.x == 0) raise_status(pg.status, PACE_DEV_BAD_INDEX);
-    page = -1;
-  }
   float temp = a.q_mul;
   if (a.temp_coef != 0.f) temp *= 1.0f + a.temp_coef * logf((float)(floor((double)(pos + 1) / a.temp_every) + 1.0));
-  for (int hh = threadIdx.x >> 5; hh < H + 2 * G; hh += warps) {
-    const bool is_q = hh < H, is_v = hh >= H + G;
+  const int rounds = (H + 2 * G + groups - 1) / groups;   // (the same for every thread: shuffles need whole warps)
+  for (int it = 0; it < rounds; ++it) {
+    const int hh = it * groups + threadIdx.x / LH;
+    const bool exists = hh < H + 2 * G, is_q = hh < H, is_v = hh >= H + G;
     const int g = is_v ? hh - H - G : hh - H, n = is_v ? vd : d;
     const T* x = src + (is_q ? hh * d : is_v ? H * d + G * d + g * vd : H * d + g * d);
-    T* dst;
-    if (is_q) dst = static_cast<T*>(a.q_out) + ((size_t)t * H + hh) * row;
-    else dst = reinterpret_cast<T*>(is_v ? pg.v : pg.k) +
-               (((size_t)(page < 0 ? 0 : page) * G + g) * pg.page_tokens + (pos - lp * pg.page_tokens)) * row;
-    float f = 1.f;
-    if (!is_v) {
-      float ss = 0.f;
-      for (int c = lane * V; c < n; c += 32 * V) {
-        float v[V];
-        Vec<T, V>::load(x + c, v);
+    float f = 1.f, first[V], ss = 0.f;
 #pragma unroll
-        for (int j = 0; j < V; ++j) ss = fmaf(v[j], v[j], ss);
-      }
-#pragma unroll
-      for (int o = 16; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      f = 1.0f / sqrtf(ss / (float)n + a.eps);
-      if (is_q) f *= temp;
-    }
-    if (!is_q && page < 0) continue;
-    for (int c = lane * V; c < row; c += 32 * V) {
+    for (int j = 0; j < V; ++j) first[j] = 0.f;
+    for (int c = lane * V; c < n && exists; c += LH * V) {
       float v[V];
-      if (c < n) Vec<T, V>::load(x + c, v);
+      Vec<T, V>::load(x + c, v);
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        ss = fmaf(v[j], v[j], ss);
+        if (c == lane * V) first[j] = v[j];
+      }
+    }
+#pragma unroll
+    for (int o = LH / 2; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!is_v) f = 1.0f / sqrtf(ss / (float)n + a.eps) * (is_q ? temp : 1.f);
+    if (!exists) continue;
+    T* dst;
+    if (is_q) {
+      dst = static_cast<T*>(a.q_out) + ((size_t)t * H + hh) * row;
+    } else {
+      if (page < 0 || page >= pg.n_pages) {
+        if (lane == 0) raise_status(pg.status, PACE_DEV_BAD_INDEX);
+        continue;
+      }
+      dst = reinterpret_cast<T*>(is_v ? pg.v : pg.k) + (((size_t)page * G + g) * pg.page_tokens + (pos - lp * pg.page_tokens)) * row;
+    }
+    for (int c = lane * V; c < row; c += LH * V) {
+      float v[V];
+      if (c == lane * V) {
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[j] = first[j];
+      } else if (c < n) {
+        Vec<T, V>::load(x + c, v);
+      }
 #pragma unroll
       for (int j = 0; j < V; ++j) v[j] = c < n ? v[j] * f : 0.f;
       Vec<T, V>::store(dst + c, v);
     }
   }
+}
+
+template <typename T, int V>
+void launch_append_heads(const pace_step_t& st, const PageRows& pg, const pace_append_norm_args_t& a, int row, cudaStream_t s) {
+  const int heads = a.n_q_heads + 2 * pg.n_kv_heads, lanes = (row + V - 1) / V;
+  auto threads = [&](int lh) {
+    const int n = (heads * lh + 31) / 32 * 32;
+    return n < 256 ? n : 256;
+  };
+  if (lanes <= 8) append_heads_kernel<T, V, 8><<<st.n_tokens, threads(8), 0, s>>>(st, pg, a, row);
+  else if (lanes <= 16) append_heads_kernel<T, V, 16><<<st.n_tokens, threads(16), 0, s>>>(st, pg, a, row);
+  else append_heads_kernel<T, V, 32><<<st.n_tokens, threads(32), 0, s>>>(st, pg, a, row);
 }
 
 template <typename T>
@@ -405,12 +427,8 @@ int launch_append_norm(const pace_kv_pool_t* p, int layer, const pace_step_t& st
   const bool vec = a.dim % V == 0 && a.vdim % V == 0 && row % V == 0 && a.qkv_stride % V == 0 && aligned16(a.qkv) &&
                    aligned16(a.q_out) && (!a.q_norm || aligned16(a.q_norm)) && (!a.k_norm || aligned16(a.k_norm));
   if (a.per_head) {
-    const int heads = a.n_q_heads + 2 * p->n_kv_heads, th = heads < 16 ? heads * 32 : 512;
-    constexpr int V4 = 4;  // 8-byte accesses of bf16: a head of 128 fills a warp
-    const bool v4 = a.dim % V4 == 0 && a.vdim % V4 == 0 && row % V4 == 0 && a.qkv_stride % V4 == 0 && aligned16(a.qkv) &&
-                    aligned16(a.q_out);
-    if (v4) append_heads_kernel<T, V4><<<st.n_tokens, th, 0, s>>>(st, pg, a, row);
-    else append_heads_kernel<T, 1><<<st.n_tokens, th, 0, s>>>(st, pg, a, row);
+    if (vec) launch_append_heads<T, V>(st, pg, a, row, s);
+    else launch_append_heads<T, 1>(st, pg, a, row, s);
     PACE_LAUNCH_CHECK("append_heads_kernel");
     note_pool_write(s);
     return PACE_OK;

@@ -49,6 +49,8 @@ __global__ void __launch_bounds__(256) latent_append_kernel(pace_step_t st, Late
   const int tid = kv ? threadIdx.x - half : threadIdx.x;
   const int n = kv ? a.kv_rank : a.q_rank;
   const T* src = static_cast<const T*>(a.down) + (size_t)t * a.down_stride + (kv ? a.q_rank : 0);
+  const int pos = st.tok_pos[t], lp = pos / lr.page_tokens;
+  const int page = kv ? latent_page(lr, st.slot[st.tok_entry[t]], lp) : 0;   // (in flight while the norm is summed)
   float ss = 0.f;
   for (int c = tid * V; c < n; c += half * V) {
     float x[V];
@@ -66,9 +68,7 @@ __global__ void __launch_bounds__(256) latent_append_kernel(pace_step_t st, Late
   const float r = 1.0f / sqrtf(ss / (float)n + a.eps);
   T* dst = kv ? nullptr : static_cast<T*>(a.cq) + (size_t)t * n;
   const float* wt = kv ? a.kv_norm : a.q_norm;
-  const int pos = st.tok_pos[t];
   if (kv) {
-    const int lp = pos / lr.page_tokens, page = latent_page(lr, st.slot[st.tok_entry[t]], lp);
     if (page < 0) {
       if (tid == 0) raise_status(lr.status, PACE_DEV_BAD_INDEX);
       return;
@@ -117,6 +117,31 @@ __global__ void rotate_heads_kernel(pace_step_t st, pace_rotate_args_t a) {
   }
 }
 
+// the same, four pairs (16 bytes of bf16) a thread
+__global__ void rotate_heads_vec_kernel(pace_step_t st, pace_rotate_args_t a) {
+  const int per = a.pad_dim / 8;
+  const size_t total = (size_t)(a.token_end - a.token_begin) * a.n_heads * per;
+  for (size_t k = blockIdx.x * (size_t)blockDim.x + threadIdx.x; k < total; k += (size_t)gridDim.x * blockDim.x) {
+    const int c = (int)(k % per) * 8, h = (int)(k / per % a.n_heads), t = a.token_begin + (int)(k / ((size_t)per * a.n_heads));
+    float x[8];
+    if (c < a.rot_dim) {
+      Vec<__nv_bfloat16, 8>::load(static_cast<const __nv_bfloat16*>(a.src) + t * a.src_row + h * a.src_head + c, x);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[j] = 0.f;
+    }
+    const int pos = st.tok_pos[t];
+    if (c / 2 + 4 <= a.rot_pairs && pos < a.table_rows) {
+      float cs[4], sn[4];
+      Vec<float, 4>::load(a.cos_table + (size_t)pos * a.rot_pairs + c / 2, cs);
+      Vec<float, 4>::load(a.sin_table + (size_t)pos * a.rot_pairs + c / 2, sn);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) turn(cs[j], sn[j], x[2 * j], x[2 * j + 1]);
+    }
+    Vec<__nv_bfloat16, 8>::store(static_cast<__nv_bfloat16*>(a.dst) + t * a.dst_row + h * a.dst_head + c, x);
+  }
+}
+
 // a thread per 16 bytes
 __global__ void latent_gather_kernel(LatentRows lr, const int32_t* __restrict__ slot, const int32_t* __restrict__ pos, int n,
                                      uint4* __restrict__ out, int pieces) {
@@ -142,10 +167,10 @@ template <typename T>
 int append_t(const pace_kv_pool_t* p, int layer, const pace_step_t& st, const pace_latent_append_args_t& a, cudaStream_t s) {
   const int row = p->head_dim * 2 / (int)sizeof(T);
   if (a.kv_rank + a.rot_dim > row) return PACE_ERR_INVALID;
-  constexpr int V = 4;
+  constexpr int V = 16 / sizeof(T);
   const bool vec = a.q_rank % V == 0 && a.kv_rank % V == 0 && a.down_stride % V == 0 && aligned16(a.down) && aligned16(a.cq) &&
                    aligned16(a.q_norm) && aligned16(a.kv_norm) && row % V == 0;
-  if (vec) latent_append_kernel<T, V><<<st.n_tokens, 256, 0, s>>>(st, latent_rows(p, layer), a, row);
+  if (vec) latent_append_kernel<T, V><<<st.n_tokens, 128, 0, s>>>(st, latent_rows(p, layer), a, row);
   else latent_append_kernel<T, 1><<<st.n_tokens, 256, 0, s>>>(st, latent_rows(p, layer), a, row);
   PACE_LAUNCH_CHECK("latent_append_kernel");
   note_pool_write(s);
@@ -185,7 +210,11 @@ int pace_rotate_heads(const pace_step_t* st, const pace_rotate_args_t* a, void* 
   if (a->rot_pairs > 0 && (!a->cos_table || !a->sin_table)) return PACE_ERR_INVALID;
   if (a->token_begin >= a->token_end || a->pad_dim == 0) return PACE_OK;
   const size_t n = (size_t)(a->token_end - a->token_begin) * a->n_heads * ((a->pad_dim + 1) / 2);
-  if (a->dtype == PACE_DTYPE_BF16) rotate_heads_kernel<__nv_bfloat16><<<blocks_for(n), 256, 0, (cudaStream_t)stream>>>(*st, *a);
+  const bool vec = a->dtype == PACE_DTYPE_BF16 && a->rot_dim % 8 == 0 && a->pad_dim % 8 == 0 && a->rot_pairs % 4 == 0 &&
+                   (a->src_row | a->src_head | a->dst_row | a->dst_head) % 8 == 0 && aligned16(a->src) && aligned16(a->dst) &&
+                   aligned16(a->cos_table) && aligned16(a->sin_table);
+  if (vec) rotate_heads_vec_kernel<<<blocks_for(n / 4), 256, 0, (cudaStream_t)stream>>>(*st, *a);
+  else if (a->dtype == PACE_DTYPE_BF16) rotate_heads_kernel<__nv_bfloat16><<<blocks_for(n), 256, 0, (cudaStream_t)stream>>>(*st, *a);
   else if (a->dtype == PACE_DTYPE_FP32) rotate_heads_kernel<float><<<blocks_for(n), 256, 0, (cudaStream_t)stream>>>(*st, *a);
   else return PACE_ERR_INVALID;
   PACE_LAUNCH_CHECK("rotate_heads_kernel");

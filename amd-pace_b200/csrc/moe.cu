@@ -6,8 +6,9 @@
 // tokens): two accumulators that share every token tile - gate and up rows of the same features (first product), two
 // neighbouring row tiles (second product).  Persistent blocks of ten warps: TMA producer, MMA issuer, eight epilogue warps;
 // two sets of accumulators in tensor memory, so that a tile is stored while the next one is computed.  The first
-// product's token rows are gathered by TMA (tile::gather4) through the router's lists; its results are written by expert,
-// and the second product reads them in place.  The tile list is made by every block from the experts' counts: nothing comes
+// product's token rows come through the router's lists: narrow tiles gather them by TMA (tile::gather4), wide ones read
+// rows that moe_spread_kernel has copied into expert order (32 gathers per 64 columns would pace a wide tile).  Its results
+// are written by expert, and the second product reads them in place.  The tile list is made by every block from the experts' counts: nothing comes
 // back to the host.
 #include "hybrid.cuh"
 #include "umma.cuh"
@@ -20,21 +21,28 @@ constexpr int kMaxExperts = 1024, kMaxTop = 64;
 // ---------------------------------------------------------------------------
 // routing
 // ---------------------------------------------------------------------------
-// A warp per token, eight at a time, `rounds` times; tokens are numbered within their expert per block first.
-__global__ void __launch_bounds__(256) moe_route_kernel(pace_moe_route_args_t a, int rounds) {
+// A warp per token.  A block numbers the tokens of an expert among its own first; one block over all tokens (WHOLE) is
+// done with that, several take their place by one atomic per expert.
+template <bool WHOLE>
+__global__ void moe_route_kernel(pace_moe_route_args_t a, int rounds) {
   extern __shared__ float sh[];
-  const int E = a.n_experts, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  float* choice = sh + warp * E;
-  int* cnt = reinterpret_cast<int*>(sh + 8 * E);   // tokens of this block per expert, then its base
+  const int E = a.n_experts, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5, slots = warps * rounds * a.top;
+  float* score = sh + warp * 2 * E;
+  float* choice = score + E;
+  int* cnt = reinterpret_cast<int*>(sh + warps * 2 * E);   // tokens of this block per expert, then the first one's number
+  int* sel = cnt + E;                                      // [token of the block][top]: expert and number in the block
+  const int t_first = blockIdx.x * warps * rounds;
   for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  const int t_first = blockIdx.x * 8 * rounds;
   for (int r = 0; r < rounds; ++r) {
-    const int t = t_first + r * 8 + warp;
+    const int local = r * warps + warp, t = t_first + local;
     if (t >= a.n_tokens) break;
     const float* z = a.logits + (size_t)t * E;
-    for (int e = lane; e < E; e += 32)
-      choice[e] = 1.0f / (1.0f + expf(-z[e])) + (a.correction ? a.correction[e] : 0.f);
+    for (int e = lane; e < E; e += 32) {
+      score[e] = 1.0f / (1.0f + expf(-z[e]));
+      choice[e] = score[e] + (a.correction ? a.correction[e] : 0.f);
+    }
+    __syncwarp();
     for (int k = 0; k < a.top; ++k) {
       float best = -INFINITY;
       int at = -1;
@@ -47,12 +55,13 @@ __global__ void __launch_bounds__(256) moe_route_kernel(pace_moe_route_args_t a,
         if (i >= 0 && (at < 0 || v > best || (v == best && i < at))) best = v, at = i;
       }
       if (at < 0) at = k;  // (scores that are not numbers: any expert)
-      if (lane == (at & 31)) choice[at] = -INFINITY;
-      if (lane == 0) {
+      if (lane == (at & 31)) {
+        choice[at] = -INFINITY;
         const size_t s = (size_t)t * a.top + k;
         a.slot_expert[s] = at;
-        a.slot_weight[s] = 1.0f / (1.0f + expf(-z[at]));
-        a.slot_rank[s] = atomicAdd(&cnt[at], 1);
+        a.slot_weight[s] = score[at];
+        sel[2 * (local * a.top + k)] = at;
+        sel[2 * (local * a.top + k) + 1] = atomicAdd(&cnt[at], 1);
       }
     }
     __syncwarp();
@@ -60,17 +69,23 @@ __global__ void __launch_bounds__(256) moe_route_kernel(pace_moe_route_args_t a,
   __syncthreads();
   for (int e = threadIdx.x; e < E; e += blockDim.x) {
     const int n = cnt[e];
-    cnt[e] = n ? atomicAdd(&a.expert_count[e], n) : 0;
+    if (WHOLE) {
+      a.expert_count[e] = n;
+      cnt[e] = 0;
+    } else {
+      cnt[e] = n ? atomicAdd(&a.expert_count[e], n) : 0;
+    }
   }
   __syncthreads();
-  const int t_last = min(a.n_tokens, t_first + 8 * rounds);
-  for (int i = threadIdx.x; i < (t_last - t_first) * a.top; i += blockDim.x) {
-    const size_t s = (size_t)t_first * a.top + i;
-    const int e = a.slot_expert[s], rank = cnt[e] + a.slot_rank[s];
-    a.slot_rank[s] = rank;
-    if (rank < a.n_tokens) a.expert_list[(size_t)e * a.n_tokens + rank] = (int)(s / a.top);
+  for (int i = threadIdx.x; i < slots; i += blockDim.x) {
+    const int t = t_first + i / a.top;
+    if (t >= a.n_tokens) break;
+    const int e = sel[2 * i], rank = cnt[e] + sel[2 * i + 1];
+    a.slot_rank[(size_t)t_first * a.top + i] = rank;
+    if (rank < a.n_tokens) a.expert_list[(size_t)e * a.n_tokens + rank] = t;
   }
 }
+size_t route_smem(int warps, int rounds, int E, int top) { return (size_t)(2 * warps + 1) * E * 4 + (size_t)warps * rounds * top * 8; }
 
 // ---------------------------------------------------------------------------
 // experts on the CUDA cores: fp32 models, sizes that are not multiples of 8
@@ -145,6 +160,27 @@ int experts_simple(const pace_moe_experts_args_t& a, cudaStream_t s) {
   return PACE_OK;
 }
 
+// token rows -> expert order, a block per token: read once, stored once per chosen expert
+__global__ void __launch_bounds__(256) moe_spread_kernel(pace_moe_experts_args_t a) {
+  __shared__ int row[kMaxTop];
+  const int t = blockIdx.x, lane = threadIdx.x & 31;
+  for (int k = threadIdx.x >> 5; k < a.top; k += blockDim.x >> 5) {
+    const int e = a.slot_expert[(size_t)t * a.top + k];
+    int n = 0;
+    for (int i = lane; i < e; i += 32) n += a.expert_count[i];
+#pragma unroll
+    for (int o = 16; o; o >>= 1) n += __shfl_xor_sync(0xffffffffu, n, o);
+    if (lane == 0) row[k] = n + a.slot_rank[(size_t)t * a.top + k];
+  }
+  __syncthreads();
+  const int pieces = a.width / 8;
+  const uint4* src = static_cast<const uint4*>(a.x) + (size_t)t * pieces;
+  for (int c = threadIdx.x; c < pieces; c += blockDim.x) {
+    const uint4 v = src[c];
+    for (int k = 0; k < a.top; ++k) static_cast<uint4*>(a.scratch)[(size_t)row[k] * pieces + c] = v;
+  }
+}
+
 // ---------------------------------------------------------------------------
 // grouped products on tcgen05
 // ---------------------------------------------------------------------------
@@ -168,8 +204,8 @@ struct Tile {
 template <int NT>
 __host__ __device__ constexpr int stage_bytes() { return 2 * kABytes + NT * 128; }
 
-// GLU: act(gate) * up over gathered tokens; otherwise plain products of the rows in place
-template <int NT, bool GLU>
+// GLU: act(gate) * up; otherwise plain products.  GATHER: token rows through the lists, otherwise in expert order.
+template <int NT, bool GLU, bool GATHER>
 __global__ void __launch_bounds__(kThreads, 1)
     moe_grouped_kernel(const GroupedParams p, const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB) {
   constexpr int STAGE = stage_bytes<NT>();
@@ -250,7 +286,7 @@ __global__ void __launch_bounds__(kThreads, 1)
       const Tile t = tile_of(i);
       const int a0 = t.e * p.a_rows + t.m * (GLU ? 128 : 256), a1 = a0 + p.a_second;
       int r[4];
-      if (GLU) {
+      if (GATHER) {
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int k = 4 * lane + j;
@@ -267,10 +303,10 @@ __global__ void __launch_bounds__(kThreads, 1)
           mbar_arrive_expect_tx(&full[s], STAGE);
           tma_load_2d(st, &tmA, ks * kKStep, a0, &full[s]);
           tma_load_2d(st + kABytes, &tmA, ks * kKStep, a1, &full[s]);
-          if (!GLU) tma_load_2d(st + 2 * kABytes, &tmB, ks * kKStep, t.row0, &full[s]);
+          if (!GATHER) tma_load_2d(st + 2 * kABytes, &tmB, ks * kKStep, t.row0, &full[s]);
         }
         __syncwarp();
-        if (GLU && lane < NT / 4) tma_gather4(st + 2 * kABytes + lane * 512, &tmB, ks * kKStep, r[0], r[1], r[2], r[3], &full[s]);
+        if (GATHER && lane < NT / 4) tma_gather4(st + 2 * kABytes + lane * 512, &tmB, ks * kKStep, r[0], r[1], r[2], r[3], &full[s]);
         ++issued;
         if (++s == S) s = 0, ph ^= 1;
       }
@@ -381,12 +417,12 @@ int sm_count() {
   return n;
 }
 
-template <int NT, bool GLU>
+template <int NT, bool GLU, bool GATHER>
 int grouped(GroupedParams p, const void* weights, const void* rows, int n_b_rows, cudaStream_t s) {
   CUtensorMap tmA, tmB;
   const uint64_t st[1] = {(uint64_t)p.K * 2};
   const uint64_t da[2] = {(uint64_t)p.K, (uint64_t)p.n_experts * p.a_rows}, db[2] = {(uint64_t)p.K, (uint64_t)n_b_rows};
-  const uint32_t ba[2] = {kKStep, 128}, bb[2] = {kKStep, GLU ? 1u : (uint32_t)NT};
+  const uint32_t ba[2] = {kKStep, 128}, bb[2] = {kKStep, GATHER ? 1u : (uint32_t)NT};
   int rc = tensor_map_bf16(&tmA, weights, 2, da, st, ba);
   if (rc == PACE_OK) rc = tensor_map_bf16(&tmB, rows, 2, db, st, bb);
   if (rc != PACE_OK) return rc;
@@ -394,13 +430,13 @@ int grouped(GroupedParams p, const void* weights, const void* rows, int n_b_rows
   if (p.n_stages > 8) p.n_stages = 8;
   p.m_tiles = (p.N + (GLU ? 127 : 255)) / (GLU ? 128 : 256);
   const int smem = p.n_stages * stage_bytes<NT>() + 1024;
-  PACE_CUDA_TRY(cudaFuncSetAttribute(moe_grouped_kernel<NT, GLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-  moe_grouped_kernel<NT, GLU><<<sm_count(), kThreads, smem, s>>>(p, tmA, tmB);
+  PACE_CUDA_TRY(cudaFuncSetAttribute(moe_grouped_kernel<NT, GLU, GATHER>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  moe_grouped_kernel<NT, GLU, GATHER><<<sm_count(), kThreads, smem, s>>>(p, tmA, tmB);
   PACE_LAUNCH_CHECK("moe_grouped_kernel");
   return PACE_OK;
 }
 
-template <int NT>
+template <int NT, bool GATHER>
 int experts_umma(const pace_moe_experts_args_t& a, cudaStream_t s) {
   GroupedParams p;
   p.count = a.expert_count;
@@ -415,14 +451,15 @@ int experts_umma(const pace_moe_experts_args_t& a, cudaStream_t s) {
   p.N = a.ff;
   p.a_rows = 2 * a.ff;
   p.a_second = a.ff;
-  const int rc = grouped<NT, true>(p, a.gate_up, a.x, a.n_tokens, s);
+  const int rc = GATHER ? grouped<NT, true, GATHER>(p, a.gate_up, a.x, a.n_tokens, s)
+                        : grouped<NT, true, GATHER>(p, a.gate_up, a.scratch, p.n_rows, s);
   if (rc != PACE_OK) return rc;
   p.out = static_cast<__nv_bfloat16*>(a.y);
   p.K = a.ff;
   p.N = a.width;
   p.a_rows = a.width;
   p.a_second = 128;
-  return grouped<NT, false>(p, a.down, a.hidden, p.n_rows, s);
+  return grouped<NT, false, false>(p, a.down, a.hidden, p.n_rows, s);
 }
 
 }  // namespace
@@ -438,10 +475,21 @@ int pace_moe_route(const pace_moe_route_args_t* a, void* stream) {
     return PACE_ERR_INVALID;
   if ((int64_t)a->n_tokens * a->top > 0x7fffffff) return PACE_ERR_UNSUPPORTED;
   const cudaStream_t s = (cudaStream_t)stream;
+  if (a->n_tokens > 0 && a->n_tokens <= 64) {
+    const int warps = a->n_tokens < 32 ? a->n_tokens : 32, rounds = (a->n_tokens + warps - 1) / warps;
+    const size_t smem = route_smem(warps, rounds, a->n_experts, a->top);
+    if (smem <= 200 * 1024) {
+      PACE_CUDA_TRY(cudaFuncSetAttribute(moe_route_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+      moe_route_kernel<true><<<1, warps * 32, smem, s>>>(*a, rounds);
+      PACE_LAUNCH_CHECK("moe_route_kernel");
+      return PACE_OK;
+    }
+  }
   PACE_CUDA_TRY(cudaMemsetAsync(a->expert_count, 0, (size_t)a->n_experts * 4, s));
   if (a->n_tokens == 0) return PACE_OK;
-  const int rounds = a->n_tokens <= 8 * 148 ? 1 : 4;
-  moe_route_kernel<<<(a->n_tokens + 8 * rounds - 1) / (8 * rounds), 256, (size_t)9 * a->n_experts * 4, s>>>(*a, rounds);
+  const size_t smem = route_smem(8, 1, a->n_experts, a->top);
+  PACE_CUDA_TRY(cudaFuncSetAttribute(moe_route_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  moe_route_kernel<false><<<(a->n_tokens + 7) / 8, 256, smem, s>>>(*a, 1);
   PACE_LAUNCH_CHECK("moe_route_kernel");
   return PACE_OK;
 }
@@ -463,9 +511,11 @@ int pace_moe_experts(const pace_moe_experts_args_t* a, void* stream) {
   const bool umma = a->width % 8 == 0 && a->ff % 8 == 0 && aligned16(a->x) && aligned16(a->gate_up) && aligned16(a->down) &&
                     aligned16(a->hidden) && aligned16(a->y);
   if (!umma) return experts_simple<__nv_bfloat16>(*a, s);
-  // tokens an expert has on average
-  const int64_t mean = (int64_t)a->n_tokens * a->top / a->n_experts;
-  return mean > 32 ? experts_umma<128>(*a, s) : experts_umma<32>(*a, s);
+  if (!a->scratch) return experts_umma<32, true>(*a, s);
+  if (!a->slot_expert || !a->slot_rank || a->top > kMaxTop || !aligned16(a->scratch)) return PACE_ERR_INVALID;
+  moe_spread_kernel<<<a->n_tokens, 256, 0, s>>>(*a);
+  PACE_LAUNCH_CHECK("moe_spread_kernel");
+  return experts_umma<128, false>(*a, s);
 }
 
 }  // extern "C"

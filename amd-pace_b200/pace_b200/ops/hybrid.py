@@ -98,6 +98,7 @@ def _span(window: Optional[int], chunk: Optional[int]):
     return (_C.SPAN_CHUNK, chunk) if chunk is not None else (_C.SPAN_ALL, 0)
 
 
+MOE_WIDE = 32           # tokens per expert from which wide token tiles are worth the copy
 PROMPT_ROWS = 64        # query rows of an entry from which the tcgen05 prompt kernel is worth a launch
 
 
@@ -211,7 +212,10 @@ def moe_experts(h: torch.Tensor, routed: Routed, gate_up: torch.Tensor, down: to
     n = h.shape[0] * routed.top
     hidden = torch.empty(n, down.shape[2], dtype=h.dtype, device=h.device)
     routed.y = torch.empty(n, down.shape[1], dtype=h.dtype, device=h.device)
-    _OPS.moe_experts(h, gate_up, down, hidden, routed.y, routed.count, routed.lists, status, routed.top, act)
+    # many tokens per expert: wide tiles, over rows that are copied into expert order first
+    scratch = torch.empty(n, h.shape[1], dtype=h.dtype, device=h.device) if n > MOE_WIDE * down.shape[0] else None
+    _OPS.moe_experts(h, gate_up, down, hidden, routed.y, scratch, routed.count, routed.lists, routed.slot_expert, routed.slot_rank,
+                     status, act)
     return routed
 
 

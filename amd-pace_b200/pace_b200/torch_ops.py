@@ -60,8 +60,8 @@ _DEFS.update({
     "glu": "(Tensor x, Tensor(a!) out, int act) -> ()",
     "moe_route": "(Tensor logits, Tensor? correction, Tensor(a!) slot_expert, Tensor(b!) slot_rank, Tensor(c!) slot_weight, "
                  "Tensor(d!) expert_count, Tensor(e!) expert_list) -> ()",
-    "moe_experts": "(Tensor x, Tensor gate_up, Tensor down, Tensor(a!) hidden, Tensor(b!) y, Tensor expert_count, "
-                   "Tensor expert_list, Tensor(c!)? status, int top, int act) -> ()",
+    "moe_experts": "(Tensor x, Tensor gate_up, Tensor down, Tensor(a!) hidden, Tensor(b!) y, Tensor(d!)? scratch, "
+                   "Tensor expert_count, Tensor expert_list, Tensor slot_expert, Tensor slot_rank, Tensor(c!)? status, int act) -> ()",
     "attn_general": "(int pool, Tensor pages, int layer, int step, Tensor q, Tensor(a!) out, int dim, int vdim, "
                     "float scale) -> ()",
     "gate_heads": "(int step, Tensor attn, Tensor gate, Tensor(a!) out, int vdim) -> ()",
@@ -299,13 +299,14 @@ def _moe_route(logits, correction, slot_expert, slot_rank, slot_weight, expert_c
         _C.check(_C.lib.pace_moe_route(C.byref(a), _stream(logits)), "pace_moe_route")
 
 
-def _moe_experts(x, gate_up, down, hidden, y, expert_count, expert_list, status, top, act):
+def _moe_experts(x, gate_up, down, hidden, y, scratch, expert_count, expert_list, slot_expert, slot_rank, status, act):
     a = _C.MoeExpertsArgs()
     a.x, a.gate_up, a.down, a.hidden, a.y = x.data_ptr(), gate_up.data_ptr(), down.data_ptr(), hidden.data_ptr(), y.data_ptr()
     a.expert_count, a.expert_list, a.status = expert_count.data_ptr(), expert_list.data_ptr(), _ptr(status)
+    a.scratch, a.slot_expert, a.slot_rank = _ptr(scratch), slot_expert.data_ptr(), slot_rank.data_ptr()
     a.n_tokens, a.width = x.shape
     a.n_experts, _, a.ff = down.shape
-    a.top, a.act, a.dtype = top, act, _dtype(x)
+    a.top, a.act, a.dtype = slot_expert.shape[1], act, _dtype(x)
     with torch.cuda.device(x.device):
         _C.check(_C.lib.pace_moe_experts(C.byref(a), _stream(x)), "pace_moe_experts")
 

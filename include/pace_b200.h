@@ -594,8 +594,9 @@ int pace_moe_route(const pace_moe_route_args_t* a, void* stream);
  * x dtype [n_tokens][width], gate_up dtype [n_experts][2 ff][width] (gate rows first), down dtype [n_experts][width][ff].
  * hidden [n_tokens * top][ff] and y [n_tokens * top][width] are written by expert: expert e's token of rank r is row
  *     expert_row(e, r) = expert_count[0] + .. + expert_count[e - 1] + r.
- * bf16 with width and ff multiples of 8: grouped products on the tcgen05 tensor cores, weights as the 128-row operand,
- * the tokens' rows gathered by TMA.  Otherwise CUDA cores.  `status` (device int32, may be NULL) takes
+ * bf16 with width and ff multiples of 8: grouped products on the tcgen05 tensor cores, weights as the 128-row operand.
+ * `scratch` (dtype [n_tokens * top][width], or NULL) chooses between tiles of 128 tokens, whose rows are first copied into
+ * expert order there, and (NULL) tiles of 32 tokens gathered by TMA, for few tokens per expert.  Otherwise CUDA cores.  `status` (device int32, may be NULL) takes
  * PACE_DEV_WAIT_TIMEOUT if a bounded wait runs out. */
 typedef struct {
   const void* x;
@@ -603,8 +604,11 @@ typedef struct {
   const void* down;
   void* hidden;
   void* y;
+  void* scratch;
   const int32_t* expert_count;
   const int32_t* expert_list;
+  const int32_t* slot_expert;   /* with scratch: the router's */
+  const int32_t* slot_rank;
   int32_t* status;
   int32_t n_tokens, n_experts, top, width, ff, act, dtype;
 } pace_moe_experts_args_t;
