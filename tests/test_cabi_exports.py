@@ -68,7 +68,8 @@ def test_dispatcher_ops_are_registered_without_a_gpu():
              "kv_read_dense", "pard_accept", "linear_skinny", "attn_decode", "attn_decode_cuda_cores",
              "attn_verify", "attn_prefill", "residual_norm", "kv_append_norm", "attn_general", "gate_heads", "norm_gate",
              "relu_squared", "causal_conv", "rglru_scan", "rglru_step", "lightning_prefill", "lightning_step",
-             "step_decode"]
+             "step_decode", "attn_span", "attn_span_prefill", "latent_append", "rotate_heads", "latent_gather", "glu", "moe_route",
+             "moe_experts"]
     for n in names:
         op = getattr(torch.ops.pace_b200, n)
         assert torch._C._dispatch_has_kernel_for_dispatch_key(f"pace_b200::{n}", "CUDA"), n
