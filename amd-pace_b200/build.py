@@ -14,7 +14,7 @@ ROOT = os.path.dirname(HERE)
 CSRC = os.path.join(HERE, "csrc")
 OUT = os.path.join(HERE, "pace_b200", "libpace_b200.so")
 SOURCES = ["kv_pool.cu", "attn_decode.cu", "attn_mma.cu", "attn_api.cu", "linear_skinny.cu",
-           "hybrid_ops.cu", "attn_general.cu", "recurrent.cu", "lightning.cu", "attn_span.cu", "attn_span_umma.cu", "latent.cu", "moe.cu"]
+           "hybrid_ops.cu", "attn_general.cu", "recurrent.cu", "lightning.cu", "attn_span.cu", "attn_span_keys.cu", "attn_span_umma.cu", "latent.cu", "moe.cu"]
 # fp32 exp, log and divide of these files are the accurate ones (they serve 32-bit models)
 PRECISE = {"hybrid_ops.cu", "attn_general.cu", "recurrent.cu", "lightning.cu", "latent.cu", "moe.cu"}
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")

@@ -11,12 +11,8 @@
 //   values   warp w: all query rows x the 16-column groups w, w + 8, ...
 // At the end every block has (maximum, sum, weighted values) of its keys in shared memory; the blocks of the cluster merge
 // them over distributed shared memory, each a part of the outputs.  No workspace, no atomics, no order that varies.
-#include <cooperative_groups.h>
-
 #include "span.cuh"
 #include "umma.cuh"
-
-namespace cg = cooperative_groups;
 
 namespace pace {
 namespace {
@@ -163,7 +159,7 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1)
       for (int k = issued > p.n_stages ? issued - p.n_stages : 0; k < issued; ++k) mbar_wait(&full[k % p.n_stages], (k / p.n_stages) & 1);
     }
     if (ns > 1) {
-      cg::cluster_group cl = cg::this_cluster();
+      cooperative_groups::cluster_group cl = cooperative_groups::this_cluster();
       cl.sync();
       cl.sync();
     }
@@ -378,43 +374,10 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1)
         }
     }
   }
-  cg::cluster_group cl = cg::this_cluster();
+  cooperative_groups::cluster_group cl = cooperative_groups::this_cluster();
   if (ns > 1) cl.sync();
   else consumer_sync();
-  const int v4 = p.dv16 / 4;
-  for (int i = share * kConsumers + tid; i < live * v4; i += ns * kConsumers) {
-    const int r = i / v4, c = (i - r * v4) * 4;
-    const int rr = r0 + r, tok = rr / p.Gq, hh = g * p.Gq + rr - tok * p.Gq;
-    float top = -INFINITY, den = 0.f;
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (p.sinks) {
-      top = p.sinks[hh] * kLog2e;
-      den = 1.f;
-    }
-    for (int k = 0; k < ns; ++k) {
-      const float2 st = ns > 1 ? *cl.map_shared_rank(ml + r, k) : ml[r];
-      if (st.x == -INFINITY) continue;
-      const float4 v = *reinterpret_cast<const float4*>(ns > 1 ? cl.map_shared_rank(O + r * OS + c, k) : O + r * OS + c);
-      const float tn = fmaxf(top, st.x);
-      const float fa = top == -INFINITY ? 0.f : fast_exp2(top - tn), fb = fast_exp2(st.x - tn);
-      top = tn;
-      den = den * fa + st.y * fb;
-      acc.x = acc.x * fa + v.x * fb;
-      acc.y = acc.y * fa + v.y * fb;
-      acc.z = acc.z * fa + v.z * fb;
-      acc.w = acc.w * fa + v.w * fb;
-    }
-    const float inv = den > 0.f ? 1.0f / den : 0.f;
-    __nv_bfloat16* dst = p.out + ((size_t)(t0 + tok) * p.H + hh) * p.out_elems + c;
-    const float y[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
-    if (c + 4 <= p.dv && (p.out_elems & 3) == 0) {
-      Vec<__nv_bfloat16, 4>::store(dst, y);
-    } else {
-#pragma unroll
-      for (int j = 0; j < 4; ++j)
-        if (c + j < p.dv) dst[j] = __float2bfloat16_rn(y[j]);
-    }
-  }
+  span_merge(O, OS, ml, S, ns, share, tid, kConsumers, live, r0, t0, g, p.Gq, p.H, p.dv, p.dv16, p.sinks, p.out, p.out_elems);
   if (ns > 1) cl.sync();  // nobody leaves while its shared memory is read
 }
 
@@ -530,7 +493,8 @@ extern "C" int pace_attn_span(const pace_kv_pool_t* p, int32_t layer, const pace
   PACE_PROFILE("attn_span", stream, "layer=%d entries=%d tokens<=%d heads=%d dims=%d/%d", layer, a->entry_end - a->entry_begin,
                a->max_tokens, a->n_q_heads, a->dim, a->vdim);
   if (a->dtype == PACE_DTYPE_BF16) {
-    const int rc = span_mma(p, layer, *st, *a, (cudaStream_t)stream);
+    int rc = attn_span_keys(p, layer, *st, *a, (cudaStream_t)stream);
+    if (rc == PACE_ERR_UNSUPPORTED) rc = span_mma(p, layer, *st, *a, (cudaStream_t)stream);
     if (rc != PACE_ERR_UNSUPPORTED) return rc;
   }
   return attn_general_span(p, layer, *st, *a, (cudaStream_t)stream);

@@ -1,6 +1,8 @@
 // Which keys a query sees: plain causality, a sliding window or chunks counted from position 0.
 #pragma once
 
+#include <cooperative_groups.h>
+
 #include "hybrid.cuh"
 
 namespace pace {
@@ -12,9 +14,73 @@ __host__ __device__ __forceinline__ int span_first(int span, int size, int pos) 
   return 0;
 }
 
-// attn_general.cu: the CUDA-core kernel behind pace_attn_span
+// attn_span_keys.cu: latents on tcgen05; attn_general.cu: the CUDA-core kernel behind pace_attn_span
+int attn_span_keys(const pace_kv_pool_t* p, int layer, const pace_step_t& st, const pace_attn_span_args_t& a, cudaStream_t s);
 int attn_general_span(const pace_kv_pool_t* p, int layer, const pace_step_t& st, const pace_attn_span_args_t& a,
                       cudaStream_t s);
+
+#ifdef __CUDACC__
+// The blocks of a cluster have (maximum, sum) ml[row] (log2 units) and weighted values O[row][stride] of their shares of the
+// keys in shared memory, at the same places; every block merges and stores its part of the outputs.  ns (at most 8): blocks
+// of the cluster, `share` this one's number; `threads` threads of the block take part, fac: 8 floats of shared memory per
+// row.  The caller has synchronised the cluster and does so again before anyone leaves.
+__device__ __forceinline__ void span_merge(const float* O, int stride, const float2* ml, float* fac, int ns, int share, int tid,
+                                           int threads, int live, int r0, int t0, int g, int Gq, int H, int dv, int dv16,
+                                           const float* sinks, __nv_bfloat16* out, int out_elems) {
+  cooperative_groups::cluster_group cl = cooperative_groups::this_cluster();
+  // what each share's values are multiplied by, per row
+  for (int r = tid; r < live; r += threads) {
+    float2 st[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k)
+      st[k] = k < ns ? (ns > 1 ? *cl.map_shared_rank(ml + r, k) : ml[r]) : make_float2(-INFINITY, 0.f);
+    const int rr = r0 + r, hh = g * Gq + rr % Gq;
+    const float sink = sinks ? sinks[hh] * kLog2e : -INFINITY;
+    float top = sink;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) top = fmaxf(top, st[k].x);
+    float den = sinks ? fast_exp2(sink - top) : 0.f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      st[k].x = st[k].x == -INFINITY ? 0.f : fast_exp2(st[k].x - top);
+      den = fmaf(st[k].y, st[k].x, den);
+    }
+    const float inv = den > 0.f ? 1.0f / den : 0.f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) fac[r * 8 + k] = st[k].x * inv;
+  }
+  asm volatile("bar.sync 1, %0;" ::"r"(threads) : "memory");
+  const int v4 = dv16 / 4;
+  for (int i = share * threads + tid; i < live * v4; i += ns * threads) {
+    const int r = i / v4, c = (i - r * v4) * 4;
+    const int rr = r0 + r, tok = rr / Gq, hh = g * Gq + rr - tok * Gq;
+    float4 v[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (k < ns && fac[r * 8 + k] != 0.f)   // (a share without keys has nothing there)
+        v[k] = *reinterpret_cast<const float4*>(ns > 1 ? cl.map_shared_rank(O + r * stride + c, k) : O + r * stride + c);
+    }
+    float y[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const float f = fac[r * 8 + k];
+      y[0] = fmaf(v[k].x, f, y[0]);
+      y[1] = fmaf(v[k].y, f, y[1]);
+      y[2] = fmaf(v[k].z, f, y[2]);
+      y[3] = fmaf(v[k].w, f, y[3]);
+    }
+    __nv_bfloat16* dst = out + ((size_t)(t0 + tok) * H + hh) * out_elems + c;
+    if (c + 4 <= dv && (out_elems & 3) == 0) {
+      Vec<__nv_bfloat16, 4>::store(dst, y);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j < dv) dst[j] = __float2bfloat16_rn(y[j]);
+    }
+  }
+}
+#endif  // __CUDACC__
 
 inline bool span_args_ok(const pace_step_t* st, const pace_attn_span_args_t* a, int n_kv_heads) {
   return a && a->q && a->out && a->n_q_heads >= 1 && n_kv_heads >= 1 && a->n_q_heads % n_kv_heads == 0 && a->dim >= 1 &&

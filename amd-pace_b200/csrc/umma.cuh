@@ -73,6 +73,8 @@ __host__ __device__ constexpr uint32_t umma_idesc(int n, bool b_mn_major) {
   return (1u << 4) | (1u << 7) | (1u << 10) | ((b_mn_major ? 1u : 0u) << 16) | ((uint32_t)(n >> 3) << 17) |
          ((uint32_t)(kUmmaRows >> 4) << 24);
 }
+// the same with A M-major (its 64-element column blocks lie LBO apart)
+__host__ __device__ constexpr uint32_t umma_idesc_at(int n) { return umma_idesc(n, false) | (1u << 15); }
 __device__ __forceinline__ void umma_bf16(uint32_t tmem_d, uint64_t a_desc, uint64_t b_desc, uint32_t idesc,
                                           uint32_t accumulate) {
   asm volatile(

@@ -88,10 +88,10 @@ def weights(cfg, seed=0, decided=False):
             mat(mix + "v", m["kv_heads"] * vd, D)
         else:
             mat(mix + "dq", m["q_rank"], D)
-            vec(mix + "dq.norm", m["q_rank"], mean=1.5)
+            vec(mix + "dq.norm", m["q_rank"], mean=1.0)
             mat(mix + "uq", H * (d + m["rot_dim"]), m["q_rank"])
             mat(mix + "dkv", m["kv_rank"] + m["rot_dim"], D)
-            vec(mix + "dkv.norm", m["kv_rank"], mean=1.5)
+            vec(mix + "dkv.norm", m["kv_rank"], mean=1.0)
             mat(mix + "uk", H * d, m["kv_rank"])
             mat(mix + "uv", H * vd, m["kv_rank"])
         if lay["type"] != L1:
