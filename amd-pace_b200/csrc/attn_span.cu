@@ -34,7 +34,7 @@ struct SpanParams {
 };
 
 struct SpanSmem {
-  int ring, q, s, ph, pl, alpha, ml, bars, obuf, total;
+  int ring, q, s, ph, pl, alpha, ml, sink, bars, obuf, total;
 };
 __host__ __device__ inline SpanSmem span_smem(int MR, int dk16, int dv16, int blocks, int n_stages) {
   SpanSmem m;
@@ -53,6 +53,7 @@ __host__ __device__ inline SpanSmem span_smem(int MR, int dk16, int dv16, int bl
   m.pl = take(MR * kPS * 2);
   m.alpha = take(MR * 4);
   m.ml = take(MR * 8);
+  m.sink = take(MR * 4);
   m.bars = take(2 * 8 * 8 + 8);
   m.total = off + 1024;  // (the ring starts at a multiple of 1024)
   return m;
@@ -105,6 +106,15 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1)
   const uint32_t s_ring = smem_u32(smem + sm.ring), s_q = smem_u32(smem + sm.q);
   const int QSB = (p.dk16 + 8) * 2;  // row stride of the queries, bytes: an odd number of 16-byte units
 
+  // the producer's page numbers: asked for now, needed behind the barrier
+  int pages_ahead = 0;
+  if (warp == kConsumers / 32) {
+    asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(&tmK)) : "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(&tmV)) : "memory");
+    const int slot = p.st.slot[e];
+    if (tile_a + lane < tile_z)
+      pages_ahead = slot >= 0 && slot < p.kv.max_seqs ? view_page(p.kv, slot, base / kKeys + tile_a + lane) : -1;
+  }
   if (tid == kConsumers) {
     *abort_flag = 0;
     for (int i = 0; i < p.n_stages; ++i) {
@@ -113,29 +123,37 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1)
     }
     fence_mbar_init();
   }
-  // values of keys no box ever brings are multiplied by zero weights and must be numbers
-  {
-    uint4* z = reinterpret_cast<uint4*>(smem + sm.ring);
-    const int used = min(p.n_stages, tile_z - tile_a) * STAGE / 16;
-    for (int i = tid; i < used; i += kThreads) z[i] = make_uint4(0, 0, 0, 0);
-    fence_proxy_async();
+  // values of keys that no box brings into a stage's first tile are multiplied by zero weights and must be numbers (later
+  // tiles find those of earlier ones)
+  for (int s = 0; s < p.n_stages && tile_a + s < tile_z; ++s) {
+    const int p0 = base + (tile_a + s) * kKeys;
+    const int row_a = max(0, key_a - p0) / kBoxRows * kBoxRows, row_z = min(kKeys, (pos_z - p0) / kBoxRows * kBoxRows + kBoxRows);
+    const int gap = kKeys - (row_z - row_a);   // rows [0, row_a) and [row_z, 64), eight pieces each
+    for (int i = tid; i < blocks * gap * 8; i += kThreads) {
+      const int b = i / (gap * 8), o = i - b * gap * 8, row = (o >> 3) < row_a ? o >> 3 : row_z + (o >> 3) - row_a;
+      *reinterpret_cast<uint4*>(smem + sm.ring + (size_t)s * STAGE + b * kBlock + row * 128 + (o & 7) * 16) = make_uint4(0, 0, 0, 0);
+    }
   }
+  if (tid < MR) {
+    const int rr = min(r0 + tid, R - 1);
+    reinterpret_cast<float*>(smem + sm.sink)[tid] = p.sinks ? p.sinks[g * p.Gq + rr % p.Gq] * kLog2e : -INFINITY;
+  }
+  fence_proxy_async();
   __syncthreads();
 
   if (warp == kConsumers / 32) {
     // ================================ producer ================================
-    const int slot = p.st.slot[e];
-    const bool slot_ok = slot >= 0 && slot < p.kv.max_seqs;
     int page = 0, s = 0, ph = 0, issued = 0;
     for (int t = tile_a; t < tile_z; ++t) {
       if (((t - tile_a) & 31) == 0) {  // the next 32 tiles' pages, one per lane
-        page = 0;
-        if (t + lane < tile_z) {
-          page = slot_ok ? view_page(p.kv, slot, base / kKeys + t + lane) : -1;
-          if (page < 0) {
-            raise_status(p.kv.status, PACE_DEV_BAD_INDEX);
-            page = 0;
-          }
+        page = pages_ahead;
+        if (t > tile_a) {
+          const int slot = p.st.slot[e];
+          page = t + lane >= tile_z ? 0 : slot >= 0 && slot < p.kv.max_seqs ? view_page(p.kv, slot, base / kKeys + t + lane) : -1;
+        }
+        if (page < 0) {
+          raise_status(p.kv.status, PACE_DEV_BAD_INDEX);
+          page = 0;
         }
       }
       const int pg = __shfl_sync(0xffffffffu, page, (t - tile_a) & 31);
@@ -377,7 +395,8 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1)
   cooperative_groups::cluster_group cl = cooperative_groups::this_cluster();
   if (ns > 1) cl.sync();
   else consumer_sync();
-  span_merge(O, OS, ml, S, ns, share, tid, kConsumers, live, r0, t0, g, p.Gq, p.H, p.dv, p.dv16, p.sinks, p.out, p.out_elems);
+  span_merge(O, OS, ml, reinterpret_cast<float*>(smem + sm.sink), S, ns, share, tid, kConsumers, live, r0, t0, g, p.Gq, p.H, p.dv,
+             p.dv16, p.out, p.out_elems);
   if (ns > 1) cl.sync();  // nobody leaves while its shared memory is read
 }
 

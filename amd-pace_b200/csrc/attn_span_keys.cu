@@ -33,7 +33,7 @@ struct KeysParams {
 };
 
 struct KeysSmem {
-  int k, q, p, s, ml, alpha, bars, total;
+  int k, q, p, s, ml, alpha, sink, bars, total;
 };
 __host__ __device__ inline KeysSmem keys_smem(int rows, int k_blocks, int dv16) {
   KeysSmem m;
@@ -51,6 +51,7 @@ __host__ __device__ inline KeysSmem keys_smem(int rows, int k_blocks, int dv16) 
   m.s = take(rows * kSS * 4, 16);
   m.ml = take(rows * 8, 8);
   m.alpha = take(rows * 4 + 16, 16);
+  m.sink = take(rows * 4, 4);
   m.bars = take((2 * kMaxBlocks + 4) * 8, 8);
   m.total = off + 1024;
   return m;
@@ -59,7 +60,9 @@ __host__ __device__ inline KeysSmem keys_smem(int rows, int k_blocks, int dv16) 
 __device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kSoftmax) : "memory"); }
 
 template <int N>  // query rows of a tile
-__global__ void __launch_bounds__(kThreads, 1) attn_span_keys_kernel(const KeysParams p, const __grid_constant__ CUtensorMap tmK) {
+__global__ void __launch_bounds__(kThreads, 1) 
+    attn_span_keys_kernel(const KeysParams p, const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                          const __grid_constant__ CUtensorMap tmPage) {
   constexpr int TPR = kSoftmax / N, PIECES = kKeys / 8 / TPR;
   extern __shared__ unsigned char smem_raw[];
   __shared__ uint32_t tmem_slot;
@@ -85,6 +88,15 @@ __global__ void __launch_bounds__(kThreads, 1) attn_span_keys_kernel(const KeysP
   volatile int* flags = reinterpret_cast<volatile int*>(alpha + N);   // [2] some row's maximum grew; [2]: the abort flag
   volatile int* abort = flags + 2;
 
+  // the producer's page numbers: asked for now, needed behind the barrier
+  int pages_ahead = 0;
+  if (warp == 8) {
+    asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(&tmQ)) : "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(&tmPage)) : "memory");
+    const int slot = p.st.slot[e];
+    if (lane < page_z - page_a)
+      pages_ahead = slot >= 0 && slot < p.kv.max_seqs ? view_page(p.kv, slot, base / kPage + page_a + lane) : -1;
+  }
   if (warp == 9) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(p.tmem_cols)
                  : "memory");
@@ -101,22 +113,20 @@ __global__ void __launch_bounds__(kThreads, 1) attn_span_keys_kernel(const KeysP
     mbar_init(o_full, 1);
     fence_mbar_init();
   }
-  // values of keys no box ever brings are multiplied by zero weights and must be numbers
+  // values of keys that no box of the first chunk brings are multiplied by zero weights and must be numbers (later chunks
+  // find those of the first one)
   if (n_chunks > 0) {
-    uint4* z = reinterpret_cast<uint4*>(smem + sm.k);
-    for (int i = tid; i < KB * kBlock / 16; i += kThreads) z[i] = make_uint4(0, 0, 0, 0);
-  }
-  // the query rows, K-major with the 128-byte swizzle
-  {
-    const int pieces = KB * 8;
-    for (int r = warp; r < N; r += kThreads / 32) {
-      const int rr = min(r0 + r, R - 1), tok = rr / p.Gq, hh = rr - tok * p.Gq;
-      const uint4* src = reinterpret_cast<const uint4*>(p.q + ((size_t)(t0 + tok) * p.H + hh) * p.q_elems);
-      for (int c = lane; c < pieces; c += 32) {
-        const uint4 v = r < live && (c + 1) * 8 <= p.q_elems && c * 8 < p.dim ? __ldg(src + c) : make_uint4(0, 0, 0, 0);
-        *reinterpret_cast<uint4*>(smem + sm.q + (c >> 3) * (N * 128) + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
-      }
+    const int p0 = base + page_a * kPage;
+    const int row_a = max(0, key_a - p0) / kBoxRows * kBoxRows, row_z = min(kKeys, (end - p0 + kBoxRows - 1) / kBoxRows * kBoxRows);
+    const int gap = kKeys - (row_z - row_a);   // rows [0, row_a) and [row_z, 128), eight pieces each
+    for (int i = tid; i < KB * gap * 8; i += kThreads) {
+      const int b = i / (gap * 8), o = i - b * gap * 8, row = (o >> 3) < row_a ? o >> 3 : row_z + (o >> 3) - row_a;
+      *reinterpret_cast<uint4*>(smem + sm.k + b * kBlock + row * 128 + (o & 7) * 16) = make_uint4(0, 0, 0, 0);
     }
+  }
+  if (tid < N) {
+    const int rr = min(r0 + tid, R - 1);
+    reinterpret_cast<float*>(smem + sm.sink)[tid] = p.sinks ? p.sinks[rr % p.Gq] * kLog2e : -INFINITY;
   }
   fence_proxy_async();  // generic-proxy writes before TMA's and the tensor core's accesses
   tc_fence_before();
@@ -126,33 +136,55 @@ __global__ void __launch_bounds__(kThreads, 1) attn_span_keys_kernel(const KeysP
 
   if (warp == 8) {
     // ================================ producer ================================
-    const int slot = p.st.slot[e];
-    const bool slot_ok = slot >= 0 && slot < p.kv.max_seqs;
     bool ok = true;
+    auto page_of = [&](int i) {   // i-th page of the share
+      int pg = 0;
+      if (i < 32) {
+        pg = __shfl_sync(0xffffffffu, pages_ahead, i);
+      } else {
+        const int slot = p.st.slot[e];
+        pg = slot >= 0 && slot < p.kv.max_seqs ? view_page(p.kv, slot, base / kPage + page_a + i) : -1;
+      }
+      if (pg < 0) {
+        if (lane == 0) raise_status(p.kv.status, PACE_DEV_BAD_INDEX);
+        pg = 0;
+      }
+      return pg;
+    };
     for (int c = 0; c < n_chunks && ok; ++c) {
       const int p0 = base + (page_a + 2 * c) * kPage;
       int page[2] = {0, 0};
 #pragma unroll
       for (int h = 0; h < 2; ++h)
-        if (p0 + h * kPage < end) {
-          page[h] = slot_ok ? view_page(p.kv, slot, p0 / kPage + h) : -1;
-          if (page[h] < 0) {
-            if (lane == 0) raise_status(p.kv.status, PACE_DEV_BAD_INDEX);
-            page[h] = 0;
-          }
-        }
+        if (p0 + h * kPage < end) page[h] = page_of(2 * c + h);
       const int box_a = max(0, key_a - p0) / kBoxRows, box_z = min(kKeys, end - p0 + kBoxRows - 1) / kBoxRows;
       for (int b = 0; b < KB; ++b) {
         if (c > 0 && !__all_sync(0xffffffffu, mbar_wait(&empty[b], (c - 1) & 1, abort))) {
           ok = false;
           break;
         }
-        if (lane == 0) mbar_arrive_expect_tx(&full[b], (uint32_t)(box_z - box_a) * kBox);
+        if (lane == 0) {
+          mbar_arrive_expect_tx(&full[b], (uint32_t)(box_z - box_a) * kBox + (c == 0 ? N * 128u : 0u));
+          if (c == 0) tma_load_2d(smem + sm.q + b * (N * 128), &tmQ, b * 64, t0 * p.H + r0, &full[b]);
+        }
         __syncwarp();
-        const int bx = box_a + lane;
-        if (bx < box_z)
-          tma_load_3d(smem + sm.k + b * kBlock + bx * kBox, &tmK, b * 64, bx * kBoxRows & (kPage - 1), page[bx * kBoxRows >= kPage ? 1 : 0],
+        // whole pages in one box each, others by 16 keys
+        const int bx = box_a + lane, half = bx >> 2;
+        const bool whole = box_a <= 4 * half && box_z >= 4 * half + 4;
+        if (bx < box_z && whole) {
+          if ((bx & 3) == 0) tma_load_3d(smem + sm.k + b * kBlock + bx * kBox, &tmPage, b * 64, 0, page[half & 1], &full[b]);
+        } else if (bx < box_z)
+          tma_load_3d(smem + sm.k + b * kBlock + bx * kBox, &tmK, b * 64, bx * kBoxRows & (kPage - 1), page[half & 1],
                       &full[b]);
+      }
+      // what the next chunk needs starts for L2 while this one is worked on
+      if (c + 1 < n_chunks) {
+        const int i = 2 * (c + 1);
+        const int pg0 = page_of(i), pg1 = p0 + 3 * kPage < end ? page_of(i + 1) : -1;
+        for (int k = lane; k < 2 * KB; k += 32) {
+          const int pg = k < KB ? pg0 : pg1;
+          if (pg >= 0) tma_prefetch_3d(&tmPage, (k < KB ? k : k - KB) * 64, 0, pg);
+        }
       }
       if (!ok)   // copies in flight land before the block's shared memory is released
         for (int b = 0; b < KB; ++b) mbar_wait(&full[b], (c - 1) & 1), mbar_wait(&full[b], c & 1, abort, 1024);
@@ -319,7 +351,7 @@ __global__ void __launch_bounds__(kThreads, 1) attn_span_keys_kernel(const KeysP
   cooperative_groups::cluster_group cl = cooperative_groups::this_cluster();
   if (ns > 1) cl.sync();
   span_merge(reinterpret_cast<float*>(smem + sm.k), p.dv16 + 4, reinterpret_cast<float2*>(smem + sm.ml),
-             reinterpret_cast<float*>(smem + sm.s), ns, share, tid, kThreads, live, r0, t0, 0, p.Gq, p.H, p.dv, p.dv16, p.sinks, p.out, p.out_elems);
+             reinterpret_cast<float*>(smem + sm.sink), reinterpret_cast<float*>(smem + sm.s), ns, share, tid, kThreads, live, r0, t0, 0, p.Gq, p.H, p.dv, p.dv16, p.out, p.out_elems);
   if (ns > 1) cl.sync();  // nobody leaves while its shared memory is read
 }
 
@@ -330,7 +362,7 @@ int sm_count() {
 }
 
 template <int N>
-int launch_keys(KeysParams& p, const CUtensorMap& tk, int max_tokens, int max_keys, int entries, cudaStream_t s) {
+int launch_keys(KeysParams& p, const CUtensorMap& tk, const CUtensorMap& tpage, int max_tokens, int max_keys, int entries, cudaStream_t s) {
   const int smem = keys_smem(N, p.k_blocks, p.dv16).total;
   if (smem > 227 * 1024 - 64) return PACE_ERR_UNSUPPORTED;
   p.tmem_cols = 128;
@@ -345,6 +377,11 @@ int launch_keys(KeysParams& p, const CUtensorMap& tk, int max_tokens, int max_ke
   int ns = 1;
   for (int k = 2; k <= 8 && units * k <= sm_count(); ++k)
     if ((pages + k - 1) / k < (pages + ns - 1) / ns) ns = k;
+  CUtensorMap tq;
+  const uint64_t dims[2] = {(uint64_t)p.q_elems, (uint64_t)p.st.n_tokens * p.H}, str[1] = {(uint64_t)p.q_elems * 2};
+  const uint32_t box[2] = {64, N};
+  const int rc = tensor_map_bf16(&tq, p.q, 2, dims, str, box);
+  if (rc != PACE_OK) return rc;
   auto* fn = attn_span_keys_kernel<N>;
   PACE_CUDA_TRY(cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
   cudaLaunchConfig_t cfg = {};
@@ -358,7 +395,7 @@ int launch_keys(KeysParams& p, const CUtensorMap& tk, int max_tokens, int max_ke
   attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
   cfg.attrs = attr;
   cfg.numAttrs = 1;
-  PACE_CUDA_TRY(cudaLaunchKernelEx(&cfg, fn, p, tk));
+  PACE_CUDA_TRY(cudaLaunchKernelEx(&cfg, fn, p, tq, tk, tpage));
   PACE_LAUNCH_CHECK("attn_span_keys_kernel");
   return PACE_OK;
 }
@@ -391,15 +428,17 @@ int attn_span_keys(const pace_kv_pool_t* pl, int layer, const pace_step_t& st, c
   p.span_size = a.span_size;
   p.scale_log2 = a.scale * kLog2e;
   if (p.k_blocks > kMaxBlocks) return PACE_ERR_UNSUPPORTED;
-  CUtensorMap tk;
+  CUtensorMap tk, tpage;
   const uint64_t row = (uint64_t)pl->head_dim;
   const uint64_t dims[3] = {row, kPage, (uint64_t)pl->n_pages}, str[2] = {row * 2, row * 2 * kPage};
   const uint32_t box[3] = {64, kBoxRows, 1};
-  const int rc = tensor_map_bf16(&tk, p.kv.k, 3, dims, str, box);
+  const uint32_t whole[3] = {64, kPage, 1};
+  int rc = tensor_map_bf16(&tk, p.kv.k, 3, dims, str, box);
+  if (rc == PACE_OK) rc = tensor_map_bf16(&tpage, p.kv.k, 3, dims, str, whole);
   if (rc != PACE_OK) return rc;
   const int E = a.entry_end - a.entry_begin;
-  return a.max_tokens * p.Gq <= 16 ? launch_keys<16>(p, tk, a.max_tokens, a.max_keys, E, s)
-                                   : launch_keys<32>(p, tk, a.max_tokens, a.max_keys, E, s);
+  return a.max_tokens * p.Gq <= 16 ? launch_keys<16>(p, tk, tpage, a.max_tokens, a.max_keys, E, s)
+                                   : launch_keys<32>(p, tk, tpage, a.max_tokens, a.max_keys, E, s);
 }
 
 }  // namespace pace

@@ -23,10 +23,10 @@ int attn_general_span(const pace_kv_pool_t* p, int layer, const pace_step_t& st,
 // The blocks of a cluster have (maximum, sum) ml[row] (log2 units) and weighted values O[row][stride] of their shares of the
 // keys in shared memory, at the same places; every block merges and stores its part of the outputs.  ns (at most 8): blocks
 // of the cluster, `share` this one's number; `threads` threads of the block take part, fac: 8 floats of shared memory per
-// row.  The caller has synchronised the cluster and does so again before anyone leaves.
-__device__ __forceinline__ void span_merge(const float* O, int stride, const float2* ml, float* fac, int ns, int share, int tid,
+// row, sink: the rows' sinks in log2 units (-infinity: none) in shared memory.  The caller has synchronised the cluster and does so again before anyone leaves.
+__device__ __forceinline__ void span_merge(const float* O, int stride, const float2* ml, const float* sink, float* fac, int ns, int share, int tid,
                                            int threads, int live, int r0, int t0, int g, int Gq, int H, int dv, int dv16,
-                                           const float* sinks, __nv_bfloat16* out, int out_elems) {
+                                           __nv_bfloat16* out, int out_elems) {
   cooperative_groups::cluster_group cl = cooperative_groups::this_cluster();
   // what each share's values are multiplied by, per row
   for (int r = tid; r < live; r += threads) {
@@ -34,12 +34,10 @@ __device__ __forceinline__ void span_merge(const float* O, int stride, const flo
 #pragma unroll
     for (int k = 0; k < 8; ++k)
       st[k] = k < ns ? (ns > 1 ? *cl.map_shared_rank(ml + r, k) : ml[r]) : make_float2(-INFINITY, 0.f);
-    const int rr = r0 + r, hh = g * Gq + rr % Gq;
-    const float sink = sinks ? sinks[hh] * kLog2e : -INFINITY;
-    float top = sink;
+    float top = sink[r];
 #pragma unroll
     for (int k = 0; k < 8; ++k) top = fmaxf(top, st[k].x);
-    float den = sinks ? fast_exp2(sink - top) : 0.f;
+    float den = sink[r] == -INFINITY ? 0.f : fast_exp2(sink[r] - top);
 #pragma unroll
     for (int k = 0; k < 8; ++k) {
       st[k].x = st[k].x == -INFINITY ? 0.f : fast_exp2(st[k].x - top);
@@ -51,6 +49,7 @@ __device__ __forceinline__ void span_merge(const float* O, int stride, const flo
   }
   asm volatile("bar.sync 1, %0;" ::"r"(threads) : "memory");
   const int v4 = dv16 / 4;
+#pragma unroll 2
   for (int i = share * threads + tid; i < live * v4; i += ns * threads) {
     const int r = i / v4, c = (i - r * v4) * 4;
     const int rr = r0 + r, tok = rr / Gq, hh = g * Gq + rr - tok * Gq;

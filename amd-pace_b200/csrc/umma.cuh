@@ -274,6 +274,10 @@ __device__ __forceinline__ void tma_load_3d(void* dst, const CUtensorMap* tm, in
       "l"(tm), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "r"(c2)
       : "memory");
 }
+// the same box on its way into L2 only
+__device__ __forceinline__ void tma_prefetch_3d(const CUtensorMap* tm, int c0, int c1, int c2) {
+  asm volatile("cp.async.bulk.prefetch.tensor.3d.L2.global.tile [%0, {%1, %2, %3}];" ::"l"(tm), "r"(c0), "r"(c1), "r"(c2) : "memory");
+}
 // four rows of a two-dimensional tensor, given by their numbers (the map's box is one row high)
 __device__ __forceinline__ void tma_gather4(void* dst, const CUtensorMap* tm, int c0, int r0, int r1, int r2, int r3,
                                             uint64_t* bar) {
