@@ -19,7 +19,8 @@ struct GeneralArgs {
   const float* sinks;
   int H, d, vd, q_row, o_row, row;   // elements of a row of q, out and the pool
   int entry0, span, span_size;
-  float scale;
+  float scale, softcap;
+  int64_t o_tok;         // elements between the rows of out
 };
 
 constexpr int kRows = 32, kKeys = 32, kRowsPerWarp = 4, kThreads = 256;
@@ -105,7 +106,11 @@ __global__ void __launch_bounds__(kThreads)
       if (last[r] < k0 || first[r] >= k0 + kKeys) continue;  // (the warp's rows agree: lanes differ in the key only)
       const int pos = k0 + lane;
       float x = -INFINITY;
-      if (pos <= last[r] && pos >= first[r]) x = s[r] * a.scale + slope[r] * (float)(pos - last[r]);
+      if (pos <= last[r] && pos >= first[r]) {
+        x = s[r] * a.scale;
+        if (a.softcap > 0.f) x = a.softcap * tanhf(x / a.softcap);
+        x += slope[r] * (float)(pos - last[r]);
+      }
       float mx = x;
 #pragma unroll
       for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -140,7 +145,7 @@ __global__ void __launch_bounds__(kThreads)
 #pragma unroll
       for (int i = 0; i < VI; ++i) acc[r][i] *= f;
     }
-    T* o = out + ((size_t)(a.rows ? a.rows[t0 + tok] : t0 + tok) * H + hh) * a.o_row;
+    T* o = out + (a.rows ? a.rows[t0 + tok] : t0 + tok) * a.o_tok + (int64_t)hh * a.o_row;
 #pragma unroll
     for (int i = 0; i < VI; ++i) {
       const int c = lane + 32 * i;
@@ -196,6 +201,8 @@ int attn_general_span(const pace_kv_pool_t* p, int layer, const pace_step_t& st,
   ga.span = a.span;
   ga.span_size = a.span_size;
   ga.scale = a.scale;
+  ga.softcap = a.softcap;
+  ga.o_tok = span_out_row(a);
   return general(make_view(p, layer, nullptr), st, ga, a.entry_end - a.entry_begin, a.max_tokens, a.dtype, s);
 }
 
@@ -225,5 +232,7 @@ extern "C" int pace_attn_general(const pace_kv_pool_t* p, int32_t layer, const p
   ga.span = PACE_SPAN_ALL;
   ga.span_size = 0;
   ga.scale = scale;
+  ga.softcap = 0.f;
+  ga.o_tok = (int64_t)H * ga.o_row;
   return general(make_view(p, layer, nullptr), *st, ga, st->n_entries, st->max_count, dtype, (cudaStream_t)stream);
 }

@@ -31,6 +31,8 @@ struct SpanParams {
   int dk16, dv16, k_blocks, v_blocks;   // sizes rounded up to 16; 64-column blocks of a stage (v_blocks 0: one plane)
   int entry0, span, span_size, n_stages;
   float scale_log2;
+  ScoreCap cap;
+  int64_t out_row;
 };
 
 struct SpanSmem {
@@ -287,7 +289,8 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1)
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const bool seen = pos + j <= spos && pos + j >= sfirst;
-          x[4 * i + j] = seen ? fmaf(sv[j], p.scale_log2, slope * (float)(pos + j - spos)) : -INFINITY;
+          const float sc = p.cap.out != 0.f ? capped(p.cap, sv[j]) : sv[j] * p.scale_log2;
+          x[4 * i + j] = seen ? fmaf(slope, (float)(pos + j - spos), sc) : -INFINITY;
           mx = fmaxf(mx, x[4 * i + j]);
         }
       }
@@ -395,8 +398,8 @@ __global__ void __launch_bounds__(kThreads, MT * NG <= 4 ? 2 : 1)
   cooperative_groups::cluster_group cl = cooperative_groups::this_cluster();
   if (ns > 1) cl.sync();
   else consumer_sync();
-  span_merge(O, OS, ml, reinterpret_cast<float*>(smem + sm.sink), S, ns, share, tid, kConsumers, live, r0, t0, g, p.Gq, p.H, p.dv,
-             p.dv16, p.out, p.out_elems);
+  span_merge(O, OS, ml, reinterpret_cast<float*>(smem + sm.sink), S, ns, share, tid, kConsumers, live, r0, t0, g, p.Gq, p.dv,
+             p.dv16, p.out, p.out_row, p.out_elems);
   if (ns > 1) cl.sync();  // nobody leaves while its shared memory is read
 }
 
@@ -452,6 +455,8 @@ int span_mma(const pace_kv_pool_t* pl, int layer, const pace_step_t& st, const p
   p.span = a.span;
   p.span_size = a.span_size;
   p.scale_log2 = a.scale * kLog2e;
+  p.cap = score_cap(a.scale, a.softcap);
+  p.out_row = span_out_row(a);
   // (q rows are read in pieces of eight: the caller keeps what lies between dim and the next multiple of 8 zero)
   if (pl->page_tokens != kKeys || a.q_elems % 8 || pl->head_dim % 8 || !aligned16(a.q) || !aligned16(pl->pages) ||
       ((uintptr_t)a.out & 7) || p.dv16 > 512 || (shared && p.dv16 > p.k_blocks * 64))

@@ -30,6 +30,7 @@ struct KeysParams {
   int k_blocks, v_tiles, v_used;   // 64-column blocks of a key, 128-element tiles of a value, blocks that values read
   int entry0, span, span_size, tmem_cols;
   float scale_log2;
+  int64_t out_row;
 };
 
 struct KeysSmem {
@@ -351,7 +352,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   cooperative_groups::cluster_group cl = cooperative_groups::this_cluster();
   if (ns > 1) cl.sync();
   span_merge(reinterpret_cast<float*>(smem + sm.k), p.dv16 + 4, reinterpret_cast<float2*>(smem + sm.ml),
-             reinterpret_cast<float*>(smem + sm.sink), reinterpret_cast<float*>(smem + sm.s), ns, share, tid, kThreads, live, r0, t0, 0, p.Gq, p.H, p.dv, p.dv16, p.out, p.out_elems);
+             reinterpret_cast<float*>(smem + sm.sink), reinterpret_cast<float*>(smem + sm.s), ns, share, tid, kThreads, live, r0, t0, 0, p.Gq, p.dv, p.dv16, p.out, p.out_row, p.out_elems);
   if (ns > 1) cl.sync();  // nobody leaves while its shared memory is read
 }
 
@@ -405,7 +406,7 @@ int launch_keys(KeysParams& p, const CUtensorMap& tk, const CUtensorMap& tpage, 
 // PACE_ERR_UNSUPPORTED: shapes beyond this kernel (nothing launched)
 int attn_span_keys(const pace_kv_pool_t* pl, int layer, const pace_step_t& st, const pace_attn_span_args_t& a, cudaStream_t s) {
   if (pl->row_format != PACE_ROWS_SHARED || pl->n_kv_heads != 1 || pl->page_tokens != kPage || pl->head_dim % 8 || a.q_elems % 8 ||
-      a.vdim > 512 || a.vdim > a.dim || !aligned16(a.q) || !aligned16(pl->pages) || ((uintptr_t)a.out & 7))
+      a.vdim > 512 || a.vdim > a.dim || a.softcap > 0.f || !aligned16(a.q) || !aligned16(pl->pages) || ((uintptr_t)a.out & 7))
     return PACE_ERR_UNSUPPORTED;
   KeysParams p;
   p.kv = make_view(pl, layer, nullptr);
@@ -427,6 +428,7 @@ int attn_span_keys(const pace_kv_pool_t* pl, int layer, const pace_step_t& st, c
   p.span = a.span;
   p.span_size = a.span_size;
   p.scale_log2 = a.scale * kLog2e;
+  p.out_row = span_out_row(a);
   if (p.k_blocks > kMaxBlocks) return PACE_ERR_UNSUPPORTED;
   CUtensorMap tk, tpage;
   const uint64_t row = (uint64_t)pl->head_dim;

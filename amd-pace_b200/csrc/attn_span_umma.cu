@@ -34,6 +34,8 @@ struct PromptParams {
   int q_elems, out_elems, H, Hkv, G, k_dim, k2_dim, vdim, nb1;
   int entry0, n_entries, n_qt, span, span_size, n_stages;
   float scale_log2;
+  ScoreCap cap;
+  int64_t out_row;
 };
 
 struct Unit {
@@ -76,14 +78,18 @@ struct Bars {
   uint64_t full[kMaxStages], empty[kMaxStages], s_full[2], s_free[2], p_full[2], o_full[2], q_ready[2], drain[3];
 };
 
-// KB, VB: 64-column blocks of a key and of a value; BIAS: distance bias
-template <int KB, int VB, bool BIAS>
+// What happens to a score in front of the softmax: nothing, a distance bias, a cap.
+enum { kPlain = 0, kBias = 1, kCap = 2 };
+
+// KB, VB: 64-column blocks of a key and of a value
+template <int KB, int VB, int MODE>
 __device__ __forceinline__ void prompt_softmax(const PromptParams& p, Bars& b, uint32_t tmem, unsigned char* qs, int n_units,
                                                volatile int* abort) {
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 7, row = tid & 127;
   const uint32_t t_lane = tmem + ((uint32_t)(row & ~31) << 16);
   const uint32_t tS = t_lane + w * kChunk, tP = t_lane + kColP + w * 32, tPl = t_lane + kColPLow + w * 32,
                  tO = t_lane + kColO + w * 128;
+  constexpr bool BIAS = MODE == kBias, LOG2 = MODE != kPlain;   // LOG2: the scores are made log2 units first
   unsigned char* qrow = qs + w * KB * (kUmmaRows * 128) + row * 128;
   const float scale = p.scale_log2;
   const uint64_t scale2 = pack64(__float_as_uint(scale), __float_as_uint(scale));
@@ -135,6 +141,33 @@ __device__ __forceinline__ void prompt_softmax(const PromptParams& p, Bars& b, u
           unpack64(fma2(pack64(a0, a1), scale2, fma2(kk, sl2, off2)), a0, a1);
         }
       }
+      if constexpr (MODE == kCap) {
+        // two capped scores share a reciprocal: 1 / a = b / (a b); the exponent's bound keeps the product finite
+        const float cin = p.cap.in, cout = p.cap.out;
+        const uint64_t cin2 = pack64(__float_as_uint(cin), __float_as_uint(cin)),
+                       one2 = pack64(0x3f800000u, 0x3f800000u), c2 = pack64(__float_as_uint(cout), __float_as_uint(cout)),
+                       zero2 = 0ull;
+#pragma unroll
+        for (int k = 0; k < 32; ++k) {
+          uint32_t& a0 = sr[k >> 4][(2 * k) & 31];
+          uint32_t& a1 = sr[k >> 4][(2 * k + 1) & 31];
+          uint32_t x0, x1;
+          unpack64(fma2(pack64(a0, a1), cin2, zero2), x0, x1);
+          const float y0 = fminf(__uint_as_float(x0), 60.f), y1 = fminf(__uint_as_float(x1), 60.f);
+          float e0, e1;
+          if (k & 1) {
+            exp2_poly2_fine(y0, y1, e0, e1);
+          } else {
+            e0 = fast_exp2(y0);
+            e1 = fast_exp2(y1);
+          }
+          uint32_t d0, d1;
+          unpack64(add2(pack64(__float_as_uint(e0), __float_as_uint(e1)), one2), d0, d1);
+          const float r = -2.0f * cout * rcp_t<__nv_bfloat16>(__uint_as_float(d0) * __uint_as_float(d1));
+          const uint64_t rr = pack64(__float_as_uint(r), __float_as_uint(r));
+          unpack64(fma2(rr, pack64(d1, d0), c2), a0, a1);
+        }
+      }
       const int lo = max(0, first - p0), hi = min(kChunk, pos + 1 - p0);  // visible keys of the chunk: [lo, hi)
       if (!__all_sync(0xffffffffu, !live || (lo <= 0 && hi >= kChunk))) {
         const unsigned seen = hi > lo ? (unsigned)(hi - lo) : 0u;
@@ -147,7 +180,7 @@ __device__ __forceinline__ void prompt_softmax(const PromptParams& p, Bars& b, u
       for (int k = 0; k < 32; ++k)
         mx4[k & 3] = max3(mx4[k & 3], __uint_as_float(sr[k >> 4][(2 * k) & 31]), __uint_as_float(sr[k >> 4][(2 * k + 1) & 31]));
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-      if (!BIAS) mx *= scale;  // scale > 0
+      if (!LOG2) mx *= scale;  // scale > 0
       const bool grow = mx > m + kLazy;
       if (__any_sync(0xffffffffu, grow)) {
         const float m_new = grow ? mx : m;
@@ -179,7 +212,7 @@ __device__ __forceinline__ void prompt_softmax(const PromptParams& p, Bars& b, u
         for (int k = 0; k < 16; ++k) {
           const uint64_t s2 = pack64(sr[hf][2 * k], sr[hf][2 * k + 1]);
           uint32_t x0, x1;
-          unpack64(BIAS ? add2(s2, ne2) : fma2(s2, scale2, ne2), x0, x1);
+          unpack64(LOG2 ? add2(s2, ne2) : fma2(s2, scale2, ne2), x0, x1);
           float p0f, p1f;
           if (k & 1) {
             exp2_poly2_fine(__uint_as_float(x0), __uint_as_float(x1), p0f, p1f);   // half of them on the FMA pipe
@@ -218,7 +251,7 @@ __device__ __forceinline__ void prompt_softmax(const PromptParams& p, Bars& b, u
       den = l * f + fast_exp2(sk - top);
     }
     const float inv = den > 0.f ? f / den : 0.f;
-    __nv_bfloat16* dst = p.out + ((size_t)(un.t0 + tok) * p.H + head) * p.out_elems;
+    __nv_bfloat16* dst = p.out + (un.t0 + tok) * p.out_row + (int64_t)head * p.out_elems;
 #pragma unroll
     for (int d0 = 0; d0 < VB * 64; d0 += 32) {
       uint32_t om[32];
@@ -328,7 +361,7 @@ __device__ __forceinline__ void prompt_issue_pv(const PromptParams& p, Bars& b, 
   }
 }
 
-template <int KB, int VB, bool BIAS>
+template <int KB, int VB, int MODE>
 __global__ void __launch_bounds__(kThreads, 1)
     attn_span_prompt_kernel(const PromptParams p, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmK2,
                             const __grid_constant__ CUtensorMap tmV) {
@@ -368,7 +401,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(&tmem_slot);
 
   if (warp < 8) {
-    prompt_softmax<KB, VB, BIAS>(p, b, tmem, qs, n_units, abort);
+    prompt_softmax<KB, VB, MODE>(p, b, tmem, qs, n_units, abort);
   } else if (warp == 8) {
     int s = 0, ph = 0, issued = 0;
     bool ok = true;
@@ -441,13 +474,15 @@ int launch_prompt(PromptParams& p, const CUtensorMap& tk, const CUtensorMap& tk2
   static_assert((226 * 1024 - 1024 - 512 - QBYTES) / STAGE >= 2, "two stages fit");
   const int smem = QBYTES + p.n_stages * STAGE + 1024;
   const int units = p.n_entries * p.Hkv * p.n_qt, blocks = std::min(units, sm_count());
-  if (p.slopes) {
-    PACE_CUDA_TRY(cudaFuncSetAttribute(attn_span_prompt_kernel<KB, VB, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    attn_span_prompt_kernel<KB, VB, true><<<blocks, kThreads, smem, s>>>(p, tk, tk2, tv);
-  } else {
-    PACE_CUDA_TRY(cudaFuncSetAttribute(attn_span_prompt_kernel<KB, VB, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    attn_span_prompt_kernel<KB, VB, false><<<blocks, kThreads, smem, s>>>(p, tk, tk2, tv);
-  }
+  auto launch = [&](auto* fn) {
+    PACE_CUDA_TRY(cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    fn<<<blocks, kThreads, smem, s>>>(p, tk, tk2, tv);
+    return PACE_OK;
+  };
+  const int rc = p.cap.out != 0.f ? launch(attn_span_prompt_kernel<KB, VB, kCap>)
+                 : p.slopes       ? launch(attn_span_prompt_kernel<KB, VB, kBias>)
+                                  : launch(attn_span_prompt_kernel<KB, VB, kPlain>);
+  if (rc != PACE_OK) return rc;
   PACE_LAUNCH_CHECK("attn_span_prompt_kernel");
   return PACE_OK;
 }
@@ -468,7 +503,7 @@ extern "C" int pace_attn_span_prefill(const pace_kv_pool_t* pl, int32_t layer, c
                  x->k_dim + x->k2_dim != a->dim || a->q_elems < a->dim))
     return PACE_ERR_INVALID;
   if (st->n_tokens == 0 || a->entry_begin == a->entry_end || a->max_tokens == 0) return PACE_OK;
-  if (a->dtype != PACE_DTYPE_BF16 || !(a->scale > 0.f) || a->vdim > 128 || a->vdim % 8 || a->out_elems % 8 || a->q_elems % 8 ||
+  if (a->dtype != PACE_DTYPE_BF16 || !(a->scale > 0.f) || a->vdim > 128 || a->vdim % 8 || a->out_elems % 8 || a->out_row % 8 || (a->slopes && a->softcap > 0.f) || a->q_elems % 8 ||
       !aligned16(a->q) || !aligned16(a->out))
     return PACE_ERR_UNSUPPORTED;
   PromptParams p;
@@ -525,6 +560,8 @@ extern "C" int pace_attn_span_prefill(const pace_kv_pool_t* pl, int32_t layer, c
   p.span = a->span;
   p.span_size = a->span_size;
   p.scale_log2 = a->scale * kLog2e;
+  p.cap = score_cap(a->scale, a->softcap);
+  p.out_row = span_out_row(*a);
   PACE_PROFILE("attn_span_prefill", stream, "layer=%d entries=%d tokens<=%d heads=%d dims=%d/%d", layer, p.n_entries, a->max_tokens,
                p.H, a->dim, a->vdim);
   const cudaStream_t s = (cudaStream_t)stream;

@@ -92,6 +92,12 @@ template <typename T> __device__ __forceinline__ float silu_t(float x) { return 
 template <typename T> __device__ __forceinline__ float gelu_tanh_t(float z) {
   return z * sigmoid_t<T>(1.5957691216057308f * (z + 0.044715f * z * z * z));
 }
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
+// ln(1 + e^x), with a relative error of a few ulp at both ends
+__device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+template <typename T> __device__ __forceinline__ float act_t(int act, float z) {
+  return act == PACE_ACT_SILU ? silu_t<T>(z) : act == PACE_ACT_GELU_TANH ? gelu_tanh_t<T>(z) : act == PACE_ACT_GELU_ERF ? gelu_erf(z) : z;
+}
 // sqrt(1 - e^x) for x <= 0 (exp_x = e^x) without cancellation: near zero 1 - e^x is the Taylor series
 // -x (1 + x/2 (1 + x/3 (1 + ...))), further out the plain difference
 template <typename T> __device__ __forceinline__ float sqrt_one_minus_exp(float x, float exp_x) {

@@ -22,11 +22,11 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(pace_step_t st, pace
     for (int k = threadIdx.x >> 5; k < a.top; k += blockDim.x >> 5) {
       const int e = a.slot_expert[(size_t)t * a.top + k];
       int n = 0;
-      for (int i = threadIdx.x & 31; i < e; i += 32) n += a.expert_count[i];
+      for (int i = threadIdx.x & 31; i < e && e < a.n_experts; i += 32) n += a.expert_count[i];
 #pragma unroll
       for (int o = 16; o; o >>= 1) n += __shfl_xor_sync(0xffffffffu, n, o);
       if ((threadIdx.x & 31) == 0) {
-        e_row[k] = n + a.slot_rank[(size_t)t * a.top + k];
+        e_row[k] = e < a.n_experts ? n + a.slot_rank[(size_t)t * a.top + k] : -1;   // -1: an identity expert
         e_w[k] = a.slot_weight[(size_t)t * a.top + k];
       }
     }
@@ -54,12 +54,25 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(pace_step_t st, pace
         for (int j = 0; j < V; ++j) yv[i][j] = 0.f;
         for (int k = 0; k < a.top; ++k) {
           float r[V];
-          Vec<T, V>::load(static_cast<const T*>(a.y) + (size_t)e_row[k] * a.y_stride + c, r);
+          Vec<T, V>::load(e_row[k] >= 0 ? static_cast<const T*>(a.y) + (size_t)e_row[k] * a.y_stride + c
+                                        : static_cast<const T*>(a.identity) + (size_t)t * W + c, r);
 #pragma unroll
           for (int j = 0; j < V; ++j) yv[i][j] = fmaf(e_w[k], r[j], yv[i][j]);
         }
       } else if (y) {
         Vec<T, V>::load(y + c, yv[i]);
+      }
+      if (a.add) {
+        float r[V];
+        Vec<T, V>::load(static_cast<const T*>(a.add) + (size_t)t * a.add_stride + c, r);
+#pragma unroll
+        for (int j = 0; j < V; ++j) yv[i][j] += r[j];
+      }
+      if (a.y_bias) {
+        float r[V];
+        Vec<float, V>::load(a.y_bias + c, r);
+#pragma unroll
+        for (int j = 0; j < V; ++j) yv[i][j] += r[j];
       }
       if (y) {
 #pragma unroll
@@ -77,9 +90,24 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(pace_step_t st, pace
         float w[V];
         if (a.w_post) Vec<float, V>::load(a.w_post + c, w);
 #pragma unroll
-        for (int j = 0; j < V; ++j) xv[i][j] += a.w_post ? yv[i][j] * r * (a.weight_offset + w[j]) : yv[i][j];
+        for (int j = 0; j < V; ++j) xv[i][j] += a.w_post ? yv[i][j] * r * (a.weight_offset + w[j]) : yv[i][j] * a.y_mul;
       }
     }
+  }
+  float em_r = 1.f;
+  if (a.embed_norm) {
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * V;
+      if (c < W && em) {
+        float e[V];
+        Vec<T, V>::load(em + c, e);
+#pragma unroll
+        for (int j = 0; j < V; ++j) ss += e[j] * e[j];
+      }
+    }
+    em_r = 1.0f / sqrtf(block_sum(ss, red) / (float)W + a.eps);
   }
   ss = 0.f;
 #pragma unroll
@@ -87,10 +115,12 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(pace_step_t st, pace
     const int c = (i * blockDim.x + threadIdx.x) * V;
     if (c < W) {
       if (em) {
-        float e[V];
+        float e[V], w[V];
         Vec<T, V>::load(em + c, e);
+        if (a.embed_norm) Vec<float, V>::load(a.embed_norm + c, w);
 #pragma unroll
-        for (int j = 0; j < V; ++j) xv[i][j] = fmaf(e[j], a.embed_scale, xv[i][j]);
+        for (int j = 0; j < V; ++j)
+          xv[i][j] = fmaf(e[j], a.embed_norm ? em_r * (a.weight_offset + w[j]) : a.embed_scale, xv[i][j]);
       }
       Vec<float, V>::store(x + c, xv[i]);
 #pragma unroll
@@ -117,6 +147,12 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(pace_step_t st, pace
 #pragma unroll
       for (int j = 0; j < V; ++j) w[j] = xv[i][j] * r * (a.weight_offset + w[j]);
       Vec<T, V>::store(h + c, w);
+      if (a.h2) {
+        Vec<float, V>::load(a.w_next2 + c, w);
+#pragma unroll
+        for (int j = 0; j < V; ++j) w[j] = xv[i][j] * r * (a.weight_offset + w[j]);
+        Vec<T, V>::store(static_cast<T*>(a.h2) + (size_t)t * W + c, w);
+      }
     }
   }
 }
@@ -511,19 +547,113 @@ __global__ void relu_squared_kernel(T* __restrict__ x, int64_t n) {
   }
 }
 
-template <typename T, int V, int ACT>
-__global__ void glu_kernel(const T* __restrict__ x, int64_t xs, T* __restrict__ out, int n_tokens, int n) {
+template <typename T, int V, int ACT, bool GATED>
+__global__ void glu_kernel(const T* __restrict__ x, int64_t xs, T* __restrict__ out, int64_t os, int n_tokens, int n) {
   const int per = n / V;
   const size_t total = (size_t)n_tokens * per;
   for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const int t = (int)(i / per), c = (int)(i % per) * V;
     float g[V], u[V];
     Vec<T, V>::load(x + (size_t)t * xs + c, g);
-    Vec<T, V>::load(x + (size_t)t * xs + n + c, u);
+    if constexpr (GATED) Vec<T, V>::load(x + (size_t)t * xs + n + c, u);
 #pragma unroll
-    for (int j = 0; j < V; ++j) u[j] *= ACT == PACE_ACT_SILU ? silu_t<T>(g[j]) : gelu_tanh_t<T>(g[j]);
-    Vec<T, V>::store(out + (size_t)t * n + c, u);
+    for (int j = 0; j < V; ++j) {
+      const float f = act_t<T>(ACT, g[j]);
+      u[j] = GATED ? u[j] * f : f;
+    }
+    Vec<T, V>::store(out + (size_t)t * os + c, u);
   }
+}
+
+__global__ void soft_cap_kernel(float* x, int64_t n, float cap) {
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x)
+    x[i] = cap * tanhf(x[i] / cap);
+}
+
+// Norms over parts of a row: LP lanes (a divisor of 32) per part, or (LP = 0) a block per part.
+template <typename T, int V, int LP>
+__global__ void part_norm_gate_kernel(pace_part_norm_gate_args_t a) {
+  __shared__ float red[32];
+  const int parts = a.n / a.part, per_block = LP ? blockDim.x / LP : 1;
+  const int64_t total = (int64_t)a.n_tokens * parts;
+  const int lane = LP ? threadIdx.x % LP : threadIdx.x, step = (LP ? LP : blockDim.x) * V;
+  int64_t i = (int64_t)blockIdx.x * per_block + (LP ? threadIdx.x / LP : 0);
+  const bool live = i < total;                 // (shuffles need whole warps)
+  if (!live) i = total - 1;
+  const int t = (int)(i / parts), c0 = (int)(i % parts) * a.part;
+  const T* o = static_cast<const T*>(a.o) + (size_t)t * a.o_stride + c0;
+  const T* gate = static_cast<const T*>(a.gate) + (size_t)t * a.gate_stride + c0;
+  T* out = static_cast<T*>(a.out) + (size_t)t * a.out_stride + c0;
+  auto value = [&](int c, float* x) {
+    Vec<T, V>::load(o + c, x);
+    if (a.gate_first) {
+      float g[V];
+      Vec<T, V>::load(gate + c, g);
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] *= silu_t<T>(g[j]);
+    }
+  };
+  float ss = 0.f, first[V];
+#pragma unroll
+  for (int j = 0; j < V; ++j) first[j] = 0.f;
+  for (int c = lane * V; c < a.part; c += step) {
+    float x[V];
+    value(c, x);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      ss = fmaf(x[j], x[j], ss);
+      if (c == lane * V) first[j] = x[j];
+    }
+  }
+  if constexpr (LP > 0) {
+#pragma unroll
+    for (int w = LP / 2; w; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
+  } else {
+    ss = block_sum(ss, red);
+  }
+  if (!live) return;
+  const float r = 1.0f / sqrtf(ss / (float)a.part + a.eps);
+  for (int c = lane * V; c < a.part; c += step) {
+    float x[V], w[V];
+    if (c == lane * V) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] = first[j];
+    } else {
+      value(c, x);
+    }
+    Vec<float, V>::load(a.w + (c0 + c) % a.w_period, w);
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[j] *= r * w[j];
+    if (!a.gate_first) {
+      float g[V];
+      Vec<T, V>::load(gate + c, g);
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] *= sigmoid_t<T>(g[j]);
+    }
+    Vec<T, V>::store(out + c, x);
+  }
+}
+
+template <typename T, int V>
+void launch_part_norm_gate(const pace_part_norm_gate_args_t& a, cudaStream_t s) {
+  const int vecs = (a.part + V - 1) / V;
+  const int64_t total = (int64_t)a.n_tokens * (a.n / a.part);
+  auto blocks = [&](int lp) { return (unsigned)((total * lp + 127) / 128); };
+  if (vecs <= 8) part_norm_gate_kernel<T, V, 8><<<blocks(8), 128, 0, s>>>(a);
+  else if (vecs <= 16) part_norm_gate_kernel<T, V, 16><<<blocks(16), 128, 0, s>>>(a);
+  else if (vecs <= 64) part_norm_gate_kernel<T, V, 32><<<blocks(32), 128, 0, s>>>(a);
+  else part_norm_gate_kernel<T, V, 0><<<(unsigned)total, vecs < 512 ? (vecs + 31) / 32 * 32 : 512, 0, s>>>(a);
+}
+
+template <typename T>
+int part_norm_gate_t(const pace_part_norm_gate_args_t& a, cudaStream_t s) {
+  constexpr int V = 16 / sizeof(T);
+  const bool vec = a.part % V == 0 && a.w_period % V == 0 && (a.o_stride | a.gate_stride | a.out_stride) % V == 0 && aligned16(a.o) &&
+                   aligned16(a.gate) && aligned16(a.out) && aligned16(a.w);
+  if (vec) launch_part_norm_gate<T, V>(a, s);
+  else launch_part_norm_gate<T, 1>(a, s);
+  PACE_LAUNCH_CHECK("part_norm_gate_kernel");
+  return PACE_OK;
 }
 
 unsigned elementwise_blocks(size_t threads_wanted) {
@@ -579,16 +709,23 @@ int relu_squared_t(void* x, int64_t n, cudaStream_t s) {
   return PACE_OK;
 }
 
-template <typename T, int ACT>
-int glu_t(const void* x, int64_t xs, void* out, int n_tokens, int n, cudaStream_t s) {
+template <typename T, int ACT, bool GATED>
+int glu_t(const void* x, int64_t xs, void* out, int64_t os, int n_tokens, int n, cudaStream_t s) {
   constexpr int V = 16 / sizeof(T);
   const size_t total = (size_t)n_tokens * n;
-  if (n % V == 0 && xs % V == 0 && aligned16(x) && aligned16(out))
-    glu_kernel<T, V, ACT><<<elementwise_blocks(total / V), 256, 0, s>>>((const T*)x, xs, (T*)out, n_tokens, n);
+  if (n % V == 0 && xs % V == 0 && os % V == 0 && aligned16(x) && aligned16(out))
+    glu_kernel<T, V, ACT, GATED><<<elementwise_blocks(total / V), 256, 0, s>>>((const T*)x, xs, (T*)out, os, n_tokens, n);
   else
-    glu_kernel<T, 1, ACT><<<elementwise_blocks(total), 256, 0, s>>>((const T*)x, xs, (T*)out, n_tokens, n);
+    glu_kernel<T, 1, ACT, GATED><<<elementwise_blocks(total), 256, 0, s>>>((const T*)x, xs, (T*)out, os, n_tokens, n);
   PACE_LAUNCH_CHECK("glu_kernel");
   return PACE_OK;
+}
+
+template <typename T, bool GATED>
+int glu_act(const void* x, int64_t xs, void* out, int64_t os, int n_tokens, int n, int act, cudaStream_t s) {
+  if (act == PACE_ACT_SILU) return glu_t<T, PACE_ACT_SILU, GATED>(x, xs, out, os, n_tokens, n, s);
+  if (act == PACE_ACT_GELU_TANH) return glu_t<T, PACE_ACT_GELU_TANH, GATED>(x, xs, out, os, n_tokens, n, s);
+  return glu_t<T, PACE_ACT_GELU_ERF, GATED>(x, xs, out, os, n_tokens, n, s);
 }
 
 bool dtype_ok(int dtype) { return dtype == PACE_DTYPE_BF16 || dtype == PACE_DTYPE_FP32; }
@@ -602,8 +739,11 @@ extern "C" {
 
 int pace_residual_norm(const pace_step_t* st, const pace_residual_norm_args_t* a, void* stream) {
   if (!step_ok(st) || !a || !a->x || a->width < 1 || !dtype_ok(a->dtype)) return PACE_ERR_INVALID;
+  if ((a->w_next2 == nullptr) != (a->h2 == nullptr) || (a->h2 && !a->w_next) || ((a->add || a->y_bias) && !a->y) ||
+      (a->add && a->add_stride < a->width) || (a->embed_norm && !a->embed))
+    return PACE_ERR_INVALID;
   if ((a->w_next && !a->h) || (a->embed && a->vocab < 1) || (a->y && a->y_stride < a->width)) return PACE_ERR_INVALID;
-  if (a->top < 0 || (a->top > 0 && (!a->y || a->top > kMaxTop || a->n_experts < a->top || !a->slot_expert || !a->slot_rank ||
+  if (a->top < 0 || (a->top > 0 && (!a->y || a->top > kMaxTop || (a->n_experts < a->top && !a->identity) || !a->slot_expert || !a->slot_rank ||
                                     !a->slot_weight || !a->expert_count)))
     return PACE_ERR_INVALID;
   if (st->n_tokens == 0) return PACE_OK;
@@ -611,7 +751,9 @@ int pace_residual_norm(const pace_step_t* st, const pace_residual_norm_args_t* a
   const cudaStream_t s = (cudaStream_t)stream;
   // four elements per access: 16 bytes of fp32, 8 of bf16
   const bool vec = a->width % 4 == 0 && a->y_stride % 4 == 0 && aligned16(a->x) && aligned16(a->y) && aligned16(a->h) &&
-                   aligned16(a->embed) && aligned16(a->w_post) && aligned16(a->w_next);
+                   aligned16(a->embed) && aligned16(a->w_post) && aligned16(a->w_next) && aligned16(a->w_next2) && aligned16(a->h2) &&
+                   aligned16(a->identity) && aligned16(a->add) && a->add_stride % 4 == 0 && aligned16(a->y_bias) &&
+                   aligned16(a->embed_norm);
   if (a->dtype == PACE_DTYPE_BF16)
     return vec ? launch_residual_norm<__nv_bfloat16, 4>(*st, *a, s) : launch_residual_norm<__nv_bfloat16, 1>(*st, *a, s);
   return vec ? launch_residual_norm<float, 4>(*st, *a, s) : launch_residual_norm<float, 1>(*st, *a, s);
@@ -654,16 +796,36 @@ int pace_relu_squared(void* x, int64_t n, int32_t dtype, void* stream) {
                                   : relu_squared_t<float>(x, n, (cudaStream_t)stream);
 }
 
-int pace_glu(const void* x, int64_t x_stride, void* out, int32_t n_tokens, int32_t n, int32_t act, int32_t dtype, void* stream) {
-  if (!x || !out || n_tokens < 0 || n < 1 || x_stride < 2 * (int64_t)n || !dtype_ok(dtype)) return PACE_ERR_INVALID;
-  if (act != PACE_ACT_SILU && act != PACE_ACT_GELU_TANH) return PACE_ERR_INVALID;
+int pace_glu(const void* x, int64_t x_stride, void* out, int64_t out_stride, int32_t n_tokens, int32_t n, int32_t act, int32_t gated,
+             int32_t dtype, void* stream) {
+  if (!x || !out || n_tokens < 0 || n < 1 || x_stride < (gated ? 2 : 1) * (int64_t)n || out_stride < n || !dtype_ok(dtype))
+    return PACE_ERR_INVALID;
+  if (act != PACE_ACT_SILU && act != PACE_ACT_GELU_TANH && act != PACE_ACT_GELU_ERF) return PACE_ERR_INVALID;
   if (n_tokens == 0) return PACE_OK;
   const cudaStream_t s = (cudaStream_t)stream;
   if (dtype == PACE_DTYPE_BF16)
-    return act == PACE_ACT_SILU ? glu_t<__nv_bfloat16, PACE_ACT_SILU>(x, x_stride, out, n_tokens, n, s)
-                                : glu_t<__nv_bfloat16, PACE_ACT_GELU_TANH>(x, x_stride, out, n_tokens, n, s);
-  return act == PACE_ACT_SILU ? glu_t<float, PACE_ACT_SILU>(x, x_stride, out, n_tokens, n, s)
-                              : glu_t<float, PACE_ACT_GELU_TANH>(x, x_stride, out, n_tokens, n, s);
+    return gated ? glu_act<__nv_bfloat16, true>(x, x_stride, out, out_stride, n_tokens, n, act, s)
+                 : glu_act<__nv_bfloat16, false>(x, x_stride, out, out_stride, n_tokens, n, act, s);
+  return gated ? glu_act<float, true>(x, x_stride, out, out_stride, n_tokens, n, act, s)
+               : glu_act<float, false>(x, x_stride, out, out_stride, n_tokens, n, act, s);
+}
+
+int pace_soft_cap(float* x, int64_t n, float cap, void* stream) {
+  if (!x || n < 0 || !(cap > 0.f)) return PACE_ERR_INVALID;
+  if (n == 0) return PACE_OK;
+  soft_cap_kernel<<<elementwise_blocks((size_t)n), 256, 0, (cudaStream_t)stream>>>(x, n, cap);
+  PACE_LAUNCH_CHECK("soft_cap_kernel");
+  return PACE_OK;
+}
+
+int pace_part_norm_gate(const pace_part_norm_gate_args_t* a, void* stream) {
+  if (!a || !a->o || !a->gate || !a->w || !a->out || a->n_tokens < 0 || a->part < 1 || a->n < a->part || a->n % a->part ||
+      a->w_period < 1 || a->o_stride < a->n || a->gate_stride < a->n || a->out_stride < a->n || !dtype_ok(a->dtype))
+    return PACE_ERR_INVALID;
+  if (a->n_tokens == 0) return PACE_OK;
+  if ((int64_t)a->n_tokens * (a->n / a->part) > 0x3fffffff) return PACE_ERR_UNSUPPORTED;
+  return a->dtype == PACE_DTYPE_BF16 ? part_norm_gate_t<__nv_bfloat16>(*a, (cudaStream_t)stream)
+                                     : part_norm_gate_t<float>(*a, (cudaStream_t)stream);
 }
 
 int pace_step_decode(int32_t* token, int32_t* tok_pos, int32_t* start, const int64_t* next, const int64_t* pos, int32_t n,

@@ -1,10 +1,10 @@
-// Mixtures of experts: routing (sigmoid scores, choice by corrected scores) and the chosen experts' gated feed-forwards
-// as grouped products.
+// Mixtures of experts: routing (sigmoid or softmax scores, choice by corrected scores) and the chosen experts'
+// feed-forwards, gated or not, as grouped products.
 //
 // Grouped product on tcgen05 (moe_grouped_kernel): the weights are the 128-row operand, the tokens the columns, so an
 // expert with a handful of tokens costs a narrow tile and not a padded one.  A tile is (expert, 2 x 128 weight rows, NT
-// tokens): two accumulators that share every token tile - gate and up rows of the same features (first product), two
-// neighbouring row tiles (second product).  Persistent blocks of ten warps: TMA producer, MMA issuer, eight epilogue warps;
+// tokens): two accumulators that share every token tile - gate and up rows of the same features (gated first product), two
+// neighbouring row tiles (everything else).  Persistent blocks of ten warps: TMA producer, MMA issuer, eight epilogue warps;
 // two sets of accumulators in tensor memory, so that a tile is stored while the next one is computed.  The first
 // product's token rows come through the router's lists: narrow tiles gather them by TMA (tile::gather4), wide ones read
 // rows that moe_spread_kernel has copied into expert order (32 gathers per 64 columns would pace a wide tile).  Its results
@@ -38,11 +38,21 @@ __global__ void moe_route_kernel(pace_moe_route_args_t a, int rounds) {
     const int local = r * warps + warp, t = t_first + local;
     if (t >= a.n_tokens) break;
     const float* z = a.logits + (size_t)t * E;
-    for (int e = lane; e < E; e += 32) {
-      score[e] = 1.0f / (1.0f + expf(-z[e]));
-      choice[e] = score[e] + (a.correction ? a.correction[e] : 0.f);
+    if (a.softmax) {
+      float top = -INFINITY, sum = 0.f;
+      for (int e = lane; e < E; e += 32) top = fmaxf(top, z[e]);
+#pragma unroll
+      for (int o = 16; o; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+      for (int e = lane; e < E; e += 32) sum += score[e] = expf(z[e] - top);
+#pragma unroll
+      for (int o = 16; o; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      for (int e = lane; e < E; e += 32) score[e] /= sum;
+    } else {
+      for (int e = lane; e < E; e += 32) score[e] = 1.0f / (1.0f + expf(-z[e]));
     }
+    for (int e = lane; e < E; e += 32) choice[e] = score[e] + (a.correction ? a.correction[e] : 0.f);
     __syncwarp();
+    float chosen = 0.f;
     for (int k = 0; k < a.top; ++k) {
       float best = -INFINITY;
       int at = -1;
@@ -55,6 +65,7 @@ __global__ void moe_route_kernel(pace_moe_route_args_t a, int rounds) {
         if (i >= 0 && (at < 0 || v > best || (v == best && i < at))) best = v, at = i;
       }
       if (at < 0) at = k;  // (scores that are not numbers: any expert)
+      chosen += score[at];
       if (lane == (at & 31)) {
         choice[at] = -INFINITY;
         const size_t s = (size_t)t * a.top + k;
@@ -65,6 +76,9 @@ __global__ void moe_route_kernel(pace_moe_route_args_t a, int rounds) {
       }
     }
     __syncwarp();
+    if (a.normalise)
+      for (int k = lane; k < a.top; k += 32)
+        a.slot_weight[(size_t)t * a.top + k] = score[sel[2 * (local * a.top + k)]] / (chosen + 1e-20f) * a.weight_scale;
   }
   __syncthreads();
   for (int e = threadIdx.x; e < E; e += blockDim.x) {
@@ -105,7 +119,7 @@ __device__ __forceinline__ bool find_row(const int32_t* count, int E, int r, int
 }
 
 // a block per row, a warp per output feature at a time
-template <typename T, bool GLU>
+template <typename T, bool FIRST>
 __global__ void __launch_bounds__(256) moe_simple_kernel(pace_moe_experts_args_t a) {
   extern __shared__ float xs[];
   __shared__ int who[2];
@@ -118,21 +132,22 @@ __global__ void __launch_bounds__(256) moe_simple_kernel(pace_moe_experts_args_t
   __syncthreads();
   const int e = who[0];
   if (e < 0) return;
-  const int K = GLU ? a.width : a.ff, N = GLU ? a.ff : a.width;
+  const int K = FIRST ? a.width : a.ff, N = FIRST ? a.ff : a.width;
+  const bool glu = FIRST && a.gated;
   const T* x;
-  if (GLU) x = static_cast<const T*>(a.x) + (size_t)a.expert_list[(size_t)e * a.n_tokens + who[1]] * K;
+  if (FIRST) x = static_cast<const T*>(a.x) + (size_t)a.expert_list[(size_t)e * a.n_tokens + who[1]] * K;
   else x = static_cast<const T*>(a.hidden) + (size_t)r * K;
   for (int c = threadIdx.x; c < K; c += blockDim.x) xs[c] = to_f<T>(x[c]);
   __syncthreads();
   const int lane = threadIdx.x & 31;
   for (int f = threadIdx.x >> 5; f < N; f += blockDim.x >> 5) {
-    const T* w0 = GLU ? static_cast<const T*>(a.gate_up) + ((size_t)e * 2 * N + f) * K
-                      : static_cast<const T*>(a.down) + ((size_t)e * N + f) * K;
+    const T* w0 = FIRST ? static_cast<const T*>(a.gate_up) + ((size_t)e * (glu ? 2 : 1) * N + f) * K
+                        : static_cast<const T*>(a.down) + ((size_t)e * N + f) * K;
     const T* w1 = w0 + (size_t)N * K;
     float s0 = 0.f, s1 = 0.f;
     for (int c = lane; c < K; c += 32) {
       s0 = fmaf(to_f<T>(w0[c]), xs[c], s0);
-      if (GLU) s1 = fmaf(to_f<T>(w1[c]), xs[c], s1);
+      if (glu) s1 = fmaf(to_f<T>(w1[c]), xs[c], s1);
     }
 #pragma unroll
     for (int o = 16; o; o >>= 1) {
@@ -140,8 +155,8 @@ __global__ void __launch_bounds__(256) moe_simple_kernel(pace_moe_experts_args_t
       s1 += __shfl_xor_sync(0xffffffffu, s1, o);
     }
     if (lane == 0) {
-      const float y = GLU ? (a.act == PACE_ACT_SILU ? silu_t<T>(s0) : gelu_tanh_t<T>(s0)) * s1 : s0;
-      (GLU ? static_cast<T*>(a.hidden) : static_cast<T*>(a.y))[(size_t)r * N + f] = from_f<T>(y);
+      const float y = FIRST ? act_t<T>(a.act, s0) * (glu ? s1 : 1.f) : s0;
+      (FIRST ? static_cast<T*>(a.hidden) : static_cast<T*>(a.y))[(size_t)r * N + f] = from_f<T>(y);
     }
   }
 }
@@ -167,17 +182,18 @@ __global__ void __launch_bounds__(256) moe_spread_kernel(pace_moe_experts_args_t
   for (int k = threadIdx.x >> 5; k < a.top; k += blockDim.x >> 5) {
     const int e = a.slot_expert[(size_t)t * a.top + k];
     int n = 0;
-    for (int i = lane; i < e; i += 32) n += a.expert_count[i];
+    for (int i = lane; i < e && e < a.n_experts; i += 32) n += a.expert_count[i];
 #pragma unroll
     for (int o = 16; o; o >>= 1) n += __shfl_xor_sync(0xffffffffu, n, o);
-    if (lane == 0) row[k] = n + a.slot_rank[(size_t)t * a.top + k];
+    if (lane == 0) row[k] = e < a.n_experts ? n + a.slot_rank[(size_t)t * a.top + k] : -1;   // -1: an identity expert
   }
   __syncthreads();
   const int pieces = a.width / 8;
   const uint4* src = static_cast<const uint4*>(a.x) + (size_t)t * pieces;
   for (int c = threadIdx.x; c < pieces; c += blockDim.x) {
     const uint4 v = src[c];
-    for (int k = 0; k < a.top; ++k) static_cast<uint4*>(a.scratch)[(size_t)row[k] * pieces + c] = v;
+    for (int k = 0; k < a.top; ++k)
+      if (row[k] >= 0) static_cast<uint4*>(a.scratch)[(size_t)row[k] * pieces + c] = v;
   }
 }
 
@@ -204,7 +220,7 @@ struct Tile {
 template <int NT>
 __host__ __device__ constexpr int stage_bytes() { return 2 * kABytes + NT * 128; }
 
-// GLU: act(gate) * up; otherwise plain products.  GATHER: token rows through the lists, otherwise in expert order.
+// GLU: act(gate) * up; otherwise act of plain products (second products: none).  GATHER: token rows through the lists, otherwise in expert order.
 template <int NT, bool GLU, bool GATHER>
 __global__ void __launch_bounds__(kThreads, 1)
     moe_grouped_kernel(const GroupedParams p, const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB) {
@@ -376,10 +392,10 @@ __global__ void __launch_bounds__(kThreads, 1)
         for (int j = 0; j < 16; ++j) {
           const float u0 = __uint_as_float(x0[j]), u1 = __uint_as_float(x1[j]);
           if constexpr (GLU) {
-            v[0][j] = (p.act == PACE_ACT_SILU ? silu_t<__nv_bfloat16>(u0) : gelu_tanh_t<__nv_bfloat16>(u0)) * u1;
+            v[0][j] = act_t<__nv_bfloat16>(p.act, u0) * u1;
           } else {
-            v[0][j] = u0;
-            v[1][j] = u1;
+            v[0][j] = act_t<__nv_bfloat16>(p.act, u0);
+            v[1][j] = act_t<__nv_bfloat16>(p.act, u1);
           }
         }
         // neighbouring lanes hold neighbouring features: they exchange one of two tokens and store pairs
@@ -449,11 +465,14 @@ int experts_umma(const pace_moe_experts_args_t& a, cudaStream_t s) {
   p.out = static_cast<__nv_bfloat16*>(a.hidden);
   p.K = a.width;
   p.N = a.ff;
-  p.a_rows = 2 * a.ff;
-  p.a_second = a.ff;
-  const int rc = GATHER ? grouped<NT, true, GATHER>(p, a.gate_up, a.x, a.n_tokens, s)
-                        : grouped<NT, true, GATHER>(p, a.gate_up, a.scratch, p.n_rows, s);
+  p.a_rows = a.gated ? 2 * a.ff : a.ff;
+  p.a_second = a.gated ? a.ff : 128;
+  const void* rows = GATHER ? a.x : a.scratch;
+  const int n_b_rows = GATHER ? a.n_tokens : p.n_rows;
+  const int rc = a.gated ? grouped<NT, true, GATHER>(p, a.gate_up, rows, n_b_rows, s)
+                         : grouped<NT, false, GATHER>(p, a.gate_up, rows, n_b_rows, s);
   if (rc != PACE_OK) return rc;
+  p.act = PACE_ACT_NONE;
   p.out = static_cast<__nv_bfloat16*>(a.y);
   p.K = a.ff;
   p.N = a.width;
@@ -498,7 +517,7 @@ int pace_moe_experts(const pace_moe_experts_args_t* a, void* stream) {
   if (!a || !a->x || !a->gate_up || !a->down || !a->hidden || !a->y || !a->expert_count || !a->expert_list || a->n_tokens < 0 ||
       a->n_experts < 1 || a->n_experts > kMaxExperts || a->top < 1 || a->width < 1 || a->ff < 1)
     return PACE_ERR_INVALID;
-  if (a->act != PACE_ACT_SILU && a->act != PACE_ACT_GELU_TANH) return PACE_ERR_INVALID;
+  if (a->act != PACE_ACT_SILU && a->act != PACE_ACT_GELU_TANH && a->act != PACE_ACT_GELU_ERF) return PACE_ERR_INVALID;
   if ((int64_t)a->n_tokens * a->top > 0x7fffffff || (int64_t)a->n_experts * 2 * a->ff > 0x7fffffff ||
       (int64_t)a->n_experts * a->width > 0x7fffffff)
     return PACE_ERR_UNSUPPORTED;

@@ -16,11 +16,26 @@ namespace {
 // inputs come from the cache after their first use.
 constexpr int kConvTokens = 4;
 
-template <typename T, int V, int NT>   // NT: number of taps where it is known at compile time, else 0
-__global__ void __launch_bounds__(256)
-    causal_conv_kernel(pace_step_t st, const T* __restrict__ in, int64_t in_stride, const float* __restrict__ taps,
-                       const float* __restrict__ bias, int n_taps, const float* __restrict__ conv_state, T* __restrict__ out,
-                       int channels) {
+template <typename T, int V, int NT, bool SILU>   // NT: number of taps where it is known at compile time, else 0
+__global__ void __launch_bounds__(256) causal_conv_kernel(pace_step_t st, pace_causal_conv_args_t a) {
+  const T* __restrict__ in = static_cast<const T*>(a.in);
+  const float *__restrict__ taps = a.taps, *__restrict__ conv_state = a.conv_state;
+  T* __restrict__ out = static_cast<T*>(a.out);
+  const int channels = a.channels, n_taps = a.n_taps;
+  const int64_t in_stride = a.in_stride;
+  auto start_from = [&](int c, float* v) {
+    if (a.bias) Vec<float, V>::load(a.bias + c, v);
+    else
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] = 0.f;
+  };
+  auto finish = [&](float* v, T* dst) {
+    if constexpr (SILU) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] = silu_t<T>(v[j]);
+    }
+    Vec<T, V>::store(dst, v);
+  };
   const int per = channels / V;
   const size_t total = (size_t)((st.n_tokens + kConvTokens - 1) / kConvTokens) * per;
   for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
@@ -35,7 +50,7 @@ __global__ void __launch_bounds__(256)
 #pragma unroll
         for (int r = 0; r < kConvTokens + NT - 1; ++r, row += in_stride) Vec<T, V>::load(row, x[r]);
         float b[V];
-        Vec<float, V>::load(bias + c, b);
+        start_from(c, b);
 #pragma unroll
         for (int r = 0; r < kConvTokens; ++r)
 #pragma unroll
@@ -50,7 +65,7 @@ __global__ void __launch_bounds__(256)
             for (int v = 0; v < V; ++v) acc[r][v] = fmaf(w[v], x[r + j][v], acc[r][v]);
         }
 #pragma unroll
-        for (int r = 0; r < kConvTokens; ++r) Vec<T, V>::store(out + (size_t)(t0 + r) * channels + c, acc[r]);
+        for (int r = 0; r < kConvTokens; ++r) finish(acc[r], out + (size_t)(t0 + r) * a.out_stride + c);
         continue;
       }
     }
@@ -61,8 +76,8 @@ __global__ void __launch_bounds__(256)
       const int t = min(t0 + r, st.n_tokens - 1), e = st.tok_entry[t];
       local[r] = t - st.cu[e];
       pos[r] = st.tok_pos[t];
-      ring[r] = conv_state + (size_t)st.slot[e] * n_taps * channels + c;
-      Vec<float, V>::load(bias + c, acc[r]);
+      ring[r] = conv_state + (size_t)st.slot[e] * a.ring_rows * a.ring_stride + c;
+      start_from(c, acc[r]);
     }
     for (int j = 0; j < n_taps; ++j) {
       const int back = n_taps - 1 - j;
@@ -73,7 +88,7 @@ __global__ void __launch_bounds__(256)
         const int t = min(t0 + r, st.n_tokens - 1);
         float x[V];
         if (local[r] >= back) Vec<T, V>::load(in + (size_t)(t - back) * in_stride + c, x);
-        else if (pos[r] >= back) Vec<float, V>::load(ring[r] + (size_t)((pos[r] - back) % n_taps) * channels, x);
+        else if (pos[r] >= back) Vec<float, V>::load(ring[r] + (size_t)((pos[r] - back) % a.ring_rows) * a.ring_stride, x);
         else continue;                                     // in front of the sequence
 #pragma unroll
         for (int v = 0; v < V; ++v) acc[r][v] = fmaf(w[v], x[v], acc[r][v]);
@@ -81,7 +96,19 @@ __global__ void __launch_bounds__(256)
     }
 #pragma unroll
     for (int r = 0; r < kConvTokens; ++r)
-      if (t0 + r < st.n_tokens) Vec<T, V>::store(out + (size_t)(t0 + r) * channels + c, acc[r]);
+      if (t0 + r < st.n_tokens) finish(acc[r], out + (size_t)(t0 + r) * a.out_stride + c);
+  }
+}
+
+// The newest inputs of every entry into its ring, behind the kernels that still read the older ones.
+template <typename T>
+__global__ void conv_store_kernel(pace_step_t st, const T* __restrict__ in, int64_t in_stride, float* __restrict__ ring, int rows,
+                                  int ring_stride, int channels) {
+  const int e = blockIdx.y, count = st.cu[e + 1] - st.cu[e], n = min(count, rows);
+  float* dst = ring + (size_t)st.slot[e] * rows * ring_stride;
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n * channels; i += gridDim.x * blockDim.x) {
+    const int j = i / channels, c = i - j * channels, l = count - 1 - j;
+    dst[(size_t)((st.start[e] + l) % rows) * ring_stride + c] = to_f<T>(in[(size_t)(st.cu[e] + l) * in_stride + c]);
   }
 }
 
@@ -583,20 +610,17 @@ int lightning_step_t(const pace_step_t& st, const pace_lightning_args_t& a, cuda
   return launch_lightning_step<T, 1>(st, a, s);
 }
 
-template <typename T>
-int causal_conv_t(const pace_step_t& st, const void* in, int64_t is, const float* taps, const float* bias, int n_taps,
-                  const float* cs, void* out, int channels, cudaStream_t s) {
+template <typename T, bool SILU>
+int causal_conv_t(const pace_step_t& st, const pace_causal_conv_args_t& a, cudaStream_t s) {
   constexpr int V = 8 / sizeof(T);      // (four bf16 or two fp32 channels: the window of rows stays in registers)
-  const bool vec = channels % V == 0 && is % V == 0 && aligned16(in) && aligned16(out) && aligned16(bias) && aligned16(cs) && aligned16(taps);
-  const size_t groups = (size_t)((st.n_tokens + kConvTokens - 1) / kConvTokens) * (channels / (vec ? V : 1));
+  const bool vec = a.channels % V == 0 && a.in_stride % V == 0 && a.out_stride % V == 0 && a.ring_stride % V == 0 &&
+                   aligned16(a.in) && aligned16(a.out) && aligned16(a.bias) && aligned16(a.conv_state) && aligned16(a.taps);
+  const size_t groups = (size_t)((st.n_tokens + kConvTokens - 1) / kConvTokens) * (a.channels / (vec ? V : 1));
   size_t blocks = (groups + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
-  if (vec && n_taps == 4)
-    causal_conv_kernel<T, V, 4><<<(unsigned)blocks, 256, 0, s>>>(st, (const T*)in, is, taps, bias, n_taps, cs, (T*)out, channels);
-  else if (vec)
-    causal_conv_kernel<T, V, 0><<<(unsigned)blocks, 256, 0, s>>>(st, (const T*)in, is, taps, bias, n_taps, cs, (T*)out, channels);
-  else
-    causal_conv_kernel<T, 1, 0><<<(unsigned)blocks, 256, 0, s>>>(st, (const T*)in, is, taps, bias, n_taps, cs, (T*)out, channels);
+  if (vec && a.n_taps == 4) causal_conv_kernel<T, V, 4, SILU><<<(unsigned)blocks, 256, 0, s>>>(st, a);
+  else if (vec) causal_conv_kernel<T, V, 0, SILU><<<(unsigned)blocks, 256, 0, s>>>(st, a);
+  else causal_conv_kernel<T, 1, 0, SILU><<<(unsigned)blocks, 256, 0, s>>>(st, a);
   PACE_LAUNCH_CHECK("causal_conv_kernel");
   return PACE_OK;
 }
@@ -641,15 +665,34 @@ using namespace pace;
 
 extern "C" {
 
-int pace_causal_conv(const pace_step_t* st, const void* in, int64_t is, const float* taps, const float* bias, int32_t n_taps,
-                     const float* cs, void* out, int32_t channels, int32_t dtype, void* stream) {
-  if (!step_ok(st) || !in || !taps || !bias || !cs || !out || n_taps < 1 || channels < 1 || !dtype_ok(dtype))
+int pace_causal_conv(const pace_step_t* st, const pace_causal_conv_args_t* a, void* stream) {
+  if (!step_ok(st) || !a || !a->in || !a->taps || !a->conv_state || !a->out || a->n_taps < 1 || a->channels < 1 ||
+      a->ring_rows < a->n_taps - 1 || a->ring_rows < 1 || a->ring_stride < a->channels || a->in_stride < a->channels ||
+      a->out_stride < a->channels || !dtype_ok(a->dtype))
     return PACE_ERR_INVALID;
   if (st->n_tokens == 0) return PACE_OK;
-  PACE_PROFILE("causal_conv", stream, "tokens=%d channels=%d", st->n_tokens, channels);
-  return dtype == PACE_DTYPE_BF16
-             ? causal_conv_t<__nv_bfloat16>(*st, in, is, taps, bias, n_taps, cs, out, channels, (cudaStream_t)stream)
-             : causal_conv_t<float>(*st, in, is, taps, bias, n_taps, cs, out, channels, (cudaStream_t)stream);
+  PACE_PROFILE("causal_conv", stream, "tokens=%d channels=%d", st->n_tokens, a->channels);
+  const cudaStream_t s = (cudaStream_t)stream;
+  if (a->dtype == PACE_DTYPE_BF16)
+    return a->silu ? causal_conv_t<__nv_bfloat16, true>(*st, *a, s) : causal_conv_t<__nv_bfloat16, false>(*st, *a, s);
+  return a->silu ? causal_conv_t<float, true>(*st, *a, s) : causal_conv_t<float, false>(*st, *a, s);
+}
+
+int pace_conv_store(const pace_step_t* st, const void* in, int64_t in_stride, float* ring, int32_t ring_rows, int32_t ring_stride,
+                    int32_t channels, int32_t dtype, void* stream) {
+  if (!step_ok(st) || !in || !ring || ring_rows < 1 || channels < 1 || ring_stride < channels || in_stride < channels ||
+      !dtype_ok(dtype))
+    return PACE_ERR_INVALID;
+  if (st->n_tokens == 0) return PACE_OK;
+  if (st->n_entries > 65535) return PACE_ERR_UNSUPPORTED;
+  const int64_t n = (int64_t)(st->max_count < ring_rows ? st->max_count : ring_rows) * channels;
+  const dim3 grid((unsigned)((n + 255) / 256 < 64 ? (n + 255) / 256 : 64), (unsigned)st->n_entries);
+  if (dtype == PACE_DTYPE_BF16)
+    conv_store_kernel<<<grid, 256, 0, (cudaStream_t)stream>>>(*st, (const __nv_bfloat16*)in, in_stride, ring, ring_rows, ring_stride, channels);
+  else
+    conv_store_kernel<<<grid, 256, 0, (cudaStream_t)stream>>>(*st, (const float*)in, in_stride, ring, ring_rows, ring_stride, channels);
+  PACE_LAUNCH_CHECK("conv_store_kernel");
+  return PACE_OK;
 }
 
 int pace_rglru_scan(const pace_step_t* st, const pace_rglru_args_t* a, void* stream) {

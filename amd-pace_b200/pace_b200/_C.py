@@ -35,7 +35,7 @@ class KVPoolStruct(C.Structure):
 ROWS_BF16, ROWS_OPAQUE, ROWS_SHARED = 0, 1, 2   # PACE_ROWS_*
 DTYPE_BF16, DTYPE_FP32 = 0, 1   # PACE_DTYPE_*
 SPAN_ALL, SPAN_WINDOW, SPAN_CHUNK = 0, 1, 2   # PACE_SPAN_*
-ACT_SILU, ACT_GELU_TANH = 0, 1  # PACE_ACT_*
+ACT_SILU, ACT_GELU_TANH, ACT_GELU_ERF = 0, 1, 2  # PACE_ACT_*
 
 ATTN_WHOLE_UNITS = 1      # PACE_ATTN_WHOLE_UNITS
 ATTN_PENDING_ROW = 2      # PACE_ATTN_PENDING_ROW
@@ -78,7 +78,9 @@ class ResidualNormArgs(C.Structure):
                [(n, C.c_int32) for n in ("width", "vocab", "restart", "dtype")] + \
                [("eps", C.c_float), ("weight_offset", C.c_float), ("embed_scale", C.c_float), ("top", C.c_int32),
                 ("n_experts", C.c_int32)] + \
-               [(n, C.c_void_p) for n in ("slot_expert", "slot_rank", "slot_weight", "expert_count")]
+               [(n, C.c_void_p) for n in ("slot_expert", "slot_rank", "slot_weight", "expert_count", "identity", "add")] + \
+               [("add_stride", C.c_int64)] + [(n, C.c_void_p) for n in ("y_bias", "embed_norm", "w_next2", "h2")] + \
+               [("y_mul", C.c_float)]
 
 
 class AppendNormArgs(C.Structure):
@@ -92,7 +94,8 @@ class AppendNormArgs(C.Structure):
 class AttnSpanArgs(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("q", "out", "slopes", "sinks")] + \
                [(n, C.c_int32) for n in ("n_q_heads", "dim", "vdim", "dtype", "q_elems", "out_elems", "entry_begin", "entry_end",
-                                         "max_tokens", "max_keys", "span", "span_size")] + [("scale", C.c_float)]
+                                         "max_tokens", "max_keys", "span", "span_size")] + \
+               [("scale", C.c_float), ("softcap", C.c_float), ("out_row", C.c_int64)]
 
 
 class AttnSpanPrefillArgs(C.Structure):
@@ -119,13 +122,14 @@ class RotateArgs(C.Structure):
 
 class MoeRouteArgs(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("logits", "correction", "slot_expert", "slot_rank", "slot_weight", "expert_count",
-                                          "expert_list")] + [(n, C.c_int32) for n in ("n_tokens", "n_experts", "top")]
+                                          "expert_list")] + \
+               [(n, C.c_int32) for n in ("n_tokens", "n_experts", "top", "softmax", "normalise")] + [("weight_scale", C.c_float)]
 
 
 class MoeExpertsArgs(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("x", "gate_up", "down", "hidden", "y", "scratch", "expert_count", "expert_list", "slot_expert",
                                           "slot_rank", "status")] + \
-               [(n, C.c_int32) for n in ("n_tokens", "n_experts", "top", "width", "ff", "act", "dtype")]
+               [(n, C.c_int32) for n in ("n_tokens", "n_experts", "top", "width", "ff", "act", "dtype", "gated")]
 
 
 class RglruArgs(C.Structure):
@@ -139,6 +143,41 @@ class LightningArgs(C.Structure):
     _fields_ = [("qkv", C.c_void_p), ("qkv_stride", C.c_int64), ("decay", C.c_void_p), ("state", C.c_void_p),
                 ("out", C.c_void_p), ("workspace", C.c_void_p), ("workspace_bytes", C.c_uint64)] + \
                [(n, C.c_int32) for n in ("heads", "dim", "vdim", "dtype")]
+
+
+class CausalConvArgs(C.Structure):
+    _fields_ = [("in_", C.c_void_p), ("in_stride", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("taps", "bias", "conv_state", "out")] + [("out_stride", C.c_int64)] + \
+               [(n, C.c_int32) for n in ("n_taps", "channels", "ring_rows", "ring_stride", "silu", "dtype")]
+
+
+class AppendConvArgs(C.Structure):
+    _fields_ = [("qkv", C.c_void_p), ("qkv_stride", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("taps", "ring", "q_norm", "k_norm", "cos_table", "sin_table", "q_out")] + \
+               [(n, C.c_int32) for n in ("n_q_heads", "dim", "vdim", "n_taps", "ring_rows", "ring_stride", "rot_pairs", "table_rows",
+                                         "store_ring", "dtype")] + [("eps", C.c_float), ("v_mul", C.c_float)]
+
+
+class PartNormGateArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("o", "gate", "w", "out")] + \
+               [(n, C.c_int64) for n in ("o_stride", "gate_stride", "out_stride")] + \
+               [(n, C.c_int32) for n in ("n_tokens", "n", "part", "w_period", "gate_first", "dtype")] + [("eps", C.c_float)]
+
+
+class SsdArgs(C.Structure):
+    _fields_ = [("xbc", C.c_void_p), ("xbc_stride", C.c_int64), ("dt_raw", C.c_void_p), ("dt_stride", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("dt_bias", "neg_a", "d_skip", "s_state", "out")] + [("out_stride", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("taps", "conv_bias", "ring", "workspace")] + [("workspace_bytes", C.c_uint64)] + \
+               [(n, C.c_int32) for n in ("heads", "groups", "state", "vdim", "n_taps", "ring_rows", "ring_stride", "dtype")]
+
+
+class DeltaArgs(C.Structure):
+    _fields_ = [("qkv", C.c_void_p), ("qkv_stride", C.c_int64), ("a_raw", C.c_void_p), ("a_stride", C.c_int64),
+                ("b_raw", C.c_void_p), ("b_stride", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("dt_bias", "neg_a", "s_state", "out")] + [("out_stride", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("taps", "ring", "workspace")] + [("workspace_bytes", C.c_uint64)] + \
+               [(n, C.c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "n_taps", "ring_rows", "ring_stride", "dtype")] + \
+               [("unit_eps", C.c_float), ("q_scale", C.c_float)]
 
 
 byref = C.byref
@@ -190,7 +229,16 @@ _SIGS = {
     "pace_latent_append": (C.c_int, [_P, C.c_int32, _S, C.POINTER(LatentAppendArgs), C.c_void_p]),
     "pace_rotate_heads": (C.c_int, [_S, C.POINTER(RotateArgs), C.c_void_p]),
     "pace_latent_gather": (C.c_int, [_P, C.c_int32, C.c_void_p, C.c_void_p, C.c_int32, C.c_void_p, C.c_void_p]),
-    "pace_glu": (C.c_int, [C.c_void_p, C.c_int64, C.c_void_p, C.c_int32, C.c_int32, C.c_int32, C.c_int32, C.c_void_p]),
+    "pace_glu": (C.c_int, [C.c_void_p, C.c_int64, C.c_void_p, C.c_int64] + [C.c_int32] * 5 + [C.c_void_p]),
+    "pace_soft_cap": (C.c_int, [C.c_void_p, C.c_int64, C.c_float, C.c_void_p]),
+    "pace_part_norm_gate": (C.c_int, [C.POINTER(PartNormGateArgs), C.c_void_p]),
+    "pace_kv_append_conv": (C.c_int, [_P, C.c_int32, _S, C.POINTER(AppendConvArgs), C.c_void_p]),
+    "pace_ssd_workspace_bytes": (C.c_uint64, [C.c_int32] * 5),
+    "pace_ssd_prefill": (C.c_int, [_S, C.POINTER(SsdArgs), C.c_void_p]),
+    "pace_ssd_step": (C.c_int, [_S, C.POINTER(SsdArgs), C.c_void_p]),
+    "pace_delta_workspace_bytes": (C.c_uint64, [C.c_int32] * 6),
+    "pace_delta_prefill": (C.c_int, [_S, C.POINTER(DeltaArgs), C.c_void_p]),
+    "pace_delta_step": (C.c_int, [_S, C.POINTER(DeltaArgs), C.c_void_p]),
     "pace_moe_route": (C.c_int, [C.POINTER(MoeRouteArgs), C.c_void_p]),
     "pace_moe_experts": (C.c_int, [C.POINTER(MoeExpertsArgs), C.c_void_p]),
     "pace_gate_heads": (C.c_int, [_S, C.c_void_p, C.c_void_p, C.c_int64, C.c_void_p, C.c_int32, C.c_int32, C.c_int32,
@@ -198,8 +246,8 @@ _SIGS = {
     "pace_norm_gate": (C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int64, C.c_void_p, C.c_int32, C.c_int32, C.c_float,
                                  C.c_int32, C.c_void_p]),
     "pace_relu_squared": (C.c_int, [C.c_void_p, C.c_int64, C.c_int32, C.c_void_p]),
-    "pace_causal_conv": (C.c_int, [_S, C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_int32, C.c_void_p, C.c_void_p,
-                                   C.c_int32, C.c_int32, C.c_void_p]),
+    "pace_causal_conv": (C.c_int, [_S, C.POINTER(CausalConvArgs), C.c_void_p]),
+    "pace_conv_store": (C.c_int, [_S, C.c_void_p, C.c_int64, C.c_void_p] + [C.c_int32] * 4 + [C.c_void_p]),
     "pace_rglru_scan": (C.c_int, [_S, C.POINTER(RglruArgs), C.c_void_p]),
     "pace_rglru_step": (C.c_int, [_S, C.POINTER(RglruArgs), C.c_void_p]),
     "pace_lightning_workspace_bytes": (C.c_uint64, [C.c_int32] * 5),

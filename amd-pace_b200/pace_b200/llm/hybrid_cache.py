@@ -1,7 +1,7 @@
 """Caches of hybrid decoders: paged K/V for attention layers, fixed-size recurrent states for the others.
 
-A model describes what each of its layer runs remembers (``KVSpec``, ``LatentSpec`` or ``StateSpec``; a layer that runs several
-times has one entry per run).  ``HybridCacheManager`` keeps one paged pool (``KVPool`` under a
+A model describes what each of its layer runs remembers (``KVSpec``, ``LatentSpec``, ``StateSpec``, or a ``JointSpec`` of them; a
+layer that runs several times has one entry per run).  ``HybridCacheManager`` keeps one paged pool (``KVPool`` under a
 ``KVCacheManager``) per distinct K/V geometry and one state array per recurrent run, all indexed by the same
 batch rows, and presents what the generation loops use of ``KVCacheManager``: lengths per row, recycling of
 finished rows, beam gather, the switches of graph capture, status checks.
@@ -39,6 +39,12 @@ class LatentSpec:
 class StateSpec:
     """Shapes per sequence of a recurrent run's fp32 arrays."""
     shapes: Tuple[Tuple[str, Tuple[int, ...]], ...]
+
+
+@dataclass(frozen=True)
+class JointSpec:
+    """A layer run that remembers several things (mixers side by side): its cache is the tuple of theirs."""
+    parts: Tuple[Union[KVSpec, LatentSpec, StateSpec], ...]
 
 
 def kv_row(spec: Union[KVSpec, LatentSpec], dtype: torch.dtype) -> Tuple[int, int]:
@@ -97,6 +103,10 @@ class PoolSet:
             bits, free = bits | b, min(free, f)
         return bits, free
 
+    def status_word(self) -> Optional[torch.Tensor]:
+        """Where kernels that belong to no pool report (None: there is no pool)."""
+        return self.pools[0].status_word() if self.pools else None
+
     def check_status(self) -> None:
         for p in self.pools:
             p.check_status()
@@ -112,14 +122,16 @@ class _GroupConfig:
 
 
 class HybridCacheManager:
-    """``specs``: one (``KVSpec``, ``LatentSpec`` or ``StateSpec``) per layer run.  ``pool_tokens``: tokens the K/V pools hold for all rows together (rounded
+    """``specs``: one (``KVSpec``, ``LatentSpec``, ``StateSpec`` or ``JointSpec``) per layer run.  ``pool_tokens``: tokens the K/V pools hold for all rows together (rounded
     down to pages); ``batch``: rows, each with a slot in every pool and state array."""
 
-    def __init__(self, specs: Sequence[Union[KVSpec, LatentSpec, StateSpec]], batch: int, pool_tokens: int, max_seq_len: int,
+    def __init__(self, specs: Sequence[Union[KVSpec, LatentSpec, StateSpec, JointSpec]], batch: int, pool_tokens: int, max_seq_len: int,
                  dtype: torch.dtype, device, cache_type: KVCacheType = KVCacheType.DYNAMIC):
         self.batch, self.max_seq_len, self.dtype = batch, max_seq_len, dtype
         self.device = torch.device(device)
         self.num_layers = len(specs)
+        joint = [len(s.parts) if isinstance(s, JointSpec) else 0 for s in specs]
+        specs = [p for s in specs for p in (s.parts if isinstance(s, JointSpec) else (s,))]
         self._lens = [0] * batch
         self.page_tokens = physical_page_tokens(None)
         n_pages = max(1, pool_tokens // self.page_tokens)
@@ -143,6 +155,8 @@ class HybridCacheManager:
             if isinstance(s, StateSpec):
                 self.caches[i] = StateCache(self, s, batch, self.device)
                 self.states.append(self.caches[i])
+        parts = iter(self.caches)
+        self.caches = [tuple(next(parts) for _ in range(n)) if n else next(parts) for n in joint]
         self.pool = PoolSet([g.pool for g in self.groups], n_pages)
         # rows map to slots 1:1: every pool is this manager's own
         self.slots = list(range(batch))

@@ -1,6 +1,6 @@
 """What decoders that run on a packed ``Step`` have in common: parameters, checkpoint reading, and the forward forms
 that the schedulers and generation loops call.  A model brings ``forward_step`` and what its layers remember."""
-from typing import Dict, List, Optional, Sequence
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 from torch import nn
@@ -27,6 +27,12 @@ class CheckpointTensors:
     def __init__(self, tensors: Dict[str, torch.Tensor]):
         self.tensors, self.used = tensors, set()
 
+    def shape(self, name: str) -> Tuple[int, ...]:
+        """For sizes that only the checkpoint names."""
+        if name not in self.tensors:
+            raise KeyError(f"checkpoint has no tensor {name}")
+        return tuple(self.tensors[name].shape)
+
     def take(self, name: str, *shape: int) -> torch.Tensor:
         if name not in self.tensors:
             raise KeyError(f"checkpoint has no tensor {name}")
@@ -49,7 +55,7 @@ class StepModel(nn.Module):
         raise NotImplementedError
 
     def cache_specs(self) -> list:
-        """What every layer run remembers (``KVSpec``, ``LatentSpec`` or ``StateSpec``), in execution order."""
+        """What every layer run remembers (``KVSpec``, ``LatentSpec``, ``StateSpec`` or ``JointSpec``), in execution order."""
         raise NotImplementedError
 
     def prepare(self, max_seq_len: int) -> None:
@@ -96,9 +102,13 @@ class StepCausalLM(nn.Module):
         self.lm_head = _Head(config.vocab_size, config.hidden_size, dtype)
 
     # -- weights and caches --------------------------------------------------------------------------
+    def load_head(self, t: CheckpointTensors) -> None:
+        self.lm_head.weight.copy_(t.take("head", *self.lm_head.weight.shape))
+
     @torch.no_grad()
     def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
-        """``embed``, ``l<i>.*`` (layers with a ``load`` method), ``final.norm``, ``head``; nothing may be left over."""
+        """``embed``, ``l<i>.*`` (layers with a ``load`` method), ``final.norm``, what ``load_head`` takes; nothing may be left
+        over."""
         t, V, W = CheckpointTensors(tensors), self.config.vocab_size, self.config.hidden_size
         self.model.embed.copy_(t.take("embed", V, W))
         done = set()
@@ -107,7 +117,7 @@ class StepCausalLM(nn.Module):
                 lay.load(t, f"l{i}.")
                 done.add(id(lay))
         self.model.norm.copy_(t.take("final.norm", W))
-        self.lm_head.weight.copy_(t.take("head", V, W))
+        self.load_head(t)
         if t.unused():
             raise ValueError(f"checkpoint tensors without a place in the model: {t.unused()[:8]}")
 

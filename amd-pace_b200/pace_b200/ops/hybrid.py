@@ -1,5 +1,5 @@
 """Operators of hybrid decoders over a packed ``Step``: fused residual norms, attention with normalised keys,
-gated linear recurrence, decayed linear attention.  Thin callers of the C ABI (include/pace_b200.h); every
+gated linear recurrence, decayed linear attention, state-space recurrence, gated delta rule, mixtures of experts.  Thin callers of the C ABI (include/pace_b200.h); every
 constant of a model is an argument.  ``torch.float32`` activations run the same functions in full 32-bit."""
 from dataclasses import dataclass
 from typing import Optional
@@ -22,29 +22,36 @@ class Routed:
     slot_expert: torch.Tensor
     slot_rank: torch.Tensor
     slot_weight: torch.Tensor
-    count: torch.Tensor
+    count: torch.Tensor          # experts with weights, without the identity experts behind them
     lists: torch.Tensor
     y: Optional[torch.Tensor] = None
+    identity: Optional[torch.Tensor] = None    # the rows identity experts hand on
 
 
 def residual_norm(step: Step, x: torch.Tensor, y: Optional[torch.Tensor] = None, w_post: Optional[torch.Tensor] = None,
                   embed: Optional[torch.Tensor] = None, w_next: Optional[torch.Tensor] = None, eps: float = 1e-6,
                   restart: bool = False, weight_offset: float = 0.0, dtype: Optional[torch.dtype] = None,
-                  embed_scale: float = 1.0, plain: bool = False, routed: Optional[Routed] = None):
-    """x (fp32, in place) takes ``rms(y) * w_post`` and, with ``embed``, the tokens' embedding rows times
-    ``embed_scale``; returns ``rms(x) * w_next`` in the activations' dtype (None without ``w_next``; with ``plain`` x
-    itself, rounded).  ``routed``: y is the weighted sum of the experts' rows, taken up on the way."""
-    h = None
+                  embed_scale: float = 1.0, plain: bool = False, routed: Optional[Routed] = None, bias: Optional[torch.Tensor] = None,
+                  y_mul: float = 1.0, embed_norm: Optional[torch.Tensor] = None, w_next2: Optional[torch.Tensor] = None):
+    """x (fp32, in place) takes ``rms(y) * w_post`` (without w_post ``y_mul * y``) and, with ``embed``, the tokens' embedding rows
+    times ``embed_scale`` or normalised (``embed_norm``); returns ``rms(x) * w_next`` in the activations' dtype (None without
+    ``w_next``; with ``plain`` x itself, rounded), with ``w_next2`` a pair of two such norms of the same x.  ``bias`` (fp32)
+    belongs to y.  ``routed``: the weighted sum of the experts' rows is (with y: is added to) the output, taken up on the way."""
+    h = h2 = add = None
     if routed is not None:
-        y = routed.y
+        y, add = routed.y, y
     if w_next is not None or plain:
         h = torch.empty(x.shape, dtype=dtype or (y if y is not None else embed).dtype, device=x.device)
+    if w_next2 is not None:
+        h2 = torch.empty_like(h)
+    more = (add, bias, embed_norm, w_next2, h2, y_mul)
     if routed is None:
-        _OPS.residual_norm(step.handle, x, y, w_post, embed, w_next, h, eps, restart, weight_offset, embed_scale)
+        _OPS.residual_norm(step.handle, x, y, w_post, embed, w_next, h, eps, restart, weight_offset, embed_scale, 0, None, None, None,
+                           None, None, *more)
     else:
         _OPS.residual_norm(step.handle, x, y, w_post, embed, w_next, h, eps, restart, weight_offset, embed_scale, routed.top,
-                           routed.slot_expert, routed.slot_rank, routed.slot_weight, routed.count)
-    return h
+                           routed.slot_expert, routed.slot_rank, routed.slot_weight, routed.count, routed.identity, *more)
+    return h if h2 is None else (h, h2)
 
 
 def step_attention(step: Step, cache, qkv: torch.Tensor, heads: int, dim: int, vdim: int, scale: float,
@@ -113,17 +120,45 @@ def span_attention(step: Step, cache, qkv: torch.Tensor, heads: int, dim: int, v
     out = torch.empty(T, heads, vdim, dtype=qkv.dtype, device=qkv.device)
     _OPS.kv_append_norm(pool.handle, pool.pages, cache.layer, step.handle, qkv, None, None, q, dim, vdim, eps, 1.0, 0.0, 1.0,
                         True)
-    rule = (slopes, sinks, dim, vdim, scale) + _span(window, chunk)
-    Ed, E = step.n_decode, step.n_entries
-    if (E > Ed and qkv.dtype == torch.bfloat16 and pool.desc.row_format == _C.ROWS_BF16
-            and step.max_count * (heads // pool.n_kv_heads) >= PROMPT_ROWS
+    _span_over_pages(step, cache, q, out, (slopes, sinks, dim, vdim, scale) + _span(window, chunk))
+    return out.view(T, heads * vdim)
+
+
+def _span_over_pages(step: Step, cache, q: torch.Tensor, out: torch.Tensor, rule: tuple, softcap: float = 0.0) -> None:
+    """The span kernels over a step's entries: those of one token, then the others (tcgen05 where it is worth a launch)."""
+    pool, Ed, E = cache.pool, step.n_decode, step.n_entries
+    tail = (softcap, out.stride(0))
+    if (E > Ed and q.dtype == torch.bfloat16 and pool.desc.row_format == _C.ROWS_BF16
+            and step.max_count * (q.shape[1] // pool.n_kv_heads) >= PROMPT_ROWS
             and _OPS.attn_span_prefill(pool.handle, pool.pages, cache.layer, step.handle, q, out, *rule, Ed, E, step.max_count,
-                                       step.max_keys, None, None, None, None, None)):
+                                       step.max_keys, None, None, None, None, None, *tail)):
         E = Ed
     for lo, hi, n in ((0, Ed, 1), (Ed, E, step.max_count)):
         if lo < hi:
-            _OPS.attn_span(pool.handle, pool.pages, cache.layer, step.handle, q, out, *rule, lo, hi, n, step.max_keys)
-    return out.view(T, heads * vdim)
+            _OPS.attn_span(pool.handle, pool.pages, cache.layer, step.handle, q, out, *rule, lo, hi, n, step.max_keys, *tail)
+
+
+def conv_attention(step: Step, cache, qkv: torch.Tensor, taps: torch.Tensor, ring: torch.Tensor, q_norm: torch.Tensor,
+                   k_norm: torch.Tensor, tables, heads: int, dim: int, vdim: int, scale: float, eps: float, softcap: float = 0.0,
+                   v_mul: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal attention behind short convolutions: every channel of q, k and v is convolved over time, queries and keys are
+    normalised per head (weights shared by the heads) and rotated by ``tables`` (None: not), then the softmax over capped
+    scores.  ``qkv`` [T, >= ...]: projection rows (q, k, v); ``taps`` fp32 [taps, channels]; ``ring`` fp32 [slots, rows,
+    channels]: the newest projections of every slot, stored here in a step of one token per entry and by ``conv_store``
+    otherwise.  Values are cached times ``v_mul``.  ``out`` [T, heads * vdim] may have a row stride of its own."""
+    pool, T = cache.pool, step.n_tokens
+    q = torch.empty(T, heads, _pool_row(pool, qkv.dtype), dtype=qkv.dtype, device=qkv.device)
+    if out is None:
+        out = torch.empty(T, heads * vdim, dtype=qkv.dtype, device=qkv.device)
+    _OPS.kv_append_conv(pool.handle, pool.pages, cache.layer, step.handle, qkv, taps, ring, q_norm, k_norm, *(tables or (None, None)),
+                        q, dim, vdim, eps, v_mul, step.decode_only)
+    _span_over_pages(step, cache, q, out.unflatten(1, (heads, vdim)), (None, None, dim, vdim, scale, _C.SPAN_ALL, 0), softcap)
+    return out
+
+
+def conv_store(step: Step, x: torch.Tensor, ring: torch.Tensor) -> None:
+    """The newest rows of ``x`` [T, >= channels] of every entry into its ring, behind the launches that read the older ones."""
+    _OPS.conv_store(step.handle, x, ring)
 
 
 def latent_attention(step: Step, cache, down: torch.Tensor, q_norm: torch.Tensor, kv_norm: torch.Tensor, q_up: torch.Tensor,
@@ -187,35 +222,46 @@ def expand_pays(step: Step, dtype: torch.dtype, heads: int, dim: int, rot_dim: i
     return step.max_count >= 32 and expanded < absorbed
 
 
-def glu(x: torch.Tensor, act: int) -> torch.Tensor:
-    """act(gate) * up of rows ``[T, 2 n]`` (gate first)."""
-    out = torch.empty(x.shape[0], x.shape[1] // 2, dtype=x.dtype, device=x.device)
+def glu(x: torch.Tensor, act: int, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """act(gate) * up of rows ``[T, 2 n]`` (gate first); ``out`` may have a row stride of its own."""
+    if out is None:
+        out = torch.empty(x.shape[0], x.shape[1] // 2, dtype=x.dtype, device=x.device)
     _OPS.glu(x, out, act)
     return out
 
 
-def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int) -> Routed:
-    """Sigmoid scores of every expert in fp32, the ``top`` largest by score + ``correction``, weighted by their scores."""
+def activate(x: torch.Tensor, act: int, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """act(x) of rows ``[T, n]``; ``out`` may have a row stride of its own."""
+    out = torch.empty_like(x) if out is None else out
+    _OPS.glu(x, out, act, False)
+    return out
+
+
+def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int, softmax: bool = False,
+              weight_scale: Optional[float] = None, identity: int = 0) -> Routed:
+    """Sigmoid (or softmax) scores of every router output in fp32, the ``top`` largest by score + ``correction``, weighted by
+    their scores (``weight_scale``: made to sum to that).  The last ``identity`` outputs are experts that hand on ``h`` itself."""
     logits = linear_f32(h, router)
     T, E = logits.shape
     ints = torch.empty(2 * T * top + E + E * T, dtype=torch.int32, device=h.device)
     a, b = T * top, 2 * T * top
     r = Routed(top, ints[:a].view(T, top), ints[a:b].view(T, top), torch.empty(T, top, dtype=torch.float32, device=h.device),
-               ints[b: b + E], ints[b + E:].view(E, T))
-    _OPS.moe_route(logits, correction, r.slot_expert, r.slot_rank, r.slot_weight, r.count, r.lists)
+               ints[b: b + E - identity], ints[b + E:].view(E, T), identity=h if identity else None)
+    _OPS.moe_route(logits, correction, r.slot_expert, r.slot_rank, r.slot_weight, ints[b: b + E], r.lists, softmax, weight_scale)
     return r
 
 
 def moe_experts(h: torch.Tensor, routed: Routed, gate_up: torch.Tensor, down: torch.Tensor, act: int,
-                status: Optional[torch.Tensor] = None) -> Routed:
-    """The chosen experts' feed-forwards, left by expert in ``routed.y`` (``residual_norm`` sums them up)."""
+                status: Optional[torch.Tensor] = None, gated: bool = True) -> Routed:
+    """The chosen experts' feed-forwards (gated: ``gate_up`` holds gate and up rows), left by expert in ``routed.y``
+    (``residual_norm`` sums them up)."""
     n = h.shape[0] * routed.top
     hidden = torch.empty(n, down.shape[2], dtype=h.dtype, device=h.device)
     routed.y = torch.empty(n, down.shape[1], dtype=h.dtype, device=h.device)
     # many tokens per expert: wide tiles, over rows that are copied into expert order first
     scratch = torch.empty(n, h.shape[1], dtype=h.dtype, device=h.device) if n > MOE_WIDE * down.shape[0] else None
     _OPS.moe_experts(h, gate_up, down, hidden, routed.y, scratch, routed.count, routed.lists, routed.slot_expert, routed.slot_rank,
-                     status, act)
+                     status, act, gated)
     return routed
 
 
@@ -231,6 +277,21 @@ def norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: fl
     out = torch.empty_like(o)
     _OPS.norm_gate(o, weight, gate, out, eps)
     return out
+
+
+def part_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, part: int, eps: float, gate_first: bool = False,
+                   out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """rms over every ``part`` elements of a row: ``rms(o) * weight * sigmoid(gate)``, or with the gate in front
+    ``rms(o * silu(gate)) * weight``; the weight repeats along the row.  ``out`` may have a row stride of its own."""
+    out = torch.empty_like(o) if out is None else out
+    _OPS.part_norm_gate(o, gate, weight, out, part, gate_first, eps)
+    return out
+
+
+def soft_cap_(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """cap * tanh(x / cap) in place (fp32)."""
+    _OPS.soft_cap(x, cap)
+    return x
 
 
 def relu_squared_(x: torch.Tensor) -> torch.Tensor:
@@ -264,6 +325,41 @@ def lightning(step: Step, qkv: torch.Tensor, decay: torch.Tensor, state: torch.T
     out = torch.empty(step.n_tokens, state.shape[1] * state.shape[3], dtype=qkv.dtype, device=qkv.device)
     op = _OPS.lightning_step if step.decode_only else _OPS.lightning_prefill
     op(step.handle, qkv, decay, state, out)
+    return out
+
+
+def ssd(step: Step, xbc: torch.Tensor, dt_raw: torch.Tensor, taps: torch.Tensor, conv_bias: Optional[torch.Tensor],
+        dt_bias: torch.Tensor, neg_a: torch.Tensor, d_skip: torch.Tensor, groups: int, state: torch.Tensor,
+        ring: torch.Tensor) -> torch.Tensor:
+    """State-space recurrence behind a short convolution with silu.  ``xbc`` [T, >= channels]: projections x (heads x vdim),
+    b and c (groups x state each); ``dt_raw`` [T, heads]; ``state`` fp32 [slots, heads, state, vdim]; ``ring`` as in
+    ``conv_attention``.  Returns [T, heads * vdim].  One token per entry: one launch, which also stores the ring."""
+    T, inner = step.n_tokens, state.shape[1] * state.shape[3]
+    out = torch.empty(T, inner, dtype=xbc.dtype, device=xbc.device)
+    if step.decode_only:
+        _OPS.ssd_step(step.handle, xbc, dt_raw, dt_bias, neg_a, d_skip, state, out, groups, taps, conv_bias, ring)
+        return out
+    u = torch.empty(T, (taps.shape[1] + 7) // 8 * 8, dtype=xbc.dtype, device=xbc.device)
+    _OPS.causal_conv(step.handle, xbc, taps, conv_bias, ring, u, True)
+    _OPS.ssd_prefill(step.handle, u, dt_raw, dt_bias, neg_a, d_skip, state, out, groups)
+    return out
+
+
+def delta_rule(step: Step, qkv: torch.Tensor, a_raw: torch.Tensor, b_raw: torch.Tensor, taps: torch.Tensor, dt_bias: torch.Tensor,
+               neg_a: torch.Tensor, kv_heads: int, state: torch.Tensor, ring: torch.Tensor, unit_eps: float,
+               q_scale: float) -> torch.Tensor:
+    """Gated delta rule with a decay per key channel behind a short convolution with silu.  ``qkv`` [T, >= channels]: projections
+    q, k (kv_heads x dim each) and v (heads x vdim); ``a_raw`` [T, heads * dim], ``b_raw`` [T, heads]; ``state`` fp32 [slots,
+    heads, dim, vdim]; ``ring`` as in ``conv_attention``.  Returns [T, heads * vdim].  One token per entry: one launch, which
+    also stores the ring."""
+    T = step.n_tokens
+    out = torch.empty(T, state.shape[1] * state.shape[3], dtype=qkv.dtype, device=qkv.device)
+    if step.decode_only:
+        _OPS.delta_step(step.handle, qkv, a_raw, b_raw, dt_bias, neg_a, state, out, kv_heads, unit_eps, q_scale, taps, ring)
+        return out
+    u = torch.empty(T, (taps.shape[1] + 7) // 8 * 8, dtype=qkv.dtype, device=qkv.device)
+    _OPS.causal_conv(step.handle, qkv, taps, None, ring, u, True)
+    _OPS.delta_prefill(step.handle, u, a_raw, b_raw, dt_bias, neg_a, state, out, kv_heads, unit_eps, q_scale)
     return out
 
 

@@ -44,30 +44,49 @@ _DEFS["linear_skinny"] = "(Tensor x, Tensor weight, Tensor(a!) out, Tensor(b!) w
 _DEFS.update({
     "residual_norm": "(int step, Tensor(a!) x, Tensor? y, Tensor? w_post, Tensor? embed, Tensor? w_next, Tensor(b!)? h, "
                      "float eps, bool restart, float weight_offset, float embed_scale=1.0, int top=0, Tensor? slot_expert=None, "
-                     "Tensor? slot_rank=None, Tensor? slot_weight=None, Tensor? expert_count=None) -> ()",
+                     "Tensor? slot_rank=None, Tensor? slot_weight=None, Tensor? expert_count=None, Tensor? identity=None, "
+                     "Tensor? add=None, Tensor? y_bias=None, Tensor? embed_norm=None, Tensor? w_next2=None, Tensor(c!)? h2=None, "
+                     "float y_mul=1.0) -> ()",
     "kv_append_norm": "(int pool, Tensor(a!) pages, int layer, int step, Tensor qkv, Tensor? q_norm, Tensor? k_norm, "
                       "Tensor(b!) q_out, int dim, int vdim, float eps, float q_mul, float temp_coef, float temp_every, "
                       "bool per_head=False) -> ()",
     "attn_span": "(int pool, Tensor pages, int layer, int step, Tensor q, Tensor(a!) out, Tensor? slopes, Tensor? sinks, int dim, "
-                 "int vdim, float scale, int span, int span_size, int entry_begin, int entry_end, int max_tokens, int max_keys) -> ()",
+                 "int vdim, float scale, int span, int span_size, int entry_begin, int entry_end, int max_tokens, int max_keys, "
+                 "float softcap=0.0, int out_row=0) -> ()",
     "attn_span_prefill": "(int pool, Tensor? pages, int layer, int step, Tensor q, Tensor(a!) out, Tensor? slopes, Tensor? sinks, "
                          "int dim, int vdim, float scale, int span, int span_size, int entry_begin, int entry_end, int max_tokens, "
-                         "int max_keys, Tensor? k, Tensor? k2, Tensor? v, Tensor? key_cu, Tensor? key_pos) -> bool",
+                         "int max_keys, Tensor? k, Tensor? k2, Tensor? v, Tensor? key_cu, Tensor? key_pos, "
+                         "float softcap=0.0, int out_row=0) -> bool",
     "latent_append": "(int pool, Tensor(a!) pages, int layer, int step, Tensor down, Tensor q_norm, Tensor kv_norm, Tensor cos, "
                      "Tensor sin, Tensor(b!) cq, int rot_dim, float eps) -> ()",
     "rotate_heads": "(int step, Tensor src, Tensor(a!) dst, Tensor cos, Tensor sin, int token_begin, int token_end, int pad_dim) -> ()",
     "latent_gather": "(int pool, Tensor pages, int layer, Tensor slot, Tensor pos, Tensor(a!) out) -> ()",
-    "glu": "(Tensor x, Tensor(a!) out, int act) -> ()",
+    "glu": "(Tensor x, Tensor(a!) out, int act, bool gated=True) -> ()",
+    "soft_cap": "(Tensor(a!) x, float cap) -> ()",
+    "part_norm_gate": "(Tensor o, Tensor gate, Tensor w, Tensor(a!) out, int part, bool gate_first, float eps) -> ()",
+    "kv_append_conv": "(int pool, Tensor(a!) pages, int layer, int step, Tensor qkv, Tensor taps, Tensor(b!) ring, Tensor q_norm, "
+                      "Tensor k_norm, Tensor? cos, Tensor? sin, Tensor(c!) q_out, int dim, int vdim, float eps, float v_mul, "
+                      "bool store_ring) -> ()",
+    "conv_store": "(int step, Tensor x, Tensor(a!) ring) -> ()",
+    "ssd_prefill": "(int step, Tensor xbc, Tensor dt_raw, Tensor dt_bias, Tensor neg_a, Tensor d_skip, Tensor(a!) state, "
+                   "Tensor(b!) out, int groups) -> ()",
+    "ssd_step": "(int step, Tensor xbc, Tensor dt_raw, Tensor dt_bias, Tensor neg_a, Tensor d_skip, Tensor(a!) state, "
+                "Tensor(b!) out, int groups, Tensor taps, Tensor? conv_bias, Tensor(c!) ring) -> ()",
+    "delta_prefill": "(int step, Tensor qkv, Tensor a_raw, Tensor b_raw, Tensor dt_bias, Tensor neg_a, Tensor(a!) state, "
+                     "Tensor(b!) out, int kv_heads, float unit_eps, float q_scale) -> ()",
+    "delta_step": "(int step, Tensor qkv, Tensor a_raw, Tensor b_raw, Tensor dt_bias, Tensor neg_a, Tensor(a!) state, "
+                  "Tensor(b!) out, int kv_heads, float unit_eps, float q_scale, Tensor taps, Tensor(c!) ring) -> ()",
     "moe_route": "(Tensor logits, Tensor? correction, Tensor(a!) slot_expert, Tensor(b!) slot_rank, Tensor(c!) slot_weight, "
-                 "Tensor(d!) expert_count, Tensor(e!) expert_list) -> ()",
+                 "Tensor(d!) expert_count, Tensor(e!) expert_list, bool softmax=False, float? weight_scale=None) -> ()",
     "moe_experts": "(Tensor x, Tensor gate_up, Tensor down, Tensor(a!) hidden, Tensor(b!) y, Tensor(d!)? scratch, "
-                   "Tensor expert_count, Tensor expert_list, Tensor slot_expert, Tensor slot_rank, Tensor(c!)? status, int act) -> ()",
+                   "Tensor expert_count, Tensor expert_list, Tensor slot_expert, Tensor slot_rank, Tensor(c!)? status, int act, "
+                   "bool gated=True) -> ()",
     "attn_general": "(int pool, Tensor pages, int layer, int step, Tensor q, Tensor(a!) out, int dim, int vdim, "
                     "float scale) -> ()",
     "gate_heads": "(int step, Tensor attn, Tensor gate, Tensor(a!) out, int vdim) -> ()",
     "norm_gate": "(Tensor o, Tensor weight, Tensor gate, Tensor(a!) out, float eps) -> ()",
     "relu_squared": "(Tensor(a!) x) -> ()",
-    "causal_conv": "(int step, Tensor x, Tensor taps, Tensor bias, Tensor conv_state, Tensor(a!) out) -> ()",
+    "causal_conv": "(int step, Tensor x, Tensor taps, Tensor? bias, Tensor conv_state, Tensor(a!) out, bool silu=False) -> ()",
     "rglru_scan": "(int step, Tensor yx, Tensor u, Tensor gates, Tensor ra_bias, Tensor ri_bias, Tensor decay_base, "
                   "Tensor(a!) state, Tensor(b!) conv_state, Tensor(c!) out, int blocks) -> ()",
     "rglru_step": "(int step, Tensor yx, Tensor gate_w, Tensor taps, Tensor conv_bias, Tensor ra_bias, Tensor ri_bias, "
@@ -189,15 +208,19 @@ def _dtype(t: torch.Tensor) -> int:
 
 
 def _residual_norm(step, x, y, w_post, embed, w_next, h, eps, restart, weight_offset, embed_scale=1.0, top=0,
-                   slot_expert=None, slot_rank=None, slot_weight=None, expert_count=None):
+                   slot_expert=None, slot_rank=None, slot_weight=None, expert_count=None, identity=None, add=None, y_bias=None,
+                   embed_norm=None, w_next2=None, h2=None, y_mul=1.0):
     a = _C.ResidualNormArgs()
     a.x, a.y, a.w_post, a.embed, a.w_next, a.h = x.data_ptr(), _ptr(y), _ptr(w_post), _ptr(embed), _ptr(w_next), _ptr(h)
     a.width, a.restart, a.eps, a.weight_offset = x.shape[1], int(restart), eps, weight_offset
     a.embed_scale, a.top = embed_scale, top
     if top:
-        a.n_experts = expert_count.numel()
+        a.n_experts = expert_count.numel()      # (identity experts are not counted here)
         a.slot_expert, a.slot_rank = slot_expert.data_ptr(), slot_rank.data_ptr()
         a.slot_weight, a.expert_count = slot_weight.data_ptr(), expert_count.data_ptr()
+    a.identity, a.add, a.y_bias, a.embed_norm = _ptr(identity), _ptr(add), _ptr(y_bias), _ptr(embed_norm)
+    a.w_next2, a.h2, a.y_mul = _ptr(w_next2), _ptr(h2), y_mul
+    a.add_stride = add.stride(0) if add is not None else 0
     a.y_stride = y.stride(0) if y is not None else x.shape[1]
     a.vocab = embed.shape[0] if embed is not None else 0
     a.dtype = _dtype(next(t for t in (h, y, embed) if t is not None))
@@ -223,7 +246,8 @@ def _attn_general(pool, pages, layer, step, q, out, dim, vdim, scale):
                                           vdim, scale, _dtype(q), _stream(pages)), "pace_attn_general")
 
 
-def _span_args(a, q, out, slopes, sinks, dim, vdim, scale, span, span_size, entry_begin, entry_end, max_tokens, max_keys):
+def _span_args(a, q, out, slopes, sinks, dim, vdim, scale, span, span_size, entry_begin, entry_end, max_tokens, max_keys, softcap=0.0, out_row=0):
+    a.softcap, a.out_row = softcap, out_row
     a.q, a.out, a.slopes, a.sinks = q.data_ptr(), out.data_ptr(), _ptr(slopes), _ptr(sinks)
     a.n_q_heads, a.dim, a.vdim, a.dtype = q.shape[1], dim, vdim, _dtype(q)
     a.q_elems, a.out_elems = q.shape[2], out.shape[2]
@@ -239,10 +263,11 @@ def _attn_span(pool, pages, layer, step, q, out, *rule):
 
 
 def _attn_span_prefill(pool, pages, layer, step, q, out, slopes, sinks, dim, vdim, scale, span, span_size, entry_begin, entry_end,
-                       max_tokens, max_keys, k=None, k2=None, v=None, key_cu=None, key_pos=None):
+                       max_tokens, max_keys, k=None, k2=None, v=None, key_cu=None, key_pos=None, softcap=0.0, out_row=0):
     """False: the kernel does not take these shapes and nothing was launched."""
     a = _C.AttnSpanPrefillArgs()
-    _span_args(a.a, q, out, slopes, sinks, dim, vdim, scale, span, span_size, entry_begin, entry_end, max_tokens, max_keys)
+    _span_args(a.a, q, out, slopes, sinks, dim, vdim, scale, span, span_size, entry_begin, entry_end, max_tokens, max_keys, softcap,
+               out_row)
     if k is not None:
         a.k, a.k_row, a.k_head, a.k_dim = k.data_ptr(), k.stride(0), k.stride(1), k.shape[2]
         a.v, a.v_row, a.v_head = v.data_ptr(), v.stride(0), v.stride(1)
@@ -284,14 +309,29 @@ def _latent_gather(pool, pages, layer, slot, pos, out):
                                            _stream(pages)), "pace_latent_gather")
 
 
-def _glu(x, out, act):
+def _glu(x, out, act, gated=True):
     with torch.cuda.device(x.device):
-        _C.check(_C.lib.pace_glu(x.data_ptr(), x.stride(0), out.data_ptr(), out.shape[0], out.shape[1], act, _dtype(x),
-                                 _stream(x)), "pace_glu")
+        _C.check(_C.lib.pace_glu(x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), out.shape[0], out.shape[1], act,
+                                 int(gated), _dtype(x), _stream(x)), "pace_glu")
 
 
-def _moe_route(logits, correction, slot_expert, slot_rank, slot_weight, expert_count, expert_list):
+def _soft_cap(x, cap):
+    with torch.cuda.device(x.device):
+        _C.check(_C.lib.pace_soft_cap(x.data_ptr(), x.numel(), cap, _stream(x)), "pace_soft_cap")
+
+
+def _part_norm_gate(o, gate, w, out, part, gate_first, eps):
+    a = _C.PartNormGateArgs()
+    a.o, a.gate, a.w, a.out = o.data_ptr(), gate.data_ptr(), w.data_ptr(), out.data_ptr()
+    a.o_stride, a.gate_stride, a.out_stride = o.stride(0), gate.stride(0), out.stride(0)
+    a.n_tokens, a.n, a.part, a.w_period, a.gate_first, a.dtype, a.eps = *o.shape, part, w.numel(), int(gate_first), _dtype(o), eps
+    with torch.cuda.device(o.device):
+        _C.check(_C.lib.pace_part_norm_gate(C.byref(a), _stream(o)), "pace_part_norm_gate")
+
+
+def _moe_route(logits, correction, slot_expert, slot_rank, slot_weight, expert_count, expert_list, softmax=False, weight_scale=None):
     a = _C.MoeRouteArgs()
+    a.softmax, a.normalise, a.weight_scale = int(softmax), int(weight_scale is not None), weight_scale or 0.0
     a.logits, a.correction, a.slot_expert, a.slot_rank = logits.data_ptr(), _ptr(correction), slot_expert.data_ptr(), slot_rank.data_ptr()
     a.slot_weight, a.expert_count, a.expert_list = slot_weight.data_ptr(), expert_count.data_ptr(), expert_list.data_ptr()
     (a.n_tokens, a.n_experts), a.top = logits.shape, slot_expert.shape[1]
@@ -299,8 +339,9 @@ def _moe_route(logits, correction, slot_expert, slot_rank, slot_weight, expert_c
         _C.check(_C.lib.pace_moe_route(C.byref(a), _stream(logits)), "pace_moe_route")
 
 
-def _moe_experts(x, gate_up, down, hidden, y, scratch, expert_count, expert_list, slot_expert, slot_rank, status, act):
+def _moe_experts(x, gate_up, down, hidden, y, scratch, expert_count, expert_list, slot_expert, slot_rank, status, act, gated=True):
     a = _C.MoeExpertsArgs()
+    a.gated = int(gated)
     a.x, a.gate_up, a.down, a.hidden, a.y = x.data_ptr(), gate_up.data_ptr(), down.data_ptr(), hidden.data_ptr(), y.data_ptr()
     a.expert_count, a.expert_list, a.status = expert_count.data_ptr(), expert_list.data_ptr(), _ptr(status)
     a.scratch, a.slot_expert, a.slot_rank = _ptr(scratch), slot_expert.data_ptr(), slot_rank.data_ptr()
@@ -328,11 +369,87 @@ def _relu_squared(x):
         _C.check(_C.lib.pace_relu_squared(x.data_ptr(), x.numel(), _dtype(x), _stream(x)), "pace_relu_squared")
 
 
-def _causal_conv(step, x, taps, bias, conv_state, out):
+def _causal_conv(step, x, taps, bias, conv_state, out, silu=False):
+    a = _C.CausalConvArgs()
+    a.in_, a.in_stride, a.taps, a.bias = x.data_ptr(), x.stride(0), taps.data_ptr(), _ptr(bias)
+    a.conv_state, a.out, a.out_stride = conv_state.data_ptr(), out.data_ptr(), out.stride(0)
+    (a.n_taps, a.channels), a.ring_rows, a.ring_stride = taps.shape, conv_state.shape[1], conv_state.stride(1)
+    a.silu, a.dtype = int(silu), _dtype(x)
     with torch.cuda.device(out.device):
-        _C.check(_C.lib.pace_causal_conv(_step(step), x.data_ptr(), x.stride(0), taps.data_ptr(), bias.data_ptr(),
-                                         taps.shape[0], conv_state.data_ptr(), out.data_ptr(), out.shape[1], _dtype(x),
-                                         _stream(out)), "pace_causal_conv")
+        _C.check(_C.lib.pace_causal_conv(_step(step), C.byref(a), _stream(out)), "pace_causal_conv")
+
+
+def _conv_store(step, x, ring):
+    with torch.cuda.device(x.device):
+        _C.check(_C.lib.pace_conv_store(_step(step), x.data_ptr(), x.stride(0), ring.data_ptr(), ring.shape[1], ring.stride(1),
+                                        ring.shape[2], _dtype(x), _stream(x)), "pace_conv_store")
+
+
+def _kv_append_conv(pool, pages, layer, step, qkv, taps, ring, q_norm, k_norm, cos, sin, q_out, dim, vdim, eps, v_mul, store_ring):
+    a = _C.AppendConvArgs()
+    a.qkv, a.qkv_stride, a.taps, a.ring = qkv.data_ptr(), qkv.stride(0), taps.data_ptr(), ring.data_ptr()
+    a.q_norm, a.k_norm, a.q_out = q_norm.data_ptr(), k_norm.data_ptr(), q_out.data_ptr()
+    if cos is not None:
+        a.cos_table, a.sin_table, (a.table_rows, a.rot_pairs) = cos.data_ptr(), sin.data_ptr(), cos.shape
+    a.n_q_heads, a.dim, a.vdim, a.n_taps = q_out.shape[1], dim, vdim, taps.shape[0]
+    a.ring_rows, a.ring_stride, a.store_ring, a.dtype = ring.shape[1], ring.stride(1), int(store_ring), _dtype(qkv)
+    a.eps, a.v_mul = eps, v_mul
+    with torch.cuda.device(pages.device):
+        _C.check(_C.lib.pace_kv_append_conv(_pool(pool), layer, _step(step), C.byref(a), _stream(pages)), "pace_kv_append_conv")
+
+
+def _workspace(a, nbytes: int, device) -> Optional[torch.Tensor]:
+    """Scratch of one launch (stream ordered: the allocator hands it out again only behind it)."""
+    if not nbytes:
+        return None
+    ws = torch.empty(nbytes, dtype=torch.uint8, device=device)
+    a.workspace, a.workspace_bytes = ws.data_ptr(), nbytes
+    return ws
+
+
+def _ssd(entry: str):
+    fn = getattr(_C.lib, entry)
+
+    def impl(step, xbc, dt_raw, dt_bias, neg_a, d_skip, state, out, groups, taps=None, conv_bias=None, ring=None):
+        a = _C.SsdArgs()
+        a.xbc, a.xbc_stride, a.dt_raw, a.dt_stride = xbc.data_ptr(), xbc.stride(0), dt_raw.data_ptr(), dt_raw.stride(0)
+        a.dt_bias, a.neg_a, a.d_skip = dt_bias.data_ptr(), neg_a.data_ptr(), d_skip.data_ptr()
+        a.s_state, a.out, a.out_stride = state.data_ptr(), out.data_ptr(), out.stride(0)
+        (_, a.heads, a.state, a.vdim), a.groups, a.dtype = state.shape, groups, _dtype(xbc)
+        if taps is not None:
+            a.taps, a.conv_bias, a.ring, a.n_taps = taps.data_ptr(), _ptr(conv_bias), ring.data_ptr(), taps.shape[0]
+            a.ring_rows, a.ring_stride = ring.shape[1], ring.stride(1)
+        with torch.cuda.device(out.device):
+            st = _C.StepStruct.from_address(step)
+            ws = None
+            if taps is None and a.dtype == _C.DTYPE_BF16:
+                ws = _workspace(a, _C.lib.pace_ssd_workspace_bytes(st.n_entries, st.max_count, a.heads, a.state, a.vdim), out.device)
+            _C.check(fn(_step(step), C.byref(a), _stream(out)), entry)
+            del ws
+    return impl
+
+
+def _delta(entry: str):
+    fn = getattr(_C.lib, entry)
+
+    def impl(step, qkv, a_raw, b_raw, dt_bias, neg_a, state, out, kv_heads, unit_eps, q_scale, taps=None, ring=None):
+        a = _C.DeltaArgs()
+        a.qkv, a.qkv_stride, a.a_raw, a.a_stride = qkv.data_ptr(), qkv.stride(0), a_raw.data_ptr(), a_raw.stride(0)
+        a.b_raw, a.b_stride, a.dt_bias, a.neg_a = b_raw.data_ptr(), b_raw.stride(0), dt_bias.data_ptr(), neg_a.data_ptr()
+        a.s_state, a.out, a.out_stride = state.data_ptr(), out.data_ptr(), out.stride(0)
+        (_, a.heads, a.dim, a.vdim), a.kv_heads, a.dtype = state.shape, kv_heads, _dtype(qkv)
+        a.unit_eps, a.q_scale = unit_eps, q_scale
+        if taps is not None:
+            a.taps, a.ring, a.n_taps, a.ring_rows, a.ring_stride = taps.data_ptr(), ring.data_ptr(), taps.shape[0], ring.shape[1], ring.stride(1)
+        with torch.cuda.device(out.device):
+            st = _C.StepStruct.from_address(step)
+            ws = None
+            if taps is None:
+                ws = _workspace(a, _C.lib.pace_delta_workspace_bytes(st.n_tokens, st.n_entries, a.heads, a.dim, a.vdim, a.dtype),
+                                out.device)
+            _C.check(fn(_step(step), C.byref(a), _stream(out)), entry)
+            del ws
+    return impl
 
 
 def _rglru_args(yx, ra_bias, ri_bias, decay_base, state, conv_state, out, blocks):
@@ -419,7 +536,9 @@ _IMPLS = {"kv_reserve": _kv_reserve, "kv_append": _kv_append, "kv_append_layers"
           "lightning_prefill": _lightning("pace_lightning_prefill"), "lightning_step": _lightning("pace_lightning_step"),
           "step_decode": _step_decode, "attn_span": _attn_span, "attn_span_prefill": _attn_span_prefill,
           "latent_append": _latent_append, "rotate_heads": _rotate_heads, "latent_gather": _latent_gather, "glu": _glu,
-          "moe_route": _moe_route, "moe_experts": _moe_experts}
+          "moe_route": _moe_route, "moe_experts": _moe_experts, "soft_cap": _soft_cap, "part_norm_gate": _part_norm_gate,
+          "kv_append_conv": _kv_append_conv, "conv_store": _conv_store, "ssd_prefill": _ssd("pace_ssd_prefill"),
+          "ssd_step": _ssd("pace_ssd_step"), "delta_prefill": _delta("pace_delta_prefill"), "delta_step": _delta("pace_delta_step")}
 for _n, _f in _IMPLS.items():
     _lib.impl(_n, _f, "CUDA")
     # shape propagation for tracers: nothing is returned, nothing to compute

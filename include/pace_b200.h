@@ -432,7 +432,11 @@ typedef struct pace_step {
  * itself).  w_post == NULL adds y as it is.  Norm weights are fp32 [width] and used as weight_offset + w (1 for
  * "one plus weight" norms).  embed is dtype [vocab][width].
  * With `top` > 0, y holds the rows of a mixture's experts (pace_moe_experts) and the sublayer's output of token t is
- *     sum over k < top of slot_weight[t][k] * y[expert_row(slot_expert[t][k], slot_rank[t][k])]. */
+ *     sum over k < top of slot_weight[t][k] * y[expert_row(slot_expert[t][k], slot_rank[t][k])],
+ * where a slot_expert of n_experts or more names an identity expert: its row is identity[t].
+ * Further terms: `add` (rows of add_stride elements) and y_bias (fp32 [width]) are added to the sublayer's output; with
+ * y_mul != 1 and no w_post the sum is multiplied by it; embed_norm normalises the embedding row (rms(row) * weight, in place of
+ * embed_scale).  h2 takes a second normalisation of the same x', with the weight w_next2. */
 typedef struct {
   float* x;
   const void* y;
@@ -448,6 +452,14 @@ typedef struct {
   const int32_t* slot_rank;     /* [n_tokens][top] */
   const float* slot_weight;     /* [n_tokens][top] */
   const int32_t* expert_count;  /* [n_experts] */
+  const void* identity;         /* dtype [n_tokens][width] */
+  const void* add;
+  int64_t add_stride;
+  const float* y_bias;
+  const float* embed_norm;
+  const float* w_next2;
+  void* h2;
+  float y_mul;
 } pace_residual_norm_args_t;
 int pace_residual_norm(const pace_step_t* step, const pace_residual_norm_args_t* a, void* stream);
 
@@ -474,6 +486,29 @@ typedef struct {
 int pace_kv_append_norm(const pace_kv_pool_t* pool, int32_t layer, const pace_step_t* step,
                         const pace_append_norm_args_t* a, void* stream);
 
+/* Projection output -> attention operands behind short causal convolutions, in one pass: every channel of q, k and v is
+ * convolved over time (taps, ring as pace_causal_conv, without bias), then q and k are normalised per head,
+ *     rms over dim * q_norm[c] (k_norm[c]; fp32 [dim], shared by the heads)
+ * and their pairs (2i, 2i + 1), i < rot_pairs, turned by the angles of the tables (as pace_latent_append); v is multiplied by
+ * v_mul.  Row t of q_out [n_tokens][n_q_heads][row elements] belongs to token t; keys and values go to their pages (reserved).
+ * qkv as pace_kv_append_norm.  store_ring: also stores the tokens' projections in the ring (one token per entry only:
+ * with more, pace_conv_store behind the launch does).  dim, vdim <= 640. */
+typedef struct {
+  const void* qkv;
+  int64_t qkv_stride;
+  const float* taps;        /* fp32 [n_taps][all channels] */
+  float* ring;
+  const float* q_norm;
+  const float* k_norm;
+  const float* cos_table;
+  const float* sin_table;
+  void* q_out;
+  int32_t n_q_heads, dim, vdim, n_taps, ring_rows, ring_stride, rot_pairs, table_rows, store_ring, dtype;
+  float eps, v_mul;
+} pace_append_conv_args_t;
+int pace_kv_append_conv(const pace_kv_pool_t* pool, int32_t layer, const pace_step_t* step, const pace_append_conv_args_t* a,
+                        void* stream);
+
 /* Causal softmax attention over the pool for any row format: q and out are dtype [q_row][n_q_heads][row
  * elements]; scores, weights and sums in fp32.  dim, vdim <= 512.  CUDA cores; the tensor-core kernels
  * (pace_attn_decode / pace_attn_prefill) take the PACE_ROWS_BF16 pools. */
@@ -485,10 +520,11 @@ int pace_attn_general(const pace_kv_pool_t* pool, int32_t layer, const pace_step
  *     PACE_SPAN_ALL     always,
  *     PACE_SPAN_WINDOW  if i - j < span_size,
  *     PACE_SPAN_CHUNK   if i / span_size == j / span_size (integer division, counted from position 0),
- * its score is scale * (q . k) - slopes[h] * (i - j) (slopes NULL: no bias), and exp(sinks[h]) is added to the
- * denominator (sinks NULL: ordinary softmax).  Query head h reads KV head h / (n_q_heads / n_kv_heads).
+ * its score is scale * (q . k), with softcap > 0 replaced by softcap * tanh(score / softcap), minus slopes[h] * (i - j) (slopes
+ * NULL: no bias), and exp(sinks[h]) is added to the denominator (sinks NULL: ordinary softmax).  Query head h reads KV head h / (n_q_heads / n_kv_heads).
  * Row t of q (dtype [n_tokens][n_q_heads][q_elems], dim elements used, zero up to the next multiple of 8) and of out
- * ([n_tokens][n_q_heads][out_elems], vdim elements written) belongs to token t.  The pool holds the step's own rows already;
+ * ([n_tokens][n_q_heads][out_elems], vdim elements written; tokens out_row elements apart where that is not 0) belongs to
+ * token t.  The pool holds the step's own rows already;
  * lengths come from the step.  PACE_ROWS_SHARED pools: the value is the first vdim elements of the key row.
  * Scores, weights and sums are fp32 (with bf16 rows the weights enter the second product as two bf16 terms).
  * max_tokens / max_keys: upper bounds, over the entries, of their tokens and of their last position + 1.
@@ -506,6 +542,8 @@ typedef struct {
   int32_t entry_begin, entry_end, max_tokens, max_keys;
   int32_t span, span_size;
   float scale;
+  float softcap;         /* 0: none */
+  int64_t out_row;       /* elements between the tokens of out; 0: n_q_heads * out_elems */
 } pace_attn_span_args_t;
 int pace_attn_span(const pace_kv_pool_t* pool, int32_t layer, const pace_step_t* step, const pace_attn_span_args_t* a,
                    void* stream);
@@ -567,15 +605,20 @@ int pace_latent_gather(const pace_kv_pool_t* pool, int32_t layer, const int32_t*
                        void* out, void* stream);
 
 /* ---- gated feed-forwards and mixtures of experts --------------------------------------------------------------------
- * pace_glu: out[t][i] = act(x[t][i]) * x[t][n + i], x rows of 2 n elements. */
+ * pace_glu: out[t][i] = act(x[t][i]) * x[t][n + i], x rows of 2 n elements; without `gated` act(x[t][i]), rows of n. */
 #define PACE_ACT_SILU 0
 #define PACE_ACT_GELU_TANH 1
-int pace_glu(const void* x, int64_t x_stride, void* out, int32_t n_tokens, int32_t n, int32_t act, int32_t dtype,
-             void* stream);
+#define PACE_ACT_GELU_ERF 2
+#define PACE_ACT_NONE 3   /* experts' second product */
+int pace_glu(const void* x, int64_t x_stride, void* out, int64_t out_stride, int32_t n_tokens, int32_t n, int32_t act,
+             int32_t gated, int32_t dtype, void* stream);
+/* x = cap * tanh(x / cap) in place, n fp32 elements. */
+int pace_soft_cap(float* x, int64_t n, float cap, void* stream);
 
-/* Router: scores = sigmoid(logits) (logits fp32 [n_tokens][n_experts]); the `top` experts with the largest scores +
- * correction (fp32 [n_experts] or NULL; ties go to the lower index) are chosen, their weights are the scores without
- * it.  slot_expert / slot_weight [n_tokens][top]; expert_count [n_experts] and slot_rank [n_tokens][top] number the tokens
+/* Router: scores = sigmoid(logits) or softmax(logits) (logits fp32 [n_tokens][n_experts]); the `top` experts with the
+ * largest scores + correction (fp32 [n_experts] or NULL; ties go to the lower index) are chosen, their weights are the scores
+ * without it; `normalise` divides them by their sum + 1e-20 and multiplies them by weight_scale.  Identity experts are the last
+ * of n_experts here; pace_moe_experts gets the number of those in front.  slot_expert / slot_weight [n_tokens][top]; expert_count [n_experts] and slot_rank [n_tokens][top] number the tokens
  * of an expert, expert_list [n_experts][n_tokens] lists them.  top <= 64, n_experts <= 1024. */
 typedef struct {
   const float* logits;
@@ -586,12 +629,14 @@ typedef struct {
   int32_t* expert_count;
   int32_t* expert_list;
   int32_t n_tokens, n_experts, top;
+  int32_t softmax, normalise;
+  float weight_scale;
 } pace_moe_route_args_t;
 int pace_moe_route(const pace_moe_route_args_t* a, void* stream);
 
 /* The chosen experts' feed-forwards: for every (token, expert) pair of the router
- *     hidden = act(gate x) * (up x),  y = down hidden
- * x dtype [n_tokens][width], gate_up dtype [n_experts][2 ff][width] (gate rows first), down dtype [n_experts][width][ff].
+ *     hidden = act(gate x) * (up x),  y = down hidden           (without `gated`: hidden = act(up x))
+ * x dtype [n_tokens][width], gate_up dtype [n_experts][2 ff][width] (gate rows first; ff rows without `gated`), down dtype [n_experts][width][ff].
  * hidden [n_tokens * top][ff] and y [n_tokens * top][width] are written by expert: expert e's token of rank r is row
  *     expert_row(e, r) = expert_count[0] + .. + expert_count[e - 1] + r.
  * bf16 with width and ff multiples of 8: grouped products on the tcgen05 tensor cores, weights as the 128-row operand.
@@ -610,7 +655,7 @@ typedef struct {
   const int32_t* slot_expert;   /* with scratch: the router's */
   const int32_t* slot_rank;
   int32_t* status;
-  int32_t n_tokens, n_experts, top, width, ff, act, dtype;
+  int32_t n_tokens, n_experts, top, width, ff, act, dtype, gated;
 } pace_moe_experts_args_t;
 int pace_moe_experts(const pace_moe_experts_args_t* a, void* stream);
 
@@ -621,15 +666,41 @@ int pace_gate_heads(const pace_step_t* step, const void* attn, const void* gate,
 /* out[t] = rms(o[t]) * w * sigmoid(gate[t]) over n elements (w fp32). */
 int pace_norm_gate(const void* o, const float* w, const void* gate, int64_t gate_stride, void* out, int32_t n_tokens,
                    int32_t n, float eps, int32_t dtype, void* stream);
+/* Norms over equal parts of a row, with a gate in front (silu) or behind (sigmoid):
+ *     gate_first:  out = rms(o * silu(gate)) * w,      otherwise:  out = rms(o) * w * sigmoid(gate)
+ * rms over every `part` elements (n a multiple of part), weight w[c % w_period] (fp32). */
+typedef struct {
+  const void* o;
+  const void* gate;
+  const float* w;
+  void* out;
+  int64_t o_stride, gate_stride, out_stride;
+  int32_t n_tokens, n, part, w_period, gate_first, dtype;
+  float eps;
+} pace_part_norm_gate_args_t;
+int pace_part_norm_gate(const pace_part_norm_gate_args_t* a, void* stream);
 /* x = relu(x)^2 in place, n elements. */
 int pace_relu_squared(void* x, int64_t n, int32_t dtype, void* stream);
 
-/* Causal depthwise convolution: out[t][c] = bias[c] + sum_j taps[j][c] in[c](pos - (n_taps - 1) + j), zeros
- * in front of the sequence.  conv_state fp32 [slots][n_taps][channels] holds each slot's newest inputs in row
- * position % n_taps (a row is overwritten only when no later token needs it).  This entry point reads it;
- * the recurrence behind it stores the new inputs. */
-int pace_causal_conv(const pace_step_t* step, const void* in, int64_t in_stride, const float* taps, const float* bias,
-                     int32_t n_taps, const float* conv_state, void* out, int32_t channels, int32_t dtype, void* stream);
+/* Causal depthwise convolution: out[t][c] = act(bias[c] + sum_j taps[j][c] in[c](pos - (n_taps - 1) + j)), zeros
+ * in front of the sequence; act is silu or nothing, bias may be NULL.  conv_state fp32 [slots][ring_rows][ring_stride] holds
+ * each slot's newest inputs in row position % ring_rows (ring_rows >= n_taps - 1, and n_taps where the launch that reads a ring
+ * or one beside it writes the current token's row).  This entry point reads it; the recurrence behind it or
+ * pace_conv_store stores the new inputs.  `conv_state` points at the first of `channels` channels of a row. */
+typedef struct {
+  const void* in;
+  int64_t in_stride;
+  const float* taps;        /* fp32 [n_taps][channels] */
+  const float* bias;
+  const float* conv_state;
+  void* out;
+  int64_t out_stride;
+  int32_t n_taps, channels, ring_rows, ring_stride, silu, dtype;
+} pace_causal_conv_args_t;
+int pace_causal_conv(const pace_step_t* step, const pace_causal_conv_args_t* a, void* stream);
+/* The newest inputs (the last ring_rows tokens at most) of every entry into its ring. */
+int pace_conv_store(const pace_step_t* step, const void* in, int64_t in_stride, float* ring, int32_t ring_rows,
+                    int32_t ring_stride, int32_t channels, int32_t dtype, void* stream);
 
 /* Real-gated linear recurrence (RG-LRU) with its branch product:
  *     r = sigmoid(gates_r + ra_bias), i = sigmoid(gates_i + ri_bias), log a = decay_base * r
@@ -680,6 +751,69 @@ typedef struct {
 uint64_t pace_lightning_workspace_bytes(int32_t n_entries, int32_t max_count, int32_t heads, int32_t dim, int32_t vdim);
 int pace_lightning_prefill(const pace_step_t* step, const pace_lightning_args_t* a, void* stream);
 int pace_lightning_step(const pace_step_t* step, const pace_lightning_args_t* a, void* stream);
+
+/* State-space recurrence with a decay per head and token (Mamba-2):
+ *     dt = softplus(dt_raw + dt_bias),  S_t = exp(neg_a dt) S_(t-1) + dt b_t x_t^T,  y_t = S_t^T c_t + d_skip x_t
+ * per head (S state x vdim; head h reads b and c of group h / (heads / groups)); neg_a = -exp(A_log), all fp32 [heads].
+ * xbc dtype [n_tokens][xbc_stride] = x (heads x vdim) | b (groups x state) | c (groups x state); dt_raw dtype
+ * [n_tokens][dt_stride].  s_state fp32 [slots][heads][state][vdim].  out dtype [n_tokens][out_stride].
+ * pace_ssd_prefill: xbc behind the convolution and silu (any counts per entry).  bf16 with state <= 128 and sizes that
+ * are multiples of 8: chunks on the tensor cores; otherwise token by token.
+ * pace_ssd_step: one token per entry; xbc in front of the convolution (taps, conv_bias, ring as pace_causal_conv; the launch
+ * stores the new rows; ring_rows >= n_taps).  state <= 512. */
+typedef struct {
+  const void* xbc;
+  int64_t xbc_stride;
+  const void* dt_raw;
+  int64_t dt_stride;
+  const float* dt_bias;
+  const float* neg_a;
+  const float* d_skip;
+  float* s_state;
+  void* out;
+  int64_t out_stride;
+  const float* taps;        /* step only */
+  const float* conv_bias;   /* step only, may be NULL */
+  float* ring;              /* step only */
+  float* workspace;         /* prefill: pace_ssd_workspace_bytes() of scratch, any content */
+  uint64_t workspace_bytes;
+  int32_t heads, groups, state, vdim, n_taps, ring_rows, ring_stride, dtype;
+} pace_ssd_args_t;
+uint64_t pace_ssd_workspace_bytes(int32_t n_entries, int32_t max_count, int32_t heads, int32_t state, int32_t vdim);
+int pace_ssd_prefill(const pace_step_t* step, const pace_ssd_args_t* a, void* stream);
+int pace_ssd_step(const pace_step_t* step, const pace_ssd_args_t* a, void* stream);
+
+/* Gated delta rule with a decay per head and key channel:
+ *     g_t = exp(neg_a softplus(a_raw + dt_bias)),  beta_t = sigmoid(b_raw)
+ *     S <- g_t S (rows);  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
+ * per head (S dim x vdim); q and k are made unit vectors per head, x / sqrt(sum(x^2) + unit_eps), q times q_scale; head h uses
+ * q / k head h / (heads / kv_heads).  qkv dtype [n_tokens][qkv_stride] = q (kv_heads x dim) | k (kv_heads x dim) |
+ * v (heads x vdim); a_raw dtype rows of heads x dim, b_raw dtype rows of heads; neg_a = -exp(A_log) fp32 [heads], dt_bias fp32
+ * [heads x dim].  s_state fp32 [slots][heads][dim][vdim].  out dtype [n_tokens][out_stride].
+ * pace_delta_prefill: qkv behind the convolution and silu.  pace_delta_step: one token per entry, qkv in front of
+ * them (taps, ring as pace_ssd_step, no bias).  dim <= 512. */
+typedef struct {
+  const void* qkv;
+  int64_t qkv_stride;
+  const void* a_raw;
+  int64_t a_stride;
+  const void* b_raw;
+  int64_t b_stride;
+  const float* dt_bias;
+  const float* neg_a;
+  float* s_state;
+  void* out;
+  int64_t out_stride;
+  const float* taps;        /* step only */
+  float* ring;              /* step only */
+  void* workspace;          /* prefill: pace_delta_workspace_bytes() of scratch, any content */
+  uint64_t workspace_bytes;
+  int32_t heads, kv_heads, dim, vdim, n_taps, ring_rows, ring_stride, dtype;
+  float unit_eps, q_scale;
+} pace_delta_args_t;
+uint64_t pace_delta_workspace_bytes(int32_t n_tokens, int32_t n_entries, int32_t heads, int32_t dim, int32_t vdim, int32_t dtype);
+int pace_delta_prefill(const pace_step_t* step, const pace_delta_args_t* a, void* stream);
+int pace_delta_step(const pace_step_t* step, const pace_delta_args_t* a, void* stream);
 
 /* Step arrays of a decode step whose tokens and positions the device holds (one token per entry):
  * token[i] = next_token[i], tok_pos[i] = start[i] = position[i]. */
