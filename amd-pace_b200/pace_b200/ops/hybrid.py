@@ -290,7 +290,8 @@ def part_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, pa
 
 def soft_cap_(x: torch.Tensor, cap: float) -> torch.Tensor:
     """cap * tanh(x / cap) in place (fp32)."""
-    _OPS.soft_cap(x, cap)
+    if x.numel():
+        _OPS.soft_cap(x, cap)
     return x
 
 
