@@ -43,7 +43,7 @@ class StateSpec:
 
 @dataclass(frozen=True)
 class JointSpec:
-    """A layer run that remembers several things (mixers side by side): its cache is the tuple of theirs."""
+    """A layer run that remembers several things (mixers side by side): its cache is the ``JointCache`` of theirs."""
     parts: Tuple[Union[KVSpec, LatentSpec, StateSpec], ...]
 
 
@@ -80,6 +80,18 @@ class StateCache:
     @property
     def seq_len(self) -> int:
         return max(self.manager.seq_lens, default=0)
+
+
+class JointCache(tuple):
+    """The caches of a ``JointSpec``; its parts have the same lengths."""
+
+    @property
+    def seq_lens(self) -> List[int]:
+        return self[0].seq_lens
+
+    @property
+    def seq_len(self) -> int:
+        return self[0].seq_len
 
 
 class PoolSet:
@@ -156,7 +168,7 @@ class HybridCacheManager:
                 self.caches[i] = StateCache(self, s, batch, self.device)
                 self.states.append(self.caches[i])
         parts = iter(self.caches)
-        self.caches = [tuple(next(parts) for _ in range(n)) if n else next(parts) for n in joint]
+        self.caches = [JointCache(next(parts) for _ in range(n)) if n else next(parts) for n in joint]
         self.pool = PoolSet([g.pool for g in self.groups], n_pages)
         # rows map to slots 1:1: every pool is this manager's own
         self.slots = list(range(batch))
