@@ -1355,6 +1355,216 @@ def run_gekupel(args):
         print(json.dumps(line), flush=True)
 
 
+# ---------------------------------------------------------------------------------------------------
+# Lesosun (capped attention beside a state-space recurrence, delta rule, mixtures with identity experts)
+# beside the decoders it resembles: Garupel (recurrences) and Gekupel (mixtures of experts)
+# ---------------------------------------------------------------------------------------------------
+LESOSUN_SIZES = {
+    "w2048": dict(width=2048, ff=8192, heads=16, kv_heads=4, dim=128, ssd_heads=32, groups=4, state=128, ssd_vdim=64, delta_heads=16,
+                  rank=128, experts=64, identity=8, top=8, expert_ff=1024),
+    "w4096": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, ssd_heads=64, groups=8, state=128, ssd_vdim=64, delta_heads=32,
+                  rank=128, experts=64, identity=8, top=8, expert_ff=1792),
+}
+
+
+def lesosun_model(size: str, dev):
+    from pace_b200.llm.registry import build_model
+    z = LESOSUN_SIZES[size]
+    left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "conv": 4, "scale": z["dim"] ** -0.5,
+            "softcap": 30.0, "rot": {"dims": 64, "base": 1e6}}
+    right = {"heads": z["ssd_heads"], "groups": z["groups"], "state": z["state"], "vdim": z["ssd_vdim"], "conv": 4, "norm_groups": z["groups"]}
+    par = {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.7}
+    delta = {"heads": z["delta_heads"], "kv_heads": z["delta_heads"], "dim": z["dim"], "vdim": z["dim"], "conv": 4}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "shared": {"ff": z["expert_ff"]},
+           "router": {"experts": z["experts"], "identity": z["identity"], "top": z["top"], "scale": 1.0}}
+    layers = [{"type": "parallel", "mixer": par, "mlp": dense}, {"type": "parallel", "mixer": par, "mlp": moe},
+              {"type": "channel_delta", "mixer": delta, "mlp": dense}, {"type": "channel_delta", "mixer": delta, "mlp": moe}]
+    cfg = {"architecture": "Lesosun", "vocab": HYBRID_VOCAB, "width": z["width"], "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+           "logit_softcap": 30.0, "layers": layers * (HYBRID_LAYERS // 4)}
+    return build_model(cfg, torch.bfloat16, dev).random_init_(5)
+
+
+@torch.inference_mode()
+def lesosun_kernels(size: str, dev):
+    """Each kernel of the Lesosun decoder alone, against its own roofline, and the like kernels of Garupel and Gekupel ("like.*")
+    on operands of the same size; phases as in ``hybrid_kernels``."""
+    from pace_b200 import _C
+    from pace_b200.llm.hybrid_cache import HybridCacheManager, JointSpec, KVSpec, StateSpec
+    from pace_b200.ops import RotaryEmbedding, hybrid
+    z = LESOSUN_SIZES[size]
+    W, H, G, D, FF = z["width"], z["heads"], z["kv_heads"], z["dim"], z["ff"]
+    SH, SG, SN, SP, DH = z["ssd_heads"], z["groups"], z["state"], z["ssd_vdim"], z["delta_heads"]
+    X, ID, top, XF, ops = z["experts"], z["identity"], z["top"], z["expert_ff"], torch.ops.pace_b200
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(
+        os.path.join(ROOT, "MEASURED_PEAKS.json")) else {"hbm_gbs": FALLBACK_HBM_GBS, "bf16_tflops_sustained": 1400.0}
+    bw, fl = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops_sustained"] * 1e12
+    g = torch.Generator(device=dev).manual_seed(2)
+
+    def rnd(*shape, dtype=torch.bfloat16):
+        return torch.randn(*shape, device=dev, generator=g, dtype=torch.float32).to(dtype)
+
+    out = {}
+    cos, sin = RotaryEmbedding({"rope_type": "precise"}, 64, 8192, 1e6, is_neox_style=False).device_tables(dev)
+    for phase, E, n, past in (("prefill", 1, 4096, 0), ("prefill_batch", 8, 512, 0), ("decode", 32, 1, 512)):
+        T, dec = E * n, n == 1
+        N = 8 if dec else 3                    # copies of every operand
+        nq, nk, nd, inner = H * D, G * D, DH * D, SH * SP
+        cl, cr = nq + 2 * nk, inner + 2 * SG * SN
+        specs = [JointSpec((KVSpec(G, D, D), StateSpec((("S", (SH, SN, SP)), ("conv", (4, cl + cr))))))] * N + \
+                [StateSpec((("S", (DH, D, D)), ("conv", (4, 3 * nd))))] * N
+        cache = HybridCacheManager(specs, E, E * (past + n + 64), past + n + 64, torch.bfloat16, dev)
+        for s_ in cache.states:
+            for name, t in s_.arrays.items():
+                t.normal_(0.0, 0.1, generator=g)
+        if past:
+            cache.begin_step(cache.step([past] * E, torch.zeros(E * past, dtype=torch.long), 1))
+        step = cache.step([n] * E, torch.zeros(T, dtype=torch.long), 1)
+        cache.begin_step(step)
+        vec = lambda k: rnd(k, dtype=torch.float32)                          # noqa: E731
+        x, y = [rnd(T, W, dtype=torch.float32) for _ in range(N)], [rnd(T, W) for _ in range(N)]
+        wp, wn = vec(W), vec(W)
+        proj = [rnd(T, cl + cr + inner + SH) for _ in range(N)]
+        dproj = [rnd(T, 3 * nd + DH + 2 * z["rank"]) for _ in range(N)]
+        dup = [rnd(T, 2 * nd) for _ in range(N)]
+        ltaps, rtaps, dtaps = rnd(4, cl, dtype=torch.float32) * 0.5, rnd(4, cr, dtype=torch.float32) * 0.5, rnd(4, 3 * nd, dtype=torch.float32) * 0.5
+        cb, dtb, na, sk = vec(cr), vec(SH) - 4.0, -vec(SH).abs() - 0.1, vec(SH)
+        ddb, dna = vec(nd) - 4.0, -vec(DH).abs() - 0.1
+        qn, kn = vec(D), vec(D)
+        qb = [torch.empty(T, H, D, dtype=torch.bfloat16, device=dev) for _ in range(N)]
+        rows = {}
+
+        def add(name, launches, nbytes, nflops=0.0):
+            us = graph_us(launches)
+            roof = max(nbytes / bw, nflops / fl) * 1e6
+            rows[name] = {"us": us, "roofline_us": roof, "frac": roof / us, "bound": "hbm" if nbytes / bw >= nflops / fl else "tensor"}
+
+        pool = cache[0][0].pool
+        ring = lambda i, lo, hi: cache[i][1]["conv"][:, :, lo:hi]            # noqa: E731
+        rg = lambda c: E * c * 4 * (4 if dec else 0)                         # noqa: E731  (decode: three ring rows read, one written)
+        add("residual_norm (two norms)", [lambda i=i: hybrid.residual_norm(step, x[i], y[i], bias=wp, y_mul=0.5, w_next=wp, w_next2=wn,
+                                                                           eps=1e-5, weight_offset=1.0) for i in range(N)],
+            T * W * (4 + 4 + 2 + 2 + 2))
+        add("like.residual_norm", [lambda i=i: hybrid.residual_norm(step, x[i], y[i], wp, w_next=wn, eps=1e-5) for i in range(N)],
+            T * W * (4 + 4 + 2 + 2))
+        add("append_conv", [lambda i=i: ops.kv_append_conv(pool.handle, pool.pages, i, step.handle, proj[i], ltaps, ring(i, 0, cl), qn, kn,
+                                                           cos, sin, qb[i], D, D, 1e-5, 0.7, dec) for i in range(N)], T * cl * 4 + rg(cl))
+        add("like.append_heads", [lambda i=i: ops.kv_append_norm(pool.handle, pool.pages, i, step.handle, proj[i], None, None, qb[i], D, D,
+                                                                 1e-5, 1.0, 0.0, 1.0, True) for i in range(N)], T * cl * 4)
+        pairs = E * sum(t + 1 for t in range(past, past + n))
+        ao = torch.empty(T, H, D, dtype=torch.bfloat16, device=dev)
+        slopes = torch.rand(H, device=dev) * 0.01
+
+        def attention(i, slopes, cap):
+            rule = (slopes, None, D, D, D ** -0.5, _C.SPAN_ALL, 0, 0, E, n, past + n)
+            if dec:
+                ops.attn_span(pool.handle, pool.pages, i, step.handle, qb[i], ao, *rule, cap)
+            else:
+                assert ops.attn_span_prefill(pool.handle, pool.pages, i, step.handle, qb[i], ao, *rule, None, None, None, None, None, cap)
+        kv_read = E * (past + n) * nk * 4 + T * nq * 4
+        add("attention (capped)", [lambda i=i: attention(i, None, 30.0) for i in range(N)], kv_read, 4.0 * nq * pairs)
+        add("like.attention (bias)", [lambda i=i: attention(i, slopes, 0.0) for i in range(N)], kv_read, 4.0 * nq * pairs)
+        # recurrences: operands once, the state read and written; flops of the chunked form
+        def ssd(i):
+            return hybrid.ssd(step, proj[i][:, cl: cl + cr], proj[i][:, cl + cr + inner: cl + cr + inner + SH], rtaps, cb, dtb, na, sk, SG,
+                              cache[i][1]["S"], ring(i, cl, cl + cr))
+        ssd_bytes = T * (cr + SH + inner) * 2 + E * SH * SN * SP * 8
+        add("ssd" if dec else "ssd with convolution", [lambda i=i: ssd(i) for i in range(N)], ssd_bytes + (rg(cr) if dec else T * cr * 4),
+            0.0 if dec else T * SH * (4 * SN * SP + 2 * 64.0 * (SN + SP)))
+
+        def delta(i):
+            return hybrid.delta_rule(step, dproj[i], dup[i][:, :nd], dproj[i][:, 3 * nd: 3 * nd + DH], dtaps, ddb, dna, DH,
+                                     cache[N + i]["S"], cache[N + i]["conv"], 1e-6, D ** -0.5)
+        delta_bytes = T * (3 * nd + nd + DH + nd) * 2 + E * DH * D * D * 8
+        add("delta" if dec else "delta with convolution", [lambda i=i: delta(i) for i in range(N)],
+            delta_bytes + (rg(3 * nd) if dec else T * 3 * nd * 4), 0.0 if dec else T * DH * (6.0 * D * D + 2 * 64.0 * 3 * D))
+        lq, decay = dproj, torch.linspace(0.9, 0.999, DH, device=dev)
+        add("like.lightning", [lambda i=i: hybrid.lightning(step, lq[i], decay, cache[N + i]["S"]) for i in range(N)],
+            T * nd * 2 * 4 + E * DH * D * D * 8, 0.0 if dec else T * DH * (4 * D * D + 4 * D * 64.0))
+        if not dec:
+            u = [torch.empty(T, max(cr, 3 * nd), dtype=torch.bfloat16, device=dev) for _ in range(N)]
+            add("convolution + silu", [lambda i=i: ops.causal_conv(step.handle, dproj[i], dtaps, None, cache[N + i]["conv"], u[i][:, :3 * nd], True)
+                                       for i in range(N)], T * 3 * nd * 4)
+            add("like.convolution", [lambda i=i: ops.causal_conv(step.handle, dproj[i], dtaps, ddb.repeat(3), cache[N + i]["conv"],
+                                                                 u[i][:, :3 * nd]) for i in range(N)], T * 3 * nd * 4)
+            so, do = torch.empty(T, inner, dtype=torch.bfloat16, device=dev), torch.empty(T, nd, dtype=torch.bfloat16, device=dev)
+            add("ssd (recurrence)", [lambda i=i: ops.ssd_prefill(step.handle, u[i][:, :cr], proj[i][:, -SH:], dtb, na, sk, cache[i][1]["S"], so, SG)
+                                     for i in range(N)], ssd_bytes, T * SH * (4 * SN * SP + 2 * 64.0 * (SN + SP)))
+            add("delta (recurrence)", [lambda i=i: ops.delta_prefill(step.handle, u[i][:, :3 * nd], dup[i][:, :nd], dproj[i][:, 3 * nd: 3 * nd + DH],
+                                                                     ddb, dna, cache[N + i]["S"], do, DH, 1e-6, D ** -0.5) for i in range(N)],
+                delta_bytes, T * DH * (6.0 * D * D + 2 * 64.0 * 3 * D))
+            add("conv_store", [lambda i=i: hybrid.conv_store(step, dproj[i], cache[N + i]["conv"]) for i in range(N)], E * 4 * 3 * nd * 6)
+        so = [rnd(T, inner) for _ in range(N)]
+        add("gate + norm (parts)", [lambda i=i: hybrid.part_norm_gate(so[i], wp.repeat(2)[:inner], proj[i][:, cl + cr: cl + cr + inner], inner // SG, 1e-5,
+                                                                      gate_first=True) for i in range(N)], T * inner * 6)
+        add("norm + gate (heads)", [lambda i=i: hybrid.part_norm_gate(dup[i][:, :nd], qn, dup[i][:, nd:], D, 1e-5, out=so[i][:, :nd] if inner >= nd else None)
+                                    for i in range(N)], T * nd * 6)
+        add("like.norm_gate", [lambda i=i: hybrid.norm_gate(so[i], wp.repeat(2)[:inner], proj[i][:, cl + cr: cl + cr + inner], 1e-5) for i in range(N)],
+            T * inner * 6)
+        # feed-forwards
+        gu = [rnd(T, 2 * FF) for _ in range(N)]
+        add("glu", [lambda i=i: hybrid.glu(gu[i], _C.ACT_SILU) for i in range(N)], T * FF * 6)
+        add("gelu (shared expert)", [lambda i=i: hybrid.activate(gu[i][:, :XF], _C.ACT_GELU_ERF, so[i][:, :XF]) for i in range(N)], T * XF * 4)
+        M = 2                                   # sets of experts (each far beyond L2)
+        router, corr = rnd(X + ID, W) * W ** -0.5, vec(X + ID) * 0.01
+        logits = [hybrid.linear_f32(y[i], router) for i in range(N)]
+        routed = [hybrid.moe_route(y[i], router, corr, top, True, 1.0, ID) for i in range(N)]
+        counts = [torch.empty(X + ID, dtype=torch.int32, device=dev) for _ in range(N)]
+        plain = [hybrid.moe_route(y[i], router[:X].contiguous(), None, top) for i in range(N)]
+        wu, wg, wd = [rnd(X, XF, W) * 0.02 for _ in range(M)], [rnd(X, 2 * XF, W) * 0.02 for _ in range(M)], [rnd(X, W, XF) * 0.02 for _ in range(M)]
+        add("moe_route", [lambda i=i: ops.moe_route(logits[i], corr, routed[i].slot_expert, routed[i].slot_rank, routed[i].slot_weight,
+                                                    counts[i], routed[i].lists, True, 1.0) for i in range(N)], T * (X + ID) * 4 + T * top * 16)
+        plogits = [t[:, :X].contiguous() for t in logits]
+        add("like.moe_route", [lambda i=i: ops.moe_route(plogits[i], None, plain[i].slot_expert, plain[i].slot_rank, plain[i].slot_weight,
+                                                         plain[i].count, plain[i].lists) for i in range(N)], T * X * 4 + T * top * 16)
+        used, slots = int((routed[0].count > 0).sum()), int(routed[0].count.sum())
+        add("moe_experts (ungated)", [lambda i=i: hybrid.moe_experts(y[i % N], routed[i % N], wu[i % M], wd[i % M], _C.ACT_GELU_ERF, gated=False)
+                                      for i in range(2 * M)],
+            used * 2 * XF * W * 2 + T * W * 2 + slots * (XF * 4 + W * 2), 4.0 * slots * XF * W)
+        used = int((plain[0].count > 0).sum())
+        add("like.moe_experts (gated)", [lambda i=i: hybrid.moe_experts(y[i % N], plain[i % N], wg[i % M], wd[i % M], _C.ACT_SILU)
+                                         for i in range(2 * M)],
+            used * 3 * XF * W * 2 + T * W * 2 + T * top * (XF * 4 + W * 2), 6.0 * T * top * XF * W)
+        for i in range(N):
+            hybrid.moe_experts(y[i], routed[i], wu[i % M], wd[i % M], _C.ACT_GELU_ERF, gated=False)
+            hybrid.moe_experts(y[i], plain[i], wg[i % M], wd[i % M], _C.ACT_SILU)
+        add("residual_norm (two norms, experts' sum)", [lambda i=i: hybrid.residual_norm(
+            step, x[i], y[i], bias=wp, routed=routed[i], y_mul=0.5, w_next=wp, w_next2=wn, eps=1e-5, weight_offset=1.0) for i in range(N)],
+            T * W * (4 + 4 + 2 + 2 + 2) + T * top * W * 2)
+        add("like.residual_norm (experts' sum)", [lambda i=i: hybrid.residual_norm(step, x[i], w_post=wp, plain=True, eps=1e-5, routed=plain[i])
+                                                  for i in range(N)], T * W * (4 + 4 + 2) + T * top * W * 2)
+        if dec:
+            lg = [rnd(T, HYBRID_VOCAB, dtype=torch.float32) for _ in range(N)]
+            add("soft_cap (logits)", [lambda i=i: hybrid.soft_cap_(lg[i], 30.0) for i in range(N)], T * HYBRID_VOCAB * 8)
+        cache.pool.check_status()
+        out[phase] = rows
+        del cache, wu, wg, wd
+        torch.cuda.empty_cache()
+    return out
+
+
+def run_lesosun(args):
+    """Side measurement: prefill and decode throughput of the Lesosun decoder beside Garupel and Gekupel at equal width, heads,
+    layer count and feed-forward sizes (random weights), and every kernel of the first against its roofline.  Prints one JSON line
+    per size."""
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    for size, z in LESOSUN_SIZES.items():
+        sampler = ClockSampler(0)
+        sampler.start()
+        line = {"workload": "lesosun", "size": size, **z, "layers": HYBRID_LAYERS, "params": {}}
+        for name, make in (("lesosun", lambda: lesosun_model(size, dev)), ("garupel", lambda: hybrid_models(size, dev)[0]),
+                           ("gekupel", lambda: gekupel_model(size, dev))):
+            model = make()
+            line["params"][name] = sum(p.numel() for p in model.parameters())
+            line[name] = hybrid_throughput(model, dev)
+            del model
+            torch.cuda.empty_cache()
+        line["kernels"] = lesosun_kernels(size, dev)
+        line["clocks"] = sampler.stop()
+        print(json.dumps(line), flush=True)
+
+
 def main():
     # stdout carries the JSON line and nothing else: whatever native libraries print to file descriptor 1
     # (NCCL's version banner on some ranks) goes to stderr, Python's own prints keep the real stdout
@@ -1373,7 +1583,7 @@ def main():
     ap.add_argument("--layers", type=int, default=CFG["n_layers"],
                     help="profiling aid: fewer layers = less device memory; the bench line is only valid at 32")
     ap.add_argument("--workload", default="decode", choices=["decode", "verify", "prefill", "rope_append", "device_loop", "serving", "linear",
-                                                                 "hybrid", "gekupel"],
+                                                                 "hybrid", "gekupel", "lesosun"],
                     help="decode = the bench line; verify / prefill = side measurements of the multi-token kernels")
     ap.add_argument("--past", type=int, default=3584, help="prefill side measurement: tokens cached before the chunk")
     ap.add_argument("--head-dim", type=int, default=128, choices=[64, 128])
@@ -1388,10 +1598,10 @@ def main():
         return
     global RANK_CORES
     RANK_CORES = pin_rank_to_cores(local_rank, world)
-    if args.workload in ("rope_append", "device_loop", "serving", "linear", "hybrid", "gekupel"):
+    if args.workload in ("rope_append", "device_loop", "serving", "linear", "hybrid", "gekupel", "lesosun"):
         if rank == 0:
             {"rope_append": run_rope, "device_loop": run_device_loop, "serving": run_serving,
-             "linear": run_linear, "hybrid": run_hybrid, "gekupel": run_gekupel}[args.workload](args)
+             "linear": run_linear, "hybrid": run_hybrid, "gekupel": run_gekupel, "lesosun": run_lesosun}[args.workload](args)
         return
     if args.workload != "decode":
         if rank == 0:
