@@ -1,6 +1,632 @@
+// Gated delta rule with a decay per key channel over many tokens, in chunks of 64 on the tensor cores.
+//
+// With G_i the sum of the chunk's log decays up to token i (a vector over the key channels), x^(G) for the elementwise product with
+// e^G, and S the state in front of the chunk, the corrections u and the outputs of a chunk are
+//     A_ij = k_i . (k_j)^(G_i - G_j)  (j < i),   P_ij = q_i . (k_j)^(G_i - G_j)  (j <= i),   T = (1 + diag(beta) A)^-1 diag(beta)
+//     U = T V - (T K^(G)) S,     O = Q^(G) S + P U,     S' = S^(G_n) + (K^(G_n - G))^T U
+// Nothing but S connects the chunks, so a first launch makes everything else side by side, a block per (chunk, head, entry):
+// W = T K^(G), T V, Q^(G), K^(G_n - G) and P; a second one walks the chunks, a block per (entry, head, 16 or 32 value columns)
+// with its part of S in fp32 accumulators.
+//
+// e^(G_i - G_j) is the product of a row's factor e^(G_i - M) and a column's e^(M - G_j), M the sum up to the middle of the row's
+// sixteen tokens: both are finite as long as eight tokens decay by less than e^60.  Sixteen rows with a channel beyond that
+// take M in front of them (both factors are then at most 1) and their own 16 x 16 block pair by pair.
+//
+// q, k, v are bf16 values; everything else is fp32: where an fp32 quantity is the operand of a bf16 product it is split into two
+// bf16 terms, of whose four products the three that matter are taken (16 bits); T is made in fp32 on the CUDA cores.
 #include "delta.cuh"
+
 namespace pace {
-bool delta_chunked_fits(const pace_delta_args_t& a) { return false; }
-int delta_chunked(const pace_step_t& st, const pace_delta_args_t& a, cudaStream_t s) { return PACE_ERR_UNSUPPORTED; }
+namespace {
+
+constexpr int kChunk = 64, kThreads = 256, kLP = kChunk + 4, kTP = kChunk + 8;
+constexpr float kRange = 86.0f;   // log2 units eight tokens may decay by on the fast path: e^60
+
+__device__ __forceinline__ void mma16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-extern "C" uint64_t pace_delta_workspace_bytes(int32_t n_tokens, int32_t n_entries, int32_t heads, int32_t dim, int32_t vdim, int32_t dtype) { return 0; }
+// (hi + lo) x (hi + lo) without the last term
+__device__ __forceinline__ void mma_split(float* c, const uint32_t* ah, const uint32_t* al, const uint32_t* bh, const uint32_t* bl) {
+  mma16816(c, ah, bh[0], bh[1]);
+  mma16816(c, ah, bl[0], bl[1]);
+  mma16816(c, al, bh[0], bh[1]);
+}
+__device__ __forceinline__ void ldsm4(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void copy16(void* dst, const void* src, bool live = true) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
+}
+
+// What the first launch leaves of a (entry, chunk, head): bf16 tiles [64][DP] (high, low halves), P [64][64], then fp32.
+template <int DP>
+struct Slot {
+  static constexpr int kTile = kChunk * DP;
+  static constexpr int kW = 0, kQ = 2 * kTile, kK = 4 * kTile, kP = 6 * kTile, kHalves = kP + 2 * kChunk * kChunk;
+  static constexpr size_t kDecay = (size_t)kHalves * 2;               // bytes: [DP] decays over the whole chunk
+  static constexpr size_t kUv = kDecay + DP * 4;                      // [64][vdim] T V
+  static __host__ __device__ size_t bytes(int vdim) { return kUv + (size_t)kChunk * vdim * 4; }
+};
+
+struct Slab {
+  unsigned char* scratch;
+  int first, n;    // chunks [first, first + n) of every entry
+};
+
+template <int DP>
+struct Prep {
+  static constexpr int QP = DP + 8, GP = DP + 8;
+  static constexpr int kK = 0, kQ = kK + kChunk * QP * 2, kG = kQ + kChunk * QP * 2, kL = kG + kChunk * GP * 4,
+                       kT = kL + kChunk * kLP * 4, kVec = kT + 2 * kChunk * kTP * 2, bytes = kVec + (3 * kChunk + 4) * 4;
+};
+
+template <int DP>
+__global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t st, pace_delta_args_t a, Slab sl) {
+  using SL = Slot<DP>;
+  using PR = Prep<DP>;
+  constexpr int QP = PR::QP, GP = PR::GP;
+  const int e = blockIdx.z, h = blockIdx.y, d = a.dim, vd = a.vdim, H = a.heads, KV = a.kv_heads, kh = h / (H / KV);
+  const int count = st.cu[e + 1] - st.cu[e], l0 = (sl.first + (int)blockIdx.x) * kChunk;
+  if (l0 >= count) return;
+  const int n_tok = min(kChunk, count - l0), t0 = st.cu[e] + l0;
+  extern __shared__ __align__(16) unsigned char sm[];
+  __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(sm + PR::kK);
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(sm + PR::kQ);
+  float* G = reinterpret_cast<float*>(sm + PR::kG);      // sums of log decays, log2 units
+  float* L = reinterpret_cast<float*>(sm + PR::kL);      // diag(beta) A, then (1 + L)^-1 in its place
+  __nv_bfloat16* t_hi = reinterpret_cast<__nv_bfloat16*>(sm + PR::kT);
+  __nv_bfloat16* t_lo = t_hi + kChunk * kTP;
+  float* fk = reinterpret_cast<float*>(sm + PR::kVec);
+  float* fq = fk + kChunk;
+  float* beta = fq + kChunk;
+  int* slow = reinterpret_cast<int*>(beta + kChunk);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  unsigned char* slot = sl.scratch + (((size_t)e * sl.n + blockIdx.x) * H + h) * SL::bytes(vd);
+  __nv_bfloat16* tiles = reinterpret_cast<__nv_bfloat16*>(slot);
+
+  // ---- operands: keys and queries as they are, log decays, unit factors ----
+  const __nv_bfloat16* qkv = static_cast<const __nv_bfloat16*>(a.qkv) + (size_t)t0 * a.qkv_stride;
+  for (int i = tid; i < kChunk * (DP / 8) * 2; i += kThreads) {
+    const int which = i / (kChunk * (DP / 8)), r = i - which * (kChunk * (DP / 8)), j = r / (DP / 8), c = (r - j * (DP / 8)) * 8;
+    const bool live = j < n_tok && c < d;
+    copy16((which ? ks : qs) + j * QP + c, qkv + (live ? (size_t)j * a.qkv_stride + (size_t)(which * KV + kh) * d + c : 0), live);
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  if (tid < 4) slow[tid] = 0;
+  if (tid < kChunk)
+    beta[tid] = tid < n_tok ? sigmoid_t<__nv_bfloat16>(
+        __bfloat162float(static_cast<const __nv_bfloat16*>(a.b_raw)[(size_t)(t0 + tid) * a.b_stride + h])) : 0.f;
+  {
+    const float neg_a = a.neg_a[h] * kLog2e;
+    const __nv_bfloat16* ar = static_cast<const __nv_bfloat16*>(a.a_raw) + (size_t)t0 * a.a_stride + (size_t)h * d;
+    for (int i = tid; i < kChunk * (DP / 2); i += kThreads) {
+      const int j = i / (DP / 2), c = (i - j * (DP / 2)) * 2;
+      float2 v = make_float2(0.f, 0.f);
+      if (j < n_tok && c < d) {
+        const float2 x = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ar + (size_t)j * a.a_stride + c));
+        const float2 b = *reinterpret_cast<const float2*>(a.dt_bias + (size_t)h * d + c);
+        v = make_float2(neg_a * softplus(x.x + b.x), neg_a * softplus(x.y + b.y));
+      }
+      *reinterpret_cast<float2*>(G + j * GP + c) = v;
+    }
+  }
+  for (int i = tid; i < kChunk * kLP; i += kThreads) L[i] = 0.f;
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  constexpr int PARTS = kThreads / DP, ROWS = kChunk / PARTS;
+  const int gc = tid % DP, part = tid / DP;
+  {
+    float s = 0.f;
+#pragma unroll 8
+    for (int j = part * ROWS; j < (part + 1) * ROWS; ++j) G[j * GP + gc] = s += G[j * GP + gc];
+  }
+  for (int j = warp * 8; j < warp * 8 + 8; ++j) {
+    float sq = 0.f, sk = 0.f;
+    for (int c = lane * 2; c < DP; c += 64) {
+      const float2 x = bf2_to_f2(*reinterpret_cast<const uint32_t*>(qs + j * QP + c)), y = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ks + j * QP + c));
+      sq = fmaf(x.x, x.x, fmaf(x.y, x.y, sq));
+      sk = fmaf(y.x, y.x, fmaf(y.y, y.y, sk));
+    }
+#pragma unroll
+    for (int o = 16; o; o >>= 1) {
+      sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      sk += __shfl_xor_sync(0xffffffffu, sk, o);
+    }
+    if (lane == 0) {
+      fq[j] = a.q_scale / sqrtf(sq + a.unit_eps);
+      fk[j] = 1.0f / sqrtf(sk + a.unit_eps);
+    }
+  }
+  __syncthreads();
+  float before = 0.f;
+  for (int p = 0; p < part; ++p) before += G[((p + 1) * ROWS - 1) * GP + gc];
+  __syncthreads();
+  if (part > 0) {
+#pragma unroll 8
+    for (int j = part * ROWS; j < (part + 1) * ROWS; ++j) G[j * GP + gc] += before;
+  }
+  __syncthreads();
+  for (int i = tid; i < 4 * DP; i += kThreads) {
+    const int b = i / DP, c = i - b * DP;
+    const float m = G[(16 * b + 7) * GP + c], s = b ? G[(16 * b - 1) * GP + c] : 0.f;
+    if (s - m > kRange || m - G[(16 * b + 15) * GP + c] > kRange) slow[b] = 1;
+  }
+  __syncthreads();
+
+  // ---- scores: warp (row block of 16, every other tile of 8 columns); the two long and the two short blocks share schedulers ----
+  {
+    const int rb = warp < 4 ? warp : 7 - warp, half = (warp >> 2) & 1;   // warps w and w + 4: row blocks w and 3 - w
+    // (half: warps 0 .. 3 take the even tiles of row block w, warps 4 .. 7 the odd ones of row block 7 - w)
+    float ck[4][4], cq[4][4];
+#pragma unroll
+    for (int s = 0; s < 4; ++s)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) ck[s][x] = cq[s][x] = 0.f;
+    const bool far = slow[rb] != 0;
+    const int i0 = 16 * rb + g, ref = far ? 16 * rb - 1 : 16 * rb + 7;
+#pragma unroll 1
+    for (int k0 = 0; k0 < DP; k0 += 16) {
+      const int c0 = k0 + 2 * t;
+      float2 m[2];
+#pragma unroll
+      for (int x = 0; x < 2; ++x) m[x] = ref >= 0 ? *reinterpret_cast<const float2*>(G + ref * GP + c0 + 8 * x) : make_float2(0.f, 0.f);
+      uint32_t kh_[4], kl_[4], qh_[4], ql_[4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int row = i0 + (x & 1) * 8, c = c0 + (x >> 1) * 8;
+        const float2 gg = *reinterpret_cast<const float2*>(G + row * GP + c);
+        const float e0 = fast_exp2(gg.x - m[x >> 1].x), e1 = fast_exp2(gg.y - m[x >> 1].y);
+        const float2 kk = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ks + row * QP + c));
+        const float2 qq = bf2_to_f2(*reinterpret_cast<const uint32_t*>(qs + row * QP + c));
+        split_bf2(kk.x * e0, kk.y * e1, kh_[x], kl_[x]);
+        split_bf2(qq.x * e0, qq.y * e1, qh_[x], ql_[x]);
+      }
+#pragma unroll
+      for (int s = 0; s < 4; ++s) {
+        if (s > rb) break;
+        const int j = 8 * (2 * s + half) + g;
+        uint32_t bh[2], bl[2];
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const float2 gg = *reinterpret_cast<const float2*>(G + j * GP + c0 + 8 * x);
+          const float2 kk = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ks + j * QP + c0 + 8 * x));
+          split_bf2(kk.x * fast_exp2(m[x].x - gg.x), kk.y * fast_exp2(m[x].y - gg.y), bh[x], bl[x]);
+        }
+        mma_split(ck[s], kh_, kl_, bh, bl);
+        mma_split(cq[s], qh_, ql_, bh, bl);
+      }
+    }
+    __nv_bfloat16 *p_hi = tiles + SL::kP, *p_lo = p_hi + kChunk * kChunk;
+#pragma unroll
+    for (int s = 0; s < 4; ++s) {
+      if (s > rb || (far && s == rb)) break;
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int i = i0 + 8 * x, j = 8 * (2 * s + half) + 2 * t;
+        const float f0 = fk[j], f1 = fk[j + 1], bi = beta[i] * fk[i], qi = fq[i];
+        L[i * kLP + j] = j < i ? ck[s][2 * x] * bi * f0 : 0.f;
+        L[i * kLP + j + 1] = j + 1 < i ? ck[s][2 * x + 1] * bi * f1 : 0.f;
+        uint32_t hi, lo;
+        split_bf2(j <= i ? cq[s][2 * x] * qi * f0 : 0.f, j + 1 <= i ? cq[s][2 * x + 1] * qi * f1 : 0.f, hi, lo);
+        *reinterpret_cast<uint32_t*>(p_hi + i * kChunk + j) = hi;
+        *reinterpret_cast<uint32_t*>(p_lo + i * kChunk + j) = lo;
+      }
+    }
+  }
+  for (int b = 0; b < 4; ++b) {
+    if (!slow[b]) continue;
+    __nv_bfloat16 *p_hi = tiles + SL::kP, *p_lo = p_hi + kChunk * kChunk;
+    const int i = 16 * b + tid / 16, j = 16 * b + tid % 16;   // one pair per thread
+    float sk = 0.f, sq = 0.f;
+    if (j <= i) {
+      for (int c = 0; c < DP; ++c) {
+        const float f = fast_exp2(G[i * GP + c] - G[j * GP + c]) * __bfloat162float(ks[j * QP + c]);
+        sk = fmaf(__bfloat162float(ks[i * QP + c]), f, sk);
+        sq = fmaf(__bfloat162float(qs[i * QP + c]), f, sq);
+      }
+    }
+    L[i * kLP + j] = j < i ? sk * beta[i] * fk[i] * fk[j] : 0.f;
+    const float p = sq * fq[i] * fk[j];
+    const __nv_bfloat16 hi = __float2bfloat16_rn(p);
+    p_hi[i * kChunk + j] = hi;
+    p_lo[i * kChunk + j] = __float2bfloat16_rn(p - __bfloat162float(hi));
+  }
+  // ---- queries and keys with their decays ----
+  for (int i = tid; i < kChunk * (DP / 2); i += kThreads) {
+    const int j = i / (DP / 2), c = (i - j * (DP / 2)) * 2;
+    const float2 gg = *reinterpret_cast<const float2*>(G + j * GP + c), ge = *reinterpret_cast<const float2*>(G + (kChunk - 1) * GP + c);
+    const float2 kk = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ks + j * QP + c));
+    const float2 qq = bf2_to_f2(*reinterpret_cast<const uint32_t*>(qs + j * QP + c));
+    uint32_t hi, lo;
+    split_bf2(qq.x * fq[j] * fast_exp2(gg.x), qq.y * fq[j] * fast_exp2(gg.y), hi, lo);
+    reinterpret_cast<uint32_t*>(tiles + SL::kQ)[i] = hi;
+    reinterpret_cast<uint32_t*>(tiles + SL::kQ + SL::kTile)[i] = lo;
+    split_bf2(kk.x * fk[j] * fast_exp2(ge.x - gg.x), kk.y * fk[j] * fast_exp2(ge.y - gg.y), hi, lo);
+    reinterpret_cast<uint32_t*>(tiles + SL::kK)[i] = hi;
+    reinterpret_cast<uint32_t*>(tiles + SL::kK + SL::kTile)[i] = lo;
+  }
+  if (tid < DP) reinterpret_cast<float*>(slot + SL::kDecay)[tid] = fast_exp2(G[(kChunk - 1) * GP + tid]);
+  __syncthreads();
+
+  // ---- (1 + L)^-1 in place of L: blocks of 16, then of 32, then of 64 ----
+  {
+    const int b = (tid >> 4) & 3, col = tid & 15;
+    float x[16];
+    if (tid < 64) {
+#pragma unroll
+      for (int i = 0; i < 16; ++i) x[i] = i == col ? 1.f : 0.f;
+      const float* Lb = L + 16 * b * kLP + 16 * b;
+#pragma unroll
+      for (int j = 0; j < 15; ++j)
+#pragma unroll
+        for (int i = j + 1; i < 16; ++i) x[i] = fmaf(-Lb[i * kLP + j], x[j], x[i]);
+    }
+    __syncthreads();
+    if (tid < 64) {
+#pragma unroll
+      for (int i = 0; i < 16; ++i) L[(16 * b + i) * kLP + 16 * b + col] = x[i];
+    }
+    __syncthreads();
+    // lower left block of a pair: -T_bb (L_ba T_aa)
+    auto combine = [&](auto size_c) {
+      constexpr int N = decltype(size_c)::value, PAIRS = kChunk / (2 * N), PER = PAIRS * N * N / kThreads;
+      float y[PER];
+#pragma unroll
+      for (int step = 0; step < 2; ++step) {
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+          const int o = k * kThreads + tid, pr = o / (N * N), i = (o - pr * N * N) / N, j = o % N, at = 2 * N * pr;
+          const float *row, *colp;
+          if (step == 0) row = L + (at + N + i) * kLP + at, colp = L + at * kLP + at + j;               // L_ba, T_aa
+          else row = L + (at + N + i) * kLP + at + N, colp = L + (at + N) * kLP + at + j;               // T_bb, the product
+          float s = 0.f;
+#pragma unroll
+          for (int x2 = 0; x2 < N; ++x2) s = fmaf(row[x2], colp[x2 * kLP], s);
+          y[k] = step ? -s : s;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+          const int o = k * kThreads + tid, pr = o / (N * N), i = (o - pr * N * N) / N, j = o % N, at = 2 * N * pr;
+          L[(at + N + i) * kLP + at + j] = y[k];
+        }
+        __syncthreads();
+      }
+    };
+    combine(std::integral_constant<int, 16>());
+    combine(std::integral_constant<int, 32>());
+  }
+  for (int i = tid; i < kChunk * kChunk / 2; i += kThreads) {
+    const int r = i / (kChunk / 2), c = (i - r * (kChunk / 2)) * 2;
+    uint32_t hi, lo;
+    split_bf2(L[r * kLP + c] * beta[c], L[r * kLP + c + 1] * beta[c + 1], hi, lo);
+    *reinterpret_cast<uint32_t*>(t_hi + r * kTP + c) = hi;
+    *reinterpret_cast<uint32_t*>(t_lo + r * kTP + c) = lo;
+  }
+  __syncthreads();
+
+  // ---- T K^(G) and T V, 16 columns at a time ----
+  const int w_items = DP / 16, items = w_items + (vd + 15) / 16;
+  for (int it = warp; it < items; it += kThreads / 32) {
+    const bool is_w = it < w_items;
+    const int n0 = (is_w ? it : it - w_items) * 16;
+    float acc[4][2][4];
+#pragma unroll
+    for (int m = 0; m < 4; ++m)
+#pragma unroll
+      for (int s = 0; s < 2; ++s)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) acc[m][s][x] = 0.f;
+#pragma unroll
+    for (int kt = 0; kt < 4; ++kt) {
+      uint32_t bh[2][2], bl[2][2];
+#pragma unroll
+      for (int s = 0; s < 2; ++s) {
+        const int c = n0 + 8 * s + g;
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const int j = 16 * kt + 2 * t + 8 * x;
+          if (is_w) {
+            const float v0 = __bfloat162float(ks[j * QP + c]) * fk[j] * fast_exp2(G[j * GP + c]);
+            const float v1 = __bfloat162float(ks[(j + 1) * QP + c]) * fk[j + 1] * fast_exp2(G[(j + 1) * GP + c]);
+            split_bf2(v0, v1, bh[s][x], bl[s][x]);
+          } else {
+            const unsigned short* v = reinterpret_cast<const unsigned short*>(qkv) + (size_t)j * a.qkv_stride + 2 * (size_t)KV * d + (size_t)h * vd + c;
+            const uint32_t lo16 = j < n_tok && c < vd ? v[0] : 0, hi16 = j + 1 < n_tok && c < vd ? v[a.qkv_stride] : 0;
+            bh[s][x] = lo16 | (hi16 << 16);
+            bl[s][x] = 0;
+          }
+        }
+      }
+#pragma unroll
+      for (int m = kt; m < 4; ++m) {
+        uint32_t ah[4], al[4];
+        ldsm4(ah, t_hi + (16 * m + (lane & 15)) * kTP + 16 * kt + (lane >> 4) * 8);
+        ldsm4(al, t_lo + (16 * m + (lane & 15)) * kTP + 16 * kt + (lane >> 4) * 8);
+#pragma unroll
+        for (int s = 0; s < 2; ++s) {
+          mma16816(acc[m][s], ah, bh[s][0], bh[s][1]);
+          mma16816(acc[m][s], al, bh[s][0], bh[s][1]);
+          if (is_w) mma16816(acc[m][s], ah, bl[s][0], bl[s][1]);
+        }
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < 4; ++m)
+#pragma unroll
+      for (int s = 0; s < 2; ++s)
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const int i = 16 * m + g + 8 * x, c = n0 + 8 * s + 2 * t;
+          if (is_w) {
+            uint32_t hi, lo;
+            split_bf2(acc[m][s][2 * x], acc[m][s][2 * x + 1], hi, lo);
+            *reinterpret_cast<uint32_t*>(tiles + SL::kW + i * DP + c) = hi;
+            *reinterpret_cast<uint32_t*>(tiles + SL::kW + SL::kTile + i * DP + c) = lo;
+          } else if (c < vd) {
+            *reinterpret_cast<float2*>(slot + SL::kUv + ((size_t)i * vd + c) * 4) = make_float2(acc[m][s][2 * x], acc[m][s][2 * x + 1]);
+          }
+        }
+  }
+}
+
+template <int DP, int VB>
+struct Walk {
+  static constexpr int QP = DP + 8, VP = VB + 8;
+  static constexpr int kW = 0, kQ = 2 * kChunk * QP, kK = 4 * kChunk * QP, kP = 6 * kChunk * QP, kS = kP + 2 * kChunk * kTP,
+                       kU = kS + 2 * DP * VP, kEnd = kU + 2 * kChunk * VP, bytes = kEnd * 2;
+};
+
+template <int DP, int VB>
+__global__ void __launch_bounds__(kThreads, 1) delta_walk_kernel(pace_step_t st, pace_delta_args_t a, Slab sl) {
+  using SL = Slot<DP>;
+  using WK = Walk<DP, VB>;
+  constexpr int QP = WK::QP, VP = WK::VP, NT = VB / 8;
+  constexpr int RG = DP / 16, CG = 8 / RG, SC = VB / CG, NS = SC / 8;   // state tile of a warp: 16 rows x SC columns
+  static_assert(NS >= 1, "a warp owns eight columns of the state at least");
+  const int e = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * VB, d = a.dim, vd = a.vdim, H = a.heads;
+  const int count = st.cu[e + 1] - st.cu[e], chunks = min(sl.n, (count + kChunk - 1) / kChunk - sl.first);
+  if (chunks <= 0) return;
+  extern __shared__ __align__(16) __nv_bfloat16 sb[];
+  __nv_bfloat16 *s_hi = sb + WK::kS, *s_lo = s_hi + DP * VP, *u_hi = sb + WK::kU, *u_lo = u_hi + kChunk * VP;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const size_t slot_bytes = SL::bytes(vd);
+  const unsigned char* slot = sl.scratch + ((size_t)e * sl.n * H + h) * slot_bytes;
+  auto fetch = [&](const unsigned char* from, int first_tile, int n_tiles) {   // [64][DP] tiles into rows of QP
+    const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(from) + first_tile * SL::kTile;
+    __nv_bfloat16* dst = sb + first_tile * kChunk * QP;
+    for (int i = tid; i < n_tiles * SL::kTile / 8; i += kThreads) {
+      const int r = i / (DP / 8), c = (i - r * (DP / 8)) * 8;
+      copy16(dst + r * QP + c, src + (size_t)r * DP + c);
+    }
+  };
+  auto fetch_wq = [&](const unsigned char* from) {
+    fetch(from, 0, 4);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  auto fetch_kp = [&](const unsigned char* from) {
+    fetch(from, 4, 2);
+    const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(from) + SL::kP;
+    for (int i = tid; i < 2 * kChunk * kChunk / 8; i += kThreads) {
+      const int r = i / (kChunk / 8), c = (i - r * (kChunk / 8)) * 8;
+      copy16(sb + WK::kP + r * kTP + c, src + r * kChunk + c);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  fetch_wq(slot);
+  float* state = a.s_state + ((size_t)st.slot[e] * H + h) * d * vd;
+  const bool fresh = st.start[e] == 0 && sl.first == 0;
+  const int sr = (warp % RG) * 16 + g, sc = (warp / RG) * SC + 2 * t;
+  float S[NS][4];
+#pragma unroll
+  for (int n = 0; n < NS; ++n)
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int r = sr + 8 * x, c = v0 + sc + 8 * n;            // (vdim is a multiple of 8: pairs are whole)
+      const float2 v = !fresh && r < d && c < vd ? *reinterpret_cast<const float2*>(state + (size_t)r * vd + c) : make_float2(0.f, 0.f);
+      S[n][2 * x] = v.x;
+      S[n][2 * x + 1] = v.y;
+    }
+  auto put_state = [&]() {
+#pragma unroll
+    for (int n = 0; n < NS; ++n)
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        uint32_t hi, lo;
+        split_bf2(S[n][2 * x], S[n][2 * x + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(s_hi + (sr + 8 * x) * VP + sc + 8 * n) = hi;
+        *reinterpret_cast<uint32_t*>(s_lo + (sr + 8 * x) * VP + sc + 8 * n) = lo;
+      }
+  };
+  put_state();
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  for (int c = 0; c < chunks; ++c, slot += (size_t)H * slot_bytes) {
+    fetch_kp(slot);
+    const int l0 = (sl.first + c) * kChunk, n_tok = min(kChunk, count - l0);
+    const float* decay = reinterpret_cast<const float*>(slot + SL::kDecay);
+    const float d0 = decay[sr], d1 = decay[sr + 8];
+    const int row = (warp & 3) * 16 + g;                       // of the tokens, for warps 0 .. 3 (W) and 4 .. 7 (Q)
+    float uv[NT][4];
+    if (warp < 4) {
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const int col = v0 + 8 * n + 2 * t;
+          const float2 v = col < vd ? *reinterpret_cast<const float2*>(slot + SL::kUv + ((size_t)(row + 8 * x) * vd + col) * 4) : make_float2(0.f, 0.f);
+          uv[n][2 * x] = v.x;
+          uv[n][2 * x + 1] = v.y;
+        }
+    }
+    // ---- what the state answers to the keys (W S) and the queries ----
+    float acc[NT][4];
+#pragma unroll
+    for (int n = 0; n < NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+    {
+      const __nv_bfloat16* ah_p = sb + (warp < 4 ? WK::kW : WK::kQ) + ((warp & 3) * 16 + (lane & 15)) * QP + (lane >> 4) * 8;
+#pragma unroll
+      for (int k0 = 0; k0 < DP; k0 += 16) {
+        uint32_t ah[4], al[4];
+        ldsm4(ah, ah_p + k0);
+        ldsm4(al, ah_p + kChunk * QP + k0);
+#pragma unroll
+        for (int n = 0; n < NT; n += 2) {
+          uint32_t bh[4], bl[4];
+          ldsm4t(bh, s_hi + (k0 + (lane & 15)) * VP + n * 8 + (lane >> 4) * 8);
+          ldsm4t(bl, s_lo + (k0 + (lane & 15)) * VP + n * 8 + (lane >> 4) * 8);
+          mma_split(acc[n], ah, al, bh, bl);
+          mma_split(acc[n + 1], ah, al, bh + 2, bl + 2);
+        }
+      }
+    }
+    if (warp < 4) {
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          uint32_t hi, lo;
+          split_bf2(uv[n][2 * x] - acc[n][2 * x], uv[n][2 * x + 1] - acc[n][2 * x + 1], hi, lo);
+          *reinterpret_cast<uint32_t*>(u_hi + (row + 8 * x) * VP + 8 * n + 2 * t) = hi;
+          *reinterpret_cast<uint32_t*>(u_lo + (row + 8 * x) * VP + 8 * n + 2 * t) = lo;
+        }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                           // U, K and P are there; W, Q and the state have been read
+    if (c + 1 < chunks) fetch_wq(slot + (size_t)H * slot_bytes);
+    // ---- the state behind the chunk ----
+#pragma unroll
+    for (int n = 0; n < NS; ++n) {
+      S[n][0] *= d0; S[n][1] *= d0;
+      S[n][2] *= d1; S[n][3] *= d1;
+    }
+    {
+      const int m0 = (warp % RG) * 16, c0 = (warp / RG) * SC;
+#pragma unroll
+      for (int k0 = 0; k0 < kChunk; k0 += 16) {
+        uint32_t ah[4], al[4];
+        const __nv_bfloat16* kp = sb + WK::kK + (k0 + (lane & 7) + (lane >> 4) * 8) * QP + m0 + ((lane >> 3) & 1) * 8;
+        ldsm4t(ah, kp);
+        ldsm4t(al, kp + kChunk * QP);
+#pragma unroll
+        for (int n = 0; n < NS; n += 2) {
+          uint32_t bh[4], bl[4];   // (with one tile of eight columns the second one is read and not used)
+          ldsm4t(bh, u_hi + (k0 + (lane & 15)) * VP + c0 + n * 8 + (lane >> 4) * 8);
+          ldsm4t(bl, u_lo + (k0 + (lane & 15)) * VP + c0 + n * 8 + (lane >> 4) * 8);
+          mma_split(S[n], ah, al, bh, bl);
+          if (n + 1 < NS) mma_split(S[n + 1 < NS ? n + 1 : n], ah, al, bh + 2, bl + 2);
+        }
+      }
+    }
+    put_state();
+    if (warp >= 4) {
+      const int m = warp - 4;
+      for (int kt = 0; kt <= m; ++kt) {
+        uint32_t ah[4], al[4];
+        const __nv_bfloat16* pp = sb + WK::kP + (16 * m + (lane & 15)) * kTP + 16 * kt + (lane >> 4) * 8;
+        ldsm4(ah, pp);
+        ldsm4(al, pp + kChunk * kTP);
+#pragma unroll
+        for (int n = 0; n < NT; n += 2) {
+          uint32_t bh[4], bl[4];
+          ldsm4t(bh, u_hi + (16 * kt + (lane & 15)) * VP + n * 8 + (lane >> 4) * 8);
+          ldsm4t(bl, u_lo + (16 * kt + (lane & 15)) * VP + n * 8 + (lane >> 4) * 8);
+          mma_split(acc[n], ah, al, bh, bl);
+          mma_split(acc[n + 1], ah, al, bh + 2, bl + 2);
+        }
+      }
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (size_t)(st.cu[e] + l0) * a.out_stride + (size_t)h * vd + v0;
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int x = 0; x < 2; ++x)
+          if (row + 8 * x < n_tok && v0 + 8 * n + 2 * t < vd)
+            *reinterpret_cast<uint32_t*>(out + (size_t)(row + 8 * x) * a.out_stride + 8 * n + 2 * t) = f2_to_bf2(acc[n][2 * x], acc[n][2 * x + 1]);
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                           // the next W and Q and the state are there; K, P and U have been read
+  }
+#pragma unroll
+  for (int n = 0; n < NS; ++n)
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int r = sr + 8 * x, c = v0 + sc + 8 * n;
+      if (r < d && c < vd) *reinterpret_cast<float2*>(state + (size_t)r * vd + c) = make_float2(S[n][2 * x], S[n][2 * x + 1]);
+    }
+}
+
+constexpr uint64_t kBudget = 256ull << 20;   // bytes of scratch a launch pair may use
+
+struct Plan {
+  int dp, slab;      // padded key size, chunks of an entry per launch pair
+  uint64_t bytes;
+};
+Plan plan_chunks(int n_entries, int max_count, int heads, int dim, int vdim) {
+  Plan p;
+  p.dp = dim <= 64 ? 64 : 128;
+  const uint64_t slot = p.dp == 64 ? Slot<64>::bytes(vdim) : Slot<128>::bytes(vdim), row = slot * heads * n_entries;
+  const int chunks = (max_count + kChunk - 1) / kChunk;
+  const uint64_t fit = kBudget / row;
+  p.slab = fit < 1 ? 1 : fit < (uint64_t)chunks ? (int)fit : chunks;
+  p.bytes = row * p.slab;
+  return p;
+}
+
+template <int DP, int VB>
+int launch_walk(const pace_step_t& st, const pace_delta_args_t& a, const Slab& sl, cudaStream_t s) {
+  PACE_CUDA_TRY(cudaFuncSetAttribute(delta_walk_kernel<DP, VB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Walk<DP, VB>::bytes));
+  const dim3 grid((unsigned)((a.vdim + VB - 1) / VB), (unsigned)a.heads, (unsigned)st.n_entries);
+  delta_walk_kernel<DP, VB><<<grid, kThreads, Walk<DP, VB>::bytes, s>>>(st, a, sl);
+  PACE_LAUNCH_CHECK("delta_walk_kernel");
+  return PACE_OK;
+}
+
+template <int DP>
+int launch_chunked(const pace_step_t& st, const pace_delta_args_t& a, const Plan& p, cudaStream_t s) {
+  PACE_CUDA_TRY(cudaFuncSetAttribute(delta_prepare_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Prep<DP>::bytes));
+  const int chunks = (st.max_count + kChunk - 1) / kChunk;
+  // few sequences and heads: narrow columns, so that more SMs take part
+  const bool narrow = (int64_t)st.n_entries * a.heads * ((a.vdim + 31) / 32) <= 74;
+  for (int c = 0; c < chunks; c += p.slab) {
+    Slab sl;
+    sl.scratch = static_cast<unsigned char*>(a.workspace);
+    sl.first = c;
+    sl.n = p.slab;
+    const int n = chunks - c < p.slab ? chunks - c : p.slab;
+    delta_prepare_kernel<DP><<<dim3((unsigned)n, (unsigned)a.heads, (unsigned)st.n_entries), kThreads, Prep<DP>::bytes, s>>>(st, a, sl);
+    PACE_LAUNCH_CHECK("delta_prepare_kernel");
+    const int rc = narrow ? launch_walk<DP, 16>(st, a, sl, s) : launch_walk<DP, 32>(st, a, sl, s);
+    if (rc != PACE_OK) return rc;
+  }
+  return PACE_OK;
+}
+
+}  // namespace
+
+// bf16, key sizes that the tiles cover and 16-byte pieces; everything else is the token-by-token kernel's
+bool delta_chunked_fits(const pace_delta_args_t& a) {
+  return a.dtype == PACE_DTYPE_BF16 && a.dim <= 128 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.qkv_stride % 8 == 0 && a.a_stride % 2 == 0 &&
+         a.out_stride % 2 == 0 && aligned16(a.qkv) && ((uintptr_t)a.a_raw & 3) == 0 && ((uintptr_t)a.dt_bias & 7) == 0 &&
+         ((uintptr_t)a.out & 3) == 0 && ((uintptr_t)a.s_state & 7) == 0;
+}
+
+int delta_chunked(const pace_step_t& st, const pace_delta_args_t& a, cudaStream_t s) {
+  const Plan p = plan_chunks(st.n_entries, st.max_count, a.heads, a.dim, a.vdim);
+  if (!a.workspace || a.workspace_bytes < p.bytes || !aligned16(a.workspace)) return PACE_ERR_INVALID;
+  return p.dp == 64 ? launch_chunked<64>(st, a, p, s) : launch_chunked<128>(st, a, p, s);
+}
+
+}  // namespace pace
+
+extern "C" uint64_t pace_delta_workspace_bytes(int32_t n_entries, int32_t max_count, int32_t heads, int32_t dim, int32_t vdim, int32_t dtype) {
+  if (n_entries <= 0 || max_count <= 0 || heads <= 0 || dim <= 0 || vdim <= 0 || dim > 128 || dtype != PACE_DTYPE_BF16) return 0;
+  return pace::plan_chunks(n_entries, max_count, heads, dim, vdim).bytes;
+}

@@ -811,7 +811,7 @@ typedef struct {
   int32_t heads, kv_heads, dim, vdim, n_taps, ring_rows, ring_stride, dtype;
   float unit_eps, q_scale;
 } pace_delta_args_t;
-uint64_t pace_delta_workspace_bytes(int32_t n_tokens, int32_t n_entries, int32_t heads, int32_t dim, int32_t vdim, int32_t dtype);
+uint64_t pace_delta_workspace_bytes(int32_t n_entries, int32_t max_count, int32_t heads, int32_t dim, int32_t vdim, int32_t dtype);
 int pace_delta_prefill(const pace_step_t* step, const pace_delta_args_t* a, void* stream);
 int pace_delta_step(const pace_step_t* step, const pace_delta_args_t* a, void* stream);
 
