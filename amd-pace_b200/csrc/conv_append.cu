@@ -13,136 +13,185 @@ struct PageRows {
   int page_tokens, n_kv_heads, max_pages_per_seq, max_seqs, n_pages;
 };
 
-constexpr int kTokens = 4, kThreads = 256;
+constexpr int kTokens = 8, kThreads = 256;
 
-// LH lanes per head row, ITEMS vectors of V elements per lane; a block takes `per` tokens, whose rows the convolution
-// reads again out of the cache.  NT: taps where known at compile time (and held in registers), else 0.
+struct Token {
+  int pos, local, slot;
+  int64_t page_row;    // row of the layer's pages for KV head 0, -1: none
+};
+
+// A block takes `per` tokens of the heads of one round: LH lanes per head row, ITEMS vectors of V elements per lane.  NT: taps
+// where known at compile time (ITEMS is then 1, and the usual tokens - one sequence, all inputs among the step's rows - keep their
+// window of rows in registers), else 0.
 template <typename T, int V, int LH, int ITEMS, int NT>
-__global__ void __launch_bounds__(kThreads) append_conv_kernel(pace_step_t st, PageRows pg, pace_append_conv_args_t a, int row, int per) {
-  const int lane = threadIdx.x % LH, groups = blockDim.x / LH, t0 = blockIdx.x * per;
-  const int n_tok = min(per, st.n_tokens - t0);
+__global__ void __launch_bounds__(kThreads, ITEMS == 1 ? 2 : 1) append_conv_kernel(pace_step_t st, PageRows pg, pace_append_conv_args_t a, int row, int per) {
+  __shared__ Token info[kTokens];
+  extern __shared__ float turn_by[];       // [per][cosines, sines][rot_pairs] of the block's tokens
+  const int lane = threadIdx.x % LH, groups = blockDim.x / LH, t0 = blockIdx.x * per, n_tok = min(per, st.n_tokens - t0);
   const int H = a.n_q_heads, G = pg.n_kv_heads, d = a.dim, vd = a.vdim, channels = (H + G) * d + G * vd;
   const int taps = NT ? NT : a.n_taps;
   const T* in = static_cast<const T*>(a.qkv);
-  // blocks of one token spread the heads over the grid's y extent, so that a decode step fills the GPU
-  const int rounds = (H + 2 * G + groups * gridDim.y - 1) / (groups * gridDim.y);   // (the same for every thread)
-  for (int it = 0; it < rounds; ++it) {
-    const int hh = (it * gridDim.y + blockIdx.y) * groups + threadIdx.x / LH;
-    const bool exists = hh < H + 2 * G, is_q = hh < H, is_v = hh >= H + G;
-    const int g = is_v ? hh - H - G : hh - H, n = exists ? (is_v ? vd : d) : 0;
-    const int ch0 = is_q ? hh * d : is_v ? (H + G) * d + g * vd : H * d + g * d;   // first channel of the head
-    float w[NT ? NT : 1][V];   // (ITEMS is 1 where NT is not 0)
-    if constexpr (NT > 0) {
-      if (lane * V < n) {
+  const int hh = blockIdx.y * groups + threadIdx.x / LH;
+  const bool exists = hh < H + 2 * G, is_q = hh < H, is_v = hh >= H + G;
+  const int g = is_v ? hh - H - G : hh - H, n = exists ? (is_v ? vd : d) : 0;
+  const int ch0 = is_q ? hh * d : is_v ? (H + G) * d + g * vd : H * d + g * d;   // first channel of the head
+  if (threadIdx.x < n_tok) {
+    const int t = t0 + threadIdx.x, e = st.tok_entry[t], pos = st.tok_pos[t], slot = st.slot[e], lp = pos / pg.page_tokens;
+    Token k;
+    k.pos = pos;
+    k.local = t - st.cu[e];
+    k.slot = slot;
+    int page = -1;
+    if (slot >= 0 && slot < pg.max_seqs && lp < pg.max_pages_per_seq) page = pg.block_table[(size_t)slot * pg.max_pages_per_seq + lp];
+    if (page < 0 || page >= pg.n_pages || (a.rot_pairs > 0 && pos >= a.table_rows)) raise_status(pg.status, PACE_DEV_BAD_INDEX);
+    k.page_row = page >= 0 && page < pg.n_pages ? (int64_t)page * G * pg.page_tokens + (pos - lp * pg.page_tokens) : -1;
+    info[threadIdx.x] = k;
+  }
+  for (int i = threadIdx.x; i < n_tok * 2 * a.rot_pairs; i += blockDim.x) {
+    const int r = i / (2 * a.rot_pairs), c = i - r * 2 * a.rot_pairs, pos = min(st.tok_pos[t0 + r], a.table_rows - 1);
+    turn_by[i] = c < a.rot_pairs ? a.cos_table[(size_t)pos * a.rot_pairs + c] : a.sin_table[(size_t)pos * a.rot_pairs + c - a.rot_pairs];
+  }
+  float nw[ITEMS][V];      // norm weights
 #pragma unroll
-        for (int j = 0; j < NT; ++j) Vec<float, V>::load(a.taps + (size_t)j * channels + ch0 + lane * V, w[j]);
+  for (int i = 0; i < ITEMS; ++i) {
+    const int c = (i * LH + lane) * V;
+    if (!is_v && c < n) Vec<float, V>::load((is_q ? a.q_norm : a.k_norm) + c, nw[i]);
+    else
+#pragma unroll
+      for (int v = 0; v < V; ++v) nw[i][v] = 1.f;
+  }
+
+  // norm, rotation and store of a token's convolved head row
+  auto finish = [&](int r, float (*y)[V]) {
+    const Token& k = info[r];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i)
+#pragma unroll
+      for (int v = 0; v < V; ++v) ss = fmaf(y[i][v], y[i][v], ss);
+#pragma unroll
+    for (int o = LH / 2; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float f = is_v ? a.v_mul : 1.0f / sqrtf(ss / (float)n + a.eps);
+    T* dst = nullptr;
+    if (is_q) dst = static_cast<T*>(a.q_out) + ((size_t)(t0 + r) * H + hh) * row;
+    else if (exists && k.page_row >= 0) dst = reinterpret_cast<T*>(is_v ? pg.v : pg.k) + (k.page_row + (int64_t)g * pg.page_tokens) * row;
+    const bool turns = !is_v;
+    const float *cs = turn_by + r * 2 * a.rot_pairs, *sn = cs + a.rot_pairs;
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {
+      const int c = (i * LH + lane) * V;
+#pragma unroll
+      for (int v = 0; v < V; ++v) y[i][v] *= f * nw[i][v];
+      // the partner of an element lies in the same vector, or (V = 1) in the neighbouring lane
+      if constexpr (V == 1) {
+        const float other = __shfl_xor_sync(0xffffffffu, y[i][0], 1);
+        if (turns && (c >> 1) < a.rot_pairs)
+          y[i][0] = (c & 1) ? y[i][0] * cs[c >> 1] + other * sn[c >> 1] : y[i][0] * cs[c >> 1] - other * sn[c >> 1];
+      } else if (turns && c < 2 * a.rot_pairs) {
+#pragma unroll
+        for (int v = 0; v < V; v += 2) {
+          const int pr = (c + v) >> 1;
+          if (pr < a.rot_pairs) {
+            const float u = y[i][v] * cs[pr] - y[i][v + 1] * sn[pr];
+            y[i][v + 1] = y[i][v + 1] * cs[pr] + y[i][v] * sn[pr];
+            y[i][v] = u;
+          }
+        }
       }
+      if (dst && c < n) Vec<T, V>::store(dst + c, y[i]);
     }
-    for (int r = 0; r < n_tok; ++r) {
-      const int t = t0 + r, e = st.tok_entry[t], local = t - st.cu[e], pos = st.tok_pos[t], slot = st.slot[e];
-      float* ring = a.ring + (size_t)slot * a.ring_rows * a.ring_stride + ch0;
-      const T* now = in + (size_t)t * a.qkv_stride + ch0;
-      float y[ITEMS][V], ss = 0.f;
+    if (dst) {                                             // what a row has beyond its head size
+      float zero[V];
 #pragma unroll
-      for (int i = 0; i < ITEMS; ++i) {
-        const int c = (i * LH + lane) * V;
+      for (int v = 0; v < V; ++v) zero[v] = 0.f;
+      for (int c = n + lane * V; c < row; c += LH * V) Vec<T, V>::store(dst + c, zero);
+    }
+  };
+
+  float w[NT ? NT : 1][V];
+  if constexpr (NT > 0) {
 #pragma unroll
-        for (int v = 0; v < V; ++v) y[i][v] = 0.f;
-        if (c >= n) continue;
-        auto tap = [&](int j, const float* wj) {
-          const int back = taps - 1 - j;
+    for (int j = 0; j < NT; ++j) {
+      if (lane * V < n) Vec<float, V>::load(a.taps + (size_t)j * channels + ch0 + lane * V, w[j]);
+      else
+#pragma unroll
+        for (int v = 0; v < V; ++v) w[j][v] = 0.f;
+    }
+  }
+  if constexpr (NT > 0 && V * sizeof(T) == 16) {
+    // (a first look without the barrier: the rows may be on their way while the tokens' places are looked up)
+    const int e0 = st.tok_entry[t0];
+    if (per > 1 && t0 - (NT - 1) >= st.cu[e0] && t0 + n_tok <= st.cu[e0 + 1]) {
+      uint4 raw[kTokens + NT - 1];
+      const T* src = in + (int64_t)(t0 - (NT - 1)) * a.qkv_stride + ch0 + (lane * V < n ? lane * V : 0);
+#pragma unroll
+      for (int r = 0; r < kTokens + NT - 1; ++r)
+        raw[r] = lane * V < n && r < n_tok + NT - 1 ? *reinterpret_cast<const uint4*>(src + r * a.qkv_stride) : make_uint4(0, 0, 0, 0);
+      __syncthreads();
+#pragma unroll
+      for (int r = 0; r < kTokens; ++r) {
+        if (r >= n_tok) break;
+        float y[1][V];
+#pragma unroll
+        for (int v = 0; v < V; ++v) y[0][v] = 0.f;
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
           float x[V];
-          if (back <= local) Vec<T, V>::load(now - (int64_t)back * a.qkv_stride + c, x);
-          else if (back <= pos) Vec<float, V>::load(ring + (size_t)((pos - back) % a.ring_rows) * a.ring_stride + c, x);
-          else return;                                     // in front of the sequence
+          Vec<T, V>::load(reinterpret_cast<const T*>(&raw[r + j]), x);
 #pragma unroll
-          for (int v = 0; v < V; ++v) y[i][v] = fmaf(wj[v], x[v], y[i][v]);
-          if (a.store_ring && back == 0) Vec<float, V>::store(ring + (size_t)(pos % a.ring_rows) * a.ring_stride + c, x);
-        };
-        if constexpr (NT > 0) {
-#pragma unroll
-          for (int j = 0; j < NT; ++j) tap(j, w[j]);
-        } else {
-          for (int j = 0; j < taps; ++j) {
-            float wj[V];
-            Vec<float, V>::load(a.taps + (size_t)j * channels + ch0 + c, wj);
-            tap(j, wj);
-          }
+          for (int v = 0; v < V; ++v) y[0][v] = fmaf(w[j][v], x[v], y[0][v]);
         }
-#pragma unroll
-        for (int v = 0; v < V; ++v) ss = fmaf(y[i][v], y[i][v], ss);
+        finish(r, y);
       }
+      return;
+    }
+  }
+  __syncthreads();
+  for (int r = 0; r < n_tok; ++r) {
+    const Token& k = info[r];
+    float* ring = a.ring + (size_t)k.slot * a.ring_rows * a.ring_stride + ch0;
+    const T* now = in + (size_t)(t0 + r) * a.qkv_stride + ch0;
+    float y[ITEMS][V];
 #pragma unroll
-      for (int o = LH / 2; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      const float f = is_v ? a.v_mul : 1.0f / sqrtf(ss / (float)n + a.eps);
-      const float* nw = is_q ? a.q_norm : a.k_norm;
-      T* dst = nullptr;
-      if (exists && is_q) {
-        dst = static_cast<T*>(a.q_out) + ((size_t)t * H + hh) * row;
-      } else if (exists) {
-        const int lp = pos / pg.page_tokens;
-        int page = -1;
-        if (slot >= 0 && slot < pg.max_seqs && lp < pg.max_pages_per_seq)
-          page = pg.block_table[(size_t)slot * pg.max_pages_per_seq + lp];
-        if (page >= 0 && page < pg.n_pages)
-          dst = reinterpret_cast<T*>(is_v ? pg.v : pg.k) + (((size_t)page * G + g) * pg.page_tokens + (pos - lp * pg.page_tokens)) * row;
-        else if (lane == 0)
-          raise_status(pg.status, PACE_DEV_BAD_INDEX);
-      }
-      const bool turns = !is_v && a.rot_pairs > 0;
-      if (turns && pos >= a.table_rows && lane == 0) raise_status(pg.status, PACE_DEV_BAD_INDEX);
+    for (int i = 0; i < ITEMS; ++i) {
+      const int c = (i * LH + lane) * V;
 #pragma unroll
-      for (int i = 0; i < ITEMS; ++i) {
-        const int c = (i * LH + lane) * V;
-        if (!is_v && c < n) {
-          float wv[V];
-          Vec<float, V>::load(nw + c, wv);
+      for (int v = 0; v < V; ++v) y[i][v] = 0.f;
+      if (c >= n) continue;
+      auto tap = [&](int j, const float* wj) {
+        const int back = taps - 1 - j;
+        float x[V];
+        if (back <= k.local) Vec<T, V>::load(now - (int64_t)back * a.qkv_stride + c, x);
+        else if (back <= k.pos) Vec<float, V>::load(ring + (size_t)((k.pos - back) % a.ring_rows) * a.ring_stride + c, x);
+        else return;                                       // in front of the sequence
 #pragma unroll
-          for (int v = 0; v < V; ++v) y[i][v] *= f * wv[v];
-        } else {
+        for (int v = 0; v < V; ++v) y[i][v] = fmaf(wj[v], x[v], y[i][v]);
+        if (a.store_ring && back == 0) Vec<float, V>::store(ring + (size_t)(k.pos % a.ring_rows) * a.ring_stride + c, x);
+      };
+      if constexpr (NT > 0) {
 #pragma unroll
-          for (int v = 0; v < V; ++v) y[i][v] *= f;
+        for (int j = 0; j < NT; ++j) tap(j, w[j]);
+      } else {
+        for (int j = 0; j < taps; ++j) {
+          float wj[V];
+          Vec<float, V>::load(a.taps + (size_t)j * channels + ch0 + c, wj);
+          tap(j, wj);
         }
-        // the partner of an element lies in the same vector, or (V = 1) in the neighbouring lane
-        if constexpr (V == 1) {
-          const float other = __shfl_xor_sync(0xffffffffu, y[i][0], 1);
-          if (turns && (c >> 1) < a.rot_pairs && pos < a.table_rows) {
-            const float cs = a.cos_table[(size_t)pos * a.rot_pairs + (c >> 1)], sn = a.sin_table[(size_t)pos * a.rot_pairs + (c >> 1)];
-            y[i][0] = (c & 1) ? y[i][0] * cs + other * sn : y[i][0] * cs - other * sn;
-          }
-        } else if (turns && pos < a.table_rows) {
-#pragma unroll
-          for (int v = 0; v < V; v += 2) {
-            const int pr = (c + v) >> 1;
-            if (pr < a.rot_pairs) {
-              const float cs = a.cos_table[(size_t)pos * a.rot_pairs + pr], sn = a.sin_table[(size_t)pos * a.rot_pairs + pr];
-              const float u = y[i][v] * cs - y[i][v + 1] * sn;
-              y[i][v + 1] = y[i][v + 1] * cs + y[i][v] * sn;
-              y[i][v] = u;
-            }
-          }
-        }
-        if (dst && c < n) Vec<T, V>::store(dst + c, y[i]);
-      }
-      if (dst) {                                           // what a row has beyond its head size
-        float zero[V];
-#pragma unroll
-        for (int v = 0; v < V; ++v) zero[v] = 0.f;
-        for (int c = n + lane * V; c < row; c += LH * V) Vec<T, V>::store(dst + c, zero);
       }
     }
+    finish(r, y);
   }
 }
 
 template <typename T, int V, int LH, int ITEMS, int NT>
 int launch(const pace_step_t& st, const PageRows& pg, const pace_append_conv_args_t& a, int row, cudaStream_t s) {
-  const int heads = a.n_q_heads + 2 * pg.n_kv_heads, per = st.n_tokens >= 148 * kTokens ? kTokens : 1,
-            blocks = (st.n_tokens + per - 1) / per;
+  const int heads = a.n_q_heads + 2 * pg.n_kv_heads, per = st.n_tokens >= 148 * kTokens ? kTokens : st.n_tokens >= 148 ? 2 : 1;
   int threads = (heads * LH + 31) / 32 * 32;
   if (threads > kThreads) threads = kThreads;
-  int split = 1;                                            // few tokens: several blocks share their heads
-  while (blocks * split < 296 && split * threads < heads * LH && split < 64) split *= 2;
-  append_conv_kernel<T, V, LH, ITEMS, NT><<<dim3((unsigned)blocks, (unsigned)split), threads, 0, s>>>(st, pg, a, row, per);
+  const int groups = threads / LH, rounds = (heads + groups - 1) / groups;
+  if (rounds > 65535) return PACE_ERR_UNSUPPORTED;
+  const size_t smem = sizeof(float) * per * 2 * a.rot_pairs;
+  append_conv_kernel<T, V, LH, ITEMS, NT><<<dim3((unsigned)((st.n_tokens + per - 1) / per), (unsigned)rounds), threads, smem, s>>>(st, pg, a, row, per);
   PACE_LAUNCH_CHECK("append_conv_kernel");
   return PACE_OK;
 }

@@ -112,10 +112,10 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(pace_step_t st, pace_del
 
 // One token per entry.  A block owns 32 V value columns of one (entry, head), its state in registers (RW rows per warp): read
 // once, decayed, read out against the key, corrected, read out against the query, written once.
-constexpr int kStepWarps = 16;
+constexpr int kStepWarps = 8;
 
 template <typename T, int V, int RW>
-__global__ void __launch_bounds__(32 * kStepWarps) delta_step_kernel(pace_step_t st, pace_delta_args_t a) {
+__global__ void __launch_bounds__(32 * kStepWarps, RW * V <= 32 ? 4 : RW * V <= 64 ? 2 : 1) delta_step_kernel(pace_step_t st, pace_delta_args_t a) {
   __shared__ float qs[512], ks[512], gs[512], vs[32 * V], us[32 * V];
   __shared__ float part[kStepWarps][32 * V];
   __shared__ float unit[2];
@@ -244,19 +244,19 @@ int delta_seq(const pace_step_t& st, const pace_delta_args_t& a, cudaStream_t s)
 template <typename T, int V>
 int delta_step_v(const pace_step_t& st, const pace_delta_args_t& a, cudaStream_t s) {
   const dim3 grid((unsigned)((a.vdim + 32 * V - 1) / (32 * V)), (unsigned)a.heads, (unsigned)st.n_entries);
-  if (a.dim <= 2 * kStepWarps) delta_step_kernel<T, V, 2><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
-  else if (a.dim <= 4 * kStepWarps) delta_step_kernel<T, V, 4><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
+  if (a.dim <= 4 * kStepWarps) delta_step_kernel<T, V, 4><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
   else if (a.dim <= 8 * kStepWarps) delta_step_kernel<T, V, 8><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
   else if (a.dim <= 16 * kStepWarps) delta_step_kernel<T, V, 16><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
-  else delta_step_kernel<T, V, 32><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
+  else if (V == 1 && a.dim <= 32 * kStepWarps) delta_step_kernel<T, 1, 32><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
+  else if (V == 1) delta_step_kernel<T, 1, 64><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
+  else return PACE_ERR_UNSUPPORTED;
   PACE_LAUNCH_CHECK("delta_step_kernel");
   return PACE_OK;
 }
 
 template <typename T>
 int delta_step_t(const pace_step_t& st, const pace_delta_args_t& a, cudaStream_t s) {
-  if (a.dim <= 128 && a.vdim % 4 == 0 && a.vdim >= 128 && aligned16(a.s_state)) return delta_step_v<T, 4>(st, a, s);
-  if (a.dim <= 256 && a.vdim % 2 == 0 && a.vdim >= 64 && aligned16(a.s_state)) return delta_step_v<T, 2>(st, a, s);
+  if (a.dim <= 128 && a.vdim % 2 == 0 && a.vdim >= 64 && aligned16(a.s_state)) return delta_step_v<T, 2>(st, a, s);
   return delta_step_v<T, 1>(st, a, s);
 }
 

@@ -73,26 +73,39 @@ __global__ void __launch_bounds__(256) ssd_seq_kernel(pace_step_t st, pace_ssd_a
   }
 }
 
-// One token per entry: the block convolves what it needs of the projections, then the state is read and written once.  A
-// block owns 32 V value columns of one (entry, head); warp w takes rows w, w + 8, ...
-template <typename T, int V>
-__global__ void __launch_bounds__(256) ssd_step_kernel(pace_step_t st, pace_ssd_args_t a) {
-  __shared__ float bs[512], cs[512], xs[32 * V];
-  __shared__ float part[8][32 * V];
+// One token per entry: the state of V CL value columns of one (entry, head) is on its way to registers while the block convolves what
+// it needs of the projections; it is read and written once.  CL lanes share a row, a thread has rows tid / CL + k 256 / CL, k < RW.
+template <typename T, int V, int CL, int RW>
+__global__ void __launch_bounds__(256, RW * V <= 32 ? 4 : RW * V <= 64 ? 2 : 1) ssd_step_kernel(pace_step_t st, pace_ssd_args_t a) {
+  constexpr int COLS = V * CL, RG = 256 / CL;      // columns of the block, rows of a pass
+  __shared__ float bs[512], cs[512], xs[COLS];
+  __shared__ float part[8][COLS];
   const int e = blockIdx.z, h = blockIdx.y, N = a.state, vd = a.vdim, H = a.heads, per_g = H / a.groups, g = h / per_g;
-  const int inner = H * vd, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, col = (blockIdx.x * 32 + lane) * V, t = st.cu[e];
-  const int pos = st.start[e], channels = inner + 2 * a.groups * N, c0 = blockIdx.x * 32 * V;
+  const int inner = H * vd, tid = threadIdx.x, warp = tid >> 5, c0 = blockIdx.x * COLS, cl = tid % CL, col = c0 + cl * V, t = st.cu[e];
+  const int pos = st.start[e], channels = inner + 2 * a.groups * N, r0 = tid / CL;
+  float* state = a.s_state + ((size_t)st.slot[e] * H + h) * N * vd;
+  float S[RW][V];
+#pragma unroll
+  for (int k = 0; k < RW; ++k) {
+    const int r = r0 + k * RG;
+    if (pos != 0 && r < N && col < vd) Vec<float, V>::load(state + (size_t)r * vd + col, S[k]);
+    else
+#pragma unroll
+      for (int j = 0; j < V; ++j) S[k][j] = 0.f;
+  }
   const T* row = static_cast<const T*>(a.xbc) + (size_t)t * a.xbc_stride;
   float* ring = a.ring + (size_t)st.slot[e] * a.ring_rows * a.ring_stride;
-  float* state = a.s_state + ((size_t)st.slot[e] * H + h) * N * vd;
   const float dt = softplus(to_f<T>(static_cast<const T*>(a.dt_raw)[(size_t)t * a.dt_stride + h]) + a.dt_bias[h]);
   const float decay = exp_t<T>(a.neg_a[h] * dt);
   const int now_row = pos % a.ring_rows;
-  for (int i = threadIdx.x; i < 2 * N + 32 * V; i += 256) {
+  for (int i = tid; i < 2 * N + COLS; i += 256) {
     int ch;
     if (i < 2 * N) ch = inner + (i < N ? 0 : a.groups * N) + g * N + (i < N ? i : i - N);
     else if (c0 + i - 2 * N < vd) ch = h * vd + c0 + i - 2 * N;
-    else continue;
+    else {
+      xs[i - 2 * N] = 0.f;
+      continue;
+    }
     const float now = to_f<T>(row[ch]);
     float acc = a.conv_bias ? a.conv_bias[ch] : 0.f;
     for (int j = 0; j < a.n_taps; ++j) {
@@ -108,36 +121,32 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(pace_step_t st, pace_ssd_
     if (i >= 2 * N || (h == g * per_g && blockIdx.x == 0)) ring[(size_t)now_row * a.ring_stride + ch] = now;
   }
   __syncthreads();
-  const bool fresh = pos == 0;
   float x[V], o[V];
 #pragma unroll
-  for (int j = 0; j < V; ++j) {
-    x[j] = col + j < vd ? xs[lane * V + j] : 0.f;
-    o[j] = 0.f;
-  }
-  if (col < vd) {
-#pragma unroll 8
-    for (int r = warp; r < N; r += 8) {
-      float s[V];
-      if (fresh) {
+  for (int j = 0; j < V; ++j) x[j] = xs[cl * V + j], o[j] = 0.f;
 #pragma unroll
-        for (int j = 0; j < V; ++j) s[j] = 0.f;
-      } else {
-        Vec<float, V>::load(state + (size_t)r * vd + col, s);
-      }
+  for (int k = 0; k < RW; ++k) {
+    const int r = r0 + k * RG;
+    if (r < N && col < vd) {
       const float b = bs[r], c = cs[r];
 #pragma unroll
       for (int j = 0; j < V; ++j) {
-        s[j] = fmaf(decay, s[j], b * x[j]);
-        o[j] = fmaf(s[j], c, o[j]);
+        S[k][j] = fmaf(decay, S[k][j], b * x[j]);
+        o[j] = fmaf(S[k][j], c, o[j]);
       }
-      Vec<float, V>::store(state + (size_t)r * vd + col, s);
+      Vec<float, V>::store(state + (size_t)r * vd + col, S[k]);
     }
   }
 #pragma unroll
-  for (int j = 0; j < V; ++j) part[warp][lane * V + j] = o[j];
+  for (int w = CL; w < 32; w <<= 1)
+#pragma unroll
+    for (int j = 0; j < V; ++j) o[j] += __shfl_xor_sync(0xffffffffu, o[j], w);
+  if ((tid & 31) < CL) {
+#pragma unroll
+    for (int j = 0; j < V; ++j) part[warp][cl * V + j] = o[j];
+  }
   __syncthreads();
-  for (int i = threadIdx.x; i < 32 * V; i += 256) {
+  for (int i = tid; i < COLS; i += 256) {
     if (c0 + i >= vd) break;
     float s = a.d_skip[h] * xs[i];
 #pragma unroll
@@ -165,19 +174,27 @@ int ssd_seq(const pace_step_t& st, const pace_ssd_args_t& a, cudaStream_t s) {
   return launch_seq<T, 64>(st, a, s);
 }
 
-template <typename T, int V>
+template <typename T, int V, int CL>
 int launch_step(const pace_step_t& st, const pace_ssd_args_t& a, cudaStream_t s) {
-  const dim3 grid((unsigned)((a.vdim + 32 * V - 1) / (32 * V)), (unsigned)a.heads, (unsigned)st.n_entries);
-  ssd_step_kernel<T, V><<<grid, 256, 0, s>>>(st, a);
+  constexpr int RG = 256 / CL;
+  const dim3 grid((unsigned)((a.vdim + CL * V - 1) / (CL * V)), (unsigned)a.heads, (unsigned)st.n_entries);
+  if (a.state <= 4 * RG) ssd_step_kernel<T, V, CL, 4><<<grid, 256, 0, s>>>(st, a);
+  else if (a.state <= 8 * RG) ssd_step_kernel<T, V, CL, 8><<<grid, 256, 0, s>>>(st, a);
+  else if (a.state <= 16 * RG) ssd_step_kernel<T, V, CL, 16><<<grid, 256, 0, s>>>(st, a);
+  else if (V * CL <= 32) ssd_step_kernel<T, 1, 32, 64><<<grid, 256, 0, s>>>(st, a);
+  else return PACE_ERR_UNSUPPORTED;
   PACE_LAUNCH_CHECK("ssd_step_kernel");
   return PACE_OK;
 }
 
 template <typename T>
 int ssd_step_t(const pace_step_t& st, const pace_ssd_args_t& a, cudaStream_t s) {
-  if (a.vdim % 4 == 0 && a.vdim >= 128 && aligned16(a.s_state)) return launch_step<T, 4>(st, a, s);
-  if (a.vdim % 2 == 0 && a.vdim >= 64 && aligned16(a.s_state)) return launch_step<T, 2>(st, a, s);
-  return launch_step<T, 1>(st, a, s);
+  if (a.vdim % 4 == 0 && aligned16(a.s_state)) {
+    if (a.vdim > 64 && a.state <= 128) return launch_step<T, 4, 32>(st, a, s);
+    if (a.vdim > 32 && a.state <= 256) return launch_step<T, 4, 16>(st, a, s);
+    return launch_step<T, 4, 8>(st, a, s);      // (256 / 8 * 16 rows: any state up to 512)
+  }
+  return launch_step<T, 1, 32>(st, a, s);
 }
 
 bool ssd_ok(const pace_step_t* st, const pace_ssd_args_t* a) {
