@@ -45,7 +45,7 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(pace_step_t st, pace_del
         const float q = r < d ? to_f<T>(row[r]) : 0.f, k = r < d ? to_f<T>(row[(size_t)G * d + r]) : 0.f;
         qs[j * dp + r] = q;
         ks[j * dp + r] = k;
-        gs[j * dp + r] = r < d ? exp_t<T>(neg_a * softplus(to_f<T>(ar[r]) + a.dt_bias[(size_t)h * d + r])) : 1.f;
+        gs[j * dp + r] = r < d ? exp_t<T>(neg_a * softplus_t<T>(to_f<T>(ar[r]) + a.dt_bias[(size_t)h * d + r])) : 1.f;
         sq = fmaf(q, q, sq);
         sk = fmaf(k, k, sk);
       }
@@ -114,14 +114,32 @@ __global__ void __launch_bounds__(256) delta_seq_kernel(pace_step_t st, pace_del
 // once, decayed, read out against the key, corrected, read out against the query, written once.
 constexpr int kStepWarps = 8;
 
-template <typename T, int V, int RW>
-__global__ void __launch_bounds__(32 * kStepWarps, RW * V <= 32 ? 4 : RW * V <= 64 ? 2 : 1) delta_step_kernel(pace_step_t st, pace_delta_args_t a) {
+template <typename T, int V, int RW, int NT>
+__global__ void __launch_bounds__(32 * kStepWarps, RW * V <= 16 ? 4 : RW * V <= 32 ? 3 : RW * V <= 64 ? 2 : 1) delta_step_kernel(pace_step_t st, pace_delta_args_t a) {
   __shared__ float qs[512], ks[512], gs[512], vs[32 * V], us[32 * V];
   __shared__ float part[kStepWarps][32 * V];
   __shared__ float unit[2];
   const int d = a.dim, vd = a.vdim, H = a.heads, G = a.kv_heads, e = blockIdx.z, h = blockIdx.y, per_g = H / G, g = h / per_g;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, c0 = blockIdx.x * 32 * V, col = c0 + lane * V, t = st.cu[e];
   const int pos = st.start[e], slot = st.slot[e], channels = 2 * G * d + H * vd;
+  constexpr int THREADS = 32 * kStepWarps, AHEAD = 2;
+  const T* row = static_cast<const T*>(a.qkv) + (size_t)t * a.qkv_stride;
+  float* ring = a.ring + (size_t)slot * a.ring_rows * a.ring_stride;
+  const int total = 2 * d + 32 * V;
+  // the i-th channel the block needs (-1: none): q and k of the head, then its columns of v
+  auto channel = [&](int i) {
+    if (i < 2 * d) return (i < d ? 0 : G * d) + g * d + (i < d ? i : i - d);
+    return i < total && c0 + i - 2 * d < vd ? 2 * G * d + h * vd + c0 + i - 2 * d : -1;
+  };
+  ConvNow<T, NT> cv[AHEAD];
+#pragma unroll
+  for (int k = 0; k < AHEAD; ++k) {
+    const int ch = channel(tid + THREADS * k);
+    if (ch >= 0) cv[k].load(row, ring, a.ring_rows, a.ring_stride, a.taps, channels, a.n_taps, nullptr, pos, ch);
+  }
+  auto decay_in = [&](int r) { return to_f<T>(static_cast<const T*>(a.a_raw)[(size_t)t * a.a_stride + (size_t)h * d + r]) + a.dt_bias[(size_t)h * d + r]; };
+  const float first_decay = tid < d ? decay_in(tid) : 0.f, neg_a = a.neg_a[h];
+  const float beta_raw = to_f<T>(static_cast<const T*>(a.b_raw)[(size_t)t * a.b_stride + h]);
   float* state = a.s_state + ((size_t)slot * H + h) * d * vd;
   float S[RW][V];
 #pragma unroll
@@ -132,36 +150,29 @@ __global__ void __launch_bounds__(32 * kStepWarps, RW * V <= 32 ? 4 : RW * V <= 
 #pragma unroll
       for (int j = 0; j < V; ++j) S[i][j] = 0.f;
   }
-  const T* row = static_cast<const T*>(a.qkv) + (size_t)t * a.qkv_stride;
-  float* ring = a.ring + (size_t)slot * a.ring_rows * a.ring_stride;
   const int now_row = pos % a.ring_rows;
-  for (int i = tid; i < 2 * d + 32 * V; i += 32 * kStepWarps) {
-    int ch;
-    if (i < 2 * d) ch = (i < d ? 0 : G * d) + g * d + (i < d ? i : i - d);
-    else if (c0 + i - 2 * d < vd) ch = 2 * G * d + h * vd + c0 + i - 2 * d;
-    else {
-      vs[i - 2 * d] = 0.f;
-      continue;
+  auto convolved = [&](int i, int ch, const ConvNow<T, NT>& in) {
+    if (ch < 0) {
+      if (i < total) vs[i - 2 * d] = 0.f;
+      return;
     }
-    const float now = to_f<T>(row[ch]);
-    float acc = 0.f;
-    for (int j = 0; j < a.n_taps; ++j) {
-      const int back = a.n_taps - 1 - j;
-      if (back > pos) continue;
-      acc = fmaf(a.taps[(size_t)j * channels + ch], back ? ring[(size_t)((pos - back) % a.ring_rows) * a.ring_stride + ch] : now, acc);
-    }
-    const float y = round_to<T>(silu_t<T>(acc));
+    const float y = round_to<T>(silu_t<T>(in.sum(ring, a.ring_rows, a.ring_stride, a.taps, channels, a.n_taps, pos, ch)));
     if (i < d) qs[i] = y;
     else if (i < 2 * d) ks[i - d] = y;
     else vs[i - 2 * d] = y;
     // the current row's place is read by nobody in this launch; one block writes a channel
-    if (i >= 2 * d || (h == g * per_g && blockIdx.x == 0)) ring[(size_t)now_row * a.ring_stride + ch] = now;
+    if (i >= 2 * d || (h == g * per_g && blockIdx.x == 0)) ring[(size_t)now_row * a.ring_stride + ch] = in.now;
+  };
+#pragma unroll
+  for (int k = 0; k < AHEAD; ++k) convolved(tid + THREADS * k, channel(tid + THREADS * k), cv[k]);
+  for (int i = tid + THREADS * AHEAD; i < total; i += THREADS) {
+    const int ch = channel(i);
+    ConvNow<T, NT> in;
+    if (ch >= 0) in.load(row, ring, a.ring_rows, a.ring_stride, a.taps, channels, a.n_taps, nullptr, pos, ch);
+    convolved(i, ch, in);
   }
-  const float neg_a = a.neg_a[h];
-  for (int r = tid; r < d; r += 32 * kStepWarps)
-    gs[r] = exp_t<T>(neg_a * softplus(to_f<T>(static_cast<const T*>(a.a_raw)[(size_t)t * a.a_stride + (size_t)h * d + r]) +
-                                      a.dt_bias[(size_t)h * d + r]));
-  const float beta = sigmoid_t<T>(to_f<T>(static_cast<const T*>(a.b_raw)[(size_t)t * a.b_stride + h]));
+  for (int r = tid; r < d; r += THREADS) gs[r] = exp_t<T>(neg_a * softplus_t<T>(r == tid ? first_decay : decay_in(r)));
+  const float beta = sigmoid_t<T>(beta_raw);
   __syncthreads();
   if (warp < 2) {
     const float* x = warp ? ks : qs;
@@ -241,17 +252,22 @@ int delta_seq(const pace_step_t& st, const pace_delta_args_t& a, cudaStream_t s)
   return launch_seq<T, 16>(st, a, s);
 }
 
-template <typename T, int V>
-int delta_step_v(const pace_step_t& st, const pace_delta_args_t& a, cudaStream_t s) {
+template <typename T, int V, int NT>
+int delta_step_taps(const pace_step_t& st, const pace_delta_args_t& a, cudaStream_t s) {
   const dim3 grid((unsigned)((a.vdim + 32 * V - 1) / (32 * V)), (unsigned)a.heads, (unsigned)st.n_entries);
-  if (a.dim <= 4 * kStepWarps) delta_step_kernel<T, V, 4><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
-  else if (a.dim <= 8 * kStepWarps) delta_step_kernel<T, V, 8><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
-  else if (a.dim <= 16 * kStepWarps) delta_step_kernel<T, V, 16><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
-  else if (V == 1 && a.dim <= 32 * kStepWarps) delta_step_kernel<T, 1, 32><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
-  else if (V == 1) delta_step_kernel<T, 1, 64><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
+  if (a.dim <= 4 * kStepWarps) delta_step_kernel<T, V, 4, NT><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
+  else if (a.dim <= 8 * kStepWarps) delta_step_kernel<T, V, 8, NT><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
+  else if (a.dim <= 16 * kStepWarps) delta_step_kernel<T, V, 16, NT><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
+  else if (V == 1 && a.dim <= 32 * kStepWarps) delta_step_kernel<T, 1, 32, 0><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
+  else if (V == 1) delta_step_kernel<T, 1, 64, 0><<<grid, 32 * kStepWarps, 0, s>>>(st, a);
   else return PACE_ERR_UNSUPPORTED;
   PACE_LAUNCH_CHECK("delta_step_kernel");
   return PACE_OK;
+}
+
+template <typename T, int V>
+int delta_step_v(const pace_step_t& st, const pace_delta_args_t& a, cudaStream_t s) {
+  return a.n_taps == 4 ? delta_step_taps<T, V, 4>(st, a, s) : delta_step_taps<T, V, 0>(st, a, s);
 }
 
 template <typename T>

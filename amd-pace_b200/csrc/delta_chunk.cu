@@ -5,7 +5,7 @@
 //     A_ij = k_i . (k_j)^(G_i - G_j)  (j < i),   P_ij = q_i . (k_j)^(G_i - G_j)  (j <= i),   T = (1 + diag(beta) A)^-1 diag(beta)
 //     U = T V - (T K^(G)) S,     O = Q^(G) S + P U,     S' = S^(G_n) + (K^(G_n - G))^T U
 // Nothing but S connects the chunks, so a first launch makes everything else side by side, a block per (chunk, head, entry):
-// W = T K^(G), T V, Q^(G), K^(G_n - G) and P; a second one walks the chunks, a block per (entry, head, 16 or 32 value columns)
+// W = T K^(G), T V, Q^(G), K^(G_n - G) and P; a second one walks the chunks, a block per (entry, head, 16 to 64 value columns)
 // with its part of S in fp32 accumulators.
 //
 // e^(G_i - G_j) is the product of a row's factor e^(G_i - M) and a column's e^(M - G_j), M the sum up to the middle of the row's
@@ -19,7 +19,7 @@
 namespace pace {
 namespace {
 
-constexpr int kChunk = 64, kThreads = 256, kLP = kChunk + 4, kTP = kChunk + 8;
+constexpr int kChunk = 64, kThreads = 256, kWalkThreads = 512, kLP = kChunk + 8, kTP = kChunk + 8;
 constexpr float kRange = 86.0f;   // log2 units eight tokens may decay by on the fast path: e^60
 
 __device__ __forceinline__ void mma16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
@@ -41,6 +41,9 @@ __device__ __forceinline__ void ldsm4(uint32_t* r, const void* p) {
 __device__ __forceinline__ void ldsm4t(uint32_t* r, const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldsm2t(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)));
 }
 __device__ __forceinline__ void copy16(void* dst, const void* src, bool live = true) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
@@ -64,8 +67,10 @@ struct Slab {
 template <int DP>
 struct Prep {
   static constexpr int QP = DP + 8, GP = DP + 8;
+  static constexpr int kVMost = 128, VP = kVMost + 8;            // value columns that pass through shared memory
   static constexpr int kK = 0, kQ = kK + kChunk * QP * 2, kG = kQ + kChunk * QP * 2, kL = kG + kChunk * GP * 4,
-                       kT = kL + kChunk * kLP * 4, kVec = kT + 2 * kChunk * kTP * 2, bytes = kVec + (3 * kChunk + 4) * 4;
+                       kV = kL + kChunk * kLP * 4, kVec = kV + kChunk * VP * 2, bytes = kVec + (3 * kChunk + 4) * 4;
+  static_assert(kChunk * kLP * 4 >= 2 * kChunk * kTP * 2, "the halves of T take the place of L");
 };
 
 template <int DP>
@@ -82,8 +87,9 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
   __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(sm + PR::kQ);
   float* G = reinterpret_cast<float*>(sm + PR::kG);      // sums of log decays, log2 units
   float* L = reinterpret_cast<float*>(sm + PR::kL);      // diag(beta) A, then (1 + L)^-1 in its place
-  __nv_bfloat16* t_hi = reinterpret_cast<__nv_bfloat16*>(sm + PR::kT);
+  __nv_bfloat16* t_hi = reinterpret_cast<__nv_bfloat16*>(sm + PR::kL);   // at the end, in L's place
   __nv_bfloat16* t_lo = t_hi + kChunk * kTP;
+  __nv_bfloat16* vs = reinterpret_cast<__nv_bfloat16*>(sm + PR::kV);
   float* fk = reinterpret_cast<float*>(sm + PR::kVec);
   float* fq = fk + kChunk;
   float* beta = fq + kChunk;
@@ -99,6 +105,15 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
     const bool live = j < n_tok && c < d;
     copy16((which ? ks : qs) + j * QP + c, qkv + (live ? (size_t)j * a.qkv_stride + (size_t)(which * KV + kh) * d + c : 0), live);
   }
+  const bool v_here = vd <= PR::kVMost;
+  if (v_here) {
+    const int pieces = (vd + 15) / 16 * 2;                 // 16 bytes each, whole items of 16 columns
+    for (int i = tid; i < kChunk * pieces; i += kThreads) {
+      const int j = i / pieces, c = (i - j * pieces) * 8;
+      const bool live = j < n_tok && c < vd;
+      copy16(vs + j * PR::VP + c, qkv + (live ? (size_t)j * a.qkv_stride + 2 * (size_t)KV * d + (size_t)h * vd + c : 0), live);
+    }
+  }
   asm volatile("cp.async.commit_group;" ::: "memory");
   if (tid < 4) slow[tid] = 0;
   if (tid < kChunk)
@@ -113,7 +128,7 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
       if (j < n_tok && c < d) {
         const float2 x = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ar + (size_t)j * a.a_stride + c));
         const float2 b = *reinterpret_cast<const float2*>(a.dt_bias + (size_t)h * d + c);
-        v = make_float2(neg_a * softplus(x.x + b.x), neg_a * softplus(x.y + b.y));
+        v = make_float2(neg_a * softplus_fast(x.x + b.x), neg_a * softplus_fast(x.y + b.y));
       }
       *reinterpret_cast<float2*>(G + j * GP + c) = v;
     }
@@ -128,19 +143,20 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
 #pragma unroll 8
     for (int j = part * ROWS; j < (part + 1) * ROWS; ++j) G[j * GP + gc] = s += G[j * GP + gc];
   }
-  for (int j = warp * 8; j < warp * 8 + 8; ++j) {
+  {
+    const int j = tid >> 2;                                // four threads a token
     float sq = 0.f, sk = 0.f;
-    for (int c = lane * 2; c < DP; c += 64) {
+    for (int c = (tid & 3) * 2; c < DP; c += 8) {
       const float2 x = bf2_to_f2(*reinterpret_cast<const uint32_t*>(qs + j * QP + c)), y = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ks + j * QP + c));
       sq = fmaf(x.x, x.x, fmaf(x.y, x.y, sq));
       sk = fmaf(y.x, y.x, fmaf(y.y, y.y, sk));
     }
 #pragma unroll
-    for (int o = 16; o; o >>= 1) {
+    for (int o = 2; o; o >>= 1) {
       sq += __shfl_xor_sync(0xffffffffu, sq, o);
       sk += __shfl_xor_sync(0xffffffffu, sk, o);
     }
-    if (lane == 0) {
+    if ((tid & 3) == 0) {
       fq[j] = a.q_scale / sqrtf(sq + a.unit_eps);
       fk[j] = 1.0f / sqrtf(sk + a.unit_eps);
     }
@@ -239,22 +255,27 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
     p_hi[i * kChunk + j] = hi;
     p_lo[i * kChunk + j] = __float2bfloat16_rn(p - __bfloat162float(hi));
   }
-  // ---- queries and keys with their decays ----
+  __syncthreads();
+  // ---- queries and keys with their decays; the halves of K^(G) take the places of the keys and the queries ----
   for (int i = tid; i < kChunk * (DP / 2); i += kThreads) {
     const int j = i / (DP / 2), c = (i - j * (DP / 2)) * 2;
     const float2 gg = *reinterpret_cast<const float2*>(G + j * GP + c), ge = *reinterpret_cast<const float2*>(G + (kChunk - 1) * GP + c);
-    const float2 kk = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ks + j * QP + c));
-    const float2 qq = bf2_to_f2(*reinterpret_cast<const uint32_t*>(qs + j * QP + c));
+    uint32_t* kp = reinterpret_cast<uint32_t*>(ks + j * QP + c);
+    uint32_t* qp = reinterpret_cast<uint32_t*>(qs + j * QP + c);
+    const float2 kk = bf2_to_f2(*kp), qq = bf2_to_f2(*qp);
+    const float e0 = fast_exp2(gg.x), e1 = fast_exp2(gg.y), k0 = kk.x * fk[j], k1 = kk.y * fk[j], f = fq[j];
     uint32_t hi, lo;
-    split_bf2(qq.x * fq[j] * fast_exp2(gg.x), qq.y * fq[j] * fast_exp2(gg.y), hi, lo);
+    split_bf2(qq.x * f * e0, qq.y * f * e1, hi, lo);
     reinterpret_cast<uint32_t*>(tiles + SL::kQ)[i] = hi;
     reinterpret_cast<uint32_t*>(tiles + SL::kQ + SL::kTile)[i] = lo;
-    split_bf2(kk.x * fk[j] * fast_exp2(ge.x - gg.x), kk.y * fk[j] * fast_exp2(ge.y - gg.y), hi, lo);
+    split_bf2(k0 * fast_exp2(ge.x - gg.x), k1 * fast_exp2(ge.y - gg.y), hi, lo);
     reinterpret_cast<uint32_t*>(tiles + SL::kK)[i] = hi;
     reinterpret_cast<uint32_t*>(tiles + SL::kK + SL::kTile)[i] = lo;
+    split_bf2(k0 * e0, k1 * e1, hi, lo);
+    *kp = hi;
+    *qp = lo;
   }
   if (tid < DP) reinterpret_cast<float*>(slot + SL::kDecay)[tid] = fast_exp2(G[(kChunk - 1) * GP + tid]);
-  __syncthreads();
 
   // ---- (1 + L)^-1 in place of L: blocks of 16, then of 32, then of 64 ----
   {
@@ -275,41 +296,51 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
       for (int i = 0; i < 16; ++i) L[(16 * b + i) * kLP + 16 * b + col] = x[i];
     }
     __syncthreads();
-    // lower left block of a pair: -T_bb (L_ba T_aa)
+    // lower left block of a pair: -T_bb (L_ba T_aa); a thread's outputs lie in one column of one pair
     auto combine = [&](auto size_c) {
-      constexpr int N = decltype(size_c)::value, PAIRS = kChunk / (2 * N), PER = PAIRS * N * N / kThreads;
-      float y[PER];
+      constexpr int N = decltype(size_c)::value, PAIRS = kChunk / (2 * N), PER = PAIRS * N * N / kThreads, RS = kThreads / (PAIRS * N);
+      const int pr = tid / (kThreads / PAIRS), at = 2 * N * pr, j = tid % N, i0 = tid % (kThreads / PAIRS) / N;
 #pragma unroll
       for (int step = 0; step < 2; ++step) {
+        const float* rows = L + (at + N + i0) * kLP + at + (step ? N : 0);            // of L_ba, then of T_bb
+        const float* cols = L + (at + (step ? N : 0)) * kLP + at + j;                 // of T_aa, then of the product
+        float y[PER];
 #pragma unroll
-        for (int k = 0; k < PER; ++k) {
-          const int o = k * kThreads + tid, pr = o / (N * N), i = (o - pr * N * N) / N, j = o % N, at = 2 * N * pr;
-          const float *row, *colp;
-          if (step == 0) row = L + (at + N + i) * kLP + at, colp = L + at * kLP + at + j;               // L_ba, T_aa
-          else row = L + (at + N + i) * kLP + at + N, colp = L + (at + N) * kLP + at + j;               // T_bb, the product
-          float s = 0.f;
+        for (int k = 0; k < PER; ++k) y[k] = 0.f;
 #pragma unroll
-          for (int x2 = 0; x2 < N; ++x2) s = fmaf(row[x2], colp[x2 * kLP], s);
-          y[k] = step ? -s : s;
+        for (int x = 0; x < N; x += 4) {
+          float c[4];
+#pragma unroll
+          for (int u = 0; u < 4; ++u) c[u] = cols[(x + u) * kLP];
+#pragma unroll
+          for (int k = 0; k < PER; ++k) {
+            const float4 r = *reinterpret_cast<const float4*>(rows + k * RS * kLP + x);
+            y[k] = fmaf(r.x, c[0], fmaf(r.y, c[1], fmaf(r.z, c[2], fmaf(r.w, c[3], y[k]))));
+          }
         }
         __syncthreads();
 #pragma unroll
-        for (int k = 0; k < PER; ++k) {
-          const int o = k * kThreads + tid, pr = o / (N * N), i = (o - pr * N * N) / N, j = o % N, at = 2 * N * pr;
-          L[(at + N + i) * kLP + at + j] = y[k];
-        }
+        for (int k = 0; k < PER; ++k) L[(at + N + i0 + k * RS) * kLP + at + j] = step ? -y[k] : y[k];
         __syncthreads();
       }
     };
     combine(std::integral_constant<int, 16>());
     combine(std::integral_constant<int, 32>());
   }
-  for (int i = tid; i < kChunk * kChunk / 2; i += kThreads) {
-    const int r = i / (kChunk / 2), c = (i - r * (kChunk / 2)) * 2;
-    uint32_t hi, lo;
-    split_bf2(L[r * kLP + c] * beta[c], L[r * kLP + c + 1] * beta[c + 1], hi, lo);
-    *reinterpret_cast<uint32_t*>(t_hi + r * kTP + c) = hi;
-    *reinterpret_cast<uint32_t*>(t_lo + r * kTP + c) = lo;
+  {
+    uint32_t hi[kChunk * kChunk / 2 / kThreads], lo[kChunk * kChunk / 2 / kThreads];
+#pragma unroll
+    for (int k = 0; k < kChunk * kChunk / 2 / kThreads; ++k) {
+      const int i = k * kThreads + tid, r = i / (kChunk / 2), c = (i - r * (kChunk / 2)) * 2;
+      split_bf2(L[r * kLP + c] * beta[c], L[r * kLP + c + 1] * beta[c + 1], hi[k], lo[k]);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kChunk * kChunk / 2 / kThreads; ++k) {
+      const int i = k * kThreads + tid, r = i / (kChunk / 2), c = (i - r * (kChunk / 2)) * 2;
+      *reinterpret_cast<uint32_t*>(t_hi + r * kTP + c) = hi[k];
+      *reinterpret_cast<uint32_t*>(t_lo + r * kTP + c) = lo[k];
+    }
   }
   __syncthreads();
 
@@ -327,23 +358,19 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
         for (int x = 0; x < 4; ++x) acc[m][s][x] = 0.f;
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt) {
-      uint32_t bh[2][2], bl[2][2];
+      uint32_t bh[4], bl[4];
+      if (is_w) {
+        ldsm4t(bh, ks + (16 * kt + (lane & 15)) * QP + n0 + (lane >> 4) * 8);
+        ldsm4t(bl, qs + (16 * kt + (lane & 15)) * QP + n0 + (lane >> 4) * 8);
+      } else if (v_here) {
+        ldsm4t(bh, vs + (16 * kt + (lane & 15)) * PR::VP + n0 + (lane >> 4) * 8);
+      } else {
 #pragma unroll
-      for (int s = 0; s < 2; ++s) {
-        const int c = n0 + 8 * s + g;
-#pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          const int j = 16 * kt + 2 * t + 8 * x;
-          if (is_w) {
-            const float v0 = __bfloat162float(ks[j * QP + c]) * fk[j] * fast_exp2(G[j * GP + c]);
-            const float v1 = __bfloat162float(ks[(j + 1) * QP + c]) * fk[j + 1] * fast_exp2(G[(j + 1) * GP + c]);
-            split_bf2(v0, v1, bh[s][x], bl[s][x]);
-          } else {
-            const unsigned short* v = reinterpret_cast<const unsigned short*>(qkv) + (size_t)j * a.qkv_stride + 2 * (size_t)KV * d + (size_t)h * vd + c;
-            const uint32_t lo16 = j < n_tok && c < vd ? v[0] : 0, hi16 = j + 1 < n_tok && c < vd ? v[a.qkv_stride] : 0;
-            bh[s][x] = lo16 | (hi16 << 16);
-            bl[s][x] = 0;
-          }
+        for (int x = 0; x < 4; ++x) {
+          const int c = n0 + 8 * (x >> 1) + g, j = 16 * kt + 2 * t + 8 * (x & 1);
+          const unsigned short* v = reinterpret_cast<const unsigned short*>(qkv) + (size_t)j * a.qkv_stride + 2 * (size_t)KV * d + (size_t)h * vd + c;
+          const uint32_t lo16 = j < n_tok && c < vd ? v[0] : 0, hi16 = j + 1 < n_tok && c < vd ? v[a.qkv_stride] : 0;
+          bh[x] = lo16 | (hi16 << 16);
         }
       }
 #pragma unroll
@@ -353,9 +380,9 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
         ldsm4(al, t_lo + (16 * m + (lane & 15)) * kTP + 16 * kt + (lane >> 4) * 8);
 #pragma unroll
         for (int s = 0; s < 2; ++s) {
-          mma16816(acc[m][s], ah, bh[s][0], bh[s][1]);
-          mma16816(acc[m][s], al, bh[s][0], bh[s][1]);
-          if (is_w) mma16816(acc[m][s], ah, bl[s][0], bl[s][1]);
+          mma16816(acc[m][s], ah, bh[2 * s], bh[2 * s + 1]);
+          mma16816(acc[m][s], al, bh[2 * s], bh[2 * s + 1]);
+          if (is_w) mma16816(acc[m][s], ah, bl[2 * s], bl[2 * s + 1]);
         }
       }
     }
@@ -385,12 +412,14 @@ struct Walk {
                        kU = kS + 2 * DP * VP, kEnd = kU + 2 * kChunk * VP, bytes = kEnd * 2;
 };
 
+// Sixteen warps: the products with the state's halves are 16 rows (of W: warps 0 .. 3 of eight, of Q: 4 .. 7) x half of the
+// columns, the state's tile 16 rows x SC columns.  The three terms of a split product have accumulators of their own.
 template <int DP, int VB>
-__global__ void __launch_bounds__(kThreads, 1) delta_walk_kernel(pace_step_t st, pace_delta_args_t a, Slab sl) {
+__global__ void __launch_bounds__(kWalkThreads, 1) delta_walk_kernel(pace_step_t st, pace_delta_args_t a, Slab sl) {
   using SL = Slot<DP>;
   using WK = Walk<DP, VB>;
-  constexpr int QP = WK::QP, VP = WK::VP, NT = VB / 8;
-  constexpr int RG = DP / 16, CG = 8 / RG, SC = VB / CG, NS = SC / 8;   // state tile of a warp: 16 rows x SC columns
+  constexpr int QP = WK::QP, VP = WK::VP, NT = VB / 16;                  // tiles of 8 columns a warp has of the token rows
+  constexpr int RG = DP / 16, CG = 16 / RG, SC = VB / CG, NS = SC / 8;   // and of the state
   static_assert(NS >= 1, "a warp owns eight columns of the state at least");
   const int e = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * VB, d = a.dim, vd = a.vdim, H = a.heads;
   const int count = st.cu[e + 1] - st.cu[e], chunks = min(sl.n, (count + kChunk - 1) / kChunk - sl.first);
@@ -403,7 +432,8 @@ __global__ void __launch_bounds__(kThreads, 1) delta_walk_kernel(pace_step_t st,
   auto fetch = [&](const unsigned char* from, int first_tile, int n_tiles) {   // [64][DP] tiles into rows of QP
     const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(from) + first_tile * SL::kTile;
     __nv_bfloat16* dst = sb + first_tile * kChunk * QP;
-    for (int i = tid; i < n_tiles * SL::kTile / 8; i += kThreads) {
+#pragma unroll 4
+    for (int i = tid; i < n_tiles * SL::kTile / 8; i += kWalkThreads) {
       const int r = i / (DP / 8), c = (i - r * (DP / 8)) * 8;
       copy16(dst + r * QP + c, src + (size_t)r * DP + c);
     }
@@ -415,7 +445,8 @@ __global__ void __launch_bounds__(kThreads, 1) delta_walk_kernel(pace_step_t st,
   auto fetch_kp = [&](const unsigned char* from) {
     fetch(from, 4, 2);
     const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(from) + SL::kP;
-    for (int i = tid; i < 2 * kChunk * kChunk / 8; i += kThreads) {
+#pragma unroll
+    for (int i = tid; i < 2 * kChunk * kChunk / 8; i += kWalkThreads) {
       const int r = i / (kChunk / 8), c = (i - r * (kChunk / 8)) * 8;
       copy16(sb + WK::kP + r * kTP + c, src + r * kChunk + c);
     }
@@ -424,7 +455,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_walk_kernel(pace_step_t st,
   fetch_wq(slot);
   float* state = a.s_state + ((size_t)st.slot[e] * H + h) * d * vd;
   const bool fresh = st.start[e] == 0 && sl.first == 0;
-  const int sr = (warp % RG) * 16 + g, sc = (warp / RG) * SC + 2 * t;
+  const int m0 = (warp % RG) * 16, c0 = (warp / RG) * SC, sr = m0 + g, sc = c0 + 2 * t;
   float S[NS][4];
 #pragma unroll
   for (int n = 0; n < NS; ++n)
@@ -446,110 +477,123 @@ __global__ void __launch_bounds__(kThreads, 1) delta_walk_kernel(pace_step_t st,
         *reinterpret_cast<uint32_t*>(s_lo + (sr + 8 * x) * VP + sc + 8 * n) = lo;
       }
   };
+  // acc += (ah + al) (bh + bl) for N tiles of 8 columns of a [k][VP] operand; the cross terms go to x1, x2
+  auto product = [&](auto n_c, float (*acc)[4], float (*x1)[4], float (*x2)[4], const uint32_t* ah, const uint32_t* al,
+                     const __nv_bfloat16* hi, const __nv_bfloat16* lo) {
+    constexpr int N = decltype(n_c)::value;
+    if constexpr (N == 1) {
+      uint32_t bh[2], bl[2];
+      ldsm2t(bh, hi + (lane & 15) * VP);
+      ldsm2t(bl, lo + (lane & 15) * VP);
+      mma16816(acc[0], ah, bh[0], bh[1]);
+      mma16816(x1[0], ah, bl[0], bl[1]);
+      mma16816(x2[0], al, bh[0], bh[1]);
+    } else {
+#pragma unroll
+      for (int n = 0; n < N; n += 2) {
+        uint32_t bh[4], bl[4];
+        ldsm4t(bh, hi + (lane & 15) * VP + n * 8 + (lane >> 4) * 8);
+        ldsm4t(bl, lo + (lane & 15) * VP + n * 8 + (lane >> 4) * 8);
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          mma16816(acc[n + u], ah, bh[2 * u], bh[2 * u + 1]);
+          mma16816(x1[n + u], ah, bl[2 * u], bl[2 * u + 1]);
+          mma16816(x2[n + u], al, bh[2 * u], bh[2 * u + 1]);
+        }
+      }
+    }
+  };
   put_state();
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
+  const int wm = warp & 7, n0 = (warp >> 3) * (VB / 2), row = (wm & 3) * 16 + g;   // token rows and columns of this warp
   for (int c = 0; c < chunks; ++c, slot += (size_t)H * slot_bytes) {
     fetch_kp(slot);
     const int l0 = (sl.first + c) * kChunk, n_tok = min(kChunk, count - l0);
     const float* decay = reinterpret_cast<const float*>(slot + SL::kDecay);
     const float d0 = decay[sr], d1 = decay[sr + 8];
-    const int row = (warp & 3) * 16 + g;                       // of the tokens, for warps 0 .. 3 (W) and 4 .. 7 (Q)
     float uv[NT][4];
-    if (warp < 4) {
+    if (wm < 4) {
 #pragma unroll
       for (int n = 0; n < NT; ++n)
 #pragma unroll
         for (int x = 0; x < 2; ++x) {
-          const int col = v0 + 8 * n + 2 * t;
+          const int col = v0 + n0 + 8 * n + 2 * t;
           const float2 v = col < vd ? *reinterpret_cast<const float2*>(slot + SL::kUv + ((size_t)(row + 8 * x) * vd + col) * 4) : make_float2(0.f, 0.f);
           uv[n][2 * x] = v.x;
           uv[n][2 * x + 1] = v.y;
         }
     }
     // ---- what the state answers to the keys (W S) and the queries ----
-    float acc[NT][4];
+    float acc[NT][4], x1[NT][4], x2[NT][4];
 #pragma unroll
-    for (int n = 0; n < NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) acc[n][x] = x1[n][x] = x2[n][x] = 0.f;
     {
-      const __nv_bfloat16* ah_p = sb + (warp < 4 ? WK::kW : WK::kQ) + ((warp & 3) * 16 + (lane & 15)) * QP + (lane >> 4) * 8;
+      const __nv_bfloat16* ap = sb + (wm < 4 ? WK::kW : WK::kQ) + ((wm & 3) * 16 + (lane & 15)) * QP + (lane >> 4) * 8;
 #pragma unroll
       for (int k0 = 0; k0 < DP; k0 += 16) {
         uint32_t ah[4], al[4];
-        ldsm4(ah, ah_p + k0);
-        ldsm4(al, ah_p + kChunk * QP + k0);
-#pragma unroll
-        for (int n = 0; n < NT; n += 2) {
-          uint32_t bh[4], bl[4];
-          ldsm4t(bh, s_hi + (k0 + (lane & 15)) * VP + n * 8 + (lane >> 4) * 8);
-          ldsm4t(bl, s_lo + (k0 + (lane & 15)) * VP + n * 8 + (lane >> 4) * 8);
-          mma_split(acc[n], ah, al, bh, bl);
-          mma_split(acc[n + 1], ah, al, bh + 2, bl + 2);
-        }
+        ldsm4(ah, ap + k0);
+        ldsm4(al, ap + kChunk * QP + k0);
+        product(std::integral_constant<int, NT>(), acc, x1, x2, ah, al, s_hi + k0 * VP + n0, s_lo + k0 * VP + n0);
       }
     }
-    if (warp < 4) {
+    if (wm < 4) {
 #pragma unroll
       for (int n = 0; n < NT; ++n)
 #pragma unroll
         for (int x = 0; x < 2; ++x) {
           uint32_t hi, lo;
-          split_bf2(uv[n][2 * x] - acc[n][2 * x], uv[n][2 * x + 1] - acc[n][2 * x + 1], hi, lo);
-          *reinterpret_cast<uint32_t*>(u_hi + (row + 8 * x) * VP + 8 * n + 2 * t) = hi;
-          *reinterpret_cast<uint32_t*>(u_lo + (row + 8 * x) * VP + 8 * n + 2 * t) = lo;
+          split_bf2(uv[n][2 * x] - (acc[n][2 * x] + (x1[n][2 * x] + x2[n][2 * x])),
+                    uv[n][2 * x + 1] - (acc[n][2 * x + 1] + (x1[n][2 * x + 1] + x2[n][2 * x + 1])), hi, lo);
+          *reinterpret_cast<uint32_t*>(u_hi + (row + 8 * x) * VP + n0 + 8 * n + 2 * t) = hi;
+          *reinterpret_cast<uint32_t*>(u_lo + (row + 8 * x) * VP + n0 + 8 * n + 2 * t) = lo;
         }
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                           // U, K and P are there; W, Q and the state have been read
     if (c + 1 < chunks) fetch_wq(slot + (size_t)H * slot_bytes);
     // ---- the state behind the chunk ----
+    float y1[NS][4], y2[NS][4];
 #pragma unroll
     for (int n = 0; n < NS; ++n) {
       S[n][0] *= d0; S[n][1] *= d0;
       S[n][2] *= d1; S[n][3] *= d1;
-    }
-    {
-      const int m0 = (warp % RG) * 16, c0 = (warp / RG) * SC;
 #pragma unroll
-      for (int k0 = 0; k0 < kChunk; k0 += 16) {
-        uint32_t ah[4], al[4];
-        const __nv_bfloat16* kp = sb + WK::kK + (k0 + (lane & 7) + (lane >> 4) * 8) * QP + m0 + ((lane >> 3) & 1) * 8;
-        ldsm4t(ah, kp);
-        ldsm4t(al, kp + kChunk * QP);
-#pragma unroll
-        for (int n = 0; n < NS; n += 2) {
-          uint32_t bh[4], bl[4];   // (with one tile of eight columns the second one is read and not used)
-          ldsm4t(bh, u_hi + (k0 + (lane & 15)) * VP + c0 + n * 8 + (lane >> 4) * 8);
-          ldsm4t(bl, u_lo + (k0 + (lane & 15)) * VP + c0 + n * 8 + (lane >> 4) * 8);
-          mma_split(S[n], ah, al, bh, bl);
-          if (n + 1 < NS) mma_split(S[n + 1 < NS ? n + 1 : n], ah, al, bh + 2, bl + 2);
-        }
-      }
+      for (int x = 0; x < 4; ++x) y1[n][x] = y2[n][x] = 0.f;
     }
+#pragma unroll
+    for (int k0 = 0; k0 < kChunk; k0 += 16) {
+      uint32_t ah[4], al[4];
+      const __nv_bfloat16* kp = sb + WK::kK + (k0 + (lane & 7) + (lane >> 4) * 8) * QP + m0 + ((lane >> 3) & 1) * 8;
+      ldsm4t(ah, kp);
+      ldsm4t(al, kp + kChunk * QP);
+      product(std::integral_constant<int, NS>(), S, y1, y2, ah, al, u_hi + k0 * VP + c0, u_lo + k0 * VP + c0);
+    }
+#pragma unroll
+    for (int n = 0; n < NS; ++n)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) S[n][x] += y1[n][x] + y2[n][x];
     put_state();
-    if (warp >= 4) {
-      const int m = warp - 4;
+    if (wm >= 4) {
+      const int m = wm - 4;
       for (int kt = 0; kt <= m; ++kt) {
         uint32_t ah[4], al[4];
         const __nv_bfloat16* pp = sb + WK::kP + (16 * m + (lane & 15)) * kTP + 16 * kt + (lane >> 4) * 8;
         ldsm4(ah, pp);
         ldsm4(al, pp + kChunk * kTP);
-#pragma unroll
-        for (int n = 0; n < NT; n += 2) {
-          uint32_t bh[4], bl[4];
-          ldsm4t(bh, u_hi + (16 * kt + (lane & 15)) * VP + n * 8 + (lane >> 4) * 8);
-          ldsm4t(bl, u_lo + (16 * kt + (lane & 15)) * VP + n * 8 + (lane >> 4) * 8);
-          mma_split(acc[n], ah, al, bh, bl);
-          mma_split(acc[n + 1], ah, al, bh + 2, bl + 2);
-        }
+        product(std::integral_constant<int, NT>(), acc, x1, x2, ah, al, u_hi + 16 * kt * VP + n0, u_lo + 16 * kt * VP + n0);
       }
-      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (size_t)(st.cu[e] + l0) * a.out_stride + (size_t)h * vd + v0;
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (size_t)(st.cu[e] + l0) * a.out_stride + (size_t)h * vd + v0 + n0;
 #pragma unroll
       for (int n = 0; n < NT; ++n)
 #pragma unroll
         for (int x = 0; x < 2; ++x)
-          if (row + 8 * x < n_tok && v0 + 8 * n + 2 * t < vd)
-            *reinterpret_cast<uint32_t*>(out + (size_t)(row + 8 * x) * a.out_stride + 8 * n + 2 * t) = f2_to_bf2(acc[n][2 * x], acc[n][2 * x + 1]);
+          if (row + 8 * x < n_tok && v0 + n0 + 8 * n + 2 * t < vd)
+            *reinterpret_cast<uint32_t*>(out + (size_t)(row + 8 * x) * a.out_stride + 8 * n + 2 * t) =
+                f2_to_bf2(acc[n][2 * x] + (x1[n][2 * x] + x2[n][2 * x]), acc[n][2 * x + 1] + (x1[n][2 * x + 1] + x2[n][2 * x + 1]));
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                           // the next W and Q and the state are there; K, P and U have been read
@@ -584,7 +628,7 @@ template <int DP, int VB>
 int launch_walk(const pace_step_t& st, const pace_delta_args_t& a, const Slab& sl, cudaStream_t s) {
   PACE_CUDA_TRY(cudaFuncSetAttribute(delta_walk_kernel<DP, VB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Walk<DP, VB>::bytes));
   const dim3 grid((unsigned)((a.vdim + VB - 1) / VB), (unsigned)a.heads, (unsigned)st.n_entries);
-  delta_walk_kernel<DP, VB><<<grid, kThreads, Walk<DP, VB>::bytes, s>>>(st, a, sl);
+  delta_walk_kernel<DP, VB><<<grid, kWalkThreads, Walk<DP, VB>::bytes, s>>>(st, a, sl);
   PACE_LAUNCH_CHECK("delta_walk_kernel");
   return PACE_OK;
 }
@@ -594,7 +638,8 @@ int launch_chunked(const pace_step_t& st, const pace_delta_args_t& a, const Plan
   PACE_CUDA_TRY(cudaFuncSetAttribute(delta_prepare_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Prep<DP>::bytes));
   const int chunks = (st.max_count + kChunk - 1) / kChunk;
   // few sequences and heads: narrow columns, so that more SMs take part
-  const bool narrow = (int64_t)st.n_entries * a.heads * ((a.vdim + 31) / 32) <= 74;
+  constexpr int WIDE = DP == 64 ? 64 : 32;
+  const bool narrow = (int64_t)st.n_entries * a.heads * ((a.vdim + WIDE - 1) / WIDE) <= 74;
   for (int c = 0; c < chunks; c += p.slab) {
     Slab sl;
     sl.scratch = static_cast<unsigned char*>(a.workspace);
@@ -603,7 +648,7 @@ int launch_chunked(const pace_step_t& st, const pace_delta_args_t& a, const Plan
     const int n = chunks - c < p.slab ? chunks - c : p.slab;
     delta_prepare_kernel<DP><<<dim3((unsigned)n, (unsigned)a.heads, (unsigned)st.n_entries), kThreads, Prep<DP>::bytes, s>>>(st, a, sl);
     PACE_LAUNCH_CHECK("delta_prepare_kernel");
-    const int rc = narrow ? launch_walk<DP, 16>(st, a, sl, s) : launch_walk<DP, 32>(st, a, sl, s);
+    const int rc = narrow ? launch_walk<DP, WIDE / 2>(st, a, sl, s) : launch_walk<DP, WIDE>(st, a, sl, s);
     if (rc != PACE_OK) return rc;
   }
   return PACE_OK;

@@ -95,6 +95,23 @@ template <typename T> __device__ __forceinline__ float gelu_tanh_t(float z) {
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
 // ln(1 + e^x), with a relative error of a few ulp at both ends
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// the same with the hardware's exponential and reciprocal: ln(1 + u) = 2 artanh(u / (2 + u)), whose argument is at most 1/3 (the
+// first term left out is below 1e-8 of the sum)
+__device__ __forceinline__ float softplus_fast(float x) {
+  const float u = fast_exp2(-fabsf(x) * kLog2e);
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(2.0f + u));
+  const float s = u * r, q = s * s;
+  float p = fmaf(q, 1.0f / 13, 1.0f / 11);
+  p = fmaf(p, q, 1.0f / 9);
+  p = fmaf(p, q, 1.0f / 7);
+  p = fmaf(p, q, 1.0f / 5);
+  p = fmaf(p, q, 1.0f / 3);
+  p = fmaf(p, q, 1.0f);
+  return fmaf(2.0f * s, p, fmaxf(x, 0.f));
+}
+template <typename T> __device__ __forceinline__ float softplus_t(float x) { return softplus_fast(x); }
+template <> __device__ __forceinline__ float softplus_t<float>(float x) { return softplus(x); }
 template <typename T> __device__ __forceinline__ float act_t(int act, float z) {
   return act == PACE_ACT_SILU ? silu_t<T>(z) : act == PACE_ACT_GELU_TANH ? gelu_tanh_t<T>(z) : act == PACE_ACT_GELU_ERF ? gelu_erf(z) : z;
 }
@@ -126,6 +143,39 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   for (int w = 0; w < warps; ++w) s += red[w];
   return s;
 }
+
+// One channel of a short convolution for the one new token of a sequence: its inputs are asked for by load() and used by sum().
+// NT: taps where known at compile time, else 0 (the inputs are then fetched by sum()).
+template <typename T, int NT> struct ConvNow {
+  float now, x[NT ? NT : 1], w[NT ? NT : 1], bias;
+  __device__ __forceinline__ void load(const T* row, const float* ring, int ring_rows, int64_t ring_stride, const float* taps, int channels,
+                                       int n_taps, const float* b, int pos, int ch) {
+    now = to_f<T>(row[ch]);
+    bias = b ? b[ch] : 0.f;
+    if constexpr (NT > 0) {
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        w[j] = taps[(size_t)j * channels + ch];
+        if (j < NT - 1) x[j] = pos >= NT - 1 - j ? ring[(size_t)((pos - (NT - 1 - j)) % ring_rows) * ring_stride + ch] : 0.f;
+      }
+    }
+  }
+  __device__ __forceinline__ float sum(const float* ring, int ring_rows, int64_t ring_stride, const float* taps, int channels, int n_taps,
+                                       int pos, int ch) const {
+    float acc = bias;
+    if constexpr (NT > 0) {
+#pragma unroll
+      for (int j = 0; j < NT; ++j) acc = fmaf(w[j], j < NT - 1 ? x[j] : now, acc);
+    } else {
+      for (int j = 0; j < n_taps; ++j) {
+        const int back = n_taps - 1 - j;
+        if (back > pos) continue;
+        acc = fmaf(taps[(size_t)j * channels + ch], back ? ring[(size_t)((pos - back) % ring_rows) * ring_stride + ch] : now, acc);
+      }
+    }
+    return acc;
+  }
+};
 
 inline bool step_ok(const pace_step_t* s) {
   return s && s->n_tokens >= 0 && s->n_entries >= 0 && s->n_tokens >= s->n_entries &&

@@ -143,7 +143,7 @@ __global__ void __launch_bounds__(STATE_ONLY ? 256 : 512, STATE_ONLY ? 2 : 1)
       float dt[2], l[2];
 #pragma unroll
       for (int k = 0; k < 2; ++k) {
-        dt[k] = lane + 32 * k < n_tok ? softplus(raw[k] + dt_bias) : 0.f;
+        dt[k] = lane + 32 * k < n_tok ? softplus_fast(raw[k] + dt_bias) : 0.f;
         l[k] = neg_a * dt[k];
       }
 #pragma unroll
