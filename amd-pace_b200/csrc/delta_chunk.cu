@@ -19,7 +19,7 @@
 namespace pace {
 namespace {
 
-constexpr int kChunk = 64, kThreads = 256, kLP = kChunk + 8, kTP = kChunk + 8;
+constexpr int kChunk = 64, kThreads = 512, kLP = kChunk + 8, kTP = kChunk + 8;
 constexpr float kRange = 86.0f;   // log2 units eight tokens may decay by on the fast path: e^60
 
 __device__ __forceinline__ void mma16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
@@ -142,19 +142,19 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
     for (int j = part * ROWS; j < (part + 1) * ROWS; ++j) G[j * GP + gc] = s += G[j * GP + gc];
   }
   {
-    const int j = tid >> 2;                                // four threads a token
+    const int j = tid >> 3;                                // eight threads a token
     float sq = 0.f, sk = 0.f;
-    for (int c = (tid & 3) * 2; c < DP; c += 8) {
+    for (int c = (tid & 7) * 2; c < DP; c += 16) {
       const float2 x = bf2_to_f2(*reinterpret_cast<const uint32_t*>(qs + j * QP + c)), y = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ks + j * QP + c));
       sq = fmaf(x.x, x.x, fmaf(x.y, x.y, sq));
       sk = fmaf(y.x, y.x, fmaf(y.y, y.y, sk));
     }
 #pragma unroll
-    for (int o = 2; o; o >>= 1) {
+    for (int o = 4; o; o >>= 1) {
       sq += __shfl_xor_sync(0xffffffffu, sq, o);
       sk += __shfl_xor_sync(0xffffffffu, sk, o);
     }
-    if ((tid & 3) == 0) {
+    if ((tid & 7) == 0) {
       fq[j] = a.q_scale / sqrtf(sq + a.unit_eps);
       fk[j] = 1.0f / sqrtf(sk + a.unit_eps);
     }
@@ -175,33 +175,32 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
   }
   __syncthreads();
 
-  // ---- scores: warp (row block of 16, every other tile of 8 columns); the two long and the two short blocks share schedulers ----
+  // ---- scores: warp (keys or queries as rows, row block of 16, every other tile of 8 columns); a scheduler's warps have long and
+  // short row blocks ----
   {
-    const int rb = warp < 4 ? warp : 7 - warp, half = (warp >> 2) & 1;   // warps w and w + 4: row blocks w and 3 - w
-    // (half: warps 0 .. 3 take the even tiles of row block w, warps 4 .. 7 the odd ones of row block 7 - w)
-    float ck[4][4], cq[4][4];
+    const bool is_q = warp >= 8;
+    const int w8 = warp & 7, rb = w8 < 4 ? w8 : 7 - w8, half = w8 >> 2;
+    float acc[4][4];
 #pragma unroll
     for (int s = 0; s < 4; ++s)
 #pragma unroll
-      for (int x = 0; x < 4; ++x) ck[s][x] = cq[s][x] = 0.f;
+      for (int x = 0; x < 4; ++x) acc[s][x] = 0.f;
     const bool far = slow[rb] != 0;
     const int i0 = 16 * rb + g, ref = far ? 16 * rb - 1 : 16 * rb + 7;
+    const __nv_bfloat16* rows = is_q ? qs : ks;
 #pragma unroll 1
     for (int k0 = 0; k0 < DP; k0 += 16) {
       const int c0 = k0 + 2 * t;
       float2 m[2];
 #pragma unroll
       for (int x = 0; x < 2; ++x) m[x] = ref >= 0 ? *reinterpret_cast<const float2*>(G + ref * GP + c0 + 8 * x) : make_float2(0.f, 0.f);
-      uint32_t kh_[4], kl_[4], qh_[4], ql_[4];
+      uint32_t ah[4], al[4];
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         const int row = i0 + (x & 1) * 8, c = c0 + (x >> 1) * 8;
         const float2 gg = *reinterpret_cast<const float2*>(G + row * GP + c);
-        const float e0 = fast_exp2(gg.x - m[x >> 1].x), e1 = fast_exp2(gg.y - m[x >> 1].y);
-        const float2 kk = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ks + row * QP + c));
-        const float2 qq = bf2_to_f2(*reinterpret_cast<const uint32_t*>(qs + row * QP + c));
-        split_bf2(kk.x * e0, kk.y * e1, kh_[x], kl_[x]);
-        split_bf2(qq.x * e0, qq.y * e1, qh_[x], ql_[x]);
+        const float2 v = bf2_to_f2(*reinterpret_cast<const uint32_t*>(rows + row * QP + c));
+        split_bf2(v.x * fast_exp2(gg.x - m[x >> 1].x), v.y * fast_exp2(gg.y - m[x >> 1].y), ah[x], al[x]);
       }
 #pragma unroll
       for (int s = 0; s < 4; ++s) {
@@ -214,8 +213,7 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
           const float2 kk = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ks + j * QP + c0 + 8 * x));
           split_bf2(kk.x * fast_exp2(m[x].x - gg.x), kk.y * fast_exp2(m[x].y - gg.y), bh[x], bl[x]);
         }
-        mma_split(ck[s], kh_, kl_, bh, bl);
-        mma_split(cq[s], qh_, ql_, bh, bl);
+        mma_split(acc[s], ah, al, bh, bl);
       }
     }
     __nv_bfloat16 *p_hi = tiles + SL::kP, *p_lo = p_hi + kChunk * kTP;
@@ -225,18 +223,21 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
         const int i = i0 + 8 * x, j = 8 * (2 * s + half) + 2 * t;
-        const float f0 = fk[j], f1 = fk[j + 1], bi = beta[i] * fk[i], qi = fq[i];
-        L[i * kLP + j] = j < i ? ck[s][2 * x] * bi * f0 : 0.f;
-        L[i * kLP + j + 1] = j + 1 < i ? ck[s][2 * x + 1] * bi * f1 : 0.f;
-        uint32_t hi, lo;
-        split_bf2(j <= i ? cq[s][2 * x] * qi * f0 : 0.f, j + 1 <= i ? cq[s][2 * x + 1] * qi * f1 : 0.f, hi, lo);
-        *reinterpret_cast<uint32_t*>(p_hi + i * kTP + j) = hi;
-        *reinterpret_cast<uint32_t*>(p_lo + i * kTP + j) = lo;
+        const float f = is_q ? fq[i] : beta[i] * fk[i], y0 = acc[s][2 * x] * f * fk[j], y1 = acc[s][2 * x + 1] * f * fk[j + 1];
+        if (is_q) {
+          uint32_t hi, lo;
+          split_bf2(j <= i ? y0 : 0.f, j + 1 <= i ? y1 : 0.f, hi, lo);
+          *reinterpret_cast<uint32_t*>(p_hi + i * kTP + j) = hi;
+          *reinterpret_cast<uint32_t*>(p_lo + i * kTP + j) = lo;
+        } else {
+          L[i * kLP + j] = j < i ? y0 : 0.f;
+          L[i * kLP + j + 1] = j + 1 < i ? y1 : 0.f;
+        }
       }
     }
   }
   for (int b = 0; b < 4; ++b) {
-    if (!slow[b]) continue;
+    if (!slow[b] || tid >= 256) continue;
     __nv_bfloat16 *p_hi = tiles + SL::kP, *p_lo = p_hi + kChunk * kTP;
     const int i = 16 * b + tid / 16, j = 16 * b + tid % 16;   // one pair per thread
     float sk = 0.f, sq = 0.f;
@@ -594,7 +595,7 @@ __global__ void __launch_bounds__(128 * GROUPS, 1) delta_walk_kernel(pace_step_t
     }
 }
 
-constexpr uint64_t kBudget = 256ull << 20;   // bytes of scratch a launch pair may use
+constexpr uint64_t kBudget = 512ull << 20;   // bytes of scratch a launch pair may use
 
 struct Plan {
   int dp, slab;      // padded key size, chunks of an entry per launch pair
