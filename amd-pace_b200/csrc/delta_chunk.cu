@@ -8,13 +8,14 @@
 // W = T K^(G), T V, Q^(G), K^(G_n - G) and P; a second one walks the chunks, a block per (entry, head, 16 or 32 value columns)
 // with its part of S in fp32 accumulators.
 //
-// e^(G_i - G_j) is the product of a row's factor e^(G_i - M) and a column's e^(M - G_j), M the sum up to the middle of the row's
-// sixteen tokens: both are finite as long as eight tokens decay by less than e^60.  Sixteen rows with a channel beyond that
-// take M in front of them (both factors are then at most 1) and their own 16 x 16 block pair by pair.
+// e^(G_i - G_j) is the product of a row's factor e^(G_i - M) and a column's e^(M - G_j), M the sum up to the middle of the column's
+// sixteen tokens: both are finite as long as eight tokens decay by less than e^60.  Sixteen columns with a channel beyond
+// that take M behind them (both factors are then at most 1 for the rows further down) and their own 16 x 16 block pair by pair.
 //
 // q, k, v are bf16 values; everything else is fp32: where an fp32 quantity is the operand of a bf16 product it is split into two
 // bf16 terms, of whose four products the three that matter are taken (16 bits); T is made in fp32 on the CUDA cores.
 #include "delta.cuh"
+#include "umma.cuh"
 
 namespace pace {
 namespace {
@@ -46,6 +47,24 @@ __device__ __forceinline__ void copy16(void* dst, const void* src, bool live = t
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
 }
 
+__device__ __forceinline__ uint64_t both(float v) { return pack64(__float_as_uint(v), __float_as_uint(v)); }
+// softplus_fast of two values, two-wide
+__device__ __forceinline__ uint64_t softplus2(float x0, float x1) {
+  const float u0 = fast_exp2(-fabsf(x0) * kLog2e), u1 = fast_exp2(-fabsf(x1) * kLog2e);
+  const uint64_t u = pack64(__float_as_uint(u0), __float_as_uint(u1));
+  uint32_t d0, d1;
+  unpack64(add2(u, both(2.0f)), d0, d1);
+  const float r0 = rcp_t<__nv_bfloat16>(__uint_as_float(d0)), r1 = rcp_t<__nv_bfloat16>(__uint_as_float(d1));
+  const uint64_t s = fma2(u, pack64(__float_as_uint(r0), __float_as_uint(r1)), 0ull), q = fma2(s, s, 0ull);
+  uint64_t p = fma2(q, both(1.0f / 13), both(1.0f / 11));
+  p = fma2(p, q, both(1.0f / 9));
+  p = fma2(p, q, both(1.0f / 7));
+  p = fma2(p, q, both(1.0f / 5));
+  p = fma2(p, q, both(1.0f / 3));
+  p = fma2(p, q, both(1.0f));
+  return fma2(add2(s, s), p, pack64(__float_as_uint(fmaxf(x0, 0.f)), __float_as_uint(fmaxf(x1, 0.f))));
+}
+
 // What the first launch leaves of a (entry, chunk, head), as it lies in shared memory later: bf16 tiles of 64 rows of QP (high,
 // low halves), P 64 rows of kTP, then fp32.
 template <int DP>
@@ -66,6 +85,7 @@ template <int DP>
 struct Prep {
   static constexpr int QP = DP + 8, GP = DP + 8;
   static constexpr int kVMost = 128, VP = kVMost + 8;            // value columns that pass through shared memory
+  static_assert(VP >= QP, "the columns' high half fits where V will be");
   static constexpr int kK = 0, kQ = kK + kChunk * QP * 2, kG = kQ + kChunk * QP * 2, kL = kG + kChunk * GP * 4,
                        kV = kL + kChunk * kLP * 4, kVec = kV + kChunk * VP * 2, bytes = kVec + (3 * kChunk + 4) * 4;
   static_assert(kChunk * kLP * 4 >= 2 * kChunk * kTP * 2, "the halves of T take the place of L");
@@ -103,35 +123,37 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
     const bool live = j < n_tok && c < d;
     copy16((which ? ks : qs) + j * QP + c, qkv + (live ? (size_t)j * a.qkv_stride + (size_t)(which * KV + kh) * d + c : 0), live);
   }
-  const bool v_here = vd <= PR::kVMost;
-  if (v_here) {
-    const int pieces = (vd + 15) / 16 * 2;                 // 16 bytes each, whole items of 16 columns
-    for (int i = tid; i < kChunk * pieces; i += kThreads) {
-      const int j = i / pieces, c = (i - j * pieces) * 8;
-      const bool live = j < n_tok && c < vd;
-      copy16(vs + j * PR::VP + c, qkv + (live ? (size_t)j * a.qkv_stride + 2 * (size_t)KV * d + (size_t)h * vd + c : 0), live);
-    }
-  }
   asm volatile("cp.async.commit_group;" ::: "memory");
   if (tid < 4) slow[tid] = 0;
   if (tid < kChunk)
     beta[tid] = tid < n_tok ? sigmoid_t<__nv_bfloat16>(
         __bfloat162float(static_cast<const __nv_bfloat16*>(a.b_raw)[(size_t)(t0 + tid) * a.b_stride + h])) : 0.f;
   {
-    const float neg_a = a.neg_a[h] * kLog2e;
-    const __nv_bfloat16* ar = static_cast<const __nv_bfloat16*>(a.a_raw) + (size_t)t0 * a.a_stride + (size_t)h * d;
-    for (int i = tid; i < kChunk * (DP / 2); i += kThreads) {
-      const int j = i / (DP / 2), c = (i - j * (DP / 2)) * 2;
-      float2 v = make_float2(0.f, 0.f);
+    // a thread has eight channels of every (kThreads / (DP / 8))-th token
+    const int c = tid % (DP / 8) * 8, j0 = tid / (DP / 8);
+    const uint64_t neg_a = both(a.neg_a[h] * kLog2e);
+    const __nv_bfloat16* ar = static_cast<const __nv_bfloat16*>(a.a_raw) + (size_t)t0 * a.a_stride + (size_t)h * d + c;
+    float bias[8];
+#pragma unroll
+    for (int x = 0; x < 8; ++x) bias[x] = c < d ? a.dt_bias[(size_t)h * d + c + x] : 0.f;
+#pragma unroll
+    for (int j = j0; j < kChunk; j += kThreads / (DP / 8)) {
+      uint64_t v[4] = {0ull, 0ull, 0ull, 0ull};
       if (j < n_tok && c < d) {
-        const float2 x = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ar + (size_t)j * a.a_stride + c));
-        const float2 b = *reinterpret_cast<const float2*>(a.dt_bias + (size_t)h * d + c);
-        v = make_float2(neg_a * softplus_fast(x.x + b.x), neg_a * softplus_fast(x.y + b.y));
+        float x[8];
+        Vec<__nv_bfloat16, 8>::load(ar + (size_t)j * a.a_stride, x);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) v[u] = fma2(softplus2(x[2 * u] + bias[2 * u], x[2 * u + 1] + bias[2 * u + 1]), neg_a, 0ull);
       }
-      *reinterpret_cast<float2*>(G + j * GP + c) = v;
+#pragma unroll
+      for (int u = 0; u < 4; u += 2) {
+        uint4 w;
+        unpack64(v[u], w.x, w.y);
+        unpack64(v[u + 1], w.z, w.w);
+        *reinterpret_cast<uint4*>(G + j * GP + c + 2 * u) = w;
+      }
     }
   }
-  for (int i = tid; i < kChunk * kLP; i += kThreads) L[i] = 0.f;
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
   constexpr int PARTS = kThreads / DP, ROWS = kChunk / PARTS;
@@ -144,10 +166,13 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
   {
     const int j = tid >> 3;                                // eight threads a token
     float sq = 0.f, sk = 0.f;
-    for (int c = (tid & 7) * 2; c < DP; c += 16) {
-      const float2 x = bf2_to_f2(*reinterpret_cast<const uint32_t*>(qs + j * QP + c)), y = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ks + j * QP + c));
-      sq = fmaf(x.x, x.x, fmaf(x.y, x.y, sq));
-      sk = fmaf(y.x, y.x, fmaf(y.y, y.y, sk));
+#pragma unroll
+    for (int c = (tid & 7) * 8; c < DP; c += 64) {
+      float x[8], y[8];
+      Vec<__nv_bfloat16, 8>::load(qs + j * QP + c, x);
+      Vec<__nv_bfloat16, 8>::load(ks + j * QP + c, y);
+#pragma unroll
+      for (int u = 0; u < 8; ++u) sq = fmaf(x[u], x[u], sq), sk = fmaf(y[u], y[u], sk);
     }
 #pragma unroll
     for (int o = 4; o; o >>= 1) {
@@ -174,68 +199,99 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
     if (s - m > kRange || m - G[(16 * b + 15) * GP + c] > kRange) slow[b] = 1;
   }
   __syncthreads();
+  // ---- columns: the keys with their factors, in two halves, where V and L will be ----
+  __nv_bfloat16 *kc_hi = vs, *kc_lo = t_hi;
+  for (int i = tid; i < kChunk * (DP / 4); i += kThreads) {
+    const int j = i / (DP / 4), c = (i - j * (DP / 4)) * 4, b = j >> 4, ref = 16 * b + (slow[b] ? 15 : 7);
+    const float4 gg = *reinterpret_cast<const float4*>(G + j * GP + c), m = *reinterpret_cast<const float4*>(G + ref * GP + c);
+    float kk[4];
+    Vec<__nv_bfloat16, 4>::load(ks + j * QP + c, kk);
+    uint2 hi, lo;
+    split_bf2(kk[0] * fast_exp2(m.x - gg.x), kk[1] * fast_exp2(m.y - gg.y), hi.x, lo.x);
+    split_bf2(kk[2] * fast_exp2(m.z - gg.z), kk[3] * fast_exp2(m.w - gg.w), hi.y, lo.y);
+    *reinterpret_cast<uint2*>(kc_hi + j * QP + c) = hi;
+    *reinterpret_cast<uint2*>(kc_lo + j * QP + c) = lo;
+  }
+  __syncthreads();
 
-  // ---- scores: warp (keys or queries as rows, row block of 16, every other tile of 8 columns); a scheduler's warps have long and
-  // short row blocks ----
+  // ---- scores: warp (keys or queries as rows, one or two of the ten 16 x 16 blocks) ----
   {
     const bool is_q = warp >= 8;
-    const int w8 = warp & 7, rb = w8 < 4 ? w8 : 7 - w8, half = w8 >> 2;
-    float acc[4][4];
-#pragma unroll
-    for (int s = 0; s < 4; ++s)
-#pragma unroll
-      for (int x = 0; x < 4; ++x) acc[s][x] = 0.f;
-    const bool far = slow[rb] != 0;
-    const int i0 = 16 * rb + g, ref = far ? 16 * rb - 1 : 16 * rb + 7;
     const __nv_bfloat16* rows = is_q ? qs : ks;
-#pragma unroll 1
-    for (int k0 = 0; k0 < DP; k0 += 16) {
-      const int c0 = k0 + 2 * t;
-      float2 m[2];
+    // (row block, column block) of a warp's first and second task; -1: none
+    constexpr int kRow[2][8] = {{0, 1, 1, 2, 2, 2, 3, 3}, {3, 3, -1, -1, -1, -1, -1, -1}};
+    constexpr int kCol[2][8] = {{0, 0, 1, 0, 1, 2, 0, 1}, {2, 3, -1, -1, -1, -1, -1, -1}};
+    float acc[2][2][4];
+    const int w8 = warp & 7;
 #pragma unroll
-      for (int x = 0; x < 2; ++x) m[x] = ref >= 0 ? *reinterpret_cast<const float2*>(G + ref * GP + c0 + 8 * x) : make_float2(0.f, 0.f);
-      uint32_t ah[4], al[4];
+    for (int task = 0; task < 2; ++task) {
 #pragma unroll
-      for (int x = 0; x < 4; ++x) {
-        const int row = i0 + (x & 1) * 8, c = c0 + (x >> 1) * 8;
-        const float2 gg = *reinterpret_cast<const float2*>(G + row * GP + c);
-        const float2 v = bf2_to_f2(*reinterpret_cast<const uint32_t*>(rows + row * QP + c));
-        split_bf2(v.x * fast_exp2(gg.x - m[x >> 1].x), v.y * fast_exp2(gg.y - m[x >> 1].y), ah[x], al[x]);
-      }
+      for (int s = 0; s < 2; ++s)
 #pragma unroll
-      for (int s = 0; s < 4; ++s) {
-        if (s > rb) break;
-        const int j = 8 * (2 * s + half) + g;
-        uint32_t bh[2], bl[2];
+        for (int x = 0; x < 4; ++x) acc[task][s][x] = 0.f;
+      int rb = -1, cb = -1;
 #pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          const float2 gg = *reinterpret_cast<const float2*>(G + j * GP + c0 + 8 * x);
-          const float2 kk = bf2_to_f2(*reinterpret_cast<const uint32_t*>(ks + j * QP + c0 + 8 * x));
-          split_bf2(kk.x * fast_exp2(m[x].x - gg.x), kk.y * fast_exp2(m[x].y - gg.y), bh[x], bl[x]);
+      for (int w = 0; w < 8; ++w)
+        if (w8 == w) rb = kRow[task][w], cb = kCol[task][w];
+      if (rb < 0 || (rb == cb && slow[cb])) continue;
+      const int i0 = 16 * rb + g, ref = 16 * cb + (slow[cb] ? 15 : 7);
+      const __nv_bfloat16* cols = kc_hi + (16 * cb + (lane & 7) + (lane >> 4) * 8) * QP + ((lane >> 3) & 1) * 8;   // two tiles of 8 columns
+      const int low = (int)(kc_lo - kc_hi);
+#pragma unroll 2
+      for (int k0 = 0; k0 < DP; k0 += 16) {
+        const int c0 = k0 + 2 * t;
+        uint32_t ah[4], al[4], bh[4], bl[4];
+        ldsm4(bh, cols + k0);
+        ldsm4(bl, cols + low + k0);
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          const int row = i0 + (x & 1) * 8, c = c0 + (x >> 1) * 8;
+          const float2 gg = *reinterpret_cast<const float2*>(G + row * GP + c), m = *reinterpret_cast<const float2*>(G + ref * GP + c);
+          const float2 v = bf2_to_f2(*reinterpret_cast<const uint32_t*>(rows + row * QP + c));
+          split_bf2(v.x * fast_exp2(gg.x - m.x), v.y * fast_exp2(gg.y - m.y), ah[x], al[x]);
         }
-        mma_split(acc[s], ah, al, bh, bl);
+        mma_split(acc[task][0], ah, al, bh, bl);
+        mma_split(acc[task][1], ah, al, bh + 2, bl + 2);
       }
     }
+    __syncthreads();                                           // the columns have been read: L takes the place of a half
+    for (int i = tid; i < kChunk * kLP / 4; i += kThreads) reinterpret_cast<float4*>(L)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    __syncthreads();
     __nv_bfloat16 *p_hi = tiles + SL::kP, *p_lo = p_hi + kChunk * kTP;
 #pragma unroll
-    for (int s = 0; s < 4; ++s) {
-      if (s > rb || (far && s == rb)) break;
+    for (int task = 0; task < 2; ++task) {
+      int rb = -1, cb = -1;
 #pragma unroll
-      for (int x = 0; x < 2; ++x) {
-        const int i = i0 + 8 * x, j = 8 * (2 * s + half) + 2 * t;
-        const float f = is_q ? fq[i] : beta[i] * fk[i], y0 = acc[s][2 * x] * f * fk[j], y1 = acc[s][2 * x + 1] * f * fk[j + 1];
-        if (is_q) {
-          uint32_t hi, lo;
-          split_bf2(j <= i ? y0 : 0.f, j + 1 <= i ? y1 : 0.f, hi, lo);
-          *reinterpret_cast<uint32_t*>(p_hi + i * kTP + j) = hi;
-          *reinterpret_cast<uint32_t*>(p_lo + i * kTP + j) = lo;
-        } else {
-          L[i * kLP + j] = j < i ? y0 : 0.f;
-          L[i * kLP + j + 1] = j + 1 < i ? y1 : 0.f;
+      for (int w = 0; w < 8; ++w)
+        if (w8 == w) rb = kRow[task][w], cb = kCol[task][w];
+      if (rb < 0 || (rb == cb && slow[cb])) continue;
+#pragma unroll
+      for (int s = 0; s < 2; ++s)
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const int i = 16 * rb + g + 8 * x, j = 16 * cb + 8 * s + 2 * t;
+          const float f = is_q ? fq[i] : beta[i] * fk[i], y0 = acc[task][s][2 * x] * f * fk[j], y1 = acc[task][s][2 * x + 1] * f * fk[j + 1];
+          if (is_q) {
+            uint32_t hi, lo;
+            split_bf2(j <= i ? y0 : 0.f, j + 1 <= i ? y1 : 0.f, hi, lo);
+            *reinterpret_cast<uint32_t*>(p_hi + i * kTP + j) = hi;
+            *reinterpret_cast<uint32_t*>(p_lo + i * kTP + j) = lo;
+          } else {
+            *reinterpret_cast<float2*>(L + i * kLP + j) = make_float2(j < i ? y0 : 0.f, j + 1 < i ? y1 : 0.f);
+          }
         }
-      }
     }
   }
+  const bool v_here = vd <= PR::kVMost;                        // (needed at the end: on their way while T is made)
+  if (v_here) {
+    const int pieces = (vd + 15) / 16 * 2;                     // 16 bytes each, whole items of 16 columns
+    for (int i = tid; i < kChunk * pieces; i += kThreads) {
+      const int j = i / pieces, c = (i - j * pieces) * 8;
+      const bool live = j < n_tok && c < vd;
+      copy16(vs + j * PR::VP + c, qkv + (live ? (size_t)j * a.qkv_stride + 2 * (size_t)KV * d + (size_t)h * vd + c : 0), live);
+    }
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
   for (int b = 0; b < 4; ++b) {
     if (!slow[b] || tid >= 256) continue;
     __nv_bfloat16 *p_hi = tiles + SL::kP, *p_lo = p_hi + kChunk * kTP;
@@ -341,6 +397,7 @@ __global__ void __launch_bounds__(kThreads, 2) delta_prepare_kernel(pace_step_t 
       *reinterpret_cast<uint32_t*>(t_lo + r * kTP + c) = lo[k];
     }
   }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
 
   // ---- T K^(G) and T V, 16 columns at a time ----
@@ -645,8 +702,8 @@ int launch_chunked(const pace_step_t& st, const pace_delta_args_t& a, const Plan
 
 // bf16, key sizes that the tiles cover and 16-byte pieces; everything else is the token-by-token kernel's
 bool delta_chunked_fits(const pace_delta_args_t& a) {
-  return a.dtype == PACE_DTYPE_BF16 && a.dim <= 128 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.qkv_stride % 8 == 0 && a.a_stride % 2 == 0 &&
-         a.out_stride % 2 == 0 && aligned16(a.qkv) && ((uintptr_t)a.a_raw & 3) == 0 && ((uintptr_t)a.dt_bias & 7) == 0 &&
+  return a.dtype == PACE_DTYPE_BF16 && a.dim <= 128 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.qkv_stride % 8 == 0 && a.a_stride % 8 == 0 &&
+         a.out_stride % 2 == 0 && aligned16(a.qkv) && aligned16(a.a_raw) &&
          ((uintptr_t)a.out & 3) == 0 && ((uintptr_t)a.s_state & 7) == 0;
 }
 
