@@ -113,7 +113,7 @@ def plain_attention(m, w, qkv, eps=1e-6):
     return ref.capped_attention(qkv.double(), m, p, "", eps).view(len(qkv), m["heads"], m["vdim"])
 
 
-SHAPES = [(BF16, 6, 2, 40, 24, 3, 16), (BF16, 8, 4, 64, 128, 4, 64), (BF16, 40, 2, 128, 64, 4, 32), (BF16, 3, 1, 22, 13, 5, 6),
+SHAPES = [(BF16, 6, 2, 40, 24, 3, 16), (BF16, 10, 5, 64, 120, 4, 48), (BF16, 40, 2, 128, 64, 4, 32), (BF16, 3, 1, 22, 13, 5, 6),
           (BF16, 4, 2, 136, 72, 2, 136), (BF16, 2, 2, 16, 16, 1, 0), (FP32, 6, 2, 40, 24, 4, 16), (FP32, 3, 3, 22, 13, 2, 22),
           (FP32, 2, 1, 136, 160, 3, 8)]
 
