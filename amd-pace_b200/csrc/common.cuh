@@ -83,9 +83,14 @@ struct KVView {
 // row planes of a layer: keys and values, or one that is both
 __host__ __device__ inline int pool_planes(const pace_kv_pool_t& p) { return p.row_format == PACE_ROWS_SHARED ? 1 : 2; }
 
+// tokens per row, rows per page
+__host__ __device__ inline int row_tokens(const pace_kv_pool_t& p) { return p.row_tokens > 1 ? p.row_tokens : 1; }
+__host__ __device__ inline int page_rows(const pace_kv_pool_t& p) { return p.page_tokens / row_tokens(p); }
+
+// (in units of rows: the page_tokens of the view are the rows of a page)
 inline KVView make_view(const pace_kv_pool_t* p, int layer, const int32_t* seq_ids) {
   KVView v;
-  const size_t page_elems = (size_t)p->n_kv_heads * p->page_tokens * p->head_dim;
+  const size_t page_elems = (size_t)p->n_kv_heads * page_rows(*p) * p->head_dim;
   const size_t region = page_elems * (size_t)p->n_pages;
   const __nv_bfloat16* base = (const __nv_bfloat16*)p->pages;
   v.k = base + (size_t)layer * pool_planes(*p) * region;
@@ -96,7 +101,7 @@ inline KVView make_view(const pace_kv_pool_t* p, int layer, const int32_t* seq_i
   v.seq_len = p->seq_len + (size_t)layer * p->max_seqs;
   v.status = p->status;
   v.fixed_len = 0;
-  v.page_tokens = p->page_tokens;
+  v.page_tokens = page_rows(*p);
   v.n_kv_heads = p->n_kv_heads;
   v.head_dim = p->head_dim;
   v.max_pages_per_seq = p->max_pages_per_seq;

@@ -565,6 +565,21 @@ __global__ void glu_kernel(const T* __restrict__ x, int64_t xs, T* __restrict__ 
   }
 }
 
+template <typename T, int V>
+__global__ void gate_per_head_kernel(T* __restrict__ x, const T* __restrict__ gate, int64_t gs, int n_tokens, int heads, int vd) {
+  const int per = vd / V;
+  const size_t total = (size_t)n_tokens * heads * per;
+  for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t th = i / per;
+    const float f = sigmoid_t<T>(to_f<T>(gate[th / heads * gs + th % heads]));
+    float v[V];
+    Vec<T, V>::load(x + i * V, v);
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[j] *= f;
+    Vec<T, V>::store(x + i * V, v);
+  }
+}
+
 __global__ void soft_cap_kernel(float* x, int64_t n, float cap) {
   for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x)
     x[i] = cap * tanhf(x[i] / cap);
@@ -586,7 +601,7 @@ __global__ void part_norm_gate_kernel(pace_part_norm_gate_args_t a) {
   T* out = static_cast<T*>(a.out) + (size_t)t * a.out_stride + c0;
   auto value = [&](int c, float* x) {
     Vec<T, V>::load(o + c, x);
-    if (a.gate_first) {
+    if (a.gate_mode == PACE_GATE_SILU_FIRST) {
       float g[V];
       Vec<T, V>::load(gate + c, g);
 #pragma unroll
@@ -624,11 +639,11 @@ __global__ void part_norm_gate_kernel(pace_part_norm_gate_args_t a) {
     Vec<float, V>::load(a.w + (c0 + c) % a.w_period, w);
 #pragma unroll
     for (int j = 0; j < V; ++j) x[j] *= r * w[j];
-    if (!a.gate_first) {
+    if (a.gate_mode != PACE_GATE_SILU_FIRST) {
       float g[V];
       Vec<T, V>::load(gate + c, g);
 #pragma unroll
-      for (int j = 0; j < V; ++j) x[j] *= sigmoid_t<T>(g[j]);
+      for (int j = 0; j < V; ++j) x[j] *= a.gate_mode == PACE_GATE_SILU ? silu_t<T>(g[j]) : sigmoid_t<T>(g[j]);
     }
     Vec<T, V>::store(out + c, x);
   }
@@ -706,6 +721,18 @@ int relu_squared_t(void* x, int64_t n, cudaStream_t s) {
   else
     relu_squared_kernel<T, 1><<<elementwise_blocks((size_t)n), 256, 0, s>>>((T*)x, n);
   PACE_LAUNCH_CHECK("relu_squared_kernel");
+  return PACE_OK;
+}
+
+template <typename T>
+int gate_per_head_t(void* x, const void* gate, int64_t gs, int n_tokens, int heads, int vd, cudaStream_t s) {
+  constexpr int V = 16 / sizeof(T);
+  const size_t n = (size_t)n_tokens * heads * vd;
+  if (vd % V == 0 && aligned16(x))
+    gate_per_head_kernel<T, V><<<elementwise_blocks(n / V), 256, 0, s>>>((T*)x, (const T*)gate, gs, n_tokens, heads, vd);
+  else
+    gate_per_head_kernel<T, 1><<<elementwise_blocks(n), 256, 0, s>>>((T*)x, (const T*)gate, gs, n_tokens, heads, vd);
+  PACE_LAUNCH_CHECK("gate_per_head_kernel");
   return PACE_OK;
 }
 
@@ -789,6 +816,13 @@ int pace_norm_gate(const void* o, const float* w, const void* gate, int64_t gs, 
                                   : norm_gate_t<float>(o, w, gate, gs, out, n_tokens, n, eps, (cudaStream_t)stream);
 }
 
+int pace_gate_per_head(void* x, const void* gate, int64_t gs, int32_t n_tokens, int32_t heads, int32_t vd, int32_t dtype, void* stream) {
+  if (!x || !gate || n_tokens < 0 || heads < 1 || vd < 1 || gs < heads || !dtype_ok(dtype)) return PACE_ERR_INVALID;
+  if (n_tokens == 0) return PACE_OK;
+  return dtype == PACE_DTYPE_BF16 ? gate_per_head_t<__nv_bfloat16>(x, gate, gs, n_tokens, heads, vd, (cudaStream_t)stream)
+                                  : gate_per_head_t<float>(x, gate, gs, n_tokens, heads, vd, (cudaStream_t)stream);
+}
+
 int pace_relu_squared(void* x, int64_t n, int32_t dtype, void* stream) {
   if (!x || n < 0 || !dtype_ok(dtype)) return PACE_ERR_INVALID;
   if (n == 0) return PACE_OK;
@@ -820,7 +854,7 @@ int pace_soft_cap(float* x, int64_t n, float cap, void* stream) {
 
 int pace_part_norm_gate(const pace_part_norm_gate_args_t* a, void* stream) {
   if (!a || !a->o || !a->gate || !a->w || !a->out || a->n_tokens < 0 || a->part < 1 || a->n < a->part || a->n % a->part ||
-      a->w_period < 1 || a->o_stride < a->n || a->gate_stride < a->n || a->out_stride < a->n || !dtype_ok(a->dtype))
+      a->w_period < 1 || a->gate_mode < PACE_GATE_SIGMOID || a->gate_mode > PACE_GATE_SILU || a->o_stride < a->n || a->gate_stride < a->n || a->out_stride < a->n || !dtype_ok(a->dtype))
     return PACE_ERR_INVALID;
   if (a->n_tokens == 0) return PACE_OK;
   if ((int64_t)a->n_tokens * (a->n / a->part) > 0x3fffffff) return PACE_ERR_UNSUPPORTED;

@@ -54,8 +54,9 @@ MetaLayout meta_layout(const pace_kv_pool_t* g) {
 bool geometry_ok(const pace_kv_pool_t* g) {
   if (!g) return false;
   if (g->n_layers <= 0 || g->n_kv_heads <= 0 || g->page_tokens <= 0 || g->n_pages <= 0 || g->max_seqs <= 0 ||
-      g->max_pages_per_seq <= 0)
+      g->max_pages_per_seq <= 0 || g->row_tokens < 0)
     return false;
+  if (row_tokens(*g) > 1 && (g->page_tokens % g->row_tokens || g->row_format == PACE_ROWS_SHARED)) return false;
   if (g->row_format == PACE_ROWS_OPAQUE || g->row_format == PACE_ROWS_SHARED) return g->head_dim > 0 && g->head_dim % 8 == 0 && g->head_dim <= 2048;
   return g->row_format == PACE_ROWS_BF16 && (g->head_dim == 64 || g->head_dim == 128);
 }
@@ -173,19 +174,21 @@ __global__ void reserve_kernel(pace_kv_pool_t p, int layer, const int32_t* __res
   const int nc = cow_count;
   if (nc == 0) return;
   // rows of a page are contiguous per head: copy rows*D elements for every (layer, K|V, head)
-  const size_t page_elems = (size_t)p.n_kv_heads * P * p.head_dim;
+  const int per = row_tokens(p), page_rows = P / per;
+  const size_t page_elems = (size_t)p.n_kv_heads * page_rows * p.head_dim;
   const size_t region = page_elems * (size_t)p.n_pages;
   uint4* base = reinterpret_cast<uint4*>(p.pages);
   const int vec_per_row = p.head_dim / 8;
   for (int c = 0; c < nc; ++c) {
-    const int src = cow[3 * c], dst = cow[3 * c + 1], rows = cow[3 * c + 2];
+    const int src = cow[3 * c], dst = cow[3 * c + 1], rows = cow[3 * c + 2] / per;   // (whole blocks only have a row)
+    if (rows == 0) continue;
     const size_t per_head = (size_t)rows * vec_per_row;
     const size_t total = (size_t)p.n_layers * pool_planes(p) * p.n_kv_heads * per_head;
     for (size_t i = threadIdx.x; i < total; i += blockDim.x) {
       const size_t lk = i / (p.n_kv_heads * per_head);
       const size_t rem = i % (p.n_kv_heads * per_head);
       const size_t h = rem / per_head, o = rem % per_head;
-      const size_t head_off = (h * P) * (size_t)p.head_dim / 8;
+      const size_t head_off = (h * page_rows) * (size_t)p.head_dim / 8;
       const size_t s = (lk * region + (size_t)src * page_elems) / 8 + head_off + o;
       const size_t d = (lk * region + (size_t)dst * page_elems) / 8 + head_off + o;
       base[d] = base[s];
@@ -712,7 +715,7 @@ bool pool_ok(const pace_kv_pool_t* p) {
          p->free_stack && p->counters && p->status && p->table_tmp;
 }
 // the entry points that move or interpret bf16 rows
-bool bf16_rows(const pace_kv_pool_t* p) { return p->row_format == PACE_ROWS_BF16; }
+bool bf16_rows(const pace_kv_pool_t* p) { return p->row_format == PACE_ROWS_BF16 && row_tokens(*p) == 1; }
 
 }  // namespace
 }  // namespace pace
@@ -726,7 +729,7 @@ const char* pace_version(void) { return "pace_b200 0.1 (sm_100a)"; }
 
 int pace_kv_pool_bytes(const pace_kv_pool_t* g, uint64_t* pages_bytes, uint64_t* meta_bytes) {
   if (!geometry_ok(g) || !pages_bytes || !meta_bytes) return PACE_ERR_INVALID;
-  *pages_bytes = (uint64_t)g->n_layers * pool_planes(*g) * g->n_pages * g->n_kv_heads * g->page_tokens * g->head_dim * 2;
+  *pages_bytes = (uint64_t)g->n_layers * pool_planes(*g) * g->n_pages * g->n_kv_heads * page_rows(*g) * g->head_dim * 2;
   *meta_bytes = meta_layout(g).total;
   return PACE_OK;
 }

@@ -29,13 +29,14 @@ class KVPoolStruct(C.Structure):
                                           "max_seqs", "max_pages_per_seq", "owns_memory")] + \
                [(n, C.c_void_p) for n in ("pages", "block_table", "seq_len", "seq_pages", "page_ref",
                                           "free_stack", "counters", "status", "table_tmp")] + \
-               [("row_format", C.c_int32)]
+               [("row_format", C.c_int32), ("row_tokens", C.c_int32)]
 
 
 ROWS_BF16, ROWS_OPAQUE, ROWS_SHARED = 0, 1, 2   # PACE_ROWS_*
 DTYPE_BF16, DTYPE_FP32 = 0, 1   # PACE_DTYPE_*
 SPAN_ALL, SPAN_WINDOW, SPAN_CHUNK = 0, 1, 2   # PACE_SPAN_*
 ACT_SILU, ACT_GELU_TANH, ACT_GELU_ERF = 0, 1, 2  # PACE_ACT_*
+GATE_SIGMOID, GATE_SILU_FIRST, GATE_SILU = 0, 1, 2  # PACE_GATE_*
 
 ATTN_WHOLE_UNITS = 1      # PACE_ATTN_WHOLE_UNITS
 ATTN_PENDING_ROW = 2      # PACE_ATTN_PENDING_ROW
@@ -161,7 +162,7 @@ class AppendConvArgs(C.Structure):
 class PartNormGateArgs(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("o", "gate", "w", "out")] + \
                [(n, C.c_int64) for n in ("o_stride", "gate_stride", "out_stride")] + \
-               [(n, C.c_int32) for n in ("n_tokens", "n", "part", "w_period", "gate_first", "dtype")] + [("eps", C.c_float)]
+               [(n, C.c_int32) for n in ("n_tokens", "n", "part", "w_period", "gate_mode", "dtype")] + [("eps", C.c_float)]
 
 
 class SsdArgs(C.Structure):
@@ -178,6 +179,37 @@ class DeltaArgs(C.Structure):
                [(n, C.c_void_p) for n in ("taps", "ring", "workspace")] + [("workspace_bytes", C.c_uint64)] + \
                [(n, C.c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "n_taps", "ring_rows", "ring_stride", "dtype")] + \
                [("unit_eps", C.c_float), ("q_scale", C.c_float)]
+
+
+class GlaArgs(C.Structure):
+    _fields_ = [("qkv", C.c_void_p), ("qkv_stride", C.c_int64), ("z", C.c_void_p), ("z_stride", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("z_bias", "s_state", "out")] + [("out_stride", C.c_int64)] + \
+               [("norm", C.c_void_p), ("gate", C.c_void_p), ("gate_stride", C.c_int64), ("workspace", C.c_void_p),
+                ("workspace_bytes", C.c_uint64)] + \
+               [(n, C.c_int32) for n in ("heads", "dim", "vdim", "dtype")] + [(n, C.c_float) for n in ("inv_tau", "q_scale", "eps")]
+
+
+class AppendRotateArgs(C.Structure):
+    _fields_ = [("qkv", C.c_void_p), ("qkv_stride", C.c_int64)] + [(n, C.c_void_p) for n in ("cos_table", "sin_table", "q_out")] + \
+               [(n, C.c_int32) for n in ("n_q_heads", "dim", "vdim", "rot_pairs", "halves", "table_rows", "block", "block_now", "dtype")]
+
+
+class AttnPooledArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("q", "out", "gate", "sinks", "mix")] + [("out_stride", C.c_int64), ("gate_stride", C.c_int64)] + \
+               [(n, C.c_int32) for n in ("n_q_heads", "dim", "vdim", "dtype", "q_elems", "window", "block", "token_begin", "token_end",
+                                         "entry_begin", "entry_end", "max_tokens", "max_keys")] + \
+               [("scale", C.c_float), ("workspace", C.c_void_p), ("workspace_bytes", C.c_uint64)]
+
+
+class ShiftNormArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("x_in", "x_out", "y")] + [("y_stride", C.c_int64)] + \
+               [(n, C.c_void_p) for n in ("y_bias", "w_post", "add", "w_next", "shift", "state", "state_out")] + \
+               [("state_stride", C.c_int64), ("h", C.c_void_p), ("width", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float)]
+
+
+class EmbedPairsArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("x", "embed", "pairs", "last_token")] + [("mul_prev", C.c_int64), ("mul_cur", C.c_int64)] + \
+               [(n, C.c_int32) for n in ("width", "vocab", "buckets", "store_last", "dtype")] + [("scale", C.c_float)]
 
 
 byref = C.byref
@@ -239,6 +271,15 @@ _SIGS = {
     "pace_delta_workspace_bytes": (C.c_uint64, [C.c_int32] * 6),
     "pace_delta_prefill": (C.c_int, [_S, C.POINTER(DeltaArgs), C.c_void_p]),
     "pace_delta_step": (C.c_int, [_S, C.POINTER(DeltaArgs), C.c_void_p]),
+    "pace_gla_workspace_bytes": (C.c_uint64, [C.c_int32] * 5),
+    "pace_gla_prefill": (C.c_int, [_S, C.POINTER(GlaArgs), C.c_void_p]),
+    "pace_gla_step": (C.c_int, [_S, C.POINTER(GlaArgs), C.c_void_p]),
+    "pace_kv_append_rotate": (C.c_int, [_P, C.c_int32, _P, C.c_int32, _S, C.POINTER(AppendRotateArgs), C.c_void_p]),
+    "pace_attn_pooled": (C.c_int, [_P, C.c_int32, _P, C.c_int32, _S, C.POINTER(AttnPooledArgs), C.c_void_p]),
+    "pace_shift_norm": (C.c_int, [_S, C.POINTER(ShiftNormArgs), C.c_void_p]),
+    "pace_embed_pairs": (C.c_int, [_S, C.POINTER(EmbedPairsArgs), C.c_void_p]),
+    "pace_state_commit": (C.c_int, [_S, C.c_void_p, C.c_void_p, C.c_int64, C.c_int64, C.c_void_p, C.c_void_p]),
+    "pace_gate_per_head": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int64] + [C.c_int32] * 4 + [C.c_void_p]),
     "pace_moe_route": (C.c_int, [C.POINTER(MoeRouteArgs), C.c_void_p]),
     "pace_moe_experts": (C.c_int, [C.POINTER(MoeExpertsArgs), C.c_void_p]),
     "pace_gate_heads": (C.c_int, [_S, C.c_void_p, C.c_void_p, C.c_int64, C.c_void_p, C.c_int32, C.c_int32, C.c_int32,

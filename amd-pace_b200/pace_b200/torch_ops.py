@@ -57,13 +57,13 @@ _DEFS.update({
                          "int dim, int vdim, float scale, int span, int span_size, int entry_begin, int entry_end, int max_tokens, "
                          "int max_keys, Tensor? k, Tensor? k2, Tensor? v, Tensor? key_cu, Tensor? key_pos, "
                          "float softcap=0.0, int out_row=0) -> bool",
-    "latent_append": "(int pool, Tensor(a!) pages, int layer, int step, Tensor down, Tensor q_norm, Tensor kv_norm, Tensor cos, "
-                     "Tensor sin, Tensor(b!) cq, int rot_dim, float eps) -> ()",
+    "latent_append": "(int pool, Tensor(a!) pages, int layer, int step, Tensor down, Tensor? q_norm, Tensor kv_norm, Tensor? cos, "
+                     "Tensor? sin, Tensor(b!)? cq, int rot_dim, float eps) -> ()",
     "rotate_heads": "(int step, Tensor src, Tensor(a!) dst, Tensor cos, Tensor sin, int token_begin, int token_end, int pad_dim) -> ()",
     "latent_gather": "(int pool, Tensor pages, int layer, Tensor slot, Tensor pos, Tensor(a!) out) -> ()",
     "glu": "(Tensor x, Tensor(a!) out, int act, bool gated=True) -> ()",
     "soft_cap": "(Tensor(a!) x, float cap) -> ()",
-    "part_norm_gate": "(Tensor o, Tensor gate, Tensor w, Tensor(a!) out, int part, bool gate_first, float eps) -> ()",
+    "part_norm_gate": "(Tensor o, Tensor gate, Tensor w, Tensor(a!) out, int part, int gate_mode, float eps) -> ()",
     "kv_append_conv": "(int pool, Tensor(a!) pages, int layer, int step, Tensor qkv, Tensor taps, Tensor(b!) ring, Tensor q_norm, "
                       "Tensor k_norm, Tensor? cos, Tensor? sin, Tensor(c!) q_out, int dim, int vdim, float eps, float v_mul, "
                       "bool store_ring) -> ()",
@@ -76,6 +76,20 @@ _DEFS.update({
                      "Tensor(b!) out, int kv_heads, float unit_eps, float q_scale) -> ()",
     "delta_step": "(int step, Tensor qkv, Tensor a_raw, Tensor b_raw, Tensor dt_bias, Tensor neg_a, Tensor(a!) state, "
                   "Tensor(b!) out, int kv_heads, float unit_eps, float q_scale, Tensor taps, Tensor(c!) ring) -> ()",
+    "gla_prefill": "(int step, Tensor qkv, Tensor z, Tensor z_bias, Tensor(a!) state, Tensor(b!) out, float inv_tau, float q_scale) -> ()",
+    "gla_step": "(int step, Tensor qkv, Tensor z, Tensor z_bias, Tensor(a!) state, Tensor(b!) out, float inv_tau, float q_scale, "
+                "Tensor norm, Tensor gate, float eps) -> ()",
+    "kv_append_rotate": "(int pool, Tensor(a!) pages, int layer, int blocks, Tensor(b!)? block_pages, int block_layer, int step, Tensor qkv, "
+                        "Tensor? cos, Tensor? sin, Tensor(c!) q_out, int dim, int vdim, bool halves, int block, bool block_now) -> ()",
+    "attn_pooled": "(int pool, Tensor pages, int layer, int blocks, Tensor? block_pages, int block_layer, int step, Tensor q, "
+                   "Tensor(a!) out, Tensor? gate, Tensor? sinks, Tensor? mix, int dim, int vdim, float scale, int window, int block, "
+                   "int token_begin, int token_end, int max_keys) -> ()",
+    "shift_norm": "(int step, Tensor x_in, Tensor(a!) x_out, Tensor? y, Tensor? y_bias, Tensor? w_post, Tensor? add, Tensor w_next, "
+                  "Tensor shift, Tensor state, Tensor(b!) state_out, Tensor(c!) h, float eps) -> ()",
+    "embed_pairs": "(int step, Tensor(a!) x, Tensor embed, float scale, Tensor? pairs, Tensor(b!)? last_token, int mul_prev, int mul_cur, "
+                   "bool store_last) -> ()",
+    "state_commit": "(int step, Tensor source, Tensor(a!) target, Tensor(b!)? last_token) -> ()",
+    "gate_per_head": "(Tensor(a!) x, Tensor gate) -> ()",
     "moe_route": "(Tensor logits, Tensor? correction, Tensor(a!) slot_expert, Tensor(b!) slot_rank, Tensor(c!) slot_weight, "
                  "Tensor(d!) expert_count, Tensor(e!) expert_list, bool softmax=False, float? weight_scale=None) -> ()",
     "moe_experts": "(Tensor x, Tensor gate_up, Tensor down, Tensor(a!) hidden, Tensor(b!) y, Tensor(d!)? scratch, "
@@ -284,10 +298,11 @@ def _attn_span_prefill(pool, pages, layer, step, q, out, slopes, sinks, dim, vdi
 
 def _latent_append(pool, pages, layer, step, down, q_norm, kv_norm, cos, sin, cq, rot_dim, eps):
     a = _C.LatentAppendArgs()
-    a.down, a.down_stride, a.q_norm, a.kv_norm = down.data_ptr(), down.stride(0), q_norm.data_ptr(), kv_norm.data_ptr()
-    a.cos_table, a.sin_table, a.cq = cos.data_ptr(), sin.data_ptr(), cq.data_ptr()
-    a.q_rank, a.kv_rank, a.rot_dim, a.rot_pairs = q_norm.numel(), kv_norm.numel(), rot_dim, cos.shape[1]
-    a.table_rows, a.dtype, a.eps = cos.shape[0], _dtype(down), eps
+    a.down, a.down_stride, a.q_norm, a.kv_norm = down.data_ptr(), down.stride(0), _ptr(q_norm), kv_norm.data_ptr()
+    a.cq, a.q_rank, a.kv_rank, a.rot_dim = _ptr(cq), 0 if q_norm is None else q_norm.numel(), kv_norm.numel(), rot_dim
+    if cos is not None:
+        a.cos_table, a.sin_table, (a.table_rows, a.rot_pairs) = cos.data_ptr(), sin.data_ptr(), cos.shape
+    a.dtype, a.eps = _dtype(down), eps
     with torch.cuda.device(pages.device):
         _C.check(_C.lib.pace_latent_append(_pool(pool), layer, _step(step), C.byref(a), _stream(pages)), "pace_latent_append")
 
@@ -320,11 +335,11 @@ def _soft_cap(x, cap):
         _C.check(_C.lib.pace_soft_cap(x.data_ptr(), x.numel(), cap, _stream(x)), "pace_soft_cap")
 
 
-def _part_norm_gate(o, gate, w, out, part, gate_first, eps):
+def _part_norm_gate(o, gate, w, out, part, gate_mode, eps):
     a = _C.PartNormGateArgs()
     a.o, a.gate, a.w, a.out = o.data_ptr(), gate.data_ptr(), w.data_ptr(), out.data_ptr()
     a.o_stride, a.gate_stride, a.out_stride = o.stride(0), gate.stride(0), out.stride(0)
-    a.n_tokens, a.n, a.part, a.w_period, a.gate_first, a.dtype, a.eps = *o.shape, part, w.numel(), int(gate_first), _dtype(o), eps
+    a.n_tokens, a.n, a.part, a.w_period, a.gate_mode, a.dtype, a.eps = *o.shape, part, w.numel(), gate_mode, _dtype(o), eps
     with torch.cuda.device(o.device):
         _C.check(_C.lib.pace_part_norm_gate(C.byref(a), _stream(o)), "pace_part_norm_gate")
 
@@ -452,6 +467,91 @@ def _delta(entry: str):
     return impl
 
 
+def _gla(entry: str):
+    fn = getattr(_C.lib, entry)
+
+    def impl(step, qkv, z, z_bias, state, out, inv_tau, q_scale, norm=None, gate=None, eps=0.0):
+        a = _C.GlaArgs()
+        a.qkv, a.qkv_stride, a.z, a.z_stride = qkv.data_ptr(), qkv.stride(0), z.data_ptr(), z.stride(0)
+        a.z_bias, a.s_state, a.out, a.out_stride = z_bias.data_ptr(), state.data_ptr(), out.data_ptr(), out.stride(0)
+        (_, a.heads, a.dim, a.vdim), a.dtype = state.shape, _dtype(qkv)
+        a.inv_tau, a.q_scale, a.eps = inv_tau, q_scale, eps
+        if norm is not None:
+            a.norm, a.gate, a.gate_stride = norm.data_ptr(), gate.data_ptr(), gate.stride(0)
+        with torch.cuda.device(out.device):
+            st = _C.StepStruct.from_address(step)
+            ws = None
+            if norm is None:
+                ws = _workspace(a, _C.lib.pace_gla_workspace_bytes(st.n_entries, st.max_count, a.heads, a.dim, a.dtype), out.device)
+            _C.check(fn(_step(step), C.byref(a), _stream(out)), entry)
+            del ws
+    return impl
+
+
+def _kv_append_rotate(pool, pages, layer, blocks, block_pages, block_layer, step, qkv, cos, sin, q_out, dim, vdim, halves, block, block_now):
+    a = _C.AppendRotateArgs()
+    a.qkv, a.qkv_stride, a.q_out = qkv.data_ptr(), qkv.stride(0), q_out.data_ptr()
+    if cos is not None:
+        a.cos_table, a.sin_table, (a.table_rows, a.rot_pairs) = cos.data_ptr(), sin.data_ptr(), cos.shape
+    a.n_q_heads, a.dim, a.vdim, a.halves = q_out.shape[1], dim, vdim, int(halves)
+    a.block, a.block_now, a.dtype = block, int(block_now), _dtype(qkv)
+    with torch.cuda.device(pages.device):
+        _C.check(_C.lib.pace_kv_append_rotate(_pool(pool), layer, _pool(blocks) if block else None, block_layer, _step(step), C.byref(a),
+                                              _stream(pages)), "pace_kv_append_rotate")
+
+
+def _pooled_args(q, out, gate, sinks, mix, dim, vdim, scale, window, block, max_keys):
+    a = _C.AttnPooledArgs()
+    a.q, a.out, a.sinks, a.mix, a.out_stride = q.data_ptr(), out.data_ptr(), _ptr(sinks), _ptr(mix), out.stride(0)
+    if gate is not None:
+        a.gate, a.gate_stride = gate.data_ptr(), gate.stride(0)
+    (_, a.n_q_heads, a.q_elems), a.dim, a.vdim, a.dtype = q.shape, dim, vdim, _dtype(q)
+    a.window, a.block, a.max_keys, a.scale = window, block, max_keys, scale
+    return a
+
+
+def _attn_pooled(pool, pages, layer, blocks, block_pages, block_layer, step, q, out, gate, sinks, mix, dim, vdim, scale, window, block,
+                 token_begin, token_end, max_keys):
+    a = _pooled_args(q, out, gate, sinks, mix, dim, vdim, scale, window, block, max_keys)
+    a.token_begin, a.token_end = token_begin, token_end
+    with torch.cuda.device(q.device):
+        _C.check(_C.lib.pace_attn_pooled(_pool(pool), layer, _pool(blocks) if block else None, block_layer, _step(step), C.byref(a),
+                                         _stream(q)), "pace_attn_pooled")
+
+
+def _shift_norm(step, x_in, x_out, y, y_bias, w_post, add, w_next, shift, state, state_out, h, eps):
+    a = _C.ShiftNormArgs()
+    a.x_in, a.x_out, a.w_next, a.shift, a.h = x_in.data_ptr(), x_out.data_ptr(), w_next.data_ptr(), shift.data_ptr(), h.data_ptr()
+    a.state, a.state_out, a.state_stride = state.data_ptr(), state_out.data_ptr(), state.stride(0)
+    a.y_bias, a.w_post, a.add = _ptr(y_bias), _ptr(w_post), _ptr(add)
+    if y is not None:
+        a.y, a.y_stride = y.data_ptr(), y.stride(0)
+    a.width, a.dtype, a.eps = x_in.shape[1], _dtype(h), eps
+    with torch.cuda.device(h.device):
+        _C.check(_C.lib.pace_shift_norm(_step(step), C.byref(a), _stream(h)), "pace_shift_norm")
+
+
+def _embed_pairs(step, x, embed, scale, pairs, last_token, mul_prev, mul_cur, store_last):
+    a = _C.EmbedPairsArgs()
+    a.x, a.embed, a.pairs, a.last_token = x.data_ptr(), embed.data_ptr(), _ptr(pairs), _ptr(last_token)
+    a.mul_prev, a.mul_cur, (a.vocab, a.width), a.store_last = mul_prev, mul_cur, embed.shape, int(store_last)
+    a.buckets, a.dtype, a.scale = pairs.shape[0] - 1 if pairs is not None else 0, _dtype(embed), scale
+    with torch.cuda.device(x.device):
+        _C.check(_C.lib.pace_embed_pairs(_step(step), C.byref(a), _stream(x)), "pace_embed_pairs")
+
+
+def _state_commit(step, source, target, last_token=None):
+    with torch.cuda.device(target.device):
+        _C.check(_C.lib.pace_state_commit(_step(step), source.data_ptr(), target.data_ptr(), source[0].numel(), source.stride(0),
+                                          _ptr(last_token), _stream(target)), "pace_state_commit")
+
+
+def _gate_per_head(x, gate):
+    with torch.cuda.device(x.device):
+        _C.check(_C.lib.pace_gate_per_head(x.data_ptr(), gate.data_ptr(), gate.stride(0), *x.shape, _dtype(x), _stream(x)),
+                 "pace_gate_per_head")
+
+
 def _rglru_args(yx, ra_bias, ri_bias, decay_base, state, conv_state, out, blocks):
     a = _C.RglruArgs()
     a.yx, a.yx_stride = yx.data_ptr(), yx.stride(0)
@@ -538,7 +638,10 @@ _IMPLS = {"kv_reserve": _kv_reserve, "kv_append": _kv_append, "kv_append_layers"
           "latent_append": _latent_append, "rotate_heads": _rotate_heads, "latent_gather": _latent_gather, "glu": _glu,
           "moe_route": _moe_route, "moe_experts": _moe_experts, "soft_cap": _soft_cap, "part_norm_gate": _part_norm_gate,
           "kv_append_conv": _kv_append_conv, "conv_store": _conv_store, "ssd_prefill": _ssd("pace_ssd_prefill"),
-          "ssd_step": _ssd("pace_ssd_step"), "delta_prefill": _delta("pace_delta_prefill"), "delta_step": _delta("pace_delta_step")}
+          "ssd_step": _ssd("pace_ssd_step"), "delta_prefill": _delta("pace_delta_prefill"), "delta_step": _delta("pace_delta_step"),
+          "gla_prefill": _gla("pace_gla_prefill"), "gla_step": _gla("pace_gla_step"), "kv_append_rotate": _kv_append_rotate,
+          "attn_pooled": _attn_pooled, "shift_norm": _shift_norm, "embed_pairs": _embed_pairs, "state_commit": _state_commit,
+          "gate_per_head": _gate_per_head}
 for _n, _f in _IMPLS.items():
     _lib.impl(_n, _f, "CUDA")
     # shape propagation for tracers: nothing is returned, nothing to compute

@@ -50,6 +50,11 @@ extern "C" {
  *   status       int32 [4]          [0] sticky PACE_DEV_* bits
  *   table_tmp    int32 [max_seqs][max_pages_per_seq + 1]   scratch of pace_kv_gather
  *
+ * row_tokens: consecutive tokens that share a row (0 or 1: a row per token).  A pool of pooled blocks has one row for every
+ * row_tokens tokens; lengths and page_tokens (a multiple of row_tokens) stay counts of tokens, so that such a pool is
+ * reserved, released and gathered with the calls and numbers of the token pool beside it, and a page has
+ * page_tokens / row_tokens rows.
+ *
  * page_tokens is the physical page size (the Python host uses 64: one page is one K/V chunk of
  * the attention kernels).  The reference's capacity (whole `tokens_per_split` segments,
  * cache.py:177-181, 292-313) is host bookkeeping on top of the pages and does not depend on it;
@@ -70,6 +75,7 @@ typedef struct pace_kv_pool {
   int32_t* status;      /* device */
   int32_t* table_tmp;   /* device */
   int32_t row_format;   /* PACE_ROWS_*: 0 = bf16 rows of 64 or 128 */
+  int32_t row_tokens;   /* 0, 1: a row per token */
 } pace_kv_pool_t;
 
 const char* pace_last_cuda_error(void);
@@ -666,8 +672,12 @@ int pace_gate_heads(const pace_step_t* step, const void* attn, const void* gate,
 /* out[t] = rms(o[t]) * w * sigmoid(gate[t]) over n elements (w fp32). */
 int pace_norm_gate(const void* o, const float* w, const void* gate, int64_t gate_stride, void* out, int32_t n_tokens,
                    int32_t n, float eps, int32_t dtype, void* stream);
-/* Norms over equal parts of a row, with a gate in front (silu) or behind (sigmoid):
- *     gate_first:  out = rms(o * silu(gate)) * w,      otherwise:  out = rms(o) * w * sigmoid(gate)
+#define PACE_GATE_SIGMOID 0
+#define PACE_GATE_SILU_FIRST 1
+#define PACE_GATE_SILU 2
+/* Norms over equal parts of a row, with a gate in front (silu) or behind (sigmoid or silu):
+ *     gate_mode PACE_GATE_SILU_FIRST:  out = rms(o * silu(gate)) * w
+ *     PACE_GATE_SIGMOID, PACE_GATE_SILU:  out = rms(o) * w * sigmoid(gate), silu(gate)
  * rms over every `part` elements (n a multiple of part), weight w[c % w_period] (fp32). */
 typedef struct {
   const void* o;
@@ -675,7 +685,7 @@ typedef struct {
   const float* w;
   void* out;
   int64_t o_stride, gate_stride, out_stride;
-  int32_t n_tokens, n, part, w_period, gate_first, dtype;
+  int32_t n_tokens, n, part, w_period, gate_mode, dtype;
   float eps;
 } pace_part_norm_gate_args_t;
 int pace_part_norm_gate(const pace_part_norm_gate_args_t* a, void* stream);
@@ -814,6 +824,124 @@ typedef struct {
 uint64_t pace_delta_workspace_bytes(int32_t n_entries, int32_t max_count, int32_t heads, int32_t dim, int32_t vdim, int32_t dtype);
 int pace_delta_prefill(const pace_step_t* step, const pace_delta_args_t* a, void* stream);
 int pace_delta_step(const pace_step_t* step, const pace_delta_args_t* a, void* stream);
+
+/* Gated linear attention with a decay per head and key channel:
+ *     alpha_t = sigmoid(z + z_bias)^inv_tau;  S <- diag(alpha_t) S + k_t v_t^T;  o_t = q_scale S^T q_t
+ * per head (S dim x vdim).  qkv dtype [n_tokens][qkv_stride] = q (heads x dim) | k (heads x dim) | v (heads x vdim); z dtype rows of
+ * heads x dim, z_bias fp32 [heads x dim].  s_state fp32 [slots][heads][dim][vdim].  out dtype [n_tokens][out_stride].
+ * pace_gla_step: one token per entry; the outputs are normalised per head and gated as well,
+ *     out = rms(o) * norm * silu(gate)           (norm fp32 [vdim], shared by the heads; gate dtype rows of heads x vdim)
+ * dim <= 512. */
+typedef struct {
+  const void* qkv;
+  int64_t qkv_stride;
+  const void* z;
+  int64_t z_stride;
+  const float* z_bias;
+  float* s_state;
+  void* out;
+  int64_t out_stride;
+  const float* norm;        /* step only */
+  const void* gate;         /* step only */
+  int64_t gate_stride;
+  void* workspace;          /* prefill: pace_gla_workspace_bytes() of scratch, any content */
+  uint64_t workspace_bytes;
+  int32_t heads, dim, vdim, dtype;
+  float inv_tau, q_scale, eps;
+} pace_gla_args_t;
+uint64_t pace_gla_workspace_bytes(int32_t n_entries, int32_t max_count, int32_t heads, int32_t dim, int32_t dtype);
+int pace_gla_prefill(const pace_step_t* step, const pace_gla_args_t* a, void* stream);
+int pace_gla_step(const pace_step_t* step, const pace_gla_args_t* a, void* stream);
+
+/* ---- attention over a window and pooled blocks -----------------------------------------------------------------------
+ * A layer has two pools of the same row geometry: tokens, and blocks of `block` tokens (row_tokens = block), whose rows are the means
+ * of the cached keys and of the cached values of a whole block.
+ * pace_kv_append_rotate: qkv dtype [n_tokens][qkv_stride] = q (n_q_heads x dim) | k (kv_heads x dim) | v (kv_heads x vdim); the
+ * first 2 rot_pairs elements of every query and key head are turned by the angles of the tables (fp32 [table_rows][rot_pairs]),
+ * element i with element i + rot_pairs (`halves`) or 2i with 2i + 1; queries go to q_out [n_tokens][n_q_heads][row elements], keys and
+ * values to their pages (reserved), rows are zero beyond dim / vdim.  With block > 0 the blocks that the step's tokens complete
+ * get their rows, by a launch behind, or with block_now (one token per entry) by the same one. */
+typedef struct {
+  const void* qkv;
+  int64_t qkv_stride;
+  const float* cos_table;
+  const float* sin_table;
+  void* q_out;
+  int32_t n_q_heads, dim, vdim, rot_pairs, halves, table_rows, block, block_now, dtype;
+} pace_append_rotate_args_t;
+int pace_kv_append_rotate(const pace_kv_pool_t* pool, int32_t layer, const pace_kv_pool_t* blocks, int32_t block_layer,
+                          const pace_step_t* step, const pace_append_rotate_args_t* a, void* stream);
+
+/* The query at position i sees the tokens j with 0 <= i - j < window and, with block > 0, the blocks b whose last token
+ * b block + block - 1 is at most i - window.  One softmax over both, score = scale * (q . k), with exp(sinks[h]) in the denominator
+ * (sinks NULL: ordinary softmax).  mix (fp32 [n_q_heads][n_q_heads], NULL: none) then mixes the heads' weights, weight_h <- sum_g
+ * mix[h][g] weight_g, in front of the values of head h's own KV head (h / (n_q_heads / kv_heads)), and gate (dtype rows of n_q_heads x
+ * vdim, NULL: none) multiplies the outputs by its sigmoid.  q dtype [n_tokens][n_q_heads][row elements]; out dtype rows of n_q_heads
+ * x vdim.  Tokens [token_begin, token_end) of the step; max_keys: upper bound of their positions + 1.
+ * pace_attn_pooled: token by token; pace_attn_pooled_prompt: entries [entry_begin, entry_end) of up to max_tokens tokens on tcgen05,
+ * with scratch of pace_attn_pooled_prompt_workspace_bytes(); answers PACE_ERR_UNSUPPORTED (nothing launched) for what it does not
+ * take: fp32, rows other than PACE_ROWS_BF16 in pages of 64 rows, scales that are not positive, more than 32 query heads per KV
+ * head. */
+typedef struct {
+  const void* q;
+  void* out;
+  const void* gate;
+  const float* sinks;
+  const float* mix;
+  int64_t out_stride, gate_stride;
+  int32_t n_q_heads, dim, vdim, dtype, q_elems, window, block, token_begin, token_end, entry_begin, entry_end, max_tokens, max_keys;
+  float scale;
+  void* workspace;
+  uint64_t workspace_bytes;
+} pace_attn_pooled_args_t;
+int pace_attn_pooled(const pace_kv_pool_t* pool, int32_t layer, const pace_kv_pool_t* blocks, int32_t block_layer,
+                     const pace_step_t* step, const pace_attn_pooled_args_t* a, void* stream);
+
+/* ---- layers that read shifted inputs ---------------------------------------------------------------------------------
+ * pace_shift_norm: between two layers,
+ *     x_out = x_in + rms(y + y_bias) * w_post + add                       (y, y_bias, add may be NULL; add, y_bias fp32 [width])
+ *     n = rms(x_out) * w_next,   h = n + (n' - n) * shift                 (element by element)
+ * with n' the n of the sequence's previous token: of the step, or state[slot] (fp32 rows of state_stride), or zeros in front of the
+ * first one.  The last n of every entry goes to state_out[slot].  x_out and state_out may be x_in and state in a step of one token per
+ * entry; otherwise they must be other buffers (pace_state_commit brings the states over).
+ * pace_embed_pairs: x = embed[token] * scale + pairs[(previous token * mul_prev + token * mul_cur) mod buckets]; pairs (dtype
+ * [buckets + 1][width], NULL: none) has one more row for a sequence's first token.  last_token int32 [slots]; store_last (one token
+ * per entry) also stores the token there.
+ * pace_state_commit: to[slot][0 .. n) = from[slot][0 .. n) for the step's slots (rows of `stride`), last_token (or NULL) [slot] =
+ * the entry's last token. */
+typedef struct {
+  const float* x_in;
+  float* x_out;
+  const void* y;
+  int64_t y_stride;
+  const float* y_bias;
+  const float* w_post;
+  const float* add;
+  const float* w_next;
+  const float* shift;
+  const float* state;
+  float* state_out;
+  int64_t state_stride;
+  void* h;
+  int32_t width, dtype;
+  float eps;
+} pace_shift_norm_args_t;
+int pace_shift_norm(const pace_step_t* step, const pace_shift_norm_args_t* a, void* stream);
+typedef struct {
+  float* x;
+  const void* embed;
+  const void* pairs;
+  int32_t* last_token;
+  int64_t mul_prev, mul_cur;
+  int32_t width, vocab, buckets, store_last, dtype;
+  float scale;
+} pace_embed_pairs_args_t;
+int pace_embed_pairs(const pace_step_t* step, const pace_embed_pairs_args_t* a, void* stream);
+int pace_state_commit(const pace_step_t* step, const float* from, float* to, int64_t n, int64_t stride, int32_t* last_token,
+                      void* stream);
+/* x[t][h][0 .. vdim) *= sigmoid(gate[t][h]) in place; x dense [n_tokens][heads][vdim]. */
+int pace_gate_per_head(void* x, const void* gate, int64_t gate_stride, int32_t n_tokens, int32_t heads, int32_t vdim, int32_t dtype,
+                       void* stream);
 
 /* Step arrays of a decode step whose tokens and positions the device holds (one token per entry):
  * token[i] = next_token[i], tok_pos[i] = start[i] = position[i]. */
