@@ -16,7 +16,7 @@ OUT = os.path.join(HERE, "pace_b200", "libpace_b200.so")
 SOURCES = ["kv_pool.cu", "attn_decode.cu", "attn_mma.cu", "attn_api.cu", "linear_skinny.cu",
            "hybrid_ops.cu", "attn_general.cu", "recurrent.cu", "lightning.cu", "attn_span.cu", "attn_span_keys.cu", "attn_span_umma.cu", "latent.cu", "moe.cu",
            "conv_append.cu", "ssd.cu", "ssd_chunk.cu", "delta.cu", "delta_chunk.cu", "rotate_append.cu", "shift_norm.cu", "attn_pooled.cu",
-           "gla.cu", "gla_chunk.cu"]
+           "attn_pooled_umma.cu", "gla.cu", "gla_chunk.cu"]
 # fp32 exp, log and divide of these files are the accurate ones (they serve 32-bit models)
 PRECISE = {"hybrid_ops.cu", "attn_general.cu", "recurrent.cu", "lightning.cu", "latent.cu", "moe.cu", "conv_append.cu",
            "ssd.cu", "ssd_chunk.cu", "delta.cu", "delta_chunk.cu", "rotate_append.cu", "shift_norm.cu", "attn_pooled.cu", "gla.cu",

@@ -444,18 +444,8 @@ extern "C" {
 
 int pace_attn_pooled(const pace_kv_pool_t* p, int32_t layer, const pace_kv_pool_t* bp, int32_t block_layer, const pace_step_t* st,
                      const pace_attn_pooled_args_t* a, void* stream) {
-  if (!p || !p->pages || !p->block_table || !step_ok(st) || !a || layer < 0 || layer >= p->n_layers) return PACE_ERR_INVALID;
-  if (!a->q || !a->out || a->n_q_heads < 1 || p->n_kv_heads < 1 || a->n_q_heads % p->n_kv_heads || a->dim < 1 || a->vdim < 1 || a->window < 1 ||
-      a->block < 0 || a->token_begin < 0 || a->token_end > st->n_tokens || a->max_keys < 0 ||
-      (a->dtype != PACE_DTYPE_BF16 && a->dtype != PACE_DTYPE_FP32) || a->out_stride < (int64_t)a->n_q_heads * a->vdim ||
-      (a->gate && a->gate_stride < (int64_t)a->n_q_heads * a->vdim))
-    return PACE_ERR_INVALID;
-  if (p->row_format == PACE_ROWS_SHARED || row_tokens(*p) != 1) return PACE_ERR_UNSUPPORTED;
-  if (a->block > 0 && (!bp || !bp->pages || !bp->block_table || block_layer < 0 || block_layer >= bp->n_layers || row_tokens(*bp) != a->block ||
-                       bp->n_kv_heads != p->n_kv_heads || bp->head_dim != p->head_dim || bp->row_format != p->row_format))
-    return PACE_ERR_INVALID;
-  const int row = a->dtype == PACE_DTYPE_BF16 ? p->head_dim : p->head_dim / 2;
-  if (a->q_elems != row || a->dim > row || a->vdim > row || (p->row_format == PACE_ROWS_BF16 && a->dtype != PACE_DTYPE_BF16)) return PACE_ERR_INVALID;
+  if (!pooled_args_ok(p, layer, bp, block_layer, st, a) || a->token_begin < 0 || a->token_end > st->n_tokens) return PACE_ERR_INVALID;
+  const int row = a->q_elems;
   if (a->token_begin >= a->token_end) return PACE_OK;
   PACE_PROFILE("attn_pooled", stream, "layer=%d tokens=%d heads=%d dims=%d/%d", layer, a->token_end - a->token_begin, a->n_q_heads, a->dim, a->vdim);
   const cudaStream_t s = (cudaStream_t)stream;

@@ -106,6 +106,7 @@ def _span(window: Optional[int], chunk: Optional[int]):
 
 
 MOE_WIDE = 32           # tokens per expert from which wide token tiles are worth the copy
+PROMPT_TOKENS = 16      # tokens of an entry from which pooled attention over tiles of tokens is worth a launch
 PROMPT_ROWS = 64        # query rows of an entry from which the tcgen05 prompt kernel is worth a launch
 
 
@@ -230,7 +231,12 @@ def pooled_attention(step: Step, cache, blocks, qkv: torch.Tensor, tables, heads
     where = (pool.handle, pool.pages, cache.layer, bp.handle, bp.pages, blocks.layer, step.handle)
     _OPS.kv_append_rotate(*where, qkv, *(tables or (None, None)), q, dim, vdim, halves, block, step.decode_only)
     rule = (q, out, gate, sinks, mix, dim, vdim, scale, window, block)
-    _OPS.attn_pooled(*where, *rule, 0, T, step.max_keys)
+    Ed, E = step.n_decode, step.n_entries
+    if (E > Ed and q.dtype == torch.bfloat16 and step.max_count >= PROMPT_TOKENS
+            and _OPS.attn_pooled_prompt(*where, *rule, Ed, E, step.max_count, step.max_keys)):
+        T = Ed
+    if T:
+        _OPS.attn_pooled(*where, *rule, 0, T, step.max_keys)
     return out
 
 

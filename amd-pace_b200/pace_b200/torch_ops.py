@@ -84,6 +84,9 @@ _DEFS.update({
     "attn_pooled": "(int pool, Tensor pages, int layer, int blocks, Tensor? block_pages, int block_layer, int step, Tensor q, "
                    "Tensor(a!) out, Tensor? gate, Tensor? sinks, Tensor? mix, int dim, int vdim, float scale, int window, int block, "
                    "int token_begin, int token_end, int max_keys) -> ()",
+    "attn_pooled_prompt": "(int pool, Tensor pages, int layer, int blocks, Tensor? block_pages, int block_layer, int step, Tensor q, "
+                          "Tensor(a!) out, Tensor? gate, Tensor? sinks, Tensor? mix, int dim, int vdim, float scale, int window, int block, "
+                          "int entry_begin, int entry_end, int max_tokens, int max_keys) -> bool",
     "shift_norm": "(int step, Tensor x_in, Tensor(a!) x_out, Tensor? y, Tensor? y_bias, Tensor? w_post, Tensor? add, Tensor w_next, "
                   "Tensor shift, Tensor state, Tensor(b!) state_out, Tensor(c!) h, float eps) -> ()",
     "embed_pairs": "(int step, Tensor(a!) x, Tensor embed, float scale, Tensor? pairs, Tensor(b!)? last_token, int mul_prev, int mul_cur, "
@@ -519,6 +522,21 @@ def _attn_pooled(pool, pages, layer, blocks, block_pages, block_layer, step, q, 
                                          _stream(q)), "pace_attn_pooled")
 
 
+def _attn_pooled_prompt(pool, pages, layer, blocks, block_pages, block_layer, step, q, out, gate, sinks, mix, dim, vdim, scale, window,
+                        block, entry_begin, entry_end, max_tokens, max_keys):
+    """False: the kernel does not take these shapes and nothing was launched."""
+    a = _pooled_args(q, out, gate, sinks, mix, dim, vdim, scale, window, block, max_keys)
+    a.entry_begin, a.entry_end, a.max_tokens = entry_begin, entry_end, max_tokens
+    with torch.cuda.device(q.device):
+        ws = _workspace(a, _C.lib.pace_attn_pooled_prompt_workspace_bytes(q.shape[0], q.shape[1], vdim), q.device)
+        rc = _C.lib.pace_attn_pooled_prompt(_pool(pool), layer, _pool(blocks) if block else None, block_layer, _step(step), C.byref(a),
+                                            _stream(q))
+        if rc != _C.PACE_ERR_UNSUPPORTED:
+            _C.check(rc, "pace_attn_pooled_prompt")
+        del ws
+    return rc == _C.PACE_OK
+
+
 def _shift_norm(step, x_in, x_out, y, y_bias, w_post, add, w_next, shift, state, state_out, h, eps):
     a = _C.ShiftNormArgs()
     a.x_in, a.x_out, a.w_next, a.shift, a.h = x_in.data_ptr(), x_out.data_ptr(), w_next.data_ptr(), shift.data_ptr(), h.data_ptr()
@@ -640,7 +658,7 @@ _IMPLS = {"kv_reserve": _kv_reserve, "kv_append": _kv_append, "kv_append_layers"
           "kv_append_conv": _kv_append_conv, "conv_store": _conv_store, "ssd_prefill": _ssd("pace_ssd_prefill"),
           "ssd_step": _ssd("pace_ssd_step"), "delta_prefill": _delta("pace_delta_prefill"), "delta_step": _delta("pace_delta_step"),
           "gla_prefill": _gla("pace_gla_prefill"), "gla_step": _gla("pace_gla_step"), "kv_append_rotate": _kv_append_rotate,
-          "attn_pooled": _attn_pooled, "shift_norm": _shift_norm, "embed_pairs": _embed_pairs, "state_commit": _state_commit,
+          "attn_pooled": _attn_pooled, "attn_pooled_prompt": _attn_pooled_prompt, "shift_norm": _shift_norm, "embed_pairs": _embed_pairs, "state_commit": _state_commit,
           "gate_per_head": _gate_per_head}
 for _n, _f in _IMPLS.items():
     _lib.impl(_n, _f, "CUDA")

@@ -1565,6 +1565,186 @@ def run_lesosun(args):
         print(json.dumps(line), flush=True)
 
 
+# ---------------------------------------------------------------------------------------------------
+# Kibotar: attention over a window and pooled blocks with mixed heads, gated linear attention, latent attention; beside the decoder
+# it resembles most, Garupel (attention and recurrences, dense relu^2 feed-forwards, norms on both sides)
+# ---------------------------------------------------------------------------------------------------
+KIBOTAR_SIZES = {
+    "w2048": dict(width=2048, ff=8192, heads=16, kv_heads=4, dim=128, window=1024, block=16, gla_heads=16, lat_heads=16, lat_dim=128,
+                  kv_rank=512),
+    "w4096": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, window=1024, block=16, gla_heads=32, lat_heads=32, lat_dim=128,
+                  kv_rank=512),
+}
+
+
+def kibotar_model(size: str, dev):
+    from pace_b200.llm.registry import build_model
+    z = KIBOTAR_SIZES[size]
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    att = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+        "mask": {"size": z["window"], "pool": z["block"]},
+        "rot": {"dims": z["dim"], "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    gla = {"type": "gla", "mlp": mlp, "mixer": {"heads": z["gla_heads"], "dim": z["dim"], "vdim": z["dim"], "tau": 16.0}}
+    lat = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": z["lat_heads"], "dim": z["lat_dim"], "vdim": z["lat_dim"], "kv_rank": z["kv_rank"], "scale": z["lat_dim"] ** -0.5}}
+    cfg = {"architecture": "Kibotar", "vocab": HYBRID_VOCAB, "width": z["width"], "norm": {"eps": 1e-5},
+           "embedding": {"scale": 8.0, "bigram": {"buckets": 20011, "mul_prev": 31, "mul_cur": 17}},
+           "layers": [gla, gla, lat, att] * (HYBRID_LAYERS // 4)}
+    return build_model(cfg, torch.bfloat16, dev).random_init_(5)
+
+
+@torch.inference_mode()
+def kibotar_kernels(size: str, dev):
+    """Each kernel of the Kibotar decoder alone, against its own roofline, and the like kernels of the other decoders ("like.*") on
+    operands of the same size; phases as in ``hybrid_kernels``."""
+    from pace_b200 import _C
+    from pace_b200.llm.hybrid_cache import BlockSpec, HybridCacheManager, JointSpec, KVSpec, LatentSpec, StateSpec
+    from pace_b200.ops import RotaryEmbedding, hybrid
+    z = KIBOTAR_SIZES[size]
+    W, H, G, D, FF, win, blk = z["width"], z["heads"], z["kv_heads"], z["dim"], z["ff"], z["window"], z["block"]
+    GH, LH, LD, R, ops = z["gla_heads"], z["lat_heads"], z["lat_dim"], z["kv_rank"], torch.ops.pace_b200
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(
+        os.path.join(ROOT, "MEASURED_PEAKS.json")) else {"hbm_gbs": FALLBACK_HBM_GBS, "bf16_tflops_sustained": 1400.0}
+    bw, fl = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops_sustained"] * 1e12
+    g = torch.Generator(device=dev).manual_seed(2)
+
+    def rnd(*shape, dtype=torch.bfloat16):
+        return torch.randn(*shape, device=dev, generator=g, dtype=torch.float32).to(dtype)
+
+    def seen(i):                               # tokens and blocks position i sees
+        return min(i + 1, win), max(0, i - win + 1) // blk
+
+    out = {}
+    tables = RotaryEmbedding({"rope_type": "precise"}, D, 8192, 500000.0).device_tables(dev)
+    turned = RotaryEmbedding({"rope_type": "precise"}, 64, 8192, 500000.0, is_neox_style=False).device_tables(dev)
+    for phase, E, n, past in (("prefill", 1, 4096, 0), ("prefill_batch", 8, 512, 0), ("decode", 32, 1, 512), ("decode_far", 8, 1, 4096)):
+        T, dec = E * n, n == 1
+        N = 8 if dec else 3                    # copies of every operand
+        nq, nk, nd = H * D, G * D, GH * D
+        specs = [JointSpec((KVSpec(G, D, D), BlockSpec(G, D, D, blk)))] * N + [StateSpec((("S", (GH, D, D)),))] * N + [LatentSpec(R, 0)] * N + \
+                [LatentSpec(R, 64)] * N + [StateSpec((("h", (N, W)), ("next", (N, W)))), StateSpec((("token", ()),), torch.int32)]
+        cache = HybridCacheManager(specs, E, E * (past + n + 64), past + n + 64, torch.bfloat16, dev)
+        for s_ in cache.states[:-1]:
+            for t in s_.arrays.values():
+                t.normal_(0.0, 0.1, generator=g)
+        if past:
+            cache.begin_step(cache.step([past] * E, torch.zeros(E * past, dtype=torch.long), 1))
+        step = cache.step([n] * E, torch.randint(0, HYBRID_VOCAB, (T,)), HYBRID_VOCAB)
+        cache.begin_step(step)
+        vec = lambda k: rnd(k, dtype=torch.float32)                          # noqa: E731
+        x, y = [rnd(T, W, dtype=torch.float32) for _ in range(N)], [rnd(T, W) for _ in range(N)]
+        spare = torch.empty(T, W, device=dev)
+        wp, wn, sh = vec(W), vec(W), vec(W)
+        qkvg = [rnd(T, 2 * nq + 2 * nk) for _ in range(N)]
+        qb = [torch.empty(T, H, D, dtype=torch.bfloat16, device=dev) for _ in range(N)]
+        rows = {}
+
+        def add(name, launches, nbytes, nflops=0.0):
+            us = graph_us(launches)
+            roof = max(nbytes / bw, nflops / fl) * 1e6
+            rows[name] = {"us": us, "roofline_us": roof, "frac": roof / us, "bound": "hbm" if nbytes / bw >= nflops / fl else "tensor"}
+
+        before = cache[4 * N]["h"]
+        after = before if dec else cache[4 * N]["next"]
+        add("shift_norm", [lambda i=i: hybrid.shift_norm(step, x[i], wn, sh, before[:, i], after[:, i], 1e-5, torch.bfloat16, y[i], None, wp, None, spare)
+                           for i in range(N)], T * W * (4 + 4 + 2 + 2) + E * W * 8)
+        add("like.residual_norm", [lambda i=i: hybrid.residual_norm(step, x[i], y[i], wp, w_next=wn, eps=1e-5) for i in range(N)],
+            T * W * (4 + 4 + 2 + 2))
+        table, pairs_t = rnd(HYBRID_VOCAB, W), rnd(20012, W)
+        add("embed_pairs", [lambda: hybrid.embed_pairs(step, table, 8.0, pairs_t, cache[4 * N + 1]["token"], 31, 17)] * N, T * W * 8)
+        add("like.embedding", [lambda i=i: hybrid.residual_norm(step, x[i], embed=table, w_next=wn, eps=1e-5, restart=True) for i in range(N)], T * W * 8)
+        if not dec:
+            add("state_commit", [lambda: hybrid.state_commit(step, cache[4 * N]["next"], before, cache[4 * N + 1]["token"])] * N, E * N * W * 8)
+        # attention: rows seen are read once, the blocks completed are made from cached rows
+        kv, bl = cache[0]
+        where = lambda i: (kv.pool.handle, kv.pool.pages, cache[i][0].layer, bl.pool.handle, bl.pool.pages, cache[i][1].layer, step.handle)   # noqa: E731
+        add("append_rotate", [lambda i=i: ops.kv_append_rotate(*where(i), qkvg[i], *tables, qb[i], D, D, True, blk, dec) for i in range(N)],
+            T * (nq + 2 * nk) * 4 + (0 if dec else T * 2 * nk * 2 * (1 + 1 / blk)))
+        add("like.append_heads", [lambda i=i: ops.kv_append_norm(kv.pool.handle, kv.pool.pages, i, step.handle, qkvg[i], None, None, qb[i], D, D,
+                                                                 1e-5, 1.0, 0.0, 1.0, True) for i in range(N)], T * (nq + 2 * nk) * 4)
+        mix, zero = torch.eye(H, device=dev) + rnd(H, H, dtype=torch.float32) * 0.1, torch.zeros(H, device=dev)
+        ao = torch.empty(T, nq, dtype=torch.bfloat16, device=dev)
+        keys = E * sum(seen(past + n - 1)) if dec else E * (n + n // blk)
+        pairs = E * sum(sum(seen(i)) for i in range(past, past + n))
+        near = E * sum(min(i + 1, win) for i in range(past, past + n))
+
+        def attention(i, mix, block):
+            rule = (qb[i], ao, qkvg[i][:, nq + 2 * nk:], zero, mix, D, D, D ** -0.5, win, block)
+            if dec:
+                ops.attn_pooled(*where(i), *rule, 0, T, past + n)
+            else:
+                assert ops.attn_pooled_prompt(*where(i), *rule, 0, E, n, past + n)
+        add("attention (pooled, mixed heads, gate)", [lambda i=i: attention(i, mix, blk) for i in range(N)], keys * nk * 4 + T * nq * 6,
+            pairs * (4.0 * nq + 2.0 * H * H))
+
+        def windowed(i):
+            rule = (None, zero, D, D, D ** -0.5, _C.SPAN_WINDOW, win, 0, E, n, past + n)
+            if dec:
+                ops.attn_span(kv.pool.handle, kv.pool.pages, i, step.handle, qb[i], ao.view(T, H, D), *rule)
+            else:
+                assert ops.attn_span_prefill(kv.pool.handle, kv.pool.pages, i, step.handle, qb[i], ao.view(T, H, D), *rule, None, None, None, None, None)
+        add("like.attention (window, sink)", [lambda i=i: windowed(i) for i in range(N)],
+            (E * min(past + n, win) if dec else T) * nk * 4 + T * nq * 4, near * 4.0 * nq)
+        gated = [rnd(step.staging_rows, H, D) for _ in range(N)]
+        add("like.gate_heads", [lambda i=i: hybrid.gate_heads(step, gated[i], qkvg[i][:, nq + 2 * nk:], D) for i in range(N)], T * nq * 6)
+        # gated linear attention: operands once, the state read and written; flops of the chunked form
+        gq, gz, zb, gw = [rnd(T, 4 * nd) for _ in range(N)], [rnd(T, nd) for _ in range(N)], vec(nd) + 2.0, vec(D)
+        rec = (lambda i: (gq[i], gz[i], zb, cache[N + i]["S"]))
+        go = [torch.empty(T, nd, dtype=torch.bfloat16, device=dev) for _ in range(N)]
+        gla_bytes, gla_flops = T * nd * 2 * 5 + E * GH * D * D * 8, 0.0 if dec else T * GH * (4.0 * D * D + 4 * D * 64.0)
+        if dec:
+            add("gla (with norm and gate)", [lambda i=i: hybrid.gla(step, *rec(i), gw, gq[i][:, 3 * nd:], 16.0, D ** -0.5, 1e-5) for i in range(N)],
+                gla_bytes + T * nd * 2)
+        else:
+            add("gla", [lambda i=i: ops.gla_prefill(step.handle, *rec(i), go[i], 1 / 16.0, D ** -0.5) for i in range(N)], gla_bytes, gla_flops)
+            add("norm + silu gate (heads)", [lambda i=i: hybrid.part_norm_gate(go[i], gw, gq[i][:, 3 * nd:], D, 1e-5, out=go[i], silu=True)
+                                             for i in range(N)], T * nd * 6)
+        decay = torch.linspace(0.9, 0.999, GH, device=dev)
+        add("like.lightning", [lambda i=i: hybrid.lightning(step, gq[i], decay, cache[N + i]["S"]) for i in range(N)],
+            T * nd * 2 * 4 + E * GH * D * D * 8, gla_flops)
+        add("like.norm_gate", [lambda i=i: hybrid.norm_gate(go[i], vec(nd), gq[i][:, 3 * nd:], 1e-5) for i in range(N)], T * nd * 6)
+        # latent attention without positions, and the one with a rotated part
+        q, down = [rnd(T, LH * LD) for _ in range(N)], [rnd(T, R + LH) for _ in range(N)]
+        qr, downr, kn, up = [rnd(T, LH * (LD + 64)) for _ in range(N)], [rnd(T, R + 64) for _ in range(N)], vec(R), rnd(2 * LH * LD, R) * 0.05
+        lp = E * sum(i + 1 for i in range(past, past + n))
+        lkeys = E * (past + n)
+        shape = lambda r: (lkeys * (R + r) * 2 + T * (R + r) * 2 + T * LH * (2 * LD + r) * 2 + up.numel() * 2,                      # noqa: E731
+                           2.0 * T * LH * 2 * LD * R + (lp * LH * 2.0 * (2 * R + r) if dec else lp * LH * 2.0 * (2 * LD + r)))
+        add("latent attention (no positions)", [lambda i=i: hybrid.latent_attention(step, cache[2 * N + i], down[i], None, kn, None, up, LH, LD, 0, LD,
+                                                                                    LD ** -0.5, 1e-5, None, q=q[i]) for i in range(N)], *shape(0))
+        add("like.latent attention (rotated part)", [lambda i=i: hybrid.latent_attention(
+            step, cache[3 * N + i], downr[i], None, kn, None, up, LH, LD, 64, LD, LD ** -0.5, 1e-5, turned, q=qr[i]) for i in range(N)], *shape(64))
+        add("gate_per_head", [lambda i=i: hybrid.gate_per_head_(q[i], down[i][:, R:], LH) for i in range(N)], T * LH * LD * 4)
+        hid = [rnd(T, FF) for _ in range(N)]
+        add("relu_squared", [lambda i=i: hybrid.relu_squared_(hid[i]) for i in range(N)], T * FF * 4)
+        cache.pool.check_status()
+        out[phase] = rows
+        del cache
+        torch.cuda.empty_cache()
+    return out
+
+
+def run_kibotar(args):
+    """Side measurement: prefill and decode throughput of the Kibotar decoder beside Garupel at equal width, heads, layer count and
+    feed-forward size (random weights), and every kernel of the first against its roofline.  Prints one JSON line per size."""
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    for size, z in KIBOTAR_SIZES.items():
+        sampler = ClockSampler(0)
+        sampler.start()
+        line = {"workload": "kibotar", "size": size, **z, "layers": HYBRID_LAYERS, "params": {}}
+        for name, make in (("kibotar", lambda: kibotar_model(size, dev)), ("garupel", lambda: hybrid_models(size, dev)[0])):
+            model = make()
+            line["params"][name] = sum(p.numel() for p in model.parameters())
+            line[name] = hybrid_throughput(model, dev)
+            del model
+            torch.cuda.empty_cache()
+        line["kernels"] = kibotar_kernels(size, dev)
+        line["clocks"] = sampler.stop()
+        print(json.dumps(line), flush=True)
+
+
 def main():
     # stdout carries the JSON line and nothing else: whatever native libraries print to file descriptor 1
     # (NCCL's version banner on some ranks) goes to stderr, Python's own prints keep the real stdout
@@ -1583,7 +1763,7 @@ def main():
     ap.add_argument("--layers", type=int, default=CFG["n_layers"],
                     help="profiling aid: fewer layers = less device memory; the bench line is only valid at 32")
     ap.add_argument("--workload", default="decode", choices=["decode", "verify", "prefill", "rope_append", "device_loop", "serving", "linear",
-                                                                 "hybrid", "gekupel", "lesosun"],
+                                                                 "hybrid", "gekupel", "lesosun", "kibotar"],
                     help="decode = the bench line; verify / prefill = side measurements of the multi-token kernels")
     ap.add_argument("--past", type=int, default=3584, help="prefill side measurement: tokens cached before the chunk")
     ap.add_argument("--head-dim", type=int, default=128, choices=[64, 128])
@@ -1598,10 +1778,11 @@ def main():
         return
     global RANK_CORES
     RANK_CORES = pin_rank_to_cores(local_rank, world)
-    if args.workload in ("rope_append", "device_loop", "serving", "linear", "hybrid", "gekupel", "lesosun"):
+    if args.workload in ("rope_append", "device_loop", "serving", "linear", "hybrid", "gekupel", "lesosun", "kibotar"):
         if rank == 0:
             {"rope_append": run_rope, "device_loop": run_device_loop, "serving": run_serving,
-             "linear": run_linear, "hybrid": run_hybrid, "gekupel": run_gekupel, "lesosun": run_lesosun}[args.workload](args)
+             "linear": run_linear, "hybrid": run_hybrid, "gekupel": run_gekupel, "lesosun": run_lesosun,
+             "kibotar": run_kibotar}[args.workload](args)
         return
     if args.workload != "decode":
         if rank == 0:
