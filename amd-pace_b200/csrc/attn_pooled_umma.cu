@@ -8,8 +8,8 @@
 // the other and adds up their shares of its outputs in fp32 (its own part of a workspace: nobody else touches it); the last one
 // multiplies by the gate and stores.
 //
-// Warps 0-3 softmax (one row per thread), 4 producer (queries, keys, values by TMA), 5 issues the products.  Chunks of 64 keys: pages of
-// pooled blocks first, then pages of tokens.  Tensor memory: two slots of 64 columns, scores and then, in their place, the weights in two
+// Warps 0-15 softmax (a row of a chunk is four threads' work, a warp per 16 columns of 32 rows), 16 producer (queries, keys, values by
+// TMA), 17 issues the products.  Chunks of 64 keys: pages of pooled blocks first, then pages of tokens.  Tensor memory: two slots of 64 columns, scores and then, in their place, the weights in two
 // bf16 terms; behind them O.
 #include <algorithm>
 
@@ -19,7 +19,8 @@
 namespace pace {
 namespace {
 
-constexpr int kChunk = 64, kBlockBytes = kChunk * 128, kThreads = 192, kMaxStages = 6;
+constexpr int kChunk = 64, kBlockBytes = kChunk * 128, kMaxStages = 6;
+constexpr int kGroups = 4, kCols = kChunk / kGroups, kSoftmax = 128 * kGroups, kThreads = kSoftmax + 64;   // softmax: warpgroups, their columns
 constexpr uint32_t kColO = 128, kColsO = 512 - kColO;
 constexpr float kLazy = 8.0f;  // log2 units a row's maximum may grow before O is rescaled
 
@@ -33,7 +34,7 @@ struct PooledParams {
   const float* mix;
   int64_t out_stride, gate_stride;
   int H, G, Gq, vdim, window, block;
-  int entry0, n_entries, n_tiles, tpw, nv, n_sub, n_stages;
+  int entry0, n_entries, n_tiles, tpw, nv, n_sub, n_stages, smem_bytes;
   float scale_log2;
 };
 
@@ -69,16 +70,38 @@ struct Bars {
   uint64_t full[kMaxStages], empty[kMaxStages], s_full[2], p_full[2], pv_done[2], q_full, q_empty, o_free, drain;
 };
 
+// behind the queries and the ring in shared memory (no static shared memory: the tiles then begin at a multiple of 1024 anyway)
+struct Small {
+  Bars b;
+  float part[kGroups][kUmmaRows];
+  uint32_t tmem_slot;
+  int abort_flag;
+};
+
+// true where any softmax thread says so; a barrier of all of them
+__device__ __forceinline__ bool softmax_any(bool v) {
+  uint32_t r;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t"
+      "setp.ne.u32 p, %1, 0;\n\t"
+      "barrier.cta.red.or.pred q, 1, %2, p;\n\t"
+      "selp.u32 %0, 1, 0, q;\n\t}"
+      : "=r"(r) : "r"((uint32_t)v), "n"(kSoftmax) : "memory");
+  return r != 0;
+}
+
 // VB: 64-column blocks of a value
 template <int VB>
-__device__ __forceinline__ void pooled_softmax(const PooledParams& p, Bars& b, uint32_t tmem, int n_units, volatile int* abort) {
-  const int row = threadIdx.x, lane = row & 31, warp = row >> 5;
+__device__ __forceinline__ void pooled_softmax(const PooledParams& p, Bars& b, uint32_t tmem, float (*part)[kUmmaRows], int n_units,
+                                               volatile int* abort) {
+  const int row = threadIdx.x & 127, lane = row & 31, warp = row >> 5, grp = threadIdx.x >> 7;
   const uint32_t t_lane = tmem + ((uint32_t)(row & ~31) << 16), tO = t_lane + kColO;
   const int hh = lane % p.Gq, base_lane = lane - hh;
   const bool in_tile = lane < p.tpw * p.Gq;
   const float scale = p.scale_log2;
   const uint64_t scale2 = pack64(__float_as_uint(scale), __float_as_uint(scale));
   int cnt = 0;  // chunks worked on
+  bool gave_up = false;   // (a wait that ran out cuts the waits behind it short; nobody leaves the common barriers)
   for (int u = blockIdx.x; u < n_units; u += gridDim.x) {
     Unit un;
     if (!get_unit(p, u, &un)) continue;
@@ -87,37 +110,44 @@ __device__ __forceinline__ void pooled_softmax(const PooledParams& p, Bars& b, u
     const int pos = un.start + (live ? tok : un.count - 1);
     const int nb = blocks_seen(pos, p.window, p.block), first = window_first(pos, p.window);
     for (int gk = un.g0; gk < un.g1; ++gk) {
-      float m = p.sinks ? p.sinks[gk * p.Gq + hh] * kLog2e : -INFINITY, l = p.sinks ? 1.f : 0.f;   // a sink: one more term of the sum
+      float m = p.sinks ? p.sinks[gk * p.Gq + hh] * kLog2e : -INFINITY, l = p.sinks && grp == 0 ? 1.f : 0.f;   // a sink: one more term of the sum
       for (int c = 0; c < un.n; ++c, ++cnt) {
         const uint32_t tS = t_lane + (cnt & 1) * kChunk;
-        if (!umma_wait(&b.s_full[cnt & 1], (cnt >> 1) & 1, abort)) return;
+        if (!gave_up) gave_up = !umma_wait(&b.s_full[cnt & 1], (cnt >> 1) & 1, abort);
         tc_fence_after();
-        uint32_t sr[2][32];
-        tmem_ld32(tS, sr[0]);
-        tmem_ld32(tS + 32, sr[1]);
+        uint32_t sr[kCols];
+        tmem_ld16(tS + grp * kCols, sr);
         tmem_wait_ld();
         const bool blk = c < un.nb_chunks;
-        const int p0 = blk ? c * kChunk : un.tbase + (c - un.nb_chunks) * kChunk;
-        const int lo = blk ? 0 : max(0, first - p0), hi = blk ? min(kChunk, nb - p0) : min(kChunk, pos + 1 - p0);   // seen keys: [lo, hi)
-        if (!__all_sync(0xffffffffu, !live || (lo <= 0 && hi >= kChunk))) {
+        const int p0 = (blk ? c * kChunk : un.tbase + (c - un.nb_chunks) * kChunk) + grp * kCols;
+        const int lo = blk ? 0 : max(0, first - p0), hi = blk ? min(kCols, nb - p0) : min(kCols, pos + 1 - p0);   // seen keys: [lo, hi)
+        if (!__all_sync(0xffffffffu, !live || (lo <= 0 && hi >= kCols))) {
           const unsigned seen = hi > lo ? (unsigned)(hi - lo) : 0u;
 #pragma unroll
-          for (int k = 0; k < 64; ++k)
-            if ((unsigned)(k - lo) >= seen) sr[k >> 5][k & 31] = 0xff800000u;  // -inf
+          for (int k = 0; k < kCols; ++k)
+            if ((unsigned)(k - lo) >= seen) sr[k] = 0xff800000u;  // -inf
         }
-        float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        float mx = max3(__uint_as_float(sr[0]), __uint_as_float(sr[1]), __uint_as_float(sr[2]));
+        float my = max3(__uint_as_float(sr[3]), __uint_as_float(sr[4]), __uint_as_float(sr[5]));
 #pragma unroll
-        for (int k = 0; k < 32; ++k)
-          mx4[k & 3] = max3(mx4[k & 3], __uint_as_float(sr[k >> 4][(2 * k) & 31]), __uint_as_float(sr[k >> 4][(2 * k + 1) & 31]));
-        const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale;  // scale > 0
-        const bool grow = mx > m + kLazy;
-        if (__any_sync(0xffffffffu, grow)) {
+        for (int k = 6; k < kCols - 2; k += 4) {
+          mx = max3(mx, __uint_as_float(sr[k]), __uint_as_float(sr[k + 1]));
+          my = max3(my, __uint_as_float(sr[k + 2]), __uint_as_float(sr[k + 3]));
+        }
+        mx = max3(fmaxf(mx, my), __uint_as_float(sr[kCols - 2]), __uint_as_float(sr[kCols - 1])) * scale;  // scale > 0
+        // behind this barrier all scores are in registers: weights may take their places
+        if (softmax_any(live && mx > m + kLazy)) {
+          part[grp][row] = mx;
+          asm volatile("bar.sync 1, %0;" ::"n"(kSoftmax) : "memory");
+#pragma unroll
+          for (int k = 0; k < kGroups; ++k) mx = fmaxf(mx, part[k][row]);
+          const bool grow = mx > m + kLazy;
           const float m_new = grow ? mx : m;
           const float alpha = grow ? ((m == -INFINITY) ? 0.f : fast_exp2(m - m_new)) : 1.f;
           if (c > 0) {  // O holds the sum of the earlier chunks
-            if (!umma_wait(&b.pv_done[(cnt - 1) & 1], ((cnt - 1) >> 1) & 1, abort)) return;
+            if (!gave_up) gave_up = !umma_wait(&b.pv_done[(cnt - 1) & 1], ((cnt - 1) >> 1) & 1, abort);
             tc_fence_after();
-            for (int d0 = 0; d0 < un.nv * VB * 64; d0 += 16) {
+            for (int d0 = grp * 16; d0 < un.nv * VB * 64; d0 += kGroups * 16) {
               uint32_t ov[16];
               tmem_ld16(tO + d0, ov);
               tmem_wait_ld();
@@ -129,30 +159,22 @@ __device__ __forceinline__ void pooled_softmax(const PooledParams& p, Bars& b, u
           }
           l *= alpha;
           m = m_new;
+          asm volatile("bar.sync 1, %0;" ::"n"(kSoftmax) : "memory");   // the maxima have been read
         }
         const float ne = (m == -INFINITY) ? 0.f : -m;
         const uint64_t ne2 = pack64(__float_as_uint(ne), __float_as_uint(ne));
         uint64_t l2[2] = {0ull, 0ull};
+        uint32_t ph[kCols / 2], pl[kCols / 2];
 #pragma unroll
-        for (int hf = 0; hf < 2; ++hf) {
-          uint32_t ph[16], pl[16];
-#pragma unroll
-          for (int k = 0; k < 16; ++k) {
-            uint32_t x0, x1;
-            unpack64(fma2(pack64(sr[hf][2 * k], sr[hf][2 * k + 1]), scale2, ne2), x0, x1);
-            float p0f, p1f;
-            if (k & 1) {
-              exp2_poly2_fine(__uint_as_float(x0), __uint_as_float(x1), p0f, p1f);   // half of them on the FMA pipe
-            } else {
-              p0f = fast_exp2(__uint_as_float(x0));
-              p1f = fast_exp2(__uint_as_float(x1));
-            }
-            l2[k & 1] = add2(l2[k & 1], pack64(__float_as_uint(p0f), __float_as_uint(p1f)));
-            split_bf2(p0f, p1f, ph[k], pl[k]);
-          }
-          tmem_st16(tS + hf * 16, ph);
-          tmem_st16(tS + 32 + hf * 16, pl);
+        for (int k = 0; k < kCols / 2; ++k) {
+          uint32_t x0, x1;
+          unpack64(fma2(pack64(sr[2 * k], sr[2 * k + 1]), scale2, ne2), x0, x1);
+          const float p0f = fast_exp2(__uint_as_float(x0)), p1f = fast_exp2(__uint_as_float(x1));
+          l2[k & 1] = add2(l2[k & 1], pack64(__float_as_uint(p0f), __float_as_uint(p1f)));
+          split_bf2(p0f, p1f, ph[k], pl[k]);
         }
+        tmem_st8(tS + grp * (kCols / 2), ph);
+        tmem_st8(tS + 32 + grp * (kCols / 2), pl);
         {
           uint32_t a0, a1, b0, b1;
           unpack64(l2[0], a0, a1);
@@ -165,70 +187,68 @@ __device__ __forceinline__ void pooled_softmax(const PooledParams& p, Bars& b, u
         if (lane == 0) mbar_arrive(&b.p_full[cnt & 1]);
       }
       // ---- this KV head's share of the unit's outputs ----
-      if (!umma_wait(&b.pv_done[(cnt - 1) & 1], ((cnt - 1) >> 1) & 1, abort)) return;
+      part[grp][row] = l;
+      asm volatile("bar.sync 1, %0;" ::"n"(kSoftmax) : "memory");
+      l = (part[0][row] + part[1][row]) + (part[2][row] + part[3][row]);
+      if (!gave_up) gave_up = !umma_wait(&b.pv_done[(cnt - 1) & 1], ((cnt - 1) >> 1) & 1, abort);
       tc_fence_after();
       const float inv = l > 0.f ? 1.0f / l : 0.f;
       const bool opens = gk == un.g0, closes = gk + 1 == un.g1;
-      for (int j = 0; j < un.nv; ++j) {
-        const int h = (un.c0 + j) * p.Gq + hh;
+      const size_t t = (size_t)(un.t0 + tok), row0 = (size_t)(un.t0 - p.st.cu[p.entry0] + tok) * p.H;
+      const int pieces = (p.vdim + 15) / 16;
+      for (int i = grp; i < un.nv * pieces; i += kGroups) {
+        const int j = i / pieces, d0 = (i - j * pieces) * 16, h = (un.c0 + j) * p.Gq + hh;
         const float* mix = p.mix ? p.mix + (size_t)h * p.H + gk * p.Gq : nullptr;
-        float* acc = p.acc + ((size_t)(un.t0 - p.st.cu[p.entry0] + tok) * p.H + h) * p.vdim;
-        const size_t t = (size_t)(un.t0 + tok);
-        for (int d0 = 0; d0 < p.vdim; d0 += 16) {
-          uint32_t raw[16];
-          tmem_ld16(tO + j * VB * 64 + d0, raw);
-          float before[16];
+        float* acc = p.acc + (row0 + h) * p.vdim;
+        uint32_t raw[16];
+        tmem_ld16(tO + j * VB * 64 + d0, raw);
+        float before[16];
 #pragma unroll
-          for (int k = 0; k < 16; k += 4) {
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (!opens && live && d0 + k < p.vdim) v = __ldcg(reinterpret_cast<const float4*>(acc + d0 + k));
-            before[k] = v.x, before[k + 1] = v.y, before[k + 2] = v.z, before[k + 3] = v.w;
+        for (int k = 0; k < 16; k += 4) {
+          float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (!opens && live && d0 + k < p.vdim) v = __ldcg(reinterpret_cast<const float4*>(acc + d0 + k));
+          before[k] = v.x, before[k + 1] = v.y, before[k + 2] = v.z, before[k + 3] = v.w;
+        }
+        __syncwarp();
+        tmem_wait_ld();
+        float o[16], y[16];
+#pragma unroll
+        for (int k = 0; k < 16; ++k) o[k] = __uint_as_float(raw[k]) * inv;
+        if (mix) {
+          const float f0 = mix[hh];
+#pragma unroll
+          for (int k = 0; k < 16; ++k) y[k] = fmaf(f0, o[k], before[k]);
+          for (int r = 1; r < p.Gq; ++r) {
+            const int g = hh + r < p.Gq ? hh + r : hh + r - p.Gq;
+            const float f = mix[g];
+            const int src = min(base_lane + g, 31);              // (lanes behind the tile's tokens: any lane)
+#pragma unroll
+            for (int k = 0; k < 16; ++k) y[k] = fmaf(f, __shfl_sync(0xffffffffu, o[k], src), y[k]);
           }
-          __syncwarp();
-          tmem_wait_ld();
-          float o[16], y[16];
+        } else {
 #pragma unroll
-          for (int k = 0; k < 16; ++k) o[k] = __uint_as_float(raw[k]) * inv;
-          if (mix) {
-            const float f0 = mix[hh];
+          for (int k = 0; k < 16; ++k) y[k] = o[k] + before[k];
+        }
+        if (live) {
 #pragma unroll
-            for (int k = 0; k < 16; ++k) y[k] = f0 * o[k];
-            for (int r = 1; r < p.Gq; ++r) {
-              const int g = hh + r < p.Gq ? hh + r : hh + r - p.Gq;
-              const float f = mix[g];
-              const int src = min(base_lane + g, 31);              // (lanes behind the tile's tokens: any lane)
+          for (int k = 0; k < 16; k += 8) {
+            if (d0 + k < p.vdim) {
+              if (!closes) {
+                __stcg(reinterpret_cast<float4*>(acc + d0 + k), make_float4(y[k], y[k + 1], y[k + 2], y[k + 3]));
+                __stcg(reinterpret_cast<float4*>(acc + d0 + k + 4), make_float4(y[k + 4], y[k + 5], y[k + 6], y[k + 7]));
+              } else {
+                if (p.gate) {
+                  float g[8];
+                  Vec<__nv_bfloat16, 8>::load(p.gate + t * p.gate_stride + (size_t)h * p.vdim + d0 + k, g);
 #pragma unroll
-              for (int k = 0; k < 16; ++k) y[k] = fmaf(f, __shfl_sync(0xffffffffu, o[k], src), y[k]);
-            }
-          } else {
-#pragma unroll
-            for (int k = 0; k < 16; ++k) y[k] = o[k];
-          }
-          if (live) {
-#pragma unroll
-            for (int k = 0; k < 16; k += 8) {
-              if (d0 + k < p.vdim) {
-                if (!opens) {
-#pragma unroll
-                  for (int x = 0; x < 8; ++x) y[k + x] += before[k + x];
+                  for (int x = 0; x < 8; ++x) y[k + x] *= sigmoid_t<__nv_bfloat16>(g[x]);
                 }
-                if (!closes) {
-                  __stcg(reinterpret_cast<float4*>(acc + d0 + k), make_float4(y[k], y[k + 1], y[k + 2], y[k + 3]));
-                  __stcg(reinterpret_cast<float4*>(acc + d0 + k + 4), make_float4(y[k + 4], y[k + 5], y[k + 6], y[k + 7]));
-                } else {
-                  if (p.gate) {
-                    float g[8];
-                    Vec<__nv_bfloat16, 8>::load(p.gate + t * p.gate_stride + (size_t)h * p.vdim + d0 + k, g);
-#pragma unroll
-                    for (int x = 0; x < 8; ++x) y[k + x] *= sigmoid_t<__nv_bfloat16>(g[x]);
-                  }
-                  Vec<__nv_bfloat16, 8>::store(p.out + t * p.out_stride + (size_t)h * p.vdim + d0 + k, y + k);
-                }
+                Vec<__nv_bfloat16, 8>::store(p.out + t * p.out_stride + (size_t)h * p.vdim + d0 + k, y + k);
               }
             }
           }
-          __syncwarp();
         }
+        __syncwarp();
       }
       tc_fence_before();
       __syncwarp();
@@ -306,33 +326,36 @@ __global__ void __launch_bounds__(kThreads, 1)
     attn_pooled_prompt_kernel(const PooledParams p, const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                               const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmBK,
                               const __grid_constant__ CUtensorMap tmBV) {
-  extern __shared__ unsigned char smem_raw[];
-  __shared__ Bars b;
-  __shared__ uint32_t tmem_slot;
-  __shared__ int abort_flag;
+  extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* qs = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   unsigned char* ring = qs + KB * kUmmaRows * 128;
-  volatile int* abort = &abort_flag;
+  Small* sm = reinterpret_cast<Small*>(ring + (size_t)p.n_stages * (KB + p.nv * VB) * kBlockBytes);
+  Bars& b = sm->b;
+  volatile int* abort = &sm->abort_flag;
+  if (reinterpret_cast<unsigned char*>(sm + 1) > smem_raw + p.smem_bytes) {     // (the tiles do not begin where they should)
+    if (threadIdx.x == 0) raise_status(p.kv.status, PACE_DEV_BAD_INDEX);
+    return;
+  }
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int n_units = p.n_entries * p.n_tiles * p.n_sub, stage_bytes = (KB + p.nv * VB) * kBlockBytes;
-  if (warp == 5) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(512) : "memory");
+  if (warp == kSoftmax / 32 + 1) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&sm->tmem_slot)), "r"(512) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
   if (tid == 0) {
-    abort_flag = 0;
+    sm->abort_flag = 0;
     for (int i = 0; i < p.n_stages; ++i) {
       mbar_init(&b.full[i], 1);
       mbar_init(&b.empty[i], 1);
     }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&b.s_full[i], 1);
-      mbar_init(&b.p_full[i], 4);
+      mbar_init(&b.p_full[i], kSoftmax / 32);
       mbar_init(&b.pv_done[i], 1);
     }
     mbar_init(&b.q_full, 1);
     mbar_init(&b.q_empty, 1);
-    mbar_init(&b.o_free, 4);
+    mbar_init(&b.o_free, kSoftmax / 32);
     mbar_init(&b.drain, 1);
     fence_mbar_init();
   }
@@ -342,11 +365,11 @@ __global__ void __launch_bounds__(kThreads, 1)
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(&tmem_slot);
+  const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(&sm->tmem_slot);
 
-  if (warp < 4) {
-    pooled_softmax<VB>(p, b, tmem, n_units, abort);
-  } else if (warp == 4) {
+  if (warp < kSoftmax / 32) {
+    pooled_softmax<VB>(p, b, tmem, sm->part, n_units, abort);
+  } else if (warp == kSoftmax / 32) {
     int s = 0, ph = 0, issued = 0, parts = 0;
     bool ok = true;
     for (int u = blockIdx.x; u < n_units && ok; u += gridDim.x) {
@@ -415,7 +438,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   if (lane == 0 && *abort) raise_status(p.kv.status, PACE_DEV_WAIT_TIMEOUT);
   tc_fence_before();
   __syncthreads();
-  if (warp == 5) {
+  if (warp == kSoftmax / 32 + 1) {
     tc_fence_after();
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512) : "memory");
   }
@@ -429,10 +452,11 @@ int sm_count() {
 
 template <int KB, int VB>
 int launch_prompt(PooledParams& p, const CUtensorMap* tm, cudaStream_t s) {
-  const int q_bytes = KB * kUmmaRows * 128, stage = (KB + p.nv * VB) * kBlockBytes, room = 226 * 1024 - 1024 - 512 - q_bytes;
+  const int q_bytes = KB * kUmmaRows * 128, stage = (KB + p.nv * VB) * kBlockBytes, most = 227 * 1024, room = most - (int)sizeof(Small) - q_bytes;
   p.n_stages = std::min(kMaxStages, room / stage);
   if (p.n_stages < 2) return PACE_ERR_UNSUPPORTED;
-  const int smem = q_bytes + p.n_stages * stage + 1024;
+  const int smem = std::min(most, q_bytes + p.n_stages * stage + (int)sizeof(Small) + 1024);
+  p.smem_bytes = smem;
   const int units = p.n_entries * p.n_tiles * p.n_sub, blocks = std::min(units, sm_count());
   PACE_CUDA_TRY(cudaFuncSetAttribute(attn_pooled_prompt_kernel<KB, VB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
   attn_pooled_prompt_kernel<KB, VB><<<blocks, kThreads, smem, s>>>(p, tm[0], tm[1], tm[2], tm[3], tm[4]);

@@ -1689,7 +1689,7 @@ def kibotar_kernels(size: str, dev):
         gated = [rnd(step.staging_rows, H, D) for _ in range(N)]
         add("like.gate_heads", [lambda i=i: hybrid.gate_heads(step, gated[i], qkvg[i][:, nq + 2 * nk:], D) for i in range(N)], T * nq * 6)
         # gated linear attention: operands once, the state read and written; flops of the chunked form
-        gq, gz, zb, gw = [rnd(T, 4 * nd) for _ in range(N)], [rnd(T, nd) for _ in range(N)], vec(nd) + 2.0, vec(D)
+        gq, gz, zb, gw, wide_w = [rnd(T, 4 * nd) for _ in range(N)], [rnd(T, nd) for _ in range(N)], vec(nd) + 2.0, vec(D), vec(nd)
         rec = (lambda i: (gq[i], gz[i], zb, cache[N + i]["S"]))
         go = [torch.empty(T, nd, dtype=torch.bfloat16, device=dev) for _ in range(N)]
         gla_bytes, gla_flops = T * nd * 2 * 5 + E * GH * D * D * 8, 0.0 if dec else T * GH * (4.0 * D * D + 4 * D * 64.0)
@@ -1703,7 +1703,7 @@ def kibotar_kernels(size: str, dev):
         decay = torch.linspace(0.9, 0.999, GH, device=dev)
         add("like.lightning", [lambda i=i: hybrid.lightning(step, gq[i], decay, cache[N + i]["S"]) for i in range(N)],
             T * nd * 2 * 4 + E * GH * D * D * 8, gla_flops)
-        add("like.norm_gate", [lambda i=i: hybrid.norm_gate(go[i], vec(nd), gq[i][:, 3 * nd:], 1e-5) for i in range(N)], T * nd * 6)
+        add("like.norm_gate", [lambda i=i: hybrid.norm_gate(go[i], wide_w, gq[i][:, 3 * nd:], 1e-5) for i in range(N)], T * nd * 6)
         # latent attention without positions, and the one with a rotated part
         q, down = [rnd(T, LH * LD) for _ in range(N)], [rnd(T, R + LH) for _ in range(N)]
         qr, downr, kn, up = [rnd(T, LH * (LD + 64)) for _ in range(N)], [rnd(T, R + 64) for _ in range(N)], vec(R), rnd(2 * LH * LD, R) * 0.05
