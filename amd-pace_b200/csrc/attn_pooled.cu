@@ -152,7 +152,7 @@ int launch_general(const KVView& kv, const KVView& bk, const pace_step_t& st, co
 // ---------------------------------------------------------------------------------------------------------------------
 // bf16 rows of 64 or 128
 // ---------------------------------------------------------------------------------------------------------------------
-constexpr int kWarps = 8, kThreads = 32 * kWarps, kMaxCluster = 8;
+constexpr int kWarps = 16, kThreads = 32 * kWarps, kMaxCluster = 8;
 
 __device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
   asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -164,8 +164,10 @@ __device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1
 // warps' outputs take the scores' place.
 struct StepSmem {
   int rows, scores, hi, lo, ml, mix, total;   // bytes
-  int pitch_s, pitch_w;                       // elements of a head's row
+  int pitch_s, pitch_w, pitch_m;              // elements of a head's row
 };
+// warps that share a task's keys, each with outputs of its own
+__host__ __device__ inline int step_sets(int tasks) { return kWarps / tasks > 1 ? kWarps / tasks : 1; }
 __host__ __device__ inline StepSmem step_smem(int H, int cap, int dp, int o_sets) {
   StepSmem m;
   int off = 0;
@@ -182,14 +184,15 @@ __host__ __device__ inline StepSmem step_smem(int H, int cap, int dp, int o_sets
   m.hi = take(H * m.pitch_w * 2);
   m.lo = take(H * m.pitch_w * 2);
   m.ml = take(H * 16);
-  m.mix = take(H * H * 4);
+  m.pitch_m = (H + 7) / 8 * 8;                // (what lies behind the last head is multiplied and not stored)
+  m.mix = take(H * m.pitch_m * 4);
   m.total = off;
   return m;
 }
 
 // DP: elements of a row; a token's keys are blocks [0, nb) in groups of 16, then tokens [first, pos] in groups of 16
 template <int DP>
-__global__ void __launch_bounds__(kThreads, 2) attn_pooled_step_kernel(KVView kv, KVView bk, pace_step_t st, pace_attn_pooled_args_t a, int cap, int o_sets) {
+__global__ void __launch_bounds__(kThreads, 1) attn_pooled_step_kernel(KVView kv, KVView bk, pace_step_t st, pace_attn_pooled_args_t a, int cap, int o_sets) {
   extern __shared__ __align__(16) unsigned char sm[];
   cg::cluster_group cl = cg::this_cluster();
   const int ns = gridDim.x, share = blockIdx.x, t = a.token_begin + blockIdx.y;
@@ -224,16 +227,23 @@ __global__ void __launch_bounds__(kThreads, 2) attn_pooled_step_kernel(KVView kv
     }
     rows[i] = pg * G * v.page_tokens + idx % v.page_tokens;
   }
-  if (a.mix)
-    for (int i = tid; i < H * H; i += kThreads) mixer[i] = a.mix[i];
+  if (a.mix)       // by key head, so that neighbouring heads lie side by side
+    for (int i = tid; i < H * H; i += kThreads) mixer[i % H * L.pitch_m + i / H] = a.mix[i];
   __syncthreads();
+  // the values are on their way to L2 while the keys are scored
+  for (int i = tid; i < n_keys * G * (DP / 64); i += kThreads) {
+    const int j = i / (G * (DP / 64)), r = i - j * (G * (DP / 64)), gi = ga + j / 16;
+    const bool blk = gi < b_groups;
+    const __nv_bfloat16* at = (blk ? bk.v : kv.v) + (size_t)(rows[j] + r / (DP / 64) * (blk ? bk.page_tokens : kv.page_tokens)) * DP + r % (DP / 64) * 64;
+    asm volatile("prefetch.global.L2 [%0];" ::"l"(at));
+  }
 
-  // warps of a KV head, the head this warp begins with
-  const int wpg = kWarps / G > 1 ? kWarps / G : 1, sub = warp % wpg, set = warp / wpg, n_sets = kWarps / wpg;
+  // a task is up to eight heads of a KV head; warps of a task, the task this warp begins with
+  const int tiles = (Gq + 7) / 8, tasks = G * tiles, wpg = step_sets(tasks), sub = warp % wpg, set = warp / wpg, n_sets = kWarps / wpg;
   const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q) + (size_t)t * H * DP;
   // ---- scores: 16 keys are the row operand, up to 8 heads the columns; lane's 8 neighbouring columns per slab of 32 ----
-  for (int gk = set; gk < G; gk += n_sets)
-    for (int h0 = 0; h0 < Gq; h0 += 8) {
+  for (int task = set; task < tasks; task += n_sets) {
+      const int gk = task / tiles, h0 = task % tiles * 8;
       uint4 qf[DP / 32];
 #pragma unroll
       for (int s = 0; s < DP / 32; ++s)
@@ -308,10 +318,17 @@ __global__ void __launch_bounds__(kThreads, 2) attn_pooled_step_kernel(KVView kv
 #pragma unroll
       for (int x = 0; x < 8; ++x) w[x] = 0.f;
       if (a.mix) {
+#pragma unroll 4
         for (int k = 0; k < H; ++k) {
           const float p = S[k * L.pitch_s + j];
 #pragma unroll
-          for (int x = 0; x < 8; ++x) w[x] = fmaf(mixer[min(h0 + x, H - 1) * H + k], p, w[x]);
+          for (int x = 0; x < 8; x += 4) {
+            const float4 f = *reinterpret_cast<const float4*>(mixer + k * L.pitch_m + h0 + x);
+            w[x] = fmaf(f.x, p, w[x]);
+            w[x + 1] = fmaf(f.y, p, w[x + 1]);
+            w[x + 2] = fmaf(f.z, p, w[x + 2]);
+            w[x + 3] = fmaf(f.w, p, w[x + 3]);
+          }
         }
       } else {
 #pragma unroll
@@ -330,8 +347,8 @@ __global__ void __launch_bounds__(kThreads, 2) attn_pooled_step_kernel(KVView kv
   // ---- values: columns of V are the row operand (two keys of a column in one register), heads the columns ----
   constexpr int NM = DP / 16, SLABS = DP / 64;                // (a row of 64: the second half of a tile is columns 4 further on)
   float* O = S;                                               // [sub][H][DP], the scores' place
-  for (int gv = set; gv < G; gv += n_sets)
-    for (int h0 = 0; h0 < Gq; h0 += 8) {
+  for (int task = set; task < tasks; task += n_sets) {
+      const int gv = task / tiles, h0 = task % tiles * 8;
       float acc[NM][4];
 #pragma unroll
       for (int m = 0; m < NM; ++m)
@@ -339,17 +356,26 @@ __global__ void __launch_bounds__(kThreads, 2) attn_pooled_step_kernel(KVView kv
         for (int x = 0; x < 4; ++x) acc[m][x] = 0.f;
       const int hr = gv * Gq + min(h0 + g, Gq - 1);           // (columns without a head are not stored)
       const __nv_bfloat16 *wh = w_hi + (size_t)hr * L.pitch_w, *wl = w_lo + (size_t)hr * L.pitch_w;
-      for (int gi = ga + sub; gi < gz; gi += wpg) {
+      uint4 next[4][SLABS];                                   // the next group's keys 2 tq, + 1, + 8, + 9
+      auto ask = [&](int gi) {
         const bool blk = gi < b_groups;
-        const __nv_bfloat16* base = blk ? bk.v : kv.v;
-        const int page_rows = blk ? bk.page_tokens : kv.page_tokens, i0 = (gi - ga) * 16;
-        uint4 v[4][SLABS];                                    // keys 2 tq, + 1, + 8, + 9
+        const __nv_bfloat16* base = (blk ? bk.v : kv.v) + (size_t)gv * (blk ? bk.page_tokens : kv.page_tokens) * DP + 8 * g;
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
-          const uint4* r = reinterpret_cast<const uint4*>(base + (size_t)(rows[i0 + 2 * tq + (x & 1) + (x >> 1) * 8] + gv * page_rows) * DP + 8 * g);
+          const uint4* r = reinterpret_cast<const uint4*>(base + (size_t)rows[(gi - ga) * 16 + 2 * tq + (x & 1) + (x >> 1) * 8] * DP);
 #pragma unroll
-          for (int s = 0; s < SLABS; ++s) v[x][s] = __ldg(r + 8 * s);
+          for (int s = 0; s < SLABS; ++s) next[x][s] = __ldg(r + 8 * s);
         }
+      };
+      if (ga + sub < gz) ask(ga + sub);
+      for (int gi = ga + sub; gi < gz; gi += wpg) {
+        const int i0 = (gi - ga) * 16;
+        uint4 v[4][SLABS];
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+#pragma unroll
+          for (int s = 0; s < SLABS; ++s) v[x][s] = next[x][s];
+        if (gi + wpg < gz) ask(gi + wpg);
         const uint32_t bh0 = *reinterpret_cast<const uint32_t*>(wh + i0 + 2 * tq), bh1 = *reinterpret_cast<const uint32_t*>(wh + i0 + 2 * tq + 8);
         const uint32_t bl0 = *reinterpret_cast<const uint32_t*>(wl + i0 + 2 * tq), bl1 = *reinterpret_cast<const uint32_t*>(wl + i0 + 2 * tq + 8);
         auto word = [](const uint4& u, int k) { return k == 0 ? u.x : k == 1 ? u.y : k == 2 ? u.z : u.w; };
@@ -379,15 +405,28 @@ __global__ void __launch_bounds__(kThreads, 2) attn_pooled_step_kernel(KVView kv
   else __syncthreads();
   // ---- the shares' outputs, every block a part of them ----
   const int vd = a.vdim, sets = wpg;
-  for (int i = share * kThreads + tid; i < H * vd; i += ns * kThreads) {
-    const int h = i / vd, c = i - h * vd;
-    float y = 0.f;
-    for (int k = 0; k < ns; ++k) {
-      const float* r = ns > 1 ? cl.map_shared_rank(O, k) : O;
-      for (int s = 0; s < sets; ++s) y += r[((size_t)s * H + h) * DP + c];
+  const int quads = (vd + 3) / 4;
+  for (int i = share * kThreads + tid; i < H * quads; i += ns * kThreads) {
+    const int h = i / quads, c = (i - h * quads) * 4;
+    float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < sets; ++s) {
+      float4 v[kMaxCluster];
+#pragma unroll
+      for (int k = 0; k < kMaxCluster; ++k) {
+        v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (k < ns) v[k] = *reinterpret_cast<const float4*>((ns > 1 ? cl.map_shared_rank(O, k) : O) + ((size_t)s * H + h) * DP + c);
+      }
+#pragma unroll
+      for (int k = 0; k < kMaxCluster; ++k) y.x += v[k].x, y.y += v[k].y, y.z += v[k].z, y.w += v[k].w;
     }
-    if (a.gate) y *= sigmoid_t<__nv_bfloat16>(__bfloat162float(static_cast<const __nv_bfloat16*>(a.gate)[(size_t)t * a.gate_stride + i]));
-    static_cast<__nv_bfloat16*>(a.out)[(size_t)t * a.out_stride + i] = __float2bfloat16_rn(y);
+    const float o[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      if (c + x >= vd) break;
+      float z = o[x];
+      if (a.gate) z *= sigmoid_t<__nv_bfloat16>(__bfloat162float(static_cast<const __nv_bfloat16*>(a.gate)[(size_t)t * a.gate_stride + h * vd + c + x]));
+      static_cast<__nv_bfloat16*>(a.out)[(size_t)t * a.out_stride + h * vd + c + x] = __float2bfloat16_rn(z);
+    }
   }
   if (ns > 1) cl.sync();                                      // nobody leaves while its shared memory is read
 }
@@ -404,10 +443,10 @@ int launch_step(const KVView& kv, const KVView& bk, const pace_step_t& st, const
   if (T > 65535) return PACE_ERR_UNSUPPORTED;
   const int64_t window = a.window < a.max_keys ? a.window : a.max_keys;
   const int64_t groups = (window + 15) / 16 + 1 + (a.block > 0 && a.max_keys > a.window ? ((a.max_keys - a.window) / a.block + 15) / 16 + 1 : 0);
-  const int o_sets = kWarps / G > 1 ? kWarps / G : 1;
+  const int o_sets = step_sets(G * ((H / G + 7) / 8));
   // the most blocks per token that are all resident at once and have two groups of keys each; more if a share has no room
   int ns = 1;
-  while (ns < kMaxCluster && (int64_t)T * ns * 2 <= 2 * sm_count() && groups >= 4 * ns) ns *= 2;
+  while (ns < kMaxCluster && (int64_t)T * ns * 2 <= sm_count() && groups >= 4 * ns) ns *= 2;
   int smem = 0, cap = 0;
   for (;; ns *= 2) {
     if (ns > kMaxCluster) return PACE_ERR_UNSUPPORTED;

@@ -896,7 +896,8 @@ typedef struct {
 } pace_attn_pooled_args_t;
 int pace_attn_pooled(const pace_kv_pool_t* pool, int32_t layer, const pace_kv_pool_t* blocks, int32_t block_layer,
                      const pace_step_t* step, const pace_attn_pooled_args_t* a, void* stream);
-uint64_t pace_attn_pooled_prompt_workspace_bytes(int32_t n_tokens, int32_t n_q_heads, int32_t vdim);
+uint64_t pace_attn_pooled_prompt_workspace_bytes(int32_t n_entries, int32_t max_tokens, int32_t n_q_heads, int32_t n_kv_heads,
+                                                 int32_t vdim, int32_t mixed);
 int pace_attn_pooled_prompt(const pace_kv_pool_t* pool, int32_t layer, const pace_kv_pool_t* blocks, int32_t block_layer,
                             const pace_step_t* step, const pace_attn_pooled_args_t* a, void* stream);
 
