@@ -69,10 +69,11 @@ __device__ __forceinline__ bool get_unit(const PooledParams& p, int u, Unit* w) 
 }
 
 struct Bars {
-  uint64_t k_full[kKeyStages], k_empty[kKeyStages], v_full[kMaxStages], v_empty[kMaxStages], s_full[kSlots], p_full[kSlots], pv_done[kSlots], q_full, q_empty, o_free, drain[2];
+  uint64_t k_full[kKeyStages], k_empty[kKeyStages], v_full[kMaxStages], v_empty[kMaxStages];
+  uint64_t s_full[kSlots], p_full[kSlots], pv_done[kSlots], q_full, q_empty, o_free, drain[2];
 };
 
-// behind the queries and the ring in shared memory (no static shared memory: the tiles then begin at a multiple of 1024 anyway)
+// behind the queries and the rings in shared memory (no static shared memory: the tiles then begin at a multiple of 1024 anyway)
 constexpr int kMixPitch = 20;     // floats of a row's 16 columns: neighbouring rows in different banks
 struct Small {
   Bars b;

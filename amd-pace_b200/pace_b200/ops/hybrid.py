@@ -106,7 +106,7 @@ def _span(window: Optional[int], chunk: Optional[int]):
 
 
 MOE_WIDE = 32           # tokens per expert from which wide token tiles are worth the copy
-PROMPT_TOKENS = 16      # tokens of an entry from which pooled attention over tiles of tokens is worth a launch
+PROMPT_TOKENS = (256, 16)    # tokens of all prompt portions, and of the longest, from which pooled attention over tiles is faster
 PROMPT_ROWS = 64        # query rows of an entry from which the tcgen05 prompt kernel is worth a launch
 
 
@@ -232,7 +232,7 @@ def pooled_attention(step: Step, cache, blocks, qkv: torch.Tensor, tables, heads
     _OPS.kv_append_rotate(*where, qkv, *(tables or (None, None)), q, dim, vdim, halves, block, step.decode_only)
     rule = (q, out, gate, sinks, mix, dim, vdim, scale, window, block)
     Ed, E = step.n_decode, step.n_entries
-    if (E > Ed and q.dtype == torch.bfloat16 and step.max_count >= PROMPT_TOKENS
+    if (E > Ed and q.dtype == torch.bfloat16 and T - Ed >= PROMPT_TOKENS[0] and step.max_count >= PROMPT_TOKENS[1]
             and _OPS.attn_pooled_prompt(*where, *rule, Ed, E, step.max_count, step.max_keys)):
         T = Ed
     if T:

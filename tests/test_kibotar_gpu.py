@@ -18,6 +18,13 @@ TOL = {BF16: 0.06, FP32: 1e-4}
 ROOT = os.path.abspath(os.path.join(os.path.dirname(__file__), ".."))
 
 
+@pytest.fixture(params=[(1, 2), None], ids=["tiles", "tokens"])
+def form(request, monkeypatch):
+    """Prompt portions take the tile form of pooled attention whatever their size, or token by token."""
+    from pace_b200.ops import hybrid
+    monkeypatch.setattr(hybrid, "PROMPT_TOKENS", request.param or (1 << 30, 2))
+
+
 def build(cfg, dtype, seed=0):
     from pace_b200.llm.registry import build_model
     w = km.weights(cfg, seed)
@@ -126,7 +133,7 @@ SHAPES = [(BF16, 6, 2, 40, 24, 37, 5, 24), (BF16, 10, 5, 64, 120, 100, 16, 32), 
 
 
 @pytest.mark.parametrize("dtype,H,G,d,vd,window,block,rot", SHAPES)
-def test_pooled_attention_at_every_position(dtype, H, G, d, vd, window, block, rot):
+def test_pooled_attention_at_every_position(dtype, H, G, d, vd, window, block, rot, form):
     """Prompts, portions and decoding against the plain form; blocks are completed inside portions, across them and by
     decoded tokens."""
     n = 330
@@ -142,7 +149,7 @@ def test_pooled_attention_at_every_position(dtype, H, G, d, vd, window, block, r
 
 @pytest.mark.parametrize("dtype", [BF16, FP32])
 @pytest.mark.parametrize("with_mix,with_gate,sinks", [(False, False, False), (True, False, True), (False, True, True)])
-def test_pooled_attention_without_its_parts(dtype, with_mix, with_gate, sinks):
+def test_pooled_attention_without_its_parts(dtype, with_mix, with_gate, sinks, form):
     m = km.att(8, 4, 32, 40, 45, 6, 16)
     qkv, gate, mix = operands(m, 200, dtype, 1)
     gate, mix = gate if with_gate else None, mix if with_mix else None
@@ -155,7 +162,7 @@ def test_pooled_attention_without_its_parts(dtype, with_mix, with_gate, sinks):
 @pytest.mark.parametrize("dtype", [BF16, FP32])
 @pytest.mark.parametrize("window,block", [(72, 16), (64, 64), (65, 5), (33, 24), (1, 8), (130, 1)])
 @pytest.mark.parametrize("tail", [[200], [1] * 200, [7, 1, 50, 2, 140]])
-def test_a_key_that_stands_out(dtype, window, block, tail):
+def test_a_key_that_stands_out(dtype, window, block, tail, form):
     """One key has nearly all the weight where it is seen: just inside and just outside the window, between window and block, and
     in the mean of its block from the first position that sees it.  Its value is recognised in every output."""
     H, G, d = 4, 2, 64
@@ -178,7 +185,7 @@ def test_a_key_that_stands_out(dtype, window, block, tail):
 
 
 @pytest.mark.parametrize("dtype", [BF16, FP32])
-def test_one_in_the_denominator(dtype):
+def test_one_in_the_denominator(dtype, form):
     """With scores far below 0 hardly any weight is left; with scores far above 0 the one does not matter."""
     for level in (-6.0, 0.0, 30.0):
         m = km.att(4, 2, 64, 64, 20, 4, 2, scale=1.0)
@@ -193,7 +200,7 @@ def test_one_in_the_denominator(dtype):
 
 
 @pytest.mark.parametrize("dtype", [BF16, FP32])
-def test_mixing_crosses_kv_heads(dtype):
+def test_mixing_crosses_kv_heads(dtype, form):
     """A permutation of the heads: head h takes another head's weights to its own values."""
     m = km.att(6, 3, 32, 16, 30, 4, 8)
     qkv, gate, _ = operands(m, 150, dtype, 6)
@@ -203,7 +210,7 @@ def test_mixing_crosses_kv_heads(dtype):
         assert row_error(attend(m, qkv, gate, mix, pooled_cache(m, dtype), 0, counts), want) < (0.03 if dtype == BF16 else 1e-5)
 
 
-def test_weights_keep_more_than_bf16():
+def test_weights_keep_more_than_bf16(form):
     """Two keys with nearly the same weight whose values nearly cancel: what is left shows the weights' rounding."""
     m = km.att(2, 1, 64, 64, 64, 64, 2, scale=1.0)
     n = 33
@@ -220,7 +227,7 @@ def test_weights_keep_more_than_bf16():
 
 
 @pytest.mark.parametrize("dtype", [BF16, FP32])
-def test_thousands_of_keys(dtype):
+def test_thousands_of_keys(dtype, form):
     """Far blocks stand out among a thousand; decoding shares a token's keys over a cluster."""
     m = km.att(4, 2, 64, 64, 90, 3, 64)
     n = 3300
@@ -439,7 +446,7 @@ def test_one_layer_models(kind, mixer, ff, dtype):
 
 @pytest.mark.parametrize("dtype", [BF16, FP32])
 @pytest.mark.parametrize("name", list(km.CONFIGS))
-def test_prompts_portions_and_decoding(name, dtype):
+def test_prompts_portions_and_decoding(name, dtype, form):
     cfg = km.CONFIGS[name]
     model, w = build(cfg, dtype)
     toks = prompt(cfg, 220, 2)
@@ -467,7 +474,7 @@ def test_loops_and_tables_of_pairs(loop, bigram):
 
 
 @pytest.mark.parametrize("dtype", [BF16, FP32])
-def test_unequal_requests_in_one_batch(dtype):
+def test_unequal_requests_in_one_batch(dtype, form):
     """Prompts, portions and decoded tokens of several requests share steps; slots and pages go round: the pool holds
     fewer tokens than all requests together, rows are freed and taken in another order."""
     cfg = km.CONFIGS["mixed"]
