@@ -20,11 +20,13 @@ __global__ void __launch_bounds__(512) shift_norm_kernel(pace_step_t st, pace_sh
     for (int j = 0; j < V; ++j) mix[i][j] = prev[i][j] = 0.f;
     if (c < W) Vec<float, V>::load(a.shift + c, mix[i]);
   }
-  // the token in front of the block's first one is made once more if it belongs to the same sequence
-  const int e0 = st.tok_entry[t0];
-  for (int t = t0 > st.cu[e0] ? t0 - 1 : t0; t < t1; ++t) {
+  // the token in front of the block's first one is made once more if it belongs to the same sequence; in a step of one token per
+  // entry nothing has to be looked up
+  const bool single = st.n_tokens == st.n_entries;
+  for (int t = !single && t0 > st.cu[st.tok_entry[t0]] ? t0 - 1 : t0; t < t1; ++t) {
     const bool own = t >= t0;
-    const int e = st.tok_entry[t];
+    const int e = single ? t : st.tok_entry[t], start = st.start[e];
+    slot = st.slot[e];
     float x[ITEMS][V], y[ITEMS][V];
     float ss = 0.f;
 #pragma unroll
@@ -45,9 +47,8 @@ __global__ void __launch_bounds__(512) shift_norm_kernel(pace_step_t st, pace_sh
         }
       }
     }
-    slot = st.slot[e];
-    if (t == st.cu[e]) {                       // the previous token is the state's, or there is none
-      const bool fresh = st.start[e] == 0;
+    if (single || t == st.cu[e]) {             // the previous token is the state's, or there is none
+      const bool fresh = start == 0;
 #pragma unroll
       for (int i = 0; i < ITEMS; ++i) {
         const int c = (i * blockDim.x + threadIdx.x) * V;
@@ -86,7 +87,7 @@ __global__ void __launch_bounds__(512) shift_norm_kernel(pace_step_t st, pace_sh
       }
     }
     const float r = 1.0f / sqrtf(block_sum(ss, red[1]) / (float)W + a.eps);
-    const bool last = t + 1 == st.cu[e + 1];
+    const bool last = single || t + 1 == st.cu[e + 1];
 #pragma unroll
     for (int i = 0; i < ITEMS; ++i) {
       const int c = (i * blockDim.x + threadIdx.x) * V;
